@@ -12,12 +12,14 @@ spec into the architecture description and the derived KV geometry.
 
 from __future__ import annotations
 
+import json
 import os
 from dataclasses import dataclass, field, fields, replace
 from math import isfinite
 from typing import Any, Mapping
 
-from .models.architecture import Qwen3VLArch, validate_tensor_parallel
+from .models.architecture import validate_tensor_parallel
+from .models.model_registry import ModelFamily, family_of_config, random_architecture, resolve_model_family
 
 COMPRESSION_MODES = (
     "off", "visual_prune", "visual_compact", "fp8_kv", "visual_compact_fp8", "scaled_fp8_kv",
@@ -25,6 +27,7 @@ COMPRESSION_MODES = (
 )
 PAGE_SIZES = (16, 32, 64, 128, 256)
 BACKENDS = ("eager", "compile", "cuda_graph", "compile_graph")
+DTYPES = ("auto", "bfloat16", "float32")
 POLICIES = ("fcfs", "vision_aware", "slo_aware")
 DEFAULT_TP_TIMEOUT = 120
 
@@ -58,6 +61,7 @@ class ModelConfig:
     logits_precision: str = "model"
     mlp_projection_mode: str = "packed"
     seed: int = 0
+    dtype: str = "auto"  # auto: bfloat16 on CUDA, float32 on the CPU; float32 on CUDA needs a family with 32-bit kernels
 
     def __post_init__(self) -> None:
         if not isinstance(self.model, str) or not self.model:
@@ -71,6 +75,8 @@ class ModelConfig:
             raise ValueError(f"unsupported logits_precision {self.logits_precision!r}")
         if self.mlp_projection_mode not in ("legacy", "packed"):
             raise ValueError(f"unsupported mlp_projection_mode {self.mlp_projection_mode!r}")
+        if self.dtype not in DTYPES:
+            raise ValueError(f"dtype must be one of {DTYPES}, got {self.dtype!r}")
 
 
 @dataclass(frozen=True)
@@ -203,6 +209,7 @@ class ExecutionConfig:
     cooperative_prefill_coalesce_min_seqs: int = 3
     programmatic_dependent_launch: bool = True
     decode_run_ahead: bool = True             # launch the next greedy decode graph before the host has read this one's tokens
+    step_logits: bool = False                 # decode graphs keep their logits for ``ModelRunner.step_logits`` (trace replay)
     device_status_check_interval: int = 256   # engine steps between reads of the kernels' status words (0 = never)
 
     def __post_init__(self) -> None:
@@ -213,7 +220,7 @@ class ExecutionConfig:
         if self.paged_decode_block_n not in (16, 32, 64, 128, 256):
             raise ValueError("paged_decode_block_n must be a power of two in [16, 256]")
         for n in ("fused_qk_rmsnorm", "fused_qk_mrope", "fused_add_rmsnorm", "packed_kv_projection",
-                  "cooperative_prefill", "programmatic_dependent_launch", "decode_run_ahead"):
+                  "cooperative_prefill", "programmatic_dependent_launch", "decode_run_ahead", "step_logits"):
             _bool(getattr(self, n), n)
         _int(self.cooperative_prefill_layer_quantum, "cooperative_prefill_layer_quantum", 1)
         _int(self.cooperative_prefill_vision_block_quantum, "cooperative_prefill_vision_block_quantum", 1)
@@ -259,7 +266,7 @@ _FLAT = {
     "model": {
         "max_model_len": "max_model_len", "tensor_parallel_size": "tensor_parallel_size",
         "tensor_parallel_timeout_seconds": "tensor_parallel_timeout_seconds",
-        "logits_precision": "logits_precision", "mlp_projection_mode": "mlp_projection_mode", "seed": "seed",
+        "logits_precision": "logits_precision", "mlp_projection_mode": "mlp_projection_mode", "seed": "seed", "dtype": "dtype",
     },
     "multimodal": {
         "image_min_pixels": "image_min_pixels", "image_max_pixels": "image_max_pixels",
@@ -306,7 +313,7 @@ _FLAT = {
         "cooperative_prefill_coalesce_ms": "cooperative_prefill_coalesce_ms",
         "cooperative_prefill_coalesce_min_seqs": "cooperative_prefill_coalesce_min_seqs",
         "enable_programmatic_dependent_launch": "programmatic_dependent_launch",
-        "enable_decode_run_ahead": "decode_run_ahead",
+        "enable_decode_run_ahead": "decode_run_ahead", "enable_step_logits": "step_logits",
         "device_status_check_interval": "device_status_check_interval",
     },
 }
@@ -376,32 +383,19 @@ class PrismConfig:
         )
 
 
-_RANDOM_ARCHS = {
-    "tiny": Qwen3VLArch.tiny,
-    "qwen3-vl-8b": Qwen3VLArch.qwen3_vl_8b,
-    "qwen3_vl_8b": Qwen3VLArch.qwen3_vl_8b,
-    "qwen3-vl-8b-2layer": Qwen3VLArch.qwen3_vl_8b_2layer,
-    # profiling aids: the language-model compute of ONE rank of an n-way tensor-parallel group
-    # (heads, KV heads, MLP width and vocabulary divided by n), run without any exchange
-    "qwen3-vl-8b-tp2-shard": lambda: Qwen3VLArch.qwen3_vl_8b().rank_shard(2),
-    "qwen3-vl-8b-tp4-shard": lambda: Qwen3VLArch.qwen3_vl_8b().rank_shard(4),
-    "qwen3-vl-8b-tp8-shard": lambda: Qwen3VLArch.qwen3_vl_8b().rank_shard(8),
-}
-
-
-def resolve_arch(model: str) -> Qwen3VLArch:
+def resolve_arch(model: str):
+    """Architecture of a checkpoint directory (by its ``config.json``) or of a ``random:<name>`` model."""
     if model.startswith("random:"):
-        name = model.split(":", 1)[1]
-        if name not in _RANDOM_ARCHS:
-            raise ValueError(f"unknown random architecture {name!r}; known: {sorted(_RANDOM_ARCHS)}")
-        return _RANDOM_ARCHS[name]()
-    return Qwen3VLArch.from_pretrained(model)
+        return random_architecture(model.split(":", 1)[1])
+    with open(os.path.join(model, "config.json"), "r", encoding="utf-8") as fh:
+        cfg = json.load(fh)
+    return family_of_config(cfg).architecture_from_config(cfg)
 
 
 class Config:
     """Resolved runtime configuration: domains + architecture + derived capacities."""
 
-    def __init__(self, model: "str | PrismConfig", arch: Qwen3VLArch | None = None, **flat_options: object) -> None:
+    def __init__(self, model: "str | PrismConfig", arch: Any | None = None, **flat_options: object) -> None:
         if isinstance(model, PrismConfig):
             if flat_options:
                 raise TypeError("flat options cannot be combined with a PrismConfig")
@@ -412,7 +406,13 @@ class Config:
             self._flat_options = dict(flat_options)  # replayed verbatim by spawned worker ranks
         self.arch = arch if arch is not None else resolve_arch(self.prism.model.model)
         validate_tensor_parallel(self.arch, self.prism.model.tensor_parallel_size)
-        self.max_model_len = min(self.prism.model.max_model_len, self.arch.text.max_position_embeddings)
+        self.family: ModelFamily = resolve_model_family(self.arch.model_type)
+        if self.kv_mode not in self.family.kv_modes:
+            raise ValueError(f"compression_mode {self.prism.cache.compression_mode!r} is not available for the {self.family.name} family")
+        if not self.family.multimodal and self.prism.cache.compression_mode != "off":
+            raise ValueError(f"compression_mode {self.prism.cache.compression_mode!r} needs visual tokens")
+        limit = self.arch.max_positions
+        self.max_model_len = self.prism.model.max_model_len if limit is None else min(self.prism.model.max_model_len, limit)
         if self.prism.scheduler.max_num_batched_tokens < self.max_model_len and not self.prism.scheduler.enable_chunked_prefill:
             raise ValueError("max_num_batched_tokens must be >= max_model_len when chunked prefill is off")
         self.eos = self.arch.eos_token_id
@@ -453,11 +453,9 @@ class Config:
         return self.prism.cache.compression_mode in ("visual_compact", "visual_compact_fp8", "visual_compact_scaled_fp8")
 
     def kv_bytes_per_page(self) -> int:
-        """Bytes of one page across all layers, K and V, on one rank (payload + scales)."""
-        t = self.arch.text
-        rows = 2 * t.num_layers * (t.num_kv_heads // self.tp) * self.kvcache_block_size
-        elem = 2 if self.kv_mode == 0 else 1
-        return rows * t.head_dim * elem + (rows * 4 if self.kv_mode == 2 else 0)
+        """Bytes of one page across all layers and planes (K and V, or the shared latent) on one rank (payload + scales)."""
+        elem = (4 if self.prism.model.dtype == "float32" else 2) if self.kv_mode == 0 else 1
+        return self.arch.kv_geometry(self.tp).bytes_per_page(self.kvcache_block_size, elem, scaled=self.kv_mode == 2)
 
     def with_cache_capacity(self, gpu_blocks: int, cpu_blocks: int) -> "Config":
         self.num_kvcache_blocks = int(gpu_blocks)

@@ -333,6 +333,17 @@ class BlockManager:
                     cow.append(pair)
         return tuple(cow)
 
+    def grow(self, seq: Sequence) -> None:
+        """Pages for tokens that arrived after admission (a prompt delivered in portions): as many as the
+        sequence's current length needs."""
+        need = seq.blocks_needed() - len(seq.block_table)
+        if need <= 0:
+            return
+        if not self._ensure_free(need):
+            raise OutOfBlocks(f"no {need} free GPU page(s) for sequence {seq.seq_id}")
+        seq.block_table.extend(self.gpu.allocate_many(need))
+        seq.block_table_version += 1
+
     def copy_on_write(self, seq: Sequence, index: int) -> tuple[int, int] | None:
         old = seq.block_table[index]
         if self.gpu.blocks[old].ref_count <= 1:

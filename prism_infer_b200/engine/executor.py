@@ -47,7 +47,7 @@ class ModelExecutor:
         # over their visual tokens (last N decoder layers) and compacted by those scores; prompts
         # that need several chunks fall back to the uniform selection at the prefix boundary
         self.attention_strategy = bool(self.compact and config.visual_pruning_strategy == "attention")
-        n_layers = config.arch.text.num_layers
+        n_layers = config.arch.num_layer_runs
         last_n = max(1, min(n_layers, int(config.visual_pruning_attention_last_n_layers)))
         self.score_layers = list(range(n_layers - last_n, n_layers))
         self.pruning_scored = PruningConfig(config.visual_pruning_keep_ratio, config.visual_pruning_min_keep_tokens,
@@ -182,6 +182,14 @@ class ModelExecutor:
             tokens = [int(t) for t in sampled]
         compactions = self._after_prefill(plan) if plan.phase is Phase.PREFILL else 0
         return ExecutionResult(tuple(tokens), (time.perf_counter() - t0) * 1e3, compactions)
+
+    def step_logits(self, plan: BatchPlan, rows):
+        """One text plan through the same preparation and model step as ``execute``; fp32 logits of the given
+        flattened token rows instead of sampled tokens (trace replay)."""
+        if not plan.kv_transfers.empty:
+            self.runners.call("apply_kv_transfers", plan.kv_transfers)
+        with profile_region("engine.model_runner", metadata={"phase": plan.phase.value, "batch": plan.batch_size}):
+            return self.runners.call("step_logits", self.preparer.prepare(plan, self._have_visual), list(rows))
 
     # ------------------------------------------------------------------------------
     def _whole_prompt(self, seq, sl) -> bool:

@@ -86,22 +86,9 @@ class LLMEngine:
         if runner_group is None:
             self._validate_environment(device)
         self.tokenizer = load_tokenizer(cfg.model, self.arch)
-        # options given by the caller win; otherwise the budgets the checkpoint's own processor files record
-        recorded = checkpoint_pixel_budgets(cfg.model) if os.path.isdir(str(cfg.model)) else {}
-        self.processor = PatchProcessor(self.arch, min_pixels=cfg.image_min_pixels or recorded.get("min_pixels"),
-                                        max_pixels=cfg.image_max_pixels or recorded.get("max_pixels"),
-                                        video_max_pixels=cfg.video_max_pixels or recorded.get("video_max_pixels"),
-                                        video_min_pixels=recorded.get("video_min_pixels"), video_fps=recorded.get("video_fps"),
-                                        video_min_frames=recorded.get("video_min_frames"), video_max_frames=recorded.get("video_max_frames"))
-        from .chat_prompt import ChatPrompt, HFProcessorAdapter
-
-        mode = cfg.chat_template
-        chat = ChatPrompt(self.tokenizer)
-        self.chat = chat if (mode == "always" or (mode == "auto" and chat.has_template)) else None
-        self.hf_processor = None
-        if cfg.hf_processor == "always":
-            self.hf_processor = HFProcessorAdapter(cfg.model, image_max_pixels=cfg.image_max_pixels,
-                                                   video_max_pixels=cfg.video_max_pixels)
+        self.processor = self.chat = self.hf_processor = None
+        if self.arch.multimodal:
+            self._load_media_front_end()
         self._ids = RequestIdAllocator()
         self.metrics = EngineMetrics()
         # CUDA engines keep a request's patches as pinned bf16 (the model's dtype): the copy to the
@@ -138,6 +125,25 @@ class LLMEngine:
         self._steps_since_status = 0
         atexit.register(self.exit)
 
+    def _load_media_front_end(self) -> None:
+        """Patch processor, chat prompts and (on request) the checkpoint's own processor of a multimodal family."""
+        cfg = self.config
+        # options given by the caller win; otherwise the budgets the checkpoint's own processor files record
+        recorded = checkpoint_pixel_budgets(cfg.model) if os.path.isdir(str(cfg.model)) else {}
+        self.processor = PatchProcessor(self.arch, min_pixels=cfg.image_min_pixels or recorded.get("min_pixels"),
+                                        max_pixels=cfg.image_max_pixels or recorded.get("max_pixels"),
+                                        video_max_pixels=cfg.video_max_pixels or recorded.get("video_max_pixels"),
+                                        video_min_pixels=recorded.get("video_min_pixels"), video_fps=recorded.get("video_fps"),
+                                        video_min_frames=recorded.get("video_min_frames"), video_max_frames=recorded.get("video_max_frames"))
+        from .chat_prompt import ChatPrompt, HFProcessorAdapter
+
+        mode = cfg.chat_template
+        chat = ChatPrompt(self.tokenizer)
+        self.chat = chat if (mode == "always" or (mode == "auto" and chat.has_template)) else None
+        if cfg.hf_processor == "always":
+            self.hf_processor = HFProcessorAdapter(cfg.model, image_max_pixels=cfg.image_max_pixels,
+                                                   video_max_pixels=cfg.video_max_pixels)
+
     def _validate_environment(self, device: str | None) -> None:
         """Fail before tokenizer, worker processes or weights exist (reference
         ``prism_infer/engine/llm_engine.py:151-167``).  A CPU engine (``device="cpu"``, the oracle
@@ -147,6 +153,10 @@ class LLMEngine:
 
         cfg = self.config
         on_cuda = torch.cuda.is_available() if device is None else str(device).startswith("cuda")
+        if cfg.prism.model.dtype == "bfloat16" and not on_cuda:
+            raise ValueError("the CPU engine computes in float32: dtype must be 'auto' or 'float32' there")
+        if cfg.prism.model.dtype == "float32" and on_cuda and not cfg.family.float32_on_cuda:
+            raise ValueError(f"dtype 'float32' on CUDA: the {cfg.family.name} family has bfloat16 kernels only")
         if on_cuda:
             validate_runtime_capabilities(True, execution_backend=cfg.prism.execution.backend,
                                           compression_mode=cfg.compression_mode)
@@ -209,6 +219,7 @@ class LLMEngine:
     def _multimodal_sequence(self, inputs: ImageInputs | VideoInputs, sp: SamplingParams | None,
                              media_key: str | None = None) -> Sequence:
         arch = self.arch
+        self._require_media()
         image_grid = getattr(inputs, "image_grid_thw", None)
         video_grid = getattr(inputs, "video_grid_thw", None)
         inputs.validate(arch)
@@ -235,11 +246,16 @@ class LLMEngine:
                                    media_key: str | None = None, raise_on_reject: bool = True) -> int:
         return self._submit(self._multimodal_sequence(inputs, sampling_params, media_key), raise_on_reject=raise_on_reject)
 
+    def _require_media(self) -> None:
+        if not self.arch.multimodal:
+            raise ValueError(f"the {self.arch.model_type} family takes text prompts only")
+
     def prepare_images(self, prompt: str | Seq[int], images: Seq[Any], *, image_marker: str | None = None) -> ImageInputs:
         """Prompt + images -> ``ImageInputs`` the way this engine was configured: chat turns around a
         string prompt when the checkpoint has a chat template, the checkpoint's Hugging Face processor
         when ``hf_processor="always"``, the built-in patch processor otherwise.  ``image_marker``
         selects the interleaved layout (images where the marker appears in the prompt)."""
+        self._require_media()
         images = list(images)
         if self.hf_processor is not None and isinstance(prompt, str):
             chat = self.hf_processor.chat
@@ -254,6 +270,7 @@ class LLMEngine:
         """Prompt + sampled frames (+ ``chat_prompt.VideoTiming``) -> ``VideoInputs``; see ``prepare_images``.
         ``frames`` may also be the path of a video file: its frames are sampled at two per second of source time
         (4 to 768 of them, evenly spaced) and their source times go into the prompt's time stamps."""
+        self._require_media()
         if isinstance(frames, (str, os.PathLike)):
             p = self.processor
             frames, file_timing = load_video_file(os.fspath(frames), fps=p.video_fps, min_frames=p.video_min_frames, max_frames=p.video_max_frames)

@@ -5,8 +5,9 @@ with packed staging ``:1219-1313``).
 
 B200-specific choices:
 
-* One KV allocation ``[2, L, pages, Hkv/tp, page, D]`` (+ fp32 scales), sized from free HBM,
-  head-major inside a page so each (page, head) is one contiguous 32 KB run of E4M3 bytes.
+* One KV allocation ``[planes, L, pages, Hkv/tp, page, D]`` (+ fp32 scales; two planes for keys and
+  values, one for a shared latent; L counts layer executions, a looped layer has one slab per pass),
+  sized from free HBM, head-major inside a page so each (page, head) is one contiguous 32 KB run of E4M3 bytes.
 * Decode runs as one CUDA graph per batch bucket (1, 2, 4, 8, 16, 32, ...).  A single packed
   pinned host buffer is copied to the device by a memcpy node *inside* the graph, and the
   sampled tokens are copied back to pinned memory by another node, so a step is: fill the
@@ -25,7 +26,8 @@ import torch
 
 from .. import ops
 from ..config import Config
-from ..models.qwen3_vl import AttnMeta, Qwen3VLModel, TPComm
+from ..models.common import AttnMeta, TPComm
+from ..models.model_registry import load_model_class
 from ..models.weights import open_weight_source
 from ..observability import profile_region
 from .contracts import KVTransferPlan
@@ -75,6 +77,7 @@ class _DecodeGraph:
         self.flip = 0
         self.step = torch.zeros(1, dtype=torch.int64, device=dev)
         self.graph: Optional[torch.cuda.CUDAGraph] = None
+        self.logits: Optional[torch.Tensor] = None  # fp32 logits the captured sampler read
         self._nps = [tuple(t.numpy() for t in self._views(h, bucket, mb)) for h in self.hosts]
         self._rows = [0, 0]  # rows of each staging buffer that hold real sequences
         for k in (0, 1):
@@ -154,7 +157,7 @@ class ModelRunner:
         self.comm = comm or TPComm()
         self.on_cuda = torch.cuda.is_available() if device is None else str(device).startswith("cuda")
         self.device = torch.device(device if device is not None else (f"cuda:{torch.cuda.current_device()}" if self.on_cuda else "cpu"))
-        self.dtype = torch.bfloat16 if self.on_cuda else torch.float32
+        self.dtype = torch.bfloat16 if self.on_cuda and config.prism.model.dtype != "float32" else torch.float32
         arch = config.arch
         if self.on_cuda:
             from ..ops import native
@@ -163,11 +166,11 @@ class ModelRunner:
             ops.set_pdl(config.programmatic_dependent_launch)
             ops.apply_tuning()
         with profile_region("runner.load_weights"):
-            self.model = Qwen3VLModel(arch, device=self.device, dtype=self.dtype, comm=self.comm)
+            self.model = load_model_class(config.family)(arch, device=self.device, dtype=self.dtype, comm=self.comm)
             source = weights.items() if weights is not None else open_weight_source(
                 config.model, arch, dtype=self.dtype, device=self.device, seed=config.seed)()
             self.model.load(source)
-            if config.logits_precision == "selective_fp32" and self.on_cuda:
+            if config.logits_precision == "selective_fp32" and self.on_cuda and hasattr(self.model, "enable_fp8_candidate_head"):
                 self.model.enable_fp8_candidate_head()
         self.page = config.kvcache_block_size
         self.max_blocks = -(-config.max_model_len // self.page)
@@ -192,8 +195,7 @@ class ModelRunner:
 
     # ------------------------------------------------------------------ KV arena
     def _allocate_kv(self) -> None:
-        cfg, t = self.config, self.config.arch.text
-        hkv = t.num_kv_heads // self.comm.size
+        cfg = self.config
         per_page = cfg.kv_bytes_per_page()
         blocks = cfg.num_kvcache_blocks
         if blocks <= 0:
@@ -206,10 +208,14 @@ class ModelRunner:
             want = int(blocks * cfg.cpu_kv_cache_ratio)
             cap = (4 << 30) // per_page if self.on_cuda else 64
             cpu_blocks = min(want, cap)
-        self.kv = ops.KVCache(t.num_layers, blocks, hkv, self.page, t.head_dim, self.kv_mode, self.device, dtype=self.dtype)
-        self.cpu_kv = ops.KVCache(t.num_layers, max(1, cpu_blocks), hkv, self.page, t.head_dim, self.kv_mode, "cpu",
-                                  dtype=self.dtype, pin_memory=self.on_cuda) if cpu_blocks > 0 else None
+        self.kv = self._new_cache(blocks, self.device)
+        self.cpu_kv = self._new_cache(max(1, cpu_blocks), "cpu", pin_memory=self.on_cuda) if cpu_blocks > 0 else None
         cfg.with_cache_capacity(blocks, cpu_blocks)
+
+    def _new_cache(self, blocks: int, device, pin_memory: bool = False) -> ops.KVCache:
+        g = self.config.arch.kv_geometry(self.comm.size)
+        return ops.KVCache(g.layers, blocks, g.heads, self.page, g.row, self.kv_mode, device, dtype=self.dtype,
+                           pin_memory=pin_memory, planes=g.planes)
 
     GRAPH_POOL_RESERVE = 1 << 30  # decode-graph pools, vision-tower activations and allocator slack
 
@@ -221,22 +227,22 @@ class ModelRunner:
         cache, and the KV arena gets ``total * gpu_memory_utilization`` minus what is allocated now, minus
         the measured peak above that, minus a fixed reserve for graph pools.  Every tensor-parallel rank
         runs the same warm-up (its collectives pair up)."""
-        cfg, t = self.config, self.config.arch.text
+        cfg = self.config
         dev = self.device
         tokens = max(1, min(int(cfg.max_num_batched_tokens), int(cfg.max_model_len)))
-        hkv = t.num_kv_heads // self.comm.size
         torch.cuda.synchronize(dev)
         base = torch.cuda.memory_allocated(dev)
         torch.cuda.reset_peak_memory_stats(dev)
         scratch_pages = -(-tokens // self.page) + 1
-        scratch = ops.KVCache(t.num_layers, scratch_pages, hkv, self.page, t.head_dim, self.kv_mode, dev, dtype=self.dtype)
+        scratch = self._new_cache(scratch_pages, dev)
         ids = torch.zeros(tokens, dtype=torch.int64, device=dev)
         pos = torch.arange(tokens, dtype=torch.int32, device=dev).repeat(3, 1).contiguous()
         slots = torch.arange(tokens, dtype=torch.int64, device=dev)
         bt = torch.arange(scratch_pages, dtype=torch.int32, device=dev).view(1, -1)
         meta = AttnMeta(is_prefill=True, block_tables=bt, slots=slots,
                         cu_seqlens_q=torch.tensor([0, tokens], dtype=torch.int32, device=dev),
-                        kv_lens=torch.tensor([tokens], dtype=torch.int32, device=dev), max_q_len=tokens, no_history=True)
+                        kv_lens=torch.tensor([tokens], dtype=torch.int32, device=dev), max_q_len=tokens, no_history=True,
+                        total_kv=tokens, max_kv_len=tokens, attended_pairs=tokens * tokens)
         hidden = self.model.forward(ids, pos, meta, scratch)
         self.model.sample(hidden[-1:], None)
         torch.cuda.synchronize(dev)
@@ -512,11 +518,13 @@ class ModelRunner:
             meta = AttnMeta(
                 is_prefill=True, block_tables=self._to_dev(inp.block_tables), slots=self._to_dev(inp.slots),
                 cu_seqlens_q=self._to_dev(inp.cu_seqlens_q), kv_lens=self._to_dev(inp.kv_lens), max_q_len=inp.max_q_len,
-                no_history=bool(torch.equal(inp.kv_lens, inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1])))
+                no_history=bool(torch.equal(inp.kv_lens, inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1])),
+                total_kv=int(inp.kv_lens.sum()), max_kv_len=int(inp.kv_lens.max()),
+                attended_pairs=int(((inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1]).long() * inp.kv_lens.long()).sum()))
             if not meta.no_history:  # key ranges for the gather + tensor-core attention over the paged cache
                 cu_kv = torch.zeros(inp.kv_lens.shape[0] + 1, dtype=torch.int32)
                 cu_kv[1:] = torch.cumsum(inp.kv_lens, 0)
-                meta.cu_seqlens_kv, meta.total_kv, meta.max_kv_len = self._to_dev(cu_kv), int(cu_kv[-1]), int(inp.kv_lens.max())
+                meta.cu_seqlens_kv = self._to_dev(cu_kv)
             ids, pos, vis_index = self._to_dev(inp.input_ids), self._to_dev(inp.positions), self._to_dev(inp.vis_index)
             if inp.score_rows:
                 from .visual_pruning import RuntimeVisualTokenScorer
@@ -541,11 +549,37 @@ class ModelRunner:
             tok = self.model.sample(rows, temps, seed=self.sample_seed, step=step)
         return tok.tolist()
 
-    def _run_prefill(self, inp: StepInputs) -> list[int]:
+    def _prefill_hidden(self, inp: StepInputs) -> tuple[AttnMeta, torch.Tensor]:
         ids, pos, meta, visual, vis_index, deep = self._prefill_inputs(inp)
         with profile_region("runner.run_model"):
-            hidden = self.model.forward(ids, pos, meta, self.kv, visual=visual, vis_index=vis_index, deepstack=deep)
-        return self._prefill_outputs(inp, meta, hidden)
+            return meta, self.model.forward(ids, pos, meta, self.kv, visual=visual, vis_index=vis_index, deepstack=deep)
+
+    def _run_prefill(self, inp: StepInputs) -> list[int]:
+        return self._prefill_outputs(inp, *self._prefill_hidden(inp))
+
+    def step_logits(self, inp: StepInputs, rows: Seq[int]) -> torch.Tensor:
+        """Run one step exactly as ``execute`` does and return the fp32 logits ``[len(rows), vocab]`` (CPU) of the
+        given flattened token rows instead of sampled tokens.  Decode steps replay the bucket's captured graph when
+        ``enable_step_logits`` let it keep its logits.  One rank."""
+        if self.comm.size != 1:
+            raise ValueError("step_logits runs on one rank")
+        self.steps_run += 1
+        self._ahead = None
+        index = torch.tensor(list(rows), dtype=torch.int64)
+        if inp.kind == "prefill":
+            _, hidden = self._prefill_hidden(inp)
+        elif self.graphs and self.config.step_logits and inp.num_seqs <= self.buckets[-1]:
+            g = self.graphs[next(b for b in self.buckets if b >= inp.num_seqs)]
+            k = g.fill(inp)
+            g.launch(k, inp.num_seqs)
+            g.wait(k, inp.num_seqs)
+            return g.logits[self._to_dev(index)].float().cpu()
+        else:
+            hidden = self._decode_hidden_eager(inp)
+        if not rows:
+            self.barrier()
+            return torch.empty((0, self.config.arch.vocab_size), dtype=torch.float32)
+        return self.model.logits(hidden[self._to_dev(index)].contiguous()).float().cpu()
 
     # ---- cooperative prefill: the same step, a few decoder layers at a time (reference
     # ``engine/model_runner.py:1346-1650``; one rank) -----------------------------------------------
@@ -577,10 +611,13 @@ class ModelRunner:
             hidden = self.model.finish_layers(state)
         return self._prefill_outputs(inp, state.meta, hidden)
 
-    def _run_decode_eager(self, inp: StepInputs) -> list[int]:
+    def _decode_hidden_eager(self, inp: StepInputs) -> torch.Tensor:
         meta = AttnMeta(is_prefill=False, block_tables=self._to_dev(inp.block_tables), slots=self._to_dev(inp.slots),
                         context_lens=self._to_dev(inp.context_lens))
-        hidden = self.model.forward(self._to_dev(inp.input_ids), self._to_dev(inp.positions), meta, self.kv)
+        return self.model.forward(self._to_dev(inp.input_ids), self._to_dev(inp.positions), meta, self.kv)
+
+    def _run_decode_eager(self, inp: StepInputs) -> list[int]:
+        hidden = self._decode_hidden_eager(inp)
         temps = self._to_dev(inp.temperatures) if bool((inp.temperatures > 0).any()) else None
         step = torch.tensor([self.steps_run], dtype=torch.int64, device=self.device)
         return self.model.sample(hidden, temps, seed=self.sample_seed, step=step).tolist()
@@ -591,6 +628,9 @@ class ModelRunner:
                         nsplit=ops.decode_splits(g.bucket, self.kv.num_kv_heads))
         hidden = self.model.forward(g.d_ids, g.d_pos, meta, self.kv)
         self.model.sample(hidden, None if g.greedy_only else g.d_temp, seed=self.sample_seed, step=g.step, out=g.tokens)
+        if self.config.step_logits:  # held, the buffer stays the graph's own; otherwise the graphs of a pool share it
+            g.logits = self.model.sampled_logits
+        self.model.sampled_logits = None
 
     def capture_graphs(self) -> None:
         """Capture one graph per bucket, largest first so smaller ones reuse its pool."""

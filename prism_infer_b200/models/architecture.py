@@ -1,4 +1,4 @@
-"""Validated Qwen3-VL architecture description.
+"""Validated architecture descriptions, one frozen dataclass tree per model family.
 
 The engine never reads a Hugging Face config object directly: it converts the
 ``config.json`` dictionary (or an ``AutoConfig`` instance) into the frozen
@@ -6,7 +6,11 @@ dataclasses below once and every later layer (weight sharding, kernels, KV sizin
 reads these.  Mirrors the contract of the reference's
 ``prism_infer/models/qwen3_vl_architecture.py:117-428`` (canonical 8B constants at
 ``:18-44``): interleaved M-RoPE only, no attention bias, SiLU text MLP, GELU-tanh
-vision MLP.
+vision MLP.  ``PoralornArch`` (end of file) is the text-only looped latent-attention family.
+
+What the engine asks of any architecture, whatever its family: ``model_type``, ``multimodal``,
+``vocab_size``, ``max_positions`` (``None``: unbounded), ``num_layer_runs``, ``eos_token_id``, the
+visual token ids (-1 where there are none), ``reserved_token_ids`` and ``kv_geometry(tp)``.
 """
 
 from __future__ import annotations
@@ -17,6 +21,21 @@ from dataclasses import asdict, dataclass, field
 from typing import Any, Mapping
 
 SUPPORTED_MODEL_TYPES = frozenset({"qwen3_vl"})
+
+
+@dataclass(frozen=True)
+class KVGeometry:
+    """Shape of one rank's paged cache: ``planes`` slabs per layer run (2: keys and values, 1: a shared
+    latent), each ``[pages, heads, page, row]``."""
+
+    planes: int
+    layers: int
+    heads: int
+    row: int
+
+    def bytes_per_page(self, page: int, element_bytes: int, scaled: bool = False) -> int:
+        rows = self.planes * self.layers * self.heads * page
+        return rows * self.row * element_bytes + (rows * 4 if scaled else 0)
 
 
 def _get(cfg: Any, *names: str, default: Any = ...) -> Any:
@@ -135,6 +154,28 @@ class Qwen3VLArch:
         ids = (self.image_token_id, self.video_token_id, self.vision_start_token_id)
         if len(set(ids)) != 3:
             raise ValueError(f"visual special token ids must be distinct: {ids}")
+
+    # ---- what the engine reads of every family ---------------------------------
+    multimodal = True
+
+    @property
+    def vocab_size(self) -> int:
+        return self.text.vocab_size
+
+    @property
+    def max_positions(self) -> int | None:
+        return self.text.max_position_embeddings
+
+    @property
+    def num_layer_runs(self) -> int:
+        return self.text.num_layers
+
+    @property
+    def reserved_token_ids(self) -> tuple[int, ...]:
+        return (self.image_token_id, self.video_token_id, self.vision_start_token_id, self.vision_end_token_id, self.eos_token_id)
+
+    def kv_geometry(self, tp: int = 1) -> KVGeometry:
+        return KVGeometry(2, self.text.num_layers, self.text.num_kv_heads // tp, self.text.head_dim)
 
     # ---- factories -----------------------------------------------------------
     @classmethod
@@ -320,10 +361,14 @@ class Qwen3VLArch:
         return asdict(self)
 
 
-def validate_tensor_parallel(arch: Qwen3VLArch, tp: int) -> None:
+def validate_tensor_parallel(arch: Any, tp: int) -> None:
     """Every sharded dimension must divide evenly (reference ``engine/llm_engine.py:117-143``)."""
     if tp < 1:
         raise ValueError("tensor_parallel_size must be >= 1")
+    if isinstance(arch, PoralornArch):
+        if tp != 1:
+            raise ValueError("the Poralorn family runs on one GPU (tensor_parallel_size 1)")
+        return
     t = arch.text
     for name, value in (
         ("num_heads", t.num_heads),
@@ -334,3 +379,191 @@ def validate_tensor_parallel(arch: Qwen3VLArch, tp: int) -> None:
     ):
         if value % tp:
             raise ValueError(f"tensor_parallel_size {tp} does not divide text {name}={value}")
+
+
+# ------------------------------------------------------------------------------- Poralorn
+@dataclass(frozen=True)
+class LatentAttentionArch:
+    """Sizes of one latent-attention mixer: ``heads`` heads whose ``dim``-wide keys and ``vdim``-wide values
+    are linear in one shared ``kv_rank``-wide latent per token (the only thing cached)."""
+
+    heads: int
+    dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+
+    def __post_init__(self) -> None:
+        for name in ("heads", "dim", "vdim", "kv_rank"):
+            if getattr(self, name) < 1:
+                raise ValueError(f"latent attention: {name} must be positive")
+
+
+@dataclass(frozen=True)
+class PoralornLayer:
+    mixer: LatentAttentionArch
+    ff: int = 0                      # width of the feed-forward, 0: the layer has none
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    """One execution of a layer.  ``loop_pass`` is the pass number on the first layer of a pass of the looped
+    section (where the loop input is formed) and ``None`` elsewhere."""
+
+    layer: int
+    loop_pass: int | None = None
+
+
+@dataclass(frozen=True)
+class PoralornArch:
+    vocab_size: int
+    width: int
+    layers: tuple[PoralornLayer, ...]
+    loop_start: int = 0              # layers loop_start .. loop_stop - 1 run loop_times times in a row
+    loop_stop: int = 0
+    loop_times: int = 0              # 0: no looped section
+    norm_eps: float = 1.0e-5
+    residual_mult: float = 1.0
+    logit_softcap: float = 0.0       # 0: logits are not capped
+    eos_token_id: int = -1
+    model_type: str = "poralorn"
+
+    multimodal = False
+    image_token_id = -1
+    video_token_id = -1
+
+    def __post_init__(self) -> None:
+        if self.vocab_size < 1 or self.width < 1 or not self.layers:
+            raise ValueError("vocab, width and layers must be given")
+        if self.loop_times < 0 or (self.has_loop and not 0 <= self.loop_start < self.loop_stop <= len(self.layers)):
+            raise ValueError(f"loop {self.loop_start} .. {self.loop_stop} x {self.loop_times} does not fit {len(self.layers)} layers")
+        if self.norm_eps < 0 or self.logit_softcap < 0:
+            raise ValueError("norm eps and logit_softcap must not be negative")
+
+    # ---- what the engine reads of every family ---------------------------------
+    @property
+    def has_loop(self) -> bool:
+        return self.loop_times > 0
+
+    @property
+    def max_positions(self) -> int | None:
+        return None                  # no position enters the computation except through the causal order
+
+    @property
+    def reserved_token_ids(self) -> tuple[int, ...]:
+        return ()
+
+    def layer_runs(self) -> tuple[LayerRun, ...]:
+        """Every layer execution in order; run ``i`` owns cache slab ``i``."""
+        if not self.has_loop:
+            return tuple(LayerRun(i) for i in range(len(self.layers)))
+        runs = [LayerRun(i) for i in range(self.loop_start)]
+        for t in range(self.loop_times):
+            runs += [LayerRun(i, t if i == self.loop_start else None) for i in range(self.loop_start, self.loop_stop)]
+        return tuple(runs + [LayerRun(i) for i in range(self.loop_stop, len(self.layers))])
+
+    @property
+    def num_layer_runs(self) -> int:
+        return len(self.layer_runs())
+
+    @property
+    def latent_row(self) -> int:
+        """Elements of one cached latent row: the widest latent, rounded up to whole 64-element tiles."""
+        return -(-max(l.mixer.kv_rank for l in self.layers) // 64) * 64
+
+    def kv_geometry(self, tp: int = 1) -> KVGeometry:
+        return KVGeometry(1, self.num_layer_runs, 1, self.latent_row)
+
+    # ---- checkpoint --------------------------------------------------------------
+    def weight_shapes(self) -> dict[str, tuple[int, ...]]:
+        s: dict[str, tuple[int, ...]] = {"embed": (self.vocab_size, self.width)}
+        if self.has_loop:
+            s["loop.in"] = (self.width, 2 * self.width)
+            s["loop.step"] = (self.loop_times, self.width)
+        for i, l in enumerate(self.layers):
+            m, p = l.mixer, f"l{i}"
+            s[f"{p}.norm1"] = ()
+            s[f"{p}.mix.q"] = (m.heads * m.dim, self.width)
+            s[f"{p}.mix.dkv"] = (m.kv_rank, self.width)
+            s[f"{p}.mix.dkv.norm"] = (m.kv_rank,)
+            s[f"{p}.mix.uk"] = (m.heads * m.dim, m.kv_rank)
+            s[f"{p}.mix.uv"] = (m.heads * m.vdim, m.kv_rank)
+            s[f"{p}.mix.g"] = (m.heads * m.vdim, self.width)
+            s[f"{p}.mix.o"] = (self.width, m.heads * m.vdim)
+            s[f"{p}.rg1"] = (self.width, self.width)
+            s[f"{p}.rg1.b"] = (self.width,)
+            if l.ff:
+                s[f"{p}.norm2"] = ()
+                s[f"{p}.mlp.up"] = (l.ff, self.width)
+                s[f"{p}.mlp.down"] = (self.width, l.ff)
+                s[f"{p}.rg2"] = (self.width, self.width)
+                s[f"{p}.rg2.b"] = (self.width,)
+        s["final.norm"] = ()
+        s["head"] = (self.vocab_size, self.width)
+        return s
+
+    @staticmethod
+    def init_kind(name: str) -> str:
+        """How random initialisation draws a tensor: ``norm``, ``bias``, ``embedding`` or ``matrix``."""
+        if name.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2"):
+            return "norm"
+        if name.endswith(".b") or name == "loop.step":
+            return "bias"
+        return "embedding" if name == "embed" else "matrix"
+
+    # ---- factories ---------------------------------------------------------------
+    @classmethod
+    def from_hf_config(cls, cfg: Mapping[str, Any]) -> "PoralornArch":
+        """From the ``config.json`` dictionary."""
+
+        def need(d: Mapping[str, Any], key: str, where: str = "config") -> Any:
+            if key not in d:
+                raise ValueError(f"Poralorn {where} is missing required field {key}")
+            return d[key]
+
+        layers = []
+        for i, entry in enumerate(need(cfg, "layers")):
+            where = f"layer {i}"
+            kind = need(entry, "type", where)
+            if kind != "latent_attention":
+                raise ValueError(f"Poralorn {where}: unsupported mixer {kind!r}")
+            m = need(entry, "mixer", where)
+            mixer = LatentAttentionArch(*(int(need(m, k, where)) for k in ("heads", "dim", "vdim", "kv_rank")),
+                                        float(need(m, "scale", where)))
+            mlp = entry.get("mlp")
+            if mlp is not None and mlp.get("kind") != "dense":
+                raise ValueError(f"Poralorn {where}: unsupported feed-forward {mlp.get('kind')!r}")
+            layers.append(PoralornLayer(mixer, int(need(mlp, "ff", where)) if mlp is not None else 0))
+        loop = cfg.get("loop") or {}
+        return cls(
+            vocab_size=int(need(cfg, "vocab")), width=int(need(cfg, "width")), layers=tuple(layers),
+            loop_start=int(need(loop, "start", "loop")) if loop else 0, loop_stop=int(need(loop, "stop", "loop")) if loop else 0,
+            loop_times=int(need(loop, "times", "loop")) if loop else 0,
+            norm_eps=float(need(need(cfg, "norm"), "eps", "norm")), residual_mult=float(need(cfg, "residual_mult")),
+            logit_softcap=float(cfg.get("logit_softcap") or 0.0))
+
+    def to_hf_config(self) -> dict[str, Any]:
+        """The ``config.json`` dictionary ``from_hf_config`` reads."""
+        out: dict[str, Any] = {"architecture": "Poralorn", "vocab": self.vocab_size, "width": self.width,
+                               "norm": {"eps": self.norm_eps}, "residual_mult": self.residual_mult,
+                               "logit_softcap": self.logit_softcap,
+                               "layers": [{"type": "latent_attention", "mixer": asdict(l.mixer),
+                                           "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None} for l in self.layers]}
+        if self.has_loop:
+            out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return out
+
+    @classmethod
+    def tiny(cls) -> "PoralornArch":
+        """The small CPU test model: five layer runs, every size different."""
+        mixers = (LatentAttentionArch(3, 32, 24, 40, 0.17), LatentAttentionArch(5, 16, 16, 72, 0.25))
+        return cls(vocab_size=300, width=160, layers=(PoralornLayer(mixers[0], 208), PoralornLayer(mixers[1]), PoralornLayer(mixers[0], 96)),
+                   loop_start=1, loop_stop=2, loop_times=3, norm_eps=1e-5, residual_mult=0.4, logit_softcap=12.0)
+
+    @classmethod
+    def like_8b(cls, layers: int = 4, *, width: int = 4096, heads: int = 32, dim: int = 128, kv_rank: int = 512,
+                ff: int = 12288, vocab_size: int = 151_936) -> "PoralornArch":
+        """Layers with the widths of an 8B-class decoder (measurement model; random weights)."""
+        mixer = LatentAttentionArch(heads, dim, dim, kv_rank, dim ** -0.5)
+        return cls(vocab_size=vocab_size, width=width, layers=(PoralornLayer(mixer, ff),) * layers, residual_mult=0.5,
+                   logit_softcap=30.0)

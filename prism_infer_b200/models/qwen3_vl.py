@@ -27,35 +27,9 @@ import torch
 
 from .. import ops
 from .architecture import Qwen3VLArch
+from .common import SMALL_T, AttnMeta, TPComm
 from .position import vision_patch_coords, vision_pos_embed_plan, vision_segments
 from .weights import LM, VIS
-
-# at or below this many tokens the GEMMs are weight-streaming: split-K + fp32 partials
-SMALL_T = 128
-
-
-@dataclass
-class AttnMeta:
-    """Device-side attention metadata of one step."""
-
-    is_prefill: bool
-    block_tables: torch.Tensor                     # [S, max_blocks] int32
-    slots: torch.Tensor                            # [T] int64 flat KV slots of the new tokens
-    # prefill
-    cu_seqlens_q: Optional[torch.Tensor] = None    # [S+1] int32
-    kv_lens: Optional[torch.Tensor] = None         # [S] int32 keys visible (history + chunk)
-    cu_seqlens_kv: Optional[torch.Tensor] = None   # [S+1] int32 running sum of kv_lens (None: the page-reading kernel)
-    total_kv: int = 0                              # sum and maximum of kv_lens, known on the host
-    max_kv_len: int = 0
-    max_q_len: int = 0
-    last_rows: Optional[torch.Tensor] = None       # [S] int64 row of each sequence's last token
-    no_history: bool = False                       # every sequence attends only to this chunk's own keys
-    # decode
-    context_lens: Optional[torch.Tensor] = None    # [B] int32 (including the new token)
-    nsplit: int = 0
-    workspace: Optional[tuple[torch.Tensor, torch.Tensor]] = None
-    # prefill with the attention pruning strategy: collects last-query attention over visual tokens
-    scorer: Optional[object] = None
 
 
 @dataclass
@@ -129,50 +103,6 @@ class LayerwiseState:
     ticket: object = None
     residual: Optional[torch.Tensor] = None
     next_layer: int = 0
-
-
-class TPComm:
-    """Collective hooks of a tensor-parallel rank; the single-rank default does nothing."""
-
-    rank = 0
-    size = 1
-
-    def reduce_partials(self, partials: torch.Tensor) -> torch.Tensor:
-        """fp32 ``[S, T, H]`` rank-local partial slabs -> slabs whose sum is the full result."""
-        return partials
-
-    def reduce_dense(self, x: torch.Tensor) -> torch.Tensor:
-        """bf16 ``[T, H]`` rank-local partial result -> summed over ranks."""
-        return x
-
-    def greedy_merge(self, local_val: torch.Tensor, local_id: torch.Tensor) -> torch.Tensor:
-        return local_id
-
-    def gather_logits(self, logits: torch.Tensor) -> torch.Tensor:
-        return logits
-
-    def all_gather_rows(self, x: torch.Tensor) -> torch.Tensor:
-        return x
-
-    def begin_step(self) -> None:
-        return None
-
-    def row_parallel(self, x: torch.Tensor, w: torch.Tensor, stages: int = 0):
-        """Row-parallel projection -> ``(dense, partials, ticket)``; exactly one is set.
-        ``stages`` caps the operand ring of a decode-sized launch (0 = as deep as fits)."""
-        T = x.shape[0]
-        # short prefills (up to 511 tokens) split K too: o_proj and down_proj have 32 weight tiles at 8B widths,
-        # one CTA each would leave 116 SMs idle
-        if T <= SMALL_T or (x.is_cuda and T <= ops.SPLIT_K_MAX_TOKENS):
-            splits = ops.choose_splits(w.shape[0], w.shape[1], T) if x.is_cuda else 1
-            if splits > 1 or T <= SMALL_T:
-                return None, ops.linear_partial(x, w, splits, stages=stages), None
-        return ops.linear(x, w), None, None
-
-    def add_rmsnorm(self, weight, eps, dense, partials, ticket, residual, extra=None, extra_index=None):
-        """``(normed, new_residual)`` from whatever ``row_parallel`` returned."""
-        return ops.add_rmsnorm(weight, eps, x=dense, partials=partials, residual=residual, extra=extra,
-                               extra_index=extra_index)
 
 
 class Qwen3VLModel:
@@ -710,8 +640,9 @@ class Qwen3VLModel:
         if (fp8_head is not None and temperature is None and self.tp == 1 and hidden.is_cuda
                 and hidden.shape[0] <= ops.LM_HEAD_FP8_BATCH and not self.__dict__.get("keep_logits")):
             # greedy rows: candidates from the E4M3 copy of the head (half the bytes), exact rerank with the bf16 rows
+            self.sampled_logits = None
             return ops.lm_head_fp8_greedy(hidden, fp8_head[0], fp8_head[1], self.lm_head, out=out)
-        logits = self.logits(hidden)
+        logits = self.sampled_logits = self.logits(hidden)
         if self.__dict__.get("keep_logits"):
             # debugging aid (eager execution): full-vocabulary fp32 logits of the last sampled rows
             self.last_logits = (logits if self.tp == 1 else self.comm.gather_logits(logits)).float().clone()

@@ -1,6 +1,7 @@
-"""Checkpoint tensors under their Hugging Face names: shapes, random init, safetensors IO.
+"""Checkpoint tensors under their checkpoint names: shapes, random init, safetensors IO.
 
-The engine keeps HF names as the single naming scheme (reference
+An architecture with ``weight_shapes()`` and ``init_kind()`` of its own (the Poralorn family) is asked for
+them; for Qwen3-VL the engine keeps HF names as the single naming scheme (reference
 ``prism_infer/utils/loader.py:17-36`` and ``prism_infer/models/qwen3_vl.py:1205-1222``):
 ``model.language_model.layers.N.self_attn.q_proj.weight``,
 ``model.visual.blocks.N.attn.qkv.weight``, ``model.visual.merger.linear_fc1.weight``,
@@ -12,7 +13,7 @@ from __future__ import annotations
 import glob
 import json
 import os
-from typing import Callable, Iterator
+from typing import Any, Callable, Iterator
 
 import torch
 
@@ -22,8 +23,10 @@ LM = "model.language_model"
 VIS = "model.visual"
 
 
-def weight_shapes(arch: Qwen3VLArch) -> dict[str, tuple[int, ...]]:
+def weight_shapes(arch: Any) -> dict[str, tuple[int, ...]]:
     """Name -> shape of every checkpoint tensor, in load order."""
+    if not isinstance(arch, Qwen3VLArch):
+        return arch.weight_shapes()
     t, v = arch.text, arch.vision
     s: dict[str, tuple[int, ...]] = {}
     s[f"{VIS}.patch_embed.proj.weight"] = (
@@ -81,8 +84,18 @@ def _is_norm_weight(name: str) -> bool:
         or ".norm2.weight" in name
 
 
+def _init_kind(arch: Any, name: str) -> str:
+    if not isinstance(arch, Qwen3VLArch):
+        return arch.init_kind(name)
+    if _is_norm_weight(name):
+        return "norm"
+    if name.endswith(".bias"):
+        return "bias"
+    return "embedding" if name.endswith(("embed_tokens.weight", "pos_embed.weight")) else "matrix"
+
+
 def iter_random_weights(
-    arch: Qwen3VLArch,
+    arch: Any,
     *,
     dtype: torch.dtype = torch.bfloat16,
     device: str | torch.device = "cpu",
@@ -98,11 +111,12 @@ def iter_random_weights(
     for index, (name, shape) in enumerate(weight_shapes(arch).items()):
         gen = torch.Generator(device=device)
         gen.manual_seed(seed * 1_000_003 + index)
-        if _is_norm_weight(name):
+        kind = _init_kind(arch, name)
+        if kind == "norm":
             w = 1.0 + 0.05 * torch.randn(shape, generator=gen, device=device, dtype=torch.float32)
-        elif name.endswith(".bias"):
+        elif kind == "bias":
             w = 0.02 * torch.randn(shape, generator=gen, device=device, dtype=torch.float32)
-        elif name.endswith("embed_tokens.weight") or name.endswith("pos_embed.weight"):
+        elif kind == "embedding":
             w = 0.05 * torch.randn(shape, generator=gen, device=device, dtype=torch.float32)
         else:
             fan_in = 1
@@ -113,7 +127,7 @@ def iter_random_weights(
         yield name, w.to(dtype)
 
 
-def random_weights(arch: Qwen3VLArch, *, dtype=torch.float32, device="cpu", seed: int = 0) -> dict[str, torch.Tensor]:
+def random_weights(arch: Any, *, dtype=torch.float32, device="cpu", seed: int = 0) -> dict[str, torch.Tensor]:
     return dict(iter_random_weights(arch, dtype=dtype, device=device, seed=seed))
 
 
@@ -132,7 +146,7 @@ def iter_safetensors(path: str) -> Iterator[tuple[str, torch.Tensor]]:
 
 def save_checkpoint(
     path: str,
-    arch: Qwen3VLArch,
+    arch: Any,
     tensors: Iterator[tuple[str, torch.Tensor]] | dict[str, torch.Tensor],
     *,
     shard_bytes: int = 4 << 30,
@@ -171,7 +185,7 @@ def save_checkpoint(
 
 
 def open_weight_source(
-    model: str, arch: Qwen3VLArch, *, dtype: torch.dtype, device, seed: int = 0
+    model: str, arch: Any, *, dtype: torch.dtype, device, seed: int = 0
 ) -> Callable[[], Iterator[tuple[str, torch.Tensor]]]:
     """``model`` is a checkpoint directory, or ``random:<anything>`` for random init."""
     if model.startswith("random:") or not glob.glob(os.path.join(model, "*.safetensors")):

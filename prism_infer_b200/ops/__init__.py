@@ -277,13 +277,17 @@ def layernorm(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float) -> 
 
 # ------------------------------------------------------------------- KV cache container
 class KVCache:
-    """One allocation for every layer: payload ``[2, L, blocks, Hkv, page, D]`` (+ scales)."""
+    """One allocation for every layer: payload ``[planes, L, blocks, Hkv, page, D]`` (+ scales).
+
+    ``planes`` is 2 (keys and values) or 1 (one shared latent row per token, from which keys and values
+    are linear; ``Hkv`` is then 1 and ``latent(layer)`` the pages)."""
 
     def __init__(self, num_layers: int, num_blocks: int, num_kv_heads: int, page: int, head_dim: int,
-                 mode: int, device, dtype: torch.dtype = torch.bfloat16, pin_memory: bool = False):
+                 mode: int, device, dtype: torch.dtype = torch.bfloat16, pin_memory: bool = False, planes: int = 2):
+        self.planes = planes
         self.num_layers, self.num_blocks, self.num_kv_heads = num_layers, num_blocks, num_kv_heads
         self.page, self.head_dim, self.mode = page, head_dim, mode
-        shape = (2, num_layers, num_blocks, num_kv_heads, page, head_dim)
+        shape = (planes, num_layers, num_blocks, num_kv_heads, page, head_dim)
         pdtype = dtype if mode == KV_BF16 else torch.float8_e4m3fn
         kw = dict(device=device)
         if pin_memory:
@@ -297,6 +301,11 @@ class KVCache:
     def v(self, layer: int) -> torch.Tensor:
         return self.payload[1, layer]
 
+    def latent(self, layer: int) -> torch.Tensor:
+        """``[blocks, page, D]`` latent rows of one layer run (single-plane caches)."""
+        assert self.planes == 1 and self.num_kv_heads == 1
+        return self.payload[0, layer, :, 0]
+
     def k_scale(self, layer: int) -> Optional[torch.Tensor]:
         return None if self.scales is None else self.scales[0, layer]
 
@@ -305,10 +314,10 @@ class KVCache:
 
     @property
     def n_slabs(self) -> int:
-        return 2 * self.num_layers
+        return self.planes * self.num_layers
 
     def bytes_per_page(self) -> int:
-        n = 2 * self.num_layers * self.num_kv_heads * self.page
+        n = self.planes * self.num_layers * self.num_kv_heads * self.page
         return n * self.head_dim * self.payload.element_size() + (n * 4 if self.scales is not None else 0)
 
     def dequant(self, kv: int, layer: int) -> torch.Tensor:

@@ -36,8 +36,13 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found; set NVCC or add it to PATH")
 
 
-def _sources() -> list[str]:
-    return sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
+def _sources(units: tuple[str, ...] = ()) -> list[str]:
+    return sorted(f for f in os.listdir(CSRC) if f.endswith(".cu") and (not units or f[:-3] in units))
+
+
+def partial_library(name: str) -> str:
+    """Path of a library that holds the kernel units of one model family only."""
+    return os.path.join(HERE, f"libprism_b200_{name}.so")
 
 
 def _stale(target: str, deps: list[str]) -> bool:
@@ -47,14 +52,29 @@ def _stale(target: str, deps: list[str]) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(verbose: bool = False, force: bool = False) -> str:
-    """Compile what changed, link, return the library path."""
+def ensure(name: str, units: tuple[str, ...]) -> str:
+    """A library with at least ``units``: the full one when it is present and newer than its sources, else the
+    family's own, compiled now if need be.  Processes that start together build one after another."""
+    import fcntl
+
+    headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
+    deps = [os.path.join(CSRC, f) for f in _sources()] + headers
+    if not _stale(LIB, deps):
+        return LIB
+    os.makedirs(BUILD, exist_ok=True)
+    with open(os.path.join(BUILD, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build(units=units, target=partial_library(name))
+
+
+def build(verbose: bool = False, force: bool = False, *, units: tuple[str, ...] = (), target: str = LIB) -> str:
+    """Compile what changed, link, return the library path.  ``units`` restricts it to some ``csrc/*.cu`` files."""
     os.makedirs(BUILD, exist_ok=True)
     nvcc = _nvcc()
     headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
     jobs = []
     objects = []
-    for src in _sources():
+    for src in _sources(units):
         obj = os.path.join(BUILD, src[:-3] + ".o")
         objects.append(obj)
         if force or _stale(obj, [os.path.join(CSRC, src), *headers]):
@@ -74,13 +94,13 @@ def build(verbose: bool = False, force: bool = False) -> str:
                     sys.stderr.write(" ".join(cmd) + "\n" + res.stdout + res.stderr)
                 if res.returncode:
                     raise RuntimeError(f"nvcc failed for {cmd[-3]}")
-    if jobs or force or _stale(LIB, objects):
-        cmd = [nvcc, "-shared", "-o", LIB, *objects, "-lcudart"]
+    if jobs or force or _stale(target, objects):
+        cmd = [nvcc, "-shared", "-o", target, *objects, "-lcudart"]
         res = subprocess.run(cmd, capture_output=True, text=True)
         if res.returncode:
             sys.stderr.write(res.stdout + res.stderr)
             raise RuntimeError("link failed")
-    return LIB
+    return target
 
 
 if __name__ == "__main__":

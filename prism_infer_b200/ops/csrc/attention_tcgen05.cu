@@ -1,5 +1,6 @@
-// Prefill and vision attention on the fifth-generation tensor cores (bf16 Q/K/V rows, head
-// dimension 128, or 72 padded to 80 with zero columns that the TMA unit fills in).
+// Prefill and vision attention on the fifth-generation tensor cores (bf16 Q/K/V rows; head
+// dimensions up to 128 that are multiples of 8, padded to 64, 80 or 128 with zero columns that the
+// TMA unit fills in).
 //
 // One CTA handles 128 query rows of one (sequence, query head) and walks the keys in tiles of
 // 64.  Warp 0 streams K/V tiles with TMA (128-byte swizzle) into a two-stage ring, one thread
@@ -52,6 +53,8 @@ struct FaArgs {
   int hd;                 // real head dimension (<= HD_PAD)
   int causal;
   float scale;
+  const __nv_bfloat16* gate;  // output gate rows [T][gate_stride], laid out like out (null: none)
+  long long gate_stride;
 };
 
 __device__ __forceinline__ void named_bar(int id, int threads) {
@@ -146,9 +149,10 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   if (warp == 0) {
     if (lane == 0 && live) {
       // ------------------------------ TMA producer ------------------------------
-      mbar_expect_tx(q_full, Q_BYTES);
+      constexpr bool TWO = HD_PAD > 64;
+      mbar_expect_tx(q_full, TWO ? Q_BYTES : Q_BYTES / 2);
       tma_load_3d(q_s, &tmQ, q_full, 0, head, q_start + q0);
-      tma_load_3d(q_s + Q_BYTES / 2, &tmQ, q_full, 64, head, q_start + q0);
+      if (TWO) tma_load_3d(q_s + Q_BYTES / 2, &tmQ, q_full, 64, head, q_start + q0);
       bool ok = true;
       int issued = 0;
       for (int j = 0; j < n_tiles && ok; ++j) {
@@ -159,11 +163,11 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         }
         uint8_t* st = ring + (size_t)s * STAGE_BYTES;
         const int row = kv_start + j * FA_BN;
-        mbar_expect_tx(&kv_full[s], STAGE_BYTES);
+        mbar_expect_tx(&kv_full[s], TWO ? STAGE_BYTES : STAGE_BYTES / 2);
         tma_load_3d(st, &tmK, &kv_full[s], 0, kvh, row);
-        tma_load_3d(st + K_BYTES / 2, &tmK, &kv_full[s], 64, kvh, row);
+        if (TWO) tma_load_3d(st + K_BYTES / 2, &tmK, &kv_full[s], 64, kvh, row);
         tma_load_3d(st + K_BYTES, &tmV, &kv_full[s], 0, kvh, row);
-        tma_load_3d(st + K_BYTES + V_BYTES / 2, &tmV, &kv_full[s], 64, kvh, row);
+        if (TWO) tma_load_3d(st + K_BYTES + V_BYTES / 2, &tmV, &kv_full[s], 64, kvh, row);
         issued = j + 1;
       }
       if (!ok) {
@@ -327,12 +331,27 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       const bool store = row < q_len;
       const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
       __nv_bfloat16* dst = a.out + (size_t)(q_start + row) * a.o_stride + (size_t)head * a.hd;
+      const __nv_bfloat16* gate = a.gate ? a.gate + (size_t)(q_start + row) * a.gate_stride + (size_t)head * a.hd : nullptr;
       for (int c = c_begin; c < c_end; ++c) {
         uint32_t r[16];
         tmem_ld16(lane_addr + TMEM_O + c * 16, r);
         tmem_ld_wait();
         uint4 v[2];
         uint32_t* w = reinterpret_cast<uint32_t*>(v);
+        if (gate != nullptr && store) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            if (c * 16 + 8 * e + 8 > a.hd) continue;
+            const uint4 g4 = *reinterpret_cast<const uint4*>(gate + c * 16 + 8 * e);
+            const __nv_bfloat162* gp = reinterpret_cast<const __nv_bfloat162*>(&g4);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float2 g = __bfloat1622float2(gp[i]);
+              r[8 * e + 2 * i] = __float_as_uint(__uint_as_float(r[8 * e + 2 * i]) * g.x);
+              r[8 * e + 2 * i + 1] = __float_as_uint(__uint_as_float(r[8 * e + 2 * i + 1]) * g.y);
+            }
+          }
+        }
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(r[2 * e]) * inv, __uint_as_float(r[2 * e + 1]) * inv);
@@ -432,14 +451,16 @@ __global__ void __launch_bounds__(GATHER_ROWS * 32) gather_pages_kernel(const Ga
 // QKV projection are fine); out [T][o_stride].  Rows and strides must be 16-byte aligned.
 static int flash_tc_impl(const void* q, long long q_stride, const void* k, const void* v, long long kv_stride, void* out,
                          long long o_stride, const void* cu_q, const void* cu_kv, int T, int Tkv, int S, int max_q_len,
-                         int Hq, int Hkv, int hd, int causal, float scale, void* stream, int pdl) {
+                         int Hq, int Hkv, int hd, int causal, float scale, void* stream, int pdl,
+                         const void* gate = nullptr, long long gate_stride = 0) {
   if (S <= 0 || max_q_len <= 0 || T <= 0 || Tkv <= 0) return 0;
   if (Hq % Hkv) return -1;
   if ((q_stride % 8) || (kv_stride % 8) || (o_stride % 8)) return -2;
   if ((reinterpret_cast<unsigned long long>(q) | reinterpret_cast<unsigned long long>(k) |
        reinterpret_cast<unsigned long long>(v) | reinterpret_cast<unsigned long long>(out)) & 15ull)
     return -3;
-  if (hd != 128 && hd != 72) return -4;
+  if (hd < 8 || hd > FA_HD || hd % 8) return -4;
+  if (gate != nullptr && ((gate_stride % 8) || (reinterpret_cast<unsigned long long>(gate) & 15ull))) return -3;
   CUtensorMap tq, tk, tv;
   int rc = prism_make_head_tensor_map(q, (unsigned long long)T, (unsigned)Hq, (unsigned)hd, (unsigned long long)q_stride, FA_BM, &tq);
   if (rc) return rc;
@@ -457,17 +478,22 @@ static int flash_tc_impl(const void* q, long long q_stride, const void* k, const
   a.hd = hd;
   a.causal = causal;
   a.scale = scale;
+  a.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  a.gate_stride = gate_stride;
   const size_t smem = 1024 + Q_BYTES + (size_t)FA_STAGES * STAGE_BYTES + 32 * 8 + 64 + 6 * FA_BM * sizeof(float);
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(flash_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(flash_tc_kernel<80>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   const int tiles = (max_q_len + FA_BM - 1) / FA_BM;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  if (hd == 128)
+  if (hd <= 64)
+    return (int)prism_launch(flash_tc_kernel<64>, dim3(tiles, Hq, S), dim3(FA_THREADS), smem, st, pdl != 0, tq, tk, tv, a);
+  if (hd > 80)
     return (int)prism_launch(flash_tc_kernel<128>, dim3(tiles, Hq, S), dim3(FA_THREADS), smem, st, pdl != 0, tq, tk, tv, a);
   return (int)prism_launch(flash_tc_kernel<80>, dim3(tiles, Hq, S), dim3(FA_THREADS), smem, st, pdl != 0, tq, tk, tv, a);
 }
@@ -478,6 +504,17 @@ PRISM_API int prism_flash_attention_tc(const void* q, long long q_stride, const 
                                        void* stream, int pdl) {
   return flash_tc_impl(q, q_stride, k, v, kv_stride, out, o_stride, cu_q, nullptr, T, T, S, max_q_len, Hq, Hkv, hd, causal,
                        scale, stream, pdl);
+}
+
+// Causal attention of new tokens over contiguous key / value rows with their own ranges (cu_kv; null: the
+// query rows' own), an optional element-wise output gate and any head dimension up to 128 that is a multiple of 8.
+PRISM_API int prism_flash_attention_tc_kv(const void* q, long long q_stride, const void* k, const void* v, long long kv_stride,
+                                          void* out, long long o_stride, const void* cu_q, const void* cu_kv, const void* gate,
+                                          long long gate_stride, int T, int Tkv, int S, int max_q_len, int Hq, int Hkv, int hd,
+                                          float scale, void* stream, int pdl) {
+  if (Hq <= 0 || Hkv <= 0) return -1;
+  return flash_tc_impl(q, q_stride, k, v, kv_stride, out, o_stride, cu_q, cu_kv, T, Tkv, S, max_q_len, Hq, Hkv, hd, 1, scale,
+                       stream, pdl, gate, gate_stride);
 }
 
 // Causal attention of new tokens over the paged cache, head dimension 128: the keys each sequence

@@ -78,6 +78,47 @@ __device__ __forceinline__ float gelu_erf(float x) {
 }
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
 
+__device__ __forceinline__ float sigmoid_fast(float x) { return 1.0f / (1.0f + __expf(-x)); }
+
+// ---- row sections of a stacked projection -------------------------------------------
+// One GEMM over several weight matrices stacked by rows: rows [row_end[i - 1], row_end[i]) are
+// scaled by alpha[i] (then the bias is added) and pass through activation act[i].
+enum PrismAct : int { PRISM_ACT_NONE = 0, PRISM_ACT_GELU_TANH = 1, PRISM_ACT_GELU_ERF = 2, PRISM_ACT_SIGMOID = 3, PRISM_ACT_SOFTCAP = 4 };
+constexpr int PRISM_MAX_SECTIONS = 8;
+struct PrismSections {
+  int n;      // 0: no sections
+  float cap;  // bound of the PRISM_ACT_SOFTCAP sections: cap * tanh(v / cap)
+  int row_end[PRISM_MAX_SECTIONS];
+  int act[PRISM_MAX_SECTIONS];
+  float alpha[PRISM_MAX_SECTIONS];
+};
+// Section of row m (rows past the last end belong to the last section).
+__device__ __forceinline__ void prism_section_of(const PrismSections& s, int m, float& alpha, int& act) {
+  alpha = s.alpha[0];
+  act = s.act[0];
+#pragma unroll
+  for (int i = 1; i < PRISM_MAX_SECTIONS; ++i)
+    if (i < s.n && m >= s.row_end[i - 1]) {
+      alpha = s.alpha[i];
+      act = s.act[i];
+    }
+}
+// Copies host arrays into the kernel argument; false when they are not a valid partition of M rows.
+static inline bool prism_fill_sections(PrismSections& s, int n, const int* row_end, const float* alpha, const int* act, float cap,
+                                       int M) {
+  if (n < 1 || n > PRISM_MAX_SECTIONS) return false;
+  s.n = n;
+  s.cap = cap;
+  for (int i = 0; i < PRISM_MAX_SECTIONS; ++i) {
+    s.row_end[i] = i < n ? row_end[i] : M;
+    s.alpha[i] = i < n ? alpha[i] : 1.0f;
+    s.act[i] = i < n ? act[i] : 0;
+    if (i < n && ((i > 0 && row_end[i] <= row_end[i - 1]) || act[i] < 0 || act[i] > PRISM_ACT_SOFTCAP)) return false;
+    if (i < n && act[i] == PRISM_ACT_SOFTCAP && !(cap > 0.0f)) return false;
+  }
+  return row_end[n - 1] == M;
+}
+
 // ---- programmatic dependent launch -------------------------------------------------
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_launch_dependents() {

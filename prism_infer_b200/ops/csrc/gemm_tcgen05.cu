@@ -17,6 +17,9 @@
 // (prism_infer/ops/csrc/cutlass_dual_gemm_swiglu.cu:85-215, mma.sync Sm80) and every
 // F.linear of prism_infer/layers/linear.py:62-190.
 //
+// Stacked projections (several weight matrices over the same activations, each with its own scale and
+// activation) run as one launch: PrismSections (common.cuh) names the row ranges.
+//
 // Programmatic dependent launch: the producer thread prefetches the first ring of weight
 // tiles (which never depend on the previous kernel) before griddepcontrol.wait, then
 // loads activations.
@@ -63,7 +66,19 @@ struct GemmArgs {
   const unsigned long long* epoch;  // local device word: sequence base of the current step (null: 0)
   float* peer_out[8];        // slab buffers (or bf16 row buffers) of this slot on every rank (incl. own)
   unsigned long long* peer_flag[8];  // flag arrays [tp] of this slot on every rank
+  PrismSections sec;         // stacked projections: scale and activation by row range (n = 0: off)
 };
+
+// One activation in 32-bit, chosen at run time (uniform over a warp for stacked projections).
+__device__ __forceinline__ float apply_act(float v, int act, float cap) {
+  switch (act) {
+    case PRISM_ACT_GELU_TANH: return gelu_tanh(v);
+    case PRISM_ACT_GELU_ERF: return gelu_erf(v);
+    case PRISM_ACT_SIGMOID: return sigmoid_fast(v);
+    case PRISM_ACT_SOFTCAP: return cap * tanhf(v / cap);
+    default: return v;
+  }
+}
 
 template <int BN, bool DUAL>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
@@ -191,9 +206,15 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       __nv_bfloat16* out_b = reinterpret_cast<__nv_bfloat16*>(a.out);
       // One compact store loop per output form; the form is chosen once, outside the column
       // loops, so the instruction stream of a tile touches only the code it needs.
-      enum { EPI_BF16_PLAIN, EPI_BF16_FULL, EPI_F32, EPI_PUSH_F32, EPI_PUSH_ROWS, EPI_DUAL };
+      enum { EPI_BF16_PLAIN, EPI_BF16_FULL, EPI_F32, EPI_PUSH_F32, EPI_PUSH_ROWS, EPI_SECTIONS, EPI_DUAL };
       int mode;
+      float sec_alpha = 1.0f;
+      int sec_act = 0;
       if (DUAL) mode = EPI_DUAL;
+      else if (a.sec.n > 0) {
+        mode = EPI_SECTIONS;
+        prism_section_of(a.sec, m, sec_alpha, sec_act);
+      }
       else if (a.n_peers > 0) mode = a.push_rows ? EPI_PUSH_ROWS : EPI_PUSH_F32;
       else if (a.out_f32) mode = EPI_F32;
       else mode = (a.bias == nullptr && a.act == 0 && a.residual == nullptr) ? EPI_BF16_PLAIN : EPI_BF16_FULL;
@@ -282,6 +303,23 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             }
             break;
           }
+          case EPI_SECTIONS: {
+            float v[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = apply_act(__uint_as_float(r[j]) * sec_alpha + bias_v, sec_act, a.sec.cap);
+            if (a.out_f32) {
+              float* dst = out_f + row0 * a.ldo + m;
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                if (j < cols) dst[(size_t)j * a.ldo] = v[j];
+            } else {
+              __nv_bfloat16* dst = out_b + row0 * a.ldo + m;
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                if (j < cols) dst[(size_t)j * a.ldo] = __float2bfloat16_rn(v[j]);
+            }
+            break;
+          }
           default: {  // EPI_DUAL: silu(gate) -> bf16, * up -> bf16 (rounding points of the eager graph)
             __nv_bfloat16* dst = out_b + row0 * a.ldo + m;
 #pragma unroll
@@ -349,6 +387,7 @@ struct PersistArgs {
   int* cta_counter;
   __nv_bfloat16* peer_out[8];
   unsigned long long* peer_flag[8];
+  PrismSections sec;  // row-major form only; row ends are multiples of 16 (a chunk lies in one section)
 };
 
 // ROWMAJOR: the A operand (128-row tiles, TMEM lanes) holds the tokens and B the weights, so an
@@ -536,6 +575,13 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
           float v[16];
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]);
+          int act = a.act;
+          if (a.sec.n > 0) {
+            float alpha;
+            prism_section_of(a.sec, f0, alpha, act);
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] *= alpha;
+          }
           if (a.bias != nullptr) {
             const uint4 b0 = *reinterpret_cast<const uint4*>(a.bias + f0), b1 = *reinterpret_cast<const uint4*>(a.bias + f0 + 8);
             const __nv_bfloat162* p0 = reinterpret_cast<const __nv_bfloat162*>(&b0);
@@ -549,12 +595,15 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
               v[8 + 2 * e + 1] += x1.y;
             }
           }
-          if (a.act == 1) {
+          if (act == PRISM_ACT_GELU_TANH) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gelu_tanh(v[j]);
-          } else if (a.act == 2) {
+          } else if (act == PRISM_ACT_GELU_ERF) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gelu_erf(v[j]);
+          } else if (act == PRISM_ACT_SIGMOID) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = sigmoid_fast(v[j]);
           }
           if (a.residual != nullptr) {
             const __nv_bfloat16* rs = a.residual + (size_t)m * a.ldr + f0;
@@ -828,7 +877,8 @@ struct PushSpec {
 static int gemm_wx_impl(const void* W, const void* X, void* out, int M, int T, int K, long long ldw, long long ldx,
                         long long ldo, int w_rows_total, const void* bias, const void* residual, long long ldr, int act,
                         int dual, int w2_row_off, int splits, int out_f32, long long split_stride, int bn_override,
-                        int stages_override, void* stream_ptr, int pdl, const PushSpec* push) {
+                        int stages_override, void* stream_ptr, int pdl, const PushSpec* push,
+                        const PrismSections* sections = nullptr) {
   if (M <= 0 || T <= 0 || K <= 0) return -1;
   if (K % 8) return -2;  // 16-byte row pitch for TMA
   if (dual && (splits > 1 || out_f32)) return -3;
@@ -859,6 +909,14 @@ static int gemm_wx_impl(const void* W, const void* X, void* out, int M, int T, i
   a.tokens_fastest = ((long long)w_rows_total * K * 2 > (100ll << 20) || (M + BM - 1) / BM > 65535) ? 1 : 0;
   a.out_f32 = out_f32;
   a.act = act;
+  a.sec.n = 0;
+  bool sections_rowmajor = true;  // the persistent row-major epilogue can serve them
+  if (sections != nullptr) {
+    if (dual || splits > 1 || push != nullptr || residual != nullptr || act != 0) return -8;
+    a.sec = *sections;
+    for (int i = 0; i < a.sec.n; ++i)
+      if (a.sec.row_end[i] % 16 || a.sec.act[i] == PRISM_ACT_SOFTCAP) sections_rowmajor = false;
+  }
   a.ldo = ldo;
   a.ldr = ldr;
   a.split_stride = split_stride;
@@ -897,8 +955,11 @@ static int gemm_wx_impl(const void* W, const void* X, void* out, int M, int T, i
   const int m_tiles = (M + BM - 1) / BM;
   const bool p = pdl != 0;
   if (g_persistent_min_tokens > 0 && T >= g_persistent_min_tokens && splits == 1 && !out_f32 && push == nullptr &&
-      bn_override <= 0 && stages_override <= 0) {
+      bn_override <= 0 && stages_override <= 0 &&
+      (sections == nullptr || (sections_rowmajor && g_persistent_rowmajor && M % 16 == 0 && ldo % 8 == 0 &&
+                               ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0))) {
     PersistArgs pa;
+    pa.sec = a.sec;
     pa.M = M;
     pa.T = T;
     pa.kb_total = a.kb_total;
@@ -993,6 +1054,18 @@ PRISM_API int prism_gemm_wx(const void* W, const void* X, void* out, int M, int 
                       out_f32, split_stride, bn_override, stages_override, stream_ptr, pdl, nullptr);
 }
 
+// Stacked projection: out[t][m] = act_i(alpha_i * (W x_t)[m] + bias[m]) for the section i that row m lies in
+// (row_end / alpha / act: host arrays of n_sections entries); bf16 or fp32 output.
+PRISM_API int prism_gemm_wx_sections(const void* W, const void* X, void* out, int M, int T, int K, long long ldw,
+                                     long long ldx, long long ldo, const void* bias, int n_sections, const void* row_end,
+                                     const void* alpha, const void* act, float cap, int out_f32, int bn_override,
+                                     int stages_override, void* stream_ptr, int pdl) {
+  PrismSections sec;
+  if (!prism_fill_sections(sec, n_sections, (const int*)row_end, (const float*)alpha, (const int*)act, cap, M)) return -9;
+  return gemm_wx_impl(W, X, out, M, T, K, ldw, ldx, ldo, M, bias, nullptr, 0, 0, 0, 0, 1, out_f32, 0, bn_override,
+                      stages_override, stream_ptr, pdl, nullptr, &sec);
+}
+
 // Fused row-parallel GEMM -> one-shot exchange: the fp32 partial of rank `my_rank`, split s,
 // lands in slab (my_rank * splits + s) of every rank's buffer (peer_out[p], p < n_peers, own
 // rank included; row stride ldo, slab stride split_stride, both in 8-byte elements).  Every
@@ -1066,6 +1139,7 @@ PRISM_API int prism_gemm_wx_scatter(const void* W, const void* X, int M, int T, 
   rc = get_tensor_map(W, (unsigned long long)M, (unsigned long long)K, (unsigned long long)ldw, 256, &tb);
   if (rc) return rc;
   PersistArgs pa;
+  pa.sec.n = 0;
   pa.dual_rm = 0;
   pa.M = T;
   pa.T = M;

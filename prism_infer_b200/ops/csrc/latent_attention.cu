@@ -1,0 +1,751 @@
+// Latent attention: every head's keys and values are linear in one shared latent row c per token,
+// k_h = U_h c and v_h = V_h c, and only c is cached (one row per token and layer run, paged).
+//
+// Absorbed form (decode steps, short portions of a prompt): with q~_h = U_h^T q_h the score is q~_h . c and the
+// head's output V_h (sum_j p_j c_j), so attention runs over the latents themselves, all heads of a token sharing
+// every latent row it reads.
+//   latent_absorb_kernel     q~ for every (token, head), and, from extra CTAs of the same launch, the RMS-normalised
+//                            latent of every new token written to its page
+//   latent_attention_kernel  16 or 32 (token, head) rows against tiles of 64 latents (32 above 512 elements), the
+//                            key range split over CTAs; mma.sync, scores and softmax in 32-bit
+//   latent_out_kernel        merges the splits, multiplies by V_h and by the output gate
+// Expanded form (whole prompts): the visible latents are gathered from their pages (gather_latents_kernel), one
+// GEMM makes keys and values of all heads, and the tcgen05 kernel of attention_tcgen05.cu attends over them.
+// The *_f32 kernels are the absorbed form in true 32-bit.
+//
+// Latent rows are padded with zeros to Rc elements (a multiple of 64), heads to dq / dv elements (multiples of 8).
+#include "mma_sync.cuh"
+
+PRISM_DEFINE_TU_STATUS(latent)
+
+namespace {
+
+typedef __nv_bfloat16 bf16;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T from_f(float v);
+template <>
+__device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
+
+// -------------------------------------------------------------------------------------------------
+// RMS norm of the projected latent and its store: one warp per token.
+// -------------------------------------------------------------------------------------------------
+template <typename T>
+struct NormStoreArgs {
+  const T* raw;            // [tokens][ld_raw]
+  long long ld_raw;
+  const T* weight;         // [R]
+  T* cache;                // [blocks][page][Rc]
+  const long long* slots;  // [tokens] flat slot, < 0: not stored
+  long long num_slots;
+  T* rows;                 // [tokens][Rc] contiguous copy (null: none)
+  int tokens, R, Rc;
+  float eps;
+};
+
+template <typename T>
+__device__ __forceinline__ void norm_store_token(const NormStoreArgs<T>& a, int t, int lane) {
+  const T* src = a.raw + (size_t)t * a.ld_raw;
+  float ss = 0.0f;
+  for (int i = lane; i < a.R; i += 32) {
+    const float v = to_f(src[i]);
+    ss += v * v;
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.R + a.eps);
+  long long slot = a.slots[t];
+  if (slot >= a.num_slots) {
+    if (lane == 0) prism_report(PRISM_ERR_BOUNDS, 3);
+    slot = -1;
+  }
+  T* page_row = slot >= 0 ? a.cache + (size_t)slot * a.Rc : nullptr;
+  T* row = a.rows ? a.rows + (size_t)t * a.Rc : nullptr;
+  for (int i = lane; i < a.Rc; i += 32) {
+    const T v = i < a.R ? from_f<T>(to_f(src[i]) * inv * to_f(a.weight[i])) : from_f<T>(0.0f);
+    if (page_row) page_row[i] = v;
+    if (row) row[i] = v;
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) latent_norm_store_kernel(const NormStoreArgs<T> a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (t < a.tokens) norm_store_token(a, t, threadIdx.x & 31);
+}
+
+// -------------------------------------------------------------------------------------------------
+// q~ = U_h^T q_h for a tile of 16 tokens, one head and 128 latent elements per CTA.  The CTAs with
+// blockIdx.y == H run the norm and store instead (those with blockIdx.x == 0; the others end).
+// -------------------------------------------------------------------------------------------------
+constexpr int ABS_N = 128, ABS_LDW = ABS_N + 8;
+
+struct AbsorbArgs {
+  const bf16* q;           // [tokens][ldq], head h at column h * dq
+  long long ldq;
+  const bf16* uk;          // [H * dq][Rc]
+  bf16* out;               // [tokens][H][Rc]
+  int H, dq, dk16;         // dk16: dq rounded up to 16
+  NormStoreArgs<bf16> ns;
+};
+
+__global__ void __launch_bounds__(128) latent_absorb_kernel(const AbsorbArgs a) {
+  extern __shared__ uint8_t smem_raw[];
+  bf16* w_s = reinterpret_cast<bf16*>(smem_raw);          // [dk16][ABS_LDW]
+  bf16* q_s = w_s + (size_t)a.dk16 * ABS_LDW;             // [16][dk16 + 8]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t0 = blockIdx.z * 16, Rc = a.ns.Rc;
+  pdl_launch_dependents();
+  if ((int)blockIdx.y == a.H) {
+    pdl_wait();
+    if (blockIdx.x == 0)
+      for (int t = t0 + warp; t < min(t0 + 16, a.ns.tokens); t += 4) norm_store_token(a.ns, t, lane);
+    return;
+  }
+  const int h = blockIdx.y, n0 = blockIdx.x * ABS_N, ldq_s = a.dk16 + 8;
+  for (int i = threadIdx.x; i < a.dk16 * (ABS_N / 8); i += 128) {  // weights do not depend on the previous kernel
+    const int k = i / (ABS_N / 8), c = (i % (ABS_N / 8)) * 8;
+    const bool ok = k < a.dq && n0 + c < Rc;
+    cp_async16(w_s + k * ABS_LDW + c, ok ? a.uk + ((size_t)h * a.dq + k) * Rc + n0 + c : a.uk, ok);
+  }
+  pdl_wait();
+  for (int i = threadIdx.x; i < 16 * (a.dk16 / 8); i += 128) {
+    const int r = i / (a.dk16 / 8), c = (i % (a.dk16 / 8)) * 8;
+    const bool ok = t0 + r < a.ns.tokens && c < a.dq;
+    cp_async16(q_s + r * ldq_s + c, ok ? a.q + (size_t)(t0 + r) * a.ldq + (size_t)h * a.dq + c : a.q, ok);
+  }
+  cp_async_commit();
+  cp_async_wait_all();
+  __syncthreads();
+  float acc[4][4] = {};
+  for (int kk = 0; kk < a.dk16; kk += 16) {
+    uint32_t qf[4];
+    ldsm_x4(qf, smem_u32(q_s + (lane & 15) * ldq_s + kk + 8 * (lane >> 4)));
+#pragma unroll
+    for (int np = 0; np < 2; ++np) {
+      uint32_t wb[4];
+      ldsm_x4_t(wb, smem_u32(w_s + (kk + (lane & 15)) * ABS_LDW + warp * 32 + np * 16 + 8 * (lane >> 4)));
+      mma_bf16(acc[2 * np], qf, wb[0], wb[1]);
+      mma_bf16(acc[2 * np + 1], qf, wb[2], wb[3]);
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < 4; ++n) {
+    const int col = n0 + warp * 32 + n * 8 + 2 * (lane & 3);
+    if (col >= Rc) continue;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int t = t0 + (lane >> 2) + 8 * half;
+      if (t < a.ns.tokens)
+        *reinterpret_cast<uint32_t*>(a.out + ((size_t)t * a.H + h) * Rc + col) = pack_bf16(acc[n][2 * half], acc[n][2 * half + 1]);
+    }
+  }
+}
+
+// -------------------------------------------------------------------------------------------------
+// Attention of (token, head) rows over paged latents.
+// -------------------------------------------------------------------------------------------------
+struct LatentAttnArgs {
+  const bf16* q;            // [tokens][H][Rc]
+  const bf16* cache;        // [blocks][page][Rc]
+  const int* block_tables;  // [S][max_blocks], < 0: hole
+  const int* cu_q;          // [S + 1] token offsets; null: sequence s is token s
+  const int* kv_lens;       // [S] visible latents of the sequence's last token
+  float* part_o;            // [tokens * H][nsplit][Rc]  (nsplit > 1)
+  float* part_ml;           // [tokens * H][nsplit][2]   maximum (base 2, scaled) and sum
+  bf16* out;                // [tokens * H][Rc] normalised (nsplit == 1)
+  int H, Rc, page, max_blocks, num_blocks, nsplit;
+  float scale;
+};
+
+template <int MT, int NT, int BN>
+__global__ void __launch_bounds__(256) latent_attention_kernel(const LatentAttnArgs a) {
+  constexpr int BM = 16 * MT;
+  constexpr int LDS = BN + 4, LDP = BN + 8;
+  extern __shared__ uint8_t smem_raw[];
+  const int Rc = a.Rc, LD = Rc + 8, nt = Rc >> 6;         // nt: 8-column tiles of the output per warp
+  bf16* q_s = reinterpret_cast<bf16*>(smem_raw);           // [BM][LD]
+  bf16* kv_s = q_s + (size_t)BM * LD;                      // [2][BN][LD]
+  float* s_s = reinterpret_cast<float*>(kv_s + (size_t)2 * BN * LD);  // [BM][LDS]
+  bf16* p_s = reinterpret_cast<bf16*>(s_s + BM * LDS);     // [BM][LDP]
+  float* fac_s = reinterpret_cast<float*>(p_s + BM * LDP); // [BM] rescale of the accumulator
+  float* m_s = fac_s + BM;                                 // [BM] running maximum
+  float* l_s = m_s + BM;                                   // [BM] running sum
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int seq = blockIdx.z, split = blockIdx.y;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int q_start = a.cu_q ? a.cu_q[seq] : seq;
+  const int q_len = a.cu_q ? a.cu_q[seq + 1] - q_start : 1;
+  const int n_rows = q_len * a.H, row0 = blockIdx.x * BM;
+  if (row0 >= n_rows) return;                              // uniform over the CTA
+  const int kv_len = clamp_context(a.kv_lens[seq], a.max_blocks, a.page);
+  const int last_t = min(row0 + BM, n_rows) - 1;
+  const int kv_end = max(0, min(kv_len, kv_len - q_len + last_t / a.H + 1));
+  const int tiles = (kv_end + BN - 1) / BN, per = (tiles + a.nsplit - 1) / a.nsplit;
+  const int tb = split * per, te = min(tiles, tb + per);
+  const size_t out_row0 = (size_t)q_start * a.H + row0;
+  const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
+  const int pieces = Rc >> 3;
+
+  auto load_tile = [&](int j, int stage) {
+    bf16* dst = kv_s + (size_t)stage * BN * LD;
+    for (int i = threadIdx.x; i < BN * pieces; i += 256) {
+      const int r = i / pieces, c = (i - r * pieces) * 8, key = j * BN + r;
+      int blk = key < kv_end ? bt[key / a.page] : -1;
+      blk = checked_page(blk, a.num_blocks);
+      const bool ok = blk >= 0;
+      cp_async16(dst + r * LD + c, ok ? a.cache + ((size_t)blk * a.page + key % a.page) * Rc + c : a.cache, ok);
+    }
+  };
+
+  for (int i = threadIdx.x; i < BM * pieces; i += 256) {
+    const int r = i / pieces, c = (i - r * pieces) * 8;
+    const bool ok = row0 + r < n_rows;
+    cp_async16(q_s + r * LD + c, ok ? a.q + (out_row0 + r) * Rc + c : a.q, ok);
+  }
+  if (tb < te) load_tile(tb, 0);
+  cp_async_commit();
+  for (int i = threadIdx.x; i < BM; i += 256) {
+    m_s[i] = -INFINITY;
+    l_s[i] = 0.0f;
+  }
+  float acc[MT][NT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < NT; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.0f;
+  const float sl2 = a.scale * 1.4426950408889634f;
+
+  for (int j = tb; j < te; ++j) {
+    const int stage = (j - tb) & 1;
+    cp_async_wait<0>();
+    __syncthreads();                 // tile j is in; every warp is done with tile j - 1
+    if (j + 1 < te) load_tile(j + 1, stage ^ 1);
+    cp_async_commit();
+    const bf16* kv = kv_s + (size_t)stage * BN * LD;
+    if (warp < BN / 8) {             // scores of keys 8 warp .. 8 warp + 7
+      float s[MT][4] = {};
+      for (int kk = 0; kk < Rc; kk += 32) {
+        uint32_t kb[4];
+        ldsm_x4(kb, smem_u32(kv + (warp * 8 + (lane & 7)) * LD + kk + 8 * (lane >> 3)));
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          uint32_t q0[4], q1[4];
+          const bf16* qp = q_s + (m * 16 + (lane & 15)) * LD + kk + 8 * (lane >> 4);
+          ldsm_x4(q0, smem_u32(qp));
+          ldsm_x4(q1, smem_u32(qp + 16));
+          mma_bf16(s[m], q0, kb[0], kb[1]);
+          mma_bf16(s[m], q1, kb[2], kb[3]);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        float* d = s_s + (m * 16 + (lane >> 2)) * LDS + warp * 8 + 2 * (lane & 3);
+        d[0] = s[m][0];
+        d[1] = s[m][1];
+        d[8 * LDS] = s[m][2];
+        d[8 * LDS + 1] = s[m][3];
+      }
+    }
+    __syncthreads();
+    // online softmax, BM / 8 rows per warp
+#pragma unroll
+    for (int i = 0; i < BM / 8; ++i) {
+      const int r = warp * (BM / 8) + i, row = row0 + r;
+      const int limit = row < n_rows ? kv_len - q_len + row / a.H + 1 : 0;
+      float v[BN / 32], mx = -INFINITY;
+#pragma unroll
+      for (int e = 0; e < BN / 32; ++e) {
+        const int c = lane + 32 * e;
+        v[e] = j * BN + c < limit ? s_s[r * LDS + c] * sl2 : -INFINITY;
+        mx = fmaxf(mx, v[e]);
+      }
+      mx = warp_max(mx);
+      const float m_old = m_s[r], m_new = fmaxf(m_old, mx);
+      const float m_use = m_new == -INFINITY ? 0.0f : m_new;
+      float sum = 0.0f;
+#pragma unroll
+      for (int e = 0; e < BN / 32; ++e) {
+        const float p = ex2_fast(v[e] - m_use);
+        sum += p;
+        p_s[r * LDP + lane + 32 * e] = __float2bfloat16_rn(p);
+      }
+      sum = warp_sum(sum);
+      __syncwarp();
+      if (lane == 0) {
+        const float f = ex2_fast(m_old - m_use);  // 0 while nothing has been seen
+        fac_s[r] = f;
+        m_s[r] = m_new;
+        l_s[r] = l_s[r] * f + sum;
+      }
+    }
+    __syncthreads();
+    // accumulate P C, columns warp * Rc / 8 ..
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float f0 = fac_s[m * 16 + (lane >> 2)], f1 = fac_s[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        acc[m][n][0] *= f0;
+        acc[m][n][1] *= f0;
+        acc[m][n][2] *= f1;
+        acc[m][n][3] *= f1;
+      }
+    }
+    const int col0 = warp * nt * 8;
+#pragma unroll
+    for (int kk = 0; kk < BN; kk += 16) {
+      uint32_t pf[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) ldsm_x4(pf[m], smem_u32(p_s + (m * 16 + (lane & 15)) * LDP + kk + 8 * (lane >> 4)));
+      const bf16* vrow = kv + (kk + (lane & 15)) * LD + col0 + 8 * (lane >> 4);
+#pragma unroll
+      for (int n = 0; n < NT; n += 2) {
+        if (n < nt) {                // a last odd tile loads its neighbour (or the row's padding) and ignores it
+          uint32_t vb[4];
+          ldsm_x4_t(vb, smem_u32(vrow + n * 8));
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            mma_bf16(acc[m][n], pf[m], vb[0], vb[1]);
+            if (n + 1 < nt) mma_bf16(acc[m][n + 1], pf[m], vb[2], vb[3]);
+          }
+        }
+      }
+    }
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  if (a.nsplit > 1 && (int)threadIdx.x < BM && row0 + (int)threadIdx.x < n_rows) {
+    float* ml = a.part_ml + ((out_row0 + threadIdx.x) * a.nsplit + split) * 2;
+    ml[0] = m_s[threadIdx.x];
+    ml[1] = l_s[threadIdx.x];
+    if (tb >= te) ml[1] = 0.0f;
+  }
+  if (a.nsplit > 1 && tb >= te) return;  // an empty split has no partial rows
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = m * 16 + (lane >> 2) + 8 * half;
+      if (row0 + r >= n_rows) continue;
+      const float l = l_s[r], inv = a.nsplit > 1 ? 1.0f : (l > 0.0f ? 1.0f / l : 0.0f);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        if (n >= nt) continue;
+        const int col = warp * nt * 8 + n * 8 + 2 * (lane & 3);
+        const float v0 = acc[m][n][2 * half] * inv, v1 = acc[m][n][2 * half + 1] * inv;
+        if (a.nsplit > 1)
+          *reinterpret_cast<float2*>(a.part_o + ((out_row0 + r) * a.nsplit + split) * Rc + col) = make_float2(v0, v1);
+        else
+          *reinterpret_cast<uint32_t*>(a.out + (out_row0 + r) * Rc + col) = pack_bf16(v0, v1);
+      }
+    }
+}
+
+// -------------------------------------------------------------------------------------------------
+// o_h = gate * V_h (merged latent output): a tile of 16 tokens, one head, 64 output elements per CTA.
+// -------------------------------------------------------------------------------------------------
+constexpr int OUT_N = 64, MAX_SPLITS = 32;
+
+struct LatentOutArgs {
+  const float* part_o;
+  const float* part_ml;
+  const bf16* lat;         // [tokens * H][Rc] (nsplit == 1)
+  const bf16* uv;          // [H * dv][Rc]
+  const bf16* gate;        // [tokens][gate_ld], head h at column h * dv (null: one)
+  long long gate_ld;
+  bf16* out;               // [tokens][ld_out]
+  long long ld_out;
+  int tokens, H, dv, Rc, nsplit;
+};
+
+__global__ void __launch_bounds__(128) latent_out_kernel(const LatentOutArgs a) {
+  extern __shared__ uint8_t smem_raw[];
+  const int Rc = a.Rc, LD = Rc + 8, pieces = Rc >> 3;
+  bf16* w_s = reinterpret_cast<bf16*>(smem_raw);   // [OUT_N][LD]
+  bf16* a_s = w_s + (size_t)OUT_N * LD;            // [16][LD]
+  __shared__ float wgt[16][MAX_SPLITS];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n0 = blockIdx.x * OUT_N, h = blockIdx.y, t0 = blockIdx.z * 16;
+  pdl_launch_dependents();
+  for (int i = threadIdx.x; i < OUT_N * pieces; i += 128) {
+    const int r = i / pieces, c = (i - r * pieces) * 8;
+    const bool ok = n0 + r < a.dv;
+    cp_async16(w_s + r * LD + c, ok ? a.uv + ((size_t)h * a.dv + n0 + r) * Rc + c : a.uv, ok);
+  }
+  cp_async_commit();
+  pdl_wait();
+  const int rows = min(16, a.tokens - t0);
+  if (a.nsplit > 1) {
+    for (int r = warp; r < rows; r += 4) {         // weights of the splits: 2^(m_s - m) / l
+      const size_t row = (size_t)(t0 + r) * a.H + h;
+      float m = -INFINITY, l = 0.0f;
+      if (lane < a.nsplit) {
+        m = a.part_ml[(row * a.nsplit + lane) * 2];
+        l = a.part_ml[(row * a.nsplit + lane) * 2 + 1];
+      }
+      const float mx = warp_max(l > 0.0f ? m : -INFINITY);
+      const float f = l > 0.0f ? ex2_fast(m - mx) : 0.0f;
+      const float sum = warp_sum(f * l);
+      if (lane < a.nsplit) wgt[r][lane] = sum > 0.0f ? f / sum : 0.0f;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < 16 * (Rc >> 2); i += 128) {
+      const int r = i / (Rc >> 2), c = (i - r * (Rc >> 2)) * 4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r < rows) {
+        const float* src = a.part_o + ((size_t)(t0 + r) * a.H + h) * a.nsplit * Rc + c;
+#pragma unroll 4
+        for (int s = 0; s < a.nsplit; ++s) {
+          const float w = wgt[r][s];
+          if (w == 0.0f) continue;                 // an empty split's rows were never written
+          const float4 p = __ldcg(reinterpret_cast<const float4*>(src + (size_t)s * Rc));
+          v.x += w * p.x;
+          v.y += w * p.y;
+          v.z += w * p.z;
+          v.w += w * p.w;
+        }
+      }
+      uint2 o;
+      o.x = pack_bf16(v.x, v.y);
+      o.y = pack_bf16(v.z, v.w);
+      *reinterpret_cast<uint2*>(a_s + r * LD + c) = o;
+    }
+  } else {
+    for (int i = threadIdx.x; i < 16 * pieces; i += 128) {
+      const int r = i / pieces, c = (i - r * pieces) * 8;
+      const bool ok = r < rows;
+      cp_async16(a_s + r * LD + c, ok ? a.lat + ((size_t)(t0 + r) * a.H + h) * Rc + c : a.lat, ok);
+    }
+    cp_async_commit();
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  float acc[2][4] = {};
+  for (int kk = 0; kk < Rc; kk += 16) {
+    uint32_t af[4], wb[4];
+    ldsm_x4(af, smem_u32(a_s + (lane & 15) * LD + kk + 8 * (lane >> 4)));
+    ldsm_x4(wb, smem_u32(w_s + (warp * 16 + (lane & 7) + 8 * (lane >> 4)) * LD + kk + 8 * ((lane >> 3) & 1)));
+    mma_bf16(acc[0], af, wb[0], wb[1]);
+    mma_bf16(acc[1], af, wb[2], wb[3]);
+  }
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    const int col = n0 + warp * 16 + n * 8 + 2 * (lane & 3);
+    if (col >= a.dv) continue;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = (lane >> 2) + 8 * half;
+      if (r >= rows) continue;
+      float g0 = 1.0f, g1 = 1.0f;
+      if (a.gate) {
+        const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(a.gate + (size_t)(t0 + r) * a.gate_ld + (size_t)h * a.dv + col));
+        g0 = g.x;
+        g1 = g.y;
+      }
+      *reinterpret_cast<uint32_t*>(a.out + (size_t)(t0 + r) * a.ld_out + (size_t)h * a.dv + col) =
+          pack_bf16(acc[n][2 * half] * g0, acc[n][2 * half + 1] * g1);
+    }
+  }
+}
+
+// -------------------------------------------------------------------------------------------------
+// Visible latents of every sequence, page by page, as contiguous rows.  One warp per row.
+// -------------------------------------------------------------------------------------------------
+struct GatherLatentArgs {
+  const uint8_t* cache;
+  const int* block_tables;
+  const int* cu_kv;        // [S + 1]
+  uint8_t* rows;           // [total][row_bytes]
+  int max_blocks, num_blocks, page, row_bytes;
+  int total;
+};
+
+__global__ void __launch_bounds__(256) gather_latents_kernel(const GatherLatentArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.y, lane = threadIdx.x & 31, j = blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int start = a.cu_kv[seq];
+  const int len = clamp_context(a.cu_kv[seq + 1] - start, a.max_blocks, a.page);
+  if (j >= len) return;
+  const long long dst = (long long)start + j;
+  if (dst < 0 || dst >= a.total) {
+    if (lane == 0) prism_report(PRISM_ERR_BOUNDS, 4);
+    return;
+  }
+  const int blk = checked_page(a.block_tables[(size_t)seq * a.max_blocks + j / a.page], a.num_blocks);
+  const uint4* src = reinterpret_cast<const uint4*>(a.cache + ((size_t)max(blk, 0) * a.page + j % a.page) * a.row_bytes);
+  uint4* out = reinterpret_cast<uint4*>(a.rows + (size_t)dst * a.row_bytes);
+  for (int i = lane; i < a.row_bytes / 16; i += 32) out[i] = blk >= 0 ? src[i] : make_uint4(0, 0, 0, 0);
+}
+
+// -------------------------------------------------------------------------------------------------
+// True 32-bit forms.
+// -------------------------------------------------------------------------------------------------
+// out[t][h * n_out + n] = gate * sum_k x[t][h * kx + k] w(h, k, n): w is [H * kx][ldw] (transposed = 0, n along the
+// row) or [H * n_out][ldw] (transposed = 1, k along the row).
+struct HeadwiseArgs {
+  const float* x;
+  long long ldx;
+  const float* w;
+  long long ldw;
+  const float* gate;
+  long long gate_ld;
+  float* out;
+  long long ldo;
+  int H, kx, n_out, transposed;
+};
+
+__global__ void __launch_bounds__(128) headwise_f32_kernel(const HeadwiseArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n = blockIdx.x * 128 + threadIdx.x, h = blockIdx.y;
+  const size_t t = blockIdx.z;
+  if (n >= a.n_out) return;
+  const float* x = a.x + t * a.ldx + (size_t)h * a.kx;
+  float v = 0.0f;
+  if (a.transposed) {
+    const float* w = a.w + ((size_t)h * a.n_out + n) * a.ldw;
+    for (int k = 0; k < a.kx; ++k) v = fmaf(x[k], w[k], v);
+  } else {
+    const float* w = a.w + (size_t)h * a.kx * a.ldw + n;
+    for (int k = 0; k < a.kx; ++k) v = fmaf(x[k], w[(size_t)k * a.ldw], v);
+  }
+  if (a.gate) v *= a.gate[t * a.gate_ld + (size_t)h * a.n_out + n];
+  a.out[t * a.ldo + (size_t)h * a.n_out + n] = v;
+}
+
+struct LatentF32Args {
+  const float* q;           // [tokens][H][Rc]
+  const float* cache;       // [blocks][page][Rc]
+  const int* block_tables;
+  const int* cu_q;
+  const int* kv_lens;
+  float* out;               // [tokens][H][Rc]
+  int H, Rc, page, max_blocks, num_blocks;
+  float scale;
+};
+
+// One CTA per (token, head) row; its four warps take every fourth key and merge at the end.
+template <int RL>
+__global__ void __launch_bounds__(128) latent_attention_f32_kernel(const LatentF32Args a) {
+  __shared__ float m_s[4], l_s[4];
+  extern __shared__ float o_s[];  // [4][Rc]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, seq = blockIdx.y;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int q_start = a.cu_q ? a.cu_q[seq] : seq;
+  const int q_len = a.cu_q ? a.cu_q[seq + 1] - q_start : 1;
+  const int row = blockIdx.x;
+  if (row >= q_len * a.H) return;
+  const int kv_len = clamp_context(a.kv_lens[seq], a.max_blocks, a.page);
+  const int limit = min(kv_len, kv_len - q_len + row / a.H + 1);
+  const size_t r = (size_t)q_start * a.H + row;
+  float q[RL], o[RL];
+#pragma unroll
+  for (int e = 0; e < RL; ++e) {
+    const int i = lane + 32 * e;
+    q[e] = i < a.Rc ? a.q[r * a.Rc + i] : 0.0f;
+    o[e] = 0.0f;
+  }
+  float m = -INFINITY, l = 0.0f;
+  for (int j = warp; j < limit; j += 4) {
+    const int blk = checked_page(a.block_tables[(size_t)seq * a.max_blocks + j / a.page], a.num_blocks);
+    if (blk < 0) continue;
+    const float* c = a.cache + ((size_t)blk * a.page + j % a.page) * a.Rc;
+    float k[RL], s = 0.0f;
+#pragma unroll
+    for (int e = 0; e < RL; ++e) {
+      const int i = lane + 32 * e;
+      k[e] = i < a.Rc ? c[i] : 0.0f;
+      s = fmaf(q[e], k[e], s);
+    }
+    s = warp_sum(s) * a.scale;
+    if (s > m) {
+      const float f = expf(m - s);  // 0 for the first key
+      m = s;
+      l *= f;
+#pragma unroll
+      for (int e = 0; e < RL; ++e) o[e] *= f;
+    }
+    const float p = expf(s - m);
+    l += p;
+#pragma unroll
+    for (int e = 0; e < RL; ++e) o[e] = fmaf(p, k[e], o[e]);
+  }
+  if (lane == 0) {
+    m_s[warp] = m;
+    l_s[warp] = l;
+  }
+#pragma unroll
+  for (int e = 0; e < RL; ++e) {
+    const int i = lane + 32 * e;
+    if (i < a.Rc) o_s[warp * a.Rc + i] = o[e];
+  }
+  __syncthreads();
+  float mx = -INFINITY;
+  for (int w = 0; w < 4; ++w)
+    if (l_s[w] > 0.0f) mx = fmaxf(mx, m_s[w]);
+  float f[4], sum = 0.0f;
+  for (int w = 0; w < 4; ++w) {
+    f[w] = l_s[w] > 0.0f ? expf(m_s[w] - mx) : 0.0f;
+    sum += f[w] * l_s[w];
+  }
+  for (int i = threadIdx.x; i < a.Rc; i += 128) {
+    float v = 0.0f;
+    for (int w = 0; w < 4; ++w) v += f[w] * o_s[w * a.Rc + i];
+    a.out[r * a.Rc + i] = sum > 0.0f ? v / sum : 0.0f;
+  }
+}
+
+template <int MT, int NT, int BN>
+int launch_latent(const LatentAttnArgs& a, int row_tiles, int S, cudaStream_t stream, bool pdl) {
+  const size_t LD = (size_t)a.Rc + 8;
+  const size_t smem = (16 * MT * LD + 2 * BN * LD) * 2 + 16 * MT * ((BN + 4) * 4 + (BN + 8) * 2 + 12);
+  static size_t configured = 0;
+  if (smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<MT, NT, BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = smem;
+  }
+  return (int)prism_launch(latent_attention_kernel<MT, NT, BN>, dim3(row_tiles, a.nsplit, S), dim3(256), smem, stream, pdl, a);
+}
+
+template <typename T>
+NormStoreArgs<T> norm_store_args(const void* raw, long long ld_raw, const void* weight, void* cache, const void* slots,
+                                 long long num_slots, void* rows, int tokens, int R, int Rc, float eps) {
+  return NormStoreArgs<T>{(const T*)raw, ld_raw, (const T*)weight, (T*)cache, (const long long*)slots, num_slots, (T*)rows,
+                          tokens, R, Rc, eps};
+}
+
+}  // namespace
+
+// Latent rows of the new tokens: RMS norm over R elements with a weight, zero padding up to Rc, stored at flat slots
+// (block * page + offset) and, when rows is given, contiguously.
+PRISM_API int prism_latent_norm_store(int f32, const void* raw, long long ld_raw, const void* weight, void* cache,
+                                      const void* slots, long long num_slots, void* rows, int tokens, int R, int Rc, float eps,
+                                      void* stream, int pdl) {
+  if (tokens <= 0) return 0;
+  if (R <= 0 || R > Rc || Rc % 64) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((tokens + 7) / 8);
+  if (f32)
+    return (int)prism_launch(latent_norm_store_kernel<float>, grid, dim3(256), 0, s, pdl != 0,
+                             norm_store_args<float>(raw, ld_raw, weight, cache, slots, num_slots, rows, tokens, R, Rc, eps));
+  return (int)prism_launch(latent_norm_store_kernel<bf16>, grid, dim3(256), 0, s, pdl != 0,
+                           norm_store_args<bf16>(raw, ld_raw, weight, cache, slots, num_slots, rows, tokens, R, Rc, eps));
+}
+
+// q~ [tokens][H][Rc] = U_h^T q_h (bf16), with the norm and store of the same tokens' latents in the same launch.
+PRISM_API int prism_latent_absorb(const void* q, long long ldq, const void* uk, void* out, const void* raw, long long ld_raw,
+                                  const void* weight, void* cache, const void* slots, long long num_slots, int tokens, int H,
+                                  int dq, int R, int Rc, float eps, void* stream, int pdl) {
+  if (tokens <= 0) return 0;
+  if (R <= 0 || R > Rc || Rc % 64 || H <= 0 || dq % 8 || ldq % 8) return -1;
+  AbsorbArgs a;
+  a.q = (const bf16*)q;
+  a.ldq = ldq;
+  a.uk = (const bf16*)uk;
+  a.out = (bf16*)out;
+  a.H = H;
+  a.dq = dq;
+  a.dk16 = (dq + 15) / 16 * 16;
+  a.ns = norm_store_args<bf16>(raw, ld_raw, weight, cache, slots, num_slots, nullptr, tokens, R, Rc, eps);
+  const size_t smem = ((size_t)a.dk16 * ABS_LDW + 16 * (a.dk16 + 8)) * 2;
+  if (smem > 220 * 1024) return -2;
+  static size_t configured = 48 * 1024;
+  if (smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(latent_absorb_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = smem;
+  }
+  const dim3 grid((Rc + ABS_N - 1) / ABS_N, H + 1, (tokens + 15) / 16);
+  return (int)prism_launch(latent_absorb_kernel, grid, dim3(128), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
+}
+
+// Causal attention of q~ over the paged latents.  nsplit > 1: unnormalised fp32 partials and their maxima / sums;
+// nsplit == 1: normalised bf16 rows in out.  Rc at most 1024.
+PRISM_API int prism_latent_attention(const void* q, const void* cache, const void* block_tables, const void* cu_q,
+                                     const void* kv_lens, void* part_o, void* part_ml, void* out, int S, int max_q_len, int H,
+                                     int Rc, int page, int max_blocks, int num_blocks, int nsplit, float scale, void* stream,
+                                     int pdl) {
+  if (S <= 0 || max_q_len <= 0) return 0;
+  if (H <= 0 || Rc % 64 || Rc <= 0 || Rc > 1024 || page <= 0 || max_blocks <= 0) return -1;
+  if (nsplit < 1 || nsplit > MAX_SPLITS || (nsplit > 1 ? (!part_o || !part_ml) : !out)) return -2;
+  LatentAttnArgs a{(const bf16*)q, (const bf16*)cache, (const int*)block_tables, (const int*)cu_q, (const int*)kv_lens,
+                   (float*)part_o, (float*)part_ml, (bf16*)out, H, Rc, page, max_blocks, num_blocks, nsplit, scale};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const long long rows = (long long)max_q_len * H;
+  const bool narrow = rows <= 16;
+  const int tiles = (int)((rows + (narrow ? 15 : 31)) / (narrow ? 16 : 32));
+  const bool p = pdl != 0;
+#define PRISM_LATENT_CASE(NT_, BN_)                                    \
+  return narrow ? launch_latent<1, NT_, BN_>(a, tiles, S, s, p) : launch_latent<2, NT_, BN_>(a, tiles, S, s, p);
+  if (Rc <= 128) PRISM_LATENT_CASE(2, 64)
+  if (Rc <= 256) PRISM_LATENT_CASE(4, 64)
+  if (Rc <= 512) PRISM_LATENT_CASE(8, 64)
+  PRISM_LATENT_CASE(16, 32)
+#undef PRISM_LATENT_CASE
+}
+
+// out [tokens][ld_out] (head h at column h * dv) = gate * V_h o~_h, o~ merged from the splits of prism_latent_attention.
+PRISM_API int prism_latent_out(const void* part_o, const void* part_ml, const void* lat, const void* uv, const void* gate,
+                               long long gate_ld, void* out, long long ld_out, int tokens, int H, int dv, int Rc, int nsplit,
+                               void* stream, int pdl) {
+  if (tokens <= 0) return 0;
+  if (H <= 0 || dv % 8 || Rc % 64 || Rc <= 0 || Rc > 1024 || nsplit < 1 || nsplit > MAX_SPLITS || gate_ld % 2 || ld_out % 2) return -1;
+  LatentOutArgs a{(const float*)part_o, (const float*)part_ml, (const bf16*)lat, (const bf16*)uv, (const bf16*)gate, gate_ld,
+                  (bf16*)out, ld_out, tokens, H, dv, Rc, nsplit};
+  const size_t smem = (size_t)(OUT_N + 16) * (Rc + 8) * 2;
+  static size_t configured = 40 * 1024;
+  if (smem > configured) {
+    cudaError_t e = cudaFuncSetAttribute(latent_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = smem;
+  }
+  const dim3 grid((dv + OUT_N - 1) / OUT_N, H, (tokens + 15) / 16);
+  return (int)prism_launch(latent_out_kernel, grid, dim3(128), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
+}
+
+// rows [total][row_bytes]: the latents each sequence sees (cu_kv), gathered from their pages.
+PRISM_API int prism_gather_latents(const void* cache, const void* block_tables, const void* cu_kv, void* rows, int S,
+                                   int max_kv_len, int total, int max_blocks, int num_blocks, int page, int row_bytes,
+                                   void* stream, int pdl) {
+  if (S <= 0 || max_kv_len <= 0 || total <= 0) return 0;
+  if (row_bytes % 16 || page <= 0 || max_blocks <= 0) return -1;
+  GatherLatentArgs a{(const uint8_t*)cache, (const int*)block_tables, (const int*)cu_kv, (uint8_t*)rows,
+                     max_blocks, num_blocks, page, row_bytes, total};
+  return (int)prism_launch(gather_latents_kernel, dim3((max_kv_len + 7) / 8, S), dim3(256), 0,
+                           reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
+}
+
+PRISM_API int prism_headwise_f32(const void* x, long long ldx, const void* w, long long ldw, const void* gate, long long gate_ld,
+                                 void* out, long long ldo, int tokens, int H, int kx, int n_out, int transposed, void* stream,
+                                 int pdl) {
+  if (tokens <= 0) return 0;
+  if (H <= 0 || kx <= 0 || n_out <= 0 || tokens > 65535) return -1;
+  HeadwiseArgs a{(const float*)x, ldx, (const float*)w, ldw, (const float*)gate, gate_ld, (float*)out, ldo, H, kx, n_out, transposed};
+  return (int)prism_launch(headwise_f32_kernel, dim3((n_out + 127) / 128, H, tokens), dim3(128), 0,
+                           reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
+}
+
+PRISM_API int prism_latent_attention_f32(const void* q, const void* cache, const void* block_tables, const void* cu_q,
+                                         const void* kv_lens, void* out, int S, int max_q_len, int H, int Rc, int page,
+                                         int max_blocks, int num_blocks, float scale, void* stream, int pdl) {
+  if (S <= 0 || max_q_len <= 0) return 0;
+  if (H <= 0 || Rc % 64 || Rc <= 0 || Rc > 1024 || page <= 0 || max_blocks <= 0) return -1;
+  LatentF32Args a{(const float*)q, (const float*)cache, (const int*)block_tables, (const int*)cu_q, (const int*)kv_lens,
+                  (float*)out, H, Rc, page, max_blocks, num_blocks, scale};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((unsigned)max_q_len * H, S);
+  const size_t smem = (size_t)4 * Rc * sizeof(float);
+  if (Rc <= 128) return (int)prism_launch(latent_attention_f32_kernel<4>, grid, dim3(128), smem, s, pdl != 0, a);
+  if (Rc <= 256) return (int)prism_launch(latent_attention_f32_kernel<8>, grid, dim3(128), smem, s, pdl != 0, a);
+  if (Rc <= 512) return (int)prism_launch(latent_attention_f32_kernel<16>, grid, dim3(128), smem, s, pdl != 0, a);
+  return (int)prism_launch(latent_attention_f32_kernel<32>, grid, dim3(128), smem, s, pdl != 0, a);
+}

@@ -1,0 +1,318 @@
+"""Ops of models with latent attention, stacked projections and a 32-bit residual stream.
+
+Same contract as the package's other ops: CUDA tensors run the kernels of ``libprism_b200.so`` (bf16, or the
+true 32-bit kernels when the tensors are fp32) and raise without them; CPU tensors run the plain-PyTorch
+statement.  Kernels: ``csrc/residual_stream.cu``, ``csrc/latent_attention.cu``, ``csrc/gemm_f32.cu``, the
+section epilogue of ``csrc/gemm_tcgen05.cu`` and the gated form of ``csrc/attention_tcgen05.cu``.
+"""
+
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import Optional, Sequence
+
+import torch
+import torch.nn.functional as F
+
+from . import SM_COUNT, KVCache, _p, _pdl, _s, choose_splits, linear, linear_partial, native
+
+ACTS = {None: 0, "gelu_tanh": 1, "gelu": 2, "sigmoid": 3, "softcap": 4}
+MAX_SPLITS = 32
+MAX_LATENT = 1024       # widest latent row of the attention kernels
+FLASH_MAX_HEAD = 128    # widest head of the tcgen05 prefill attention
+EXPAND_MAX_SCRATCH_BYTES = 2 << 30
+
+
+# ------------------------------------------------------------------------------ stacked projections
+class Sections:
+    """Row ranges of a stacked weight matrix: ``(rows, alpha, act)`` each; ``cap`` bounds ``softcap`` sections
+    (``cap * tanh(v / cap)``)."""
+
+    def __init__(self, parts: Sequence[tuple[int, float, Optional[str]]], cap: float = 0.0) -> None:
+        self.parts = [(int(r), float(a), act) for r, a, act in parts]
+        self.cap = float(cap)
+        n = len(self.parts)
+        ends, total = [], 0
+        for rows, _, _ in self.parts:
+            total += rows
+            ends.append(total)
+        self.rows = total
+        self.row_end = (ctypes.c_int * n)(*ends)
+        self.alpha = (ctypes.c_float * n)(*(a for _, a, _ in self.parts))
+        self.act = (ctypes.c_int * n)(*(ACTS[act] for _, _, act in self.parts))
+
+    def args(self) -> tuple:
+        return (len(self.parts), ctypes.addressof(self.row_end), ctypes.addressof(self.alpha), ctypes.addressof(self.act), self.cap)
+
+
+def _apply(y: torch.Tensor, act: Optional[str], cap: float) -> torch.Tensor:
+    if act == "gelu":
+        return F.gelu(y)
+    if act == "gelu_tanh":
+        return F.gelu(y, approximate="tanh")
+    if act == "sigmoid":
+        return torch.sigmoid(y)
+    return cap * torch.tanh(y / cap) if act == "softcap" else y
+
+
+def linear_sections(x: torch.Tensor, w: torch.Tensor, sections: Sections, *, bias: Optional[torch.Tensor] = None,
+                    out_f32: bool = False, stages: int = 0) -> torch.Tensor:
+    """``act_i(alpha_i * x @ w_i.T + bias_i)`` for every row section ``i`` of ``w``, side by side in one ``[T, M]``."""
+    T, K = x.shape
+    M = w.shape[0]
+    assert sections.rows == M
+    if not x.is_cuda:
+        y = F.linear(x.float(), w.float())
+        cols, parts = 0, []
+        for rows, alpha, act in sections.parts:
+            z = y[:, cols:cols + rows] * alpha
+            if bias is not None:
+                z = z + bias[cols:cols + rows].float()
+            parts.append(_apply(z, act, sections.cap))
+            cols += rows
+        y = torch.cat(parts, dim=1)
+        return y if out_f32 else y.to(x.dtype)
+    assert x.stride(1) == 1 and w.stride(1) == 1 and x.dtype == w.dtype
+    n, ends, alpha, act, cap = sections.args()
+    if x.dtype == torch.float32:
+        out = torch.empty((T, M), dtype=torch.float32, device=x.device)
+        native.call("prism_gemm_f32", _p(w), _p(x), _p(out), M, T, K, w.stride(0), x.stride(0), out.stride(0), _p(bias), n, ends,
+                    alpha, act, cap, _s(), _pdl())
+        return out
+    out = torch.empty((T, M), dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
+    native.call("prism_gemm_wx_sections", _p(w), _p(x), _p(out), M, T, K, w.stride(0), x.stride(0), out.stride(0), _p(bias), n,
+                ends, alpha, act, cap, 1 if out_f32 else 0, 0, stages, _s(), _pdl())
+    return out
+
+
+def linear_slabs(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """fp32 slabs ``[S, T, M]`` whose sum is ``x @ w.T``, for any number of tokens."""
+    if x.is_cuda and x.dtype == torch.float32:
+        T, K = x.shape
+        out = torch.empty((1, T, w.shape[0]), dtype=torch.float32, device=x.device)
+        native.call("prism_gemm_f32", _p(w), _p(x), _p(out), w.shape[0], T, K, w.stride(0), x.stride(0), out.stride(1), None, 0,
+                    None, None, None, 0.0, _s(), _pdl())
+        return out
+    return linear_partial(x, w, choose_splits(w.shape[0], w.shape[1], x.shape[0]) if x.is_cuda else 1)
+
+
+# --------------------------------------------------------------------------------- residual stream
+@dataclass
+class Branch:
+    """Output of a sublayer on its way into the stream: fp32 ``slabs [S, T, W]`` or ``rows [T, W]``, with an
+    element-wise ``gate [T, W]``."""
+
+    slabs: Optional[torch.Tensor] = None
+    rows: Optional[torch.Tensor] = None
+    gate: Optional[torch.Tensor] = None
+
+    def value(self) -> torch.Tensor:
+        v = self.slabs.sum(0) if self.slabs is not None else self.rows.float()
+        return v if self.gate is None else v * self.gate.float()
+
+
+def stream_update(x: torch.Tensor, width: int, eps: float, *, keep: bool, ids: Optional[torch.Tensor] = None,
+                  table: Optional[torch.Tensor] = None, a: Optional[Branch] = None, b: Optional[Branch] = None, mult: float = 1.0,
+                  bias: Optional[torch.Tensor] = None, norm_out: Optional[torch.Tensor] = None,
+                  raw_out: Optional[torch.Tensor] = None, embed_out: Optional[torch.Tensor] = None) -> None:
+    """``x [T, W]`` (fp32, in place) ``= (x if keep) + table[ids] + mult * (a + b) + bias``, and what follows reads of
+    it: ``norm_out`` the rows over their root mean square (``width`` real columns, the rest are zero), ``raw_out``
+    the rows themselves, ``embed_out`` the embedding rows, each in its own type."""
+    T, W = x.shape
+    if not x.is_cuda:
+        new = x.clone() if keep else torch.zeros_like(x)
+        for branch in (a, b):
+            if branch is not None:
+                new += mult * branch.value()
+        if bias is not None:
+            new += bias.float()
+        if ids is not None:
+            emb = table[ids].float()
+            new += emb
+            if embed_out is not None:
+                embed_out.copy_(emb)
+        x.copy_(new)
+        if raw_out is not None:
+            raw_out.copy_(new)
+        if norm_out is not None:
+            norm_out.copy_(new / torch.sqrt(new.pow(2).sum(-1, keepdim=True) / width + eps))
+        return
+    kinds = [t.dtype for t in (table, bias, norm_out, raw_out, embed_out) if t is not None]
+    for branch in (a, b):
+        if branch is not None:
+            kinds += [t.dtype for t in (branch.rows, branch.gate) if t is not None]
+    assert x.dtype == torch.float32 and x.is_contiguous() and len(set(kinds)) == 1
+    gate_ld = 0
+    flat: list = []
+    for branch in (a, b):
+        if branch is None:
+            flat += [None, 0, 0, None, 0, None]
+            continue
+        s, r, g = branch.slabs, branch.rows, branch.gate
+        assert s is None or (s.stride(1) == W and s.stride(2) == 1)
+        if g is not None:
+            assert gate_ld in (0, g.stride(0))
+            gate_ld = g.stride(0)
+        flat += [_p(s), s.stride(0) if s is not None else 0, s.shape[0] if s is not None else 0, _p(r),
+                 r.stride(0) if r is not None else 0, _p(g)]
+    ld = lambda t: t.stride(0) if t is not None else 0  # noqa: E731
+    native.call("prism_stream_update", 1 if kinds[0] == torch.float32 else 0, T, _p(x), 1 if keep else 0, _p(ids), _p(table),
+                table.shape[0] if table is not None else 0, *flat, gate_ld, float(mult), _p(bias), _p(norm_out), ld(norm_out),
+                _p(raw_out), ld(raw_out), _p(embed_out), ld(embed_out), W, width, float(eps), _s(),
+                0 if ids is not None else _pdl())  # the first kernel of a step may follow a copy: full dependency
+
+
+# -------------------------------------------------------------------------------- latent attention
+@dataclass
+class LatentWeights:
+    """What a latent-attention layer multiplies latents with.  ``uk [H * dq, Rc]`` and ``uv [H * dv, Rc]`` are the two
+    halves of ``ukv``; ``norm [R]`` is the latent's RMS-norm weight.  ``dq`` / ``dv`` are the padded head widths, ``Rc``
+    the padded latent width; padding is zero."""
+
+    heads: int
+    dq: int
+    dv: int
+    rank: int
+    scale: float
+    norm: torch.Tensor
+    ukv: torch.Tensor
+
+    @property
+    def uk(self) -> torch.Tensor:
+        return self.ukv[:self.heads * self.dq]
+
+    @property
+    def uv(self) -> torch.Tensor:
+        return self.ukv[self.heads * self.dq:]
+
+
+def latent_norm_store(raw: torch.Tensor, lw: LatentWeights, eps: float, slots: torch.Tensor, cache: KVCache, layer: int, *,
+                      rows: Optional[torch.Tensor] = None) -> None:
+    """RMS-normalise the projected latents ``raw [T, R]`` with their weight and store them at flat ``slots`` (negative =
+    skip) of a single-plane cache, and into ``rows [T, Rc]`` when given."""
+    T, Rc = raw.shape[0], cache.head_dim
+    if not raw.is_cuda:
+        v = raw[:, :lw.rank].float()
+        c = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps) * lw.norm.float()
+        keep = slots >= 0
+        pages = cache.latent(layer)
+        pages[slots[keep] // cache.page, slots[keep] % cache.page, :lw.rank] = c[keep].to(pages.dtype)
+        pages[slots[keep] // cache.page, slots[keep] % cache.page, lw.rank:] = 0
+        if rows is not None:
+            rows.zero_()
+            rows[:, :lw.rank] = c.to(rows.dtype)
+        return
+    native.call("prism_latent_norm_store", 1 if raw.dtype == torch.float32 else 0, _p(raw), raw.stride(0), _p(lw.norm),
+                _p(cache.latent(layer)), _p(slots), cache.num_blocks * cache.page, _p(rows), T, lw.rank, Rc, float(eps), _s(), _pdl())
+
+
+def latent_splits(sequences: int, rows: int) -> int:
+    """CTAs per key range: one CTA per SM is resident, so no more than fill the device once."""
+    tiles = sequences * max(1, -(-rows // (16 if rows <= 16 else 32)))
+    return max(1, min(MAX_SPLITS, SM_COUNT // tiles))
+
+
+def latent_attention_absorbed(
+    q: torch.Tensor, raw: torch.Tensor, gate: Optional[torch.Tensor], lw: LatentWeights, eps: float, slots: torch.Tensor,
+    cache: KVCache, layer: int, block_tables: torch.Tensor, kv_lens: torch.Tensor, *, cu_seqlens_q: Optional[torch.Tensor] = None,
+    max_q_len: int = 1, nsplit: int = 0,
+) -> torch.Tensor:
+    """Store the new tokens' latents, then causal attention of their heads over the paged latents in the absorbed
+    form, times the output ``gate``: ``[T, H * dv]``.
+
+    ``q [T, H * dq]``, ``raw [T, R]`` and ``gate [T, H * dv]`` may be column ranges of a stacked projection.  Without
+    ``cu_seqlens_q`` every token is its own sequence (a decode step)."""
+    T, H, Rc = q.shape[0], lw.heads, cache.head_dim
+    if not q.is_cuda:
+        latent_norm_store(raw, lw, eps, slots, cache, layer)
+        qa = torch.einsum("thd,hdr->thr", q.reshape(T, H, lw.dq).float(), lw.uk.float().view(H, lw.dq, Rc))
+        lat = torch.zeros((T, H, Rc), dtype=torch.float32)
+        pages = cache.latent(layer).float()
+        cu = cu_seqlens_q.tolist() if cu_seqlens_q is not None else list(range(T + 1))
+        for s, (lo, hi) in enumerate(zip(cu[:-1], cu[1:])):
+            n = int(kv_lens[s])
+            if n == 0:
+                continue
+            pos = torch.arange(n)
+            blk = block_tables[s, pos // cache.page].long()
+            c = pages[blk.clamp_min(0), pos % cache.page]
+            sc = torch.einsum("thr,nr->thn", qa[lo:hi], c) * lw.scale
+            seen = (pos[None, :] <= torch.arange(n - (hi - lo), n)[:, None]) & (blk >= 0)[None, :]
+            sc = sc.masked_fill(~seen[:, None, :], float("-inf"))
+            lat[lo:hi] = torch.einsum("thn,nr->thr", torch.softmax(sc, dim=-1), c)
+        o = torch.einsum("thr,hvr->thv", lat, lw.uv.float().view(H, lw.dv, Rc)).reshape(T, H * lw.dv)
+        return (o if gate is None else o * gate.float()).to(q.dtype)
+    S = T if cu_seqlens_q is None else cu_seqlens_q.shape[0] - 1
+    dev = q.device
+    pages = cache.latent(layer)
+    page_args = (_p(pages), _p(block_tables), _p(cu_seqlens_q), _p(kv_lens))
+    assert block_tables.dtype == torch.int32 and kv_lens.dtype == torch.int32 and slots.dtype == torch.int64
+    gate_ld = gate.stride(0) if gate is not None else 0
+    if q.dtype == torch.float32:
+        latent_norm_store(raw, lw, eps, slots, cache, layer)
+        qa = torch.empty((T, H, Rc), dtype=torch.float32, device=dev)
+        native.call("prism_headwise_f32", _p(q), q.stride(0), _p(lw.uk), Rc, None, 0, _p(qa), H * Rc, T, H, lw.dq, Rc, 0, _s(), _pdl())
+        lat = torch.empty_like(qa)
+        native.call("prism_latent_attention_f32", _p(qa), *page_args, _p(lat), S, max_q_len, H, Rc, cache.page, block_tables.shape[1],
+                    cache.num_blocks, float(lw.scale), _s(), _pdl())
+        out = torch.empty((T, H * lw.dv), dtype=torch.float32, device=dev)
+        native.call("prism_headwise_f32", _p(lat), H * Rc, _p(lw.uv), Rc, _p(gate), gate_ld, _p(out), H * lw.dv, T, H, Rc, lw.dv, 1,
+                    _s(), _pdl())
+        return out
+    if nsplit <= 0:
+        nsplit = latent_splits(S, max_q_len * H)
+    qa = torch.empty((T, H, Rc), dtype=torch.bfloat16, device=dev)
+    native.call("prism_latent_absorb", _p(q), q.stride(0), _p(lw.uk), _p(qa), _p(raw), raw.stride(0), _p(lw.norm), _p(pages), _p(slots),
+                cache.num_blocks * cache.page, T, H, lw.dq, lw.rank, Rc, float(eps), _s(), _pdl())
+    part_o = part_ml = lat = None
+    if nsplit > 1:
+        part_o = torch.empty((T * H, nsplit, Rc), dtype=torch.float32, device=dev)
+        part_ml = torch.empty((T * H, nsplit, 2), dtype=torch.float32, device=dev)
+    else:
+        lat = torch.empty((T * H, Rc), dtype=torch.bfloat16, device=dev)
+    native.call("prism_latent_attention", _p(qa), *page_args, _p(part_o), _p(part_ml), _p(lat), S, max_q_len, H, Rc, cache.page,
+                block_tables.shape[1], cache.num_blocks, nsplit, float(lw.scale), _s(), _pdl())
+    out = torch.empty((T, H * lw.dv), dtype=torch.bfloat16, device=dev)
+    native.call("prism_latent_out", _p(part_o), _p(part_ml), _p(lat), _p(lw.uv), _p(gate), gate_ld, _p(out), out.stride(0), T, H, lw.dv,
+                Rc, nsplit, _s(), _pdl())
+    return out
+
+
+def expanded_is_cheaper(lw: LatentWeights, row: int, total_kv: int, attended_pairs: int) -> bool:
+    """Whether a prompt step runs faster with explicit keys and values.  Per attended pair the absorbed form
+    multiplies 2 x ``row`` elements per head, the expanded form ``dq + dv``, on a tensor-core path that is about
+    2.5 times as fast, but it first makes keys and values of every visible latent."""
+    if lw.dq != lw.dv or lw.dq > FLASH_MAX_HEAD:
+        return False
+    if total_kv * 2 * (row + lw.heads * (lw.dq + lw.dv)) > EXPAND_MAX_SCRATCH_BYTES:
+        return False
+    absorbed = attended_pairs * 2 * row
+    expanded = (attended_pairs + total_kv * row) * (lw.dq + lw.dv)
+    return expanded < 2.5 * absorbed
+
+
+def latent_attention_expanded(
+    q: torch.Tensor, raw: torch.Tensor, gate: Optional[torch.Tensor], lw: LatentWeights, eps: float, slots: torch.Tensor,
+    cache: KVCache, layer: int, block_tables: torch.Tensor, cu_seqlens_q: torch.Tensor, max_q_len: int, *,
+    cu_seqlens_kv: Optional[torch.Tensor] = None, total_kv: int = 0, max_kv_len: int = 0,
+) -> torch.Tensor:
+    """The same result from explicit keys and values (bf16, CUDA): the visible latents as contiguous rows (the new
+    tokens' own without ``cu_seqlens_kv``, else gathered from their pages), one GEMM for the keys and values of all
+    heads, and the tcgen05 attention kernel with the gate in its epilogue."""
+    T, H, Rc = q.shape[0], lw.heads, cache.head_dim
+    dev, S = q.device, cu_seqlens_q.shape[0] - 1
+    assert q.is_cuda and q.dtype == torch.bfloat16 and lw.dq == lw.dv
+    total = T if cu_seqlens_kv is None else int(total_kv)
+    c = torch.empty((total, Rc), dtype=torch.bfloat16, device=dev)
+    latent_norm_store(raw, lw, eps, slots, cache, layer, rows=c if cu_seqlens_kv is None else None)
+    if cu_seqlens_kv is not None:
+        native.call("prism_gather_latents", _p(cache.latent(layer)), _p(block_tables), _p(cu_seqlens_kv), _p(c), S, int(max_kv_len),
+                    total, block_tables.shape[1], cache.num_blocks, cache.page, Rc * 2, _s(), _pdl())
+    kv = linear(c, lw.ukv)
+    k, v = kv[:, :H * lw.dq], kv[:, H * lw.dq:]
+    out = torch.empty((T, H * lw.dv), dtype=torch.bfloat16, device=dev)
+    native.call("prism_flash_attention_tc_kv", _p(q), q.stride(0), _p(k), _p(v), kv.stride(0), _p(out), out.stride(0),
+                _p(cu_seqlens_q), _p(cu_seqlens_kv), _p(gate), gate.stride(0) if gate is not None else 0, T, total, S, int(max_q_len),
+                H, H, lw.dq, float(lw.scale), _s(), _pdl())
+    return out

@@ -27,6 +27,17 @@ _T = {"p": ctypes.c_void_p, "i": ctypes.c_int, "l": ctypes.c_longlong, "f": ctyp
 # name -> argument signature (p pointer, i int, l int64, f float, u uint64)
 _SIGNATURES = {
     "prism_gemm_wx": "pppiiilllippliiiiiliipi",
+    "prism_gemm_wx_sections": "pppiiilllpipppfiiipi",
+    "prism_gemm_f32": "pppiiilllpipppfpi",
+    "prism_stream_update": "iipippl" "plipl" "p" "plipl" "p" "lfp" "plplpl" "iifpi",
+    "prism_latent_norm_store": "iplppplpiiifpi",
+    "prism_latent_absorb": "plppplppp" "liiiiifpi",
+    "prism_latent_attention": "pppppppp" "iiiiiiiifpi",
+    "prism_latent_out": "ppppplpl" "iiiiipi",
+    "prism_gather_latents": "ppppiiiiiiipi",
+    "prism_headwise_f32": "plplplpliiiiipi",
+    "prism_latent_attention_f32": "ppppppiiiiiiifpi",
+    "prism_flash_attention_tc_kv": "plpplplppp" "liiiiiiifpi",
     "prism_gemm_effective_splits": "ii",
     "prism_gemm_clear_tensor_maps": "",
     "prism_add_rmsnorm": "plipppppppiifpi",
@@ -74,11 +85,20 @@ _SIGNATURES = {
     "prism_decode_layers_timeline_stamps": "",
     "prism_decode_layers_seq_step": "i",
 }
-_STATUS_UNITS = ("gemm", "norm", "attn", "attn_tc", "kvops", "sampler", "comm", "decode_layers", "lm_head_fp8")
+_STATUS_UNITS = ("gemm", "norm", "attn", "attn_tc", "kvops", "sampler", "comm", "decode_layers", "lm_head_fp8",
+                 "latent", "stream", "gemm_f32")
 
 
 class NativeError(RuntimeError):
     pass
+
+
+def use_library(path: str) -> None:
+    """Bind another library than the full one (one family's kernel units); before the first call."""
+    global LIB_PATH
+    if _lib is not None and path != LIB_PATH:
+        raise NativeError(f"{LIB_PATH} is already loaded")
+    LIB_PATH = path
 
 
 def available() -> bool:

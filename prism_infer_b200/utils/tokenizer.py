@@ -40,6 +40,4 @@ def load_tokenizer(model: str, arch) -> object:
         from transformers import AutoTokenizer
 
         return AutoTokenizer.from_pretrained(model, use_fast=True)
-    reserved = (arch.image_token_id, arch.video_token_id, arch.vision_start_token_id, arch.vision_end_token_id,
-                arch.eos_token_id)
-    return IdTokenizer(arch.text.vocab_size, reserved, arch.eos_token_id)
+    return IdTokenizer(arch.vocab_size, arch.reserved_token_ids, arch.eos_token_id)
