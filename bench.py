@@ -16,6 +16,7 @@ it waits for the current one, so host work overlaps device work).  ``first_token
 generated token ids of the request, so that runs at different N can be compared by eye.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
+    python bench.py --workload latent-layers     (benchmarks/bench_latent_layers.py)
 """
 
 from __future__ import annotations
@@ -108,7 +109,15 @@ def main() -> None:
     ap.add_argument("--model", default="random:qwen3-vl-8b")
     ap.add_argument("--kv-pages", type=int, default=0)
     ap.add_argument("--logits-precision", default="", choices=["", "model", "fp32", "selective_fp32"])
+    ap.add_argument("--workload", default="headline", choices=["headline", "latent-layers"],
+                    help="latent-layers: layer throughput and kernel rooflines of the latent-attention family beside the grouped-query "
+                         "family at equal size (one GPU; its own JSON line)")
+    ap.add_argument("--sizes", default="2048,4096,8192", help="layer widths of --workload latent-layers")
     args = ap.parse_args()
+    if args.workload == "latent-layers":
+        from benchmarks import bench_latent_layers
+
+        raise SystemExit(bench_latent_layers.main(["--sizes", args.sizes, "--steps", str(args.steps), "--warmup", str(args.warmup)]))
     if args.impl == "reference":
         run_reference(args)
         return

@@ -45,15 +45,59 @@ struct NormStoreArgs {
   T* rows;                 // [tokens][Rc] contiguous copy (null: none)
   int tokens, R, Rc;
   float eps;
+  int vec;                 // 1: raw rows and the weight start on 16-byte boundaries
 };
 
+struct F8 {
+  float v[8];
+};
+__device__ __forceinline__ F8 load8(const float* p) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  return F8{{a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w}};
+}
+__device__ __forceinline__ F8 load8(const bf16* p) {
+  const uint4 raw = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+  F8 f;
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float2 t = __bfloat1622float2(h[e]);
+    f.v[2 * e] = t.x;
+    f.v[2 * e + 1] = t.y;
+  }
+  return f;
+}
+__device__ __forceinline__ void store8(float* p, const F8& f) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(f.v[0], f.v[1], f.v[2], f.v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(f.v[4], f.v[5], f.v[6], f.v[7]);
+}
+__device__ __forceinline__ void store8(bf16* p, const F8& f) {
+  uint4 o;
+  uint32_t* w = reinterpret_cast<uint32_t*>(&o);
+#pragma unroll
+  for (int e = 0; e < 4; ++e) w[e] = pack_bf16(f.v[2 * e], f.v[2 * e + 1]);
+  *reinterpret_cast<uint4*>(p) = o;
+}
+
+constexpr int NORM_VEC = 4;  // 8-element pieces per lane: rows of up to 1024 elements
+
+// A last piece that is not whole (and every piece of unaligned rows) is read element by element.
 template <typename T>
 __device__ __forceinline__ void norm_store_token(const NormStoreArgs<T>& a, int t, int lane) {
   const T* src = a.raw + (size_t)t * a.ld_raw;
+  F8 x[NORM_VEC];
   float ss = 0.0f;
-  for (int i = lane; i < a.R; i += 32) {
-    const float v = to_f(src[i]);
-    ss += v * v;
+#pragma unroll
+  for (int k = 0; k < NORM_VEC; ++k) {
+    const int i = (lane + 32 * k) * 8;
+    if (a.vec && i + 8 <= a.R) {
+      x[k] = load8(src + i);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[k].v[e] = i + e < a.R ? to_f(src[i + e]) : 0.0f;
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += x[k].v[e] * x[k].v[e];
   }
   const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.R + a.eps);
   long long slot = a.slots[t];
@@ -63,10 +107,21 @@ __device__ __forceinline__ void norm_store_token(const NormStoreArgs<T>& a, int 
   }
   T* page_row = slot >= 0 ? a.cache + (size_t)slot * a.Rc : nullptr;
   T* row = a.rows ? a.rows + (size_t)t * a.Rc : nullptr;
-  for (int i = lane; i < a.Rc; i += 32) {
-    const T v = i < a.R ? from_f<T>(to_f(src[i]) * inv * to_f(a.weight[i])) : from_f<T>(0.0f);
-    if (page_row) page_row[i] = v;
-    if (row) row[i] = v;
+#pragma unroll
+  for (int k = 0; k < NORM_VEC; ++k) {
+    const int i = (lane + 32 * k) * 8;
+    if (i >= a.Rc) continue;
+    F8 w;
+    if (a.vec && i + 8 <= a.R) {
+      w = load8(a.weight + i);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w.v[e] = i + e < a.R ? to_f(a.weight[i + e]) : 0.0f;
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) w.v[e] *= x[k].v[e] * inv;
+    if (page_row) store8(page_row + i, w);
+    if (row) store8(row + i, w);
   }
 }
 
@@ -80,7 +135,7 @@ __global__ void __launch_bounds__(256) latent_norm_store_kernel(const NormStoreA
 
 // -------------------------------------------------------------------------------------------------
 // q~ = U_h^T q_h for a tile of 16 tokens, one head and 128 latent elements per CTA.  The CTAs with
-// blockIdx.y == H run the norm and store instead (those with blockIdx.x == 0; the others end).
+// blockIdx.y == H run the norm and store instead, one token per warp.
 // -------------------------------------------------------------------------------------------------
 constexpr int ABS_N = 128, ABS_LDW = ABS_N + 8;
 
@@ -102,8 +157,7 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const AbsorbArgs a) 
   pdl_launch_dependents();
   if ((int)blockIdx.y == a.H) {
     pdl_wait();
-    if (blockIdx.x == 0)
-      for (int t = t0 + warp; t < min(t0 + 16, a.ns.tokens); t += 4) norm_store_token(a.ns, t, lane);
+    for (int t = t0 + blockIdx.x * 4 + warp; t < min(t0 + 16, a.ns.tokens); t += 4 * gridDim.x) norm_store_token(a.ns, t, lane);
     return;
   }
   const int h = blockIdx.y, n0 = blockIdx.x * ABS_N, ldq_s = a.dk16 + 8;
@@ -162,23 +216,48 @@ struct LatentAttnArgs {
   float scale;
 };
 
+// One row of a tile: `bytes` (a multiple of 16) from global to shared memory, completing on `bar`.
+__device__ __forceinline__ void bulk_row(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
+               "l"(src), "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
+}
+
+// Shared-memory bytes of a launch (the kernel lays its buffers out in this order).
+template <int MT, int BN>
+__host__ __device__ constexpr size_t latent_smem_bytes(int Rc) {
+  return (size_t)(16 * MT + 2 * BN) * (Rc + 8) * 2 + (size_t)(8 / (BN / 16)) * 16 * MT * (BN + 4) * 4 + (size_t)16 * MT * (BN + 8) * 2 +
+         4 * 16 * MT * 4 + 3 * 8;
+}
+
+// BM = 16 MT rows of one sequence against its latents in tiles of BN keys.  Eight warps:
+//   scores    warp (kg, kh) takes 16 keys and one of KH slices of the latent; its query fragments stay in registers
+//             for the whole kernel where they fit (QREG), the slices are added when the softmax reads them
+//   softmax   BM / 8 rows per warp
+//   output    every warp accumulates Rc / 8 columns of P C in registers
+// Latent rows come by one bulk copy each, issued by one thread per row, two tiles in flight.  Tiles that hold only
+// latents of earlier steps are fetched before the previous kernel has finished.
 template <int MT, int NT, int BN>
-__global__ void __launch_bounds__(256) latent_attention_kernel(const LatentAttnArgs a) {
+__global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAttnArgs a) {
   constexpr int BM = 16 * MT;
+  constexpr int KG = BN / 16, KH = 8 / KG;
+  constexpr bool QREG = NT <= 8;
+  constexpr int QS = QREG ? NT * 4 / KH : 1;              // 16-element steps of a warp's slice (compile-time bound)
   constexpr int LDS = BN + 4, LDP = BN + 8;
-  extern __shared__ uint8_t smem_raw[];
+  extern __shared__ __align__(128) uint8_t smem_raw[];
   const int Rc = a.Rc, LD = Rc + 8, nt = Rc >> 6;         // nt: 8-column tiles of the output per warp
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);           // [BM][LD]
   bf16* kv_s = q_s + (size_t)BM * LD;                      // [2][BN][LD]
-  float* s_s = reinterpret_cast<float*>(kv_s + (size_t)2 * BN * LD);  // [BM][LDS]
-  bf16* p_s = reinterpret_cast<bf16*>(s_s + BM * LDS);     // [BM][LDP]
+  float* s_s = reinterpret_cast<float*>(kv_s + (size_t)2 * BN * LD);  // [KH][BM][LDS]
+  bf16* p_s = reinterpret_cast<bf16*>(s_s + KH * BM * LDS);  // [BM][LDP]
   float* fac_s = reinterpret_cast<float*>(p_s + BM * LDP); // [BM] rescale of the accumulator
   float* m_s = fac_s + BM;                                 // [BM] running maximum
   float* l_s = m_s + BM;                                   // [BM] running sum
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int* lim_s = reinterpret_cast<int*>(l_s + BM);           // [BM] keys a row sees
+  uint64_t* bars = reinterpret_cast<uint64_t*>(lim_s + BM);  // two tiles, then the queries
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int seq = blockIdx.z, split = blockIdx.y;
   pdl_launch_dependents();
-  pdl_wait();
   const int q_start = a.cu_q ? a.cu_q[seq] : seq;
   const int q_len = a.cu_q ? a.cu_q[seq + 1] - q_start : 1;
   const int n_rows = q_len * a.H, row0 = blockIdx.x * BM;
@@ -190,79 +269,132 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatentAttnA
   const int tb = split * per, te = min(tiles, tb + per);
   const size_t out_row0 = (size_t)q_start * a.H + row0;
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
-  const int pieces = Rc >> 3;
+  const uint32_t row_bytes = (uint32_t)Rc * 2;
 
-  auto load_tile = [&](int j, int stage) {
-    bf16* dst = kv_s + (size_t)stage * BN * LD;
-    for (int i = threadIdx.x; i < BN * pieces; i += 256) {
-      const int r = i / pieces, c = (i - r * pieces) * 8, key = j * BN + r;
-      int blk = key < kv_end ? bt[key / a.page] : -1;
-      blk = checked_page(blk, a.num_blocks);
-      const bool ok = blk >= 0;
-      cp_async16(dst + r * LD + c, ok ? a.cache + ((size_t)blk * a.page + key % a.page) * Rc + c : a.cache, ok);
+  if (tid == 0) {
+    mbar_init(&bars[0], BN);
+    mbar_init(&bars[1], BN);
+    mbar_init(&bars[2], BM);
+    fence_barrier_init();
+  }
+  __syncthreads();
+
+  auto issue = [&](int j) {                                // threads 0 .. BN - 1: one latent row each
+    if (tid < BN && j < te) {
+      const int stage = (j - tb) & 1, key = j * BN + tid;
+      bf16* dst = kv_s + ((size_t)stage * BN + tid) * LD;
+      const int blk = key < kv_end ? checked_page(bt[key / a.page], a.num_blocks) : -1;
+      if (blk >= 0) {
+        fence_proxy_async();
+        mbar_expect_tx(&bars[stage], row_bytes);
+        bulk_row(dst, a.cache + ((size_t)blk * a.page + key % a.page) * Rc, row_bytes, &bars[stage]);
+      } else {                                             // past the end, or a hole: zeros
+        for (int c = 0; c < Rc; c += 8) *reinterpret_cast<uint4*>(dst + c) = make_uint4(0, 0, 0, 0);
+        fence_proxy_async();
+        mbar_arrive(&bars[stage]);
+      }
     }
   };
+  const int old_tiles = max(0, kv_len - q_len) / BN;       // tiles that hold latents of earlier steps only
+  const bool pre0 = tb < old_tiles, pre1 = tb + 1 < old_tiles;
+  if (pre0) issue(tb);
+  if (pre1) issue(tb + 1);
+  if (tid < BM) {
+    const int row = row0 + tid;
+    m_s[tid] = -INFINITY;
+    l_s[tid] = 0.0f;
+    lim_s[tid] = row < n_rows ? kv_len - q_len + row / a.H + 1 : 0;
+  }
+  pdl_wait();
+  if (tb < te && tid < BM) {
+    bf16* dst = q_s + (size_t)tid * LD;
+    if (row0 + tid < n_rows) {
+      mbar_expect_tx(&bars[2], row_bytes);
+      bulk_row(dst, a.q + (out_row0 + tid) * Rc, row_bytes, &bars[2]);
+    } else {
+      for (int c = 0; c < Rc; c += 8) *reinterpret_cast<uint4*>(dst + c) = make_uint4(0, 0, 0, 0);
+      mbar_arrive(&bars[2]);
+    }
+  }
+  if (!pre0) issue(tb);
+  if (!pre1) issue(tb + 1);
 
-  for (int i = threadIdx.x; i < BM * pieces; i += 256) {
-    const int r = i / pieces, c = (i - r * pieces) * 8;
-    const bool ok = row0 + r < n_rows;
-    cp_async16(q_s + r * LD + c, ok ? a.q + (out_row0 + r) * Rc + c : a.q, ok);
-  }
-  if (tb < te) load_tile(tb, 0);
-  cp_async_commit();
-  for (int i = threadIdx.x; i < BM; i += 256) {
-    m_s[i] = -INFINITY;
-    l_s[i] = 0.0f;
-  }
   float acc[MT][NT][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int n = 0; n < NT; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.0f;
   const float sl2 = a.scale * 1.4426950408889634f;
+  const int kg = warp % KG, kh = warp / KG, steps = (Rc >> 4) / KH, k0 = kh * steps * 16;
+  const bf16* q_frag = q_s + (size_t)(lane & 15) * LD + k0 + 8 * (lane >> 4);
+  uint32_t qf[MT][QS][4];
+  if (tb < te) {
+    (void)mbar_wait(&bars[2], 0, 31);
+    if (QREG) {
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int k = 0; k < QS; ++k)
+          if (k < steps) ldsm_x4(qf[m][k], smem_u32(q_frag + (size_t)m * 16 * LD + k * 16));
+    }
+  }
 
   for (int j = tb; j < te; ++j) {
     const int stage = (j - tb) & 1;
-    cp_async_wait<0>();
-    __syncthreads();                 // tile j is in; every warp is done with tile j - 1
-    if (j + 1 < te) load_tile(j + 1, stage ^ 1);
-    cp_async_commit();
+    (void)mbar_wait(&bars[stage], ((j - tb) >> 1) & 1, 32 + stage);
     const bf16* kv = kv_s + (size_t)stage * BN * LD;
-    if (warp < BN / 8) {             // scores of keys 8 warp .. 8 warp + 7
-      float s[MT][4] = {};
-      for (int kk = 0; kk < Rc; kk += 32) {
-        uint32_t kb[4];
-        ldsm_x4(kb, smem_u32(kv + (warp * 8 + (lane & 7)) * LD + kk + 8 * (lane >> 3)));
+    {
+      float s[MT][2][4] = {};
+      const bf16* kp = kv + (size_t)(kg * 16 + (lane & 7) + 8 * (lane >> 4)) * LD + k0 + 8 * ((lane >> 3) & 1);
+      if (QREG) {
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t q0[4], q1[4];
-          const bf16* qp = q_s + (m * 16 + (lane & 15)) * LD + kk + 8 * (lane >> 4);
-          ldsm_x4(q0, smem_u32(qp));
-          ldsm_x4(q1, smem_u32(qp + 16));
-          mma_bf16(s[m], q0, kb[0], kb[1]);
-          mma_bf16(s[m], q1, kb[2], kb[3]);
+        for (int k = 0; k < QS; ++k)
+          if (k < steps) {
+            uint32_t kb[4];
+            ldsm_x4(kb, smem_u32(kp + k * 16));
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+              mma_bf16(s[m][0], qf[m][k], kb[0], kb[1]);
+              mma_bf16(s[m][1], qf[m][k], kb[2], kb[3]);
+            }
+          }
+      } else {
+#pragma unroll 4
+        for (int k = 0; k < steps; ++k) {
+          uint32_t kb[4];
+          ldsm_x4(kb, smem_u32(kp + k * 16));
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            uint32_t q[4];
+            ldsm_x4(q, smem_u32(q_frag + (size_t)m * 16 * LD + k * 16));
+            mma_bf16(s[m][0], q, kb[0], kb[1]);
+            mma_bf16(s[m][1], q, kb[2], kb[3]);
+          }
         }
       }
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        float* d = s_s + (m * 16 + (lane >> 2)) * LDS + warp * 8 + 2 * (lane & 3);
-        d[0] = s[m][0];
-        d[1] = s[m][1];
-        d[8 * LDS] = s[m][2];
-        d[8 * LDS + 1] = s[m][3];
-      }
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          float* d = s_s + ((size_t)kh * BM + m * 16 + (lane >> 2)) * LDS + kg * 16 + n * 8 + 2 * (lane & 3);
+          *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
+          *reinterpret_cast<float2*>(d + 8 * LDS) = make_float2(s[m][n][2], s[m][n][3]);
+        }
     }
     __syncthreads();
     // online softmax, BM / 8 rows per warp
 #pragma unroll
     for (int i = 0; i < BM / 8; ++i) {
-      const int r = warp * (BM / 8) + i, row = row0 + r;
-      const int limit = row < n_rows ? kv_len - q_len + row / a.H + 1 : 0;
+      const int r = warp * (BM / 8) + i;
+      const int limit = lim_s[r] - j * BN;
       float v[BN / 32], mx = -INFINITY;
 #pragma unroll
       for (int e = 0; e < BN / 32; ++e) {
         const int c = lane + 32 * e;
-        v[e] = j * BN + c < limit ? s_s[r * LDS + c] * sl2 : -INFINITY;
+        float t = s_s[r * LDS + c];
+#pragma unroll
+        for (int h = 1; h < KH; ++h) t += s_s[(h * BM + r) * LDS + c];
+        v[e] = c < limit ? t * sl2 : -INFINITY;
         mx = fmaxf(mx, v[e]);
       }
       mx = warp_max(mx);
@@ -303,7 +435,7 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatentAttnA
       uint32_t pf[MT][4];
 #pragma unroll
       for (int m = 0; m < MT; ++m) ldsm_x4(pf[m], smem_u32(p_s + (m * 16 + (lane & 15)) * LDP + kk + 8 * (lane >> 4)));
-      const bf16* vrow = kv + (kk + (lane & 15)) * LD + col0 + 8 * (lane >> 4);
+      const bf16* vrow = kv + (size_t)(kk + (lane & 15)) * LD + col0 + 8 * (lane >> 4);
 #pragma unroll
       for (int n = 0; n < NT; n += 2) {
         if (n < nt) {                // a last odd tile loads its neighbour (or the row's padding) and ignores it
@@ -317,14 +449,14 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatentAttnA
         }
       }
     }
+    __syncthreads();                 // every warp is done with this tile: its buffer takes the tile after the next
+    issue(j + 2);
   }
-  cp_async_wait<0>();
   __syncthreads();
-  if (a.nsplit > 1 && (int)threadIdx.x < BM && row0 + (int)threadIdx.x < n_rows) {
-    float* ml = a.part_ml + ((out_row0 + threadIdx.x) * a.nsplit + split) * 2;
-    ml[0] = m_s[threadIdx.x];
-    ml[1] = l_s[threadIdx.x];
-    if (tb >= te) ml[1] = 0.0f;
+  if (a.nsplit > 1 && tid < BM && row0 + tid < n_rows) {
+    float* ml = a.part_ml + ((out_row0 + tid) * a.nsplit + split) * 2;
+    ml[0] = m_s[tid];
+    ml[1] = l_s[tid];
   }
   if (a.nsplit > 1 && tb >= te) return;  // an empty split has no partial rows
 #pragma unroll
@@ -350,7 +482,7 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatentAttnA
 // -------------------------------------------------------------------------------------------------
 // o_h = gate * V_h (merged latent output): a tile of 16 tokens, one head, 64 output elements per CTA.
 // -------------------------------------------------------------------------------------------------
-constexpr int OUT_N = 64, MAX_SPLITS = 32;
+constexpr int OUT_N = 64, OUT_THREADS = 256, MAX_SPLITS = 64;
 
 struct LatentOutArgs {
   const float* part_o;
@@ -364,93 +496,132 @@ struct LatentOutArgs {
   int tokens, H, dv, Rc, nsplit;
 };
 
-__global__ void __launch_bounds__(128) latent_out_kernel(const LatentOutArgs a) {
-  extern __shared__ uint8_t smem_raw[];
+// Weighted sum of the splits for 16 tokens of one head, as bf16 rows in shared memory.  A thread keeps ITEMS x BATCH
+// independent 16-byte loads in flight.
+template <int ITEMS, int BATCH>
+__device__ __forceinline__ void merge_splits(const LatentOutArgs& a, bf16* a_s, int LD, const float (*wgt)[MAX_SPLITS], const int* used,
+                                             int t0, int h) {
+  const int per_row = a.Rc >> 2, total = 16 * per_row;
+  for (int i0 = threadIdx.x; i0 < total; i0 += OUT_THREADS * ITEMS) {
+    float4 v[ITEMS];
+    int r[ITEMS], c[ITEMS], n_max = 0;
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+      const int i = min(i0 + k * OUT_THREADS, total - 1);
+      r[k] = i / per_row;
+      c[k] = (i - r[k] * per_row) * 4;
+      v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      n_max = max(n_max, used[r[k]]);
+    }
+    for (int s0 = 0; s0 < n_max; s0 += BATCH) {
+      float4 p[ITEMS][BATCH];
+#pragma unroll
+      for (int k = 0; k < ITEMS; ++k) {
+        const float* src = a.part_o + (((size_t)(t0 + r[k]) * a.H + h) * a.nsplit + s0) * a.Rc + c[k];
+#pragma unroll
+        for (int s = 0; s < BATCH; ++s)  // an empty split's rows were never written: weight zero, not read
+          p[k][s] = (s0 + s < used[r[k]] && wgt[r[k]][s0 + s] > 0.0f) ? __ldcg(reinterpret_cast<const float4*>(src + (size_t)s * a.Rc))
+                                                                      : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int k = 0; k < ITEMS; ++k)
+#pragma unroll
+        for (int s = 0; s < BATCH; ++s) {
+          const float w = s0 + s < used[r[k]] ? wgt[r[k]][s0 + s] : 0.0f;
+          v[k].x += w * p[k][s].x;
+          v[k].y += w * p[k][s].y;
+          v[k].z += w * p[k][s].z;
+          v[k].w += w * p[k][s].w;
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+      if (i0 + k * OUT_THREADS >= total) continue;
+      uint2 o;
+      o.x = pack_bf16(v[k].x, v[k].y);
+      o.y = pack_bf16(v[k].z, v[k].w);
+      *reinterpret_cast<uint2*>(a_s + (size_t)r[k] * LD + c[k]) = o;
+    }
+  }
+}
+
+__global__ void __launch_bounds__(OUT_THREADS) latent_out_kernel(const LatentOutArgs a) {
+  extern __shared__ __align__(128) uint8_t smem_raw[];
   const int Rc = a.Rc, LD = Rc + 8, pieces = Rc >> 3;
   bf16* w_s = reinterpret_cast<bf16*>(smem_raw);   // [OUT_N][LD]
   bf16* a_s = w_s + (size_t)OUT_N * LD;            // [16][LD]
   __shared__ float wgt[16][MAX_SPLITS];
+  __shared__ int used[16];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n0 = blockIdx.x * OUT_N, h = blockIdx.y, t0 = blockIdx.z * 16;
   pdl_launch_dependents();
-  for (int i = threadIdx.x; i < OUT_N * pieces; i += 128) {
-    const int r = i / pieces, c = (i - r * pieces) * 8;
+  for (int r = warp; r < OUT_N; r += OUT_THREADS / 32) {
     const bool ok = n0 + r < a.dv;
-    cp_async16(w_s + r * LD + c, ok ? a.uv + ((size_t)h * a.dv + n0 + r) * Rc + c : a.uv, ok);
+    const bf16* src = ok ? a.uv + ((size_t)h * a.dv + n0 + r) * Rc : a.uv;
+    for (int c = lane * 8; c < Rc; c += 256) cp_async16(w_s + (size_t)r * LD + c, ok ? src + c : src, ok);
   }
   cp_async_commit();
   pdl_wait();
   const int rows = min(16, a.tokens - t0);
   if (a.nsplit > 1) {
-    for (int r = warp; r < rows; r += 4) {         // weights of the splits: 2^(m_s - m) / l
-      const size_t row = (size_t)(t0 + r) * a.H + h;
-      float m = -INFINITY, l = 0.0f;
-      if (lane < a.nsplit) {
-        m = a.part_ml[(row * a.nsplit + lane) * 2];
-        l = a.part_ml[(row * a.nsplit + lane) * 2 + 1];
+    for (int r = warp; r < 16; r += OUT_THREADS / 32) {  // weights of the splits: 2^(m_s - m) / l
+      float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+      if (r < rows) {
+        const float2* ml = reinterpret_cast<const float2*>(a.part_ml) + ((size_t)(t0 + r) * a.H + h) * a.nsplit;
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+          if (lane + 32 * e < a.nsplit) {
+            const float2 v = ml[lane + 32 * e];
+            m[e] = v.y > 0.0f ? v.x : -INFINITY;
+            l[e] = v.y;
+          }
       }
-      const float mx = warp_max(l > 0.0f ? m : -INFINITY);
-      const float f = l > 0.0f ? ex2_fast(m - mx) : 0.0f;
-      const float sum = warp_sum(f * l);
-      if (lane < a.nsplit) wgt[r][lane] = sum > 0.0f ? f / sum : 0.0f;
+      const float mx = warp_max(fmaxf(m[0], m[1]));
+      const float f0 = l[0] > 0.0f ? ex2_fast(m[0] - mx) : 0.0f, f1 = l[1] > 0.0f ? ex2_fast(m[1] - mx) : 0.0f;
+      const float sum = warp_sum(f0 * l[0] + f1 * l[1]);
+      const float inv = sum > 0.0f ? 1.0f / sum : 0.0f;
+      wgt[r][lane] = f0 * inv;
+      wgt[r][lane + 32] = f1 * inv;
+      const unsigned b0 = __ballot_sync(0xffffffffu, f0 > 0.0f), b1 = __ballot_sync(0xffffffffu, f1 > 0.0f);
+      if (lane == 0) used[r] = b1 ? 64 - __clz(b1) : (b0 ? 32 - __clz(b0) : 0);
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < 16 * (Rc >> 2); i += 128) {
-      const int r = i / (Rc >> 2), c = (i - r * (Rc >> 2)) * 4;
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (r < rows) {
-        const float* src = a.part_o + ((size_t)(t0 + r) * a.H + h) * a.nsplit * Rc + c;
-#pragma unroll 4
-        for (int s = 0; s < a.nsplit; ++s) {
-          const float w = wgt[r][s];
-          if (w == 0.0f) continue;                 // an empty split's rows were never written
-          const float4 p = __ldcg(reinterpret_cast<const float4*>(src + (size_t)s * Rc));
-          v.x += w * p.x;
-          v.y += w * p.y;
-          v.z += w * p.z;
-          v.w += w * p.w;
-        }
-      }
-      uint2 o;
-      o.x = pack_bf16(v.x, v.y);
-      o.y = pack_bf16(v.z, v.w);
-      *reinterpret_cast<uint2*>(a_s + r * LD + c) = o;
-    }
+    if (a.nsplit <= 4) merge_splits<4, 4>(a, a_s, LD, wgt, used, t0, h);
+    else if (a.nsplit <= 16) merge_splits<2, 16>(a, a_s, LD, wgt, used, t0, h);
+    else merge_splits<1, 32>(a, a_s, LD, wgt, used, t0, h);
   } else {
-    for (int i = threadIdx.x; i < 16 * pieces; i += 128) {
-      const int r = i / pieces, c = (i - r * pieces) * 8;
+    for (int r = warp; r < 16; r += OUT_THREADS / 32) {
       const bool ok = r < rows;
-      cp_async16(a_s + r * LD + c, ok ? a.lat + ((size_t)(t0 + r) * a.H + h) * Rc + c : a.lat, ok);
+      const bf16* src = ok ? a.lat + ((size_t)(t0 + r) * a.H + h) * Rc : a.lat;
+      for (int c = lane * 8; c < Rc; c += 256) cp_async16(a_s + (size_t)r * LD + c, ok ? src + c : src, ok);
     }
     cp_async_commit();
   }
   cp_async_wait<0>();
   __syncthreads();
-  float acc[2][4] = {};
-  for (int kk = 0; kk < Rc; kk += 16) {
-    uint32_t af[4], wb[4];
-    ldsm_x4(af, smem_u32(a_s + (lane & 15) * LD + kk + 8 * (lane >> 4)));
-    ldsm_x4(wb, smem_u32(w_s + (warp * 16 + (lane & 7) + 8 * (lane >> 4)) * LD + kk + 8 * ((lane >> 3) & 1)));
-    mma_bf16(acc[0], af, wb[0], wb[1]);
-    mma_bf16(acc[1], af, wb[2], wb[3]);
+  float acc[2][4] = {};                              // even and odd steps: two independent chains, 8 columns per warp
+#pragma unroll 4
+  for (int kk = 0; kk < Rc; kk += 32) {
+    uint32_t a0[4], a1[4], wb[4];
+    ldsm_x4(wb, smem_u32(w_s + (size_t)(warp * 8 + (lane & 7)) * LD + kk + 8 * (lane >> 3)));
+    ldsm_x4(a0, smem_u32(a_s + (size_t)(lane & 15) * LD + kk + 8 * (lane >> 4)));
+    ldsm_x4(a1, smem_u32(a_s + (size_t)(lane & 15) * LD + kk + 16 + 8 * (lane >> 4)));
+    mma_bf16(acc[0], a0, wb[0], wb[1]);
+    mma_bf16(acc[1], a1, wb[2], wb[3]);
   }
+  const int col = n0 + warp * 8 + 2 * (lane & 3);
+  if (col >= a.dv) return;
 #pragma unroll
-  for (int n = 0; n < 2; ++n) {
-    const int col = n0 + warp * 16 + n * 8 + 2 * (lane & 3);
-    if (col >= a.dv) continue;
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int r = (lane >> 2) + 8 * half;
-      if (r >= rows) continue;
-      float g0 = 1.0f, g1 = 1.0f;
-      if (a.gate) {
-        const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(a.gate + (size_t)(t0 + r) * a.gate_ld + (size_t)h * a.dv + col));
-        g0 = g.x;
-        g1 = g.y;
-      }
-      *reinterpret_cast<uint32_t*>(a.out + (size_t)(t0 + r) * a.ld_out + (size_t)h * a.dv + col) =
-          pack_bf16(acc[n][2 * half] * g0, acc[n][2 * half + 1] * g1);
+  for (int half = 0; half < 2; ++half) {
+    const int r = (lane >> 2) + 8 * half;
+    if (r >= rows) continue;
+    float v0 = acc[0][2 * half] + acc[1][2 * half], v1 = acc[0][2 * half + 1] + acc[1][2 * half + 1];
+    if (a.gate) {
+      const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(a.gate + (size_t)(t0 + r) * a.gate_ld + (size_t)h * a.dv + col));
+      v0 *= g.x;
+      v1 *= g.y;
     }
+    *reinterpret_cast<uint32_t*>(a.out + (size_t)(t0 + r) * a.ld_out + (size_t)h * a.dv + col) = pack_bf16(v0, v1);
   }
 }
 
@@ -605,8 +776,7 @@ __global__ void __launch_bounds__(128) latent_attention_f32_kernel(const LatentF
 
 template <int MT, int NT, int BN>
 int launch_latent(const LatentAttnArgs& a, int row_tiles, int S, cudaStream_t stream, bool pdl) {
-  const size_t LD = (size_t)a.Rc + 8;
-  const size_t smem = (16 * MT * LD + 2 * BN * LD) * 2 + 16 * MT * ((BN + 4) * 4 + (BN + 8) * 2 + 12);
+  const size_t smem = latent_smem_bytes<MT, BN>(a.Rc);
   static size_t configured = 0;
   if (smem > configured) {
     cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<MT, NT, BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -620,7 +790,8 @@ template <typename T>
 NormStoreArgs<T> norm_store_args(const void* raw, long long ld_raw, const void* weight, void* cache, const void* slots,
                                  long long num_slots, void* rows, int tokens, int R, int Rc, float eps) {
   return NormStoreArgs<T>{(const T*)raw, ld_raw, (const T*)weight, (T*)cache, (const long long*)slots, num_slots, (T*)rows,
-                          tokens, R, Rc, eps};
+                          tokens, R, Rc, eps,
+                          ld_raw * sizeof(T) % 16 == 0 && ((reinterpret_cast<uintptr_t>(raw) | reinterpret_cast<uintptr_t>(weight)) & 15) == 0};
 }
 
 }  // namespace
@@ -631,7 +802,7 @@ PRISM_API int prism_latent_norm_store(int f32, const void* raw, long long ld_raw
                                       const void* slots, long long num_slots, void* rows, int tokens, int R, int Rc, float eps,
                                       void* stream, int pdl) {
   if (tokens <= 0) return 0;
-  if (R <= 0 || R > Rc || Rc % 64) return -1;
+  if (R <= 0 || R > Rc || Rc % 64 || Rc > 1024) return -1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid((tokens + 7) / 8);
   if (f32)
@@ -646,7 +817,7 @@ PRISM_API int prism_latent_absorb(const void* q, long long ldq, const void* uk, 
                                   const void* weight, void* cache, const void* slots, long long num_slots, int tokens, int H,
                                   int dq, int R, int Rc, float eps, void* stream, int pdl) {
   if (tokens <= 0) return 0;
-  if (R <= 0 || R > Rc || Rc % 64 || H <= 0 || dq % 8 || ldq % 8) return -1;
+  if (R <= 0 || R > Rc || Rc % 64 || H <= 0 || dq % 8 || ldq % 8 || Rc > 1024) return -1;
   AbsorbArgs a;
   a.q = (const bf16*)q;
   a.ldq = ldq;
@@ -681,7 +852,8 @@ PRISM_API int prism_latent_attention(const void* q, const void* cache, const voi
                    (float*)part_o, (float*)part_ml, (bf16*)out, H, Rc, page, max_blocks, num_blocks, nsplit, scale};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const long long rows = (long long)max_q_len * H;
-  const bool narrow = rows <= 16;
+  // 16-row tiles read the latents once per 16 heads instead of 32: worth it while they still fit the device in one wave
+  const bool narrow = rows <= 16 || (rows + 15) / 16 * nsplit * S <= 148;
   const int tiles = (int)((rows + (narrow ? 15 : 31)) / (narrow ? 16 : 32));
   const bool p = pdl != 0;
 #define PRISM_LATENT_CASE(NT_, BN_)                                    \
@@ -709,7 +881,7 @@ PRISM_API int prism_latent_out(const void* part_o, const void* part_ml, const vo
     configured = smem;
   }
   const dim3 grid((dv + OUT_N - 1) / OUT_N, H, (tokens + 15) / 16);
-  return (int)prism_launch(latent_out_kernel, grid, dim3(128), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
+  return (int)prism_launch(latent_out_kernel, grid, dim3(OUT_THREADS), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
 }
 
 // rows [total][row_bytes]: the latents each sequence sees (cu_kv), gathered from their pages.

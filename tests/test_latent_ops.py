@@ -227,7 +227,7 @@ class Scene:
         device, dtype = self.backend
         yield "absorbed", self.absorbed()
         if dtype == torch.bfloat16:
-            for n in (1, 2, 7, 32):
+            for n in (1, 2, 7, 33, 64):
                 yield f"absorbed, {n} splits", self.absorbed(n)
             if self.lw.dq == self.lw.dv and self.lw.dq <= 128:
                 yield "expanded", self.expanded()
