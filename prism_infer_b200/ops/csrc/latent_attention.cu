@@ -233,7 +233,8 @@ __host__ __device__ constexpr size_t latent_smem_bytes(int Rc) {
 // BM = 16 MT rows of one sequence against its latents in tiles of BN keys.  Eight warps:
 //   scores    warp (kg, kh) takes 16 keys and one of KH slices of the latent; its query fragments stay in registers
 //             for the whole kernel where they fit (QREG), the slices are added when the softmax reads them
-//   softmax   BM / 8 rows per warp
+//   softmax   BM / 8 rows per warp; a row's reference maximum is only raised when a tile exceeds it by more than
+//             2^8 (the weights stay below 256), so the accumulators are rarely rescaled
 //   output    every warp accumulates Rc / 8 columns of P C in registers
 // Latent rows come by one bulk copy each, issued by one thread per row, two tiles in flight.  Tiles that hold only
 // latents of earlier steps are fetched before the previous kernel has finished.
@@ -279,11 +280,15 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
   }
   __syncthreads();
 
-  auto issue = [&](int j) {                                // threads 0 .. BN - 1: one latent row each
+  auto page_of = [&](int j) {                              // threads 0 .. BN - 1: the page of one latent row of tile j
+    const int key = j * BN + tid;
+    return tid < BN && j < te && key < kv_end ? bt[key / a.page] : -1;
+  };
+  auto issue = [&](int j, int page_id) {
     if (tid < BN && j < te) {
       const int stage = (j - tb) & 1, key = j * BN + tid;
       bf16* dst = kv_s + ((size_t)stage * BN + tid) * LD;
-      const int blk = key < kv_end ? checked_page(bt[key / a.page], a.num_blocks) : -1;
+      const int blk = checked_page(page_id, a.num_blocks);
       if (blk >= 0) {
         fence_proxy_async();
         mbar_expect_tx(&bars[stage], row_bytes);
@@ -297,8 +302,9 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
   };
   const int old_tiles = max(0, kv_len - q_len) / BN;       // tiles that hold latents of earlier steps only
   const bool pre0 = tb < old_tiles, pre1 = tb + 1 < old_tiles;
-  if (pre0) issue(tb);
-  if (pre1) issue(tb + 1);
+  const int page0 = page_of(tb), page1 = page_of(tb + 1);
+  if (pre0) issue(tb, page0);
+  if (pre1) issue(tb + 1, page1);
   if (tid < BM) {
     const int row = row0 + tid;
     m_s[tid] = -INFINITY;
@@ -316,8 +322,8 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
       mbar_arrive(&bars[2]);
     }
   }
-  if (!pre0) issue(tb);
-  if (!pre1) issue(tb + 1);
+  if (!pre0) issue(tb, page0);
+  if (!pre1) issue(tb + 1, page1);
 
   float acc[MT][NT][4];
 #pragma unroll
@@ -341,6 +347,7 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
 
   for (int j = tb; j < te; ++j) {
     const int stage = (j - tb) & 1;
+    const int next_page = page_of(j + 2);
     (void)mbar_wait(&bars[stage], ((j - tb) >> 1) & 1, 32 + stage);
     const bf16* kv = kv_s + (size_t)stage * BN * LD;
     {
@@ -398,7 +405,7 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
         mx = fmaxf(mx, v[e]);
       }
       mx = warp_max(mx);
-      const float m_old = m_s[r], m_new = fmaxf(m_old, mx);
+      const float m_old = m_s[r], m_new = mx > m_old + 8.0f ? mx : m_old;
       const float m_use = m_new == -INFINITY ? 0.0f : m_new;
       float sum = 0.0f;
 #pragma unroll
@@ -421,12 +428,14 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
       const float f0 = fac_s[m * 16 + (lane >> 2)], f1 = fac_s[m * 16 + (lane >> 2) + 8];
+      if (__any_sync(0xffffffffu, f0 != 1.0f || f1 != 1.0f)) {
 #pragma unroll
-      for (int n = 0; n < NT; ++n) {
-        acc[m][n][0] *= f0;
-        acc[m][n][1] *= f0;
-        acc[m][n][2] *= f1;
-        acc[m][n][3] *= f1;
+        for (int n = 0; n < NT; ++n) {
+          acc[m][n][0] *= f0;
+          acc[m][n][1] *= f0;
+          acc[m][n][2] *= f1;
+          acc[m][n][3] *= f1;
+        }
       }
     }
     const int col0 = warp * nt * 8;
@@ -450,7 +459,7 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
       }
     }
     __syncthreads();                 // every warp is done with this tile: its buffer takes the tile after the next
-    issue(j + 2);
+    issue(j + 2, next_page);
   }
   __syncthreads();
   if (a.nsplit > 1 && tid < BM && row0 + tid < n_rows) {
@@ -547,7 +556,7 @@ __device__ __forceinline__ void merge_splits(const LatentOutArgs& a, bf16* a_s, 
 
 __global__ void __launch_bounds__(OUT_THREADS) latent_out_kernel(const LatentOutArgs a) {
   extern __shared__ __align__(128) uint8_t smem_raw[];
-  const int Rc = a.Rc, LD = Rc + 8, pieces = Rc >> 3;
+  const int Rc = a.Rc, LD = Rc + 8;
   bf16* w_s = reinterpret_cast<bf16*>(smem_raw);   // [OUT_N][LD]
   bf16* a_s = w_s + (size_t)OUT_N * LD;            // [16][LD]
   __shared__ float wgt[16][MAX_SPLITS];
