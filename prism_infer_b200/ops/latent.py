@@ -1,6 +1,6 @@
 """Ops of models with latent attention, stacked projections and a 32-bit residual stream.
 
-Same contract as the package's other ops: CUDA tensors run the kernels of ``libprism_b200.so`` (bf16, or the
+As with the package's other ops, CUDA tensors run the kernels of ``libprism_b200.so`` (bf16, or the
 true 32-bit kernels when the tensors are fp32) and raise without them; CPU tensors run the plain-PyTorch
 statement.  Kernels: ``csrc/residual_stream.cu``, ``csrc/latent_attention.cu``, ``csrc/gemm_f32.cu``, the
 section epilogue of ``csrc/gemm_tcgen05.cu`` and the gated form of ``csrc/attention_tcgen05.cu``.

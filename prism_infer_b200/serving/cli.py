@@ -33,7 +33,7 @@ def load_engine_options(path: str | None) -> dict[str, object]:
 
 
 def build_parser() -> argparse.ArgumentParser:
-    ap = argparse.ArgumentParser(prog="prism-serve", description="Serve Qwen3-VL over HTTP / SSE")
+    ap = argparse.ArgumentParser(prog="prism-serve", description="Serve a model over HTTP / SSE")
     ap.add_argument("--model", required=True)
     ap.add_argument("--engine-config", default=None)
     ap.add_argument("--host", default="127.0.0.1")

@@ -3,7 +3,7 @@
 The report covers the Python distributions the package leans on, the in-tree kernel library (present, loadable, built
 for which sources), the CUDA devices with their free memory, the run that is planned (execution backend, KV mode,
 tensor-parallel size, page budget) and, with ``--model``, the checkpoint directory (required files, safetensors shards,
-that its configuration is a Qwen3-VL one and which sharded dimensions the tensor-parallel size has to divide).
+that its configuration names a model family of this package and which sharded dimensions the tensor-parallel size has to divide).
 Failures make the exit status non-zero; warnings do not.  ``--json`` prints the machine-readable report only.  Nothing is
 loaded onto a GPU.  The reference ships the same kind of tool as ``scripts/check_environment.py``.
 
@@ -83,18 +83,29 @@ def inspect_checkpoint(model: str | None, tp: int) -> tuple[dict[str, Any], list
             config = json.loads((path / "config.json").read_text(encoding="utf-8"))
         except (OSError, json.JSONDecodeError) as exc:
             errors.append(f"config.json cannot be read: {exc}")
-    model_type, archs = config.get("model_type"), config.get("architectures") or []
-    if config and model_type != "qwen3_vl" and not any("Qwen3VL" in str(a) for a in archs):
-        errors.append(f"config.json does not describe a Qwen3-VL model (model_type={model_type!r}, architectures={archs!r})")
-    if config and not errors:
-        from ..models.architecture import Qwen3VLArch, validate_tensor_parallel
+    model_type, archs = config.get("model_type", config.get("architecture")), config.get("architectures") or []
+    family = None
+    if config:
+        from ..models.model_registry import family_of_config, known_model_types
 
         try:
-            arch = Qwen3VLArch.from_hf_config(config)
+            family = family_of_config(config)
+        except ValueError:
+            errors.append(f"config.json does not describe a supported model ({', '.join(known_model_types())}): model_type={model_type!r}, "
+                          f"architectures={archs!r}")
+    if family is not None and not errors:
+        from ..models.architecture import validate_tensor_parallel
+
+        try:
+            arch = family.architecture_from_config(config)
             validate_tensor_parallel(arch, tp)
-            rep["text"] = {"layers": arch.text.num_layers, "hidden": arch.text.hidden_size, "heads": arch.text.num_heads,
-                           "kv_heads": arch.text.num_kv_heads, "head_dim": arch.text.head_dim, "vocabulary": arch.text.vocab_size}
-            rep["vision"] = {"depth": arch.vision.depth, "hidden": arch.vision.hidden_size, "heads": arch.vision.num_heads}
+            if family.multimodal:
+                rep["text"] = {"layers": arch.text.num_layers, "hidden": arch.text.hidden_size, "heads": arch.text.num_heads,
+                               "kv_heads": arch.text.num_kv_heads, "head_dim": arch.text.head_dim, "vocabulary": arch.text.vocab_size}
+                rep["vision"] = {"depth": arch.vision.depth, "hidden": arch.vision.hidden_size, "heads": arch.vision.num_heads}
+            else:
+                rep["text"] = {"layer_runs": arch.num_layer_runs, "vocabulary": arch.vocab_size,
+                               "cache_row": arch.kv_geometry(tp).row, "cache_planes": arch.kv_geometry(tp).planes}
         except Exception as exc:
             errors.append(f"configuration rejected: {exc}")
     rep.update({"status": "fail" if errors else "pass", "model_type": model_type, "architectures": list(archs),

@@ -29,7 +29,7 @@ CASES = {
     # the loop covers every layer and runs once
     "once": config([(mixer(4, 32, 32, 64, 0.18), 96)], vocab=160, width=64, loop=(0, 1, 1), mult=1.0),
     # the loop is the last layer
-    "tail": config([(mixer(4, 64, 64, 128, 0.125), 160), (mixer(4, 64, 64, 128, 0.1), 160)], vocab=192, width=128, loop=(1, 2, 4), mult=0.25,
+    "tail": config([(mixer(4, 72, 72, 136, 0.12), 160), (mixer(4, 72, 72, 136, 0.1), 160)], vocab=192, width=128, loop=(1, 2, 4), mult=0.25,
                    cap=20.0),
     # no loop, wide heads (no square tensor-core path), wide latent
     "wide": config([(mixer(2, 160, 96, 320, 0.08), 64), (mixer(9, 48, 48, 600, 0.14), 0)], vocab=128, width=112),

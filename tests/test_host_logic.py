@@ -654,7 +654,7 @@ def test_environment_check_reports_checkpoint_and_plan_problems(tmp_path, capsys
     (bad / "config.json").write_text(json.dumps({"model_type": "llama", "architectures": ["LlamaForCausalLM"]}))
     rc = ce.main(["--allow-cpu", "--model", str(bad), "--json"])
     rep = json.loads(capsys.readouterr().out)
-    assert rc == 1 and any("no *.safetensors" in e for e in rep["errors"]) and any("does not describe a Qwen3-VL" in e for e in rep["errors"])
+    assert rc == 1 and any("no *.safetensors" in e for e in rep["errors"]) and any("does not describe a supported model" in e for e in rep["errors"])
     assert ce.main(["--allow-cpu", "--model", str(tmp_path / "nowhere"), "--json"]) == 1
     capsys.readouterr()
     assert ce.main(["--allow-cpu", "--model", "random:nope", "--json"]) == 1

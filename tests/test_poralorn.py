@@ -86,6 +86,28 @@ def test_loading_checks_names_and_shapes(model):
     m.load({**w, "unknown.tensor": torch.zeros(3)}.items())
 
 
+def test_environment_check_knows_the_family(model):
+    from prism_infer_b200.utils.check_environment import inspect_checkpoint
+
+    rep, errors, _ = inspect_checkpoint(model("uneven")[3], 1)
+    assert rep["status"] == "pass" and not errors and rep["text"]["layer_runs"] == 5
+    assert inspect_checkpoint(model("uneven")[3], 2)[1]
+
+
+def test_partial_kernel_library(tmp_path, monkeypatch):
+    """Without an up-to-date full library only the family's own kernel units are compiled, into a library of their own."""
+    from prism_infer_b200.models.model_registry import resolve_model_family
+    from prism_infer_b200.ops import build
+
+    units = resolve_model_family("poralorn").kernel_units
+    assert {u + ".cu" for u in units} <= set(build._sources())
+    asked = {}
+    monkeypatch.setattr(build, "build", lambda **kw: asked.update(kw) or kw["target"])
+    monkeypatch.setattr(build, "BUILD", str(tmp_path))
+    monkeypatch.setattr(build, "LIB", str(tmp_path / "absent.so"))
+    assert build.ensure("poralorn", units) == build.partial_library("poralorn") and asked["units"] == units
+
+
 def test_cache_geometry():
     arch = PoralornArch.from_hf_config(cases.CASES["uneven"])
     g = arch.kv_geometry()
@@ -279,6 +301,21 @@ def test_greedy_generation(model, options, backend):
     if backend[0] != "cpu":
         llm.check_device_status()
         assert llm.graph_metadata()["decode_steps"]["graph_batch_sizes"]
+    llm.exit()
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["auto", "float32"])
+def test_cache_sized_from_free_memory(cuda_device, dtype):
+    """Default cache sizing (a measured warm-up prefill) and graph decode on production widths."""
+    llm = LLM("random:poralorn-8b-like-4layer" if dtype == "auto" else "random:poralorn-tiny", dtype=dtype, gpu_memory_utilization=0.3,
+              max_num_seqs=8, max_num_batched_tokens=2048, cpu_kv_cache_ratio=0.0)
+    sizing = llm.graph_metadata()["kv_sizing"]
+    assert sizing["budget_bytes"] > 0 and llm.scheduler.block_manager.gpu.num_blocks > 100
+    prompts = [cases.tokens(n, 200, seed=n) for n in (700, 3, 41)]
+    together = llm.generate(prompts, SamplingParams(temperature=0.0, max_tokens=6, ignore_eos=True), use_tqdm=False)
+    assert all(len(o["token_ids"]) == 6 for o in together)
+    llm.check_device_status()
     llm.exit()
 
 
