@@ -6,7 +6,8 @@ with packed staging ``:1219-1313``).
 B200-specific choices:
 
 * One KV allocation ``[planes, L, pages, Hkv/tp, page, D]`` (+ fp32 scales; two planes for keys and
-  values, one for a shared latent; L counts layer executions, a looped layer has one slab per pass),
+  values, one where a token has a single row per layer, whose width may then differ from layer to layer;
+  L counts layer executions, a looped layer has one slab per pass),
   sized from free HBM, head-major inside a page so each (page, head) is one contiguous 32 KB run of E4M3 bytes.
 * Decode runs as one CUDA graph per batch bucket (1, 2, 4, 8, 16, 32, ...).  A single packed
   pinned host buffer is copied to the device by a memcpy node *inside* the graph, and the
@@ -215,7 +216,7 @@ class ModelRunner:
     def _new_cache(self, blocks: int, device, pin_memory: bool = False) -> ops.KVCache:
         g = self.config.arch.kv_geometry(self.comm.size)
         return ops.KVCache(g.layers, blocks, g.heads, self.page, g.row, self.kv_mode, device, dtype=self.dtype,
-                           pin_memory=pin_memory, planes=g.planes)
+                           pin_memory=pin_memory, planes=g.planes, rows=g.rows)
 
     GRAPH_POOL_RESERVE = 1 << 30  # decode-graph pools, vision-tower activations and allocator slack
 

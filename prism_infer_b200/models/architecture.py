@@ -6,7 +6,8 @@ dataclasses below once and every later layer (weight sharding, kernels, KV sizin
 reads these.  Mirrors the contract of the reference's
 ``prism_infer/models/qwen3_vl_architecture.py:117-428`` (canonical 8B constants at
 ``:18-44``): interleaved M-RoPE only, no attention bias, SiLU text MLP, GELU-tanh
-vision MLP.  ``PoralornArch`` (end of file) is the text-only looped latent-attention family.
+vision MLP.  ``PoralornArch`` and ``DolidraArch`` (end of file) are text-only looped families: latent attention, and
+windowed attention with a mixture of experts.
 
 What the engine asks of any architecture, whatever its family: ``model_type``, ``multimodal``,
 ``vocab_size``, ``max_positions`` (``None``: unbounded), ``num_layer_runs``, ``eos_token_id``, the
@@ -16,6 +17,7 @@ visual token ids (-1 where there are none), ``reserved_token_ids`` and ``kv_geom
 from __future__ import annotations
 
 import json
+import math
 import os
 from dataclasses import asdict, dataclass, field
 from typing import Any, Mapping
@@ -25,15 +27,23 @@ SUPPORTED_MODEL_TYPES = frozenset({"qwen3_vl"})
 
 @dataclass(frozen=True)
 class KVGeometry:
-    """Shape of one rank's paged cache: ``planes`` slabs per layer run (2: keys and values, 1: a shared
-    latent), each ``[pages, heads, page, row]``."""
+    """Shape of one rank's paged cache: ``planes`` slabs per layer run (2: keys and values, 1: one row per token,
+    a shared latent or all heads' keys and values), each ``[pages, heads, page, row]``.  ``rows`` gives every layer
+    run a row width of its own (single plane, one head)."""
 
     planes: int
     layers: int
     heads: int
     row: int
+    rows: tuple[int, ...] = ()
+
+    def __post_init__(self) -> None:
+        if self.rows and (self.planes != 1 or self.heads != 1 or len(self.rows) != self.layers or self.row != max(self.rows)):
+            raise ValueError("row widths per layer run need a single-plane, single-head cache and one width per layer run")
 
     def bytes_per_page(self, page: int, element_bytes: int, scaled: bool = False) -> int:
+        if self.rows:
+            return sum(self.rows) * page * element_bytes
         rows = self.planes * self.layers * self.heads * page
         return rows * self.row * element_bytes + (rows * 4 if scaled else 0)
 
@@ -365,9 +375,9 @@ def validate_tensor_parallel(arch: Any, tp: int) -> None:
     """Every sharded dimension must divide evenly (reference ``engine/llm_engine.py:117-143``)."""
     if tp < 1:
         raise ValueError("tensor_parallel_size must be >= 1")
-    if isinstance(arch, PoralornArch):
+    if isinstance(arch, LoopedStack):
         if tp != 1:
-            raise ValueError("the Poralorn family runs on one GPU (tensor_parallel_size 1)")
+            raise ValueError(f"the {type(arch).__name__.removesuffix('Arch')} family runs on one GPU (tensor_parallel_size 1)")
         return
     t = arch.text
     for name, value in (
@@ -379,6 +389,74 @@ def validate_tensor_parallel(arch: Any, tp: int) -> None:
     ):
         if value % tp:
             raise ValueError(f"tensor_parallel_size {tp} does not divide text {name}={value}")
+
+
+# ----------------------------------------------------------------------- looped layer stacks
+@dataclass(frozen=True)
+class LayerRun:
+    """One execution of a layer.  ``loop_pass`` is the pass number on the first layer of a pass of the looped
+    section (where a loop input may be formed) and ``None`` elsewhere."""
+
+    layer: int
+    loop_pass: int | None = None
+
+
+class LoopedStack:
+    """What the text-only families with a looped section share: layers ``loop_start .. loop_stop - 1`` run
+    ``loop_times`` times in a row (0: no looped section), every run with its own cache slab."""
+
+    multimodal = False
+    image_token_id = -1
+    video_token_id = -1
+
+    def check_stack(self) -> None:
+        if self.vocab_size < 1 or self.width < 1 or not self.layers:
+            raise ValueError("vocab, width and layers must be given")
+        if self.loop_times < 0 or (self.has_loop and not 0 <= self.loop_start < self.loop_stop <= len(self.layers)):
+            raise ValueError(f"loop {self.loop_start} .. {self.loop_stop} x {self.loop_times} does not fit {len(self.layers)} layers")
+        if self.norm_eps < 0:
+            raise ValueError("norm eps must not be negative")
+
+    @property
+    def has_loop(self) -> bool:
+        return self.loop_times > 0
+
+    @property
+    def max_positions(self) -> int | None:
+        return None                  # nothing bounds a position
+
+    @property
+    def reserved_token_ids(self) -> tuple[int, ...]:
+        return ()
+
+    def layer_runs(self) -> tuple[LayerRun, ...]:
+        """Every layer execution in order; run ``i`` owns cache slab ``i``."""
+        if not self.has_loop:
+            return tuple(LayerRun(i) for i in range(len(self.layers)))
+        runs = [LayerRun(i) for i in range(self.loop_start)]
+        for t in range(self.loop_times):
+            runs += [LayerRun(i, t if i == self.loop_start else None) for i in range(self.loop_start, self.loop_stop)]
+        return tuple(runs + [LayerRun(i) for i in range(self.loop_stop, len(self.layers))])
+
+    @property
+    def num_layer_runs(self) -> int:
+        return len(self.layer_runs())
+
+
+def _field_reader(family: str):
+    """``need(dictionary, key, where)``: a required field of a family's ``config.json``."""
+
+    def need(d: Mapping[str, Any], key: str, where: str = "config") -> Any:
+        if key not in d:
+            raise ValueError(f"{family} {where} is missing required field {key}")
+        return d[key]
+
+    return need
+
+
+def _loop_fields(cfg: Mapping[str, Any], need) -> dict[str, int]:
+    loop = cfg.get("loop") or {}
+    return {f"loop_{k}": int(need(loop, k, "loop")) if loop else 0 for k in ("start", "stop", "times")}
 
 
 # ------------------------------------------------------------------------------- Poralorn
@@ -406,16 +484,7 @@ class PoralornLayer:
 
 
 @dataclass(frozen=True)
-class LayerRun:
-    """One execution of a layer.  ``loop_pass`` is the pass number on the first layer of a pass of the looped
-    section (where the loop input is formed) and ``None`` elsewhere."""
-
-    layer: int
-    loop_pass: int | None = None
-
-
-@dataclass(frozen=True)
-class PoralornArch:
+class PoralornArch(LoopedStack):
     vocab_size: int
     width: int
     layers: tuple[PoralornLayer, ...]
@@ -428,44 +497,12 @@ class PoralornArch:
     eos_token_id: int = -1
     model_type: str = "poralorn"
 
-    multimodal = False
-    image_token_id = -1
-    video_token_id = -1
-
     def __post_init__(self) -> None:
-        if self.vocab_size < 1 or self.width < 1 or not self.layers:
-            raise ValueError("vocab, width and layers must be given")
-        if self.loop_times < 0 or (self.has_loop and not 0 <= self.loop_start < self.loop_stop <= len(self.layers)):
-            raise ValueError(f"loop {self.loop_start} .. {self.loop_stop} x {self.loop_times} does not fit {len(self.layers)} layers")
-        if self.norm_eps < 0 or self.logit_softcap < 0:
-            raise ValueError("norm eps and logit_softcap must not be negative")
+        self.check_stack()
+        if self.logit_softcap < 0:
+            raise ValueError("logit_softcap must not be negative")
 
     # ---- what the engine reads of every family ---------------------------------
-    @property
-    def has_loop(self) -> bool:
-        return self.loop_times > 0
-
-    @property
-    def max_positions(self) -> int | None:
-        return None                  # no position enters the computation except through the causal order
-
-    @property
-    def reserved_token_ids(self) -> tuple[int, ...]:
-        return ()
-
-    def layer_runs(self) -> tuple[LayerRun, ...]:
-        """Every layer execution in order; run ``i`` owns cache slab ``i``."""
-        if not self.has_loop:
-            return tuple(LayerRun(i) for i in range(len(self.layers)))
-        runs = [LayerRun(i) for i in range(self.loop_start)]
-        for t in range(self.loop_times):
-            runs += [LayerRun(i, t if i == self.loop_start else None) for i in range(self.loop_start, self.loop_stop)]
-        return tuple(runs + [LayerRun(i) for i in range(self.loop_stop, len(self.layers))])
-
-    @property
-    def num_layer_runs(self) -> int:
-        return len(self.layer_runs())
-
     @property
     def latent_row(self) -> int:
         """Elements of one cached latent row: the widest latent, rounded up to whole 64-element tiles."""
@@ -515,12 +552,7 @@ class PoralornArch:
     @classmethod
     def from_hf_config(cls, cfg: Mapping[str, Any]) -> "PoralornArch":
         """From the ``config.json`` dictionary."""
-
-        def need(d: Mapping[str, Any], key: str, where: str = "config") -> Any:
-            if key not in d:
-                raise ValueError(f"Poralorn {where} is missing required field {key}")
-            return d[key]
-
+        need = _field_reader("Poralorn")
         layers = []
         for i, entry in enumerate(need(cfg, "layers")):
             where = f"layer {i}"
@@ -534,11 +566,8 @@ class PoralornArch:
             if mlp is not None and mlp.get("kind") != "dense":
                 raise ValueError(f"Poralorn {where}: unsupported feed-forward {mlp.get('kind')!r}")
             layers.append(PoralornLayer(mixer, int(need(mlp, "ff", where)) if mlp is not None else 0))
-        loop = cfg.get("loop") or {}
         return cls(
-            vocab_size=int(need(cfg, "vocab")), width=int(need(cfg, "width")), layers=tuple(layers),
-            loop_start=int(need(loop, "start", "loop")) if loop else 0, loop_stop=int(need(loop, "stop", "loop")) if loop else 0,
-            loop_times=int(need(loop, "times", "loop")) if loop else 0,
+            vocab_size=int(need(cfg, "vocab")), width=int(need(cfg, "width")), layers=tuple(layers), **_loop_fields(cfg, need),
             norm_eps=float(need(need(cfg, "norm"), "eps", "norm")), residual_mult=float(need(cfg, "residual_mult")),
             logit_softcap=float(cfg.get("logit_softcap") or 0.0))
 
@@ -567,3 +596,266 @@ class PoralornArch:
         mixer = LatentAttentionArch(heads, dim, dim, kv_rank, dim ** -0.5)
         return cls(vocab_size=vocab_size, width=width, layers=(PoralornLayer(mixer, ff),) * layers, residual_mult=0.5,
                    logit_softcap=30.0)
+
+
+# -------------------------------------------------------------------------------- Dolidra
+@dataclass(frozen=True)
+class RotaryArch:
+    """Rotation of the first ``dims`` columns of a head (pairs ``(i, i + dims / 2)``).  ``factor`` > 0 rescales the
+    frequencies by wavelength: long ones are divided by it, those below ``original / high`` stay, a ramp between."""
+
+    base: float
+    dims: int
+    factor: float = 0.0
+    low: float = 0.0
+    high: float = 0.0
+    original: float = 0.0
+
+    def __post_init__(self) -> None:
+        if self.dims < 0 or self.dims % 2:
+            raise ValueError(f"rotary dims must be even, got {self.dims}")
+
+    def inv_freq(self) -> list[float]:
+        out = []
+        for i in range(self.dims // 2):
+            f = self.base ** (-2.0 * i / self.dims)
+            if self.factor > 0.0:
+                wavelength = 2.0 * math.pi / f
+                if wavelength > self.original / self.low:
+                    f /= self.factor
+                elif wavelength >= self.original / self.high:
+                    keep = (self.original / wavelength - self.low) / (self.high - self.low)
+                    f = (1.0 - keep) * f / self.factor + keep * f
+            out.append(f)
+        return out
+
+
+@dataclass(frozen=True)
+class WindowAttentionArch:
+    """One windowed attention mixer.  ``maps`` 2: differential attention (two maps over the same values, the second
+    subtracted); ``qk_norm``: RMS norm over the whole query and the whole key projection; ``gate``: one sigmoid output
+    gate per head; a query sees the ``window`` newest positions (its own included) and the first ``keep_first``."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotaryArch
+    window: int
+    keep_first: int = 0
+    maps: int = 1
+    diff: float = 0.0
+    bias: bool = False
+    qk_norm: bool = False
+    gate: bool = False
+
+    def __post_init__(self) -> None:
+        for name in ("heads", "kv_heads", "dim", "vdim", "window"):
+            if getattr(self, name) < 1:
+                raise ValueError(f"windowed attention: {name} must be positive")
+        if self.heads % self.kv_heads:
+            raise ValueError(f"windowed attention: {self.heads} query heads over {self.kv_heads} key/value heads")
+        if self.rot.dims > self.dim or self.keep_first < 0 or self.maps not in (1, 2):
+            raise ValueError("windowed attention: rot.dims must not exceed dim, keep_first must not be negative, maps is 1 or 2")
+
+    @property
+    def dq(self) -> int:
+        """Key width of one map of one head, padded to whole tensor-core steps; ``dv`` likewise for values."""
+        return -(-self.dim // 16) * 16
+
+    @property
+    def dv(self) -> int:
+        return -(-self.vdim // 16) * 16
+
+    @property
+    def cache_row(self) -> int:
+        """Elements a token's keys and values take: ``[key heads x maps x dq | value heads x dv]``."""
+        return self.kv_heads * (self.maps * self.dq + self.dv)
+
+
+@dataclass(frozen=True)
+class MixtureArch:
+    """Routed experts: ``top`` of ``experts`` gated feed-forwards of width ``ff`` per token, and one of width
+    ``shared_ff`` (0: none) for every token."""
+
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0
+
+    def __post_init__(self) -> None:
+        if self.experts < 1 or not 1 <= self.top <= self.experts or self.ff < 1 or self.shared_ff < 0:
+            raise ValueError(f"mixture of experts: {self.top} of {self.experts} experts of width {self.ff}, shared {self.shared_ff}")
+
+
+@dataclass(frozen=True)
+class DolidraLayer:
+    mixer: WindowAttentionArch
+    ff: int = 0                      # width of a dense feed-forward
+    moe: MixtureArch | None = None   # or a mixture; neither: the layer has no feed-forward
+
+    @property
+    def has_ff(self) -> bool:
+        return self.ff > 0 or self.moe is not None
+
+
+@dataclass(frozen=True)
+class DolidraArch(LoopedStack):
+    vocab_size: int
+    width: int
+    layers: tuple[DolidraLayer, ...]
+    side_dim: int                    # width of a layer's part of the per-token side table
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 0
+    norm_eps: float = 1.0e-5
+    eos_token_id: int = -1
+    model_type: str = "dolidra"
+
+    def __post_init__(self) -> None:
+        self.check_stack()
+        if self.side_dim < 1:
+            raise ValueError("token_side.dim must be positive")
+
+    def kv_geometry(self, tp: int = 1) -> KVGeometry:
+        rows = tuple(self.layers[r.layer].mixer.cache_row for r in self.layer_runs())
+        return KVGeometry(1, len(rows), 1, max(rows), rows)
+
+    # ---- checkpoint --------------------------------------------------------------
+    def weight_shapes(self) -> dict[str, tuple[int, ...]]:
+        W, D = self.width, self.side_dim
+        s: dict[str, tuple[int, ...]] = {"embed": (self.vocab_size, W), "side.embed": (self.vocab_size, len(self.layers) * D)}
+
+        def ff(prefix: str, width: int) -> None:
+            s[f"{prefix}.gate"] = s[f"{prefix}.up"] = (width, W)
+            s[f"{prefix}.down"] = (W, width)
+
+        for i, l in enumerate(self.layers):
+            m, p = l.mixer, f"l{i}"
+            for n in ("norm1", "norm1b") + (("norm2", "norm2b") if l.has_ff else ()):
+                s[f"{p}.{n}"] = (W,)
+            sizes = {"q": m.heads * m.maps * m.dim, "k": m.kv_heads * m.maps * m.dim, "v": m.kv_heads * m.vdim}
+            for n, rows in sizes.items():
+                s[f"{p}.mix.{n}"] = (rows, W)
+                if m.bias:
+                    s[f"{p}.mix.{n}.b"] = (rows,)
+            if m.maps == 2:
+                for n in ("lq1", "lk1", "lq2", "lk2"):
+                    s[f"{p}.mix.{n}"] = (m.dim,)
+            if m.qk_norm:
+                s[f"{p}.mix.q.norm"], s[f"{p}.mix.k.norm"] = (sizes["q"],), (sizes["k"],)
+            if m.gate:
+                s[f"{p}.mix.g"] = (m.heads, W)
+            s[f"{p}.mix.o"] = (W, m.heads * m.vdim)
+            if l.moe is not None:
+                s[f"{p}.mlp.router"] = (l.moe.experts, W)
+                for e in range(l.moe.experts):
+                    ff(f"{p}.mlp.e{e}", l.moe.ff)
+                if l.moe.shared_ff:
+                    ff(f"{p}.mlp.shared", l.moe.shared_ff)
+            elif l.ff:
+                ff(f"{p}.mlp", l.ff)
+            s[f"{p}.side.gate"], s[f"{p}.side.proj"], s[f"{p}.side.norm"] = (D, W), (W, D), (W,)
+        s["final.norm"] = (W,)
+        s["head"] = (self.vocab_size, W)
+        return s
+
+    @staticmethod
+    def init_kind(name: str) -> str:
+        """How random initialisation draws a tensor: ``norm``, ``bias``, ``embedding`` or ``matrix``."""
+        last = name.rsplit(".", 1)[-1]
+        if last.startswith("norm"):
+            return "norm"
+        if last in ("b", "lq1", "lk1", "lq2", "lk2"):
+            return "bias"
+        return "embedding" if name in ("embed", "side.embed") else "matrix"
+
+    # ---- factories ---------------------------------------------------------------
+    @classmethod
+    def from_hf_config(cls, cfg: Mapping[str, Any]) -> "DolidraArch":
+        """From the ``config.json`` dictionary."""
+        need = _field_reader("Dolidra")
+        layers = []
+        for i, entry in enumerate(need(cfg, "layers")):
+            where = f"layer {i}"
+            kind = need(entry, "type", where)
+            if kind not in ("attention", "attention_2"):
+                raise ValueError(f"Dolidra {where}: unsupported mixer {kind!r}")
+            m = need(entry, "mixer", where)
+            rot, mask = need(m, "rot", where), need(m, "mask", where)
+            scaling = rot.get("scaling") or {}
+            rotary = RotaryArch(float(need(rot, "base", where)), int(need(rot, "dims", where)),
+                                *(float(need(scaling, k, where)) for k in ("factor", "low", "high", "original")) if scaling else ())
+            common = dict(heads=int(need(m, "heads", where)), kv_heads=int(need(m, "kv_heads", where)), dim=int(need(m, "dim", where)),
+                          vdim=int(need(m, "vdim", where)), scale=float(need(m, "scale", where)), rot=rotary,
+                          window=int(need(mask, "size", where)), keep_first=int(mask.get("keep_first") or 0))
+            if kind == "attention":
+                mixer = WindowAttentionArch(**common, maps=2, diff=float(need(m, "diff", where)), bias=True)
+            else:
+                mixer = WindowAttentionArch(**common, qk_norm=True, gate=True)
+            mlp = entry.get("mlp")
+            if mlp is None:
+                layers.append(DolidraLayer(mixer))
+            elif mlp.get("kind") == "dense":
+                layers.append(DolidraLayer(mixer, ff=int(need(mlp, "ff", where))))
+            elif mlp.get("kind") == "moe":
+                router, shared = need(mlp, "router", where), mlp.get("shared") or {}
+                layers.append(DolidraLayer(mixer, moe=MixtureArch(
+                    int(need(router, "experts", where)), int(need(router, "top", where)), int(need(need(mlp, "expert", where), "ff", where)),
+                    int(need(shared, "ff", where)) if shared else 0)))
+            else:
+                raise ValueError(f"Dolidra {where}: unsupported feed-forward {mlp.get('kind')!r}")
+        return cls(vocab_size=int(need(cfg, "vocab")), width=int(need(cfg, "width")), layers=tuple(layers),
+                   side_dim=int(need(need(cfg, "token_side"), "dim", "token_side")), **_loop_fields(cfg, need),
+                   norm_eps=float(need(need(cfg, "norm"), "eps", "norm")))
+
+    def to_hf_config(self) -> dict[str, Any]:
+        """The ``config.json`` dictionary ``from_hf_config`` reads."""
+
+        def layer(l: DolidraLayer) -> dict[str, Any]:
+            m, r = l.mixer, l.mixer.rot
+            rot: dict[str, Any] = {"base": r.base, "dims": r.dims}
+            if r.factor > 0.0:
+                rot["scaling"] = {"factor": r.factor, "low": r.low, "high": r.high, "original": r.original}
+            mixer: dict[str, Any] = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "rot": rot,
+                                     "mask": {"size": m.window}}
+            if m.maps == 2:
+                mixer["diff"] = m.diff
+            if m.keep_first or m.maps == 1:
+                mixer["mask"]["keep_first"] = m.keep_first
+            mlp: dict[str, Any] | None = {"kind": "dense", "ff": l.ff} if l.ff else None
+            if l.moe is not None:
+                mlp = {"kind": "moe", "router": {"experts": l.moe.experts, "top": l.moe.top}, "expert": {"ff": l.moe.ff}}
+                if l.moe.shared_ff:
+                    mlp["shared"] = {"ff": l.moe.shared_ff}
+            return {"type": "attention" if m.maps == 2 else "attention_2", "mixer": mixer, "mlp": mlp}
+
+        out: dict[str, Any] = {"architecture": "Dolidra", "vocab": self.vocab_size, "width": self.width, "norm": {"eps": self.norm_eps},
+                               "token_side": {"dim": self.side_dim}, "layers": [layer(l) for l in self.layers]}
+        if self.has_loop:
+            out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return out
+
+    @classmethod
+    def tiny(cls) -> "DolidraArch":
+        """The small CPU test model: every size different, both mixers, all three kinds of feed-forward, five layer runs."""
+        scaled = RotaryArch(20000.0, 24, 4.0, 1.0, 4.0, 64.0)
+        diff = WindowAttentionArch(3, 1, 24, 40, 0.2, scaled, window=19, maps=2, diff=0.45, bias=True)
+        kept = WindowAttentionArch(4, 2, 32, 16, 0.17, RotaryArch(5000.0, 8), window=11, keep_first=3, qk_norm=True, gate=True)
+        return cls(vocab_size=310, width=144, side_dim=20, layers=(DolidraLayer(diff, ff=176), DolidraLayer(kept, moe=MixtureArch(5, 2, 48, 72)),
+                                                                   DolidraLayer(diff)), loop_start=1, loop_stop=2, loop_times=3)
+
+    @classmethod
+    def like_8b(cls, layers: int = 4, *, width: int = 4096, heads: int = 16, kv_heads: int = 4, dim: int = 128, window: int = 1024,
+                ff: int = 12288, experts: int = 32, top: int = 4, expert_ff: int = 1536, side_dim: int = 256,
+                vocab_size: int = 151_936) -> "DolidraArch":
+        """Layers with the widths of an 8B-class decoder (measurement model; random weights): differential layers with
+        dense and with routed feed-forwards in turn, every fourth layer with kept first tokens and twice the heads."""
+        rot = RotaryArch(1.0e6, dim, 8.0, 1.0, 4.0, 8192.0)
+        diff = WindowAttentionArch(heads, kv_heads, dim, dim, dim ** -0.5, rot, window=window, maps=2, diff=0.6, bias=True)
+        kept = WindowAttentionArch(2 * heads, 2 * kv_heads, dim, dim, dim ** -0.5, RotaryArch(1.0e6, dim), window=window, keep_first=16,
+                                   qk_norm=True, gate=True)
+        moe = MixtureArch(experts, top, expert_ff, expert_ff)
+        kinds = [DolidraLayer(kept if i % 4 == 2 else diff, **({"moe": moe} if i % 2 else {"ff": ff})) for i in range(layers)]
+        return cls(vocab_size=vocab_size, width=width, layers=tuple(kinds), side_dim=side_dim)

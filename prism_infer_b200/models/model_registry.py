@@ -56,12 +56,28 @@ def _poralorn_random() -> dict[str, Callable[[], Any]]:
             "poralorn-8b-like-4layer": PoralornArch.like_8b}
 
 
+def _dolidra_arch(cfg: Any):
+    from .architecture import DolidraArch
+
+    return DolidraArch.from_hf_config(cfg)
+
+
+def _dolidra_random() -> dict[str, Callable[[], Any]]:
+    from .architecture import DolidraArch
+
+    return {"dolidra-tiny": DolidraArch.tiny, "dolidra-8b-like": lambda: DolidraArch.like_8b(36),
+            "dolidra-8b-like-4layer": DolidraArch.like_8b}
+
+
 _FAMILIES = {
     "qwen3_vl": ModelFamily("qwen3_vl", True, _qwen3_vl_arch, "prism_infer_b200.models.qwen3_vl:Qwen3VLModel", _qwen3_vl_random()),
     "poralorn": ModelFamily("poralorn", False, _poralorn_arch, "prism_infer_b200.models.poralorn:PoralornModel", _poralorn_random(),
                             float32_on_cuda=True, kv_modes=(0,),
                             kernel_units=("gemm_tcgen05", "gemm_f32", "attention_tcgen05", "latent_attention", "residual_stream",
                                           "kv_ops", "sampler")),
+    "dolidra": ModelFamily("dolidra", False, _dolidra_arch, "prism_infer_b200.models.dolidra:DolidraModel", _dolidra_random(),
+                           float32_on_cuda=True, kv_modes=(0,),
+                           kernel_units=("gemm_tcgen05", "gemm_f32", "window_attention", "moe", "residual_stream", "kv_ops", "sampler")),
 }
 
 

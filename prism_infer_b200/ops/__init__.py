@@ -140,8 +140,16 @@ def effective_splits(k: int, splits: int) -> int:
     return (kb + per - 1) // per
 
 
+def glu_act(z: torch.Tensor, act: str) -> torch.Tensor:
+    return F.gelu(z, approximate="tanh") if act == "gelu_tanh" else F.silu(z)
+
+
+GLU_ACTS = {"silu": 1, "gelu_tanh": 2}  # 0: silu with the rounding points of the eager graph (gate_up_swiglu)
+
+
 def gate_up_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, *, bn: int = 0) -> torch.Tensor:
-    """``silu(x @ Wg.T) * (x @ Wu.T)`` with ``w_gate_up = [Wg ; Wu]`` of shape ``[2I, K]``."""
+    """``silu(x @ Wg.T) * (x @ Wu.T)`` with ``w_gate_up = [Wg ; Wu]`` of shape ``[2I, K]``; gate, up and silu are each
+    rounded to the tensor's type."""
     T, K = x.shape
     I = w_gate_up.shape[0] // 2
     if not x.is_cuda:
@@ -153,10 +161,35 @@ def gate_up_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional[torch
         return y
     if out is None:
         out = torch.empty((T, I), dtype=torch.bfloat16, device=x.device)
+    _gate_up(x, w_gate_up, out, 0, bn)
+    return out
+
+
+def _gate_up(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int, bn: int = 0) -> None:
+    I = w.shape[0] // 2
     native.call(
-        "prism_gemm_wx", _p(w_gate_up), _p(x), _p(out), I, T, K, w_gate_up.stride(0), x.stride(0), out.stride(0),
-        2 * I, None, None, 0, 0, 1, I, 1, 0, 0, bn, 0, _s(), _pdl(),
+        "prism_gemm_wx", _p(w), _p(x), _p(out), I, x.shape[0], x.shape[1], w.stride(0), x.stride(0), out.stride(0),
+        2 * I, None, None, 0, act, 1, I, 1, 0, 0, bn, 0, _s(), _pdl(),
     )
+
+
+def gate_up_glu(x: torch.Tensor, w_gate_up: torch.Tensor, act: str) -> torch.Tensor:
+    """``act(x @ Wg.T) * (x @ Wu.T)``, activation and product in 32-bit; ``act`` is ``silu`` or ``gelu_tanh``.  bf16 or
+    (true 32-bit kernels) fp32."""
+    T = x.shape[0]
+    I = w_gate_up.shape[0] // 2
+    if not x.is_cuda:
+        gu = F.linear(x.float(), w_gate_up.float())
+        return (glu_act(gu[:, :I], act) * gu[:, I:]).to(x.dtype)
+    assert x.dtype == w_gate_up.dtype and x.stride(1) == 1 and w_gate_up.stride(1) == 1
+    out = torch.empty((T, I), dtype=x.dtype, device=x.device)
+    if x.dtype == torch.float32:
+        gu = torch.empty((T, 2 * I), dtype=torch.float32, device=x.device)
+        native.call("prism_gemm_f32", _p(w_gate_up), _p(x), _p(gu), 2 * I, T, x.shape[1], w_gate_up.stride(0), x.stride(0), 2 * I,
+                    None, 0, None, None, None, 0.0, _s(), _pdl())
+        native.call("prism_glu_f32", _p(gu), _p(out), T, I, GLU_ACTS[act], _s(), _pdl())
+    else:
+        _gate_up(x, w_gate_up, out, GLU_ACTS[act])
     return out
 
 
@@ -279,12 +312,15 @@ def layernorm(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float) -> 
 class KVCache:
     """One allocation for every layer: payload ``[planes, L, blocks, Hkv, page, D]`` (+ scales).
 
-    ``planes`` is 2 (keys and values) or 1 (one shared latent row per token, from which keys and values
-    are linear; ``Hkv`` is then 1 and ``latent(layer)`` the pages)."""
+    ``planes`` is 2 (keys and values) or 1 (one row per token: a shared latent, or all heads' keys and values side
+    by side; ``Hkv`` is then 1 and ``token_rows(layer)`` the pages).  ``rows`` gives every layer of a single-plane
+    cache a row width of its own; the payload is then flat, one ``[blocks, page, rows[l]]`` slab after another."""
 
     def __init__(self, num_layers: int, num_blocks: int, num_kv_heads: int, page: int, head_dim: int,
-                 mode: int, device, dtype: torch.dtype = torch.bfloat16, pin_memory: bool = False, planes: int = 2):
+                 mode: int, device, dtype: torch.dtype = torch.bfloat16, pin_memory: bool = False, planes: int = 2,
+                 rows: Sequence[int] = ()):
         self.planes = planes
+        self.rows = tuple(int(r) for r in rows)
         self.num_layers, self.num_blocks, self.num_kv_heads = num_layers, num_blocks, num_kv_heads
         self.page, self.head_dim, self.mode = page, head_dim, mode
         shape = (planes, num_layers, num_blocks, num_kv_heads, page, head_dim)
@@ -292,6 +328,13 @@ class KVCache:
         kw = dict(device=device)
         if pin_memory:
             kw = dict(device="cpu", pin_memory=True)
+        if self.rows:
+            assert planes == 1 and num_kv_heads == 1 and mode == KV_BF16 and len(self.rows) == num_layers
+            starts = [0]
+            for r in self.rows:
+                starts.append(starts[-1] + num_blocks * page * r)
+            shape = (starts[-1],)
+            self._starts = starts
         self.payload = torch.zeros(shape, dtype=pdtype, **kw)
         self.scales = torch.zeros(shape[:-1], dtype=torch.float32, **kw) if mode == KV_FP8_SCALED else None
 
@@ -301,10 +344,25 @@ class KVCache:
     def v(self, layer: int) -> torch.Tensor:
         return self.payload[1, layer]
 
-    def latent(self, layer: int) -> torch.Tensor:
-        """``[blocks, page, D]`` latent rows of one layer run (single-plane caches)."""
+    def token_rows(self, layer: int) -> torch.Tensor:
+        """``[blocks, page, D]`` rows of one layer run (single-plane caches)."""
         assert self.planes == 1 and self.num_kv_heads == 1
+        if self.rows:
+            return self.payload[self._starts[layer]:self._starts[layer + 1]].view(self.num_blocks, self.page, self.rows[layer])
         return self.payload[0, layer, :, 0]
+
+    latent = token_rows
+
+    def slab_groups(self) -> list[torch.Tensor]:
+        """The payload as ``[slabs, blocks, Hkv, page, D]`` views, one per run of layers with equal rows."""
+        if not self.rows:
+            return [self.payload.view(-1, *self.payload.shape[2:])]
+        out, lo = [], 0
+        for hi in range(1, self.num_layers + 1):
+            if hi == self.num_layers or self.rows[hi] != self.rows[lo]:
+                out.append(self.payload[self._starts[lo]:self._starts[hi]].view(hi - lo, self.num_blocks, 1, self.page, self.rows[lo]))
+                lo = hi
+        return out
 
     def k_scale(self, layer: int) -> Optional[torch.Tensor]:
         return None if self.scales is None else self.scales[0, layer]
@@ -317,6 +375,8 @@ class KVCache:
         return self.planes * self.num_layers
 
     def bytes_per_page(self) -> int:
+        if self.rows:
+            return sum(self.rows) * self.page * self.payload.element_size()
         n = self.planes * self.num_layers * self.num_kv_heads * self.page
         return n * self.head_dim * self.payload.element_size() + (n * 4 if self.scales is not None else 0)
 
@@ -503,12 +563,15 @@ def decode_splits(batch: int, num_kv_heads: int) -> int:
 
 
 _DECODE_COUNTERS: dict = {}
+_RETIRED_COUNTERS: list = []  # outgrown counters stay allocated: captured graphs hold their addresses
 
 
 def _decode_counters(device, n: int) -> torch.Tensor:
     """Zero-initialised, self-resetting arrival counters shared by all decode launches."""
     t = _DECODE_COUNTERS.get(str(device))
     if t is None or t.numel() < n:
+        if t is not None:
+            _RETIRED_COUNTERS.append(t)
         t = torch.zeros(max(n, 8192), dtype=torch.int32, device=device)
         _DECODE_COUNTERS[str(device)] = t
     return t
@@ -707,7 +770,8 @@ def kv_page_copy(src: KVCache, dst: KVCache, src_blocks: Sequence[int], dst_bloc
     if not on_gpu:
         for i in range(n):
             r = src.page if rows is None else int(rows[i])
-            dst.payload[:, :, dst_blocks[i], :, :r] = src.payload[:, :, src_blocks[i], :, :r]
+            for s, d in zip(src.slab_groups(), dst.slab_groups()):
+                d[:, dst_blocks[i], :, :r] = s[:, src_blocks[i], :, :r]
             if src.scales is not None:
                 dst.scales[:, :, dst_blocks[i], :, :r] = src.scales[:, :, src_blocks[i], :, :r]
         return
@@ -716,13 +780,13 @@ def kv_page_copy(src: KVCache, dst: KVCache, src_blocks: Sequence[int], dst_bloc
     db = torch.tensor(list(dst_blocks), dtype=torch.int32, device=dev)
     nr = None if rows is None else torch.tensor(list(rows), dtype=torch.int32, device=dev)
     es = src.payload.element_size()
-    native.call(
-        "prism_kv_page_copy", _p(src.payload), _p(dst.payload), src.payload.stride(1) * es, dst.payload.stride(1) * es,
-        src.head_dim * es, _p(src.scales), _p(dst.scales),
-        src.scales.stride(1) * 4 if src.scales is not None else 0,
-        dst.scales.stride(1) * 4 if dst.scales is not None else 0,
-        _p(sb), _p(db), _p(nr), n, src.num_kv_heads, src.page, src.n_slabs, _s(),
-    )
+    for s, d in zip(src.slab_groups(), dst.slab_groups()):
+        native.call(
+            "prism_kv_page_copy", _p(s), _p(d), s.stride(0) * es, d.stride(0) * es, s.shape[-1] * es, _p(src.scales), _p(dst.scales),
+            src.scales.stride(1) * 4 if src.scales is not None else 0,
+            dst.scales.stride(1) * 4 if dst.scales is not None else 0,
+            _p(sb), _p(db), _p(nr), n, src.num_kv_heads, src.page, s.shape[0], _s(),
+        )
 
 
 def kv_compact(cache: KVCache, src_slots: torch.Tensor, dst_slots: torch.Tensor) -> None:
@@ -734,22 +798,22 @@ def kv_compact(cache: KVCache, src_slots: torch.Tensor, dst_slots: torch.Tensor)
     if not cache.payload.is_cuda:
         sb, so = src_slots.long() // cache.page, src_slots.long() % cache.page
         db, do = dst_slots.long() // cache.page, dst_slots.long() % cache.page
-        tmp = cache.payload[:, :, sb, :, so].clone()
-        cache.payload[:, :, db, :, do] = tmp
+        for slabs in cache.slab_groups():
+            slabs[:, db, :, do] = slabs[:, sb, :, so].clone()
         if cache.scales is not None:
             tmp_s = cache.scales[:, :, sb, :, so].clone()
             cache.scales[:, :, db, :, do] = tmp_s
         return
     es = cache.payload.element_size()
-    rb = cache.head_dim * es
-    rows = cache.n_slabs * cache.num_kv_heads * R
-    temp = torch.empty(rows * rb, dtype=torch.uint8, device=cache.payload.device)
-    stemp = torch.empty(rows, dtype=torch.float32, device=cache.payload.device) if cache.scales is not None else None
-    native.call(
-        "prism_kv_compact", _p(cache.payload), cache.payload.stride(1) * es, rb, _p(cache.scales),
-        cache.scales.stride(1) * 4 if cache.scales is not None else 0, _p(temp), _p(stemp),
-        _p(src_slots), _p(dst_slots), R, cache.num_kv_heads, cache.page, cache.n_slabs, _s(),
-    )
+    for slabs in cache.slab_groups():
+        rb, rows = slabs.shape[-1] * es, slabs.shape[0] * cache.num_kv_heads * R
+        temp = torch.empty(rows * rb, dtype=torch.uint8, device=slabs.device)
+        stemp = torch.empty(rows, dtype=torch.float32, device=slabs.device) if cache.scales is not None else None
+        native.call(
+            "prism_kv_compact", _p(slabs), slabs.stride(0) * es, rb, _p(cache.scales),
+            cache.scales.stride(1) * 4 if cache.scales is not None else 0, _p(temp), _p(stemp),
+            _p(src_slots), _p(dst_slots), R, cache.num_kv_heads, cache.page, slabs.shape[0], _s(),
+        )
 
 
 # ------------------------------------------------------------------------------ sampler

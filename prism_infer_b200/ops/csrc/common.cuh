@@ -77,6 +77,13 @@ __device__ __forceinline__ float gelu_erf(float x) {
   return 0.5f * x * (1.0f + erff(x * 0.7071067811865476f));
 }
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
+// Gated linear units of the two-matrix GEMM epilogues.  SILU_ROUNDED keeps the rounding points of an eager bf16 graph;
+// the others stay in 32-bit until the product is stored.
+enum PrismGlu : int { PRISM_GLU_SILU_ROUNDED = 0, PRISM_GLU_SILU = 1, PRISM_GLU_GELU_TANH = 2 };
+__device__ __forceinline__ float glu(float g, float u, int act) {
+  if (act == PRISM_GLU_SILU_ROUNDED) return bf16_round(silu(bf16_round(g))) * bf16_round(u);
+  return (act == PRISM_GLU_GELU_TANH ? gelu_tanh(g) : silu(g)) * u;
+}
 
 __device__ __forceinline__ float sigmoid_fast(float x) { return 1.0f / (1.0f + __expf(-x)); }
 
@@ -253,6 +260,10 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
       : "memory");
 }
 __device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+// One column: thread t of the warp receives lane (taddr.lane + t).
+__device__ __forceinline__ void tmem_ld1(uint32_t taddr, uint32_t& r) {
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x1.b32 {%0}, [%1];" : "=r"(r) : "r"(taddr) : "memory");
+}
 // Store counterpart: thread t writes lane (taddr.lane + t), columns taddr.col .. +15.
 __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
   asm volatile(

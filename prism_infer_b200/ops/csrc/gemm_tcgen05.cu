@@ -17,6 +17,10 @@
 // (prism_infer/ops/csrc/cutlass_dual_gemm_swiglu.cu:85-215, mma.sync Sm80) and every
 // F.linear of prism_infer/layers/linear.py:62-190.
 //
+// Grouped form (mixture of experts): the weights of all experts are stacked by rows and a table on the device names, per
+// tile, the expert and the consecutive activation rows it serves; decode-sized steps run the split-K kernel with one
+// expert per blockIdx.y, prompts the persistent kernel with tokens on the TMEM lanes.
+//
 // Stacked projections (several weight matrices over the same activations, each with its own scale and
 // activation) run as one launch: PrismSections (common.cuh) names the row ranges.
 //
@@ -67,6 +71,11 @@ struct GemmArgs {
   float* peer_out[8];        // slab buffers (or bf16 row buffers) of this slot on every rank (incl. own)
   unsigned long long* peer_flag[8];  // flag arrays [tp] of this slot on every rank
   PrismSections sec;         // stacked projections: scale and activation by row range (n = 0: off)
+  // grouped form: blockIdx.y is an entry of the table, expert e's weights start at row e * group_rows of W
+  const int4* groups;        // (expert, first row, rows, -)
+  const int* n_groups;
+  const int* row_token;      // column of every row (the whole step is one token tile); null: consecutive rows of X
+  int group_rows;
 };
 
 // One activation in 32-bit, chosen at run time (uniform over a warp for stacked projections).
@@ -80,7 +89,7 @@ __device__ __forceinline__ float apply_act(float v, int act, float cap) {
   }
 }
 
-template <int BN, bool DUAL>
+template <int BN, bool DUAL, bool GROUPED = false>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, const GemmArgs a) {
   constexpr int X_TILE_BYTES = BN * BK * 2;
@@ -103,8 +112,17 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
   // Rasterisation.  When the weight matrix does not fit the 126 MB L2, token tiles vary
   // fastest so the CTAs that share a weight tile run together and it leaves DRAM once;
   // otherwise feature tiles vary fastest (measured faster while everything is L2-resident).
-  const int m0 = (a.tokens_fastest ? blockIdx.y : blockIdx.x) * BM;
-  const int n0 = (a.tokens_fastest ? blockIdx.x : blockIdx.y) * BN;
+  const int m0 = (!GROUPED && a.tokens_fastest ? blockIdx.y : blockIdx.x) * BM;
+  int n0 = (a.tokens_fastest ? blockIdx.x : blockIdx.y) * BN;
+  int w_row = m0;            // first row of the weight tile in W
+  int4 group = make_int4(0, 0, 0, 0);
+  if (GROUPED) {
+    pdl_wait();              // the table comes from the previous kernels
+    if ((int)blockIdx.y >= *a.n_groups) return;
+    group = a.groups[blockIdx.y];
+    w_row = group.x * a.group_rows + m0;
+    n0 = a.row_token ? 0 : group.y;
+  }
   const int split = blockIdx.z;
   const int kb_begin = split * a.kb_per_split;
   const int kb_end = min(a.kb_total, kb_begin + a.kb_per_split);
@@ -137,8 +155,8 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       for (int i = 0; i < pre; ++i) {
         uint8_t* st = smem + (size_t)i * STAGE_BYTES;
         mbar_expect_tx(&full[i], STAGE_BYTES);
-        tma_load_2d(st, &tmW, &full[i], (kb_begin + i) * BK, m0);
-        if (DUAL) tma_load_2d(st + W_TILE_BYTES, &tmW, &full[i], (kb_begin + i) * BK, a.w2_row_off + m0);
+        tma_load_2d(st, &tmW, &full[i], (kb_begin + i) * BK, w_row);
+        if (DUAL) tma_load_2d(st + W_TILE_BYTES, &tmW, &full[i], (kb_begin + i) * BK, a.w2_row_off + w_row);
       }
       pdl_wait();  // activations come from the previous kernel
       for (int i = 0; i < pre; ++i) {
@@ -154,8 +172,8 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         if (!ok) break;
         uint8_t* st = smem + (size_t)s * STAGE_BYTES;
         mbar_expect_tx(&full[s], STAGE_BYTES);
-        tma_load_2d(st, &tmW, &full[s], (kb_begin + kb) * BK, m0);
-        if (DUAL) tma_load_2d(st + W_TILE_BYTES, &tmW, &full[s], (kb_begin + kb) * BK, a.w2_row_off + m0);
+        tma_load_2d(st, &tmW, &full[s], (kb_begin + kb) * BK, w_row);
+        if (DUAL) tma_load_2d(st + W_TILE_BYTES, &tmW, &full[s], (kb_begin + kb) * BK, a.w2_row_off + w_row);
         tma_load_2d(st + W_STAGE_BYTES, &tmX, &full[s], (kb_begin + kb) * BK, n0);
         issued = kb + 1;
       }
@@ -218,7 +236,18 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       else if (a.n_peers > 0) mode = a.push_rows ? EPI_PUSH_ROWS : EPI_PUSH_F32;
       else if (a.out_f32) mode = EPI_F32;
       else mode = (a.bias == nullptr && a.act == 0 && a.residual == nullptr) ? EPI_BF16_PLAIN : EPI_BF16_FULL;
-      const int n_valid = min(BN, a.T - n0);
+      const int n_valid = GROUPED ? min(BN, group.z) : min(BN, a.T - n0);
+      if (GROUPED && DUAL && a.row_token != nullptr) {
+        // the tile holds every token of the step: each row of this expert reads its token's column
+        for (int i = 0; i < group.z; ++i) {
+          const int c = a.row_token[group.y + i];
+          uint32_t rg, ru;
+          tmem_ld1(t_lane + c, rg);
+          tmem_ld1(t_lane + BN + c, ru);
+          tmem_ld_wait();
+          if (m_ok) out_b[(size_t)(group.y + i) * a.ldo + m] = __float2bfloat16_rn(glu(__uint_as_float(rg), __uint_as_float(ru), a.act));
+        }
+      } else {
       unsigned long long push_seq = 0;
       if (mode == EPI_PUSH_F32)
         push_seq = (((a.epoch ? *a.epoch : 0ull) + (unsigned long long)a.point) & 0xffffffffull) << 32;
@@ -320,19 +349,15 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             }
             break;
           }
-          default: {  // EPI_DUAL: silu(gate) -> bf16, * up -> bf16 (rounding points of the eager graph)
+          default: {  // EPI_DUAL
             __nv_bfloat16* dst = out_b + row0 * a.ldo + m;
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              if (j < cols) {
-                const float g = bf16_round(__uint_as_float(r[j]));
-                const float u = bf16_round(__uint_as_float(r2[j]));
-                dst[(size_t)j * a.ldo] = __float2bfloat16_rn(bf16_round(silu(g)) * u);
-              }
-            }
+            for (int j = 0; j < 16; ++j)
+              if (j < cols) dst[(size_t)j * a.ldo] = __float2bfloat16_rn(glu(__uint_as_float(r[j]), __uint_as_float(r2[j]), a.act));
             break;
           }
         }
+      }
       }
     }
   }
@@ -388,6 +413,9 @@ struct PersistArgs {
   __nv_bfloat16* peer_out[8];
   unsigned long long* peer_flag[8];
   PrismSections sec;  // row-major form only; row ends are multiples of 16 (a chunk lies in one section)
+  const int4* groups;  // grouped form (row-major): token tile i is entry i of the table, m_tiles its capacity
+  const int* n_groups;
+  int group_rows;      // weight rows per expert
 };
 
 // ROWMAJOR: the A operand (128-row tiles, TMEM lanes) holds the tokens and B the weights, so an
@@ -395,7 +423,7 @@ struct PersistArgs {
 // and output move as 16-byte vectors instead of sixteen strided 2-byte accesses (the strided
 // residual loads made the vision projections 6x slower than their main loop).  In that form
 // a.M counts tokens and a.T features.
-template <int BN, bool DUAL, bool ROWMAJOR = false>
+template <int BN, bool DUAL, bool ROWMAJOR = false, bool GROUPED = false>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                           const PersistArgs a) {
@@ -418,7 +446,12 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
-  const int num_tiles = a.m_tiles * a.n_tiles;
+  int m_tiles = a.m_tiles;
+  if (GROUPED) {
+    pdl_wait();  // the table comes from the previous kernels
+    m_tiles = min(m_tiles, *a.n_groups);
+  }
+  const int num_tiles = m_tiles * a.n_tiles;
   const int num_kb = a.kb_total;
 
   if (threadIdx.x == 0) {
@@ -446,9 +479,14 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
 
   // tile id -> (m0, n0); consecutive ids share a weight tile (tokens fastest) or an
   // activation tile (features fastest)
-#define PRISM_TILE_COORDS(tile_, m0_, n0_)                                             \
-  const int m0_ = (a.tokens_fastest ? (tile_) / a.n_tiles : (tile_) % a.m_tiles) * BM; \
-  const int n0_ = (a.tokens_fastest ? (tile_) % a.n_tiles : (tile_) / a.m_tiles) * BN;
+  // m0 / n0: first activation row / output feature; w0: row of the weight matrix the expert starts at; m_end: rows past it
+  // belong to another tile
+#define PRISM_TILE_COORDS(tile_, m0_, n0_)                                         \
+  const int mt_ = a.tokens_fastest ? (tile_) / a.n_tiles : (tile_) % m_tiles;      \
+  const int4 g_ = GROUPED ? a.groups[mt_] : make_int4(0, mt_ * BM, 0, 0);          \
+  const int m0_ = g_.y, w0 = GROUPED ? g_.x * a.group_rows : 0;                    \
+  const int m_end = GROUPED ? min(a.M, g_.y + g_.z) : a.M;                         \
+  const int n0_ = (a.tokens_fastest ? (tile_) % a.n_tiles : (tile_) / m_tiles) * BN;
 
   if (warp == 0) {
     if (lane == 0) {
@@ -471,10 +509,10 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
           if (DUAL) tma_load_2d(st + W_TILE_BYTES, &tmW, &full[s], kb * BK, a.w2_row_off + m0);
           if (ROWMAJOR && a.dual_rm) {
             // one 256-row B tile made of 128 gate rows and the matching 128 up rows
-            tma_load_2d(st + W_STAGE_BYTES, &tmX, &full[s], kb * BK, n0 / 2);
-            tma_load_2d(st + W_STAGE_BYTES + X_TILE_BYTES / 2, &tmX, &full[s], kb * BK, a.w2_row_off + n0 / 2);
+            tma_load_2d(st + W_STAGE_BYTES, &tmX, &full[s], kb * BK, w0 + n0 / 2);
+            tma_load_2d(st + W_STAGE_BYTES + X_TILE_BYTES / 2, &tmX, &full[s], kb * BK, w0 + a.w2_row_off + n0 / 2);
           } else {
-            tma_load_2d(st + W_STAGE_BYTES, &tmX, &full[s], kb * BK, n0);
+            tma_load_2d(st + W_STAGE_BYTES, &tmX, &full[s], kb * BK, w0 + n0);
           }
         }
       }
@@ -534,7 +572,7 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
       tc_fence_after();
       PRISM_TILE_COORDS(tile, m0, n0)
       const int m = m0 + q * 32 + lane;
-      const bool m_ok = m < a.M;
+      const bool m_ok = m < m_end;
       const uint32_t t_lane = tmem_base + buf * ACC_COLS + ((uint32_t)(q * 32) << 16);
       const int n_valid = min(BN, a.T - n0);
       if (ROWMAJOR && a.dual_rm) {
@@ -551,9 +589,8 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
           __nv_bfloat162* op = reinterpret_cast<__nv_bfloat162*>(o);
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
-            const float g0 = bf16_round(__uint_as_float(rg[2 * e])), g1 = bf16_round(__uint_as_float(rg[2 * e + 1]));
-            const float u0 = bf16_round(__uint_as_float(ru[2 * e])), u1 = bf16_round(__uint_as_float(ru[2 * e + 1]));
-            op[e] = __floats2bfloat162_rn(bf16_round(silu(g0)) * u0, bf16_round(silu(g1)) * u1);
+            op[e] = __floats2bfloat162_rn(glu(__uint_as_float(rg[2 * e]), __uint_as_float(ru[2 * e]), a.act),
+                                          glu(__uint_as_float(rg[2 * e + 1]), __uint_as_float(ru[2 * e + 1]), a.act));
           }
           __nv_bfloat16* dst = a.out + (size_t)m * a.ldo + f_base + c0;
           *reinterpret_cast<uint4*>(dst) = o[0];
@@ -651,13 +688,8 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
         __nv_bfloat16* dst = a.out + row0 * a.ldo + m;
         if (DUAL) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) {
-            if (j < cols) {
-              const float g = bf16_round(__uint_as_float(r[j]));
-              const float u = bf16_round(__uint_as_float(r2[j]));
-              dst[(size_t)j * a.ldo] = __float2bfloat16_rn(bf16_round(silu(g)) * u);
-            }
-          }
+          for (int j = 0; j < 16; ++j)
+            if (j < cols) dst[(size_t)j * a.ldo] = __float2bfloat16_rn(glu(__uint_as_float(r[j]), __uint_as_float(r2[j]), a.act));
         } else if (plain) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
@@ -776,9 +808,9 @@ int get_tensor_map(const void* ptr, unsigned long long rows, unsigned long long 
 
 int g_small_tile_smem_cap = 0;
 
-template <int BN, bool DUAL>
+template <int BN, bool DUAL, bool GROUPED = false>
 int launch_gemm(const CUtensorMap& tw, const CUtensorMap& tx, GemmArgs& a, int m_tiles, int splits, int stages_override,
-                cudaStream_t stream, bool pdl) {
+                cudaStream_t stream, bool pdl, int max_groups = 0) {
   constexpr int STAGE_BYTES = W_TILE_BYTES * (DUAL ? 2 : 1) + BN * BK * 2;
   int max_stages = (SMEM_LIMIT - 1024 - 512) / STAGE_BYTES;
   if (max_stages > 16) max_stages = 16;
@@ -796,13 +828,13 @@ int launch_gemm(const CUtensorMap& tw, const CUtensorMap& tx, GemmArgs& a, int m
   const size_t smem = (size_t)stages * STAGE_BYTES + 1024 + (2 * stages + 1) * 8 + 48;
   static int configured_smem = 0;
   if ((int)smem > configured_smem) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_wx_kernel<BN, DUAL>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_LIMIT);
+    cudaError_t e = cudaFuncSetAttribute(gemm_wx_kernel<BN, DUAL, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_LIMIT);
     if (e != cudaSuccess) return (int)e;
     configured_smem = SMEM_LIMIT;
   }
-  const int n_tiles = (a.T + BN - 1) / BN;
-  dim3 grid = a.tokens_fastest ? dim3(n_tiles, m_tiles, splits) : dim3(m_tiles, n_tiles, splits);
-  cudaError_t e = prism_launch(gemm_wx_kernel<BN, DUAL>, grid, dim3(GEMM_THREADS), smem, stream, pdl, tw, tx, a);
+  const int n_tiles = GROUPED ? max_groups : (a.T + BN - 1) / BN;
+  dim3 grid = !GROUPED && a.tokens_fastest ? dim3(n_tiles, m_tiles, splits) : dim3(m_tiles, n_tiles, splits);
+  cudaError_t e = prism_launch(gemm_wx_kernel<BN, DUAL, GROUPED>, grid, dim3(GEMM_THREADS), smem, stream, pdl, tw, tx, a);
   return (int)e;
 }
 
@@ -811,7 +843,7 @@ int g_persistent_min_tokens = 512;  // 0 disables the persistent form
 int g_persistent_rowmajor = 1;      // 1: tokens on the TMEM lanes for the non-dual persistent GEMM
 int g_sm_count = 0;
 
-template <int BN, bool DUAL, bool ROWMAJOR = false>
+template <int BN, bool DUAL, bool ROWMAJOR = false, bool GROUPED = false>
 int launch_persistent(const CUtensorMap& tw, const CUtensorMap& tx, PersistArgs& a, cudaStream_t stream, bool pdl) {
   constexpr int STAGE_BYTES = W_TILE_BYTES * (DUAL ? 2 : 1) + BN * BK * 2;
   int stages = (SMEM_LIMIT - 1024 - 512) / STAGE_BYTES;
@@ -821,7 +853,7 @@ int launch_persistent(const CUtensorMap& tw, const CUtensorMap& tx, PersistArgs&
   const size_t smem = (size_t)stages * STAGE_BYTES + 1024 + (2 * stages + 4) * 8 + 64;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_wx_persistent_kernel<BN, DUAL, ROWMAJOR>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_LIMIT);
+    cudaError_t e = cudaFuncSetAttribute(gemm_wx_persistent_kernel<BN, DUAL, ROWMAJOR, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_LIMIT);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
@@ -832,7 +864,7 @@ int launch_persistent(const CUtensorMap& tw, const CUtensorMap& tx, PersistArgs&
   }
   const int tiles = a.m_tiles * a.n_tiles;
   const int grid = tiles < g_sm_count ? tiles : g_sm_count;
-  return (int)prism_launch(gemm_wx_persistent_kernel<BN, DUAL, ROWMAJOR>, dim3(grid), dim3(GEMM_THREADS), smem, stream, pdl, tw, tx, a);
+  return (int)prism_launch(gemm_wx_persistent_kernel<BN, DUAL, ROWMAJOR, GROUPED>, dim3(grid), dim3(GEMM_THREADS), smem, stream, pdl, tw, tx, a);
 }
 
 }  // namespace
@@ -917,6 +949,9 @@ static int gemm_wx_impl(const void* W, const void* X, void* out, int M, int T, i
     for (int i = 0; i < a.sec.n; ++i)
       if (a.sec.row_end[i] % 16 || a.sec.act[i] == PRISM_ACT_SOFTCAP) sections_rowmajor = false;
   }
+  a.groups = nullptr;
+  a.n_groups = a.row_token = nullptr;
+  a.group_rows = 0;
   a.ldo = ldo;
   a.ldr = ldr;
   a.split_stride = split_stride;
@@ -960,6 +995,9 @@ static int gemm_wx_impl(const void* W, const void* X, void* out, int M, int T, i
                                ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0))) {
     PersistArgs pa;
     pa.sec = a.sec;
+    pa.groups = nullptr;
+    pa.n_groups = nullptr;
+    pa.group_rows = 0;
     pa.M = M;
     pa.T = T;
     pa.kb_total = a.kb_total;
@@ -987,8 +1025,8 @@ static int gemm_wx_impl(const void* W, const void* X, void* out, int M, int T, i
                                         reinterpret_cast<unsigned long long>(residual);
     pa.dual_rm = 0;
     if (dual && g_persistent_rowmajor && M % 16 == 0 && ldo % 8 == 0 && (vec_addr & 15ull) == 0 && bias == nullptr &&
-        residual == nullptr && act == 0) {
-      // SwiGLU with tokens on the TMEM lanes: one N = 256 MMA per step over [128 gate rows | 128 up rows]
+        residual == nullptr) {
+      // gated unit with tokens on the TMEM lanes: one N = 256 MMA per step over [128 gate rows | 128 up rows]
       CUtensorMap ta, tb;
       rc = get_tensor_map(X, (unsigned long long)T, (unsigned long long)K, (unsigned long long)ldx, BM, &ta);
       if (rc) return rc;
@@ -1064,6 +1102,86 @@ PRISM_API int prism_gemm_wx_sections(const void* W, const void* X, void* out, in
   if (!prism_fill_sections(sec, n_sections, (const int*)row_end, (const float*)alpha, (const int*)act, cap, M)) return -9;
   return gemm_wx_impl(W, X, out, M, T, K, ldw, ldx, ldo, M, bias, nullptr, 0, 0, 0, 0, 1, out_f32, 0, bn_override,
                       stages_override, stream_ptr, pdl, nullptr, &sec);
+}
+
+// Experts' projections of a decode-sized step.  W stacks the experts' matrices (act != 0: M gate rows then M up rows each, the
+// output is act(gate) * up in bf16; act == 0: M rows each, the output fp32 split-K slabs).  Entry i of the table is
+// (expert, first row, rows, -) with rows <= T.  row_token != null: X holds the step's T <= 128 tokens and output row n belongs
+// to token row_token[n]; null: X and the output share their row numbers.
+PRISM_API int prism_gemm_grouped_small(const void* W, const void* X, void* out, int M, int T, int X_rows, int K, long long ldx,
+                                       long long ldo, const void* groups, int max_groups, const void* n_groups, const void* row_token,
+                                       int N, int experts, int act, int splits, long long split_stride, void* stream, int pdl) {
+  if (M <= 0 || T <= 0 || T > 128 || K <= 0 || K % 8 || max_groups <= 0 || max_groups > 65535 || experts <= 0 || !groups || !n_groups) return -1;
+  const bool dual = act != 0;
+  if (act < 0 || act > PRISM_GLU_GELU_TANH || (dual != (row_token != nullptr)) || (dual && splits > 1) || X_rows < (dual ? T : N)) return -2;
+  GemmArgs a = {};
+  a.M = M;
+  a.T = N;
+  a.kb_total = (K + BK - 1) / BK;
+  if (splits < 1) splits = 1;
+  if (splits > a.kb_total) splits = a.kb_total;
+  a.kb_per_split = (a.kb_total + splits - 1) / splits;
+  splits = (a.kb_total + a.kb_per_split - 1) / a.kb_per_split;
+  a.w2_row_off = M;
+  a.out_f32 = dual ? 0 : 1;
+  a.act = act;
+  a.ldo = ldo;
+  a.split_stride = split_stride;
+  a.out = out;
+  a.groups = (const int4*)groups;
+  a.n_groups = (const int*)n_groups;
+  a.row_token = (const int*)row_token;
+  a.group_rows = dual ? 2 * M : M;
+  const int bn = T <= 16 ? 16 : (T <= 32 ? 32 : (T <= 64 ? 64 : 128));
+  CUtensorMap tw, tx;
+  int rc = get_tensor_map(W, (unsigned long long)experts * a.group_rows, (unsigned long long)K, (unsigned long long)K, BM, &tw);
+  if (rc) return rc;
+  rc = get_tensor_map(X, (unsigned long long)X_rows, (unsigned long long)K, (unsigned long long)ldx, (unsigned)bn, &tx);
+  if (rc) return rc;
+  const int m_tiles = (M + BM - 1) / BM;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const bool p = pdl != 0;
+#define PRISM_GROUPED_CASE(BN_)                                                                case BN_:                                                                                      return dual ? launch_gemm<BN_, true, true>(tw, tx, a, m_tiles, splits, 0, s, p, max_groups)                 : launch_gemm<BN_, false, true>(tw, tx, a, m_tiles, splits, 0, s, p, max_groups);
+  switch (bn) {
+    PRISM_GROUPED_CASE(16)
+    PRISM_GROUPED_CASE(32)
+    PRISM_GROUPED_CASE(64)
+    PRISM_GROUPED_CASE(128)
+  }
+#undef PRISM_GROUPED_CASE
+  return -6;
+}
+
+// Experts' projections of a prompt: X [N][K] and out [N][ldo] (bf16) in expert order, table entries of at most 128 rows.
+// act != 0: W [experts][M gate rows, M up rows][K], out = act(gate) * up; act == 0: W [experts][M][K].  M a multiple of 16.
+PRISM_API int prism_gemm_grouped(const void* W, const void* X, void* out, int M, int N, int K, long long ldx, long long ldo,
+                                 const void* groups, int max_groups, const void* n_groups, int experts, int act, void* stream, int pdl) {
+  if (M <= 0 || M % 16 || N <= 0 || K <= 0 || K % 8 || max_groups <= 0 || experts <= 0 || !groups || !n_groups) return -1;
+  if (act < 0 || act > PRISM_GLU_GELU_TANH || ldo % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return -2;
+  const bool dual = act != 0;
+  PersistArgs pa = {};
+  pa.sec.n = 0;
+  pa.dual_rm = dual ? 1 : 0;
+  pa.M = N;
+  pa.T = dual ? 2 * M : M;
+  pa.kb_total = (K + BK - 1) / BK;
+  pa.w2_row_off = M;
+  pa.m_tiles = max_groups;
+  pa.n_tiles = dual ? (M + 127) / 128 : (M + 255) / 256;
+  pa.tokens_fastest = 1;  // consecutive tiles share a token tile: the features of one expert follow one another
+  pa.act = act;
+  pa.ldo = ldo;
+  pa.out = reinterpret_cast<__nv_bfloat16*>(out);
+  pa.rows_per_owner = 1;
+  pa.groups = (const int4*)groups;
+  pa.n_groups = (const int*)n_groups;
+  pa.group_rows = dual ? 2 * M : M;
+  CUtensorMap ta, tb;
+  int rc = get_tensor_map(X, (unsigned long long)N, (unsigned long long)K, (unsigned long long)ldx, BM, &ta);
+  if (rc) return rc;
+  rc = get_tensor_map(W, (unsigned long long)experts * pa.group_rows, (unsigned long long)K, (unsigned long long)K, dual ? 128 : 256, &tb);
+  if (rc) return rc;
+  return launch_persistent<256, false, true, true>(ta, tb, pa, reinterpret_cast<cudaStream_t>(stream), pdl != 0);
 }
 
 // Fused row-parallel GEMM -> one-shot exchange: the fp32 partial of rank `my_rank`, split s,

@@ -1,0 +1,251 @@
+// Routing and dispatch of a mixture of experts.
+//
+// Every token has `top` routed slots and `always` more that name experts E .. E + always - 1.  Pairs (token, slot) get a
+// row each, sorted by expert and, within one, by token: the grouped GEMMs then read an expert's tokens as consecutive
+// rows.  The order is a function of the routing alone.
+//
+//   moe_route_kernel   one CTA per chunk of tokens: sum of the router's split-K slabs, top-k (one warp per token), softmax
+//                      over the chosen logits, count per expert and rank of each pair within its chunk and expert.  With a
+//                      single chunk it also places the pairs.
+//   moe_place_kernel   one CTA per chunk: first row of every expert, then rows of the chunk's pairs
+//   moe_gather_kernel  copies a token's row to the rows of its pairs
+#include "common.cuh"
+
+PRISM_DEFINE_TU_STATUS(moe)
+
+namespace {
+
+typedef __nv_bfloat16 bf16;
+
+constexpr int ROUTE_THREADS = 1024, ROUTE_WARPS = ROUTE_THREADS / 32;
+constexpr int MAX_EXPERTS = 1024;  // routed and always-on together: one thread each in the prefix sums
+
+struct RouteArgs {
+  const float* logits;     // [P][T][ld] fp32 slabs
+  long long slab_stride, ld;
+  int P;
+  const long long* slots;  // cache slot of each token, < 0: takes no part
+  int* expert;             // [T][K] expert of each pair (-1: none)
+  int* pos;                // [T][K] rank within chunk and expert, then the pair's row (-1: none)
+  float* weight;           // [T][K]
+  int* row_token;          // [T * K]
+  int* counts;             // [chunks][E + always]
+  int4* groups;            // (expert, first row, rows, 0)
+  int max_groups;
+  int* n_groups;
+  int T, top, E, always, chunk, tile;
+};
+
+// Exclusive prefix sum over the block of one value per thread; *total gets the sum.
+__device__ __forceinline__ int block_scan(int v, int* warp_sums, int* total) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  int x = v;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int y = __shfl_up_sync(0xffffffffu, x, o);
+    if (lane >= o) x += y;
+  }
+  if (lane == 31) warp_sums[warp] = x;
+  __syncthreads();
+  if (warp == 0) {
+    int s = warp_sums[lane];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int y = __shfl_up_sync(0xffffffffu, s, o);
+      if (lane >= o) s += y;
+    }
+    warp_sums[lane] = s;
+  }
+  __syncthreads();
+  const int before = warp > 0 ? warp_sums[warp - 1] : 0;
+  *total = warp_sums[31];
+  __syncthreads();
+  return before + x - v;
+}
+
+// Rows of a chunk's pairs from the experts' first rows, and (writer) the table of tiles.  count: pairs of expert
+// threadIdx.x over all tokens, before: those in earlier chunks.
+__device__ __forceinline__ void place(const RouteArgs& a, int t0, int n, int count, int before, bool writer, int* scan_s, int* base_s) {
+  const int e = threadIdx.x, all = a.E + a.always, K = a.top + a.always;
+  int total;
+  const int first = block_scan(e < all ? count : 0, scan_s, &total);
+  if (e < all) base_s[e] = first + before;
+  const int tiles = e < all ? (count + a.tile - 1) / a.tile : 0;
+  int n_tiles;
+  const int g0 = block_scan(tiles, scan_s, &n_tiles);
+  if (writer) {
+    for (int i = 0; i < tiles; ++i)
+      if (g0 + i < a.max_groups) a.groups[g0 + i] = make_int4(e, first + i * a.tile, min(a.tile, count - i * a.tile), 0);
+    if (e == 0) {
+      *a.n_groups = min(n_tiles, a.max_groups);
+      if (n_tiles > a.max_groups) prism_report(PRISM_ERR_BOUNDS, 1);
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < n * K; i += blockDim.x) {
+    const size_t pair = (size_t)t0 * K + i;
+    const int x = a.expert[pair];
+    if (x < 0) continue;
+    const int row = base_s[x] + a.pos[pair];
+    a.pos[pair] = row;
+    a.row_token[row] = t0 + i / K;
+  }
+}
+
+__global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArgs a) {
+  extern __shared__ int expert_s[];            // [chunk * K]
+  __shared__ int count_s[MAX_EXPERTS], base_s[MAX_EXPERTS], scan_s[32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t0 = blockIdx.x * a.chunk, n = min(a.chunk, a.T - t0), all = a.E + a.always, K = a.top + a.always;
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int i = warp; i < n; i += ROUTE_WARPS) {
+    const size_t t = (size_t)t0 + i;
+    const bool live = a.slots[t] >= 0;
+    // lane l holds experts l, l + 32, ...: the next best is found by a maximum over (value, lowest expert)
+    float v[MAX_EXPERTS / 32];
+#pragma unroll
+    for (int c = 0; c < MAX_EXPERTS / 32; ++c) {
+      v[c] = -INFINITY;
+      if (c * 32 < a.E) {
+        const int e = c * 32 + lane;
+        if (e < a.E) {
+          float s = 0.0f;
+          for (int p = 0; p < a.P; ++p) s += __ldcg(a.logits + (size_t)p * a.slab_stride + t * a.ld + e);
+          v[c] = s;
+        }
+      }
+    }
+    float best0 = 0.0f, sum = 0.0f;
+    for (int k = 0; k < a.top; ++k) {
+      float bv = -INFINITY;
+      int be = MAX_EXPERTS;
+#pragma unroll
+      for (int c = 0; c < MAX_EXPERTS / 32; ++c)
+        if (c * 32 < a.E && v[c] > bv) {
+          bv = v[c];
+          be = c * 32 + lane;
+        }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+        const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+        if (ov > bv || (ov == bv && oe < be)) {
+          bv = ov;
+          be = oe;
+        }
+      }
+      if (be >= a.E) be = 0;                   // no finite logit left: any expert, weight from its own logit
+#pragma unroll
+      for (int c = 0; c < MAX_EXPERTS / 32; ++c)
+        if (be == c * 32 + lane) v[c] = -INFINITY;
+      if (k == 0) best0 = bv;
+      const float w = expf(bv - best0);
+      sum += w;
+      if (lane == 0) {
+        expert_s[i * K + k] = live ? be : -1;
+        a.weight[t * K + k] = w;
+      }
+    }
+    __syncwarp();
+    const float inv = 1.0f / sum;
+    for (int k = lane; k < K; k += 32) {
+      if (k >= a.top) expert_s[i * K + k] = live ? a.E + k - a.top : -1;
+      a.weight[t * K + k] = live ? (k < a.top ? a.weight[t * K + k] * inv : 1.0f) : 0.0f;
+    }
+  }
+  __syncthreads();
+  // count and rank: one warp per expert looks at 32 pairs at a time
+  for (int e = warp; e < all; e += ROUTE_WARPS) {
+    int c = 0;
+    for (int i0 = 0; i0 < n * K; i0 += 32) {
+      const int i = i0 + lane;
+      const bool hit = i < n * K && expert_s[i] == e;
+      const unsigned m = __ballot_sync(0xffffffffu, hit);
+      if (hit) a.pos[(size_t)t0 * K + i] = c + __popc(m & ((1u << lane) - 1));
+      c += __popc(m);
+    }
+    if (lane == 0) count_s[e] = c;
+  }
+  for (int i = threadIdx.x; i < n * K; i += ROUTE_THREADS) {
+    a.expert[(size_t)t0 * K + i] = expert_s[i];
+    if (expert_s[i] < 0) a.pos[(size_t)t0 * K + i] = -1;
+  }
+  __syncthreads();
+  if (gridDim.x > 1) {
+    for (int e = threadIdx.x; e < all; e += ROUTE_THREADS) a.counts[(size_t)blockIdx.x * all + e] = count_s[e];
+    return;
+  }
+  place(a, t0, n, (int)threadIdx.x < all ? count_s[threadIdx.x] : 0, 0, true, scan_s, base_s);
+}
+
+__global__ void __launch_bounds__(ROUTE_THREADS) moe_place_kernel(const RouteArgs a) {
+  __shared__ int base_s[MAX_EXPERTS], scan_s[32];
+  const int t0 = blockIdx.x * a.chunk, n = min(a.chunk, a.T - t0), all = a.E + a.always;
+  pdl_launch_dependents();
+  pdl_wait();
+  int count = 0, before = 0;
+  if ((int)threadIdx.x < all)
+    for (int c = 0; c < (int)gridDim.x; ++c) {
+      const int v = a.counts[(size_t)c * all + threadIdx.x];
+      count += v;
+      if (c < (int)blockIdx.x) before += v;
+    }
+  place(a, t0, n, count, before, blockIdx.x == 0, scan_s, base_s);
+}
+
+// grid (tokens): row t of x to every row of its pairs
+__global__ void __launch_bounds__(256) moe_gather_kernel(const bf16* x, long long ldx, const int* pos, bf16* rows, int K, int W, int N) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const uint4* src = reinterpret_cast<const uint4*>(x + t * ldx);
+  for (int i = threadIdx.x; i < W / 8; i += 256) {
+    const uint4 v = src[i];
+    for (int k = 0; k < K; ++k) {
+      const int r = pos[t * K + k];
+      if (r >= 0 && r < N) reinterpret_cast<uint4*>(rows + (size_t)r * W)[i] = v;
+    }
+  }
+}
+
+int check_route(const RouteArgs& a) {
+  if (a.top < 1 || a.top > a.E || a.always < 0 || a.E + a.always > MAX_EXPERTS || a.chunk < 1 || a.tile < 1 || a.max_groups < 1) return -1;
+  if ((long long)a.T * (a.top + a.always) > 0x7fffffffll || a.chunk * (a.top + a.always) > 10240) return -2;
+  return 0;
+}
+
+}  // namespace
+
+// logits: P fp32 slabs [T][ld] of E columns.  expert, pos, weight [T][top + always]; row_token [T * (top + always)]; counts
+// [chunks][E + always]; groups [max_groups] int4 and n_groups: tiles of at most `tile` rows of one expert.  With more than
+// one chunk prism_moe_place must follow.
+PRISM_API int prism_moe_route(const void* logits, long long slab_stride, long long ld, int P, const void* slots, void* expert, void* pos,
+                              void* weight, void* row_token, void* counts, void* groups, int max_groups, void* n_groups, int T, int top,
+                              int E, int always, int chunk, int tile, void* stream, int pdl) {
+  if (T <= 0) return 0;
+  RouteArgs a{(const float*)logits, slab_stride, ld, P, (const long long*)slots, (int*)expert, (int*)pos, (float*)weight, (int*)row_token,
+              (int*)counts, (int4*)groups, max_groups, (int*)n_groups, T, top, E, always, chunk, tile};
+  if (int rc = check_route(a)) return rc;
+  const size_t smem = (size_t)chunk * (top + always) * sizeof(int);
+  return (int)prism_launch(moe_route_kernel, dim3((T + chunk - 1) / chunk), dim3(ROUTE_THREADS), smem, reinterpret_cast<cudaStream_t>(stream),
+                           pdl != 0, a);
+}
+
+PRISM_API int prism_moe_place(void* expert, void* pos, void* weight, void* row_token, void* counts, void* groups, int max_groups,
+                              void* n_groups, int T, int top, int E, int always, int chunk, int tile, void* stream, int pdl) {
+  if (T <= 0) return 0;
+  RouteArgs a{nullptr, 0, 0, 0, nullptr, (int*)expert, (int*)pos, (float*)weight, (int*)row_token, (int*)counts, (int4*)groups, max_groups,
+              (int*)n_groups, T, top, E, always, chunk, tile};
+  if (int rc = check_route(a)) return rc;
+  return (int)prism_launch(moe_place_kernel, dim3((T + chunk - 1) / chunk), dim3(ROUTE_THREADS), 0, reinterpret_cast<cudaStream_t>(stream),
+                           pdl != 0, a);
+}
+
+// rows [T * K][W] (bf16, W a multiple of 8): x[t] at every pos[t][k] >= 0.
+PRISM_API int prism_moe_gather(const void* x, long long ldx, const void* pos, void* rows, int T, int K, int W, void* stream, int pdl) {
+  if (T <= 0) return 0;
+  if (K <= 0 || W <= 0 || W % 8 || ldx % 8) return -1;
+  return (int)prism_launch(moe_gather_kernel, dim3(T), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream), pdl != 0, (const bf16*)x, ldx,
+                           (const int*)pos, (bf16*)rows, K, W, T * K);
+}

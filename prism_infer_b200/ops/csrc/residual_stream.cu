@@ -4,9 +4,11 @@
 //   start     x = table[id]                                     (embedding)
 //   pass      x = sum of the loop projection's slabs + step     (input of a looped section)
 //   layer     x += mult * (gate_a * a + gate_b * b)             (two parallel sublayers, either may be absent)
-// and what the next operation reads of it: the RMS-normalised row (gains are scalars that the next
-// GEMM's epilogue applies), or the row itself (the loop projection's input, with the embedding beside it).
-// a and b come as fp32 split-K slabs, summed here in a fixed order, or as rows of the compute type.
+//   layer     x += norm(a) * w                                  (a norm behind the sublayer)
+// and what the next operation reads of it: the RMS-normalised row (with a weight, or with a scalar gain that the
+// next GEMM's epilogue applies), or the row itself (the loop projection's input, with the embedding beside it).
+// a and b come as fp32 split-K slabs, summed here in a fixed order, or as rows of the compute type; a may also be
+// the weighted sum of several (token, expert) rows.
 #include "common.cuh"
 
 PRISM_DEFINE_TU_STATUS(stream)
@@ -47,6 +49,10 @@ struct Branch {
   long long ld;
   const T* gate;           // [T][gate_ld] (null: one)
   long long gate_ld;
+  const int* pos;          // [T][K]: rows of slabs / rows whose weighted sum is the value (null: row t itself)
+  const float* weight;     // [T][K]
+  int K;
+  const T* post_w;         // weight of the norm behind the sublayer (null: none)
 };
 
 template <typename T>
@@ -59,7 +65,8 @@ struct StreamArgs {
   Branch<T> a, b;
   float mult;
   const T* bias;           // [W] (null: none)
-  T* norm_out;             // rows x / sqrt(mean(x^2) + eps) (null: not wanted)
+  const T* norm_w;         // [W] (null: one)
+  T* norm_out;             // rows x / sqrt(mean(x^2) + eps) * norm_w (null: not wanted)
   long long norm_ld;
   T* raw_out;              // rows x in the compute type
   long long raw_ld;
@@ -69,37 +76,69 @@ struct StreamArgs {
   float eps;
 };
 
+// Columns i .. i + 3 of row r of a branch, slabs summed.
 template <typename T>
-__device__ __forceinline__ void add_branch(const Branch<T>& br, size_t t, int W, int i, float mult, F4& acc) {
-  if (br.slabs == nullptr && br.rows == nullptr) return;
-  F4 d;
-  if (br.slabs != nullptr) {
-    d = F4{{0.0f, 0.0f, 0.0f, 0.0f}};
-    const float* p0 = br.slabs + t * W + i;
+__device__ __forceinline__ F4 branch_row(const Branch<T>& br, size_t r, int W, int i) {
+  if (br.slabs == nullptr) return load4(br.rows + r * br.ld + i);
+  F4 d{{0.0f, 0.0f, 0.0f, 0.0f}};
+  const float* p0 = br.slabs + r * W + i;
 #pragma unroll 8
-    for (int p = 0; p < br.P; ++p) {
-      const float4 v = __ldcg(reinterpret_cast<const float4*>(p0 + (size_t)p * br.slab_stride));
-      d.v[0] += v.x;
-      d.v[1] += v.y;
-      d.v[2] += v.z;
-      d.v[3] += v.w;
+  for (int p = 0; p < br.P; ++p) {
+    const float4 v = __ldcg(reinterpret_cast<const float4*>(p0 + (size_t)p * br.slab_stride));
+    d.v[0] += v.x;
+    d.v[1] += v.y;
+    d.v[2] += v.z;
+    d.v[3] += v.w;
+  }
+  return d;
+}
+
+template <typename T>
+__device__ __forceinline__ F4 branch_value(const Branch<T>& br, size_t t, int W, int i) {
+  F4 d;
+  if (br.pos != nullptr) {
+    d = F4{{0.0f, 0.0f, 0.0f, 0.0f}};
+#pragma unroll 4
+    for (int k = 0; k < br.K; ++k) {
+      const int r = __ldg(br.pos + t * br.K + k);
+      if (r < 0) continue;
+      const float w = __ldg(br.weight + t * br.K + k);
+      const F4 v = branch_row(br, (size_t)r, W, i);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) d.v[e] += w * v.v[e];
     }
   } else {
-    d = load4(br.rows + t * br.ld + i);
+    d = branch_row(br, t, W, i);
   }
   if (br.gate != nullptr) {
     const F4 g = load4(br.gate + t * br.gate_ld + i);
 #pragma unroll
     for (int e = 0; e < 4; ++e) d.v[e] *= g.v[e];
   }
+  return d;
+}
+
+template <typename T>
+__device__ __forceinline__ void add_branch(const Branch<T>& br, size_t t, int W, int i, float mult, F4& acc) {
+  if (br.slabs == nullptr && br.rows == nullptr) return;
+  const F4 d = branch_value(br, t, W, i);
 #pragma unroll
   for (int e = 0; e < 4; ++e) acc.v[e] += mult * d.v[e];
+}
+
+// Sum over the block; every thread returns it.  red: 32 floats, free for the next use after the caller's next barrier.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  return warp_sum(lane < nw ? red[lane] : 0.0f);
 }
 
 template <typename T>
 __global__ void __launch_bounds__(1024) stream_update_kernel(const StreamArgs<T> a) {
   extern __shared__ float row[];  // W floats
-  __shared__ float red[32];
+  __shared__ float red[2][32];
   const size_t t = blockIdx.x;
   pdl_launch_dependents();
   pdl_wait();
@@ -109,10 +148,26 @@ __global__ void __launch_bounds__(1024) stream_update_kernel(const StreamArgs<T>
     if (id >= 0 && id < a.vocab) emb = a.table + (size_t)id * a.W;
     else if (threadIdx.x == 0) prism_report(PRISM_ERR_BOUNDS, 1);
   }
-  float ss = 0.0f;
+  float ss = 0.0f, post = 0.0f;
+  if (a.a.post_w != nullptr) {  // the branch's own root mean square first; a thread meets its own columns again below
+    float bs = 0.0f;
+    for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4) {
+      const F4 d = branch_value(a.a, t, a.W, i);
+      store4(row + i, d);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) bs += d.v[e] * d.v[e];
+    }
+    post = a.mult / sqrtf(block_sum(bs, red[0]) / (float)a.W_real + a.eps);
+  }
   for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4) {
     F4 acc{{0.0f, 0.0f, 0.0f, 0.0f}};
-    add_branch(a.a, t, a.W, i, a.mult, acc);
+    if (a.a.post_w != nullptr) {
+      const F4 d = load4(row + i), w = load4(a.a.post_w + i);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc.v[e] = d.v[e] * post * w.v[e];
+    } else {
+      add_branch(a.a, t, a.W, i, a.mult, acc);
+    }
     add_branch(a.b, t, a.W, i, a.mult, acc);
     if (a.keep) {
       const F4 x = load4(a.x + t * a.W + i);
@@ -139,25 +194,69 @@ __global__ void __launch_bounds__(1024) stream_update_kernel(const StreamArgs<T>
     for (int e = 0; e < 4; ++e) ss += acc.v[e] * acc.v[e];
   }
   if (a.norm_out == nullptr) return;
-  ss = warp_sum(ss);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  if (lane == 0) red[warp] = ss;
-  __syncthreads();
-  ss = warp_sum(lane < nw ? red[lane] : 0.0f);
-  const float inv = 1.0f / sqrtf(ss / (float)a.W_real + a.eps);
+  const float inv = 1.0f / sqrtf(block_sum(ss, red[1]) / (float)a.W_real + a.eps);
   for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4) {
     F4 v = load4(row + i);
 #pragma unroll
     for (int e = 0; e < 4; ++e) v.v[e] *= inv;
+    if (a.norm_w != nullptr) {
+      const F4 w = load4(a.norm_w + i);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v.v[e] *= w.v[e];
+    }
     store4(a.norm_out + t * a.norm_ld + i, v);
   }
+}
+
+// -------------------------------------------------------------------------------------------------
+// g[t][d] = gelu_tanh(z[t][d]) * table[ids[t]][offset + d]: the gate of a per-token side table.
+// -------------------------------------------------------------------------------------------------
+template <typename T>
+struct SideArgs {
+  Branch<T> z;
+  const T* table;
+  long long vocab, table_ld, offset;
+  const long long* ids;
+  T* out;                  // [T][D]
+  int D;
+  long long total;         // T * D / 4
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) token_side_gate_kernel(const SideArgs<T> a) {
+  pdl_launch_dependents();
+  const long long n = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (n >= a.total) return;
+  const size_t t = (size_t)(n * 4 / a.D);
+  const int d = (int)(n * 4 - (long long)t * a.D);
+  const long long id = a.ids[t];
+  F4 e{{0.0f, 0.0f, 0.0f, 0.0f}};  // the table does not depend on the previous kernel
+  if (id >= 0 && id < a.vocab) e = load4(a.table + (size_t)id * a.table_ld + a.offset + d);
+  else prism_report(PRISM_ERR_BOUNDS, 2);
+  pdl_wait();
+  F4 z = branch_value(a.z, t, a.D, d);
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const float v = z.v[k];
+    z.v[k] = 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v))) * e.v[k];
+  }
+  store4(a.out + t * a.D + d, z);
+}
+
+template <typename T>
+int launch_side(const void* slabs, long long slab_stride, int P, const void* rows, long long ld, const void* table, long long vocab,
+                long long table_ld, long long offset, const void* ids, void* out, int T_rows, int D, cudaStream_t stream, bool pdl) {
+  SideArgs<T> a{Branch<T>{(const float*)slabs, slab_stride, P, (const T*)rows, ld, nullptr, 0, nullptr, nullptr, 0, nullptr},
+                (const T*)table, vocab, table_ld, offset, (const long long*)ids, (T*)out, D, (long long)T_rows * D / 4};
+  return (int)prism_launch(token_side_gate_kernel<T>, dim3((unsigned)((a.total + 255) / 256)), dim3(256), 0, stream, pdl, a);
 }
 
 template <typename T>
 int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* table, long long vocab, const void* a_slabs,
                   long long a_stride, int a_P, const void* a_rows, long long a_ld, const void* a_gate, const void* b_slabs,
                   long long b_stride, int b_P, const void* b_rows, long long b_ld, const void* b_gate, long long gate_ld,
-                  float mult, const void* bias, void* norm_out, long long norm_ld, void* raw_out, long long raw_ld,
+                  const void* a_pos, const void* a_weight, int a_K, const void* a_post, float mult, const void* bias,
+                  const void* norm_w, void* norm_out, long long norm_ld, void* raw_out, long long raw_ld,
                   void* embed_out, long long embed_ld, int W, int W_real, float eps, cudaStream_t stream, bool pdl) {
   StreamArgs<T> a;
   a.x = (float*)x;
@@ -165,10 +264,12 @@ int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* ta
   a.ids = (const long long*)ids;
   a.table = (const T*)table;
   a.vocab = vocab;
-  a.a = Branch<T>{(const float*)a_slabs, a_stride, a_P, (const T*)a_rows, a_ld, (const T*)a_gate, gate_ld};
-  a.b = Branch<T>{(const float*)b_slabs, b_stride, b_P, (const T*)b_rows, b_ld, (const T*)b_gate, gate_ld};
+  a.a = Branch<T>{(const float*)a_slabs, a_stride, a_P, (const T*)a_rows, a_ld, (const T*)a_gate, gate_ld,
+                  (const int*)a_pos, (const float*)a_weight, a_K, (const T*)a_post};
+  a.b = Branch<T>{(const float*)b_slabs, b_stride, b_P, (const T*)b_rows, b_ld, (const T*)b_gate, gate_ld, nullptr, nullptr, 0, nullptr};
   a.mult = mult;
   a.bias = (const T*)bias;
+  a.norm_w = (const T*)norm_w;
   a.norm_out = (T*)norm_out;
   a.norm_ld = norm_ld;
   a.raw_out = (T*)raw_out;
@@ -195,17 +296,31 @@ int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* ta
 PRISM_API int prism_stream_update(int f32, int T, void* x, int keep, const void* ids, const void* table, long long vocab,
                                   const void* a_slabs, long long a_stride, int a_P, const void* a_rows, long long a_ld,
                                   const void* a_gate, const void* b_slabs, long long b_stride, int b_P, const void* b_rows,
-                                  long long b_ld, const void* b_gate, long long gate_ld, float mult, const void* bias,
-                                  void* norm_out, long long norm_ld, void* raw_out, long long raw_ld, void* embed_out,
+                                  long long b_ld, const void* b_gate, long long gate_ld, const void* a_pos,
+                                  const void* a_weight, int a_K, const void* a_post, float mult, const void* bias,
+                                  const void* norm_w, void* norm_out, long long norm_ld, void* raw_out, long long raw_ld, void* embed_out,
                                   long long embed_ld, int W, int W_real, float eps, void* stream, int pdl) {
   if (T <= 0) return 0;
   if (W <= 0 || W % 8 || W_real <= 0 || W_real > W || W > 32768) return -1;
   if ((a_ld | b_ld | gate_ld | norm_ld | raw_ld | embed_ld) % 4) return -2;
+  if ((a_pos != nullptr && (a_K <= 0 || !a_weight)) || ((a_pos || a_post) && !a_slabs && !a_rows)) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return f32 ? launch_stream<float>(T, x, keep, ids, table, vocab, a_slabs, a_stride, a_P, a_rows, a_ld, a_gate, b_slabs, b_stride,
-                                    b_P, b_rows, b_ld, b_gate, gate_ld, mult, bias, norm_out, norm_ld, raw_out, raw_ld, embed_out,
+                                    b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, mult, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,
                                     embed_ld, W, W_real, eps, s, pdl != 0)
              : launch_stream<bf16>(T, x, keep, ids, table, vocab, a_slabs, a_stride, a_P, a_rows, a_ld, a_gate, b_slabs, b_stride,
-                                   b_P, b_rows, b_ld, b_gate, gate_ld, mult, bias, norm_out, norm_ld, raw_out, raw_ld, embed_out,
+                                   b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, mult, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,
                                    embed_ld, W, W_real, eps, s, pdl != 0);
+}
+
+// g [T][D] = gelu_tanh(z) * table[ids[t]][offset ..]; z as fp32 slabs or rows of the compute type.  D, table_ld and offset
+// multiples of 4.
+PRISM_API int prism_token_side_gate(int f32, const void* slabs, long long slab_stride, int P, const void* rows, long long ld,
+                                    const void* table, long long vocab, long long table_ld, long long offset, const void* ids,
+                                    void* out, int T, int D, void* stream, int pdl) {
+  if (T <= 0) return 0;
+  if (D <= 0 || (D | table_ld | offset | ld) % 4 || offset + D > table_ld || (!slabs && !rows)) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  return f32 ? launch_side<float>(slabs, slab_stride, P, rows, ld, table, vocab, table_ld, offset, ids, out, T, D, s, pdl != 0)
+             : launch_side<bf16>(slabs, slab_stride, P, rows, ld, table, vocab, table_ld, offset, ids, out, T, D, s, pdl != 0);
 }

@@ -29,7 +29,19 @@ _SIGNATURES = {
     "prism_gemm_wx": "pppiiilllippliiiiiliipi",
     "prism_gemm_wx_sections": "pppiiilllpipppfiiipi",
     "prism_gemm_f32": "pppiiilllpipppfpi",
-    "prism_stream_update": "iipippl" "plipl" "p" "plipl" "p" "lfp" "plplpl" "iifpi",
+    "prism_gemm_f32_grouped": "pppiiilllpippiipi",
+    "prism_glu_f32": "ppiiipi",
+    "prism_gemm_grouped_small": "pppiiiillpippiiiilpi",
+    "prism_gemm_grouped": "pppiiillpipiipi",
+    "prism_moe_route": "pllippppppp" "ip" "iiiiiipi",
+    "prism_moe_place": "pppppp" "ip" "iiiiiipi",
+    "prism_moe_gather": "plppiiipi",
+    "prism_window_prepare": "ipliplppp" "ppplppp" "iiiiiiiiii" "fpi",
+    "prism_window_decode": "pppppppl" "ppp" "iiiiiiiiiiiiiii" "ffffpi",
+    "prism_window_prefill_tc": "pppppppl" "iiiiiiiiiiiiiii" "ffffpi",
+    "prism_window_attention_simple": "ipppppppl" "iiiiiiiiiiiiii" "ffffpi",
+    "prism_token_side_gate": "ipliplplllppiipi",
+    "prism_stream_update": "iipippl" "plipl" "p" "plipl" "p" "lppipfpp" "plplpl" "iifpi",
     "prism_latent_norm_store": "iplppplpiiifpi",
     "prism_latent_absorb": "plppplppp" "liiiiifpi",
     "prism_latent_attention": "pppppppp" "iiiiiiiifpi",
@@ -86,7 +98,7 @@ _SIGNATURES = {
     "prism_decode_layers_seq_step": "i",
 }
 _STATUS_UNITS = ("gemm", "norm", "attn", "attn_tc", "kvops", "sampler", "comm", "decode_layers", "lm_head_fp8",
-                 "latent", "stream", "gemm_f32")
+                 "latent", "stream", "gemm_f32", "window", "moe")
 
 
 class NativeError(RuntimeError):
