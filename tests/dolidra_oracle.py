@@ -64,17 +64,17 @@ def visible(i, window, keep_first=0):
     return [j for j in range(i + 1) if i - j < window or j < keep_first]
 
 
-def masked_attention(q, k, v, scale, window, keep_first=0):
-    """q [T, H, d], k [T, G, d], v [T, G, e] -> [T, H, e]."""
+def masked_attention(q, k, v, scale, window, keep_first=0, first=0):
+    """q [T, H, d] at positions ``first ..``, k [N, G, d], v [N, G, e] -> [T, H, e]."""
     share = q.shape[1] // k.shape[1]
-    out = torch.zeros(q.shape[0], q.shape[1], v.shape[2], dtype=torch.float64)
+    k, v = k.repeat_interleave(share, 1), v.repeat_interleave(share, 1)
+    out = []
     for i in range(q.shape[0]):
-        seen = visible(i, window, keep_first)
-        for h in range(q.shape[1]):
-            s = (k[seen, h // share] @ q[i, h]) * scale
-            e = torch.exp(s - s.max())
-            out[i, h] = (e / e.sum()) @ v[seen, h // share]
-    return out
+        seen = visible(first + i, window, keep_first)
+        s = torch.einsum("hd,jhd->hj", q[i], k[seen]) * scale
+        e = torch.exp(s - s.max(-1, keepdim=True).values)
+        out.append(torch.einsum("hj,jhe->he", e / e.sum(-1, keepdim=True), v[seen]))
+    return torch.stack(out)
 
 
 def difference_weight(w, p, diff):

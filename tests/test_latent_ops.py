@@ -9,28 +9,10 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
 import poralorn_oracle as oracle  # noqa: E402
+from op_helpers import BACKENDS, close, rand  # noqa: E402
 
 from prism_infer_b200 import ops  # noqa: E402
 from prism_infer_b200.ops import latent as lat  # noqa: E402
-
-CPU = pytest.param(("cpu", torch.float32), id="cpu")
-GPU32 = pytest.param(("cuda:0", torch.float32), marks=pytest.mark.gpu, id="gpu-float32")
-GPU16 = pytest.param(("cuda:0", torch.bfloat16), marks=pytest.mark.gpu, id="gpu-bfloat16")
-BACKENDS = [CPU, GPU32, GPU16]
-
-
-def rand(*shape, seed=0, scale=1.0, dtype=torch.float32, device="cpu"):
-    """Values every type can hold: drawn on the CPU and rounded to bf16."""
-    g = torch.Generator().manual_seed(seed)
-    return (torch.randn(*shape, generator=g) * scale).to(torch.bfloat16).to(dtype).to(device)
-
-
-def close(got, want, dtype, tol16=0.012, tol32=2e-5):
-    got, want = got.detach().double().cpu(), want.double()
-    assert got.shape == want.shape
-    err = (got - want).abs().max() / want.abs().max().clamp_min(1e-6)
-    assert float(err) < (tol16 if dtype == torch.bfloat16 else tol32), float(err)
-
 
 # ------------------------------------------------------------------------------------------ projections
 @pytest.mark.parametrize("backend", BACKENDS)
