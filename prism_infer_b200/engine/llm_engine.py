@@ -169,6 +169,7 @@ class LLMEngine:
         if self._closed:
             return
         self._closed = True
+        atexit.unregister(self.exit)  # the registration would keep a closed engine and its device memory alive
         try:
             self.runners.close()
         except Exception:  # pragma: no cover - shutdown must not raise

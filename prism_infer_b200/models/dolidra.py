@@ -286,7 +286,7 @@ class DolidraModel:
 
     def _project(self, x: torch.Tensor, w: torch.Tensor) -> lat.Branch:
         """A projection whose sum the next kernel forms: split-K slabs for up to a few hundred tokens, rows for long prompts."""
-        if self.device.type == "cuda" and self.dtype == torch.float32:
+        if self.device.type == "cuda" and (self.dtype == torch.float32 or ops.narrow_splits(w.shape[0], w.shape[1], x.shape[0]) > 1):
             return lat.Branch(slabs=lat.linear_slabs(x, w))
         dense, partials, _ = self.comm.row_parallel(x, w)
         return lat.Branch(slabs=partials, rows=dense)

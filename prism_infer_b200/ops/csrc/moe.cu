@@ -92,6 +92,8 @@ __device__ __forceinline__ void place(const RouteArgs& a, int t0, int n, int cou
   }
 }
 
+// C: groups of 32 routed experts
+template <int C>
 __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArgs a) {
   extern __shared__ int expert_s[];            // [chunk * K]
   __shared__ int count_s[MAX_EXPERTS], base_s[MAX_EXPERTS], scan_s[32];
@@ -103,26 +105,24 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArg
     const size_t t = (size_t)t0 + i;
     const bool live = a.slots[t] >= 0;
     // lane l holds experts l, l + 32, ...: the next best is found by a maximum over (value, lowest expert)
-    float v[MAX_EXPERTS / 32];
+    float v[C];
 #pragma unroll
-    for (int c = 0; c < MAX_EXPERTS / 32; ++c) {
-      v[c] = -INFINITY;
-      if (c * 32 < a.E) {
-        const int e = c * 32 + lane;
-        if (e < a.E) {
-          float s = 0.0f;
-          for (int p = 0; p < a.P; ++p) s += __ldcg(a.logits + (size_t)p * a.slab_stride + t * a.ld + e);
-          v[c] = s;
-        }
+    for (int c = 0; c < C; ++c) {
+      const int e = c * 32 + lane;
+      float s = 0.0f;
+      if (e < a.E) {
+#pragma unroll 16
+        for (int p = 0; p < a.P; ++p) s += __ldcg(a.logits + (size_t)p * a.slab_stride + t * a.ld + e);
       }
+      v[c] = e < a.E ? s : -INFINITY;
     }
     float best0 = 0.0f, sum = 0.0f;
     for (int k = 0; k < a.top; ++k) {
       float bv = -INFINITY;
       int be = MAX_EXPERTS;
 #pragma unroll
-      for (int c = 0; c < MAX_EXPERTS / 32; ++c)
-        if (c * 32 < a.E && v[c] > bv) {
+      for (int c = 0; c < C; ++c)
+        if (v[c] > bv) {
           bv = v[c];
           be = c * 32 + lane;
         }
@@ -137,7 +137,7 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArg
       }
       if (be >= a.E) be = 0;                   // no finite logit left: any expert, weight from its own logit
 #pragma unroll
-      for (int c = 0; c < MAX_EXPERTS / 32; ++c)
+      for (int c = 0; c < C; ++c)
         if (be == c * 32 + lane) v[c] = -INFINITY;
       if (k == 0) best0 = bv;
       const float w = expf(bv - best0);
@@ -228,8 +228,13 @@ PRISM_API int prism_moe_route(const void* logits, long long slab_stride, long lo
               (int*)counts, (int4*)groups, max_groups, (int*)n_groups, T, top, E, always, chunk, tile};
   if (int rc = check_route(a)) return rc;
   const size_t smem = (size_t)chunk * (top + always) * sizeof(int);
-  return (int)prism_launch(moe_route_kernel, dim3((T + chunk - 1) / chunk), dim3(ROUTE_THREADS), smem, reinterpret_cast<cudaStream_t>(stream),
-                           pdl != 0, a);
+  const dim3 grid((T + chunk - 1) / chunk), block(ROUTE_THREADS);
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (E <= 32) return (int)prism_launch(moe_route_kernel<1>, grid, block, smem, st, pdl != 0, a);
+  if (E <= 64) return (int)prism_launch(moe_route_kernel<2>, grid, block, smem, st, pdl != 0, a);
+  if (E <= 128) return (int)prism_launch(moe_route_kernel<4>, grid, block, smem, st, pdl != 0, a);
+  if (E <= 256) return (int)prism_launch(moe_route_kernel<8>, grid, block, smem, st, pdl != 0, a);
+  return (int)prism_launch(moe_route_kernel<MAX_EXPERTS / 32>, grid, block, smem, st, pdl != 0, a);
 }
 
 PRISM_API int prism_moe_place(void* expert, void* pos, void* weight, void* row_token, void* counts, void* groups, int max_groups,

@@ -135,12 +135,14 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return warp_sum(lane < nw ? red[lane] : 0.0f);
 }
 
-template <typename T>
-__global__ void __launch_bounds__(1024) stream_update_kernel(const StreamArgs<T> a) {
-  extern __shared__ float row[];  // W floats
+// A thread holds U groups of four columns in registers from the first load to the last store.
+template <typename T, int U>
+__global__ void __launch_bounds__(U == 1 ? 1024 : 512) stream_update_kernel(const StreamArgs<T> a) {
   __shared__ float red[2][32];
   const size_t t = blockIdx.x;
+  const int i0 = threadIdx.x * 4, step = blockDim.x * 4;
   pdl_launch_dependents();
+  F4 acc[U], x[U];
   pdl_wait();
   const T* emb = nullptr;
   if (a.ids != nullptr) {
@@ -148,55 +150,67 @@ __global__ void __launch_bounds__(1024) stream_update_kernel(const StreamArgs<T>
     if (id >= 0 && id < a.vocab) emb = a.table + (size_t)id * a.W;
     else if (threadIdx.x == 0) prism_report(PRISM_ERR_BOUNDS, 1);
   }
-  float ss = 0.0f, post = 0.0f;
-  if (a.a.post_w != nullptr) {  // the branch's own root mean square first; a thread meets its own columns again below
-    float bs = 0.0f;
-    for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4) {
-      const F4 d = branch_value(a.a, t, a.W, i);
-      store4(row + i, d);
+  const bool has_a = a.a.slabs != nullptr || a.a.rows != nullptr;
+  float bs = 0.0f;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) bs += d.v[e] * d.v[e];
+  for (int u = 0; u < U; ++u) {
+    const int i = i0 + u * step;
+    acc[u] = x[u] = F4{{0.0f, 0.0f, 0.0f, 0.0f}};
+    if (i < a.W) {
+      if (a.keep) x[u] = load4(a.x + t * a.W + i);
+      if (has_a) acc[u] = branch_value(a.a, t, a.W, i);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) bs += acc[u].v[e] * acc[u].v[e];
     }
-    post = a.mult / sqrtf(block_sum(bs, red[0]) / (float)a.W_real + a.eps);
   }
-  for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4) {
-    F4 acc{{0.0f, 0.0f, 0.0f, 0.0f}};
-    if (a.a.post_w != nullptr) {
-      const F4 d = load4(row + i), w = load4(a.a.post_w + i);
+  if (a.a.post_w != nullptr) {  // the branch over its own root mean square
+    const float post = a.mult / sqrtf(block_sum(bs, red[0]) / (float)a.W_real + a.eps);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc.v[e] = d.v[e] * post * w.v[e];
-    } else {
-      add_branch(a.a, t, a.W, i, a.mult, acc);
-    }
-    add_branch(a.b, t, a.W, i, a.mult, acc);
-    if (a.keep) {
-      const F4 x = load4(a.x + t * a.W + i);
+    for (int u = 0; u < U; ++u) {
+      if (i0 + u * step >= a.W) continue;
+      const F4 w = load4(a.a.post_w + i0 + u * step);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc.v[e] += x.v[e];
+      for (int e = 0; e < 4; ++e) acc[u].v[e] *= post * w.v[e];
     }
+  } else if (has_a) {
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[u].v[e] *= a.mult;
+  }
+  float ss = 0.0f;
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int i = i0 + u * step;
+    if (i >= a.W) continue;
+    add_branch(a.b, t, a.W, i, a.mult, acc[u]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[u].v[e] += x[u].v[e];
     if (a.bias != nullptr) {
       const F4 s = load4(a.bias + i);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc.v[e] += s.v[e];
+      for (int e = 0; e < 4; ++e) acc[u].v[e] += s.v[e];
     }
     if (emb != nullptr) {
       const F4 v = load4(emb + i);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc.v[e] += v.v[e];
+      for (int e = 0; e < 4; ++e) acc[u].v[e] += v.v[e];
       if (a.embed_out != nullptr) store4(a.embed_out + t * a.embed_ld + i, v);
     } else if (a.embed_out != nullptr) {
       store4(a.embed_out + t * a.embed_ld + i, F4{{0.0f, 0.0f, 0.0f, 0.0f}});
     }
-    store4(a.x + t * a.W + i, acc);
-    if (a.raw_out != nullptr) store4(a.raw_out + t * a.raw_ld + i, acc);
-    store4(row + i, acc);
+    store4(a.x + t * a.W + i, acc[u]);
+    if (a.raw_out != nullptr) store4(a.raw_out + t * a.raw_ld + i, acc[u]);
 #pragma unroll
-    for (int e = 0; e < 4; ++e) ss += acc.v[e] * acc.v[e];
+    for (int e = 0; e < 4; ++e) ss += acc[u].v[e] * acc[u].v[e];
   }
   if (a.norm_out == nullptr) return;
   const float inv = 1.0f / sqrtf(block_sum(ss, red[1]) / (float)a.W_real + a.eps);
-  for (int i = threadIdx.x * 4; i < a.W; i += blockDim.x * 4) {
-    F4 v = load4(row + i);
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int i = i0 + u * step;
+    if (i >= a.W) continue;
+    F4 v = acc[u];
 #pragma unroll
     for (int e = 0; e < 4; ++e) v.v[e] *= inv;
     if (a.norm_w != nullptr) {
@@ -279,14 +293,16 @@ int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* ta
   a.W = W;
   a.W_real = W_real;
   a.eps = eps;
-  int threads = (W / 4 + 31) / 32 * 32;
-  if (threads > 1024) threads = 1024;
-  const size_t smem = (size_t)W * sizeof(float);
-  if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(stream_update_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
+  // a few rows: as many threads as there are groups of four columns; many rows: several groups per thread
+  const int groups = W / 4;
+  const int U = groups <= 1024 && (T_rows < 256 || groups < 256) ? 1 : (groups <= 2048 ? 4 : (groups <= 4096 ? 8 : 16));
+  const dim3 grid(T_rows), block(((groups + U - 1) / U + 31) / 32 * 32);
+  switch (U) {
+    case 1: return (int)prism_launch(stream_update_kernel<T, 1>, grid, block, 0, stream, pdl, a);
+    case 4: return (int)prism_launch(stream_update_kernel<T, 4>, grid, block, 0, stream, pdl, a);
+    case 8: return (int)prism_launch(stream_update_kernel<T, 8>, grid, block, 0, stream, pdl, a);
   }
-  return (int)prism_launch(stream_update_kernel<T>, dim3(T_rows), dim3(threads), smem, stream, pdl, a);
+  return (int)prism_launch(stream_update_kernel<T, 16>, grid, block, 0, stream, pdl, a);
 }
 
 }  // namespace

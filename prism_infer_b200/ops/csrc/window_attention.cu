@@ -88,17 +88,39 @@ __device__ __forceinline__ float4 projected4(const PrepareArgs<T>& a, size_t t, 
   return v;
 }
 
+// A unit is four columns of a map of a head and, inside the rotated part, their four partners half the rotated width on.
+struct PrepareUnit {
+  int c, d;      // column of q | k, and inside the map
+  bool pair;
+};
 template <typename T>
-__global__ void __launch_bounds__(512) window_prepare_kernel(const PrepareArgs<T> a) {
-  extern __shared__ float sm[];
-  float* val = sm;                       // [nq + nk]
-  float* cs = sm + a.nq + a.nk;          // [rot / 2] cosines, then sines
+__device__ __forceinline__ PrepareUnit prepare_unit(const PrepareArgs<T>& a, int u, int per_map) {
+  const int pairs = a.rot >> 3, map = u / per_map, r = u - map * per_map;
+  PrepareUnit p;
+  p.pair = r < pairs;
+  p.d = p.pair ? r * 4 : a.rot + (r - pairs) * 4;
+  p.c = map * a.dq + p.d;
+  return p;
+}
+__device__ __forceinline__ float sum_sq(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+__device__ __forceinline__ float4 mul4(float4 v, float f, float4 w) { return make_float4(v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w); }
+
+// Threads keep their first PREP_U units in registers between the norm's sum and the rotation; others are read again.
+// Widths whose rotated half is not a multiple of four go element by element.
+constexpr int PREP_U = 2;
+
+template <typename T>
+__global__ void __launch_bounds__(512, 1) window_prepare_kernel(const PrepareArgs<T> a) {
+  extern __shared__ float cs[];          // [rot / 2] cosines, then sines
   __shared__ float red[2][16];
   const size_t t = blockIdx.x;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, half = a.rot >> 1;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, half = a.rot >> 1, nt = blockDim.x;
   pdl_launch_dependents();
   const float pos = (float)a.positions[t];
-  for (int i = tid; i < half; i += blockDim.x) sincosf(pos * a.freq[i], &cs[half + i], &cs[i]);
+  for (int i = tid; i < half; i += nt) sincosf(pos * a.freq[i], &cs[half + i], &cs[i]);
+  const int nqk = a.nq + a.nk, total = nqk + a.nv;
+  const bool vec = (half & 3) == 0, norm = a.q_w != nullptr;
+  const int per_map = vec ? (a.rot >> 3) + ((a.dq - a.rot) >> 2) : 1, units = vec ? nqk / a.dq * per_map : 0;
   pdl_wait();
   long long slot = a.slots[t];
   if (slot >= a.num_slots) {
@@ -106,21 +128,22 @@ __global__ void __launch_bounds__(512) window_prepare_kernel(const PrepareArgs<T
     slot = -1;
   }
   T* page_row = slot >= 0 ? a.cache + (size_t)slot * (a.nk + a.nv) : nullptr;
-  const int nqk = a.nq + a.nk, total = nqk + a.nv;
-  float sq = 0.0f, sk = 0.0f;
-  for (int c = tid * 4; c < total; c += blockDim.x * 4) {
-    const float4 v = projected4(a, t, c);
-    if (c < nqk) {
-      store4(val + c, v);
-      const float s = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-      if (c < a.nq) sq += s;
-      else sk += s;
-    } else if (page_row) {
-      store4(page_row + a.nk + (c - nqk), v);
+  float4 lo[PREP_U], hi[PREP_U];
+  PrepareUnit pu[PREP_U];
+#pragma unroll
+  for (int k = 0; k < PREP_U; ++k) {
+    const int u = tid + k * nt;
+    lo[k] = hi[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (u < units) {
+      pu[k] = prepare_unit(a, u, per_map);
+      lo[k] = projected4(a, t, pu[k].c);
+      if (pu[k].pair) hi[k] = projected4(a, t, pu[k].c + half);
     }
   }
+  if (page_row)
+    for (int c = tid * 4; c < a.nv; c += nt * 4) store4(page_row + a.nk + c, projected4(a, t, nqk + c));
   if (a.gate != nullptr)
-    for (int h = tid; h * 4 < a.H; h += blockDim.x) {
+    for (int h = tid; h * 4 < a.H; h += nt) {
       const float4 v = projected4(a, t, total + 4 * h);
       const float z[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
@@ -128,7 +151,21 @@ __global__ void __launch_bounds__(512) window_prepare_kernel(const PrepareArgs<T
         if (4 * h + e < a.H) a.gate[t * a.H + 4 * h + e] = 1.0f / (1.0f + expf(-z[e]));
     }
   float iq = 1.0f, ik = 1.0f;
-  if (a.q_w != nullptr) {
+  if (norm) {
+    float sq = 0.0f, sk = 0.0f;
+    if (vec) {
+#pragma unroll
+      for (int k = 0; k < PREP_U; ++k)
+        if (tid + k * nt < units) (pu[k].c < a.nq ? sq : sk) += sum_sq(lo[k]) + sum_sq(hi[k]);
+      for (int u = tid + PREP_U * nt; u < units; u += nt) {
+        const PrepareUnit p = prepare_unit(a, u, per_map);
+        float ss = sum_sq(projected4(a, t, p.c));
+        if (p.pair) ss += sum_sq(projected4(a, t, p.c + half));
+        (p.c < a.nq ? sq : sk) += ss;
+      }
+    } else {
+      for (int c = tid * 4; c < nqk; c += nt * 4) (c < a.nq ? sq : sk) += sum_sq(projected4(a, t, c));
+    }
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     if (lane == 0) {
@@ -137,38 +174,52 @@ __global__ void __launch_bounds__(512) window_prepare_kernel(const PrepareArgs<T
     }
   }
   __syncthreads();
-  if (a.q_w != nullptr) {
-    const int nw = blockDim.x >> 5;
-    sq = warp_sum(lane < nw ? red[0][lane] : 0.0f);
-    sk = warp_sum(lane < nw ? red[1][lane] : 0.0f);
-    iq = 1.0f / sqrtf(sq / (float)a.q_real + a.eps);
-    ik = 1.0f / sqrtf(sk / (float)a.k_real + a.eps);
-    for (int c = tid * 4; c < nqk; c += blockDim.x * 4) {
-      const float inv = c < a.nq ? iq : ik;
-      const float4 w = c < a.nq ? load4(a.q_w + c) : load4(a.k_w + c - a.nq);
-      float4 v = load4(val + c);
-      v.x *= inv * w.x;
-      v.y *= inv * w.y;
-      v.z *= inv * w.z;
-      v.w *= inv * w.w;
-      store4(val + c, v);
-    }
-    __syncthreads();
+  if (norm) {
+    const int nw = nt >> 5;
+    iq = 1.0f / sqrtf(warp_sum(lane < nw ? red[0][lane] : 0.0f) / (float)a.q_real + a.eps);
+    ik = 1.0f / sqrtf(warp_sum(lane < nw ? red[1][lane] : 0.0f) / (float)a.k_real + a.eps);
   }
-  for (int c = tid * 4; c < nqk; c += blockDim.x * 4) {
-    const int d0 = c % a.dq;
-    float o[4];
+  auto weight4 = [&](int c) { return c < a.nq ? load4(a.q_w + c) : load4(a.k_w + c - a.nq); };
+  auto write4 = [&](int c, float4 v) {
+    if (c < a.nq) store4(a.q_out + t * a.nq + c, v);
+    else if (page_row) store4(page_row + c - a.nq, v);
+  };
+  if (vec) {
+    auto finish = [&](const PrepareUnit& p, float4 x, float4 y) {
+      if (norm) {
+        const float inv = p.c < a.nq ? iq : ik;
+        x = mul4(x, inv, weight4(p.c));
+        if (p.pair) y = mul4(y, inv, weight4(p.c + half));
+      }
+      if (p.pair) {
+        const float4 co = load4(cs + p.d), si = load4(cs + half + p.d);
+        write4(p.c, make_float4(x.x * co.x - y.x * si.x, x.y * co.y - y.y * si.y, x.z * co.z - y.z * si.z, x.w * co.w - y.w * si.w));
+        write4(p.c + half, make_float4(y.x * co.x + x.x * si.x, y.y * co.y + x.y * si.y, y.z * co.z + x.z * si.z, y.w * co.w + x.w * si.w));
+      } else {
+        write4(p.c, x);
+      }
+    };
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int d = d0 + e;
-      const float v = val[c + e];
-      if (d < half) o[e] = v * cs[d] - val[c + e + half] * cs[half + d];
-      else if (d < a.rot) o[e] = v * cs[d - half] + val[c + e - half] * cs[d];
-      else o[e] = v;
+    for (int k = 0; k < PREP_U; ++k)
+      if (tid + k * nt < units) finish(pu[k], lo[k], hi[k]);
+    for (int u = tid + PREP_U * nt; u < units; u += nt) {
+      const PrepareUnit p = prepare_unit(a, u, per_map);
+      finish(p, projected4(a, t, p.c), p.pair ? projected4(a, t, p.c + half) : make_float4(0.f, 0.f, 0.f, 0.f));
     }
-    const float4 r = make_float4(o[0], o[1], o[2], o[3]);
-    if (c < a.nq) store4(a.q_out + t * a.nq + c, r);
-    else if (page_row) store4(page_row + c - a.nq, r);
+    return;
+  }
+  auto value = [&](int c) {
+    const float4 v = projected4(a, t, c & ~3);
+    const float f = (c & 2) ? ((c & 1) ? v.w : v.z) : ((c & 1) ? v.y : v.x);
+    return norm ? f * (c < a.nq ? iq * to_f(a.q_w[c]) : ik * to_f(a.k_w[c - a.nq])) : f;
+  };
+  for (int c = tid; c < nqk; c += nt) {
+    const int d = c % a.dq;
+    float o = value(c);
+    if (d < half) o = o * cs[d] - value(c + half) * cs[half + d];
+    else if (d < a.rot) o = o * cs[d - half] + value(c - half) * cs[d];
+    if (c < a.nq) put(a.q_out + t * a.nq + c, o);
+    else if (page_row) put(page_row + c - a.nq, o);
   }
 }
 
@@ -209,19 +260,29 @@ __device__ __forceinline__ TileList tile_list(int p_first, int p_last, int windo
 // =====================================================================================
 // Decode.  Rows of a CTA: up to 16 MT (head, map) pairs of one value head; a row's query sits in its own map's
 // columns of a maps x dq wide row and is zero elsewhere, so both maps are scored by one product with the concatenated
-// keys and weight the same values.  Each of the four warps owns 16 keys of every 64-key tile and streams them by
-// cp.async through its own ring; the warps meet only at the end.
+// keys and weight the same values.  Each of the four warps owns 16 keys of every 64-key tile and streams their rows by
+// bulk copies (one per lane: 16 key rows, 16 value rows) through its own ring; the warps meet only at the end.  Tiles
+// that hold only keys of earlier steps are fetched before the previous kernel has finished.
 // =====================================================================================
 constexpr int DEC_TILE = 64;
 
-template <int MT, int DVT>
+// `bytes` (a multiple of 16) from global to shared memory, completing on `bar`.
+__device__ __forceinline__ void bulk_row(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
+               "l"(src), "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
+}
+
+// KS: 16-element steps of the query kept in registers (0: read from shared memory every tile)
+template <int MT, int DVT, int KS>
 __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> a, const int stages) {
   extern __shared__ __align__(128) uint8_t smem_raw[];
   const int KD = a.maps * a.dq, LDQ = KD + 8, LDR = KD + a.dv + 8;  // an odd number of 16-byte steps: no bank conflicts
   constexpr int BM = 16 * MT;
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);                   // [BM][LDQ]
   bf16* ring = q_s + BM * LDQ;                                      // [4 warps][stages][16][LDR]
-  __shared__ float m_s[4][BM], l_s[4][BM];
+  __shared__ float m_s[4][BM], l_s[4][BM], f_s[4][BM], L_s[BM];
+  __shared__ __align__(8) uint64_t bars[4][4];
   __shared__ int last_s;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int share = a.H / a.G, rows_all = share * a.maps, blocks = (rows_all + BM - 1) / BM;
@@ -237,29 +298,34 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
   const int lo = pos - a.window;                                    // keys after lo are inside the window
   bf16* my = ring + (size_t)warp * stages * 16 * LDR;
-  const int kc = KD >> 3, chunks = kc + (a.dv >> 3);
+  if (lane < stages) mbar_init(&bars[warp][lane], 1);
+  fence_barrier_init();
+  __syncwarp();
 
   auto issue = [&](int t) {                                         // this warp's 16 keys of list entry t
-    if (t < te) {
-      const int key = tl.id(t) * DEC_TILE + warp * 16 + (lane & 15);
-      int blk = key < ctx ? checked_page(bt[key / a.page], a.num_blocks) : -1;
-      const long long row = blk >= 0 ? (long long)blk * a.page + key % a.page : -1;
-      bf16* dst = my + (size_t)((t - tb) % stages) * 16 * LDR;
-#pragma unroll 4
-      for (int i = 0; i < 16; ++i) {
-        const long long r = __shfl_sync(0xffffffffu, row, i);
-        const bf16* src = a.cache + (size_t)(r < 0 ? 0 : r) * a.R;
-        for (int c = lane; c < chunks; c += 32) {
-          const bool is_k = c < kc;
-          const int col = is_k ? kvh * KD + c * 8 : a.G * KD + kvh * a.dv + (c - kc) * 8;
-          cp_async16(dst + i * LDR + c * 8, src + col, r >= 0);
-        }
-      }
+    if (t >= te) return;
+    const int st = (t - tb) % stages, r = lane & 15;
+    const int key = tl.id(t) * DEC_TILE + warp * 16 + r;
+    const int blk = key < ctx ? checked_page(bt[key / a.page], a.num_blocks) : -1;
+    const bool ok = blk >= 0, is_k = lane < 16;
+    const unsigned live = __ballot_sync(0xffffffffu, ok) & 0xffffu;
+    if (lane == 0) mbar_expect_tx(&bars[warp][st], (uint32_t)__popc(live) * (uint32_t)(KD + a.dv) * 2u);
+    bf16* dst = my + ((size_t)st * 16 + r) * LDR + (is_k ? 0 : KD);
+    const int n = is_k ? KD : a.dv;
+    if (ok) {
+      const bf16* src = a.cache + ((size_t)blk * a.page + key % a.page) * a.R + (is_k ? kvh * KD : a.G * KD + kvh * a.dv);
+      fence_proxy_async();
+      bulk_row(dst, src, (uint32_t)n * 2u, &bars[warp][st]);
+    } else {                                                        // past the end, or a hole: zeros
+      for (int c = 0; c < n; c += 8) *reinterpret_cast<uint4*>(dst + c) = make_uint4(0, 0, 0, 0);
     }
-    cp_async_commit();
   };
+  // the newest key was written by the kernel before this one, all others in earlier steps
+  auto is_old = [&](int t) { return t < te && tl.id(t) * DEC_TILE + DEC_TILE <= pos; };
+  int ahead = 0;
+  while (ahead < stages - 1 && is_old(tb + ahead)) issue(tb + ahead++);
   pdl_wait();
-  for (int s = 0; s < stages - 1; ++s) issue(tb + s);
+  while (ahead < stages - 1) issue(tb + ahead++);
 
   for (int i = tid; i < BM * (LDQ / 8); i += 128) {
     const int r = i / (LDQ / 8), c = (i % (LDQ / 8)) * 8;
@@ -281,31 +347,52 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
     for (int n = 0; n < DVT; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.0f;
   }
   const float sl2 = a.scale * 1.4426950408889634f;
-  const int dvt = a.dv >> 3;
+  const int dvt = a.dv >> 3, ksteps = KD >> 4;
+  const bf16* qp = q_s + (lane & 15) * LDQ + 8 * (lane >> 4);
+  uint32_t qr[MT][KS > 0 ? KS : 1][4];
+  if (KS > 0) {
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int k = 0; k < KS; ++k)
+        if (k < ksteps) ldsm_x4(qr[m][k], smem_u32(qp + m * 16 * LDQ + k * 16));
+  }
   for (int t = tb; t < te; ++t) {
+    const int i = t - tb;
     issue(t + stages - 1);
-    // stages is 2, 3 or 4: all but the newest stages - 1 groups have landed
-    if (stages == 4) cp_async_wait<3>();
-    else if (stages == 3) cp_async_wait<2>();
-    else cp_async_wait<1>();
+    (void)mbar_wait(&bars[warp][i % stages], (i / stages) & 1, 51);
     __syncwarp();
-    const bf16* kv = my + (size_t)((t - tb) % stages) * 16 * LDR;
+    const bf16* kv = my + (size_t)(i % stages) * 16 * LDR;
     float s[MT][2][4] = {};
     const bf16* kp = kv + ((lane & 7) + 8 * (lane >> 4)) * LDR + 8 * ((lane >> 3) & 1);
-    const bf16* qp = q_s + (lane & 15) * LDQ + 8 * (lane >> 4);
-#pragma unroll 4
-    for (int kk = 0; kk < KD; kk += 16) {
-      uint32_t kb[4];
-      ldsm_x4(kb, smem_u32(kp + kk));
+    if (KS > 0) {
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        uint32_t qf[4];
-        ldsm_x4(qf, smem_u32(qp + m * 16 * LDQ + kk));
-        mma_bf16(s[m][0], qf, kb[0], kb[1]);
-        mma_bf16(s[m][1], qf, kb[2], kb[3]);
+      for (int k = 0; k < KS; ++k)
+        if (k < ksteps) {
+          uint32_t kb[4];
+          ldsm_x4(kb, smem_u32(kp + k * 16));
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            mma_bf16(s[m][0], qr[m][k], kb[0], kb[1]);
+            mma_bf16(s[m][1], qr[m][k], kb[2], kb[3]);
+          }
+        }
+    } else {
+#pragma unroll 4
+      for (int k = 0; k < ksteps; ++k) {
+        uint32_t kb[4];
+        ldsm_x4(kb, smem_u32(kp + k * 16));
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          uint32_t qf[4];
+          ldsm_x4(qf, smem_u32(qp + m * 16 * LDQ + k * 16));
+          mma_bf16(s[m][0], qf, kb[0], kb[1]);
+          mma_bf16(s[m][1], qf, kb[2], kb[3]);
+        }
       }
     }
     const int j0 = tl.id(t) * DEC_TILE + warp * 16;
+    const bool whole = j0 + 15 <= pos && (j0 > lo || j0 + 16 <= a.keep);  // every key of the warp is visible
     uint32_t pf[MT][4];
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
@@ -315,7 +402,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int j = j0 + n * 8 + t4 * 2 + (e & 1);
-          const bool ok = j <= pos && (j > lo || j < a.keep);
+          const bool ok = whole || (j <= pos && (j > lo || j < a.keep));
           s[m][n][e] = ok ? s[m][n][e] * sl2 : -INFINITY;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[m][n][e]);
         }
@@ -324,7 +411,8 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
       for (int r = 0; r < 2; ++r) {
         mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
         mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-        const float mn = fmaxf(m_run[m][r], mx[r]);
+        // the reference only rises when a tile exceeds it by more than 2^8: the weights stay below 256
+        const float mn = mx[r] > m_run[m][r] + 8.0f ? mx[r] : m_run[m][r];
         use[r] = mn == -INFINITY ? 0.0f : mn;
         corr[r] = ex2_fast(m_run[m][r] - use[r]);  // 0 before the first visible key
         m_run[m][r] = mn;
@@ -367,72 +455,63 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
     }
     __syncwarp();
   }
-  cp_async_wait_all();
-  __syncthreads();
+  __syncthreads();                                                  // every row that was issued has been waited for
 
-  // ---- the four warps meet: maxima and sums, then the weighted accumulators in shared memory
+  // ---- the four warps meet: accumulators, maxima and sums in shared memory
+  float* acc_s = reinterpret_cast<float*>(smem_raw);                // [4][BM][dv + 4]
+  const int LDA = a.dv + 4;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
+      const int row = m * 16 + g + 8 * r;
       float l = l_run[m][r];
       l += __shfl_xor_sync(0xffffffffu, l, 1);
       l += __shfl_xor_sync(0xffffffffu, l, 2);
       if (t4 == 0) {
-        m_s[warp][m * 16 + g + 8 * r] = m_run[m][r];
-        l_s[warp][m * 16 + g + 8 * r] = l;
+        m_s[warp][row] = m_run[m][r];
+        l_s[warp][row] = l;
+      }
+      if (row < rows) {
+#pragma unroll
+        for (int n = 0; n < DVT; ++n)
+          if (n < dvt)
+            *reinterpret_cast<float2*>(acc_s + ((size_t)warp * BM + row) * LDA + n * 8 + t4 * 2) = make_float2(o[m][n][2 * r], o[m][n][2 * r + 1]);
       }
     }
   __syncthreads();
-  float* acc_s = reinterpret_cast<float*>(smem_raw);                // [BM][dv + 4]
-  const int LDA = a.dv + 4;
-  for (int w = 0; w < 4; ++w) {
-    if (warp == w) {
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int row = m * 16 + g + 8 * r;
-          float mx = -INFINITY;
-#pragma unroll
-          for (int v = 0; v < 4; ++v) mx = fmaxf(mx, m_s[v][row]);
-          const float f = m_run[m][r] == -INFINITY ? 0.0f : ex2_fast(m_run[m][r] - mx);
-#pragma unroll
-          for (int n = 0; n < DVT; ++n)
-            if (n < dvt) {
-              float2* d = reinterpret_cast<float2*>(acc_s + row * LDA + n * 8 + t4 * 2);
-              float2 v = make_float2(o[m][n][2 * r] * f, o[m][n][2 * r + 1] * f);
-              if (w > 0) {
-                const float2 old = *d;
-                v.x += old.x;
-                v.y += old.y;
-              }
-              *d = v;
-            }
-        }
-    }
-    __syncthreads();
-  }
-  __shared__ float M_s[BM], L_s[BM];
+  const int group = seq * gridDim.y + blockIdx.y, per_row4 = a.dv >> 2;
+  const size_t base = ((size_t)group * a.nsplit + split) * BM;
   if (tid < BM) {
     float mx = -INFINITY, l = 0.0f;
 #pragma unroll
     for (int v = 0; v < 4; ++v) mx = fmaxf(mx, m_s[v][tid]);
 #pragma unroll
-    for (int v = 0; v < 4; ++v) l += m_s[v][tid] == -INFINITY ? 0.0f : l_s[v][tid] * ex2_fast(m_s[v][tid] - mx);
-    M_s[tid] = mx;
+    for (int v = 0; v < 4; ++v) {
+      const float f = m_s[v][tid] == -INFINITY ? 0.0f : ex2_fast(m_s[v][tid] - mx);
+      f_s[v][tid] = f;
+      l += l_s[v][tid] * f;
+    }
     L_s[tid] = l;
+    if (a.nsplit > 1 && tid < rows) *reinterpret_cast<float2*>(a.part_ml + (base + tid) * 2) = make_float2(mx, l);
   }
   __syncthreads();
-  const int group = seq * gridDim.y + blockIdx.y, per_row4 = a.dv >> 2;
+  for (int i = tid; i < rows * per_row4; i += 128) {
+    const int r = i / per_row4, c = (i % per_row4) * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float f = f_s[w][r];
+      const float4 p = load4(acc_s + ((size_t)w * BM + r) * LDA + c);
+      v.x += f * p.x;
+      v.y += f * p.y;
+      v.z += f * p.z;
+      v.w += f * p.w;
+    }
+    if (a.nsplit == 1) store4(acc_s + r * LDA + c, v);              // read by this thread only
+    else if (tb < te) store4(a.part_o + (base + r) * a.dv + c, v);
+  }
   if (a.nsplit > 1) {
-    const size_t base = ((size_t)group * a.nsplit + split) * BM;
-    if (tid < rows) *reinterpret_cast<float2*>(a.part_ml + (base + tid) * 2) = make_float2(M_s[tid], L_s[tid]);
-    if (tb < te)
-      for (int i = tid; i < rows * per_row4; i += 128) {
-        const int r = i / per_row4, c = (i % per_row4) * 4;
-        store4(a.part_o + (base + r) * a.dv + c, load4(acc_s + r * LDA + c));
-      }
     __threadfence();
     __syncthreads();
     if (tid == 0) {
@@ -462,18 +541,17 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
 #pragma unroll 8
       for (int s = 0; s < a.nsplit; ++s) {
         const float f = coef[r * a.nsplit + s];
-        if (f > 0.0f) {                                             // an empty split's rows were never written
-          const float4 p = __ldcg(reinterpret_cast<const float4*>(src + (size_t)s * BM * a.dv));
-          v.x += f * p.x;
-          v.y += f * p.y;
-          v.z += f * p.z;
-          v.w += f * p.w;
-        }
+        // an empty split's rows were never written
+        const float4 p = f > 0.0f ? __ldcg(reinterpret_cast<const float4*>(src + (size_t)s * BM * a.dv)) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v.x += f * p.x;
+        v.y += f * p.y;
+        v.z += f * p.z;
+        v.w += f * p.w;
       }
       store4(acc_s + r * LDA + c, v);
     }
-    __syncthreads();
   }
+  __syncthreads();
   // ---- combine maps, gate, store: one head per warp
   for (int hh = warp; hh < rows / a.maps; hh += 4) {
     const int r = hh * a.maps, h = head0 + hh;
@@ -710,13 +788,17 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       if (!ok) break;
       tc_fence_after();
       float v[PKT];
-#pragma unroll
-      for (int k = 0; k < PKT / 16; ++k) {
-        uint32_t r[16];
-        tmem_ld16(lanes + (s * 2 + b) * PKT + k * 16, r);
+      {
+        uint32_t(&r0)[16] = *reinterpret_cast<uint32_t(*)[16]>(&v[0]);
+        uint32_t(&r1)[16] = *reinterpret_cast<uint32_t(*)[16]>(&v[16]);
+        uint32_t(&r2)[16] = *reinterpret_cast<uint32_t(*)[16]>(&v[32]);
+        uint32_t(&r3)[16] = *reinterpret_cast<uint32_t(*)[16]>(&v[48]);
+        const uint32_t src = lanes + (s * 2 + b) * PKT;
+        tmem_ld16(src, r0);
+        tmem_ld16(src + 16, r1);
+        tmem_ld16(src + 32, r2);
+        tmem_ld16(src + 48, r3);
         tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 16; ++i) v[k * 16 + i] = __uint_as_float(r[i]) * sl2;
       }
       if (j0 + PKT - 1 > last_key || !(j0 > low || j0 + PKT <= a.keep)) {
 #pragma unroll
@@ -725,9 +807,10 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           if (j > last_key || (j <= low && j >= a.keep)) v[i] = -INFINITY;
         }
       }
-      float mx = v[0];
+      float m4[4] = {v[0], v[1], v[2], v[3]};
 #pragma unroll
-      for (int i = 1; i < PKT; ++i) mx = fmaxf(mx, v[i]);
+      for (int i = 4; i < PKT; ++i) m4[i & 3] = fmaxf(m4[i & 3], v[i]);
+      const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * sl2;  // scale > 0: the scaled maximum
       if (c == 0) {
         m_ref = mx;
       } else {
@@ -753,19 +836,20 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         }
       }
       const float m_use = m_ref == -INFINITY ? 0.0f : m_ref;
-      float sum = 0.0f;
+      float sum0 = 0.0f, sum1 = 0.0f;
 #pragma unroll
       for (int k = 0; k < PKT / 32; ++k) {
         uint32_t packed[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float p0 = ex2_fast(v[k * 32 + 2 * i] - m_use), p1 = ex2_fast(v[k * 32 + 2 * i + 1] - m_use);
-          sum += p0 + p1;
+          const float p0 = ex2_fast(fmaf(v[k * 32 + 2 * i], sl2, -m_use)), p1 = ex2_fast(fmaf(v[k * 32 + 2 * i + 1], sl2, -m_use));
+          sum0 += p0;
+          sum1 += p1;
           packed[i] = pack_bf16(p0, p1);
         }
         tmem_st16(lanes + (s * 2 + b) * PKT + k * 16, packed);
       }
-      l_run += sum;
+      l_run += sum0 + sum1;
       tmem_st_wait();
       tc_fence_before();
       mbar_arrive(&p_full[s * 2 + b]);
@@ -973,23 +1057,22 @@ int check_sizes(int H, int G, int maps, int dq, int dv, int vdim, int R, int pag
   return 0;
 }
 
-template <int MT, int DVT>
+template <int MT, int DVT, int KS>
 int launch_decode(const WinArgs<bf16>& a, int S, int blocks, cudaStream_t stream, bool pdl) {
   const int ldq = a.maps * a.dq + 8, ldr = ldq + a.dv;
   const size_t q_bytes = (size_t)16 * MT * ldq * 2, stage = (size_t)4 * 16 * ldr * 2;
-  const size_t merge = (size_t)16 * MT * (a.dv + 4 + a.nsplit) * 4;
-  int stages = 3;
-  if (q_bytes + stages * stage > 220 * 1024) stages = 2;
+  const size_t merge = (size_t)16 * MT * (4 * (a.dv + 4) + a.nsplit) * 4;
+  int stages = q_bytes + 3 * stage <= 72 * 1024 ? 3 : 2;  // three CTAs per SM where they fit
   size_t smem = q_bytes + stages * stage;
   if (smem < merge) smem = merge;
   if (smem > 227 * 1024) return -5;
   static size_t configured = 40 * 1024;
   if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<MT, DVT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(window_decode_kernel<MT, DVT, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  return (int)prism_launch(window_decode_kernel<MT, DVT>, dim3(S, a.G * blocks, a.nsplit), dim3(128), smem, stream, pdl, a, stages);
+  return (int)prism_launch(window_decode_kernel<MT, DVT, KS>, dim3(S, a.G * blocks, a.nsplit), dim3(128), smem, stream, pdl, a, stages);
 }
 
 template <typename T>
@@ -1012,15 +1095,9 @@ int launch_prepare(const void* slabs, long long slab_stride, int P, const void* 
   PrepareArgs<T> a{(const float*)slabs, slab_stride, P, (const T*)rows, ld, (const T*)bias, (const T*)q_w, (const T*)k_w,
                    (const float*)freq, (const int*)positions, (const long long*)slots, num_slots, (T*)q_out, (T*)cache, (float*)gate,
                    M, nq, nk, nv, H, dq, rot, q_real, k_real, eps};
-  const size_t smem = (size_t)(nq + nk + rot) * sizeof(float);
-  if (smem > 220 * 1024) return -5;
-  static size_t configured = 48 * 1024;
-  if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(window_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
-    configured = smem;
-  }
-  const int threads = M >= 2048 ? 512 : (M >= 512 ? 256 : 128);
+  const size_t smem = (size_t)(rot + 4) * sizeof(float);
+  if (smem > 48 * 1024) return -5;
+  const int threads = M >= 4096 && tokens <= 128 ? 512 : (M >= 512 ? 256 : 128);
   return (int)prism_launch(window_prepare_kernel<T>, dim3(tokens), dim3(threads), smem, stream, pdl, a);
 }
 
@@ -1063,9 +1140,14 @@ PRISM_API int prism_window_decode(const void* q, const void* cache, const void* 
   const int blocks = (H / G * maps + 16 * mt - 1) / (16 * mt);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const bool p = pdl != 0;
-  if (dv <= 64) return mt == 1 ? launch_decode<1, 8>(a, S, blocks, s, p) : launch_decode<2, 8>(a, S, blocks, s, p);
-  if (dv <= 128) return mt == 1 ? launch_decode<1, 16>(a, S, blocks, s, p) : launch_decode<2, 16>(a, S, blocks, s, p);
-  return launch_decode<1, 32>(a, S, blocks, s, p);
+  const bool regs = maps * dq <= 256;
+  if (dv <= 64)
+    return mt == 2 ? launch_decode<2, 8, 0>(a, S, blocks, s, p)
+                   : (regs ? launch_decode<1, 8, 16>(a, S, blocks, s, p) : launch_decode<1, 8, 0>(a, S, blocks, s, p));
+  if (dv <= 128)
+    return mt == 2 ? launch_decode<2, 16, 0>(a, S, blocks, s, p)
+                   : (regs ? launch_decode<1, 16, 16>(a, S, blocks, s, p) : launch_decode<1, 16, 0>(a, S, blocks, s, p));
+  return launch_decode<1, 32, 0>(a, S, blocks, s, p);
 }
 
 // Prompts and portions (cu_q: token offsets of the sequences), head widths up to 128, pages of a multiple of 8 rows.
@@ -1075,7 +1157,7 @@ PRISM_API int prism_window_prefill_tc(const void* q, const void* cache, const vo
                                       float scale, float lam, float gain, float eps, void* stream, int pdl) {
   if (T <= 0 || S <= 0 || max_q_len <= 0) return 0;
   if (int rc = check_sizes(H, G, maps, dq, dv, vdim, R, page, max_blocks, window, keep)) return rc;
-  if (dq > 128 || dv > 128 || page % 8 || !cu_q || num_blocks <= 0 || out_ld % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return -3;
+  if (dq > 128 || dv > 128 || page % 8 || !cu_q || num_blocks <= 0 || !(scale > 0.0f) || out_ld % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return -3;
   PrefillArgs p;
   p.w = win_args<bf16>(q, cache, block_tables, cu_q, kv_lens, gate, out, out_ld, H, G, maps, dq, dv, vdim, R, page, max_blocks, num_blocks,
                        window, keep, scale, lam, gain, eps);

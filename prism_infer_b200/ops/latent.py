@@ -15,7 +15,7 @@ from typing import Optional, Sequence
 import torch
 import torch.nn.functional as F
 
-from . import SM_COUNT, KVCache, _p, _pdl, _s, choose_splits, linear, linear_partial, native
+from . import SM_COUNT, KVCache, _p, _pdl, _s, choose_splits, linear, linear_partial, narrow_splits, native
 
 ACTS = {None: 0, "gelu_tanh": 1, "gelu": 2, "sigmoid": 3, "softcap": 4}
 MAX_SPLITS = 64
@@ -103,7 +103,8 @@ def linear_slabs(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         native.call("prism_gemm_f32", _p(w), _p(x), _p(out), w.shape[0], T, K, w.stride(0), x.stride(0), out.stride(1), None, 0,
                     None, None, None, 0.0, _s(), _pdl())
         return out
-    return linear_partial(x, w, choose_splits(w.shape[0], w.shape[1], x.shape[0]) if x.is_cuda else 1)
+    m, k, tokens = w.shape[0], w.shape[1], x.shape[0]
+    return linear_partial(x, w, max(choose_splits(m, k, tokens), narrow_splits(m, k, tokens)) if x.is_cuda else 1)
 
 
 # --------------------------------------------------------------------------------- residual stream

@@ -157,13 +157,13 @@ def _attention_cpu(q, spec, gate, pages, page, block_tables, kv_lens, cu):
 
 
 def _decode_geometry(spec: WindowSpec, batch: int, reach: int) -> tuple[int, int]:
-    """(16-row tiles per CTA, key splits): two CTAs' worth of work per SM where the visible keys allow it."""
+    """(16-row tiles per CTA, key splits): up to three CTAs per SM where the visible keys allow it."""
     rows = spec.heads // spec.kv_heads * spec.maps
     mt = 1 if rows <= 16 or spec.dv > 128 else 2
     blocks = batch * spec.kv_heads * -(-rows // (16 * mt))
     seen = min(reach, spec.window + KEY_TILE) + min(reach, spec.keep_first)
     tiles = max(1, -(-seen // KEY_TILE))
-    return mt, max(1, min(MAX_SPLITS, tiles, 2 * SM_COUNT // max(1, blocks)))
+    return mt, max(1, min(MAX_SPLITS, tiles, 3 * SM_COUNT // max(1, blocks)))
 
 
 def window_attention(q: torch.Tensor, spec: WindowSpec, gate: Optional[torch.Tensor], cache: KVCache, layer: int,
@@ -198,7 +198,7 @@ def window_attention(q: torch.Tensor, spec: WindowSpec, gate: Optional[torch.Ten
             counters = _decode_counters(q.device, S * blocks)
         native.call("prism_window_decode", *head, _p(po), _p(ml), _p(counters), S, *sizes, mt, ns, *tail)
         return out
-    if fast and not decode and spec.dq <= TC_MAX_HEAD and spec.dv <= TC_MAX_HEAD and cache.page % 8 == 0:
+    if fast and not decode and spec.dq <= TC_MAX_HEAD and spec.dv <= TC_MAX_HEAD and cache.page % 8 == 0 and spec.scale > 0.0:
         native.call("prism_window_prefill_tc", *head, T, S, int(max_q_len), *sizes, *tail)
         return out
     native.call("prism_window_attention_simple", 1 if q.dtype == torch.float32 else 0, *head, S, int(max_q_len), *sizes, *tail)

@@ -1,6 +1,7 @@
 """The Poralorn family through the engine (configuration, loading, paged latents, portions, mixed batches, greedy
 generation) against the plain statement in ``poralorn_oracle.py``: on the CPU in 32-bit, on a B200 in 32-bit and bf16."""
 
+import gc
 import json
 import os
 import subprocess
@@ -317,6 +318,9 @@ def test_cache_sized_from_free_memory(cuda_device, dtype):
     assert all(len(o["token_ids"]) == 6 for o in together)
     llm.check_device_status()
     llm.exit()
+    del llm
+    gc.collect()  # the cache takes a third of the device: give it back before the next test
+    torch.cuda.empty_cache()
 
 
 @pytest.mark.parametrize("backend", BACKENDS)
