@@ -95,21 +95,7 @@ __device__ __forceinline__ F4 branch_row(const Branch<T>& br, size_t r, int W, i
 
 template <typename T>
 __device__ __forceinline__ F4 branch_value(const Branch<T>& br, size_t t, int W, int i) {
-  F4 d;
-  if (br.pos != nullptr) {
-    d = F4{{0.0f, 0.0f, 0.0f, 0.0f}};
-#pragma unroll 4
-    for (int k = 0; k < br.K; ++k) {
-      const int r = __ldg(br.pos + t * br.K + k);
-      if (r < 0) continue;
-      const float w = __ldg(br.weight + t * br.K + k);
-      const F4 v = branch_row(br, (size_t)r, W, i);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) d.v[e] += w * v.v[e];
-    }
-  } else {
-    d = branch_row(br, t, W, i);
-  }
+  F4 d = branch_row(br, t, W, i);
   if (br.gate != nullptr) {
     const F4 g = load4(br.gate + t * br.gate_ld + i);
 #pragma unroll
@@ -137,7 +123,7 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 
 // A thread holds U groups of four columns in registers from the first load to the last store.
 template <typename T, int U>
-__global__ void __launch_bounds__(U == 1 ? 1024 : 512) stream_update_kernel(const StreamArgs<T> a) {
+__global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_update_kernel(const StreamArgs<T> a) {
   __shared__ float red[2][32];
   const size_t t = blockIdx.x;
   const int i0 = threadIdx.x * 4, step = blockDim.x * 4;
@@ -157,12 +143,28 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512) stream_update_kernel(cons
     const int i = i0 + u * step;
     acc[u] = x[u] = F4{{0.0f, 0.0f, 0.0f, 0.0f}};
     if (i < a.W) {
-      if (a.keep) x[u] = load4(a.x + t * a.W + i);
-      if (has_a) acc[u] = branch_value(a.a, t, a.W, i);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) bs += acc[u].v[e] * acc[u].v[e];
+      if (U == 1 && a.keep) x[u] = load4(a.x + t * a.W + i);
+      if (has_a && a.a.pos == nullptr) acc[u] = branch_value(a.a, t, a.W, i);
     }
   }
+  if (a.a.pos != nullptr) {  // all of a thread's columns of one row at a time
+    for (int k = 0; k < a.a.K; ++k) {
+      const int r = __ldg(a.a.pos + t * a.a.K + k);
+      if (r < 0) continue;
+      const float w = __ldg(a.a.weight + t * a.a.K + k);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        if (i0 + u * step >= a.W) continue;
+        const F4 v = branch_row(a.a, (size_t)r, a.W, i0 + u * step);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[u].v[e] += w * v.v[e];
+      }
+    }
+  }
+#pragma unroll
+  for (int u = 0; u < U; ++u)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) bs += acc[u].v[e] * acc[u].v[e];
   if (a.a.post_w != nullptr) {  // the branch over its own root mean square
     const float post = a.mult / sqrtf(block_sum(bs, red[0]) / (float)a.W_real + a.eps);
 #pragma unroll
@@ -183,6 +185,7 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512) stream_update_kernel(cons
   for (int u = 0; u < U; ++u) {
     const int i = i0 + u * step;
     if (i >= a.W) continue;
+    if (U > 1 && a.keep) x[u] = load4(a.x + t * a.W + i);
     add_branch(a.b, t, a.W, i, a.mult, acc[u]);
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[u].v[e] += x[u].v[e];
@@ -319,7 +322,7 @@ PRISM_API int prism_stream_update(int f32, int T, void* x, int keep, const void*
   if (T <= 0) return 0;
   if (W <= 0 || W % 8 || W_real <= 0 || W_real > W || W > 32768) return -1;
   if ((a_ld | b_ld | gate_ld | norm_ld | raw_ld | embed_ld) % 4) return -2;
-  if ((a_pos != nullptr && (a_K <= 0 || !a_weight)) || ((a_pos || a_post) && !a_slabs && !a_rows)) return -3;
+  if ((a_pos != nullptr && (a_K <= 0 || !a_weight || a_gate)) || ((a_pos || a_post) && !a_slabs && !a_rows)) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return f32 ? launch_stream<float>(T, x, keep, ids, table, vocab, a_slabs, a_stride, a_P, a_rows, a_ld, a_gate, b_slabs, b_stride,
                                     b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, mult, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,

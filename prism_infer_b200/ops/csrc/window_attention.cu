@@ -59,6 +59,7 @@ struct PrepareArgs {
   float* gate;             // [T][H] (null: no gates)
   int M, nq, nk, nv, H, dq, rot, q_real, k_real;
   float eps;
+  int shift;               // 2^shift unit places per map
 };
 
 template <typename T>
@@ -89,28 +90,29 @@ __device__ __forceinline__ float4 projected4(const PrepareArgs<T>& a, size_t t, 
 }
 
 // A unit is four columns of a map of a head and, inside the rotated part, their four partners half the rotated width on.
+// Units are numbered with 2^shift places per map, so that a unit's map and place come without a division.
 struct PrepareUnit {
-  int c, d;      // column of q | k, and inside the map
+  int c, d;      // column of q | k (< 0: an unused place), and inside the map
   bool pair;
 };
 template <typename T>
-__device__ __forceinline__ PrepareUnit prepare_unit(const PrepareArgs<T>& a, int u, int per_map) {
-  const int pairs = a.rot >> 3, map = u / per_map, r = u - map * per_map;
+__device__ __forceinline__ PrepareUnit prepare_unit(const PrepareArgs<T>& a, int u) {
+  const int pairs = a.rot >> 3, map = u >> a.shift, r = u & ((1 << a.shift) - 1);
   PrepareUnit p;
   p.pair = r < pairs;
   p.d = p.pair ? r * 4 : a.rot + (r - pairs) * 4;
-  p.c = map * a.dq + p.d;
+  p.c = p.d < a.dq && map * a.dq < a.nq + a.nk ? map * a.dq + p.d : -1;
   return p;
 }
 __device__ __forceinline__ float sum_sq(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 __device__ __forceinline__ float4 mul4(float4 v, float f, float4 w) { return make_float4(v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w); }
 
-// Threads keep their first PREP_U units in registers between the norm's sum and the rotation; others are read again.
-// Widths whose rotated half is not a multiple of four go element by element.
-constexpr int PREP_U = 2;
-
-template <typename T>
-__global__ void __launch_bounds__(512, 1) window_prepare_kernel(const PrepareArgs<T> a) {
+// Threads keep their first U units in registers between the norm's sum and the rotation; others are read again.
+// FEW tokens: more threads per token, norm weights fetched before the previous kernel has finished.  Widths whose rotated
+// half is not a multiple of four go element by element.
+template <typename T, bool FEW>
+__global__ void __launch_bounds__(FEW ? 512 : 256, FEW ? 1 : 4) window_prepare_kernel(const PrepareArgs<T> a) {
+  constexpr int U = 2;
   extern __shared__ float cs[];          // [rot / 2] cosines, then sines
   __shared__ float red[2][16];
   const size_t t = blockIdx.x;
@@ -120,7 +122,20 @@ __global__ void __launch_bounds__(512, 1) window_prepare_kernel(const PrepareArg
   for (int i = tid; i < half; i += nt) sincosf(pos * a.freq[i], &cs[half + i], &cs[i]);
   const int nqk = a.nq + a.nk, total = nqk + a.nv;
   const bool vec = (half & 3) == 0, norm = a.q_w != nullptr;
-  const int per_map = vec ? (a.rot >> 3) + ((a.dq - a.rot) >> 2) : 1, units = vec ? nqk / a.dq * per_map : 0;
+  const int units = vec ? (nqk / a.dq) << a.shift : 0;
+  PrepareUnit pu[U];
+  float4 w_lo[FEW ? U : 1], w_hi[FEW ? U : 1];
+  auto weight4 = [&](int c) { return c < a.nq ? load4(a.q_w + c) : load4(a.k_w + c - a.nq); };
+#pragma unroll
+  for (int k = 0; k < U; ++k) {
+    const int u = tid + k * nt;
+    pu[k].c = -1;
+    if (u < units) pu[k] = prepare_unit(a, u);
+    if (FEW && norm && pu[k].c >= 0) {
+      w_lo[k] = weight4(pu[k].c);
+      if (pu[k].pair) w_hi[k] = weight4(pu[k].c + half);
+    }
+  }
   pdl_wait();
   long long slot = a.slots[t];
   if (slot >= a.num_slots) {
@@ -128,14 +143,11 @@ __global__ void __launch_bounds__(512, 1) window_prepare_kernel(const PrepareArg
     slot = -1;
   }
   T* page_row = slot >= 0 ? a.cache + (size_t)slot * (a.nk + a.nv) : nullptr;
-  float4 lo[PREP_U], hi[PREP_U];
-  PrepareUnit pu[PREP_U];
+  float4 lo[U], hi[U];
 #pragma unroll
-  for (int k = 0; k < PREP_U; ++k) {
-    const int u = tid + k * nt;
+  for (int k = 0; k < U; ++k) {
     lo[k] = hi[k] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (u < units) {
-      pu[k] = prepare_unit(a, u, per_map);
+    if (pu[k].c >= 0) {
       lo[k] = projected4(a, t, pu[k].c);
       if (pu[k].pair) hi[k] = projected4(a, t, pu[k].c + half);
     }
@@ -155,10 +167,10 @@ __global__ void __launch_bounds__(512, 1) window_prepare_kernel(const PrepareArg
     float sq = 0.0f, sk = 0.0f;
     if (vec) {
 #pragma unroll
-      for (int k = 0; k < PREP_U; ++k)
-        if (tid + k * nt < units) (pu[k].c < a.nq ? sq : sk) += sum_sq(lo[k]) + sum_sq(hi[k]);
-      for (int u = tid + PREP_U * nt; u < units; u += nt) {
-        const PrepareUnit p = prepare_unit(a, u, per_map);
+      for (int k = 0; k < U; ++k) (pu[k].c < a.nq ? sq : sk) += sum_sq(lo[k]) + sum_sq(hi[k]);
+      for (int u = tid + U * nt; u < units; u += nt) {
+        const PrepareUnit p = prepare_unit(a, u);
+        if (p.c < 0) continue;
         float ss = sum_sq(projected4(a, t, p.c));
         if (p.pair) ss += sum_sq(projected4(a, t, p.c + half));
         (p.c < a.nq ? sq : sk) += ss;
@@ -179,17 +191,16 @@ __global__ void __launch_bounds__(512, 1) window_prepare_kernel(const PrepareArg
     iq = 1.0f / sqrtf(warp_sum(lane < nw ? red[0][lane] : 0.0f) / (float)a.q_real + a.eps);
     ik = 1.0f / sqrtf(warp_sum(lane < nw ? red[1][lane] : 0.0f) / (float)a.k_real + a.eps);
   }
-  auto weight4 = [&](int c) { return c < a.nq ? load4(a.q_w + c) : load4(a.k_w + c - a.nq); };
   auto write4 = [&](int c, float4 v) {
     if (c < a.nq) store4(a.q_out + t * a.nq + c, v);
     else if (page_row) store4(page_row + c - a.nq, v);
   };
   if (vec) {
-    auto finish = [&](const PrepareUnit& p, float4 x, float4 y) {
+    auto finish = [&](const PrepareUnit& p, float4 x, float4 y, float4 wx, float4 wy) {
       if (norm) {
         const float inv = p.c < a.nq ? iq : ik;
-        x = mul4(x, inv, weight4(p.c));
-        if (p.pair) y = mul4(y, inv, weight4(p.c + half));
+        x = mul4(x, inv, wx);
+        if (p.pair) y = mul4(y, inv, wy);
       }
       if (p.pair) {
         const float4 co = load4(cs + p.d), si = load4(cs + half + p.d);
@@ -199,12 +210,18 @@ __global__ void __launch_bounds__(512, 1) window_prepare_kernel(const PrepareArg
         write4(p.c, x);
       }
     };
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int k = 0; k < PREP_U; ++k)
-      if (tid + k * nt < units) finish(pu[k], lo[k], hi[k]);
-    for (int u = tid + PREP_U * nt; u < units; u += nt) {
-      const PrepareUnit p = prepare_unit(a, u, per_map);
-      finish(p, projected4(a, t, p.c), p.pair ? projected4(a, t, p.c + half) : make_float4(0.f, 0.f, 0.f, 0.f));
+    for (int k = 0; k < U; ++k)
+      if (pu[k].c >= 0) {
+        if (FEW) finish(pu[k], lo[k], hi[k], w_lo[k], w_hi[k]);
+        else finish(pu[k], lo[k], hi[k], norm ? weight4(pu[k].c) : zero, norm && pu[k].pair ? weight4(pu[k].c + half) : zero);
+      }
+    for (int u = tid + U * nt; u < units; u += nt) {
+      const PrepareUnit p = prepare_unit(a, u);
+      if (p.c < 0) continue;
+      finish(p, projected4(a, t, p.c), p.pair ? projected4(a, t, p.c + half) : zero, norm ? weight4(p.c) : zero,
+             norm && p.pair ? weight4(p.c + half) : zero);
     }
     return;
   }
@@ -1094,11 +1111,13 @@ int launch_prepare(const void* slabs, long long slab_stride, int P, const void* 
                    float eps, cudaStream_t stream, bool pdl) {
   PrepareArgs<T> a{(const float*)slabs, slab_stride, P, (const T*)rows, ld, (const T*)bias, (const T*)q_w, (const T*)k_w,
                    (const float*)freq, (const int*)positions, (const long long*)slots, num_slots, (T*)q_out, (T*)cache, (float*)gate,
-                   M, nq, nk, nv, H, dq, rot, q_real, k_real, eps};
+                   M, nq, nk, nv, H, dq, rot, q_real, k_real, eps, 0};
+  while ((1 << a.shift) < rot / 8 + (dq - rot) / 4) ++a.shift;
   const size_t smem = (size_t)(rot + 4) * sizeof(float);
   if (smem > 48 * 1024) return -5;
-  const int threads = M >= 4096 && tokens <= 128 ? 512 : (M >= 512 ? 256 : 128);
-  return (int)prism_launch(window_prepare_kernel<T>, dim3(tokens), dim3(threads), smem, stream, pdl, a);
+  if (tokens <= 256)
+    return (int)prism_launch(window_prepare_kernel<T, true>, dim3(tokens), dim3(M >= 4096 ? 512 : 256), smem, stream, pdl, a);
+  return (int)prism_launch(window_prepare_kernel<T, false>, dim3(tokens), dim3(256), smem, stream, pdl, a);
 }
 
 }  // namespace
