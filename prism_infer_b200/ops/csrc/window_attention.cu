@@ -601,15 +601,15 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
 //   two maps            the two maps of one head: own queries and keys, shared values
 //   one map, even group two heads of one value head: shared keys and values
 //   one map, odd group  two consecutive query tiles of one head: shared keys and values
-// Warp 0 streams key and value tiles of 64 rows from the pages by TMA, one thread of warp 1 issues the MMAs; warps
-// 2 - 5 and 6 - 9 are the softmax of stream 0 and 1, one thread per query row.
+// Warp 0 streams key and value tiles of 64 rows from the pages by TMA, one thread of warp 1 issues the MMAs of stream 0
+// and one of warp 10 those of stream 1; warps 2 - 5 and 6 - 9 are the streams' softmax, one thread per query row.
 //   S[s][b] = Q_s K^T (two buffers per stream), P written over S as bf16, O_s += P V with P read from TMEM.
 // A tile that no row of a stream sees is skipped for that stream; every role derives the same list.
 // TMEM: S 4 x 64 columns, O 2 x 128.  Every wait is bounded; on a timeout the roles unwind and TMEM is freed.
 // =====================================================================================
 constexpr int PT = 128;          // query rows per stream
 constexpr int PKT = 64;          // keys per tile
-constexpr int PRE_THREADS = 320;
+constexpr int PRE_THREADS = 352;
 constexpr int Q_ATOM = PT * 128, KV_ATOM = PKT * 128;   // bytes of a 64-column atom
 constexpr int TM_O = 256;
 
@@ -659,7 +659,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       mbar_init(&p_full[i], 128);
       mbar_init(&pv_done[i], 1);
       mbar_init(&kv_full[i], 1);
-      mbar_init(&kv_empty[i], 1);
+      mbar_init(&kv_empty[i], 2);
     }
     fence_barrier_init();
     tma_prefetch_desc(&tmQ);
@@ -728,29 +728,35 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       if (!ok)
         for (int t = max(0, issued - p.stages); t < issued; ++t) (void)mbar_wait(&kv_full[t % p.stages], (t / p.stages) & 1, 42);
     }
-  } else if (warp == 1) {
+  } else if (warp == 1 || warp == 10) {
     if (lane == 0 && live) {
-      // ------------------------------ MMA issuer ------------------------------
+      // ------------------------------ MMA issuer of one stream ------------------------------
+      const int s = warp == 1 ? 0 : 1;
       const uint32_t idesc_s = umma_idesc_bf16(PT, PKT);
       const uint32_t idesc_o = umma_idesc_bf16(PT, a.dv) | UMMA_B_MN_MAJOR;
       const int ksteps = a.dq >> 4;
-      int sc[2] = {0, 0}, pc[2] = {0, 0};
+      // descriptors of stage 0; a stage further on is stage_bytes / 16 higher
+      const uint64_t q_desc = umma_desc_sw128(smem_u32(q_s + s * q_bytes));
+      const uint64_t k_desc = umma_desc_sw128(smem_u32(ring + (p.k_maps == 2 ? s * k_bytes : 0)));
+      const uint64_t v_desc = umma_desc_sw128_mn(smem_u32(ring + p.k_maps * k_bytes), KV_ATOM);
+      const uint32_t s_tmem = tmem_base + s * 2 * PKT, o_tmem = tmem_base + TM_O + s * 128;
+      int sc = 0, pc = 0, st_next = 0, st = 0;
+      uint32_t ph_next = 0;
       bool ok = mbar_wait(q_full, 0, 43);
-      auto score = [&](int t) {
-        const uint32_t st = smem_u32(ring + (size_t)(t % p.stages) * stage_bytes);
+      auto score = [&](int t) {  // S of tile t, which is in stage st_next
+        if (active(s, t)) {
+          const uint64_t kd = k_desc + (uint64_t)((uint32_t)(st_next * stage_bytes) >> 4);
+          const uint32_t d = s_tmem + (sc & 1) * PKT;
 #pragma unroll
-        for (int s = 0; s < 2; ++s) {
-          if (!active(s, t)) continue;
-          const int b = sc[s] & 1;
-          const uint32_t qb = smem_u32(q_s + s * q_bytes), kb = st + (p.k_maps == 2 ? s * k_bytes : 0);
-          const uint32_t d = tmem_base + (s * 2 + b) * PKT;
-          for (int k = 0; k < ksteps; ++k) {
-            const uint64_t da = umma_desc_sw128(qb + (k >> 2) * Q_ATOM) + 2 * (k & 3);
-            const uint64_t db = umma_desc_sw128(kb + (k >> 2) * KV_ATOM) + 2 * (k & 3);
-            tc_mma_f16(d, da, db, idesc_s, k != 0);
-          }
-          tc_commit(&s_full[s * 2 + b]);
-          ++sc[s];
+          for (int k = 0; k < 8; ++k)
+            if (k < ksteps)
+              tc_mma_f16(d, q_desc + ((k >> 2) * (Q_ATOM >> 4) + 2 * (k & 3)), kd + ((k >> 2) * (KV_ATOM >> 4) + 2 * (k & 3)), idesc_s, k != 0);
+          tc_commit(&s_full[s * 2 + (sc & 1)]);
+          ++sc;
+        }
+        if (++st_next == p.stages) {
+          st_next = 0;
+          ph_next ^= 1;
         }
       };
       if (ok) ok = mbar_wait(&kv_full[0], 0, 44);
@@ -760,29 +766,24 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       }
       for (int t = 0; t < n_tiles && ok; ++t) {
         if (t + 1 < n_tiles) {
-          ok = mbar_wait(&kv_full[(t + 1) % p.stages], ((t + 1) / p.stages) & 1, 45);
+          ok = mbar_wait(&kv_full[st_next], ph_next, 45);
           if (!ok) break;
           tc_fence_after();
           score(t + 1);  // into the buffer whose P V was issued before: it is read first
         }
-        const uint32_t vt = smem_u32(ring + (size_t)(t % p.stages) * stage_bytes + p.k_maps * k_bytes);
-#pragma unroll
-        for (int s = 0; s < 2; ++s) {
-          if (!ok || !active(s, t)) continue;
-          const int b = pc[s] & 1;
-          ok = mbar_wait(&p_full[s * 2 + b], (pc[s] >> 1) & 1, 46);
-          if (!ok) continue;
+        if (active(s, t)) {
+          const int b = pc & 1;
+          ok = mbar_wait(&p_full[s * 2 + b], (pc >> 1) & 1, 46);
+          if (!ok) break;
           tc_fence_after();
-          const uint32_t pt = tmem_base + (s * 2 + b) * PKT, d = tmem_base + TM_O + s * 128;
+          const uint64_t vd = v_desc + (uint64_t)((uint32_t)(st * stage_bytes) >> 4);
 #pragma unroll
-          for (int k = 0; k < PKT / 16; ++k) {
-            const uint64_t db = umma_desc_sw128_mn(vt + k * 2048, KV_ATOM);
-            tc_mma_f16_ts(d, pt + k * 8, db, idesc_o, (pc[s] | k) != 0);
-          }
+          for (int k = 0; k < PKT / 16; ++k) tc_mma_f16_ts(o_tmem, s_tmem + b * PKT + k * 8, vd + k * (2048 >> 4), idesc_o, (pc | k) != 0);
           tc_commit(&pv_done[s * 2 + b]);
-          ++pc[s];
+          ++pc;
         }
-        if (ok) tc_commit(&kv_empty[t % p.stages]);
+        tc_commit(&kv_empty[st]);  // one arrival per stream
+        if (++st == p.stages) st = 0;
       }
     }
   } else if (live) {
