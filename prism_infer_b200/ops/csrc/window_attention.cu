@@ -107,19 +107,35 @@ __device__ __forceinline__ PrepareUnit prepare_unit(const PrepareArgs<T>& a, int
 __device__ __forceinline__ float sum_sq(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 __device__ __forceinline__ float4 mul4(float4 v, float f, float4 w) { return make_float4(v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w); }
 
+constexpr int PREP_PARTS = 4;
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+__device__ __forceinline__ float cluster_load(const float* own, int rank) {
+  float v;
+  asm volatile(
+      "{\n\t.reg .b32 a;\n\t"
+      "mapa.shared::cluster.u32 a, %1, %2;\n\t"
+      "ld.shared::cluster.f32 %0, [a];\n\t}"
+      : "=f"(v)
+      : "r"(smem_u32(own)), "r"(rank)
+      : "memory");
+  return v;
+}
+
 // Threads keep their first U units in registers between the norm's sum and the rotation; others are read again.
-// FEW tokens: more threads per token, norm weights fetched before the previous kernel has finished.  Widths whose rotated
-// half is not a multiple of four go element by element.
+// FEW tokens: a cluster of PREP_PARTS CTAs per token, norm weights fetched before the previous kernel has finished.  Widths
+// whose rotated half is not a multiple of four go element by element.
 template <typename T, bool FEW>
-__global__ void __launch_bounds__(FEW ? 512 : 256, FEW ? 1 : 4) window_prepare_kernel(const PrepareArgs<T> a) {
-  constexpr int U = 2;
+__device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
+  constexpr int U = 2, PARTS = FEW ? PREP_PARTS : 1;
   extern __shared__ float cs[];          // [rot / 2] cosines, then sines
-  __shared__ float red[2][16];
-  const size_t t = blockIdx.x;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, half = a.rot >> 1, nt = blockDim.x;
+  __shared__ float red[2][8], part_s[2];
+  const size_t t = blockIdx.x / PARTS;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = a.rot >> 1;
+  const int part = blockIdx.x % PARTS, tid = part * blockDim.x + threadIdx.x, nt = PARTS * blockDim.x;  // threads of the token
   pdl_launch_dependents();
   const float pos = (float)a.positions[t];
-  for (int i = tid; i < half; i += nt) sincosf(pos * a.freq[i], &cs[half + i], &cs[i]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * a.freq[i], &cs[half + i], &cs[i]);
   const int nqk = a.nq + a.nk, total = nqk + a.nv;
   const bool vec = (half & 3) == 0, norm = a.q_w != nullptr;
   const int units = vec ? (nqk / a.dq) << a.shift : 0;
@@ -187,9 +203,26 @@ __global__ void __launch_bounds__(FEW ? 512 : 256, FEW ? 1 : 4) window_prepare_k
   }
   __syncthreads();
   if (norm) {
-    const int nw = nt >> 5;
-    iq = 1.0f / sqrtf(warp_sum(lane < nw ? red[0][lane] : 0.0f) / (float)a.q_real + a.eps);
-    ik = 1.0f / sqrtf(warp_sum(lane < nw ? red[1][lane] : 0.0f) / (float)a.k_real + a.eps);
+    const int nw = blockDim.x >> 5;
+    float sq = warp_sum(lane < nw ? red[0][lane] : 0.0f), sk = warp_sum(lane < nw ? red[1][lane] : 0.0f);
+    if (FEW) {                           // the parts of a token add up through distributed shared memory, in their order
+      if (threadIdx.x == 0) {
+        part_s[0] = sq;
+        part_s[1] = sk;
+      }
+      __syncwarp();
+      cluster_arrive();
+      cluster_wait();
+      sq = sk = 0.0f;
+#pragma unroll
+      for (int r = 0; r < PARTS; ++r) {
+        sq += cluster_load(&part_s[0], r);
+        sk += cluster_load(&part_s[1], r);
+      }
+      cluster_arrive();                  // a part leaves only after the others have read its sums
+    }
+    iq = 1.0f / sqrtf(sq / (float)a.q_real + a.eps);
+    ik = 1.0f / sqrtf(sk / (float)a.k_real + a.eps);
   }
   auto write4 = [&](int c, float4 v) {
     if (c < a.nq) store4(a.q_out + t * a.nq + c, v);
@@ -223,21 +256,34 @@ __global__ void __launch_bounds__(FEW ? 512 : 256, FEW ? 1 : 4) window_prepare_k
       finish(p, projected4(a, t, p.c), p.pair ? projected4(a, t, p.c + half) : zero, norm ? weight4(p.c) : zero,
              norm && p.pair ? weight4(p.c + half) : zero);
     }
-    return;
+  } else {
+    auto value = [&](int c) {
+      const float4 v = projected4(a, t, c & ~3);
+      const float f = (c & 2) ? ((c & 1) ? v.w : v.z) : ((c & 1) ? v.y : v.x);
+      return norm ? f * (c < a.nq ? iq * to_f(a.q_w[c]) : ik * to_f(a.k_w[c - a.nq])) : f;
+    };
+    for (int c = tid; c < nqk; c += nt) {
+      const int d = c % a.dq;
+      float o = value(c);
+      if (d < half) o = o * cs[d] - value(c + half) * cs[half + d];
+      else if (d < a.rot) o = o * cs[d - half] + value(c - half) * cs[d];
+      if (c < a.nq) put(a.q_out + t * a.nq + c, o);
+      else if (page_row) put(page_row + c - a.nq, o);
+    }
   }
-  auto value = [&](int c) {
-    const float4 v = projected4(a, t, c & ~3);
-    const float f = (c & 2) ? ((c & 1) ? v.w : v.z) : ((c & 1) ? v.y : v.x);
-    return norm ? f * (c < a.nq ? iq * to_f(a.q_w[c]) : ik * to_f(a.k_w[c - a.nq])) : f;
-  };
-  for (int c = tid; c < nqk; c += nt) {
-    const int d = c % a.dq;
-    float o = value(c);
-    if (d < half) o = o * cs[d] - value(c + half) * cs[half + d];
-    else if (d < a.rot) o = o * cs[d - half] + value(c - half) * cs[d];
-    if (c < a.nq) put(a.q_out + t * a.nq + c, o);
-    else if (page_row) put(page_row + c - a.nq, o);
+  if (FEW && norm) {
+    __syncwarp();
+    cluster_wait();
   }
+}
+
+template <typename T>
+__global__ void __cluster_dims__(PREP_PARTS, 1, 1) __launch_bounds__(256) window_prepare_few_kernel(const PrepareArgs<T> a) {
+  prepare_token<T, true>(a);
+}
+template <typename T>
+__global__ void __launch_bounds__(256, 4) window_prepare_kernel(const PrepareArgs<T> a) {
+  prepare_token<T, false>(a);
 }
 
 // =====================================================================================
@@ -1116,9 +1162,10 @@ int launch_prepare(const void* slabs, long long slab_stride, int P, const void* 
   while ((1 << a.shift) < rot / 8 + (dq - rot) / 4) ++a.shift;
   const size_t smem = (size_t)(rot + 4) * sizeof(float);
   if (smem > 48 * 1024) return -5;
-  if (tokens <= 256)
-    return (int)prism_launch(window_prepare_kernel<T, true>, dim3(tokens), dim3(M >= 4096 ? 512 : 256), smem, stream, pdl, a);
-  return (int)prism_launch(window_prepare_kernel<T, false>, dim3(tokens), dim3(256), smem, stream, pdl, a);
+  // with a norm the cluster's exchange costs more than it spreads from a few dozen tokens on
+  if (tokens <= (q_w != nullptr ? 16 : 256))
+    return (int)prism_launch(window_prepare_few_kernel<T>, dim3(tokens * PREP_PARTS), dim3(M >= 4096 ? 256 : 128), smem, stream, pdl, a);
+  return (int)prism_launch(window_prepare_kernel<T>, dim3(tokens), dim3(256), smem, stream, pdl, a);
 }
 
 }  // namespace
