@@ -123,13 +123,13 @@ __device__ __forceinline__ float cluster_load(const float* own, int rank) {
 }
 
 // Threads keep their first U units in registers between the norm's sum and the rotation; others are read again.
-// FEW tokens: a cluster of PREP_PARTS CTAs per token, norm weights fetched before the previous kernel has finished.  Widths
+// PARTS CTAs (a cluster) per token; FEW tokens: norm weights fetched before the previous kernel has finished.  Widths
 // whose rotated half is not a multiple of four go element by element.
-template <typename T, bool FEW>
+template <typename T, int PARTS, bool FEW>
 __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
-  constexpr int U = 2, PARTS = FEW ? PREP_PARTS : 1;
+  constexpr int U = 2;
   extern __shared__ float cs[];          // [rot / 2] cosines, then sines
-  __shared__ float red[2][8], part_s[2];
+  __shared__ float red[2][16], part_s[2];
   const size_t t = blockIdx.x / PARTS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = a.rot >> 1;
   const int part = blockIdx.x % PARTS, tid = part * blockDim.x + threadIdx.x, nt = PARTS * blockDim.x;  // threads of the token
@@ -205,7 +205,7 @@ __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
   if (norm) {
     const int nw = blockDim.x >> 5;
     float sq = warp_sum(lane < nw ? red[0][lane] : 0.0f), sk = warp_sum(lane < nw ? red[1][lane] : 0.0f);
-    if (FEW) {                           // the parts of a token add up through distributed shared memory, in their order
+    if (PARTS > 1) {                     // the parts of a token add up through distributed shared memory, in their order
       if (threadIdx.x == 0) {
         part_s[0] = sq;
         part_s[1] = sk;
@@ -271,7 +271,7 @@ __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
       else if (page_row) put(page_row + c - a.nq, o);
     }
   }
-  if (FEW && norm) {
+  if (PARTS > 1 && norm) {
     __syncwarp();
     cluster_wait();
   }
@@ -279,11 +279,15 @@ __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
 
 template <typename T>
 __global__ void __cluster_dims__(PREP_PARTS, 1, 1) __launch_bounds__(256) window_prepare_few_kernel(const PrepareArgs<T> a) {
-  prepare_token<T, true>(a);
+  prepare_token<T, PREP_PARTS, true>(a);
+}
+template <typename T>
+__global__ void __launch_bounds__(512) window_prepare_mid_kernel(const PrepareArgs<T> a) {
+  prepare_token<T, 1, true>(a);
 }
 template <typename T>
 __global__ void __launch_bounds__(256, 4) window_prepare_kernel(const PrepareArgs<T> a) {
-  prepare_token<T, false>(a);
+  prepare_token<T, 1, false>(a);
 }
 
 // =====================================================================================
@@ -1163,8 +1167,9 @@ int launch_prepare(const void* slabs, long long slab_stride, int P, const void* 
   const size_t smem = (size_t)(rot + 4) * sizeof(float);
   if (smem > 48 * 1024) return -5;
   // with a norm the cluster's exchange costs more than it spreads from a few dozen tokens on
-  if (tokens <= (q_w != nullptr ? 16 : 256))
+  if (tokens <= (q_w != nullptr ? 48 : 256))
     return (int)prism_launch(window_prepare_few_kernel<T>, dim3(tokens * PREP_PARTS), dim3(M >= 4096 ? 256 : 128), smem, stream, pdl, a);
+  if (tokens <= 256) return (int)prism_launch(window_prepare_mid_kernel<T>, dim3(tokens), dim3(M >= 4096 ? 512 : 256), smem, stream, pdl, a);
   return (int)prism_launch(window_prepare_kernel<T>, dim3(tokens), dim3(256), smem, stream, pdl, a);
 }
 

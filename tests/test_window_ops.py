@@ -66,12 +66,13 @@ def pad_heads(t, heads, real, padded):
 
 @pytest.mark.parametrize("backend", BACKENDS)
 @pytest.mark.parametrize("source", ["slabs", "rows"])
+@pytest.mark.parametrize("T", [5, 60, 300])
 @pytest.mark.parametrize("name,bias,norm,rot", [("pair-of-maps", True, False, 24), ("plain", False, True, 16), ("ragged", True, True, 12),
                                                 ("own-keys", False, False, 0), ("widest", True, True, 128), ("odd-group", False, True, 2)])
-def test_prepare(backend, source, name, bias, norm, rot):
+def test_prepare(backend, source, name, bias, norm, rot, T):
     device, dtype = backend
     sp = dataclasses.replace(SPECS[name], rot_dims=rot)
-    T, page, H, G, M, d, e = 5, 16, sp.heads, sp.kv_heads, sp.maps, sp.dim, sp.vdim
+    page, H, G, M, d, e = 16, sp.heads, sp.kv_heads, sp.maps, sp.dim, sp.vdim
     freq = torch.tensor(oracle.frequencies({"base": 300.0, "dims": rot}).tolist())
     parts = [(H * M, d, sp.dq), (G * M, d, sp.dq), (G, e, sp.dv)]
 
@@ -81,7 +82,7 @@ def test_prepare(backend, source, name, bias, norm, rot):
         flat = torch.cat([pad_heads(x, n, r, p) for x, (n, r, p) in zip(real, parts)] + ([real[3]] if sp.gate else []), 1)
         return real, torch.nn.functional.pad(flat, (0, sp.proj_cols - flat.shape[1]))
 
-    (q, k, v, g), flat = stack(1)
+    (q, k, v, zg), flat = stack(1)
     (bq, bk, bv, bg), flat_b = stack(20, 1)
     qn, kn = 0.5 + rand(H * M * d, seed=40).abs(), 0.5 + rand(G * M * d, seed=41).abs()
     w = window.WindowWeights(
@@ -93,9 +94,11 @@ def test_prepare(backend, source, name, bias, norm, rot):
         proj = Branch(slabs=torch.stack([a, b, flat - a - b]).to(device))
     else:
         proj = Branch(rows=flat.to(device, dtype))
-    positions = torch.tensor([0, 3, 17, 400, 2], dtype=torch.int32)
-    slots = torch.tensor([5, 16, -1, 40, 63])
-    cache = ops.KVCache(2, 4, 1, page, sp.k_cols + sp.v_cols, ops.KV_BF16, device, dtype=dtype, planes=1)
+    g = torch.Generator().manual_seed(T)
+    positions = torch.cat([torch.tensor([0, 3, 17, 400, 2]), torch.randint(0, 500, (T - 5,), generator=g)]).int()
+    slots = torch.randperm(16 * page * 2, generator=g)[:T]
+    slots[2] = -1
+    cache = ops.KVCache(2, 32, 1, page, sp.k_cols + sp.v_cols, ops.KV_BF16, device, dtype=dtype, planes=1)
     cache.payload.fill_(7.0)
     q_got, gate = window.qkv_prepare(proj, sp, w, positions.to(device), slots.to(device), cache, 1)
 
@@ -113,12 +116,12 @@ def test_prepare(backend, source, name, bias, norm, rot):
     flat_cache = cache.token_rows(1).reshape(-1, row.shape[1])
     keep = slots >= 0
     close(flat_cache[slots[keep].to(device)], row[keep], dtype, tol32=1e-4)
-    untouched = torch.ones(64, dtype=torch.bool)
+    untouched = torch.ones(32 * page, dtype=torch.bool)
     untouched[slots[keep]] = False
     assert bool((flat_cache.cpu()[untouched] == 7.0).all()) and bool((cache.token_rows(0) == 7.0).all())
     assert (gate is not None) == sp.gate
     if sp.gate:
-        close(gate, oracle.sigmoid(g.double() + (bg.double() if bias else 0.0)), torch.float32)
+        close(gate, oracle.sigmoid(zg.double() + (bg.double() if bias else 0.0)), torch.float32)
 
 
 # ----------------------------------------------------------------------------------------------- attention
