@@ -389,7 +389,12 @@ def resolve_arch(model: str):
         return random_architecture(model.split(":", 1)[1])
     with open(os.path.join(model, "config.json"), "r", encoding="utf-8") as fh:
         cfg = json.load(fh)
-    return family_of_config(cfg).architecture_from_config(cfg)
+    arch = family_of_config(cfg).architecture_from_config(cfg)
+    if hasattr(arch, "with_tensor_shapes"):  # sizes that only the tensors tell
+        from .models.weights import checkpoint_shapes
+
+        arch = arch.with_tensor_shapes(checkpoint_shapes(model))
+    return arch
 
 
 class Config:
@@ -418,6 +423,7 @@ class Config:
         self.eos = self.arch.eos_token_id
         self.num_kvcache_blocks = self.prism.cache.num_gpu_blocks
         self.num_cpu_blocks = 0
+        self.num_cpu_state_slots = 0
 
     # flat read access used across the engine ------------------------------------
     _flat_domain: dict[str, str] = {}  # field name -> domain, resolved once (the step loop reads flat names)
@@ -438,6 +444,14 @@ class Config:
     @property
     def tp(self) -> int:
         return self.prism.model.tensor_parallel_size
+
+    @property
+    def state_slots(self) -> int:
+        """Slots of recurrent state on the device: one per running sequence (0: the family has none)."""
+        return self.prism.scheduler.max_num_seqs if self.arch.state_sizes() else 0
+
+    def state_bytes_per_slot(self) -> int:
+        return 8 * sum(self.arch.state_sizes())   # two versions, 32-bit
 
     @property
     def kvcache_block_size(self) -> int:

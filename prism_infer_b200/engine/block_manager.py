@@ -9,6 +9,7 @@
   transfer) and only computes its own question.  Entries may occupy any free page of the
   pool and are evicted on demand, lowest ``benefit_tokens * (1 + hits) / resident_pages``
   first.
+* Slots of recurrent state, for families that have one: allocated with the pages, given back with them, swapped with them.
 * Copy-on-write, append, swap-out / swap-in (hashes, scales and layouts survive) and the
   plan / commit halves of physical compaction.
 
@@ -23,7 +24,7 @@ import struct
 from dataclasses import dataclass
 from typing import Sequence as Seq
 
-from .block_pool import CpuBlockPool, GpuBlockPool, OutOfBlocks
+from .block_pool import CpuBlockPool, GpuBlockPool, OutOfBlocks, StateSlotPool
 from .contracts import KVTransferPlan
 from .kv_layout import CompactionPlan, KVLayout
 from .sequence import Sequence
@@ -86,10 +87,15 @@ class PrefixCacheCounters:
 
 
 class BlockManager:
-    def __init__(self, num_gpu_blocks: int, page: int, num_cpu_blocks: int = 0, *, enable_prefix_caching: bool = True) -> None:
+    def __init__(self, num_gpu_blocks: int, page: int, num_cpu_blocks: int = 0, *, enable_prefix_caching: bool = True,
+                 num_state_slots: int = 0, num_cpu_state_slots: int = 0) -> None:
+        if num_state_slots and enable_prefix_caching:
+            raise ValueError("pages of equal prefixes cannot be shared where sequences carry recurrent state")
         self.page = page
         self.gpu = GpuBlockPool(num_gpu_blocks)
         self.cpu = CpuBlockPool(num_cpu_blocks)
+        self.state = StateSlotPool(num_state_slots) if num_state_slots else None
+        self.cpu_state = StateSlotPool(num_cpu_state_slots)
         self.enable_prefix_caching = enable_prefix_caching
         self.entries: dict[str, PrefixEntry] = {}
         self.counters = PrefixCacheCounters()
@@ -175,14 +181,25 @@ class BlockManager:
 
     # --------------------------------------------------------------------- allocate
     def can_allocate(self, seq: Sequence) -> bool:
+        if self.state is not None and self.state.num_free == 0:
+            return False
         entry = self.probe_multimodal_prefix(seq) if seq.is_multimodal else None
         need = self._pages_for_hit(seq, entry) if entry is not None else seq.blocks_needed(len(seq))
         return self.num_free_with_eviction() >= need
 
     def allocate(self, seq: Sequence, *, expected_hit: bool | None = None) -> KVTransferPlan:
-        """Give ``seq`` pages for its whole prompt; returns the copies that must run first."""
+        """Give ``seq`` pages for its whole prompt and a state slot; returns the copies that must run first."""
         if seq.block_table:
             raise RuntimeError(f"sequence {seq.seq_id} already owns pages")
+        if self.state is not None:
+            slot = self.state.allocate()
+            try:
+                self._allocate_dense(seq, share=False)
+            except OutOfBlocks:
+                self.state.release(slot)
+                raise
+            seq.state_slot = slot
+            return KVTransferPlan()
         if seq.is_multimodal:
             entry = self.probe_multimodal_prefix(seq)
             if entry is None and expected_hit:
@@ -303,6 +320,11 @@ class BlockManager:
         for p in seq.cpu_block_table:
             self.cpu.release(p)
         seq.cpu_block_table = []
+        if seq.state_slot >= 0:
+            self.state.release(seq.state_slot)
+        if seq.cpu_state_slot >= 0:
+            self.cpu_state.release(seq.cpu_state_slot)
+        seq.state_slot = seq.cpu_state_slot = -1
         seq.num_computed_tokens = 0
         seq.kv_layout = None
 
@@ -359,7 +381,7 @@ class BlockManager:
 
     # ------------------------------------------------------------------------- swap
     def can_swap_out(self, seq: Sequence) -> bool:
-        return self.cpu.num_free >= len(seq.block_table)
+        return self.cpu.num_free >= len(seq.block_table) and (seq.state_slot < 0 or self.cpu_state.num_free > 0)
 
     def swap_out(self, seq: Sequence) -> tuple[tuple[int, int], ...]:
         cpu_pages = self.cpu.allocate_many(len(seq.block_table))
@@ -377,7 +399,7 @@ class BlockManager:
         return tuple(pairs)
 
     def can_swap_in(self, seq: Sequence) -> bool:
-        return self.num_free_with_eviction() >= len(seq.cpu_block_table)
+        return self.num_free_with_eviction() >= len(seq.cpu_block_table) and (seq.cpu_state_slot < 0 or self.state.num_free > 0)
 
     def swap_in(self, seq: Sequence) -> tuple[tuple[int, int], ...]:
         n = len(seq.cpu_block_table)
@@ -396,6 +418,23 @@ class BlockManager:
         seq.cpu_block_table = []
         seq.block_table_version += 1
         return tuple(pairs)
+
+    def swap_out_state(self, seq: Sequence) -> tuple[tuple[int, int], ...]:
+        """The state's part of ``swap_out``: its (device slot, CPU slot), if the sequence has state."""
+        if seq.state_slot < 0:
+            return ()
+        pair = (seq.state_slot, self.cpu_state.allocate())
+        self.state.release(seq.state_slot)
+        seq.state_slot, seq.cpu_state_slot = -1, pair[1]
+        return (pair,)
+
+    def swap_in_state(self, seq: Sequence) -> tuple[tuple[int, int], ...]:
+        if seq.cpu_state_slot < 0:
+            return ()
+        pair = (seq.cpu_state_slot, self.state.allocate())
+        self.cpu_state.release(seq.cpu_state_slot)
+        seq.state_slot, seq.cpu_state_slot = pair[1], -1
+        return (pair,)
 
     # ------------------------------------------------------------------- compaction
     def build_compaction_plan(self, seq: Sequence, retained_positions: Seq[int], prefix_len: int) -> CompactionPlan | None:

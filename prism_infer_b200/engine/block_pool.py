@@ -1,6 +1,6 @@
 """Page allocators: a reference-counted GPU pool with a content-hash index, and a CPU
 swap-page pool with all-or-nothing allocation (reference
-``prism_infer/engine/block_pool.py:17-267``)."""
+``prism_infer/engine/block_pool.py:17-267``); slots of recurrent state."""
 
 from __future__ import annotations
 
@@ -92,6 +92,29 @@ class GpuBlockPool:
         if blk.hash is not None and self.hash_to_block.get(blk.hash) == bid:
             del self.hash_to_block[blk.hash]
         blk.hash, blk.token_ids = None, ()
+
+
+class StateSlotPool:
+    """Slots of recurrent state, one per sequence.  A slot's contents mean nothing to its next owner: a sequence's
+    first token starts from zero whatever the slot holds."""
+
+    def __init__(self, num_slots: int) -> None:
+        self.num_slots = num_slots
+        self.free: deque[int] = deque(range(num_slots))
+
+    @property
+    def num_free(self) -> int:
+        return len(self.free)
+
+    def allocate(self) -> int:
+        if not self.free:
+            raise OutOfBlocks("no free state slot")
+        return self.free.popleft()
+
+    def release(self, slot: int) -> None:
+        if slot in self.free or not 0 <= slot < self.num_slots:
+            raise RuntimeError(f"state slot {slot} is not in use")
+        self.free.append(slot)
 
 
 class CpuBlockPool:

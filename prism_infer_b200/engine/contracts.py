@@ -30,16 +30,20 @@ class PrefillSlice:
 
 @dataclass(frozen=True)
 class KVTransferPlan:
-    """Page traffic to apply before the model runs, in this order."""
+    """Page and state traffic to apply before the model runs, in this order (the order in which the scheduler plans it:
+    a CPU page read by a swap-in may be handed out again by a later swap-out, a device page freed by a swap-out may be the
+    target of a copy)."""
 
+    swap_in: tuple[tuple[int, int], ...] = ()             # (cpu page, gpu page)
+    swap_out: tuple[tuple[int, int], ...] = ()            # (gpu page, cpu page)
     copy_prefix: tuple[tuple[int, int, int], ...] = ()   # (src page, dst page, rows)
     copy_on_write: tuple[tuple[int, int], ...] = ()       # (src page, dst page)
-    swap_out: tuple[tuple[int, int], ...] = ()            # (gpu page, cpu page)
-    swap_in: tuple[tuple[int, int], ...] = ()             # (cpu page, gpu page)
+    state_in: tuple[tuple[int, int], ...] = ()            # (cpu slot, gpu slot), with swap_in
+    state_out: tuple[tuple[int, int], ...] = ()           # (gpu slot, cpu slot), with swap_out
 
     @property
     def empty(self) -> bool:
-        return not (self.copy_prefix or self.copy_on_write or self.swap_out or self.swap_in)
+        return not (self.copy_prefix or self.copy_on_write or self.swap_out or self.swap_in or self.state_out or self.state_in)
 
 
 @dataclass(frozen=True)

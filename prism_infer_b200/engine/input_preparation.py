@@ -70,6 +70,7 @@ class StepInputs(_TensorStatePickle):
     slots: torch.Tensor                    # [T] int64
     block_tables: torch.Tensor             # [S, max_blocks] int32
     temperatures: torch.Tensor             # [S] fp32 (0 = greedy)
+    state_slots: Optional[torch.Tensor] = None    # [S] int32 slot of each sequence's recurrent state
     # prefill only
     cu_seqlens_q: Optional[torch.Tensor] = None   # [S+1] int32
     kv_lens: Optional[torch.Tensor] = None        # [S] int32
@@ -94,7 +95,7 @@ class StepInputs(_TensorStatePickle):
     def pack_decode(self, area: memoryview) -> int:
         """Write the step into ``area``; returns the bytes used, or 0 when this step does not fit
         the fixed form (not a decode step, unexpected dtypes, area too small)."""
-        if self.kind != "decode" or self.context_lens is None or self.block_tables.dim() != 2:
+        if self.kind != "decode" or self.context_lens is None or self.block_tables.dim() != 2 or self.state_slots is not None:
             return 0
         B, W = (int(v) for v in self.block_tables.shape)
         want = ((self.input_ids, torch.int64, B), (self.slots, torch.int64, B), (self.positions, torch.int32, 3 * B),
@@ -149,6 +150,12 @@ class ModelInputPreparer:
             if table:
                 bt[i, : len(table)] = table
         return torch.from_numpy(bt)
+
+    @staticmethod
+    def _state_slots(seqs: tuple[Sequence, ...]) -> Optional[torch.Tensor]:
+        if seqs[0].state_slot < 0:
+            return None
+        return torch.tensor([s.state_slot for s in seqs], dtype=torch.int32)
 
     def prepare(self, plan: BatchPlan, have_visual: set[int] | None = None) -> StepInputs:
         if plan.phase is Phase.PREFILL:
@@ -210,6 +217,7 @@ class ModelInputPreparer:
             slots=cat(slot_parts),
             block_tables=self._block_table(plan.seqs),
             temperatures=temps,
+            state_slots=self._state_slots(plan.seqs),
             cu_seqlens_q=torch.tensor(cu, dtype=torch.int32),
             kv_lens=torch.tensor(kv_lens, dtype=torch.int32),
             max_q_len=max(s.length for s in plan.slices),
@@ -248,5 +256,6 @@ class ModelInputPreparer:
             slots=torch.from_numpy(slots),
             block_tables=self._block_table(seqs),
             temperatures=torch.from_numpy(temps),
+            state_slots=self._state_slots(seqs),
             context_lens=torch.from_numpy(ctx),
         )

@@ -31,6 +31,7 @@ from ..models.common import AttnMeta, TPComm
 from ..models.model_registry import load_model_class
 from ..models.weights import open_weight_source
 from ..observability import profile_region
+from ..ops.recurrent import StateCache
 from .contracts import KVTransferPlan
 from .input_preparation import StepInputs
 from .kv_layout import CompactionPlan
@@ -64,14 +65,16 @@ class _DecodeGraph:
         self.off_ctx = al(self.off_pos + 3 * bucket * 4)
         self.off_temp = al(self.off_ctx + bucket * 4)
         self.off_bt = al(self.off_temp + bucket * 4)
-        self.nbytes = al(self.off_bt + bucket * mb * 4)
+        self.off_state = al(self.off_bt + bucket * mb * 4)
+        self.has_state = runner.state is not None
+        self.nbytes = al(self.off_state + bucket * 4) if self.has_state else self.off_state
         pin = runner.on_cuda
         # Two pinned staging buffers and two token read-back buffers, used alternately: the host may stage step n + 1
         # while the copies of step n are still pending (one step runs ahead at most).  The copies run outside the
         # captured graph, which therefore reads and writes fixed device buffers only.
         self.hosts = [torch.zeros(self.nbytes, dtype=torch.uint8, pin_memory=pin) for _ in range(2)]
         self.dev = torch.zeros(self.nbytes, dtype=torch.uint8, device=dev)
-        self.d_ids, self.d_slots, self.d_pos, self.d_ctx, self.d_temp, self.d_bt = self._views(self.dev, bucket, mb)
+        self.d_ids, self.d_slots, self.d_pos, self.d_ctx, self.d_temp, self.d_bt, self.d_state = self._views(self.dev, bucket, mb)
         self.tokens = torch.zeros(bucket, dtype=torch.int64, device=dev)
         self.tokens_hosts = [torch.zeros(bucket, dtype=torch.int64, pin_memory=pin) for _ in range(2)]
         self.done = [torch.cuda.Event() for _ in range(2)] if pin else [None, None]
@@ -99,10 +102,11 @@ class _DecodeGraph:
         ctx = buf[self.off_ctx:self.off_ctx + b * 4].view(torch.int32)
         temp = buf[self.off_temp:self.off_temp + b * 4].view(torch.float32)
         bt = buf[self.off_bt:self.off_bt + b * mb * 4].view(torch.int32).view(b, mb)
-        return ids, slots, pos, ctx, temp, bt
+        state = buf[self.off_state:self.off_state + (b * 4 if self.has_state else 0)].view(torch.int32)
+        return ids, slots, pos, ctx, temp, bt, state
 
     def reset_rows(self, k: int, start: int) -> None:
-        """Padding rows of staging buffer ``k``: token 0, no slot, empty context, no pages."""
+        """Padding rows of staging buffer ``k``: token 0, no slot, empty context, no pages, no state."""
         n = self._nps[k]
         n[0][start:] = 0
         n[1][start:] = -1
@@ -110,6 +114,7 @@ class _DecodeGraph:
         n[3][start:] = 0
         n[4][start:] = 0
         n[5][start:] = -1
+        n[6][start:] = -1
 
     def fill(self, inp: StepInputs, *, ahead: int = 0) -> int:
         """Stage one step's inputs in the next pinned buffer.  Writes go through numpy views of the
@@ -120,7 +125,7 @@ class _DecodeGraph:
         self.flip ^= 1
         k = self.flip
         n = inp.num_seqs
-        ids, slots, pos, ctx, temp, bt = self._nps[k]
+        ids, slots, pos, ctx, temp, bt, state = self._nps[k]
         ids[:n] = inp.input_ids.numpy()
         slots[:n] = inp.slots.numpy() + ahead
         pos[:, :n] = inp.positions.numpy() + ahead
@@ -129,6 +134,8 @@ class _DecodeGraph:
         w = inp.block_tables.shape[1]
         bt[:n, :w] = inp.block_tables.numpy()
         bt[:n, w:] = -1
+        if self.has_state:
+            state[:n] = inp.state_slots.numpy()
         if n < self._rows[k]:
             self.reset_rows(k, n)
         self._rows[k] = n
@@ -176,6 +183,7 @@ class ModelRunner:
         self.page = config.kvcache_block_size
         self.max_blocks = -(-config.max_model_len // self.page)
         self.kv_mode = config.kv_mode
+        self._allocate_state()
         self._allocate_kv()
         self._visual: dict[int, tuple[torch.Tensor, list[torch.Tensor]]] = {}
         self._visual_cache: dict[str, tuple[torch.Tensor, list[torch.Tensor]]] = {}
@@ -194,7 +202,20 @@ class ModelRunner:
         if self.on_cuda and config.prism.execution.uses_graphs:
             self.capture_graphs()
 
-    # ------------------------------------------------------------------ KV arena
+    # ----------------------------------------------------------- recurrent state, KV arena
+    def _allocate_state(self) -> None:
+        """Slots of recurrent state, in front of the KV arena, which takes what memory is left."""
+        cfg = self.config
+        sizes = cfg.arch.state_sizes()
+        self.state = self.cpu_state = None
+        if not sizes:
+            return
+        self.state = StateCache(sizes, cfg.state_slots, self.device)
+        if cfg.cpu_kv_cache_ratio > 0:
+            cap = (4 << 30) // cfg.state_bytes_per_slot() if self.on_cuda else 64
+            cfg.num_cpu_state_slots = max(1, min(cfg.state_slots, cap))
+            self.cpu_state = StateCache(sizes, cfg.num_cpu_state_slots, "cpu", pin_memory=self.on_cuda)
+
     def _allocate_kv(self) -> None:
         cfg = self.config
         per_page = cfg.kv_bytes_per_page()
@@ -243,7 +264,7 @@ class ModelRunner:
         meta = AttnMeta(is_prefill=True, block_tables=bt, slots=slots,
                         cu_seqlens_q=torch.tensor([0, tokens], dtype=torch.int32, device=dev),
                         kv_lens=torch.tensor([tokens], dtype=torch.int32, device=dev), max_q_len=tokens, no_history=True,
-                        total_kv=tokens, max_kv_len=tokens, attended_pairs=tokens * tokens)
+                        total_kv=tokens, max_kv_len=tokens, attended_pairs=tokens * tokens, **self._state_meta([0]))
         hidden = self.model.forward(ids, pos, meta, scratch)
         self.model.sample(hidden[-1:], None)
         torch.cuda.synchronize(dev)
@@ -257,9 +278,29 @@ class ModelRunner:
                           "budget_bytes": int(budget)}
         return max(1, budget // per_page)
 
+    def _state_meta(self, slots) -> dict[str, object]:
+        """The recurrent state's part of a step's metadata."""
+        if self.state is None:
+            return {}
+        if not isinstance(slots, torch.Tensor):
+            slots = torch.tensor(slots, dtype=torch.int32)
+        return {"state": self.state, "state_slots": slots if slots.device == self.device else self._to_dev(slots)}
+
     # --------------------------------------------------------------- page traffic
     def apply_kv_transfers(self, tr: KVTransferPlan) -> None:
-        """Order matters: prefix-row copies, copy-on-write, swap-out, swap-in."""
+        """Order matters: swap-in, swap-out (pages and recurrent state), prefix-row copies, copy-on-write."""
+        if tr.swap_in:
+            with profile_region("engine.kv.swap_in"):
+                ops.kv_page_copy(self.cpu_kv, self.kv, [c for c, _ in tr.swap_in], [g for _, g in tr.swap_in])
+        for c, g in tr.state_in:
+            self.state.copy_slot(self.cpu_state, c, g)
+        for g, c in tr.state_out:
+            self.cpu_state.copy_slot(self.state, g, c)
+        if tr.swap_out:
+            with profile_region("engine.kv.swap_out"):
+                ops.kv_page_copy(self.kv, self.cpu_kv, [g for g, _ in tr.swap_out], [c for _, c in tr.swap_out])
+                if self.on_cuda:
+                    torch.cuda.current_stream().synchronize()
         if tr.copy_prefix:
             with profile_region("engine.kv.copy_prefix"):
                 ops.kv_page_copy(self.kv, self.kv, [s for s, _, _ in tr.copy_prefix], [d for _, d, _ in tr.copy_prefix],
@@ -267,14 +308,6 @@ class ModelRunner:
         if tr.copy_on_write:
             with profile_region("engine.kv.copy_on_write"):
                 ops.kv_page_copy(self.kv, self.kv, [s for s, _ in tr.copy_on_write], [d for _, d in tr.copy_on_write])
-        if tr.swap_out:
-            with profile_region("engine.kv.swap_out"):
-                ops.kv_page_copy(self.kv, self.cpu_kv, [g for g, _ in tr.swap_out], [c for _, c in tr.swap_out])
-                if self.on_cuda:
-                    torch.cuda.current_stream().synchronize()
-        if tr.swap_in:
-            with profile_region("engine.kv.swap_in"):
-                ops.kv_page_copy(self.cpu_kv, self.kv, [c for c, _ in tr.swap_in], [g for _, g in tr.swap_in])
 
     def compact_kv(self, plans: Seq[CompactionPlan]) -> None:
         with profile_region("engine.kv.visual_compact"):
@@ -521,7 +554,8 @@ class ModelRunner:
                 cu_seqlens_q=self._to_dev(inp.cu_seqlens_q), kv_lens=self._to_dev(inp.kv_lens), max_q_len=inp.max_q_len,
                 no_history=bool(torch.equal(inp.kv_lens, inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1])),
                 total_kv=int(inp.kv_lens.sum()), max_kv_len=int(inp.kv_lens.max()),
-                attended_pairs=int(((inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1]).long() * inp.kv_lens.long()).sum()))
+                attended_pairs=int(((inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1]).long() * inp.kv_lens.long()).sum()),
+                **self._state_meta(inp.state_slots))
             if not meta.no_history:  # key ranges for the gather + tensor-core attention over the paged cache
                 cu_kv = torch.zeros(inp.kv_lens.shape[0] + 1, dtype=torch.int32)
                 cu_kv[1:] = torch.cumsum(inp.kv_lens, 0)
@@ -614,7 +648,7 @@ class ModelRunner:
 
     def _decode_hidden_eager(self, inp: StepInputs) -> torch.Tensor:
         meta = AttnMeta(is_prefill=False, block_tables=self._to_dev(inp.block_tables), slots=self._to_dev(inp.slots),
-                        context_lens=self._to_dev(inp.context_lens))
+                        context_lens=self._to_dev(inp.context_lens), **self._state_meta(inp.state_slots))
         return self.model.forward(self._to_dev(inp.input_ids), self._to_dev(inp.positions), meta, self.kv)
 
     def _run_decode_eager(self, inp: StepInputs) -> list[int]:
@@ -626,7 +660,7 @@ class ModelRunner:
     # ---------------------------------------------------------------- CUDA graphs
     def _decode_body(self, g: _DecodeGraph) -> None:
         meta = AttnMeta(is_prefill=False, block_tables=g.d_bt, slots=g.d_slots, context_lens=g.d_ctx,
-                        nsplit=ops.decode_splits(g.bucket, self.kv.num_kv_heads))
+                        nsplit=ops.decode_splits(g.bucket, self.kv.num_kv_heads), **self._state_meta(g.d_state))
         hidden = self.model.forward(g.d_ids, g.d_pos, meta, self.kv)
         self.model.sample(hidden, None if g.greedy_only else g.d_temp, seed=self.sample_seed, step=g.step, out=g.tokens)
         if self.config.step_logits:  # held, the buffer stays the graph's own; otherwise the graphs of a pool share it
@@ -673,7 +707,8 @@ class ModelRunner:
         samples, copied on the device.  The next call takes the launch over if its inputs are the predicted ones
         (the ids must be the tokens this step returned); otherwise the launch is left to finish unobserved: it wrote
         one K / V row per sequence at a position past that sequence's end, which nothing reads before it is written
-        again, and every later kernel is ordered after it on the stream."""
+        again, and the version of its recurrent state that belongs to one token more (the other version, which the
+        repeated step reads, stays as it was); every later kernel is ordered after it on the stream."""
         n = inp.num_seqs
         bucket = next(b for b in self.buckets if b >= n)
         greedy = bucket in self.greedy_graphs and not bool((inp.temperatures > 0).any())

@@ -36,9 +36,12 @@ class Scheduler:
         self.max_vision_patches = config.max_vision_patches_per_batch
         self.max_model_len = config.max_model_len
         self.eos = config.eos
+        slots = getattr(config, "state_slots", 0)
+        # pages of equal prefixes are shared only where attention is all there is: a recurrent state is not kept at page borders
         self.block_manager = block_manager or BlockManager(
             config.num_kvcache_blocks, config.kvcache_block_size, config.num_cpu_blocks,
-            enable_prefix_caching=config.enable_prefix_caching)
+            enable_prefix_caching=config.enable_prefix_caching and not slots, num_state_slots=slots,
+            num_cpu_state_slots=config.num_cpu_state_slots if slots else 0)
         self.policy = policy or make_policy(config)
         self.metrics = metrics
         self.clock_ns = clock_ns
@@ -210,10 +213,13 @@ class Scheduler:
         bm = self.block_manager
         swap_in: list[tuple[int, int]] = []
         swap_out: list[tuple[int, int]] = []
+        state_in: list[tuple[int, int]] = []
+        state_out: list[tuple[int, int]] = []
         cow: list[tuple[int, int]] = []
         while self.swapped and len(self.running) < self.max_num_seqs and bm.can_swap_in(self.swapped[0]):
             seq = self.swapped.popleft()
             swap_in.extend(bm.swap_in(seq))
+            state_in.extend(bm.swap_in_state(seq))
             seq.lifecycle.transition(RequestState.DECODING, "swap_in")
             self.running.append(seq)
             self.counters["swap_in"] += 1
@@ -224,7 +230,9 @@ class Scheduler:
                 continue
             while not bm.can_append(seq):
                 victim = self.policy.pick_victim([s for s in self.running if s.state is RequestState.DECODING])
-                swap_out.extend(self.preempt(victim))
+                pages, states = self.preempt(victim)
+                swap_out.extend(pages)
+                state_out.extend(states)
                 preempted = True
                 if victim is seq:
                     break
@@ -238,29 +246,32 @@ class Scheduler:
             batch = [s for s in batch if s in self.running and s.state is RequestState.DECODING]
         if not batch:
             if swap_out:
-                return BatchPlan(Phase.IDLE, kv_transfers=KVTransferPlan(swap_out=tuple(swap_out)))
+                return BatchPlan(Phase.IDLE, kv_transfers=KVTransferPlan(swap_in=tuple(swap_in), swap_out=tuple(swap_out),
+                                                                         state_in=tuple(state_in), state_out=tuple(state_out)))
             return None
-        return BatchPlan(Phase.DECODE, tuple(batch), (), KVTransferPlan(copy_on_write=tuple(cow), swap_out=tuple(swap_out),
-                                                                          swap_in=tuple(swap_in)), len(batch), 0)
+        return BatchPlan(Phase.DECODE, tuple(batch), (), KVTransferPlan(
+            copy_on_write=tuple(cow), swap_out=tuple(swap_out), swap_in=tuple(swap_in), state_out=tuple(state_out),
+            state_in=tuple(state_in)), len(batch), 0)
 
     # ---------------------------------------------------------------------- preempt
-    def preempt(self, seq: Sequence) -> tuple[tuple[int, int], ...]:
-        """Free ``seq``'s GPU pages: swap to CPU pages if possible, else recompute later."""
+    def preempt(self, seq: Sequence) -> tuple[tuple[tuple[int, int], ...], tuple[tuple[int, int], ...]]:
+        """Free ``seq``'s GPU pages and state slot: swap to CPU pages if possible, else recompute later.  Returns the pairs
+        of pages and of state slots to copy out."""
         self.running.remove(seq)
         bm = self.block_manager
         if seq.state is RequestState.DECODING and bm.can_swap_out(seq) and bm.cpu.num_blocks > 0:
-            pairs = bm.swap_out(seq)
+            pairs, states = bm.swap_out(seq), bm.swap_out_state(seq)
             seq.lifecycle.transition(RequestState.SWAPPED, "preempt_swap")
             self.swapped.append(seq)
             self.counters["preempt_swap"] += 1
             self.counters["peak_swapped"] = max(self.counters["peak_swapped"], len(self.swapped))
-            return pairs
+            return pairs, states
         bm.deallocate(seq)
         seq.num_cached_tokens = 0
         seq.lifecycle.transition(RequestState.WAITING, "preempt_recompute")
         self.waiting.appendleft(seq)
         self.counters["preempt_recompute"] += 1
-        return ()
+        return (), ()
 
     # ------------------------------------------------------------------ postprocess
     def postprocess(self, plan: BatchPlan, tokens: Iterable[int | None]) -> list[RequestOutput]:

@@ -47,6 +47,8 @@ class Sequence:
         self.lifecycle = RequestLifecycle(seq_id)
         self.block_table: list[int] = []
         self.cpu_block_table: list[int] = []
+        self.state_slot = -1              # slot of its recurrent state on the device / swapped out
+        self.cpu_state_slot = -1
         self.block_table_version = 0
         self.num_computed_tokens = 0      # logical tokens whose KV exists
         self.num_cached_tokens = 0        # logical tokens served from a cache at admission

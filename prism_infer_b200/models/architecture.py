@@ -6,12 +6,12 @@ dataclasses below once and every later layer (weight sharding, kernels, KV sizin
 reads these.  Mirrors the contract of the reference's
 ``prism_infer/models/qwen3_vl_architecture.py:117-428`` (canonical 8B constants at
 ``:18-44``): interleaved M-RoPE only, no attention bias, SiLU text MLP, GELU-tanh
-vision MLP.  ``PoralornArch`` and ``DolidraArch`` (end of file) are text-only looped families: latent attention, and
-windowed attention with a mixture of experts.
+vision MLP.  ``PoralornArch``, ``DolidraArch`` and ``BokoraxArch`` (end of file) are text-only families: latent attention,
+windowed attention with a mixture of experts, and recurrent layers between attention layers.
 
 What the engine asks of any architecture, whatever its family: ``model_type``, ``multimodal``,
 ``vocab_size``, ``max_positions`` (``None``: unbounded), ``num_layer_runs``, ``eos_token_id``, the
-visual token ids (-1 where there are none), ``reserved_token_ids`` and ``kv_geometry(tp)``.
+visual token ids (-1 where there are none), ``reserved_token_ids``, ``kv_geometry(tp)`` and ``state_sizes()``.
 """
 
 from __future__ import annotations
@@ -19,7 +19,7 @@ from __future__ import annotations
 import json
 import math
 import os
-from dataclasses import asdict, dataclass, field
+from dataclasses import asdict, dataclass, field, replace
 from typing import Any, Mapping
 
 SUPPORTED_MODEL_TYPES = frozenset({"qwen3_vl"})
@@ -183,6 +183,9 @@ class Qwen3VLArch:
     @property
     def reserved_token_ids(self) -> tuple[int, ...]:
         return (self.image_token_id, self.video_token_id, self.vision_start_token_id, self.vision_end_token_id, self.eos_token_id)
+
+    def state_sizes(self) -> tuple[int, ...]:
+        return ()
 
     def kv_geometry(self, tp: int = 1) -> KVGeometry:
         return KVGeometry(2, self.text.num_layers, self.text.num_kv_heads // tp, self.text.head_dim)
@@ -429,6 +432,10 @@ class LoopedStack:
     def reserved_token_ids(self) -> tuple[int, ...]:
         return ()
 
+    def state_sizes(self) -> tuple[int, ...]:
+        """fp32 elements that a sequence's recurrent state takes in each recurrent layer run (none: attention only)."""
+        return ()
+
     def layer_runs(self) -> tuple[LayerRun, ...]:
         """Every layer execution in order; run ``i`` owns cache slab ``i``."""
         if not self.has_loop:
@@ -602,7 +609,8 @@ class PoralornArch(LoopedStack):
 @dataclass(frozen=True)
 class RotaryArch:
     """Rotation of the first ``dims`` columns of a head (pairs ``(i, i + dims / 2)``).  ``factor`` > 0 rescales the
-    frequencies by wavelength: long ones are divided by it, those below ``original / high`` stay, a ramp between."""
+    frequencies by wavelength: long ones are divided by it, those below ``original / high`` stay, a ramp between; without
+    ``original`` all of them are divided."""
 
     base: float
     dims: int
@@ -619,7 +627,9 @@ class RotaryArch:
         out = []
         for i in range(self.dims // 2):
             f = self.base ** (-2.0 * i / self.dims)
-            if self.factor > 0.0:
+            if self.factor > 0.0 and self.original == 0.0:
+                f /= self.factor
+            elif self.factor > 0.0:
                 wavelength = 2.0 * math.pi / f
                 if wavelength > self.original / self.low:
                     f /= self.factor
@@ -630,11 +640,17 @@ class RotaryArch:
         return out
 
 
+NO_WINDOW = 1 << 30              # a window that no sequence outgrows
+
+
 @dataclass(frozen=True)
 class WindowAttentionArch:
     """One windowed attention mixer.  ``maps`` 2: differential attention (two maps over the same values, the second
-    subtracted); ``qk_norm``: RMS norm over the whole query and the whole key projection; ``gate``: one sigmoid output
-    gate per head; a query sees the ``window`` newest positions (its own included) and the first ``keep_first``."""
+    subtracted); ``qk_norm``: RMS norm over the whole query and the whole key projection, or (``head_norm``) over every
+    head with one weight for all; ``gate``: one sigmoid output gate per head; a query sees the ``window`` newest positions
+    (its own included) and the first ``keep_first``.  ``tied_values``: the values are the keys as projected; ``softcap``
+    bounds the scores (0: no bound); ``sink``: a learned score per head in the softmax's denominator; ``kv_from``: the layer
+    whose cached keys and values it reads instead of its own (-1: none)."""
 
     heads: int
     kv_heads: int
@@ -649,6 +665,11 @@ class WindowAttentionArch:
     bias: bool = False
     qk_norm: bool = False
     gate: bool = False
+    head_norm: bool = False
+    tied_values: bool = False
+    softcap: float = 0.0
+    sink: bool = False
+    kv_from: int = -1
 
     def __post_init__(self) -> None:
         for name in ("heads", "kv_heads", "dim", "vdim", "window"):
@@ -658,6 +679,10 @@ class WindowAttentionArch:
             raise ValueError(f"windowed attention: {self.heads} query heads over {self.kv_heads} key/value heads")
         if self.rot.dims > self.dim or self.keep_first < 0 or self.maps not in (1, 2):
             raise ValueError("windowed attention: rot.dims must not exceed dim, keep_first must not be negative, maps is 1 or 2")
+        if self.tied_values and (self.vdim != self.dim or self.maps != 1):
+            raise ValueError("windowed attention: values that are the keys have the keys' width, and one map")
+        if self.softcap < 0.0:
+            raise ValueError("windowed attention: softcap must not be negative")
 
     @property
     def dq(self) -> int:
@@ -677,16 +702,34 @@ class WindowAttentionArch:
 @dataclass(frozen=True)
 class MixtureArch:
     """Routed experts: ``top`` of ``experts`` gated feed-forwards of width ``ff`` per token, and one of width
-    ``shared_ff`` (0: none) for every token."""
+    ``shared_ff`` (0: none) for every token, times a sigmoid per token with ``shared_gate``.  The weights are the softmax over
+    the chosen logits, or (``scored``) the chosen scores of a softmax over all, divided by their sum and times ``scale``; then
+    a learned correction enters the choice only, ``identity`` more router outputs stand for the input itself, and the
+    choice is among the ``groups_kept`` best of ``groups`` equal groups of neighbours."""
 
     experts: int
     top: int
     ff: int
     shared_ff: int = 0
+    scored: bool = False
+    identity: int = 0
+    groups: int = 1
+    groups_kept: int = 1
+    scale: float = 1.0
+    shared_gate: bool = False
+
+    @property
+    def outputs(self) -> int:
+        """Router outputs that can be chosen."""
+        return self.experts + self.identity
 
     def __post_init__(self) -> None:
-        if self.experts < 1 or not 1 <= self.top <= self.experts or self.ff < 1 or self.shared_ff < 0:
+        if self.experts < 1 or not 1 <= self.top <= self.outputs or self.ff < 1 or self.shared_ff < 0 or self.identity < 0:
             raise ValueError(f"mixture of experts: {self.top} of {self.experts} experts of width {self.ff}, shared {self.shared_ff}")
+        if not 1 <= self.groups_kept <= self.groups or self.outputs % self.groups or self.top > self.outputs // self.groups * self.groups_kept:
+            raise ValueError(f"mixture of experts: {self.top} of {self.outputs} in {self.groups_kept} of {self.groups} groups")
+        if not self.scored and (self.identity or self.groups > 1 or self.scale != 1.0):
+            raise ValueError("mixture of experts: identity experts, groups and a scale belong to scored routing")
 
 
 @dataclass(frozen=True)
@@ -859,3 +902,252 @@ class DolidraArch(LoopedStack):
         moe = MixtureArch(experts, top, expert_ff, expert_ff)
         kinds = [DolidraLayer(kept if i % 4 == 2 else diff, **({"moe": moe} if i % 2 else {"ff": ff})) for i in range(layers)]
         return cls(vocab_size=vocab_size, width=width, layers=tuple(kinds), side_dim=side_dim)
+
+
+# -------------------------------------------------------------------------------- Bokorax
+@dataclass(frozen=True)
+class TimeMixArch:
+    """A recurrent mixer with a matrix state per head (``dim`` x ``dim``): decay per key channel, data-dependent through a
+    projection of rank ``decay_rank`` (a checkpoint's tensor shapes give it), and a bonus for the current token.  Every
+    projection reads its own blend of the token's row and the previous token's."""
+
+    heads: int
+    dim: int
+    decay_rank: int = 64
+
+    def __post_init__(self) -> None:
+        if self.heads < 1 or self.dim < 1 or self.decay_rank < 1:
+            raise ValueError(f"time mixing: {self.heads} heads of {self.dim}, decay rank {self.decay_rank}")
+
+    @property
+    def dp(self) -> int:
+        """Head width padded to whole tensor-core steps."""
+        return -(-self.dim // 16) * 16
+
+    def state_size(self, width: int) -> int:
+        """fp32 elements of a sequence's state: ``[heads, dp, dp]`` and the previous token's row."""
+        return self.heads * self.dp * self.dp + -(-width // 16) * 16
+
+
+@dataclass(frozen=True)
+class BokoraxLayer:
+    mixer: WindowAttentionArch | TimeMixArch
+    moe: MixtureArch | None = None
+
+    @property
+    def recurrent(self) -> bool:
+        return isinstance(self.mixer, TimeMixArch)
+
+    @property
+    def owns_cache(self) -> bool:
+        return not self.recurrent and self.mixer.kv_from < 0
+
+
+@dataclass(frozen=True)
+class BokoraxArch(LoopedStack):
+    vocab_size: int
+    width: int
+    layers: tuple[BokoraxLayer, ...]
+    embed_scale: float = 1.0
+    logit_scale: float = 1.0
+    norm_eps: float = 1.0e-6
+    eos_token_id: int = -1
+    model_type: str = "bokorax"
+
+    loop_start = loop_stop = loop_times = 0   # every layer runs once
+
+    def __post_init__(self) -> None:
+        self.check_stack()
+        for i, l in enumerate(self.layers):
+            if l.recurrent or l.owns_cache:
+                continue
+            m, j = l.mixer, l.mixer.kv_from
+            owner = self.layers[j] if j < i else None
+            if owner is None or not owner.owns_cache:
+                raise ValueError(f"Bokorax layer {i}: kv_from {j} does not name an earlier layer with keys of its own")
+            if (m.kv_heads, m.dim, m.vdim) != (owner.mixer.kv_heads, owner.mixer.dim, owner.mixer.vdim):
+                raise ValueError(f"Bokorax layer {i}: keys and values of layer {j} have other sizes")
+
+    def cache_slab(self, layer: int) -> int:
+        """Cache slab a layer's attention reads (-1: a recurrent layer)."""
+        l = self.layers[layer]
+        if l.recurrent:
+            return -1
+        owner = layer if l.owns_cache else l.mixer.kv_from
+        return sum(o.owns_cache for o in self.layers[:owner])
+
+    def state_slab(self, layer: int) -> int:
+        return sum(l.recurrent for l in self.layers[:layer]) if self.layers[layer].recurrent else -1
+
+    def kv_geometry(self, tp: int = 1) -> KVGeometry:
+        rows = tuple(l.mixer.cache_row for l in self.layers if l.owns_cache) or (16,)   # pages count tokens even without keys
+        return KVGeometry(1, len(rows), 1, max(rows), rows)
+
+    def state_sizes(self) -> tuple[int, ...]:
+        return tuple(l.mixer.state_size(self.width) for l in self.layers if l.recurrent)
+
+    # ---- checkpoint --------------------------------------------------------------
+    def weight_shapes(self) -> dict[str, tuple[int, ...]]:
+        W = self.width
+        s: dict[str, tuple[int, ...]] = {"embed": (self.vocab_size, W)}
+
+        def ff(prefix: str, width: int) -> None:
+            s[f"{prefix}.gate"] = s[f"{prefix}.up"] = (width, W)
+            s[f"{prefix}.down"] = (W, width)
+
+        for i, l in enumerate(self.layers):
+            m, p = l.mixer, f"l{i}"
+            s[f"{p}.norm1"] = (W,)
+            if l.recurrent:
+                C = m.heads * m.dim
+                for n in "rkvgw":
+                    s[f"{p}.mix.mu.{n}"] = (W,)
+                for n in "rkvg":
+                    s[f"{p}.mix.{n}"] = (C, W)
+                s[f"{p}.mix.w1"], s[f"{p}.mix.w2"], s[f"{p}.mix.w0"] = (m.decay_rank, W), (C, m.decay_rank), (C,)
+                s[f"{p}.mix.u"], s[f"{p}.mix.norm"], s[f"{p}.mix.o"] = (m.heads, m.dim), (C,), (W, C)
+            else:
+                sizes = {"q": m.heads * m.dim}
+                if m.kv_from < 0:
+                    sizes["k"] = m.kv_heads * m.dim
+                    if not m.tied_values:
+                        sizes["v"] = m.kv_heads * m.vdim
+                for n, rows in sizes.items():
+                    s[f"{p}.mix.{n}"] = (rows, W)
+                    if m.qk_norm and n != "v":
+                        s[f"{p}.mix.{n}.norm"] = (m.dim if m.head_norm else rows,)
+                if m.sink:
+                    s[f"{p}.mix.sink"] = (m.heads,)
+                if m.gate:
+                    s[f"{p}.mix.g"] = (m.heads, W)
+                s[f"{p}.mix.o"] = (W, m.heads * m.vdim)
+            if l.moe is not None:
+                s[f"{p}.norm2"] = (W,)
+                s[f"{p}.mlp.router"], s[f"{p}.mlp.correction"] = (l.moe.outputs, W), (l.moe.outputs,)
+                for e in range(l.moe.experts):
+                    ff(f"{p}.mlp.e{e}", l.moe.ff)
+                if l.moe.shared_ff:
+                    ff(f"{p}.mlp.shared", l.moe.shared_ff)
+                    s[f"{p}.mlp.shared.sg"] = (1, W)
+        s["final.norm"] = (W,)
+        s["head"] = (self.vocab_size, W)
+        return s
+
+    def with_tensor_shapes(self, shapes: Mapping[str, tuple[int, ...]]) -> "BokoraxArch":
+        """The sizes that only a checkpoint's tensors tell: the rank of every decay projection."""
+        def sized(i: int, l: BokoraxLayer) -> BokoraxLayer:
+            shape = shapes.get(f"l{i}.mix.w1") if l.recurrent else None
+            return replace(l, mixer=replace(l.mixer, decay_rank=int(shape[0]))) if shape else l
+
+        return replace(self, layers=tuple(sized(i, l) for i, l in enumerate(self.layers)))
+
+    @staticmethod
+    def init_kind(name: str) -> str:
+        """How random initialisation draws a tensor: ``norm``, ``bias``, ``embedding`` or ``matrix``."""
+        last = name.rsplit(".", 1)[-1]
+        if last in ("norm1", "norm2", "w0", "u", "sink", "correction") or name == "final.norm" or ".mu." in name:
+            return "bias"            # norm weights around zero among them
+        if last == "norm":
+            return "norm"
+        return "embedding" if name == "embed" else "matrix"
+
+    # ---- factories ---------------------------------------------------------------
+    @classmethod
+    def from_hf_config(cls, cfg: Mapping[str, Any]) -> "BokoraxArch":
+        """From the ``config.json`` dictionary."""
+        need = _field_reader("Bokorax")
+
+        def attention(m: Mapping[str, Any], where: str, **kw) -> WindowAttentionArch:
+            rot, mask = need(m, "rot", where), m.get("mask") or {}
+            scaling = rot.get("scaling") or {}
+            return WindowAttentionArch(
+                heads=int(need(m, "heads", where)), kv_heads=int(need(m, "kv_heads", where)), dim=int(need(m, "dim", where)),
+                vdim=int(need(m, "vdim", where)), scale=float(need(m, "scale", where)),
+                rot=RotaryArch(float(need(rot, "base", where)), int(need(rot, "dims", where)),
+                               float(need(scaling, "factor", where)) if scaling else 0.0),
+                window=int(need(mask, "size", where)) if mask else NO_WINDOW, qk_norm=True,
+                kv_from=-1 if m.get("kv_from") is None else int(m["kv_from"]), softcap=float(m.get("softcap") or 0.0), **kw)
+
+        layers = []
+        for i, entry in enumerate(need(cfg, "layers")):
+            where = f"layer {i}"
+            kind, m = need(entry, "type", where), need(entry, "mixer", where)
+            if kind == "attention":
+                mixer = attention(m, where, tied_values=True)
+            elif kind == "attention_2":
+                mixer = attention(m, where, head_norm=True, gate=True, sink=True)
+            elif kind == "wkv":
+                mixer = TimeMixArch(int(need(m, "heads", where)), int(need(m, "dim", where)))
+            else:
+                raise ValueError(f"Bokorax {where}: unsupported mixer {kind!r}")
+            mlp = entry.get("mlp")
+            if mlp is None:
+                layers.append(BokoraxLayer(mixer))
+                continue
+            if mlp.get("kind") != "moe":
+                raise ValueError(f"Bokorax {where}: unsupported feed-forward {mlp.get('kind')!r}")
+            router, shared = need(mlp, "router", where), mlp.get("shared") or {}
+            groups = router.get("groups") or {"count": 1, "keep": 1}
+            layers.append(BokoraxLayer(mixer, MixtureArch(
+                int(need(router, "experts", where)), int(need(router, "top", where)), int(need(need(mlp, "expert", where), "ff", where)),
+                int(need(shared, "ff", where)) if shared else 0, scored=True, identity=int(router.get("identity") or 0),
+                groups=int(need(groups, "count", where)), groups_kept=int(need(groups, "keep", where)),
+                scale=float(router.get("scale", 1.0)), shared_gate=bool(shared))))
+        return cls(vocab_size=int(need(cfg, "vocab")), width=int(need(cfg, "width")), layers=tuple(layers),
+                   embed_scale=float(need(need(cfg, "embedding"), "scale", "embedding")), logit_scale=float(need(cfg, "logit_scale")),
+                   norm_eps=float(need(need(cfg, "norm"), "eps", "norm")))
+
+    def to_hf_config(self) -> dict[str, Any]:
+        """The ``config.json`` dictionary ``from_hf_config`` reads."""
+
+        def layer(l: BokoraxLayer) -> dict[str, Any]:
+            m = l.mixer
+            mixer: dict[str, Any] = {"heads": m.heads, "dim": m.dim}
+            if not l.recurrent:
+                rot: dict[str, Any] = {"base": m.rot.base, "dims": m.rot.dims}
+                if m.rot.factor > 0.0:
+                    rot["scaling"] = {"factor": m.rot.factor}
+                mixer |= {"kv_heads": m.kv_heads, "vdim": m.vdim, "scale": m.scale, "rot": rot}
+                if m.window != NO_WINDOW:
+                    mixer["mask"] = {"size": m.window}
+                if m.softcap:
+                    mixer["softcap"] = m.softcap
+                if m.kv_from >= 0:
+                    mixer["kv_from"] = m.kv_from
+            mlp: dict[str, Any] | None = None
+            if l.moe is not None:
+                mlp = {"kind": "moe", "expert": {"ff": l.moe.ff},
+                       "router": {"experts": l.moe.experts, "top": l.moe.top, "identity": l.moe.identity, "scale": l.moe.scale,
+                                  "groups": {"count": l.moe.groups, "keep": l.moe.groups_kept}}}
+                if l.moe.shared_ff:
+                    mlp["shared"] = {"ff": l.moe.shared_ff}
+            return {"type": "wkv" if l.recurrent else ("attention" if m.tied_values else "attention_2"), "mixer": mixer, "mlp": mlp}
+
+        return {"architecture": "Bokorax", "vocab": self.vocab_size, "width": self.width, "norm": {"eps": self.norm_eps},
+                "embedding": {"scale": self.embed_scale}, "logit_scale": self.logit_scale, "layers": [layer(l) for l in self.layers]}
+
+    @classmethod
+    def tiny(cls) -> "BokoraxArch":
+        """The small CPU test model: every size different, all three mixers, a layer that reads another's keys."""
+        wkv = TimeMixArch(3, 24, 12)
+        tied = WindowAttentionArch(4, 2, 40, 40, 0.16, RotaryArch(9000.0, 24), window=21, qk_norm=True, tied_values=True)
+        sink = WindowAttentionArch(6, 2, 32, 24, 0.18, RotaryArch(30000.0, 16, 3.0), window=NO_WINDOW, qk_norm=True, gate=True,
+                                   head_norm=True, softcap=20.0, sink=True)
+        moe = MixtureArch(6, 2, 40, 56, scored=True, identity=2, groups=4, groups_kept=2, scale=1.5, shared_gate=True)
+        return cls(vocab_size=300, width=112, layers=(BokoraxLayer(wkv, moe), BokoraxLayer(sink, moe), BokoraxLayer(tied), BokoraxLayer(wkv),
+                                                      BokoraxLayer(replace(sink, kv_from=1), moe)), embed_scale=4.0, logit_scale=1.5)
+
+    @classmethod
+    def like_8b(cls, layers: int = 4, *, width: int = 4096, heads: int = 32, kv_heads: int = 8, dim: int = 128, state_dim: int = 64,
+                window: int = 1024, experts: int = 24, identity: int = 8, top: int = 4, expert_ff: int = 1536,
+                vocab_size: int = 151_936) -> "BokoraxArch":
+        """Layers with the widths of an 8B-class decoder (measurement model; random weights): recurrent, causal, windowed
+        and, with the causal layer's keys, causal again, in turn."""
+        wkv = TimeMixArch(width // state_dim, state_dim)
+        tied = WindowAttentionArch(heads, kv_heads, dim, dim, dim ** -0.5, RotaryArch(1.0e6, dim), window=window, qk_norm=True, tied_values=True)
+        sink = WindowAttentionArch(heads, kv_heads, dim, dim, dim ** -0.5, RotaryArch(1.0e6, dim, 4.0), window=NO_WINDOW, qk_norm=True,
+                                   gate=True, head_norm=True, softcap=30.0, sink=True)
+        moe = MixtureArch(experts, top, expert_ff, expert_ff, scored=True, identity=identity, groups=4, groups_kept=2, scale=2.5,
+                          shared_gate=True)
+        kinds = [(wkv, sink, tied, replace(sink, kv_from=i - 2))[i % 4] for i in range(layers)]
+        return cls(vocab_size=vocab_size, width=width, layers=tuple(BokoraxLayer(m, moe) for m in kinds), embed_scale=8.0)

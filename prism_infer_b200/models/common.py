@@ -36,6 +36,9 @@ class AttnMeta:
     workspace: Optional[tuple[torch.Tensor, torch.Tensor]] = None
     # prefill with the attention pruning strategy: collects last-query attention over visual tokens
     scorer: Optional[object] = None
+    # recurrent layers: the state container and the slot of each sequence (decode: of each row, < 0: padding)
+    state: Optional[object] = None                 # ops.recurrent.StateCache
+    state_slots: Optional[torch.Tensor] = None     # [S] int32
     attended_pairs: int = 0                        # sum over the sequences of query rows x visible keys, known on the host
 
 

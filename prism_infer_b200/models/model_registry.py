@@ -69,6 +69,19 @@ def _dolidra_random() -> dict[str, Callable[[], Any]]:
             "dolidra-8b-like-4layer": DolidraArch.like_8b}
 
 
+def _bokorax_arch(cfg: Any):
+    from .architecture import BokoraxArch
+
+    return BokoraxArch.from_hf_config(cfg)
+
+
+def _bokorax_random() -> dict[str, Callable[[], Any]]:
+    from .architecture import BokoraxArch
+
+    return {"bokorax-tiny": BokoraxArch.tiny, "bokorax-8b-like": lambda: BokoraxArch.like_8b(36),
+            "bokorax-8b-like-4layer": BokoraxArch.like_8b}
+
+
 _FAMILIES = {
     "qwen3_vl": ModelFamily("qwen3_vl", True, _qwen3_vl_arch, "prism_infer_b200.models.qwen3_vl:Qwen3VLModel", _qwen3_vl_random()),
     "poralorn": ModelFamily("poralorn", False, _poralorn_arch, "prism_infer_b200.models.poralorn:PoralornModel", _poralorn_random(),
@@ -78,6 +91,10 @@ _FAMILIES = {
     "dolidra": ModelFamily("dolidra", False, _dolidra_arch, "prism_infer_b200.models.dolidra:DolidraModel", _dolidra_random(),
                            float32_on_cuda=True, kv_modes=(0,),
                            kernel_units=("gemm_tcgen05", "gemm_f32", "window_attention", "moe", "residual_stream", "kv_ops", "sampler")),
+    "bokorax": ModelFamily("bokorax", False, _bokorax_arch, "prism_infer_b200.models.bokorax:BokoraxModel", _bokorax_random(),
+                           float32_on_cuda=True, kv_modes=(0,),
+                           kernel_units=("gemm_tcgen05", "gemm_f32", "window_attention", "recurrence", "moe", "residual_stream", "kv_ops",
+                                         "sampler")),
 }
 
 

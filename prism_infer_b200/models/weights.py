@@ -144,6 +144,18 @@ def iter_safetensors(path: str) -> Iterator[tuple[str, torch.Tensor]]:
                 yield name, fh.get_tensor(name)
 
 
+def checkpoint_shapes(path: str) -> dict[str, tuple[int, ...]]:
+    """Name -> shape of every tensor in ``path/*.safetensors``, from the file headers."""
+    from safetensors import safe_open
+
+    shapes: dict[str, tuple[int, ...]] = {}
+    for file in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with safe_open(file, "pt", "cpu") as fh:
+            for name in fh.keys():
+                shapes[name] = tuple(fh.get_slice(name).get_shape())
+    return shapes
+
+
 def save_checkpoint(
     path: str,
     arch: Any,

@@ -6,7 +6,9 @@
 //
 //   moe_route_kernel   one CTA per chunk of tokens: sum of the router's split-K slabs, top-k (one warp per token), softmax
 //                      over the chosen logits, count per expert and rank of each pair within its chunk and expert.  With a
-//                      single chunk it also places the pairs.
+//                      single chunk it also places the pairs.  Scored form: the softmax is over all outputs, a correction
+//                      enters the choice only, which is among the best groups of neighbours; outputs E .. choices - 1 stand
+//                      for the token's own row (their weights are summed up for the kernel that adds the branch).
 //   moe_place_kernel   one CTA per chunk: first row of every expert, then rows of the chunk's pairs
 //   moe_gather_kernel  copies a token's row to the rows of its pairs
 #include "common.cuh"
@@ -34,6 +36,13 @@ struct RouteArgs {
   int max_groups;
   int* n_groups;
   int T, top, E, always, chunk, tile;
+  // scored form (correction != null)
+  const float* correction;  // [choices]
+  float* self_weight;       // [T] weight of the token's own row
+  int choices;              // outputs that can be chosen, the E experts first; E without the scored form
+  int sets, keep;           // the best `keep` of `sets` equal runs of neighbours are open to choice
+  int always_col;           // logit whose sigmoid weighs the always-on experts (-1: weight one)
+  float scale;
 };
 
 // Exclusive prefix sum over the block of one value per thread; *total gets the sum.
@@ -92,8 +101,58 @@ __device__ __forceinline__ void place(const RouteArgs& a, int t0, int n, int cou
   }
 }
 
-// C: groups of 32 routed experts
+// choice [C]: lane l's values of outputs l, l + 32, ...  Outputs outside the best groups become -inf.
 template <int C>
+__device__ __forceinline__ void keep_best_groups(float (&choice)[C], const RouteArgs& a, int lane) {
+  const int size = a.choices / a.sets;
+  int of[C];                       // group of each of the lane's outputs
+#pragma unroll
+  for (int c = 0; c < C; ++c) of[c] = (c * 32 + lane) / size;
+  float best[C];                   // lane l: scores of groups l, l + 32, ...
+#pragma unroll
+  for (int c = 0; c < C; ++c) best[c] = -INFINITY;
+  for (int g = 0; g < a.sets; ++g) {
+    float m = -INFINITY;
+#pragma unroll
+    for (int c = 0; c < C; ++c)
+      if (of[c] == g) m = fmaxf(m, choice[c]);
+    m = warp_max(m);
+#pragma unroll
+    for (int c = 0; c < C; ++c)
+      if (c * 32 + lane == g) best[c] = m;
+  }
+  unsigned open = 0;
+  for (int k = 0; k < a.keep; ++k) {
+    float bv = -INFINITY;
+    int bg = MAX_EXPERTS;
+#pragma unroll
+    for (int c = 0; c < C; ++c)
+      if (best[c] > bv) {
+        bv = best[c];
+        bg = c * 32 + lane;
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int og = __shfl_xor_sync(0xffffffffu, bg, o);
+      if (ov > bv || (ov == bv && og < bg)) {
+        bv = ov;
+        bg = og;
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+      if (of[c] == bg) open |= 1u << c;
+      if (c * 32 + lane == bg) best[c] = -INFINITY;
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < C; ++c)
+    if (!(open >> c & 1u)) choice[c] = -INFINITY;
+}
+
+// C: groups of 32 outputs
+template <int C, bool SCORED>
 __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArgs a) {
   extern __shared__ int expert_s[];            // [chunk * K]
   __shared__ int count_s[MAX_EXPERTS], base_s[MAX_EXPERTS], scan_s[32];
@@ -110,13 +169,35 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArg
     for (int c = 0; c < C; ++c) {
       const int e = c * 32 + lane;
       float s = 0.0f;
-      if (e < a.E) {
+      if (e < a.choices) {
 #pragma unroll 16
         for (int p = 0; p < a.P; ++p) s += __ldcg(a.logits + (size_t)p * a.slab_stride + t * a.ld + e);
       }
-      v[c] = e < a.E ? s : -INFINITY;
+      v[c] = e < a.choices ? s : -INFINITY;
     }
-    float best0 = 0.0f, sum = 0.0f;
+    float always_w = 1.0f, score[SCORED ? C : 1];
+    if (SCORED) {
+      if (a.always_col >= 0) {
+        float s = 0.0f;
+#pragma unroll 16
+        for (int p = 0; p < a.P; ++p) s += __ldcg(a.logits + (size_t)p * a.slab_stride + t * a.ld + a.always_col);
+        always_w = 1.0f / (1.0f + expf(-s));
+      }
+      float m = v[0], total = 0.0f;
+#pragma unroll
+      for (int c = 1; c < C; ++c) m = fmaxf(m, v[c]);
+      m = warp_max(m);
+#pragma unroll
+      for (int c = 0; c < C; ++c) total += score[c] = expf(v[c] - m);
+      total = 1.0f / warp_sum(total);
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        score[c] *= total;
+        if (c * 32 + lane < a.choices) v[c] = score[c] + a.correction[c * 32 + lane];
+      }
+      if (a.sets > a.keep) keep_best_groups(v, a, lane);
+    }
+    float best0 = 0.0f, sum = 0.0f, self = 0.0f;
     for (int k = 0; k < a.top; ++k) {
       float bv = -INFINITY;
       int be = MAX_EXPERTS;
@@ -135,24 +216,35 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArg
           be = oe;
         }
       }
-      if (be >= a.E) be = 0;                   // no finite logit left: any expert, weight from its own logit
+      if (be >= a.choices) be = 0;             // no finite logit left: any expert, weight from its own logit
 #pragma unroll
       for (int c = 0; c < C; ++c)
         if (be == c * 32 + lane) v[c] = -INFINITY;
-      if (k == 0) best0 = bv;
-      const float w = expf(bv - best0);
+      float w;
+      if (SCORED) {
+        float mine = 0.0f;
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+          if (be == c * 32 + lane) mine = score[c];
+        w = __shfl_sync(0xffffffffu, mine, be & 31);
+        if (be >= a.E) self += w;
+      } else {
+        if (k == 0) best0 = bv;
+        w = expf(bv - best0);
+      }
       sum += w;
       if (lane == 0) {
-        expert_s[i * K + k] = live ? be : -1;
-        a.weight[t * K + k] = w;
+        expert_s[i * K + k] = live && be < a.E ? be : -1;
+        a.weight[t * K + k] = be < a.E ? w : 0.0f;
       }
     }
     __syncwarp();
-    const float inv = 1.0f / sum;
+    const float inv = SCORED ? a.scale / (sum + 1e-20f) : 1.0f / sum;
     for (int k = lane; k < K; k += 32) {
       if (k >= a.top) expert_s[i * K + k] = live ? a.E + k - a.top : -1;
-      a.weight[t * K + k] = live ? (k < a.top ? a.weight[t * K + k] * inv : 1.0f) : 0.0f;
+      a.weight[t * K + k] = live ? (k < a.top ? a.weight[t * K + k] * inv : always_w) : 0.0f;
     }
+    if (SCORED && lane == 0) a.self_weight[t] = live ? self * inv : 0.0f;
   }
   __syncthreads();
   // count and rank: one warp per expert looks at 32 pairs at a time
@@ -210,38 +302,49 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const bf16* x, long lon
 }
 
 int check_route(const RouteArgs& a) {
-  if (a.top < 1 || a.top > a.E || a.always < 0 || a.E + a.always > MAX_EXPERTS || a.chunk < 1 || a.tile < 1 || a.max_groups < 1) return -1;
+  if (a.top < 1 || a.top > a.choices || a.choices < a.E || a.choices > MAX_EXPERTS || a.always < 0 || a.E + a.always > MAX_EXPERTS || a.chunk < 1 || a.tile < 1 || a.max_groups < 1) return -1;
   if ((long long)a.T * (a.top + a.always) > 0x7fffffffll || a.chunk * (a.top + a.always) > 10240) return -2;
+  if (a.correction != nullptr && (!a.self_weight || a.sets < 1 || a.choices % a.sets || a.keep < 1 || a.keep > a.sets)) return -3;
   return 0;
+}
+
+template <int C>
+int launch_route(const RouteArgs& a, size_t smem, cudaStream_t st, bool pdl) {
+  const dim3 grid((a.T + a.chunk - 1) / a.chunk), block(ROUTE_THREADS);
+  return (int)(a.correction != nullptr ? prism_launch(moe_route_kernel<C, true>, grid, block, smem, st, pdl, a)
+                                       : prism_launch(moe_route_kernel<C, false>, grid, block, smem, st, pdl, a));
 }
 
 }  // namespace
 
 // logits: P fp32 slabs [T][ld] of E columns.  expert, pos, weight [T][top + always]; row_token [T * (top + always)]; counts
 // [chunks][E + always]; groups [max_groups] int4 and n_groups: tiles of at most `tile` rows of one expert.  With more than
-// one chunk prism_moe_place must follow.
+// one chunk prism_moe_place must follow.  correction != null: the scored form, with the logits of `choices` outputs (the E
+// experts, then those that stand for the token's own row, whose weight goes to self_weight [T]) and, at column always_col if
+// that is not negative, the one whose sigmoid weighs the always-on experts.
 PRISM_API int prism_moe_route(const void* logits, long long slab_stride, long long ld, int P, const void* slots, void* expert, void* pos,
                               void* weight, void* row_token, void* counts, void* groups, int max_groups, void* n_groups, int T, int top,
-                              int E, int always, int chunk, int tile, void* stream, int pdl) {
+                              int E, int always, int chunk, int tile, const void* correction, void* self_weight, int choices,
+                              int sets, int keep, int always_col, float scale, void* stream, int pdl) {
   if (T <= 0) return 0;
   RouteArgs a{(const float*)logits, slab_stride, ld, P, (const long long*)slots, (int*)expert, (int*)pos, (float*)weight, (int*)row_token,
-              (int*)counts, (int4*)groups, max_groups, (int*)n_groups, T, top, E, always, chunk, tile};
+              (int*)counts, (int4*)groups, max_groups, (int*)n_groups, T, top, E, always, chunk, tile, (const float*)correction,
+              (float*)self_weight, choices, sets, keep, always_col, scale};
   if (int rc = check_route(a)) return rc;
   const size_t smem = (size_t)chunk * (top + always) * sizeof(int);
-  const dim3 grid((T + chunk - 1) / chunk), block(ROUTE_THREADS);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  if (E <= 32) return (int)prism_launch(moe_route_kernel<1>, grid, block, smem, st, pdl != 0, a);
-  if (E <= 64) return (int)prism_launch(moe_route_kernel<2>, grid, block, smem, st, pdl != 0, a);
-  if (E <= 128) return (int)prism_launch(moe_route_kernel<4>, grid, block, smem, st, pdl != 0, a);
-  if (E <= 256) return (int)prism_launch(moe_route_kernel<8>, grid, block, smem, st, pdl != 0, a);
-  return (int)prism_launch(moe_route_kernel<MAX_EXPERTS / 32>, grid, block, smem, st, pdl != 0, a);
+  if (choices <= 32) return launch_route<1>(a, smem, st, pdl != 0);
+  if (choices <= 64) return launch_route<2>(a, smem, st, pdl != 0);
+  if (choices <= 128) return launch_route<4>(a, smem, st, pdl != 0);
+  if (choices <= 256) return launch_route<8>(a, smem, st, pdl != 0);
+  return launch_route<MAX_EXPERTS / 32>(a, smem, st, pdl != 0);
 }
 
 PRISM_API int prism_moe_place(void* expert, void* pos, void* weight, void* row_token, void* counts, void* groups, int max_groups,
                               void* n_groups, int T, int top, int E, int always, int chunk, int tile, void* stream, int pdl) {
   if (T <= 0) return 0;
   RouteArgs a{nullptr, 0, 0, 0, nullptr, (int*)expert, (int*)pos, (float*)weight, (int*)row_token, (int*)counts, (int4*)groups, max_groups,
-              (int*)n_groups, T, top, E, always, chunk, tile};
+              (int*)n_groups, T, top, E, always, chunk, tile, nullptr, nullptr, top > E ? top : E, 1, 1, -1, 1.0f};
   if (int rc = check_route(a)) return rc;
   return (int)prism_launch(moe_place_kernel, dim3((T + chunk - 1) / chunk), dim3(ROUTE_THREADS), 0, reinterpret_cast<cudaStream_t>(stream),
                            pdl != 0, a);

@@ -8,7 +8,7 @@
 // and what the next operation reads of it: the RMS-normalised row (with a weight, or with a scalar gain that the
 // next GEMM's epilogue applies), or the row itself (the loop projection's input, with the embedding beside it).
 // a and b come as fp32 split-K slabs, summed here in a fixed order, or as rows of the compute type; a may also be
-// the weighted sum of several (token, expert) rows.
+// the weighted sum of several (token, expert) rows, and of the stream's own row.
 #include "common.cuh"
 
 PRISM_DEFINE_TU_STATUS(stream)
@@ -53,6 +53,7 @@ struct Branch {
   const float* weight;     // [T][K]
   int K;
   const T* post_w;         // weight of the norm behind the sublayer (null: none)
+  const float* self_w;     // [T]: weight of the stream's row in the sum (null: none)
 };
 
 template <typename T>
@@ -64,6 +65,8 @@ struct StreamArgs {
   long long vocab;
   Branch<T> a, b;
   float mult;
+  float emb_mult;          // factor on the embedding rows
+  float w_offset;          // added to the weights of both norms (1: weights stored around zero)
   const T* bias;           // [W] (null: none)
   const T* norm_w;         // [W] (null: one)
   T* norm_out;             // rows x / sqrt(mean(x^2) + eps) * norm_w (null: not wanted)
@@ -161,6 +164,16 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
       }
     }
   }
+  if (a.a.self_w != nullptr) {
+    const float w = __ldg(a.a.self_w + t);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (i0 + u * step >= a.W) continue;
+      const F4 v = U == 1 && a.keep ? x[u] : load4(a.x + t * a.W + i0 + u * step);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[u].v[e] += w * v.v[e];
+    }
+  }
 #pragma unroll
   for (int u = 0; u < U; ++u)
 #pragma unroll
@@ -172,7 +185,7 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
       if (i0 + u * step >= a.W) continue;
       const F4 w = load4(a.a.post_w + i0 + u * step);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc[u].v[e] *= post * w.v[e];
+      for (int e = 0; e < 4; ++e) acc[u].v[e] *= post * (a.w_offset + w.v[e]);
     }
   } else if (has_a) {
 #pragma unroll
@@ -195,7 +208,9 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
       for (int e = 0; e < 4; ++e) acc[u].v[e] += s.v[e];
     }
     if (emb != nullptr) {
-      const F4 v = load4(emb + i);
+      F4 v = load4(emb + i);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v.v[e] *= a.emb_mult;
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[u].v[e] += v.v[e];
       if (a.embed_out != nullptr) store4(a.embed_out + t * a.embed_ld + i, v);
@@ -219,7 +234,7 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
     if (a.norm_w != nullptr) {
       const F4 w = load4(a.norm_w + i);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v.v[e] *= w.v[e];
+      for (int e = 0; e < 4; ++e) v.v[e] *= a.w_offset + w.v[e];
     }
     store4(a.norm_out + t * a.norm_ld + i, v);
   }
@@ -263,7 +278,7 @@ __global__ void __launch_bounds__(256) token_side_gate_kernel(const SideArgs<T> 
 template <typename T>
 int launch_side(const void* slabs, long long slab_stride, int P, const void* rows, long long ld, const void* table, long long vocab,
                 long long table_ld, long long offset, const void* ids, void* out, int T_rows, int D, cudaStream_t stream, bool pdl) {
-  SideArgs<T> a{Branch<T>{(const float*)slabs, slab_stride, P, (const T*)rows, ld, nullptr, 0, nullptr, nullptr, 0, nullptr},
+  SideArgs<T> a{Branch<T>{(const float*)slabs, slab_stride, P, (const T*)rows, ld, nullptr, 0, nullptr, nullptr, 0, nullptr, nullptr},
                 (const T*)table, vocab, table_ld, offset, (const long long*)ids, (T*)out, D, (long long)T_rows * D / 4};
   return (int)prism_launch(token_side_gate_kernel<T>, dim3((unsigned)((a.total + 255) / 256)), dim3(256), 0, stream, pdl, a);
 }
@@ -272,8 +287,8 @@ template <typename T>
 int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* table, long long vocab, const void* a_slabs,
                   long long a_stride, int a_P, const void* a_rows, long long a_ld, const void* a_gate, const void* b_slabs,
                   long long b_stride, int b_P, const void* b_rows, long long b_ld, const void* b_gate, long long gate_ld,
-                  const void* a_pos, const void* a_weight, int a_K, const void* a_post, float mult, const void* bias,
-                  const void* norm_w, void* norm_out, long long norm_ld, void* raw_out, long long raw_ld,
+                  const void* a_pos, const void* a_weight, int a_K, const void* a_post, const void* a_self, float mult,
+                  float emb_mult, float w_offset, const void* bias, const void* norm_w, void* norm_out, long long norm_ld, void* raw_out, long long raw_ld,
                   void* embed_out, long long embed_ld, int W, int W_real, float eps, cudaStream_t stream, bool pdl) {
   StreamArgs<T> a;
   a.x = (float*)x;
@@ -282,9 +297,12 @@ int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* ta
   a.table = (const T*)table;
   a.vocab = vocab;
   a.a = Branch<T>{(const float*)a_slabs, a_stride, a_P, (const T*)a_rows, a_ld, (const T*)a_gate, gate_ld,
-                  (const int*)a_pos, (const float*)a_weight, a_K, (const T*)a_post};
-  a.b = Branch<T>{(const float*)b_slabs, b_stride, b_P, (const T*)b_rows, b_ld, (const T*)b_gate, gate_ld, nullptr, nullptr, 0, nullptr};
+                  (const int*)a_pos, (const float*)a_weight, a_K, (const T*)a_post,
+                  (const float*)a_self};
+  a.b = Branch<T>{(const float*)b_slabs, b_stride, b_P, (const T*)b_rows, b_ld, (const T*)b_gate, gate_ld, nullptr, nullptr, 0, nullptr, nullptr};
   a.mult = mult;
+  a.emb_mult = emb_mult;
+  a.w_offset = w_offset;
   a.bias = (const T*)bias;
   a.norm_w = (const T*)norm_w;
   a.norm_out = (T*)norm_out;
@@ -311,24 +329,25 @@ int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* ta
 }  // namespace
 
 // f32: 1 = table, rows, gates, bias and outputs are fp32, 0 = bf16.  W a multiple of 8; every row stride a
-// multiple of 4 elements.
+// multiple of 4 elements.  a_self [T] (with a branch a): weight of the old stream row in it.  w_offset: added to norm weights.
 PRISM_API int prism_stream_update(int f32, int T, void* x, int keep, const void* ids, const void* table, long long vocab,
                                   const void* a_slabs, long long a_stride, int a_P, const void* a_rows, long long a_ld,
                                   const void* a_gate, const void* b_slabs, long long b_stride, int b_P, const void* b_rows,
                                   long long b_ld, const void* b_gate, long long gate_ld, const void* a_pos,
-                                  const void* a_weight, int a_K, const void* a_post, float mult, const void* bias,
+                                  const void* a_weight, int a_K, const void* a_post, const void* a_self, float mult,
+                                  float emb_mult, float w_offset, const void* bias,
                                   const void* norm_w, void* norm_out, long long norm_ld, void* raw_out, long long raw_ld, void* embed_out,
                                   long long embed_ld, int W, int W_real, float eps, void* stream, int pdl) {
   if (T <= 0) return 0;
   if (W <= 0 || W % 8 || W_real <= 0 || W_real > W || W > 32768) return -1;
   if ((a_ld | b_ld | gate_ld | norm_ld | raw_ld | embed_ld) % 4) return -2;
-  if ((a_pos != nullptr && (a_K <= 0 || !a_weight || a_gate)) || ((a_pos || a_post) && !a_slabs && !a_rows)) return -3;
+  if ((a_pos != nullptr && (a_K <= 0 || !a_weight || a_gate)) || ((a_pos || a_post || a_self) && !a_slabs && !a_rows)) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return f32 ? launch_stream<float>(T, x, keep, ids, table, vocab, a_slabs, a_stride, a_P, a_rows, a_ld, a_gate, b_slabs, b_stride,
-                                    b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, mult, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,
+                                    b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, a_self, mult, emb_mult, w_offset, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,
                                     embed_ld, W, W_real, eps, s, pdl != 0)
              : launch_stream<bf16>(T, x, keep, ids, table, vocab, a_slabs, a_stride, a_P, a_rows, a_ld, a_gate, b_slabs, b_stride,
-                                   b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, mult, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,
+                                   b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, a_self, mult, emb_mult, w_offset, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,
                                    embed_ld, W, W_real, eps, s, pdl != 0);
 }
 

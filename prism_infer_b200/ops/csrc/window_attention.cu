@@ -2,9 +2,11 @@
 //   row = [key heads x maps x dq | value heads x dv],
 // plain (one map) or differential (two maps: every head has two queries and two keys over one value; the outputs
 // are combined as (a1 - lam a2) over its root mean square, times a constant).  A query at position i sees key j when
-// j <= i and (i - j < window or j < keep).
+// j <= i and (i - j < window or j < keep).  Scores may be bounded (cap tanh(s / cap)) and a sink per head may take part in
+// the denominator of the softmax.
 //
-//   window_prepare_kernel      bias, norm over the whole query and key rows, rotation, page store, head gates
+//   window_prepare_kernel      bias, norm over the whole query and key rows or over each head, rotation, page store (values:
+//                              columns of their own, or the keys as projected), head gates
 //   window_decode_kernel       one query token per sequence: mma.sync over key tiles of 64, key range split over CTAs,
 //                              the last CTA of a (sequence, value head) merges the splits and combines maps / gates
 //   window_prefill_tc_kernel   128 query rows on tcgen05, two softmax streams per CTA (the two maps of a head, two
@@ -48,7 +50,7 @@ struct PrepareArgs {
   const T* rows;           // [T][ld]
   long long ld;
   const T* bias;           // [M] (null: none)
-  const T* q_w;            // norm weights over the whole query / key row (null: no norm)
+  const T* q_w;            // norm weights over the whole query / key row, or of one head (null: no norm)
   const T* k_w;
   const float* freq;       // [rot / 2]
   const int* positions;
@@ -58,6 +60,7 @@ struct PrepareArgs {
   T* cache;                // [slots][nk + nv]
   float* gate;             // [T][H] (null: no gates)
   int M, nq, nk, nv, H, dq, rot, q_real, k_real;
+  int v_col, gate_col;     // first column of the values and of the gates (tied values: the keys' first column)
   float eps;
   int shift;               // 2^shift unit places per map
 };
@@ -123,12 +126,13 @@ __device__ __forceinline__ float cluster_load(const float* own, int rank) {
 }
 
 // Threads keep their first U units in registers between the norm's sum and the rotation; others are read again.
-// PARTS CTAs (a cluster) per token; FEW tokens: norm weights fetched before the previous kernel has finished.  Widths
-// whose rotated half is not a multiple of four go element by element.
-template <typename T, int PARTS, bool FEW>
+// PARTS CTAs (a cluster) per token; FEW tokens: norm weights fetched before the previous kernel has finished; HEAD: norms
+// per head.  Widths whose rotated half is not a multiple of four go element by element.
+template <typename T, int PARTS, bool FEW, bool HEAD>
 __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
   constexpr int U = 2;
-  extern __shared__ float cs[];          // [rot / 2] cosines, then sines
+  extern __shared__ float cs[];          // [rot / 2] cosines, then sines, then the heads' norm factors where they are not
+                                         // formed in registers
   __shared__ float red[2][16], part_s[2];
   const size_t t = blockIdx.x / PARTS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = a.rot >> 1;
@@ -136,20 +140,30 @@ __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
   pdl_launch_dependents();
   const float pos = (float)a.positions[t];
   for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * a.freq[i], &cs[half + i], &cs[i]);
-  const int nqk = a.nq + a.nk, total = nqk + a.nv;
-  const bool vec = (half & 3) == 0, norm = a.q_w != nullptr;
+  const int nqk = a.nq + a.nk;
+  const bool vec = (half & 3) == 0, any_norm = a.q_w != nullptr, norm = any_norm && !HEAD;
+  const bool seg = HEAD && any_norm && vec && a.shift <= 5;  // the units of a head are neighbouring lanes
   const int units = vec ? (nqk / a.dq) << a.shift : 0;
+  float* hinv = cs + 2 * half;
   PrepareUnit pu[U];
   float4 w_lo[FEW ? U : 1], w_hi[FEW ? U : 1];
-  auto weight4 = [&](int c) { return c < a.nq ? load4(a.q_w + c) : load4(a.k_w + c - a.nq); };
+  auto weight4 = [&](const PrepareUnit& p, int o) {
+    if (HEAD) return load4((p.c < a.nq ? a.q_w : a.k_w) + p.d + o);
+    return p.c < a.nq ? load4(a.q_w + p.c + o) : load4(a.k_w + p.c + o - a.nq);
+  };
+  // 1 / root mean square of a unit's head from the sums of squares of its units (every lane of the warp)
+  auto segment_inv = [&](float ss) {
+    for (int o = 1; o < 1 << a.shift; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    return 1.0f / sqrtf(ss / (float)a.q_real + a.eps);
+  };
 #pragma unroll
   for (int k = 0; k < U; ++k) {
     const int u = tid + k * nt;
     pu[k].c = -1;
     if (u < units) pu[k] = prepare_unit(a, u);
-    if (FEW && norm && pu[k].c >= 0) {
-      w_lo[k] = weight4(pu[k].c);
-      if (pu[k].pair) w_hi[k] = weight4(pu[k].c + half);
+    if (FEW && any_norm && pu[k].c >= 0) {
+      w_lo[k] = weight4(pu[k], 0);
+      if (pu[k].pair) w_hi[k] = weight4(pu[k], half);
     }
   }
   pdl_wait();
@@ -169,16 +183,27 @@ __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
     }
   }
   if (page_row)
-    for (int c = tid * 4; c < a.nv; c += nt * 4) store4(page_row + a.nk + c, projected4(a, t, nqk + c));
+    for (int c = tid * 4; c < a.nv; c += nt * 4) store4(page_row + a.nk + c, projected4(a, t, a.v_col + c));
   if (a.gate != nullptr)
     for (int h = tid; h * 4 < a.H; h += nt) {
-      const float4 v = projected4(a, t, total + 4 * h);
+      const float4 v = projected4(a, t, a.gate_col + 4 * h);
       const float z[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
       for (int e = 0; e < 4; ++e)
         if (4 * h + e < a.H) a.gate[t * a.H + 4 * h + e] = 1.0f / (1.0f + expf(-z[e]));
     }
-  float iq = 1.0f, ik = 1.0f;
+  float iq = 1.0f, ik = 1.0f, unit_inv[U];
+  if (seg) {
+#pragma unroll
+    for (int k = 0; k < U; ++k) unit_inv[k] = segment_inv(sum_sq(lo[k]) + sum_sq(hi[k]));
+  } else if (HEAD && any_norm) {
+    for (int h = warp; h < nqk / a.dq; h += blockDim.x >> 5) {
+      float ss = 0.0f;
+      for (int c = lane * 4; c < a.dq; c += 128) ss += sum_sq(projected4(a, t, h * a.dq + c));
+      ss = warp_sum(ss);
+      if (lane == 0) hinv[h] = 1.0f / sqrtf(ss / (float)a.q_real + a.eps);
+    }
+  }
   if (norm) {
     float sq = 0.0f, sk = 0.0f;
     if (vec) {
@@ -229,9 +254,9 @@ __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
     else if (page_row) store4(page_row + c - a.nq, v);
   };
   if (vec) {
-    auto finish = [&](const PrepareUnit& p, float4 x, float4 y, float4 wx, float4 wy) {
-      if (norm) {
-        const float inv = p.c < a.nq ? iq : ik;
+    auto finish = [&](const PrepareUnit& p, float4 x, float4 y, float4 wx, float4 wy, float own) {
+      if (any_norm) {
+        const float inv = !HEAD ? (p.c < a.nq ? iq : ik) : (seg ? own : hinv[p.c / a.dq]);
         x = mul4(x, inv, wx);
         if (p.pair) y = mul4(y, inv, wy);
       }
@@ -247,19 +272,27 @@ __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
 #pragma unroll
     for (int k = 0; k < U; ++k)
       if (pu[k].c >= 0) {
-        if (FEW) finish(pu[k], lo[k], hi[k], w_lo[k], w_hi[k]);
-        else finish(pu[k], lo[k], hi[k], norm ? weight4(pu[k].c) : zero, norm && pu[k].pair ? weight4(pu[k].c + half) : zero);
+        if (FEW) finish(pu[k], lo[k], hi[k], w_lo[k], w_hi[k], unit_inv[k]);
+        else finish(pu[k], lo[k], hi[k], any_norm ? weight4(pu[k], 0) : zero, any_norm && pu[k].pair ? weight4(pu[k], half) : zero, unit_inv[k]);
       }
-    for (int u = tid + U * nt; u < units; u += nt) {
-      const PrepareUnit p = prepare_unit(a, u);
-      if (p.c < 0) continue;
-      finish(p, projected4(a, t, p.c), p.pair ? projected4(a, t, p.c + half) : zero, norm ? weight4(p.c) : zero,
-             norm && p.pair ? weight4(p.c + half) : zero);
+    for (int u0 = tid - (HEAD ? lane : 0) + U * nt; u0 < units; u0 += nt) {  // per head whole warps: segment_inv takes every lane
+      const int u = u0 + (HEAD ? lane : 0);
+      PrepareUnit p{-1, 0, false};
+      if (u < units) p = prepare_unit(a, u);
+      if (!HEAD && p.c < 0) continue;
+      float4 x = zero, y = zero;
+      if (p.c >= 0) {
+        x = projected4(a, t, p.c);
+        if (p.pair) y = projected4(a, t, p.c + half);
+      }
+      const float own = seg ? segment_inv(sum_sq(x) + sum_sq(y)) : 1.0f;
+      if (p.c >= 0) finish(p, x, y, any_norm ? weight4(p, 0) : zero, any_norm && p.pair ? weight4(p, half) : zero, own);
     }
   } else {
     auto value = [&](int c) {
       const float4 v = projected4(a, t, c & ~3);
       const float f = (c & 2) ? ((c & 1) ? v.w : v.z) : ((c & 1) ? v.y : v.x);
+      if (HEAD && any_norm) return f * hinv[c / a.dq] * to_f((c < a.nq ? a.q_w : a.k_w)[c % a.dq]);
       return norm ? f * (c < a.nq ? iq * to_f(a.q_w[c]) : ik * to_f(a.k_w[c - a.nq])) : f;
     };
     for (int c = tid; c < nqk; c += nt) {
@@ -277,17 +310,17 @@ __device__ __forceinline__ void prepare_token(const PrepareArgs<T>& a) {
   }
 }
 
-template <typename T>
+template <typename T, bool HEAD>
 __global__ void __cluster_dims__(PREP_PARTS, 1, 1) __launch_bounds__(256) window_prepare_few_kernel(const PrepareArgs<T> a) {
-  prepare_token<T, PREP_PARTS, true>(a);
+  prepare_token<T, PREP_PARTS, true, HEAD>(a);
 }
-template <typename T>
+template <typename T, bool HEAD>
 __global__ void __launch_bounds__(512) window_prepare_mid_kernel(const PrepareArgs<T> a) {
-  prepare_token<T, 1, true>(a);
+  prepare_token<T, 1, true, HEAD>(a);
 }
-template <typename T>
+template <typename T, bool HEAD>
 __global__ void __launch_bounds__(256, 4) window_prepare_kernel(const PrepareArgs<T> a) {
-  prepare_token<T, 1, false>(a);
+  prepare_token<T, 1, false, HEAD>(a);
 }
 
 // =====================================================================================
@@ -301,14 +334,29 @@ struct WinArgs {
   const int* cu_q;          // [S + 1] token offsets; null: sequence s is token s
   const int* kv_lens;       // [S] keys up to and including the sequence's last token
   const float* gate;        // [tokens][H] (null: one)
+  const float* sink;        // [H] (null: none); one map only
   T* out;                   // [tokens][out_ld]
   long long out_ld;
   float* part_o;            // decode partials [CTA group][nsplit][rows][dv]
   float* part_ml;           // [CTA group][nsplit][rows][2]
   int* counters;            // [CTA groups], zero-initialised, self-resetting
   int H, G, maps, dq, dv, vdim, R, page, max_blocks, num_blocks, window, keep, nsplit;
-  float scale, lam, gain, eps;
+  float scale, lam, gain, eps, cap;  // cap 0: scores are not bounded
 };
+
+// cap tanh(s scale / cap) times log2(e), as 1 - 2 / (exp(2x) + 1): a = 2 scale log2(e) / cap, b = cap log2(e).  The absolute
+// error is a few 2^-24 of cap.
+__device__ __forceinline__ float capped_log2(float s, float a, float b) { return b - __fdividef(2.0f * b, ex2_fast(s * a) + 1.0f); }
+
+// Factor on accumulated values whose weights sum to l relative to 2^m: one over the denominator, with the sink's part in it.
+__device__ __forceinline__ float softmax_factor(float l, float m, const float* sink, int h) {
+  if (!(l > 0.0f)) return 0.0f;
+  if (sink == nullptr) return 1.0f / l;
+  const float s = sink[h] * 1.4426950408889634f;
+  if (s <= m) return 1.0f / (l + ex2_fast(s - m));
+  const float f = ex2_fast(m - s);
+  return f / (l * f + 1.0f);
+}
 
 // Key tiles a query range [p_first, p_last] touches: the kept tiles before the window's first tile, then the window's.
 struct TileList {
@@ -348,7 +396,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
   constexpr int BM = 16 * MT;
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);                   // [BM][LDQ]
   bf16* ring = q_s + BM * LDQ;                                      // [4 warps][stages][16][LDR]
-  __shared__ float m_s[4][BM], l_s[4][BM], f_s[4][BM], L_s[BM];
+  __shared__ float m_s[4][BM], l_s[4][BM], f_s[4][BM], L_s[BM], M_s[BM];
   __shared__ __align__(8) uint64_t bars[4][4];
   __shared__ int last_s;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
@@ -414,6 +462,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
     for (int n = 0; n < DVT; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.0f;
   }
   const float sl2 = a.scale * 1.4426950408889634f;
+  const float cap_a = a.cap > 0.0f ? 2.0f * sl2 / a.cap : 0.0f, cap_b = a.cap * 1.4426950408889634f;
   const int dvt = a.dv >> 3, ksteps = KD >> 4;
   const bf16* qp = q_s + (lane & 15) * LDQ + 8 * (lane >> 4);
   uint32_t qr[MT][KS > 0 ? KS : 1][4];
@@ -470,7 +519,8 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
         for (int e = 0; e < 4; ++e) {
           const int j = j0 + n * 8 + t4 * 2 + (e & 1);
           const bool ok = whole || (j <= pos && (j > lo || j < a.keep));
-          s[m][n][e] = ok ? s[m][n][e] * sl2 : -INFINITY;
+          const float z = a.cap > 0.0f ? capped_log2(s[m][n][e], cap_a, cap_b) : s[m][n][e] * sl2;
+          s[m][n][e] = ok ? z : -INFINITY;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[m][n][e]);
         }
       float use[2], corr[2], sum[2] = {0.0f, 0.0f};
@@ -560,6 +610,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
       l += l_s[v][tid] * f;
     }
     L_s[tid] = l;
+    M_s[tid] = mx;
     if (a.nsplit > 1 && tid < rows) *reinterpret_cast<float2*>(a.part_ml + (base + tid) * 2) = make_float2(mx, l);
   }
   __syncthreads();
@@ -598,7 +649,10 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
       const float f = ml.x == -INFINITY ? 0.0f : ex2_fast(ml.x - mx);
       const float l = warp_sum(f * ml.y);
       if (lane < a.nsplit) coef[r * a.nsplit + lane] = f;
-      if (lane == 0) L_s[r] = l;
+      if (lane == 0) {
+        L_s[r] = l;
+        M_s[r] = mx;
+      }
     }
     __syncthreads();
     for (int i = tid; i < rows * per_row4; i += 128) {
@@ -622,7 +676,7 @@ __global__ void __launch_bounds__(128) window_decode_kernel(const WinArgs<bf16> 
   // ---- combine maps, gate, store: one head per warp
   for (int hh = warp; hh < rows / a.maps; hh += 4) {
     const int r = hh * a.maps, h = head0 + hh;
-    const float i1 = L_s[r] > 0.0f ? 1.0f / L_s[r] : 0.0f;
+    const float i1 = softmax_factor(L_s[r], M_s[r], a.sink, h);
     float f1 = i1, f2 = 0.0f, post = 1.0f;
     if (a.maps == 2) {
       f2 = L_s[r + 1] > 0.0f ? a.lam / L_s[r + 1] : 0.0f;
@@ -675,6 +729,7 @@ __device__ __forceinline__ void named_bar(int id, int threads) {
   asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory");
 }
 
+template <bool CAPPED>
 __global__ void __launch_bounds__(PRE_THREADS, 1)
 window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                          const __grid_constant__ CUtensorMap tmV, const PrefillArgs p) {
@@ -843,7 +898,8 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     const int last_key = min(pos_off + row, kv_len - 1);
     const int low = last_key - a.window;                             // keys after low are inside the window
     const uint32_t lanes = tmem_base + ((uint32_t)(q4 * 32) << 16);
-    const float sl2 = a.scale * 1.4426950408889634f;
+    const float scale2 = a.scale * 1.4426950408889634f, sl2 = CAPPED ? 1.0f : scale2;  // capped scores are in powers of two already
+    const float cap_a = CAPPED ? 2.0f * scale2 / a.cap : 0.0f, cap_b = a.cap * 1.4426950408889634f;
     constexpr float RAISE = 8.0f;  // the reference maximum rises only when a tile exceeds it by 2^8
     float m_ref = -INFINITY, l_run = 0.0f;
     bool ok = true;
@@ -867,6 +923,10 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         tmem_ld16(src + 32, r2);
         tmem_ld16(src + 48, r3);
         tmem_ld_wait();
+      }
+      if (CAPPED) {
+#pragma unroll
+        for (int i = 0; i < PKT; ++i) v[i] = capped_log2(v[i], cap_a, cap_b);
       }
       if (j0 + PKT - 1 > last_key || !(j0 > low || j0 + PKT <= a.keep)) {
 #pragma unroll
@@ -972,7 +1032,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     } else if (__all_sync(0xffffffffu, ok) && rows_here) {
       tc_fence_after();
       const int h = p.pair_heads ? head0 + s : head0;
-      float f = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+      float f = softmax_factor(l_run, m_ref, a.sink, h);
       if (a.gate != nullptr && store) f *= a.gate[(size_t)(q_start + row) * a.H + h];
       bf16* dst = a.out + (size_t)(q_start + row) * a.out_ld + (size_t)h * a.dv;
       for (int k = 0; k < chunks; ++k) {
@@ -1047,6 +1107,7 @@ __global__ void __launch_bounds__(128) window_simple_kernel(const WinArgs<T> a) 
         if (i < a.dq) s = fmaf(q[mp][e], to_f(k[mp * a.dq + i]), s);
       }
       s = warp_sum(s) * a.scale;
+      if (a.cap > 0.0f) s = a.cap * tanhf(s / a.cap);
       if (s > m[mp]) {
         const float f = expf(m[mp] - s);  // 0 for the first key
         m[mp] = s;
@@ -1081,6 +1142,10 @@ __global__ void __launch_bounds__(128) window_simple_kernel(const WinArgs<T> a) 
     float mx = -INFINITY, sum = 0.0f;
     for (int w = 0; w < 4; ++w)
       if (l_s[w][mp] > 0.0f) mx = fmaxf(mx, m_s[w][mp]);
+    if (a.sink != nullptr && mx > -INFINITY) {
+      mx = fmaxf(mx, a.sink[h]);
+      sum = expf(a.sink[h] - mx);
+    }
     for (int w = 0; w < 4; ++w) {
       f[mp][w] = l_s[w][mp] > 0.0f ? expf(m_s[w][mp] - mx) : 0.0f;
       sum += f[mp][w] * l_s[w][mp];
@@ -1112,14 +1177,17 @@ __global__ void __launch_bounds__(128) window_simple_kernel(const WinArgs<T> a) 
 
 template <typename T>
 WinArgs<T> win_args(const void* q, const void* cache, const void* block_tables, const void* cu_q, const void* kv_lens,
-                    const void* gate, void* out, long long out_ld, int H, int G, int maps, int dq, int dv, int vdim, int R, int page,
-                    int max_blocks, int num_blocks, int window, int keep, float scale, float lam, float gain, float eps) {
+                    const void* gate, const void* sink, void* out, long long out_ld, int H, int G, int maps, int dq, int dv, int vdim,
+                    int R, int page, int max_blocks, int num_blocks, int window, int keep, float scale, float lam, float gain, float eps,
+                    float cap) {
   return WinArgs<T>{(const T*)q, (const T*)cache, (const int*)block_tables, (const int*)cu_q, (const int*)kv_lens, (const float*)gate,
-                    (T*)out, out_ld, nullptr, nullptr, nullptr, H, G, maps, dq, dv, vdim, R, page, max_blocks, num_blocks, window, keep, 1,
-                    scale, lam, gain, eps};
+                    (const float*)sink, (T*)out, out_ld, nullptr, nullptr, nullptr, H, G, maps, dq, dv, vdim, R, page, max_blocks, num_blocks,
+                    window, keep, 1, scale, lam, gain, eps, cap};
 }
 
-int check_sizes(int H, int G, int maps, int dq, int dv, int vdim, int R, int page, int max_blocks, int window, int keep) {
+int check_sizes(int H, int G, int maps, int dq, int dv, int vdim, int R, int page, int max_blocks, int window, int keep, const void* sink,
+                float cap) {
+  if ((sink != nullptr && maps != 1) || !(cap >= 0.0f)) return -7;
   if (H <= 0 || G <= 0 || H % G || maps < 1 || maps > 2 || page <= 0 || max_blocks <= 0 || window < 1 || keep < 0) return -1;
   if (dq <= 0 || dq % 16 || dv <= 0 || dv % 16 || vdim <= 0 || vdim > dv || R != G * (maps * dq + dv)) return -2;
   return 0;
@@ -1159,52 +1227,58 @@ template <typename T>
 int launch_prepare(const void* slabs, long long slab_stride, int P, const void* rows, long long ld, const void* bias, const void* q_w,
                    const void* k_w, const void* freq, const void* positions, const void* slots, long long num_slots, void* q_out,
                    void* cache, void* gate, int tokens, int M, int nq, int nk, int nv, int H, int dq, int rot, int q_real, int k_real,
-                   float eps, cudaStream_t stream, bool pdl) {
+                   int head_norm, int tied, float eps, cudaStream_t s, bool pdl) {
   PrepareArgs<T> a{(const float*)slabs, slab_stride, P, (const T*)rows, ld, (const T*)bias, (const T*)q_w, (const T*)k_w,
                    (const float*)freq, (const int*)positions, (const long long*)slots, num_slots, (T*)q_out, (T*)cache, (float*)gate,
-                   M, nq, nk, nv, H, dq, rot, q_real, k_real, eps, 0};
+                   M, nq, nk, nv, H, dq, rot, q_real, k_real, tied ? nq : nq + nk, nq + nk + (tied ? 0 : nv), eps, 0};
   while ((1 << a.shift) < rot / 8 + (dq - rot) / 4) ++a.shift;
-  const size_t smem = (size_t)(rot + 4) * sizeof(float);
+  const size_t smem = (size_t)(rot + 4 + (head_norm ? (nq + nk) / dq : 0)) * sizeof(float);
   if (smem > 48 * 1024) return -5;
   // with a norm the cluster's exchange costs more than it spreads from a few dozen tokens on
-  if (tokens <= (q_w != nullptr ? 48 : 256))
-    return (int)prism_launch(window_prepare_few_kernel<T>, dim3(tokens * PREP_PARTS), dim3(M >= 4096 ? 256 : 128), smem, stream, pdl, a);
-  if (tokens <= 256) return (int)prism_launch(window_prepare_mid_kernel<T>, dim3(tokens), dim3(M >= 4096 ? 512 : 256), smem, stream, pdl, a);
-  return (int)prism_launch(window_prepare_kernel<T>, dim3(tokens), dim3(256), smem, stream, pdl, a);
+  if (tokens <= (q_w != nullptr && !head_norm ? 48 : 256))
+    return (int)prism_launch(head_norm ? window_prepare_few_kernel<T, true> : window_prepare_few_kernel<T, false>, dim3(tokens * PREP_PARTS),
+                             dim3(M >= 4096 ? 256 : 128), smem, s, pdl, a);
+  if (tokens <= 256)
+    return (int)prism_launch(head_norm ? window_prepare_mid_kernel<T, true> : window_prepare_mid_kernel<T, false>, dim3(tokens),
+                             dim3(M >= 4096 ? 512 : 256), smem, s, pdl, a);
+  return (int)prism_launch(head_norm ? window_prepare_kernel<T, true> : window_prepare_kernel<T, false>, dim3(tokens), dim3(256), smem, s, pdl, a);
 }
 
 }  // namespace
 
 // Stacked projection (fp32 slabs or rows of the compute type) -> queries, cache rows, sigmoid gates.  Columns: nq queries,
-// nk keys, nv values, then (gate != null) one gate per head; dq columns per map of a head, the first rot of them rotated.
+// nk keys, nv values (tied: none, the nv = nk values are the keys before norm and rotation), then (gate != null) one gate per
+// head; dq columns per map of a head, the first rot of them rotated.  head_norm: q_w and k_w [dq] hold for every head of
+// q_real = k_real columns.  nk = nv = 0: queries only.
 PRISM_API int prism_window_prepare(int f32, const void* slabs, long long slab_stride, int P, const void* rows, long long ld,
                                    const void* bias, const void* q_w, const void* k_w, const void* freq, const void* positions,
                                    const void* slots, long long num_slots, void* q_out, void* cache, void* gate, int tokens, int M,
-                                   int nq, int nk, int nv, int H, int dq, int rot, int q_real, int k_real, float eps, void* stream,
-                                   int pdl) {
+                                   int nq, int nk, int nv, int H, int dq, int rot, int q_real, int k_real, int head_norm, int tied,
+                                   float eps, void* stream, int pdl) {
   if (tokens <= 0) return 0;
-  if (dq <= 0 || dq % 16 || nq % dq || nk % dq || nv % 16 || M % 16 || M < nq + nk + nv + (gate ? H : 0)) return -1;
+  if (dq <= 0 || dq % 16 || nq % dq || nk % dq || nv % 16 || M % 16 || M < nq + nk + (tied ? 0 : nv) + (gate ? H : 0)) return -1;
+  if ((tied && nv != nk) || (head_norm && q_real != k_real)) return -3;
   if (rot < 0 || rot % 2 || rot > dq || (q_w != nullptr) != (k_w != nullptr) || (!slabs && (!rows || ld % 4))) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return f32 ? launch_prepare<float>(slabs, slab_stride, P, rows, ld, bias, q_w, k_w, freq, positions, slots, num_slots, q_out, cache, gate,
-                                     tokens, M, nq, nk, nv, H, dq, rot, q_real, k_real, eps, s, pdl != 0)
+                                     tokens, M, nq, nk, nv, H, dq, rot, q_real, k_real, head_norm, tied, eps, s, pdl != 0)
              : launch_prepare<bf16>(slabs, slab_stride, P, rows, ld, bias, q_w, k_w, freq, positions, slots, num_slots, q_out, cache, gate,
-                                    tokens, M, nq, nk, nv, H, dq, rot, q_real, k_real, eps, s, pdl != 0);
+                                    tokens, M, nq, nk, nv, H, dq, rot, q_real, k_real, head_norm, tied, eps, s, pdl != 0);
 }
 
 // One query token per sequence.  mt: 16-row tiles per CTA (1 or 2); nsplit > 1 needs the partial buffers
 // ([S * G * blocks][nsplit][16 mt][dv] and [...][2] floats) and zeroed counters [S * G * blocks].
 PRISM_API int prism_window_decode(const void* q, const void* cache, const void* block_tables, const void* cu_q, const void* kv_lens,
-                                  const void* gate, void* out, long long out_ld, void* part_o, void* part_ml, void* counters, int S,
+                                  const void* gate, const void* sink, void* out, long long out_ld, void* part_o, void* part_ml, void* counters, int S,
                                   int H, int G, int maps, int dq, int dv, int vdim, int R, int page, int max_blocks, int num_blocks,
-                                  int window, int keep, int mt, int nsplit, float scale, float lam, float gain, float eps,
+                                  int window, int keep, int mt, int nsplit, float scale, float lam, float gain, float eps, float cap,
                                   void* stream, int pdl) {
   if (S <= 0) return 0;
-  if (int rc = check_sizes(H, G, maps, dq, dv, vdim, R, page, max_blocks, window, keep)) return rc;
+  if (int rc = check_sizes(H, G, maps, dq, dv, vdim, R, page, max_blocks, window, keep, sink, cap)) return rc;
   if (maps * dq > 512 || dv > 256 || (mt != 1 && mt != 2) || (mt == 2 && dv > 128) || out_ld % 2 || cu_q != nullptr) return -3;
   if (nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_o || !part_ml || !counters))) return -4;
-  WinArgs<bf16> a = win_args<bf16>(q, cache, block_tables, cu_q, kv_lens, gate, out, out_ld, H, G, maps, dq, dv, vdim, R, page, max_blocks,
-                                   num_blocks, window, keep, scale, lam, gain, eps);
+  WinArgs<bf16> a = win_args<bf16>(q, cache, block_tables, cu_q, kv_lens, gate, sink, out, out_ld, H, G, maps, dq, dv, vdim, R, page, max_blocks,
+                                   num_blocks, window, keep, scale, lam, gain, eps, cap);
   a.part_o = (float*)part_o;
   a.part_ml = (float*)part_ml;
   a.counters = (int*)counters;
@@ -1224,15 +1298,15 @@ PRISM_API int prism_window_decode(const void* q, const void* cache, const void* 
 
 // Prompts and portions (cu_q: token offsets of the sequences), head widths up to 128, pages of a multiple of 8 rows.
 PRISM_API int prism_window_prefill_tc(const void* q, const void* cache, const void* block_tables, const void* cu_q, const void* kv_lens,
-                                      const void* gate, void* out, long long out_ld, int T, int S, int max_q_len, int H, int G, int maps,
+                                      const void* gate, const void* sink, void* out, long long out_ld, int T, int S, int max_q_len, int H, int G, int maps,
                                       int dq, int dv, int vdim, int R, int page, int max_blocks, int num_blocks, int window, int keep,
-                                      float scale, float lam, float gain, float eps, void* stream, int pdl) {
+                                      float scale, float lam, float gain, float eps, float cap, void* stream, int pdl) {
   if (T <= 0 || S <= 0 || max_q_len <= 0) return 0;
-  if (int rc = check_sizes(H, G, maps, dq, dv, vdim, R, page, max_blocks, window, keep)) return rc;
+  if (int rc = check_sizes(H, G, maps, dq, dv, vdim, R, page, max_blocks, window, keep, sink, cap)) return rc;
   if (dq > 128 || dv > 128 || page % 8 || !cu_q || num_blocks <= 0 || !(scale > 0.0f) || out_ld % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return -3;
   PrefillArgs p;
-  p.w = win_args<bf16>(q, cache, block_tables, cu_q, kv_lens, gate, out, out_ld, H, G, maps, dq, dv, vdim, R, page, max_blocks, num_blocks,
-                       window, keep, scale, lam, gain, eps);
+  p.w = win_args<bf16>(q, cache, block_tables, cu_q, kv_lens, gate, sink, out, out_ld, H, G, maps, dq, dv, vdim, R, page, max_blocks, num_blocks,
+                       window, keep, scale, lam, gain, eps, cap);
   p.k_maps = maps;
   p.pair_heads = maps == 1 && (H / G) % 2 == 0;
   p.box = 64;
@@ -1255,32 +1329,34 @@ PRISM_API int prism_window_prefill_tc(const void* q, const void* cache, const vo
   p.stages = 4;
   while (p.stages > 2 && fixed + p.stages * stage > 227 * 1024) --p.stages;
   const size_t smem = fixed + p.stages * stage;
-  static size_t configured = 0;
-  if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(window_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  void (*kernel)(const CUtensorMap, const CUtensorMap, const CUtensorMap, const PrefillArgs) =
+      cap > 0.0f ? window_prefill_tc_kernel<true> : window_prefill_tc_kernel<false>;
+  static size_t configured[2] = {0, 0};
+  if (smem > configured[cap > 0.0f]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    configured = smem;
+    configured[cap > 0.0f] = smem;
   }
   const int rows_per_cta = maps == 1 && !p.pair_heads ? 2 * PT : PT;
   const dim3 grid((max_q_len + rows_per_cta - 1) / rows_per_cta, p.pair_heads ? H / 2 : H, S);
-  return (int)prism_launch(window_prefill_tc_kernel, grid, dim3(PRE_THREADS), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, tq, tk,
+  return (int)prism_launch(kernel, grid, dim3(PRE_THREADS), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, tq, tk,
                            tv, p);
 }
 
 // Any sizes up to 512 elements per head, decode (cu_q null) and prompts, fp32 or bf16 storage.
 PRISM_API int prism_window_attention_simple(int f32, const void* q, const void* cache, const void* block_tables, const void* cu_q,
-                                            const void* kv_lens, const void* gate, void* out, long long out_ld, int S, int max_q_len,
+                                            const void* kv_lens, const void* gate, const void* sink, void* out, long long out_ld, int S, int max_q_len,
                                             int H, int G, int maps, int dq, int dv, int vdim, int R, int page, int max_blocks,
-                                            int num_blocks, int window, int keep, float scale, float lam, float gain, float eps,
+                                            int num_blocks, int window, int keep, float scale, float lam, float gain, float eps, float cap,
                                             void* stream, int pdl) {
   if (S <= 0 || max_q_len <= 0) return 0;
-  if (int rc = check_sizes(H, G, maps, dq, dv, vdim, R, page, max_blocks, window, keep)) return rc;
+  if (int rc = check_sizes(H, G, maps, dq, dv, vdim, R, page, max_blocks, window, keep, sink, cap)) return rc;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (f32)
-    return launch_simple<float>(win_args<float>(q, cache, block_tables, cu_q, kv_lens, gate, out, out_ld, H, G, maps, dq, dv, vdim, R, page,
-                                                max_blocks, num_blocks, window, keep, scale, lam, gain, eps),
+    return launch_simple<float>(win_args<float>(q, cache, block_tables, cu_q, kv_lens, gate, sink, out, out_ld, H, G, maps, dq, dv, vdim, R, page,
+                                                max_blocks, num_blocks, window, keep, scale, lam, gain, eps, cap),
                                 S, max_q_len, s, pdl != 0);
-  return launch_simple<bf16>(win_args<bf16>(q, cache, block_tables, cu_q, kv_lens, gate, out, out_ld, H, G, maps, dq, dv, vdim, R, page,
-                                            max_blocks, num_blocks, window, keep, scale, lam, gain, eps),
+  return launch_simple<bf16>(win_args<bf16>(q, cache, block_tables, cu_q, kv_lens, gate, sink, out, out_ld, H, G, maps, dq, dv, vdim, R, page,
+                                            max_blocks, num_blocks, window, keep, scale, lam, gain, eps, cap),
                              S, max_q_len, s, pdl != 0);
 }

@@ -113,7 +113,8 @@ class Branch:
     """Output of a sublayer on its way into the stream: fp32 ``slabs [S, T, W]`` or ``rows [T, W]``, with an
     element-wise ``gate [T, W]``.  With ``pos [T, K]`` the slabs or rows are those of (token, slot) pairs instead and a
     token's value is the sum of ``weight[t, k]`` times row ``pos[t, k]`` (negative: nothing).  ``post_norm [W]``: the
-    value is divided by its root mean square and multiplied by this weight before it is added."""
+    value is divided by its root mean square and multiplied by this weight before it is added.  ``self_weight [T]``: the
+    stream's own row, as it was, joins the value with this weight."""
 
     slabs: Optional[torch.Tensor] = None
     rows: Optional[torch.Tensor] = None
@@ -121,6 +122,7 @@ class Branch:
     pos: Optional[torch.Tensor] = None
     weight: Optional[torch.Tensor] = None
     post_norm: Optional[torch.Tensor] = None
+    self_weight: Optional[torch.Tensor] = None
 
     def value(self) -> torch.Tensor:
         v = self.slabs.sum(0) if self.slabs is not None else self.rows.float()
@@ -132,25 +134,29 @@ class Branch:
 def stream_update(x: torch.Tensor, width: int, eps: float, *, keep: bool, ids: Optional[torch.Tensor] = None,
                   table: Optional[torch.Tensor] = None, a: Optional[Branch] = None, b: Optional[Branch] = None, mult: float = 1.0,
                   bias: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, norm_out: Optional[torch.Tensor] = None,
-                  raw_out: Optional[torch.Tensor] = None, embed_out: Optional[torch.Tensor] = None) -> None:
-    """``x [T, W]`` (fp32, in place) ``= (x if keep) + table[ids] + mult * (a + b) + bias``, and what follows reads of
+                  raw_out: Optional[torch.Tensor] = None, embed_out: Optional[torch.Tensor] = None, embed_mult: float = 1.0,
+                  norm_offset: float = 0.0) -> None:
+    """``x [T, W]`` (fp32, in place) ``= (x if keep) + embed_mult * table[ids] + mult * (a + b) + bias``, and what follows reads of
     it: ``norm_out`` the rows over their root mean square (``width`` real columns, the rest are zero), times
     ``norm_weight`` if given, ``raw_out`` the rows themselves, ``embed_out`` the embedding rows, each in its own type.
-    Only ``a`` may consist of pairs or be normalised (``Branch.post_norm``)."""
-    assert b is None or (b.pos is None and b.post_norm is None)
+    Only ``a`` may consist of pairs or be normalised (``Branch.post_norm``).  ``norm_offset`` is added to the norm weights (1:
+    weights stored around zero)."""
+    assert b is None or (b.pos is None and b.post_norm is None and b.self_weight is None)
     T, W = x.shape
     if not x.is_cuda:
         new = x.clone() if keep else torch.zeros_like(x)
         for branch in (a, b):
             if branch is not None:
                 v = branch.value()
+                if branch.self_weight is not None:
+                    v = v + branch.self_weight[:, None] * x
                 if branch.post_norm is not None:
-                    v = v / torch.sqrt(v.pow(2).sum(-1, keepdim=True) / width + eps) * branch.post_norm.float()
+                    v = v / torch.sqrt(v.pow(2).sum(-1, keepdim=True) / width + eps) * (norm_offset + branch.post_norm.float())
                 new += mult * v
         if bias is not None:
             new += bias.float()
         if ids is not None:
-            emb = table[ids].float()
+            emb = table[ids].float() * embed_mult
             new += emb
             if embed_out is not None:
                 embed_out.copy_(emb)
@@ -159,7 +165,7 @@ def stream_update(x: torch.Tensor, width: int, eps: float, *, keep: bool, ids: O
             raw_out.copy_(new)
         if norm_out is not None:
             n = new / torch.sqrt(new.pow(2).sum(-1, keepdim=True) / width + eps)
-            norm_out.copy_(n if norm_weight is None else n * norm_weight.float())
+            norm_out.copy_(n if norm_weight is None else n * (norm_offset + norm_weight.float()))
         return
     kinds = [t.dtype for t in (table, bias, norm_weight, norm_out, raw_out, embed_out) if t is not None]
     for branch in (a, b):
@@ -182,9 +188,9 @@ def stream_update(x: torch.Tensor, width: int, eps: float, *, keep: bool, ids: O
     ld = lambda t: t.stride(0) if t is not None else 0  # noqa: E731
     pairs = a is not None and a.pos is not None
     extra = (_p(a.pos) if pairs else None, _p(a.weight) if pairs else None, a.pos.shape[1] if pairs else 0,
-             _p(a.post_norm) if a is not None else None)
+             _p(a.post_norm) if a is not None else None, _p(a.self_weight) if a is not None else None)
     native.call("prism_stream_update", 1 if kinds[0] == torch.float32 else 0, T, _p(x), 1 if keep else 0, _p(ids), _p(table),
-                table.shape[0] if table is not None else 0, *flat, gate_ld, *extra, float(mult), _p(bias), _p(norm_weight), _p(norm_out), ld(norm_out),
+                table.shape[0] if table is not None else 0, *flat, gate_ld, *extra, float(mult), float(embed_mult), float(norm_offset), _p(bias), _p(norm_weight), _p(norm_out), ld(norm_out),
                 _p(raw_out), ld(raw_out), _p(embed_out), ld(embed_out), W, width, float(eps), _s(),
                 0 if ids is not None else _pdl())  # the first kernel of a step may follow a copy: full dependency
 

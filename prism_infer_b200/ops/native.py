@@ -33,15 +33,20 @@ _SIGNATURES = {
     "prism_glu_f32": "ppiiipi",
     "prism_gemm_grouped_small": "pppiiiillpippiiiilpi",
     "prism_gemm_grouped": "pppiiillpipiipi",
-    "prism_moe_route": "pllippppppp" "ip" "iiiiiipi",
+    "prism_moe_route": "pllippppppp" "ip" "iiiiii" "ppiiiifpi",
     "prism_moe_place": "pppppp" "ip" "iiiiiipi",
     "prism_moe_gather": "plppiiipi",
-    "prism_window_prepare": "ipliplppp" "ppplppp" "iiiiiiiiii" "fpi",
-    "prism_window_decode": "pppppppl" "ppp" "iiiiiiiiiiiiiii" "ffffpi",
-    "prism_window_prefill_tc": "pppppppl" "iiiiiiiiiiiiiii" "ffffpi",
-    "prism_window_attention_simple": "ipppppppl" "iiiiiiiiiiiiii" "ffffpi",
+    "prism_window_prepare": "ipliplppp" "ppplppp" "iiiiiiiiiiii" "fpi",
+    "prism_window_decode": "ppppppppl" "ppp" "iiiiiiiiiiiiiii" "fffffpi",
+    "prism_window_prefill_tc": "ppppppppl" "iiiiiiiiiiiiiii" "fffffpi",
+    "prism_window_attention_simple": "ippppppppl" "iiiiiiiiiiiiii" "fffffpi",
+    "prism_token_mix": "ipliipppp" "iippippi" "pi",
+    "prism_tanh_split": "iplipl" "piipi",
+    "prism_state_step": "ipliippp" "ii" "plipl" "plipl" "ppppp" "iiii" "fpi",
+    "prism_state_scan": "ipliipppp" "ii" "plipl" "ppp" "iiipi",
+    "prism_head_norm_gate": "ip" "plipl" "pp" "iiii" "fpi",
     "prism_token_side_gate": "ipliplplllppiipi",
-    "prism_stream_update": "iipippl" "plipl" "p" "plipl" "p" "lppipfpp" "plplpl" "iifpi",
+    "prism_stream_update": "iipippl" "plipl" "p" "plipl" "p" "lppippfffpp" "plplpl" "iifpi",
     "prism_latent_norm_store": "iplppplpiiifpi",
     "prism_latent_absorb": "plppplppp" "liiiiifpi",
     "prism_latent_attention": "pppppppp" "iiiiiiiifpi",
@@ -98,7 +103,7 @@ _SIGNATURES = {
     "prism_decode_layers_seq_step": "i",
 }
 _STATUS_UNITS = ("gemm", "norm", "attn", "attn_tc", "kvops", "sampler", "comm", "decode_layers", "lm_head_fp8",
-                 "latent", "stream", "gemm_f32", "window", "moe")
+                 "latent", "stream", "gemm_f32", "window", "moe", "recurrence")
 
 
 class NativeError(RuntimeError):
