@@ -94,7 +94,7 @@ def prefill_ms(runner, tokens: int, steps: int, warmup: int) -> float:
     meta = AttnMeta(is_prefill=True, block_tables=torch.arange(pages, dtype=torch.int32, device=dev).view(1, -1),
                     slots=torch.arange(tokens, device=dev), cu_seqlens_q=torch.tensor([0, tokens], dtype=torch.int32, device=dev),
                     kv_lens=torch.tensor([tokens], dtype=torch.int32, device=dev), max_q_len=tokens, no_history=True, total_kv=tokens,
-                    max_kv_len=tokens, attended_pairs=tokens * tokens)
+                    max_kv_len=tokens, attended_pairs=tokens * tokens, **runner._state_meta([0]))
     return events_ms(lambda _: runner.model.forward(ids, pos, meta, cache), steps, warmup)
 
 
@@ -106,7 +106,8 @@ def decode_ms(runner, batch: int, context: int, steps: int, warmup: int) -> floa
     last = context - 1
     slots = table[:, last // runner.page].long() * runner.page + last % runner.page
     inp = StepInputs(kind="decode", input_ids=torch.randint(0, VOCAB - 8, (batch,)), positions=torch.full((3, batch), last, dtype=torch.int32),
-                     slots=slots, block_tables=table, temperatures=torch.zeros(batch), context_lens=torch.full((batch,), context, dtype=torch.int32))
+                     slots=slots, block_tables=table, temperatures=torch.zeros(batch), context_lens=torch.full((batch,), context, dtype=torch.int32),
+                     state_slots=torch.arange(batch, dtype=torch.int32) if runner.state is not None else None)
     runner.execute(inp)
     runner.time_decode_graph(warmup)
     return runner.time_decode_graph(steps)
@@ -146,10 +147,11 @@ class Kernels:
         self.bw, self.rate = peaks()
         self.rows: list[dict] = []
 
-    def time(self, family: str, name: str, like: str, fn, sets: int, nbytes: float, flops: float = 0.0) -> None:
-        """``fn(i)`` runs operand set ``i``; ``sets`` of them together exceed L2."""
+    def time(self, family: str, name: str, like: str, fn, sets: int, nbytes: float, flops: float = 0.0, rate: float = 0.0) -> None:
+        """``fn(i)`` runs operand set ``i``; ``sets`` of them together exceed L2.  ``rate``: FLOP/s of work that is not the tensor
+        cores'."""
         graph_ms = self._graph(fn, sets)
-        roof = max(nbytes / self.bw, flops / self.rate) * 1e3
+        roof = max(nbytes / self.bw, flops / (rate or self.rate)) * 1e3
         self.rows.append({"width": self.width, "family": family, "kernel": name, "like": like, "us": round(graph_ms * 1e3, 2),
                           "roofline_us": round(roof * 1e3, 2), "fraction": round(roof / graph_ms, 3)})
 
