@@ -384,7 +384,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 
 
 // ------------------------------------------------------------------------------------
-// Persistent form for prefill-sized problems (no split-K, bf16 output): one CTA per SM walks
+// Persistent form for prefill-sized problems (no split-K, bf16 output, or fp32 with tokens on the lanes): one CTA per SM walks
 // a strided list of output tiles.  The TMA producer runs ahead across tile boundaries, the
 // MMA thread alternates between two TMEM accumulators when both fit (BN * (DUAL ? 2 : 1)
 // <= 256 columns), and the epilogue warps drain one accumulator while the next tile's MMAs
@@ -397,6 +397,7 @@ struct PersistArgs {
   int m_tiles, n_tiles;
   int tokens_fastest;
   int act;
+  int out_f32;  // row-major form without residual or scatter: out is float
   long long ldo, ldr;
   const __nv_bfloat16* bias;
   const __nv_bfloat16* residual;
@@ -655,6 +656,12 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
               v[8 + 2 * e] = bf16_round(v[8 + 2 * e]) + x1.x;
               v[8 + 2 * e + 1] = bf16_round(v[8 + 2 * e + 1]) + x1.y;
             }
+          }
+          if (a.out_f32) {
+            float4* dst = reinterpret_cast<float4*>(reinterpret_cast<float*>(a.out) + (size_t)m * a.ldo + f0);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) dst[e] = make_float4(v[4 * e], v[4 * e + 1], v[4 * e + 2], v[4 * e + 3]);
+            continue;
           }
           uint4 o[2];
           __nv_bfloat162* op = reinterpret_cast<__nv_bfloat162*>(o);
@@ -989,7 +996,7 @@ static int gemm_wx_impl(const void* W, const void* X, void* out, int M, int T, i
   if (rc) return rc;
   const int m_tiles = (M + BM - 1) / BM;
   const bool p = pdl != 0;
-  if (g_persistent_min_tokens > 0 && T >= g_persistent_min_tokens && splits == 1 && !out_f32 && push == nullptr &&
+  if (g_persistent_min_tokens > 0 && T >= g_persistent_min_tokens && splits == 1 && (!out_f32 || sections != nullptr) && push == nullptr &&
       bn_override <= 0 && stages_override <= 0 &&
       (sections == nullptr || (sections_rowmajor && g_persistent_rowmajor && M % 16 == 0 && ldo % 8 == 0 &&
                                ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0))) {
@@ -1005,6 +1012,7 @@ static int gemm_wx_impl(const void* W, const void* X, void* out, int M, int T, i
     pa.m_tiles = m_tiles;
     pa.tokens_fastest = a.tokens_fastest;
     pa.act = act;
+    pa.out_f32 = out_f32;
     pa.ldo = ldo;
     pa.ldr = ldr;
     pa.bias = a.bias;
@@ -1267,6 +1275,7 @@ PRISM_API int prism_gemm_wx_scatter(const void* W, const void* X, int M, int T, 
   pa.n_tiles = (M + 255) / 256;
   pa.tokens_fastest = 0;
   pa.act = 0;
+  pa.out_f32 = 0;
   pa.ldo = M;
   pa.ldr = 0;
   pa.bias = nullptr;

@@ -15,6 +15,8 @@
 //   o_t = (S + diag(u) k v^T)^T r,   S <- diag(d) S + k v^T.
 #include "common.cuh"
 
+#include <type_traits>
+
 PRISM_DEFINE_TU_STATUS(recurrence)
 
 namespace {
@@ -32,6 +34,7 @@ __device__ __forceinline__ float4 load4(const bf16* p) {
   const float2 a = __bfloat1622float2(h[0]), b = __bfloat1622float2(h[1]);
   return make_float4(a.x, a.y, b.x, b.y);
 }
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ void store4(bf16* p, float4 v) {
   uint2 o;
@@ -73,6 +76,35 @@ __device__ __forceinline__ float proj1(const Proj<T>& p, size_t row, int c) {
   for (int i = 0; i < p.P; ++i) v += __ldcg(s + (size_t)i * p.slab_stride);
   return v;
 }
+
+// The same in two steps, so that many loads are under way before the first value is needed: what memory holds, and its value.
+__device__ __forceinline__ float4 raw_value(float4 r) { return r; }
+__device__ __forceinline__ float4 raw_value(uint2 r) {
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&r);
+  const float2 a = __bfloat1622float2(h[0]), b = __bfloat1622float2(h[1]);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename T, bool SLABS>
+struct RawProj {
+  typedef typename std::conditional<SLABS || std::is_same<T, float>::value, float4, uint2>::type type;
+  static __device__ __forceinline__ type zero() { return type{}; }
+  static __device__ __forceinline__ type load(const Proj<T>& p, size_t row, int c) {
+    if constexpr (SLABS) {
+      const float* s = p.slabs + row * p.ld + c;
+      float4 v = __ldcg(reinterpret_cast<const float4*>(s));
+      for (int i = 1; i < p.P; ++i) {
+        const float4 x = __ldcg(reinterpret_cast<const float4*>(s + (size_t)i * p.slab_stride));
+        v.x += x.x;
+        v.y += x.y;
+        v.z += x.z;
+        v.w += x.w;
+      }
+      return v;
+    } else {
+      return __ldcg(reinterpret_cast<const type*>(p.rows + row * p.ld + c));
+    }
+  }
+};
 
 // The state slots of a layer and the sequences of a step.
 struct StateArgs {
@@ -181,9 +213,9 @@ __global__ void __launch_bounds__(256) tanh_split_kernel(const Proj<T> z, T* out
 }
 
 // =====================================================================================
-// One token per sequence.  grid (heads, sequences).  Thread (ty, tx) owns value columns 4 tx .. 4 tx + 3 of key rows
-// ty, ty + rows, ...; up to NV of its state elements (float4) are fetched before the previous kernel has finished: they
-// were written by an earlier step.
+// One token per sequence.  grid (heads, sequences), NT threads.  Thread (ty, tx) owns value columns 4 tx .. 4 tx + 3 of key
+// rows ty, ty + rows, ...; up to NV of its state elements (float4) are fetched before the previous kernel has finished:
+// they were written by an earlier step.
 // =====================================================================================
 template <typename T>
 struct StepArgs {
@@ -199,23 +231,21 @@ struct StepArgs {
   float eps;
 };
 
-constexpr int STEP_THREADS = 256;
-
-template <typename T, int NV>
-__global__ void __launch_bounds__(STEP_THREADS) state_step_kernel(const StepArgs<T> a) {
+template <typename T, int NV, int NT>
+__global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_step_kernel(const StepArgs<T> a) {
   extern __shared__ float sm[];
   const int n = a.n, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, s = blockIdx.y;
-  float *r_s = sm, *k_s = sm + n, *v_s = sm + 2 * n, *g_s = sm + 3 * n, *d_s = sm + 4 * n, *t_s = sm + 5 * n;
+  float *r_s = sm, *k_s = sm + n, *v_s = sm + 2 * n, *g_s = sm + 3 * n, *d_s = sm + 4 * n, *b_s = sm + 5 * n, *t_s = sm + 6 * n;
   float* o_s = t_s + a.rank;                      // [rows][n] partial outputs
-  __shared__ float red[STEP_THREADS / 32], bonus_s;
-  const int c4 = n >> 2, rows = STEP_THREADS / c4, tx = tid % c4, ty = tid / c4;
+  __shared__ float red[NT / 32];
+  const int c4 = n >> 2, rows = NT / c4, tx = tid % c4, ty = tid / c4;
   pdl_launch_dependents();
   const Span sp = span_of(a.st, s);
   const size_t C = (size_t)a.H * n, hc = (size_t)h * n;
   T* out = a.out + (size_t)s * C + hc;
   if (sp.new_version == nullptr) {
     pdl_wait();
-    for (int c = tid; c < n; c += STEP_THREADS) put(out + c, 0.0f);
+    for (int c = tid; c < n; c += NT) put(out + c, 0.0f);
     return;
   }
   const float* old_s = sp.old_version ? sp.old_version + (size_t)h * n * n : nullptr;
@@ -227,22 +257,25 @@ __global__ void __launch_bounds__(STEP_THREADS) state_step_kernel(const StepArgs
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int key = ty + i * rows;
-      S[i] = active && key < n && old_s ? __ldcg(reinterpret_cast<const float4*>(old_s + (size_t)key * n) + tx) : zero;
+      S[i] = active && key < n && old_s ? __ldcs(reinterpret_cast<const float4*>(old_s + (size_t)key * n) + tx) : zero;
     }
   }
+  for (int i = tid * 128; i < n * a.rank * (int)sizeof(T); i += NT * 128)   // the head's rows of the decay projection
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(a.w2 + hc * a.rank) + i));
   pdl_wait();
   // the projections' sums, and the narrow one's tanh
-  for (int i = tid; i < 4 * c4 + a.rank; i += STEP_THREADS) {
+  for (int i = tid; i < 4 * c4 + a.rank; i += NT) {
     if (i < 4 * c4) {
-      const int m = i / c4, c = (i % c4) * 4;
+      const int m = i / c4, c = (i - m * c4) * 4;
       store4(sm + m * n + c, proj4(a.p, (size_t)m * a.tokens + s, (int)hc + c));
     } else {
       t_s[i - 4 * c4] = tanhf(proj1(a.w1, (size_t)s, i - 4 * c4));
     }
   }
   __syncthreads();
-  // decay: eight lanes per channel over the rank
-  for (int c0 = 0; c0 < n; c0 += STEP_THREADS / 8) {
+  // decay and bonus: eight lanes per channel over the rank
+#pragma unroll 4
+  for (int c0 = 0; c0 < n; c0 += NT / 8) {
     const int c = c0 + (tid >> 3);
     float z = 0.0f;
     if (c < n)
@@ -253,28 +286,23 @@ __global__ void __launch_bounds__(STEP_THREADS) state_step_kernel(const StepArgs
     z += __shfl_xor_sync(0xffffffffu, z, 1);
     z += __shfl_xor_sync(0xffffffffu, z, 2);
     z += __shfl_xor_sync(0xffffffffu, z, 4);
-    if (c < n && (tid & 7) == 0) d_s[c] = expf(-expf(z + to_f(a.w0[hc + c])));
+    if (c < n && (tid & 7) == 0) {
+      d_s[c] = expf(-expf(z + to_f(a.w0[hc + c])));
+      b_s[c] = r_s[c] * to_f(a.u[hc + c]) * k_s[c];
+    }
   }
-  float b = 0.0f;
-  for (int c = tid; c < n; c += STEP_THREADS) b += r_s[c] * to_f(a.u[hc + c]) * k_s[c];
-  b = warp_sum(b);
-  if (lane == 0) red[warp] = b;
   __syncthreads();
-  if (tid == 0) {
-    float t = 0.0f;
-    for (int i = 0; i < STEP_THREADS / 32; ++i) t += red[i];
-    bonus_s = t;
-  }
   if (active) {
     const float4 v = load4(v_s + 4 * tx);
     float4 o = zero;
     auto step = [&](int key, float4 st) {
-      const float r = r_s[key], k = k_s[key], d = d_s[key];
-      o.x = fmaf(r, st.x, o.x);
-      o.y = fmaf(r, st.y, o.y);
-      o.z = fmaf(r, st.z, o.z);
-      o.w = fmaf(r, st.w, o.w);
-      store4(new_s + (size_t)key * n + 4 * tx, make_float4(fmaf(d, st.x, k * v.x), fmaf(d, st.y, k * v.y), fmaf(d, st.z, k * v.z), fmaf(d, st.w, k * v.w)));
+      const float r = r_s[key], k = k_s[key], d = d_s[key], b = b_s[key];
+      o.x = fmaf(b, v.x, fmaf(r, st.x, o.x));
+      o.y = fmaf(b, v.y, fmaf(r, st.y, o.y));
+      o.z = fmaf(b, v.z, fmaf(r, st.z, o.z));
+      o.w = fmaf(b, v.w, fmaf(r, st.w, o.w));
+      __stcs(reinterpret_cast<float4*>(new_s + (size_t)key * n) + tx,
+             make_float4(fmaf(d, st.x, k * v.x), fmaf(d, st.y, k * v.y), fmaf(d, st.z, k * v.z), fmaf(d, st.w, k * v.w)));
     };
     if (NV > 0) {
 #pragma unroll
@@ -282,17 +310,18 @@ __global__ void __launch_bounds__(STEP_THREADS) state_step_kernel(const StepArgs
         if (ty + i * rows < n) step(ty + i * rows, S[i]);
     } else {
 #pragma unroll 8
-      for (int key = ty; key < n; key += rows) step(key, old_s ? __ldcg(reinterpret_cast<const float4*>(old_s + (size_t)key * n) + tx) : zero);
+      for (int key = ty; key < n; key += rows) step(key, old_s ? __ldcs(reinterpret_cast<const float4*>(old_s + (size_t)key * n) + tx) : zero);
     }
     store4(o_s + (size_t)ty * n + 4 * tx, o);
   }
   // the last token's row, a share per head
-  for (int c = (h * STEP_THREADS + tid) * 4; c < a.st.W; c += a.H * STEP_THREADS * 4)
+  for (int c = (h * NT + tid) * 4; c < a.st.W; c += a.H * NT * 4)
     store4(sp.new_version + a.st.carry + c, load4(a.st.x + (size_t)s * a.st.W + c));
   __syncthreads();
   float ss = 0.0f;
-  for (int c = tid; c < n; c += STEP_THREADS) {
-    float o = bonus_s * v_s[c];
+  for (int c = tid; c < n; c += NT) {
+    float o = 0.0f;
+#pragma unroll 8
     for (int i = 0; i < rows; ++i) o += o_s[(size_t)i * n + c];
     o_s[c] = o;                                   // column c is this thread's
     ss += o * o;
@@ -300,19 +329,17 @@ __global__ void __launch_bounds__(STEP_THREADS) state_step_kernel(const StepArgs
   ss = warp_sum(ss);
   if (lane == 0) red[warp] = ss;
   __syncthreads();
-  ss = warp_sum(lane < STEP_THREADS / 32 ? red[lane] : 0.0f);
+  ss = warp_sum(lane < NT / 32 ? red[lane] : 0.0f);
   const float inv = 1.0f / sqrtf(ss / (float)a.n_real + a.eps);
-  for (int c = tid; c < n; c += STEP_THREADS) {
-    const float g = g_s[c];
-    put(out + c, o_s[c] * inv * to_f(a.norm[hc + c]) * (g / (1.0f + expf(-g))));
-  }
+  for (int c = tid; c < n; c += NT) put(out + c, o_s[c] * inv * to_f(a.norm[hc + c]) * silu_f(g_s[c]));
 }
 
 // =====================================================================================
-// Many tokens per sequence.  grid (heads x column blocks of 32, sequences).  Four warps hold the state: a lane owns one
-// value column and every fourth group of four keys of it (KT keys in all), so a token costs KT / 4 times three 16-byte
-// shared-memory reads and the products in registers.  Four more warps fill the next block of TB tokens: sums of the
-// projections' slabs, decays, the bonus' scalar per token.
+// Many tokens per sequence.  grid (heads x column blocks of 32, sequences).  Four warps hold the state: a lane owns KL keys of
+// four value columns, sixteen lanes the keys of a column, so that a token costs a lane three 16-byte shared-memory reads per
+// four keys and one for the values; the lanes' partial outputs of four tokens are summed by one reduce-scatter.  Four more
+// warps feed blocks of TB tokens: while a block is worked on they turn the next one's raw rows, already in registers, into
+// what the products need (decays, the bonus' scalar per token) and fetch rows of the blocks behind it.
 // =====================================================================================
 constexpr int TB = 16;
 constexpr int SCAN_COLS = 32;
@@ -328,36 +355,24 @@ struct ScanArgs {
   int tokens, H, n;
 };
 
-__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
-  unsigned long long d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
-  unsigned long long d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ unsigned long long pair_of(float lo, float hi) {
-  unsigned long long d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ float pair_sum(unsigned long long v) {
-  float lo, hi;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-  return lo + hi;
-}
+template <int KL>
+struct ScanTile {
+  static constexpr int NP = 16 * KL;                            // keys, padded to the lanes' share
+  static constexpr int G = NP / 4;                              // groups of four keys
+  static constexpr int ITEMS = TB * G / 128;                    // (token, group) items of a loader thread
+  static constexpr int PARTS = G > 32 ? G / 32 : 1;             // warps that share a token's bonus
+  static constexpr int K = TB * NP, D = 2 * TB * NP, V = 3 * TB * NP, BONUS = V + TB * SCAN_COLS;
+  static constexpr int FLOATS = BONUS + TB * PARTS;             // one buffer: [r | k | d][TB][NP], v [TB][32], bonus
+};
 
-template <typename T, int KT>
+template <typename T, int KL, bool SLABS>
 __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs<T> a) {
-  extern __shared__ __align__(16) float sm[];
-  constexpr int NP = 4 * KT;                      // keys, padded to the lanes' share
+  extern __shared__ __align__(16) float sm[];                   // two buffers, then outputs [2][TB][32]
+  using Tile = ScanTile<KL>;
+  constexpr int NP = Tile::NP, G = Tile::G, ITEMS = Tile::ITEMS;
   const int n = a.n, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int blocks = (n + SCAN_COLS - 1) / SCAN_COLS, h = blockIdx.x / blocks, col0 = blockIdx.x % blocks * SCAN_COLS, s = blockIdx.y;
-  // two buffers of [r | k | d][TB][NP], v [TB][32], bonus [TB]; then outputs [TB][32] of the block under way
-  const int buf = 3 * TB * NP + TB * SCAN_COLS + TB;
-  float* out_s = sm + 2 * buf;
+  float* out_s = sm + 2 * Tile::FLOATS;
   pdl_launch_dependents();
   const Span sp = span_of(a.st, s);
   const size_t C = (size_t)a.H * n, hc = (size_t)h * n;
@@ -369,138 +384,239 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
       if (col0 + i % SCAN_COLS < n) a.o[(size_t)(sp.first + i / SCAN_COLS) * C + hc + col0 + i % SCAN_COLS] = 0.0f;
     return;
   }
-  auto fill = [&](int b, int w) {                 // one warp's tokens of block b
-    float* dst = sm + (b & 1) * buf;
+  if (warp >= 4) {
+    // ------------------------------ loaders ------------------------------
+    const int tid = threadIdx.x - 128, g = tid % G, c = g * 4;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const bool in = c < n;
+    const float4 u = in ? load4(a.u + hc + c) : zero;
+    const int vi = tid >> 3, vc = (tid & 7) * 4;                // 16 tokens x 8 groups of value columns
+    const bool v_in = col0 + vc < n;
+    using Raw = RawProj<T, SLABS>;
+    struct Rows {                                               // of one block
+      typename Raw::type r[ITEMS], k[ITEMS], v;
+      float4 z[ITEMS];
+    };
+    constexpr int AHEAD = ITEMS <= 4 ? 2 : 1;                   // blocks held in registers
+    Rows held[AHEAD];
+    auto fetch = [&](Rows& x, int b) {
+      if (b >= nb) return;
 #pragma unroll
-    for (int q = 0; q < TB / 4; ++q) {
-      const int i = w + 4 * q, tok = b * TB + i;
-      if (tok >= sp.len) continue;
-      const size_t t = (size_t)(sp.first + tok);
-      float bonus = 0.0f;
-      for (int c = lane * 4; c < NP; c += 128) {
-        float4 r = make_float4(0.f, 0.f, 0.f, 0.f), k = r, d = r;
-        if (c < n) {
-          r = proj4(a.p, t, (int)hc + c);
-          k = proj4(a.p, (size_t)a.tokens + t, (int)hc + c);
-          const float4 z = __ldcg(reinterpret_cast<const float4*>(a.z + t * C + hc + c)), u = load4(a.u + hc + c);
-          d = make_float4(expf(-expf(z.x)), expf(-expf(z.y)), expf(-expf(z.z)), expf(-expf(z.w)));
-          bonus += r.x * u.x * k.x + r.y * u.y * k.y + r.z * u.z * k.z + r.w * u.w * k.w;
+      for (int q = 0; q < ITEMS; ++q) {
+        const int tok = b * TB + tid / G + q * (128 / G);
+        x.r[q] = x.k[q] = Raw::zero();
+        x.z[q] = zero;
+        if (tok >= sp.len) x.z[q].x = x.z[q].y = x.z[q].z = x.z[q].w = -INFINITY;   // past the end: decay one, nothing added
+        else if (in) {
+          const size_t t = (size_t)(sp.first + tok);
+          x.r[q] = Raw::load(a.p, t, (int)hc + c);
+          x.k[q] = Raw::load(a.p, (size_t)a.tokens + t, (int)hc + c);
+          x.z[q] = __ldcg(reinterpret_cast<const float4*>(a.z + t * C + hc + c));
         }
-        store4(dst + i * NP + c, r);
-        store4(dst + (TB + i) * NP + c, k);
-        store4(dst + (2 * TB + i) * NP + c, d);
       }
-      if (lane * 4 < SCAN_COLS)
-        store4(dst + 3 * TB * NP + i * SCAN_COLS + lane * 4,
-               col0 + lane * 4 < n ? proj4(a.p, (size_t)2 * a.tokens + t, (int)hc + col0 + lane * 4) : make_float4(0.f, 0.f, 0.f, 0.f));
-      bonus = warp_sum(bonus);
-      if (lane == 0) dst[3 * TB * NP + TB * SCAN_COLS + i] = bonus;
+      x.v = Raw::zero();
+      if (v_in && b * TB + vi < sp.len) x.v = Raw::load(a.p, (size_t)2 * a.tokens + sp.first + b * TB + vi, (int)hc + col0 + vc);
+    };
+    auto store = [&](const Rows& x, int b) {
+      if (b >= nb) return;
+      float* dst = sm + (b & 1) * Tile::FLOATS;
+#pragma unroll
+      for (int q = 0; q < ITEMS; ++q) {
+        const int i = tid / G + q * (128 / G);
+        float4 d = zero;
+        if (in) d = make_float4(expf(-expf(x.z[q].x)), expf(-expf(x.z[q].y)), expf(-expf(x.z[q].z)), expf(-expf(x.z[q].w)));
+        const float4 rq = raw_value(x.r[q]), kq = raw_value(x.k[q]);
+        store4(dst + i * NP + c, rq);
+        store4(dst + Tile::K + i * NP + c, kq);
+        store4(dst + Tile::D + i * NP + c, d);
+        float bonus = rq.x * u.x * kq.x + rq.y * u.y * kq.y + rq.z * u.z * kq.z + rq.w * u.w * kq.w;
+#pragma unroll
+        for (int o = (G < 32 ? G : 32) / 2; o > 0; o >>= 1) bonus += __shfl_xor_sync(0xffffffffu, bonus, o);
+        if (g % 32 == 0) dst[Tile::BONUS + i * Tile::PARTS + g / 32] = bonus;
+      }
+      store4(dst + Tile::V + vi * SCAN_COLS + vc, raw_value(x.v));
+    };
+#pragma unroll
+    for (int e = 0; e < AHEAD; ++e) fetch(held[e], e);
+    store(held[0], 0);
+    fetch(held[0], AHEAD);
+    __syncthreads();
+    for (int b0 = 0; b0 < nb; b0 += AHEAD) {
+#pragma unroll
+      for (int e = 0; e < AHEAD; ++e) {
+        const int b = b0 + e;
+        if (b >= nb) break;
+        store(held[(e + 1) % AHEAD], b + 1);
+        fetch(held[(e + 1) % AHEAD], b + 1 + AHEAD);
+        __syncthreads();
+      }
     }
-  };
-  const bool loader = warp >= 4;
-  const int lk = lane & 3, col = (warp & 3) * 8 + (lane >> 2);     // column of the block
+    // the last token's row, a share per CTA
+    const float* last = a.st.x + (size_t)(sp.first + sp.len - 1) * a.st.W;
+    for (int i = (blockIdx.x * 128 + tid) * 4; i < a.st.W; i += gridDim.x * 512) store4(sp.new_version + a.st.carry + i, load4(last + i));
+    return;
+  }
+  // ------------------------------ state ------------------------------
+  const int kl = lane & 15, col = warp * 8 + (lane >> 4) * 4;    // first of the lane's columns in the block
   const bool live = col0 + col < n;
-  unsigned long long S[KT / 2];                   // keys 16 g + 4 lk + {0, 1}, {2, 3}
-  if (loader) {
-    fill(0, warp - 4);
-  } else {
+  unsigned long long S[KL / 2][4];                // keys 64 g + 4 kl + {0, 1}, {2, 3}
+  {
     const float* src = sp.old_version ? sp.old_version + (size_t)h * n * n + col0 + col : nullptr;
 #pragma unroll
-    for (int g = 0; g < KT / 4; ++g)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int key = 16 * g + 4 * lk + 2 * e;
-        const bool in = live && src && key < n;   // n is a multiple of 16
-        S[2 * g + e] = pair_of(in ? src[(size_t)key * n] : 0.0f, in ? src[(size_t)(key + 1) * n] : 0.0f);
+    for (int p = 0; p < KL / 2; ++p) {
+      const int key = 64 * (p >> 1) + 4 * kl + 2 * (p & 1);
+      float4 lo = make_float4(0.f, 0.f, 0.f, 0.f), hi = lo;
+      if (live && src && key < n) {               // n is a multiple of 16
+        lo = load4(src + (size_t)key * n);
+        hi = load4(src + (size_t)(key + 1) * n);
       }
+      S[p][0] = pair_of(lo.x, hi.x);
+      S[p][1] = pair_of(lo.y, hi.y);
+      S[p][2] = pair_of(lo.z, hi.z);
+      S[p][3] = pair_of(lo.w, hi.w);
+    }
   }
   __syncthreads();
   for (int b = 0; b < nb; ++b) {
-    if (loader) {
-      if (b + 1 < nb) fill(b + 1, warp - 4);
-    } else {
-      const float* src = sm + (b & 1) * buf;
-      const int cnt = min(TB, sp.len - b * TB);
-#pragma unroll 2
-      for (int i = 0; i < cnt; ++i) {
-        const float v = src[3 * TB * NP + i * SCAN_COLS + col];
-        const unsigned long long vv = pair_of(v, v);
-        unsigned long long o0 = 0, o1 = 0;
+    const float* __restrict__ src = sm + (b & 1) * Tile::FLOATS;
+    const float* __restrict__ rp = src + 4 * kl;
+    const int cnt = min(TB, sp.len - b * TB);
+    float* __restrict__ out_b = out_s + (b & 1) * TB * SCAN_COLS;
+    // partial outputs [token][column] of four tokens, and of the four before them, whose sum over the lanes goes on meanwhile
+    float x[16], done[16];
+    auto tokens4 = [&](int i0) {
 #pragma unroll
-        for (int g = 0; g < KT / 4; ++g) {
-          const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(src + i * NP + 16 * g + 4 * lk);
-          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(src + (TB + i) * NP + 16 * g + 4 * lk);
-          const ulonglong2 d = *reinterpret_cast<const ulonglong2*>(src + (2 * TB + i) * NP + 16 * g + 4 * lk);
-          o0 = fma2(r.x, S[2 * g], o0);
-          o1 = fma2(r.y, S[2 * g + 1], o1);
-          S[2 * g] = fma2(d.x, S[2 * g], mul2(k.x, vv));
-          S[2 * g + 1] = fma2(d.y, S[2 * g + 1], mul2(k.y, vv));
+      for (int q = 0; q < 4; ++q) {
+        const int i = i0 + q;
+        const float4 v = load4(src + Tile::V + i * SCAN_COLS + col);
+        const unsigned long long vv[4] = {pair_of(v.x, v.x), pair_of(v.y, v.y), pair_of(v.z, v.z), pair_of(v.w, v.w)};
+        unsigned long long o[4];
+#pragma unroll
+        for (int g = 0; g < KL / 4; ++g) {
+          const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(rp + i * NP + 64 * g);
+          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(rp + Tile::K + i * NP + 64 * g);
+          const ulonglong2 d = *reinterpret_cast<const ulonglong2*>(rp + Tile::D + i * NP + 64 * g);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            o[c] = g == 0 ? mul2(r.x, S[0][c]) : fma2(r.x, S[2 * g][c], o[c]);
+            S[2 * g][c] = fma2(d.x, S[2 * g][c], mul2(k.x, vv[c]));
+          }
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            o[c] = fma2(r.y, S[2 * g + 1][c], o[c]);
+            S[2 * g + 1][c] = fma2(d.y, S[2 * g + 1][c], mul2(k.y, vv[c]));
+          }
         }
-        float o = pair_sum(o0) + pair_sum(o1);
-        o += __shfl_xor_sync(0xffffffffu, o, 1);
-        o += __shfl_xor_sync(0xffffffffu, o, 2);
-        if (lk == 0) out_s[(b & 1) * TB * SCAN_COLS + i * SCAN_COLS + col] = fmaf(src[3 * TB * NP + TB * SCAN_COLS + i], v, o);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float2 f = unpair(o[c]);
+          x[4 * q + c] = f.x + f.y;
+        }
       }
-      // a warp's eight columns of the block
-      __syncwarp();
-      for (int i = lane >> 1; i < cnt; i += 16) {
-        const int c = (warp & 3) * 8 + (lane & 1) * 4;
-        if (col0 + c < n)
-          store4(a.o + (size_t)(sp.first + b * TB + i) * C + hc + col0 + c, load4(out_s + (b & 1) * TB * SCAN_COLS + i * SCAN_COLS + c));
+    };
+    auto finish4 = [&](int i0) {                  // sixteen lanes, sixteen sums: lane kl ends up with value kl
+      const int i = i0 + (kl >> 2), c = col + (kl & 3);
+      float bonus = src[Tile::BONUS + i * Tile::PARTS];
+#pragma unroll
+      for (int e = 1; e < Tile::PARTS; ++e) bonus += src[Tile::BONUS + i * Tile::PARTS + e];
+      const float v = src[Tile::V + i * SCAN_COLS + c];
+#pragma unroll
+      for (int m = 8; m > 0; m >>= 1) {
+        const bool up = (kl & m) != 0;
+#pragma unroll
+        for (int e = 0; e < m; ++e) {
+          const float send = up ? done[e] : done[e + m], own = up ? done[e + m] : done[e];
+          done[e] = own + __shfl_xor_sync(0xffffffffu, send, m);
+        }
       }
+      out_b[i * SCAN_COLS + c] = fmaf(bonus, v, done[0]);
+    };
+    auto keep = [&]() {
+#pragma unroll
+      for (int e = 0; e < 16; ++e) done[e] = x[e];
+    };
+    tokens4(0);
+    keep();
+    if (cnt > TB - 4) {
+#pragma unroll
+      for (int i0 = 4; i0 < TB; i0 += 4) {
+        tokens4(i0);
+        finish4(i0 - 4);
+        keep();
+      }
+      finish4(TB - 4);
+    } else {
+      int i0 = 4;
+      for (; i0 < cnt; i0 += 4) {                 // tokens past the end leave the state as it is
+        finish4(i0 - 4);
+        tokens4(i0);
+        keep();
+      }
+      finish4(i0 - 4);
+    }
+    // a warp's eight columns of the block
+    __syncwarp();
+    for (int i = lane >> 1; i < cnt; i += 16) {
+      const int c = warp * 8 + (lane & 1) * 4;
+      if (col0 + c < n) store4(a.o + (size_t)(sp.first + b * TB + i) * C + hc + col0 + c, load4(out_b + i * SCAN_COLS + c));
     }
     __syncthreads();
   }
-  if (!loader) {
-    float* dst = sp.new_version + (size_t)h * n * n + col0 + col;
+  if (!live) return;
+  float* dst = sp.new_version + (size_t)h * n * n + col0 + col;
 #pragma unroll
-    for (int g = 0; g < KT / 4; ++g)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int key = 16 * g + 4 * lk + 2 * e;
-        if (live && key < n) {
-          float lo, hi;
-          asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(S[2 * g + e]));
-          dst[(size_t)key * n] = lo;
-          dst[(size_t)(key + 1) * n] = hi;
-        }
-      }
-  } else {                                        // the last token's row, a share per CTA
-    const float* x = a.st.x + (size_t)(sp.first + sp.len - 1) * a.st.W;
-    for (int c = (blockIdx.x * 128 + threadIdx.x - 128) * 4; c < a.st.W; c += gridDim.x * 512)
-      store4(sp.new_version + a.st.carry + c, load4(x + c));
+  for (int p = 0; p < KL / 2; ++p) {
+    const int key = 64 * (p >> 1) + 4 * kl + 2 * (p & 1);
+    if (key >= n) continue;
+    const float2 f0 = unpair(S[p][0]), f1 = unpair(S[p][1]), f2 = unpair(S[p][2]), f3 = unpair(S[p][3]);
+    store4(dst + (size_t)key * n, make_float4(f0.x, f1.x, f2.x, f3.x));
+    store4(dst + (size_t)(key + 1) * n, make_float4(f0.y, f1.y, f2.y, f3.y));
   }
 }
 
-// out = o / rms(o) * norm * silu(gate) per head; one warp per (token, head)
-template <typename T>
+// out = o / rms(o) * norm * silu(gate) per head.  A lane holds eight columns, L lanes a head; four rows of a warp at a time.
+template <typename T, int L, bool SLABS>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, const Proj<T> p, const T* norm, T* out, int tokens, int H, int n,
                                                              int n_real, float eps) {
+  constexpr int ROWS = 4;
+  const int lane = threadIdx.x & 31, c = (lane % L) * 8;
+  const long long total = (long long)tokens * H, first = ((long long)blockIdx.x * 8 + (threadIdx.x >> 5)) * (32 / L) * ROWS + lane / L;
   pdl_launch_dependents();
   pdl_wait();
-  const long long i = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (i >= (long long)tokens * H) return;
-  const int lane = threadIdx.x & 31;
-  const size_t t = (size_t)(i / H);
-  const int hc = (int)(i % H) * n;
-  const float* row = o + t * (size_t)H * n + hc;
-  float4 v[2];
-  float ss = 0.0f;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  using Raw = RawProj<T, SLABS>;
+  float4 v[ROWS][2];
+  typename Raw::type g[ROWS][2];
+  long long t[ROWS];
+  int hc[ROWS];
+  bool in[ROWS];
 #pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const int c = (lane + 32 * e) * 4;
-    v[e] = c < n ? __ldcg(reinterpret_cast<const float4*>(row + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
-    ss += v[e].x * v[e].x + v[e].y * v[e].y + v[e].z * v[e].z + v[e].w * v[e].w;
+  for (int q = 0; q < ROWS; ++q) {
+    const long long i = first + q * (32 / L);
+    in[q] = i < total && c < n;
+    t[q] = in[q] ? i / H : 0;
+    hc[q] = in[q] ? (int)(i - t[q] * H) * n + c : 0;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      v[q][e] = in[q] ? __ldcg(reinterpret_cast<const float4*>(o + t[q] * (size_t)H * n + hc[q] + 4 * e)) : zero;
+      g[q][e] = in[q] ? Raw::load(p, (size_t)3 * tokens + t[q], hc[q] + 4 * e) : Raw::zero();
+    }
   }
-  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)n_real + eps);
 #pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const int c = (lane + 32 * e) * 4;
-    if (c >= n) continue;
-    const float4 g = proj4(p, (size_t)3 * tokens + t, hc + c), w = load4(norm + hc + c);
-    auto silu_f = [](float z) { return z / (1.0f + expf(-z)); };
-    store4(out + t * (size_t)H * n + hc + c, make_float4(v[e].x * inv * w.x * silu_f(g.x), v[e].y * inv * w.y * silu_f(g.y),
-                                                         v[e].z * inv * w.z * silu_f(g.z), v[e].w * inv * w.w * silu_f(g.w)));
+  for (int q = 0; q < ROWS; ++q) {
+    float ss = 0.0f;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) ss += v[q][e].x * v[q][e].x + v[q][e].y * v[q][e].y + v[q][e].z * v[q][e].z + v[q][e].w * v[q][e].w;
+#pragma unroll
+    for (int x = L / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+    const float inv = 1.0f / sqrtf(ss / (float)n_real + eps);
+    if (!in[q]) continue;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const float4 w = load4(norm + hc[q] + 4 * e), x = v[q][e], z = raw_value(g[q][e]);
+      store4(out + t[q] * (size_t)H * n + hc[q] + 4 * e, make_float4(x.x * inv * w.x * silu_f(z.x), x.y * inv * w.y * silu_f(z.y),
+                                                                   x.z * inv * w.z * silu_f(z.z), x.w * inv * w.w * silu_f(z.w)));
+    }
   }
 }
 
@@ -525,22 +641,22 @@ int allow_smem(K kernel, size_t smem, size_t& configured) {
   return (int)e;
 }
 
-template <typename T, int NV>
+template <typename T, int NV, int NT>
 int launch_step(const StepArgs<T>& a, cudaStream_t stream, bool pdl) {
-  const int rows = STEP_THREADS / (a.n / 4);
-  const size_t smem = (size_t)(5 * a.n + a.rank + rows * a.n) * sizeof(float);
+  const int rows = NT / (a.n / 4);
+  const size_t smem = (size_t)(6 * a.n + a.rank + rows * a.n) * sizeof(float);
   static size_t configured = 48 * 1024;
-  if (int rc = allow_smem(state_step_kernel<T, NV>, smem, configured)) return rc;
-  return (int)prism_launch(state_step_kernel<T, NV>, dim3(a.H, a.st.S), dim3(STEP_THREADS), smem, stream, pdl, a);
+  if (int rc = allow_smem(state_step_kernel<T, NV, NT>, smem, configured)) return rc;
+  return (int)prism_launch(state_step_kernel<T, NV, NT>, dim3(a.H, a.st.S), dim3(NT), smem, stream, pdl, a);
 }
 
-template <typename T, int KT>
+template <typename T, int KL, bool SLABS>
 int launch_scan(const ScanArgs<T>& a, cudaStream_t stream, bool pdl) {
-  const size_t smem = (size_t)(2 * (3 * TB * 4 * KT + TB * SCAN_COLS + TB) + 2 * TB * SCAN_COLS) * sizeof(float);
+  const size_t smem = (size_t)(2 * ScanTile<KL>::FLOATS + 2 * TB * SCAN_COLS) * sizeof(float);
   static size_t configured = 48 * 1024;
-  if (int rc = allow_smem(state_scan_kernel<T, KT>, smem, configured)) return rc;
+  if (int rc = allow_smem(state_scan_kernel<T, KL, SLABS>, smem, configured)) return rc;
   const dim3 grid(a.H * ((a.n + SCAN_COLS - 1) / SCAN_COLS), a.st.S);
-  return (int)prism_launch(state_scan_kernel<T, KT>, grid, dim3(SCAN_THREADS), smem, stream, pdl, a);
+  return (int)prism_launch(state_scan_kernel<T, KL, SLABS>, grid, dim3(SCAN_THREADS), smem, stream, pdl, a);
 }
 
 template <typename T>
@@ -600,10 +716,10 @@ PRISM_API int prism_state_step(int f32, void* state, long long row, int num_slot
     using T = decltype(type);
     StepArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), proj_of<T>(w1_slabs, w1_stride, w1_P, w1_rows, w1_ld), (const T*)w2,
                   (const T*)w0, (const T*)u, (const T*)norm, (T*)out, S, H, n, n_real, rank, eps};
-    const int rows = STEP_THREADS / (n / 4), nv = (n + rows - 1) / rows;
-    if (nv <= 4) return launch_step<T, 4>(a, s, pdl != 0);
-    if (nv <= 16) return launch_step<T, 16>(a, s, pdl != 0);
-    return launch_step<T, 0>(a, s, pdl != 0);
+    // float4s of the state per thread
+    if (n <= 64) return launch_step<T, 8, 128>(a, s, pdl != 0);
+    if (n <= 128) return launch_step<T, 16, 256>(a, s, pdl != 0);
+    return launch_step<T, 0, 256>(a, s, pdl != 0);
   };
   return f32 ? run(float()) : run(bf16());
 }
@@ -622,10 +738,13 @@ PRISM_API int prism_state_scan(int f32, void* state, long long row, int num_slot
   auto run = [&](auto type) -> int {
     using T = decltype(type);
     ScanArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), (const float*)z, (const T*)u, (float*)o, T_rows, H, n};
-    if (n <= 32) return launch_scan<T, 8>(a, s, pdl != 0);
-    if (n <= 64) return launch_scan<T, 16>(a, s, pdl != 0);
-    if (n <= 128) return launch_scan<T, 32>(a, s, pdl != 0);
-    return launch_scan<T, 64>(a, s, pdl != 0);
+    auto sized = [&](auto slabs) -> int {
+      constexpr bool SLABS = decltype(slabs)::value;
+      if (n <= 64) return launch_scan<T, 4, SLABS>(a, s, pdl != 0);
+      if (n <= 128) return launch_scan<T, 8, SLABS>(a, s, pdl != 0);
+      return launch_scan<T, 16, SLABS>(a, s, pdl != 0);
+    };
+    return p_slabs ? sized(std::true_type()) : sized(std::false_type());
   };
   return f32 ? run(float()) : run(bf16());
 }
@@ -636,10 +755,19 @@ PRISM_API int prism_head_norm_gate(int f32, const void* o, const void* p_slabs, 
                                    void* stream, int pdl) {
   if (T_rows <= 0) return 0;
   if (H <= 0 || n <= 0 || n % 16 || n > 256 || n_real <= 0 || n_real > n || (!p_slabs && !p_rows) || p_ld % 4) return -1;
-  const dim3 grid((unsigned)(((long long)T_rows * H + 7) / 8));
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return f32 ? (int)prism_launch(head_norm_gate_kernel<float>, grid, dim3(256), 0, s, pdl != 0, (const float*)o,
-                                 proj_of<float>(p_slabs, p_stride, p_P, p_rows, p_ld), (const float*)norm, (float*)out, T_rows, H, n, n_real, eps)
-             : (int)prism_launch(head_norm_gate_kernel<bf16>, grid, dim3(256), 0, s, pdl != 0, (const float*)o,
-                                 proj_of<bf16>(p_slabs, p_stride, p_P, p_rows, p_ld), (const bf16*)norm, (bf16*)out, T_rows, H, n, n_real, eps);
+  auto run = [&](auto type, auto lanes) -> int {
+    using T = decltype(type);
+    constexpr int L = decltype(lanes)::value, PER_CTA = 8 * (32 / L) * 4;
+    const dim3 grid((unsigned)(((long long)T_rows * H + PER_CTA - 1) / PER_CTA));
+    return (int)prism_launch(p_slabs ? head_norm_gate_kernel<T, L, true> : head_norm_gate_kernel<T, L, false>, grid, dim3(256), 0, s, pdl != 0,
+                             (const float*)o, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), (const T*)norm, (T*)out, T_rows, H, n, n_real, eps);
+  };
+  auto sized = [&](auto type) -> int {
+    if (n <= 32) return run(type, std::integral_constant<int, 4>());
+    if (n <= 64) return run(type, std::integral_constant<int, 8>());
+    if (n <= 128) return run(type, std::integral_constant<int, 16>());
+    return run(type, std::integral_constant<int, 32>());
+  };
+  return f32 ? sized(float()) : sized(bf16());
 }

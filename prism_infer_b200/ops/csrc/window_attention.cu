@@ -348,6 +348,28 @@ struct WinArgs {
 // error is a few 2^-24 of cap.
 __device__ __forceinline__ float capped_log2(float s, float a, float b) { return b - __fdividef(2.0f * b, ex2_fast(s * a) + 1.0f); }
 
+// The same by tanh's power series up to x^9, all on the multiply-add pipe: cap tanh(x) log2(e) with x = s scale / cap.  For
+// |x| < CAP_SERIES the first term left out is below 4e-7 of cap.
+constexpr float CAP_SERIES = 0.4f;
+struct CapSeries {
+  unsigned long long a0, a1, a2, a3, a4;   // the same value in both halves
+  __device__ __forceinline__ CapSeries(float scale, float cap) {
+    const float x = cap > 0.0f ? scale / cap : 0.0f, q = x * x, f = cap * 1.4426950408889634f * x;
+    auto both = [](float v) { return pair_of(v, v); };
+    a0 = both(f);
+    a1 = both(f * q * (-1.0f / 3.0f));
+    a2 = both(f * q * q * (2.0f / 15.0f));
+    a3 = both(f * q * q * q * (-17.0f / 315.0f));
+    a4 = both(f * q * q * q * q * (62.0f / 2835.0f));
+  }
+  __device__ __forceinline__ void operator()(float& u, float& v) const {
+    const unsigned long long s = pair_of(u, v), q = mul2(s, s);
+    const float2 r = unpair(mul2(s, fma2(q, fma2(q, fma2(q, fma2(q, a4, a3), a2), a1), a0)));
+    u = r.x;
+    v = r.y;
+  }
+};
+
 // Factor on accumulated values whose weights sum to l relative to 2^m: one over the denominator, with the sink's part in it.
 __device__ __forceinline__ float softmax_factor(float l, float m, const float* sink, int h) {
   if (!(l > 0.0f)) return 0.0f;
@@ -900,6 +922,8 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     const uint32_t lanes = tmem_base + ((uint32_t)(q4 * 32) << 16);
     const float scale2 = a.scale * 1.4426950408889634f, sl2 = CAPPED ? 1.0f : scale2;  // capped scores are in powers of two already
     const float cap_a = CAPPED ? 2.0f * scale2 / a.cap : 0.0f, cap_b = a.cap * 1.4426950408889634f;
+    const CapSeries series(a.scale, CAPPED ? a.cap : 0.0f);
+    const float small = CAPPED ? CAP_SERIES * a.cap / a.scale : 0.0f;
     constexpr float RAISE = 8.0f;  // the reference maximum rises only when a tile exceeds it by 2^8
     float m_ref = -INFINITY, l_run = 0.0f;
     bool ok = true;
@@ -925,8 +949,16 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         tmem_ld_wait();
       }
       if (CAPPED) {
+        float h4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-        for (int i = 0; i < PKT; ++i) v[i] = capped_log2(v[i], cap_a, cap_b);
+        for (int i = 0; i < PKT; ++i) h4[i & 3] = fmaxf(h4[i & 3], fabsf(v[i]));
+        if (__all_sync(0xffffffffu, fmaxf(fmaxf(h4[0], h4[1]), fmaxf(h4[2], h4[3])) < small)) {
+#pragma unroll
+          for (int i = 0; i < PKT; i += 2) series(v[i], v[i + 1]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < PKT; ++i) v[i] = capped_log2(v[i], cap_a, cap_b);
+        }
       }
       if (j0 + PKT - 1 > last_key || !(j0 > low || j0 + PKT <= a.keep)) {
 #pragma unroll
