@@ -125,14 +125,13 @@ class Kernels(base.Kernels):
         t = torch.empty(T, 2 * RANK, device=dev, dtype=torch.bfloat16)
         self.time("bokorax", f"tanh in two parts, {tag}", "", lambda i: native.call("prism_tanh_split", 0, *z1_args, t.data_ptr(), T, RANK, st(),
                                                                                     rec._pdl()), 4, z1.numel() * 4 + T * RANK * 4)
-        z = lat.linear_sections(t, w(0).w2, w(0)._decay, bias=w(0).w0, out_f32=True)
+        d = lat.linear_sections(t, w(0).w2, w(0)._decay, bias=w(0).w0, out_f32=True)
         self.time("bokorax", f"decay projection, wide, {tag}", "", lambda i: lat.linear_sections(t, w(i).w2, w(i)._decay, bias=w(i).w0, out_f32=True),
                   len(ws), C * RANK * 4 + T * (RANK * 4 + C * 4), 4.0 * C * RANK * T)
-        z.clamp_(-6.0, 0.0)
         o = torch.empty(T, C, device=dev)
 
         def scan(i):
-            native.call("prism_state_scan", 0, *views[i].args(sp), x.data_ptr(), batch, W, *p_args, z.data_ptr(), w(i).u.data_ptr(), o.data_ptr(), T, H,
+            native.call("prism_state_scan", 0, *views[i].args(sp), x.data_ptr(), batch, W, *p_args, d.data_ptr(), w(i).u.data_ptr(), o.data_ptr(), T, H,
                         n, st(), rec._pdl())
 
         # per state element: output product, decay product, key-value product and their sums

@@ -601,6 +601,10 @@ class LLMEngine:
         out["kv_pages_total"] = float(pool.num_blocks)
         out["kv_pages_used"] = float(pool.num_blocks - pool.num_free)
         out["kv_bytes_per_page"] = float(self.config.kv_bytes_per_page())
+        state = self.scheduler.block_manager.state
+        if state is not None:
+            out["state_slots_total"] = float(state.num_slots)
+            out["state_slots_used"] = float(state.num_slots - state.num_free)
         for k, v in self.scheduler.block_manager.prefix_cache_metadata().items():
             if isinstance(v, (int, float)) and not isinstance(v, bool) and k not in ("free_pages", "total_pages"):
                 out[f"prefix_cache_{k}"] = float(v)

@@ -780,6 +780,7 @@ class ModelRunner:
                 "launches_per_decode_graph": {str(b): getattr(g, "launches", 0) for b, g in self.graphs.items()},
                 "staging_bytes": {str(b): g.nbytes for b, g in self.graphs.items()},
                 "weight_bytes": self.model.weight_bytes(), "kv_sizing": getattr(self, "kv_sizing", None),
+                "state_bytes": self.state.bytes() if self.state is not None else 0,
                 "decode_run_ahead": dict(self.run_ahead_counters),
                 "decode_steps": {k: {str(n): c for n, c in sorted(v.items())} for k, v in self.decode_counters.items()}}
 

@@ -85,6 +85,8 @@ __device__ __forceinline__ float glu(float g, float u, int act) {
   return (act == PRISM_GLU_GELU_TANH ? gelu_tanh(g) : silu(g)) * u;
 }
 
+// Decay of a recurrence from the logarithm of its rate, in 32-bit.
+__device__ __forceinline__ float decay_of(float x) { return expf(-expf(x)); }
 __device__ __forceinline__ float sigmoid_fast(float x) { return 1.0f / (1.0f + __expf(-x)); }
 
 // ---- packed pairs of floats: two fused multiply-adds per instruction -----------------
@@ -112,7 +114,8 @@ __device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigne
 // ---- row sections of a stacked projection -------------------------------------------
 // One GEMM over several weight matrices stacked by rows: rows [row_end[i - 1], row_end[i]) are
 // scaled by alpha[i] (then the bias is added) and pass through activation act[i].
-enum PrismAct : int { PRISM_ACT_NONE = 0, PRISM_ACT_GELU_TANH = 1, PRISM_ACT_GELU_ERF = 2, PRISM_ACT_SIGMOID = 3, PRISM_ACT_SOFTCAP = 4 };
+enum PrismAct : int { PRISM_ACT_NONE = 0, PRISM_ACT_GELU_TANH = 1, PRISM_ACT_GELU_ERF = 2, PRISM_ACT_SIGMOID = 3, PRISM_ACT_SOFTCAP = 4,
+                      PRISM_ACT_DECAY = 5 };
 constexpr int PRISM_MAX_SECTIONS = 8;
 struct PrismSections {
   int n;      // 0: no sections
@@ -142,7 +145,7 @@ static inline bool prism_fill_sections(PrismSections& s, int n, const int* row_e
     s.row_end[i] = i < n ? row_end[i] : M;
     s.alpha[i] = i < n ? alpha[i] : 1.0f;
     s.act[i] = i < n ? act[i] : 0;
-    if (i < n && ((i > 0 && row_end[i] <= row_end[i - 1]) || act[i] < 0 || act[i] > PRISM_ACT_SOFTCAP)) return false;
+    if (i < n && ((i > 0 && row_end[i] <= row_end[i - 1]) || act[i] < 0 || act[i] > PRISM_ACT_DECAY)) return false;
     if (i < n && act[i] == PRISM_ACT_SOFTCAP && !(cap > 0.0f)) return false;
   }
   return row_end[n - 1] == M;

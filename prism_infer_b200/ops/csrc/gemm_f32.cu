@@ -30,6 +30,7 @@ __device__ __forceinline__ float act_f32(float v, int act, float cap) {
     case PRISM_ACT_GELU_ERF: return gelu_erf(v);
     case PRISM_ACT_SIGMOID: return 1.0f / (1.0f + expf(-v));
     case PRISM_ACT_SOFTCAP: return cap * tanhf(v / cap);
+    case PRISM_ACT_DECAY: return decay_of(v);
     default: return v;
   }
 }

@@ -85,6 +85,7 @@ __device__ __forceinline__ float apply_act(float v, int act, float cap) {
     case PRISM_ACT_GELU_ERF: return gelu_erf(v);
     case PRISM_ACT_SIGMOID: return sigmoid_fast(v);
     case PRISM_ACT_SOFTCAP: return cap * tanhf(v / cap);
+    case PRISM_ACT_DECAY: return decay_of(v);
     default: return v;
   }
 }
@@ -642,6 +643,9 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
           } else if (act == PRISM_ACT_SIGMOID) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = sigmoid_fast(v[j]);
+          } else if (act == PRISM_ACT_DECAY) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = decay_of(v[j]);
           }
           if (a.residual != nullptr) {
             const __nv_bfloat16* rs = a.residual + (size_t)m * a.ldr + f0;

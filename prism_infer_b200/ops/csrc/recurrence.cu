@@ -287,7 +287,7 @@ __global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_st
     z += __shfl_xor_sync(0xffffffffu, z, 2);
     z += __shfl_xor_sync(0xffffffffu, z, 4);
     if (c < n && (tid & 7) == 0) {
-      d_s[c] = expf(-expf(z + to_f(a.w0[hc + c])));
+      d_s[c] = decay_of(z + to_f(a.w0[hc + c]));
       b_s[c] = r_s[c] * to_f(a.u[hc + c]) * k_s[c];
     }
   }
@@ -339,9 +339,8 @@ __global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_st
 // four value columns, sixteen lanes the keys of a column, so that a token costs a lane three 16-byte shared-memory reads per
 // four keys and one for the values; the lanes' partial outputs of four tokens are summed by one reduce-scatter.  Four more
 // warps feed blocks of TB tokens: while a block is worked on they turn the next one's raw rows, already in registers, into
-// what the products need (decays, the bonus' scalar per token) and fetch rows of the blocks behind it.
+// what the products need (fp32, the bonus' scalar per token) and fetch rows of the blocks behind it.
 // =====================================================================================
-constexpr int TB = 16;
 constexpr int SCAN_COLS = 32;
 constexpr int SCAN_THREADS = 256;
 
@@ -349,7 +348,7 @@ template <typename T>
 struct ScanArgs {
   StateArgs st;
   Proj<T> p;               // r, k, v: rows m * tokens + t
-  const float* z;          // [tokens][heads * n]: decay exp(-exp(z))
+  const float* d;          // [tokens][heads * n] decays
   const T* u;              // [heads * n]
   float* o;                // [tokens][heads * n]
   int tokens, H, n;
@@ -357,6 +356,7 @@ struct ScanArgs {
 
 template <int KL>
 struct ScanTile {
+  static constexpr int TB = KL == 4 ? 32 : 16;                  // tokens of a block
   static constexpr int NP = 16 * KL;                            // keys, padded to the lanes' share
   static constexpr int G = NP / 4;                              // groups of four keys
   static constexpr int ITEMS = TB * G / 128;                    // (token, group) items of a loader thread
@@ -369,7 +369,7 @@ template <typename T, int KL, bool SLABS>
 __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs<T> a) {
   extern __shared__ __align__(16) float sm[];                   // two buffers, then outputs [2][TB][32]
   using Tile = ScanTile<KL>;
-  constexpr int NP = Tile::NP, G = Tile::G, ITEMS = Tile::ITEMS;
+  constexpr int TB = Tile::TB, NP = Tile::NP, G = Tile::G, ITEMS = Tile::ITEMS;
   const int n = a.n, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int blocks = (n + SCAN_COLS - 1) / SCAN_COLS, h = blockIdx.x / blocks, col0 = blockIdx.x % blocks * SCAN_COLS, s = blockIdx.y;
   float* out_s = sm + 2 * Tile::FLOATS;
@@ -390,12 +390,12 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     const bool in = c < n;
     const float4 u = in ? load4(a.u + hc + c) : zero;
-    const int vi = tid >> 3, vc = (tid & 7) * 4;                // 16 tokens x 8 groups of value columns
+    const int vi = tid >> 3, vc = (tid & 7) * 4;                // a token in sixteen, a group of value columns
     const bool v_in = col0 + vc < n;
     using Raw = RawProj<T, SLABS>;
     struct Rows {                                               // of one block
-      typename Raw::type r[ITEMS], k[ITEMS], v;
-      float4 z[ITEMS];
+      typename Raw::type r[ITEMS], k[ITEMS], v[TB / 16];
+      float4 d[ITEMS];
     };
     constexpr int AHEAD = ITEMS <= 4 ? 2 : 1;                   // blocks held in registers
     Rows held[AHEAD];
@@ -405,17 +405,20 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
       for (int q = 0; q < ITEMS; ++q) {
         const int tok = b * TB + tid / G + q * (128 / G);
         x.r[q] = x.k[q] = Raw::zero();
-        x.z[q] = zero;
-        if (tok >= sp.len) x.z[q].x = x.z[q].y = x.z[q].z = x.z[q].w = -INFINITY;   // past the end: decay one, nothing added
+        x.d[q] = zero;
+        if (tok >= sp.len) x.d[q].x = x.d[q].y = x.d[q].z = x.d[q].w = 1.0f;   // past the end: no decay, nothing added
         else if (in) {
           const size_t t = (size_t)(sp.first + tok);
           x.r[q] = Raw::load(a.p, t, (int)hc + c);
           x.k[q] = Raw::load(a.p, (size_t)a.tokens + t, (int)hc + c);
-          x.z[q] = __ldcg(reinterpret_cast<const float4*>(a.z + t * C + hc + c));
+          x.d[q] = __ldcg(reinterpret_cast<const float4*>(a.d + t * C + hc + c));
         }
       }
-      x.v = Raw::zero();
-      if (v_in && b * TB + vi < sp.len) x.v = Raw::load(a.p, (size_t)2 * a.tokens + sp.first + b * TB + vi, (int)hc + col0 + vc);
+#pragma unroll
+      for (int q = 0; q < TB / 16; ++q) {
+        const int tok = b * TB + vi + 16 * q;
+        x.v[q] = v_in && tok < sp.len ? Raw::load(a.p, (size_t)2 * a.tokens + sp.first + tok, (int)hc + col0 + vc) : Raw::zero();
+      }
     };
     auto store = [&](const Rows& x, int b) {
       if (b >= nb) return;
@@ -423,18 +426,17 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
 #pragma unroll
       for (int q = 0; q < ITEMS; ++q) {
         const int i = tid / G + q * (128 / G);
-        float4 d = zero;
-        if (in) d = make_float4(expf(-expf(x.z[q].x)), expf(-expf(x.z[q].y)), expf(-expf(x.z[q].z)), expf(-expf(x.z[q].w)));
         const float4 rq = raw_value(x.r[q]), kq = raw_value(x.k[q]);
         store4(dst + i * NP + c, rq);
         store4(dst + Tile::K + i * NP + c, kq);
-        store4(dst + Tile::D + i * NP + c, d);
+        store4(dst + Tile::D + i * NP + c, x.d[q]);
         float bonus = rq.x * u.x * kq.x + rq.y * u.y * kq.y + rq.z * u.z * kq.z + rq.w * u.w * kq.w;
 #pragma unroll
         for (int o = (G < 32 ? G : 32) / 2; o > 0; o >>= 1) bonus += __shfl_xor_sync(0xffffffffu, bonus, o);
         if (g % 32 == 0) dst[Tile::BONUS + i * Tile::PARTS + g / 32] = bonus;
       }
-      store4(dst + Tile::V + vi * SCAN_COLS + vc, raw_value(x.v));
+#pragma unroll
+      for (int q = 0; q < TB / 16; ++q) store4(dst + Tile::V + (vi + 16 * q) * SCAN_COLS + vc, raw_value(x.v[q]));
     };
 #pragma unroll
     for (int e = 0; e < AHEAD; ++e) fetch(held[e], e);
@@ -652,7 +654,7 @@ int launch_step(const StepArgs<T>& a, cudaStream_t stream, bool pdl) {
 
 template <typename T, int KL, bool SLABS>
 int launch_scan(const ScanArgs<T>& a, cudaStream_t stream, bool pdl) {
-  const size_t smem = (size_t)(2 * ScanTile<KL>::FLOATS + 2 * TB * SCAN_COLS) * sizeof(float);
+  const size_t smem = (size_t)(2 * ScanTile<KL>::FLOATS + 2 * ScanTile<KL>::TB * SCAN_COLS) * sizeof(float);
   static size_t configured = 48 * 1024;
   if (int rc = allow_smem(state_scan_kernel<T, KL, SLABS>, smem, configured)) return rc;
   const dim3 grid(a.H * ((a.n + SCAN_COLS - 1) / SCAN_COLS), a.st.S);
@@ -724,10 +726,10 @@ PRISM_API int prism_state_step(int f32, void* state, long long row, int num_slot
   return f32 ? run(float()) : run(bf16());
 }
 
-// Prompts and portions.  p: r, k, v (and the gate) of all T tokens one after another; z [T][H n] fp32; o [T][H n] fp32.
+// Prompts and portions.  p: r, k, v (and the gate) of all T tokens one after another; decay [T][H n] and o [T][H n] fp32.
 PRISM_API int prism_state_scan(int f32, void* state, long long row, int num_slots, int carry, const void* slots, const void* cu_q,
                                const void* kv_lens, const void* x, int S, int W, const void* p_slabs, long long p_stride, int p_P,
-                               const void* p_rows, long long p_ld, const void* z, const void* u, void* o, int T_rows, int H, int n,
+                               const void* p_rows, long long p_ld, const void* decay, const void* u, void* o, int T_rows, int H, int n,
                                void* stream, int pdl) {
   if (T_rows <= 0) return 0;
   if (int rc = check_state(row, num_slots, carry, S, W)) return rc;
@@ -737,7 +739,7 @@ PRISM_API int prism_state_scan(int f32, void* state, long long row, int num_slot
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   auto run = [&](auto type) -> int {
     using T = decltype(type);
-    ScanArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), (const float*)z, (const T*)u, (float*)o, T_rows, H, n};
+    ScanArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), (const float*)decay, (const T*)u, (float*)o, T_rows, H, n};
     auto sized = [&](auto slabs) -> int {
       constexpr bool SLABS = decltype(slabs)::value;
       if (n <= 64) return launch_scan<T, 4, SLABS>(a, s, pdl != 0);

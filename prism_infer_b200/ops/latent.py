@@ -17,7 +17,7 @@ import torch.nn.functional as F
 
 from . import SM_COUNT, KVCache, _p, _pdl, _s, choose_splits, linear, linear_partial, narrow_splits, native
 
-ACTS = {None: 0, "gelu_tanh": 1, "gelu": 2, "sigmoid": 3, "softcap": 4}
+ACTS = {None: 0, "gelu_tanh": 1, "gelu": 2, "sigmoid": 3, "softcap": 4, "decay": 5}
 MAX_SPLITS = 64
 MAX_LATENT = 1024       # widest latent row of the attention kernels
 FLASH_MAX_HEAD = 128    # widest head of the tcgen05 prefill attention
@@ -27,7 +27,7 @@ EXPAND_MAX_SCRATCH_BYTES = 2 << 30
 # ------------------------------------------------------------------------------ stacked projections
 class Sections:
     """Row ranges of a stacked weight matrix: ``(rows, alpha, act)`` each; ``cap`` bounds ``softcap`` sections
-    (``cap * tanh(v / cap)``)."""
+    (``cap * tanh(v / cap)``); ``decay`` is ``exp(-exp(v))``."""
 
     def __init__(self, parts: Sequence[tuple[int, float, Optional[str]]], cap: float = 0.0) -> None:
         self.parts = [(int(r), float(a), act) for r, a, act in parts]
@@ -53,6 +53,8 @@ def _apply(y: torch.Tensor, act: Optional[str], cap: float) -> torch.Tensor:
         return F.gelu(y, approximate="tanh")
     if act == "sigmoid":
         return torch.sigmoid(y)
+    if act == "decay":
+        return torch.exp(-torch.exp(y))
     return cap * torch.tanh(y / cap) if act == "softcap" else y
 
 

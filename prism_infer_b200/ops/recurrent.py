@@ -86,7 +86,7 @@ class TimeMixWeights:
 
     def __post_init__(self) -> None:
         self.w2_once = self.w2[:, :self.w2.shape[1] // 2].contiguous()
-        self._decay = Sections([(self.w2.shape[0], 1.0, None)])
+        self._decay = Sections([(self.w2.shape[0], 1.0, "decay")])
 
     def refresh(self) -> None:
         """After loading: what is derived from the loaded tensors."""
@@ -209,9 +209,9 @@ def time_mix(x: torch.Tensor, spec: TimeMixSpec, w: TimeMixWeights, st: StateVie
         return out
     t = torch.empty((T, 2 * spec.rank), dtype=dtype, device=dev)
     native.call("prism_tanh_split", f32, *_proj_args(Branch(slabs=z1)), _p(t), T, spec.rank, _s(), _pdl())
-    z = linear_sections(t, w.w2, w._decay, bias=w.w0, out_f32=True)
+    d = linear_sections(t, w.w2, w._decay, bias=w.w0, out_f32=True)
     o = torch.empty((T, spec.cols), dtype=torch.float32, device=dev)
-    native.call("prism_state_scan", f32, *st.args(spec), _p(x), S, spec.width, *_proj_args(p), _p(z), _p(w.u), _p(o), T, spec.heads, spec.n,
+    native.call("prism_state_scan", f32, *st.args(spec), _p(x), S, spec.width, *_proj_args(p), _p(d), _p(w.u), _p(o), T, spec.heads, spec.n,
                 _s(), _pdl())
     native.call("prism_head_norm_gate", f32, _p(o), *_proj_args(p), _p(w.norm), _p(out), T, spec.heads, spec.n, spec.dim, float(spec.eps), _s(),
                 _pdl())
