@@ -94,7 +94,7 @@ class Kernels(base.Kernels):
         cache = rec.StateCache([sp.carry + W] * sets, batch, dev)
         x = torch.randn(T, W, device=dev)
         ws = [rec.TimeMixWeights(torch.rand(5, W, device=dev).bfloat16(), self.matrix(4 * C, W).view(4, C, W), self.matrix(RANK, W),
-                                 self.matrix(C, 2 * RANK), torch.full((C,), -2.0, device=dev).bfloat16(), self.matrix(1, C)[0], self.matrix(1, C)[0])
+                                 self.matrix(C, RANK), torch.full((C,), -2.0, device=dev).bfloat16(), self.matrix(1, C)[0], self.matrix(1, C)[0])
               for _ in range(min(sets, 8))]
         slots = torch.arange(batch, dtype=torch.int32, device=dev)
         lens = torch.full((batch,), 64 + tokens, dtype=torch.int32, device=dev)
@@ -117,17 +117,14 @@ class Kernels(base.Kernels):
         if decode:
             def step(i):
                 m = w(i)
-                native.call("prism_state_step", 0, *views[i].args(sp, cu=False), x.data_ptr(), batch, W, *p_args, *z1_args, m.w2_once.data_ptr(),
+                native.call("prism_state_step", 0, *views[i].args(sp, cu=False), x.data_ptr(), batch, W, *p_args, *z1_args, m.w2.data_ptr(),
                             m.w0.data_ptr(), m.u.data_ptr(), m.norm.data_ptr(), out.data_ptr(), H, n, n, RANK, 1e-6, st(), rec._pdl())
 
             self.time("bokorax", f"state step, {tag}", "", step, sets, 2 * state_bytes + wide_out + C * (RANK + 3) * 2 + batch * C * 2)
             return
-        t = torch.empty(T, 2 * RANK, device=dev, dtype=torch.bfloat16)
-        self.time("bokorax", f"tanh in two parts, {tag}", "", lambda i: native.call("prism_tanh_split", 0, *z1_args, t.data_ptr(), T, RANK, st(),
-                                                                                    rec._pdl()), 4, z1.numel() * 4 + T * RANK * 4)
-        d = lat.linear_sections(t, w(0).w2, w(0)._decay, bias=w(0).w0, out_f32=True)
-        self.time("bokorax", f"decay projection, wide, {tag}", "", lambda i: lat.linear_sections(t, w(i).w2, w(i)._decay, bias=w(i).w0, out_f32=True),
-                  len(ws), C * RANK * 4 + T * (RANK * 4 + C * 4), 4.0 * C * RANK * T)
+        d = rec.decays(z1, w(0))
+        self.time("bokorax", f"decays, {tag}", "stacked projection", lambda i: rec.decays(z1, w(i)), len(ws),
+                  C * RANK * 2 + z1.numel() * 4 + T * C * 4, 4.0 * C * RANK * T)
         o = torch.empty(T, C, device=dev)
 
         def scan(i):

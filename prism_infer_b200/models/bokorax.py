@@ -42,7 +42,7 @@ class BokoraxLayerWeights(LayerWeights):           # norms: norm1, norm2
         yield from super().tensors()
         if self.mix is not None:
             m = self.mix
-            yield from (m.mu, m.rkvg, m.w1, m.w2, m.w2_once, m.w0, m.u, m.norm)
+            yield from (m.mu, m.rkvg, m.w1, m.w2, m.w0, m.u, m.norm)
 
 
 class BokoraxModel(WindowedDecoder):
@@ -65,7 +65,7 @@ class BokoraxModel(WindowedDecoder):
     def _alloc_time_mix(self, w: BokoraxLayerWeights, m: TimeMixArch) -> None:
         w.mix_spec = s = rec.TimeMixSpec(m.heads, m.dim, padded(m.decay_rank), self.W, self.arch.norm_eps)
         w.mix = rec.TimeMixWeights(mu=self._z(5, self.W), rkvg=self._z(4, s.cols, self.W), w1=self._z(s.rank, self.W),
-                                   w2=self._z(s.cols, 2 * s.rank), w0=self._z(s.cols), u=self._z(s.cols), norm=self._z(s.cols))
+                                   w2=self._z(s.cols, s.rank), w0=self._z(s.cols), u=self._z(s.cols), norm=self._z(s.cols))
         w.o = self._z(self.W, s.cols)
 
     # ------------------------------------------------------------------- loading
@@ -87,8 +87,7 @@ class BokoraxModel(WindowedDecoder):
         elif sub == "w1":
             self._into(m.w1[:t.shape[0], :width], t)
         elif sub == "w2":
-            for first in (0, s.rank):
-                self._into(heads(m.w2)[..., first:first + rank], t.view(H, d, rank))
+            self._into(heads(m.w2)[..., :rank], t.view(H, d, rank))
         elif sub in ("w0", "u", "norm"):
             self._into(heads(getattr(m, sub)), t.view(H, d))
         elif sub == "o":
@@ -96,11 +95,6 @@ class BokoraxModel(WindowedDecoder):
         else:
             return False
         return True
-
-    def _loaded(self) -> None:
-        for w in self.weights:
-            if w.mix is not None:
-                w.mix.refresh()
 
     # ---------------------------------------------------------------------- text
     def _reads_stream(self, layer: int) -> Optional[bool]:

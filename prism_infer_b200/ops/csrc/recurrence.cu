@@ -6,14 +6,14 @@
 // starts from zero whatever its slot holds.
 //
 //   token_mix_kernel      five blends of a token's row with the previous token's, and the table of a grouped projection
-//   tanh_split_kernel     tanh of a narrow projection as a sum of two numbers of the compute type
+//   decay_project_kernel  decays of many tokens from the narrow projection's rows (bf16; fp32 takes the 32-bit GEMM)
 //   state_step_kernel     one token per sequence: decay, output, state update, norm per head, gate
 //   state_scan_kernel     many tokens of a sequence: the state stays in registers, loader warps feed token blocks
 //   head_norm_gate_kernel norm per head and gate behind the scan
 //
 // Per head, with r, k, v, the decay d = exp(-exp(z)) and the bonus u (all fp32):
 //   o_t = (S + diag(u) k v^T)^T r,   S <- diag(d) S + k v^T.
-#include "common.cuh"
+#include "mma_sync.cuh"
 
 #include <type_traits>
 
@@ -196,20 +196,140 @@ __global__ void __launch_bounds__(256) token_mix_kernel(const MixArgs<T> a) {
   }
 }
 
-// out[t] = [hi, lo] with hi + lo = tanh(z_t) to about twice the type's precision: the next projection multiplies both.
-template <typename T>
-__global__ void __launch_bounds__(256) tanh_split_kernel(const Proj<T> z, T* out, int R, long long total) {
+// =====================================================================================
+// decay[t][c] = exp(-exp(w0[c] + W2[c] . tanh(z_t))), the narrow rows z summed on the way in.  A CTA makes 64 tokens x
+// `tiles` times 128 channels; tanh(z) enters the products as the sum of two bf16 numbers, so that only the weights' own rounding is left.
+// =====================================================================================
+constexpr int DP_TOKENS = 64, DP_COLS = 128, DP_K = 128;
+struct DecayArgs {
+  const float* z;          // [P][T][ld] slabs whose sum is the narrow projection
+  long long stride, ld;
+  int P;
+  const bf16* w2;          // [C][R]
+  const bf16* w0;          // [C]
+  float* out;              // [T][C]
+  int T, C, R, tiles;
+};
+
+// Place of a block's thread in a matrix of `groups` groups per row, 256 places on with every step.
+struct Walk {
+  int row, group, groups, rows_on, groups_on;
+  __device__ __forceinline__ Walk(int i, int groups_) : row(i / groups_), group(i % groups_), groups(groups_), rows_on(256 / groups_), groups_on(256 % groups_) {}
+  __device__ __forceinline__ void next() {
+    row += rows_on;
+    group += groups_on;
+    if (group >= groups) {
+      group -= groups;
+      ++row;
+    }
+  }
+};
+// With the hardware's exponential: absolute errors of a few 2^-23.
+__device__ __forceinline__ float tanh_exp(float x) { return 1.0f - __fdividef(2.0f, __expf(2.0f * x) + 1.0f); }
+__device__ __forceinline__ float decay_fast(float x) { return __expf(-__expf(x)); }
+
+__global__ void __launch_bounds__(256, 3) decay_project_kernel(const DecayArgs a) {
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  const int LD = min(DP_K, a.R) + 8;
+  bf16* hi_s = reinterpret_cast<bf16*>(smem_raw);               // [64][LD]
+  bf16* lo_s = hi_s + DP_TOKENS * LD;
+  bf16* w_s = lo_s + DP_TOKENS * LD;                            // [128][LD]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, t0 = blockIdx.y * DP_TOKENS;
+  const int wt = (warp & 3) * 16, wc = (warp >> 2) * 64;        // the warp's tokens and channels
+  pdl_launch_dependents();
+  for (int tile = 0; tile < a.tiles; ++tile) {
+    const int c0 = (blockIdx.x * a.tiles + tile) * DP_COLS;
+    if (c0 >= a.C) break;
+    float acc[8][4] = {};
+    for (int k0 = 0; k0 < a.R; k0 += DP_K) {
+      const int kn = min(DP_K, a.R - k0);                         // a multiple of 16
+      if (tile + k0 > 0) __syncthreads();
+      Walk w(tid, kn / 8);
+      while (w.row < DP_COLS) {                   // four groups at a time, all their loads first
+        uint4 v[4];
+        int at[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q, w.next()) {
+          at[q] = w.row < DP_COLS ? w.row * LD + w.group * 8 : -1;
+          v[q] = __ldg(reinterpret_cast<const uint4*>(a.w2 + (size_t)min(c0 + w.row, a.C - 1) * a.R + k0 + w.group * 8));
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+          if (at[q] >= 0) *reinterpret_cast<uint4*>(w_s + at[q]) = v[q];   // channels past the end are not stored
+      }
+      if (tile + k0 == 0) pdl_wait();             // the weights do not depend on the previous kernel
+      Walk z(tid, kn / 4);
+      while ((tile == 0 || a.R > DP_K) && z.row < DP_TOKENS) {
+        float4 v[4];
+        int at[4];
+        size_t src[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q, z.next()) {
+          at[q] = z.row < DP_TOKENS ? z.row * LD + z.group * 4 : -1;
+          src[q] = (size_t)min(t0 + z.row, a.T - 1) * a.ld + k0 + z.group * 4;   // rows past the end are not stored
+          v[q] = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll 2
+        for (int p = 0; p < a.P; ++p) {
+          const float* slab = a.z + (size_t)p * a.stride;
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            const float4 x = __ldcg(reinterpret_cast<const float4*>(slab + src[q]));
+            v[q].x += x.x;
+            v[q].y += x.y;
+            v[q].z += x.z;
+            v[q].w += x.w;
+          }
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          if (at[q] < 0) continue;
+          const float4 x = make_float4(tanh_exp(v[q].x), tanh_exp(v[q].y), tanh_exp(v[q].z), tanh_exp(v[q].w));
+          const float4 h = make_float4(bf16_round(x.x), bf16_round(x.y), bf16_round(x.z), bf16_round(x.w));
+          store4(hi_s + at[q], h);
+          store4(lo_s + at[q], make_float4(x.x - h.x, x.y - h.y, x.z - h.z, x.w - h.w));
+        }
+      }
+      __syncthreads();
+      const bf16* hp = hi_s + (wt + (lane & 15)) * LD + 8 * (lane >> 4);
+      const bf16* lp = lo_s + (wt + (lane & 15)) * LD + 8 * (lane >> 4);
+      const bf16* wp = w_s + (wc + (lane & 7) + 8 * (lane >> 4)) * LD + 8 * ((lane >> 3) & 1);
+      for (int k = 0; k < kn; k += 16) {
+        uint32_t h[4], l[4];
+        ldsm_x4(h, smem_u32(hp + k));
+        ldsm_x4(l, smem_u32(lp + k));
+#pragma unroll
+        for (int n = 0; n < 8; n += 2) {
+          uint32_t b[4];
+          ldsm_x4(b, smem_u32(wp + n * 8 * LD + k));
+          mma_bf16(acc[n], h, b[0], b[1]);
+          mma_bf16(acc[n], l, b[0], b[1]);
+          mma_bf16(acc[n + 1], h, b[2], b[3]);
+          mma_bf16(acc[n + 1], l, b[2], b[3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < 8; ++n) {
+      const int c = c0 + wc + n * 8 + (lane & 3) * 2;             // C is a multiple of 16
+      if (c >= a.C) continue;
+      const float b0 = to_f(a.w0[c]), b1 = to_f(a.w0[c + 1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = t0 + wt + (lane >> 2) + 8 * e;
+        if (t < a.T)
+          *reinterpret_cast<float2*>(a.out + (size_t)t * a.C + c) = make_float2(decay_fast(acc[n][2 * e] + b0), decay_fast(acc[n][2 * e + 1] + b1));
+      }
+    }
+  }
+}
+
+// out = tanh of the summed rows, fp32
+__global__ void __launch_bounds__(256) tanh_f32_kernel(const Proj<float> z, float* out, int R, long long total) {
   pdl_launch_dependents();
   pdl_wait();
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
-  if (i >= total) return;
-  const long long t = i / R;
-  const int c = (int)(i - t * R);
-  const float v = tanhf(proj1(z, (size_t)t, c));
-  T hi;
-  put(&hi, v);
-  out[t * 2 * R + c] = hi;
-  put(out + t * 2 * R + R + c, v - to_f(hi));
+  if (i < total) out[i] = tanhf(proj1(z, (size_t)(i / R), (int)(i % R)));
 }
 
 // =====================================================================================
@@ -689,16 +809,30 @@ PRISM_API int prism_token_mix(int f32, void* state, long long row, int num_slots
              : launch_mix<bf16>(st, mu, out, T, groups, n_groups, tile, s, pdl != 0);
 }
 
-// out [T][2 R] = [hi, lo], hi + lo = tanh(z).  z as fp32 slabs or rows of the compute type.
-PRISM_API int prism_tanh_split(int f32, const void* slabs, long long slab_stride, int P, const void* rows, long long ld, void* out, int T,
-                               int R, void* stream, int pdl) {
+// bf16: decay [T][C] fp32 = exp(-exp(w0 + W2 tanh(z))), z the sum of P fp32 slabs [T][ld] of R columns, w2 [C][R].  R and C
+// multiples of 16.
+PRISM_API int prism_decay_project(const void* slabs, long long slab_stride, int P, long long ld, const void* w2, const void* w0, void* out,
+                                  int T, int C, int R, void* stream, int pdl) {
   if (T <= 0) return 0;
-  if (R <= 0 || (!slabs && !rows)) return -1;
+  if (C <= 0 || C % 16 || R <= 0 || R % 16 || !slabs || P < 1 || ld % 4 || ld < R || (reinterpret_cast<uintptr_t>(w2) & 15)) return -1;
+  DecayArgs a{(const float*)slabs, slab_stride, ld, P, (const bf16*)w2, (const bf16*)w0, (float*)out, T, C, R, 1};
+  const int col_tiles = (C + DP_COLS - 1) / DP_COLS, token_tiles = (T + DP_TOKENS - 1) / DP_TOKENS;
+  const int across = 3 * 148 / token_tiles;       // CTAs side by side: three per SM, and no second wave, where that is possible
+  a.tiles = (col_tiles + (across > 1 ? across : 1) - 1) / (across > 1 ? across : 1);
+  const size_t smem = (size_t)(2 * DP_TOKENS + DP_COLS) * ((R < DP_K ? R : DP_K) + 8) * sizeof(bf16);
+  static size_t configured = 48 * 1024;
+  if (int rc = allow_smem(decay_project_kernel, smem, configured)) return rc;
+  const dim3 grid((col_tiles + a.tiles - 1) / a.tiles, token_tiles);
+  return (int)prism_launch(decay_project_kernel, grid, dim3(256), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
+}
+
+// out [T][R] = tanh(z), fp32
+PRISM_API int prism_tanh_f32(const void* slabs, long long slab_stride, int P, void* out, int T, int R, void* stream, int pdl) {
+  if (T <= 0) return 0;
+  if (R <= 0 || !slabs) return -1;
   const long long total = (long long)T * R;
-  const dim3 grid((unsigned)((total + 255) / 256));
-  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return f32 ? (int)prism_launch(tanh_split_kernel<float>, grid, dim3(256), 0, s, pdl != 0, proj_of<float>(slabs, slab_stride, P, rows, ld), (float*)out, R, total)
-             : (int)prism_launch(tanh_split_kernel<bf16>, grid, dim3(256), 0, s, pdl != 0, proj_of<bf16>(slabs, slab_stride, P, rows, ld), (bf16*)out, R, total);
+  return (int)prism_launch(tanh_f32_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream),
+                           pdl != 0, proj_of<float>(slabs, slab_stride, P, nullptr, R), (float*)out, R, total);
 }
 
 // One token per sequence (token s belongs to sequence s).  p: r, k, v, gate of all tokens one after another, fp32 slabs or

@@ -41,7 +41,8 @@ _SIGNATURES = {
     "prism_window_prefill_tc": "ppppppppl" "iiiiiiiiiiiiiii" "fffffpi",
     "prism_window_attention_simple": "ippppppppl" "iiiiiiiiiiiiii" "fffffpi",
     "prism_token_mix": "ipliipppp" "iippippi" "pi",
-    "prism_tanh_split": "iplipl" "piipi",
+    "prism_decay_project": "plil" "ppp" "iiipi",
+    "prism_tanh_f32": "plip" "iipi",
     "prism_state_step": "ipliippp" "ii" "plipl" "plipl" "ppppp" "iiii" "fpi",
     "prism_state_scan": "ipliipppp" "ii" "plipl" "ppp" "iiipi",
     "prism_head_norm_gate": "ip" "plipl" "pp" "iiii" "fpi",

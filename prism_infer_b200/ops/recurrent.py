@@ -79,18 +79,13 @@ class TimeMixWeights:
     mu: torch.Tensor         # [5, W] blends of r, k, v, gate, decay
     rkvg: torch.Tensor       # [4, H n, W]
     w1: torch.Tensor         # [rank, W]
-    w2: torch.Tensor         # [H n, 2 rank]: the second projection twice, for the two parts of its input
+    w2: torch.Tensor         # [H n, rank]
     w0: torch.Tensor         # [H n]
     u: torch.Tensor          # [H n]
     norm: torch.Tensor       # [H n]
 
     def __post_init__(self) -> None:
-        self.w2_once = self.w2[:, :self.w2.shape[1] // 2].contiguous()
         self._decay = Sections([(self.w2.shape[0], 1.0, "decay")])
-
-    def refresh(self) -> None:
-        """After loading: what is derived from the loaded tensors."""
-        self.w2_once.copy_(self.w2[:, :self.w2.shape[1] // 2])
 
 
 @dataclass
@@ -129,7 +124,7 @@ def _time_mix_cpu(x: torch.Tensor, spec: TimeMixSpec, w: TimeMixWeights, st: Sta
         mixed = [(h + (prev - h) * w.mu[m].float()).to(dtype) for m in range(5)]
         r, k, v, g = (F.linear(mixed[m].float(), w.rkvg[m].float()).view(-1, H, n) for m in range(4))
         t = torch.tanh(F.linear(mixed[4].float(), w.w1.float()))
-        d = torch.exp(-torch.exp(F.linear(t, w.w2_once.float()) + w.w0.float())).view(-1, H, n)
+        d = torch.exp(-torch.exp(F.linear(t, w.w2.float()) + w.w0.float())).view(-1, H, n)
         u = w.u.float().view(H, n)
         S = old[:spec.carry].view(H, n, n)
         o = torch.empty_like(r)
@@ -189,6 +184,19 @@ def wide_projections(mixed: torch.Tensor, w: torch.Tensor, table: tuple) -> Bran
     return Branch(rows=y)
 
 
+def decays(z: torch.Tensor, w: TimeMixWeights) -> torch.Tensor:
+    """``exp(-exp(w0 + W2 tanh(z)))`` in 32-bit, ``[T, H n]``, of the narrow projection's slabs ``z [S, T, rank]``."""
+    _, T, R = z.shape
+    C = w.w2.shape[0]
+    if w.w2.dtype == torch.float32:
+        t = torch.empty((T, R), dtype=torch.float32, device=z.device)
+        native.call("prism_tanh_f32", _p(z), z.stride(0), z.shape[0], _p(t), T, R, _s(), _pdl())
+        return linear_sections(t, w.w2, w._decay, bias=w.w0, out_f32=True)
+    d = torch.empty((T, C), dtype=torch.float32, device=z.device)
+    native.call("prism_decay_project", _p(z), z.stride(0), z.shape[0], z.stride(1), _p(w.w2), _p(w.w0), _p(d), T, C, R, _s(), _pdl())
+    return d
+
+
 def time_mix(x: torch.Tensor, spec: TimeMixSpec, w: TimeMixWeights, st: StateView) -> torch.Tensor:
     """The mixer up to its output projection for the step's rows ``x [T, W]`` (fp32): ``[T, H n]``, with the state taken from and
     put back into the sequences' slots.  Rows of sequences without a slot are zero."""
@@ -205,11 +213,9 @@ def time_mix(x: torch.Tensor, spec: TimeMixSpec, w: TimeMixWeights, st: StateVie
     out = torch.empty((T, spec.cols), dtype=dtype, device=dev)
     if st.cu_seqlens_q is None:
         native.call("prism_state_step", f32, *st.args(spec, cu=False), _p(x), S, spec.width, *_proj_args(p), *_proj_args(Branch(slabs=z1)),
-                    _p(w.w2_once), _p(w.w0), _p(w.u), _p(w.norm), _p(out), spec.heads, spec.n, spec.dim, spec.rank, float(spec.eps), _s(), _pdl())
+                    _p(w.w2), _p(w.w0), _p(w.u), _p(w.norm), _p(out), spec.heads, spec.n, spec.dim, spec.rank, float(spec.eps), _s(), _pdl())
         return out
-    t = torch.empty((T, 2 * spec.rank), dtype=dtype, device=dev)
-    native.call("prism_tanh_split", f32, *_proj_args(Branch(slabs=z1)), _p(t), T, spec.rank, _s(), _pdl())
-    d = linear_sections(t, w.w2, w._decay, bias=w.w0, out_f32=True)
+    d = decays(z1, w)
     o = torch.empty((T, spec.cols), dtype=torch.float32, device=dev)
     native.call("prism_state_scan", f32, *st.args(spec), _p(x), S, spec.width, *_proj_args(p), _p(d), _p(w.u), _p(o), T, spec.heads, spec.n,
                 _s(), _pdl())

@@ -42,17 +42,15 @@ class Mixer:
         def z(*shape):
             return torch.zeros(shape, dtype=dtype, device=device)
 
-        m = rec.TimeMixWeights(z(5, s.width), z(4, s.cols, s.width), z(s.rank, s.width), z(s.cols, 2 * s.rank), z(s.cols), z(s.cols), z(s.cols))
+        m = rec.TimeMixWeights(z(5, s.width), z(4, s.cols, s.width), z(s.rank, s.width), z(s.cols, s.rank), z(s.cols), z(s.cols), z(s.cols))
         for i, n in enumerate("rkvgw"):
             m.mu[i, :W] = p["mu." + n].to(device, dtype)
         for i, n in enumerate("rkvg"):
             m.rkvg[i].view(H, s.n, s.width)[:, :d, :W] = p[n].view(H, d, W).to(device, dtype)
         m.w1[:R, :W] = p["w1"].to(device, dtype)
-        for first in (0, s.rank):
-            m.w2.view(H, s.n, -1)[:, :d, first:first + R] = p["w2"].view(H, d, R).to(device, dtype)
+        m.w2.view(H, s.n, -1)[:, :d, :R] = p["w2"].view(H, d, R).to(device, dtype)
         for n in ("w0", "u", "norm"):
             getattr(m, n).view(H, s.n)[:, :d] = p[n].reshape(H, d).to(device, dtype)
-        m.refresh()
         self.packed = m
         self.cache = rec.StateCache([8, s.carry + s.width], slots, device)
         for i in range(2):
@@ -192,6 +190,23 @@ def test_a_far_token_is_remembered(backend, decode):
     y = x.clone()
     y[20] = x[21]
     assert float((m.want(y)[400] - want[400]).abs().max()) > 0.2 * float(want[400].abs().max())
+
+
+@pytest.mark.parametrize("backend", [GPU32, GPU16])
+@pytest.mark.parametrize("T,C,R,S", [(1, 16, 16, 1), (70, 144, 48, 3), (129, 256, 64, 2), (64, 128, 128, 1), (600, 400, 208, 2)])
+def test_decays(backend, T, C, R, S):
+    """From rates that forget at once to rates that forget nothing in thousands of tokens; close to 32-bit in both types."""
+    device, dtype = backend
+    z, w2, w0 = rand(S, T, R, seed=1, scale=1.0), rand(C, R, seed=2, scale=2 * R ** -0.5), torch.linspace(-9.0, 3.0, C).to(torch.bfloat16).float()
+    w = rec.TimeMixWeights(*(torch.zeros(1),) * 3, w2.to(device, dtype), w0.to(device, dtype), *(torch.zeros(1),) * 2)
+    got = rec.decays(z.to(device), w).double().cpu()
+    rate = torch.exp(torch.tanh(z.double().sum(0)) @ w2.double().T + w0.double())
+    assert float((got - torch.exp(-rate)).abs().max()) < (2e-6 if dtype == torch.float32 else 1e-4)
+    slow = rate < 0.1
+    assert float(((-torch.log(got) - rate).abs() / rate)[slow & (rate > 1e-2)].max()) < (1e-4 if dtype == torch.float32 else 1e-3)
+    from prism_infer_b200.ops import native
+
+    native.check_status()
 
 
 @pytest.mark.parametrize("backend", [GPU32, GPU16])

@@ -350,3 +350,20 @@ def test_own_row_and_scaled_embedding(backend, width, T):
     lat.stream_update(x, width, 1e-5, keep=False, ids=ids.to(device), table=table.to(device, dtype), embed_mult=2.7, raw_out=raw)
     close(x, table[ids].double() * 2.7, torch.float32, tol32=1e-6)
     close(raw, table[ids].double() * 2.7, dtype)
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+@pytest.mark.parametrize("T", [3, 140, 600])
+@pytest.mark.parametrize("M,K", [(272, 96), (1024, 64), (97, 80)])
+def test_scaled_and_decay_sections_in_32_bit(backend, T, M, K):
+    """Sections of a stacked projection with fp32 output: a scale (logits), and decays; few tokens, and enough for the persistent form."""
+    device, dtype = backend
+    x, w, bias = rand(T, K, seed=1), rand(M, K, seed=2, scale=K ** -0.5), rand(M, seed=3)
+    y = x.double() @ w.double().T
+    args = x.to(device, dtype), w.to(device, dtype)
+    got = lat.linear_sections(*args, lat.Sections([(M, 2.5, None)]), out_f32=True)
+    close(got, y * 2.5, dtype, tol16=1e-5)
+    first = M // 2 // 16 * 16
+    got = lat.linear_sections(*args, lat.Sections([(first, 1.0, "decay"), (M - first, -0.5, None)]), bias=bias.to(device, dtype), out_f32=True)
+    close(got[:, :first], torch.exp(-torch.exp(y[:, :first] + bias[:first].double())), dtype, tol16=1e-5)
+    close(got[:, first:], -0.5 * y[:, first:] + bias[first:].double(), dtype, tol16=1e-5)
