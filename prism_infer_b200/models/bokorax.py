@@ -97,16 +97,12 @@ class BokoraxModel(WindowedDecoder):
         return True
 
     # ---------------------------------------------------------------------- text
-    def _reads_stream(self, layer: int) -> Optional[bool]:
-        """Whether layer ``layer``'s mixer reads the stream itself (recurrent) rather than its copy; None behind the last."""
-        return self.arch.layers[layer].recurrent if layer < len(self.weights) else None
-
     def _hand_on(self, st: LayerLoopState, layer: int) -> dict:
-        """What an update writes for the mixer of ``layer``, or for the head behind the last one."""
-        reads = self._reads_stream(layer)
-        if reads is None:
+        """What an update writes for the mixer of ``layer`` (a recurrent one reads the stream itself), or for the head behind the
+        last one."""
+        if layer == len(self.weights):
             return {"norm_weight": self.final_norm, "norm_out": st.n}
-        return {} if reads else {"raw_out": st.raw}
+        return {} if self.weights[layer].mix is not None else {"raw_out": st.raw}
 
     def _embed(self, st: LayerLoopState) -> None:
         self._update(st, keep=False, ids=st.ids, table=self.embed, embed_mult=self.arch.embed_scale, **self._hand_on(st, 0))

@@ -1,8 +1,6 @@
 """Plain, slow statement of the Bokorax design in float64, one function per mechanism.  Works on a whole sequence at
 once, no cache, no padding, one query or token at a time; shares no code with the package."""
 
-import math
-
 import torch
 
 

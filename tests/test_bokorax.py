@@ -193,6 +193,30 @@ def test_block_manager_hands_out_state_slots():
         bm.state.release(0)
 
 
+@pytest.mark.parametrize("backend", BACKENDS)
+def test_page_and_state_traffic_runs_in_the_order_it_is_planned(model, backend):
+    """A plan may read a CPU page (a state slot) for one sequence and hand it to another, and overwrite a device page that it has
+    just swapped out."""
+    from prism_infer_b200.engine.contracts import KVTransferPlan
+
+    llm = cases.engine(model("plain")[3], backend, cpu_kv_cache_ratio=0.5)
+    r = llm.runners.runner
+    for l in range(2):
+        for cache, base in ((r.kv, 100.0), (r.cpu_kv, 500.0)):
+            rows = cache.token_rows(l)
+            rows.copy_((base + torch.arange(float(rows.shape[0])))[:, None, None].expand(rows.shape))
+        for state, base in ((r.state, 1.0), (r.cpu_state, 50.0)):
+            t = state.layer(l)
+            t.copy_((base + torch.arange(float(t.shape[0])))[:, None, None].expand(t.shape))
+    r.apply_kv_transfers(KVTransferPlan(swap_in=((0, 3),), swap_out=((5, 0),), copy_on_write=((2, 5),), state_in=((1, 0),), state_out=((2, 1),)))
+    r.barrier()
+    for l in range(2):
+        kv, cpu, st, cst = r.kv.token_rows(l), r.cpu_kv.token_rows(l), r.state.layer(l), r.cpu_state.layer(l)
+        assert [float(kv[i].float().mean()) for i in (3, 5, 2)] == [500.0, 102.0, 102.0] and float(cpu[0].float().mean()) == 105.0
+        assert [float(st[i].mean()) for i in (0, 2)] == [51.0, 3.0] and float(cst[1].mean()) == 3.0
+    llm.exit()
+
+
 # ----------------------------------------------------------------------------------------- whole forward
 @pytest.mark.parametrize("backend", BACKENDS)
 @pytest.mark.parametrize("name", list(cases.CASES))
