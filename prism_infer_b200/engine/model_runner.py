@@ -264,7 +264,8 @@ class ModelRunner:
         meta = AttnMeta(is_prefill=True, block_tables=bt, slots=slots,
                         cu_seqlens_q=torch.tensor([0, tokens], dtype=torch.int32, device=dev),
                         kv_lens=torch.tensor([tokens], dtype=torch.int32, device=dev), max_q_len=tokens, no_history=True,
-                        total_kv=tokens, max_kv_len=tokens, attended_pairs=tokens * tokens, **self._state_meta([0]))
+                        total_kv=tokens, max_kv_len=tokens, attended_pairs=tokens * tokens, host_lens=[(tokens, tokens)],
+                        **self._state_meta([0]))
         hidden = self.model.forward(ids, pos, meta, scratch)
         self.model.sample(hidden[-1:], None)
         torch.cuda.synchronize(dev)
@@ -554,6 +555,7 @@ class ModelRunner:
                 cu_seqlens_q=self._to_dev(inp.cu_seqlens_q), kv_lens=self._to_dev(inp.kv_lens), max_q_len=inp.max_q_len,
                 no_history=bool(torch.equal(inp.kv_lens, inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1])),
                 total_kv=int(inp.kv_lens.sum()), max_kv_len=int(inp.kv_lens.max()),
+                host_lens=list(zip((inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1]).tolist(), inp.kv_lens.tolist())),
                 attended_pairs=int(((inp.cu_seqlens_q[1:] - inp.cu_seqlens_q[:-1]).long() * inp.kv_lens.long()).sum()),
                 **self._state_meta(inp.state_slots))
             if not meta.no_history:  # key ranges for the gather + tensor-core attention over the paged cache

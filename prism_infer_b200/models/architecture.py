@@ -6,8 +6,9 @@ dataclasses below once and every later layer (weight sharding, kernels, KV sizin
 reads these.  Mirrors the contract of the reference's
 ``prism_infer/models/qwen3_vl_architecture.py:117-428`` (canonical 8B constants at
 ``:18-44``): interleaved M-RoPE only, no attention bias, SiLU text MLP, GELU-tanh
-vision MLP.  ``PoralornArch``, ``DolidraArch`` and ``BokoraxArch`` (end of file) are text-only families: latent attention,
-windowed attention with a mixture of experts, and recurrent layers between attention layers.
+vision MLP.  ``PoralornArch``, ``DolidraArch``, ``BokoraxArch`` and ``FosulixArch`` (end of file) are text-only families: latent
+attention, windowed attention with a mixture of experts, recurrent layers between attention layers, and gated linear attention
+between windowed latent attention under a depth average.
 
 What the engine asks of any architecture, whatever its family: ``model_type``, ``multimodal``,
 ``vocab_size``, ``max_positions`` (``None``: unbounded), ``num_layer_runs``, ``eos_token_id``, the
@@ -466,22 +467,58 @@ def _loop_fields(cfg: Mapping[str, Any], need) -> dict[str, int]:
     return {f"loop_{k}": int(need(loop, k, "loop")) if loop else 0 for k in ("start", "stop", "times")}
 
 
+NO_WINDOW = 1 << 30              # a window that no sequence outgrows
+
+
 # ------------------------------------------------------------------------------- Poralorn
 @dataclass(frozen=True)
 class LatentAttentionArch:
     """Sizes of one latent-attention mixer: ``heads`` heads whose ``dim``-wide keys and ``vdim``-wide values
-    are linear in one shared ``kv_rank``-wide latent per token (the only thing cached)."""
+    are linear in one shared ``kv_rank``-wide latent per token (the only thing cached).  ``q_rank``: the queries go through a
+    normalised latent of their own (0: straight from the input); ``rot_dim`` more columns of every query, and of one key part
+    all heads share (cached beside the latent), are rotated as ``rot`` says; a query sees the ``window`` newest positions;
+    ``kv_from``: the layer whose cached rows it reads instead of its own (-1: none)."""
 
     heads: int
     dim: int
     vdim: int
     kv_rank: int
     scale: float
+    q_rank: int = 0
+    rot_dim: int = 0
+    rot: RotaryArch | None = None
+    window: int = NO_WINDOW
+    kv_from: int = -1
 
     def __post_init__(self) -> None:
-        for name in ("heads", "dim", "vdim", "kv_rank"):
+        for name in ("heads", "dim", "vdim", "kv_rank", "window"):
             if getattr(self, name) < 1:
                 raise ValueError(f"latent attention: {name} must be positive")
+        if self.q_rank < 0 or self.rot_dim < 0 or self.rot_dim != (self.rot.dims if self.rot is not None else 0):
+            raise ValueError("latent attention: q_rank must not be negative, rot.dims is rot_dim")
+
+    @property
+    def rot_start(self) -> int:
+        """Column of a query or key head at which its rotated part starts; ``dq`` the whole head, padded, ``dv`` a value head."""
+        return -(-self.dim // 8) * 8
+
+    @property
+    def dq(self) -> int:
+        return -(-(self.rot_start + self.rot_dim) // 16) * 16
+
+    @property
+    def dv(self) -> int:
+        return -(-self.vdim // 16) * 16
+
+    @property
+    def row_rot_start(self) -> int:
+        """Column of a cached row at which the rotated key part starts."""
+        return -(-self.kv_rank // 16) * 16
+
+    @property
+    def cache_row(self) -> int:
+        """Elements of a cached row, latent and rotated key part, in whole 64-element tiles."""
+        return -(-(self.row_rot_start + self.rot_dim) // 64) * 64
 
 
 @dataclass(frozen=True)
@@ -583,7 +620,8 @@ class PoralornArch(LoopedStack):
         out: dict[str, Any] = {"architecture": "Poralorn", "vocab": self.vocab_size, "width": self.width,
                                "norm": {"eps": self.norm_eps}, "residual_mult": self.residual_mult,
                                "logit_softcap": self.logit_softcap,
-                               "layers": [{"type": "latent_attention", "mixer": asdict(l.mixer),
+                               "layers": [{"type": "latent_attention",
+                                           "mixer": {k: getattr(l.mixer, k) for k in ("heads", "dim", "vdim", "kv_rank", "scale")},
                                            "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None} for l in self.layers]}
         if self.has_loop:
             out["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
@@ -608,9 +646,10 @@ class PoralornArch(LoopedStack):
 # -------------------------------------------------------------------------------- Dolidra
 @dataclass(frozen=True)
 class RotaryArch:
-    """Rotation of the first ``dims`` columns of a head (pairs ``(i, i + dims / 2)``).  ``factor`` > 0 rescales the
-    frequencies by wavelength: long ones are divided by it, those below ``original / high`` stay, a ramp between; without
-    ``original`` all of them are divided."""
+    """Rotation of the first ``dims`` columns of a head (pairs ``(i, i + dims / 2)``, or neighbours where the mixer says so).
+    ``factor`` > 0 rescales the frequencies by wavelength: long ones are divided by it, those below ``original / high`` stay, a
+    ramp between; without ``original`` all of them are divided.  With ``fast`` and ``slow`` (turns over ``original`` positions)
+    the ramp is over the pairs' numbers instead (YaRN), and sines and cosines are scaled by ``amplitude``."""
 
     base: float
     dims: int
@@ -618,12 +657,35 @@ class RotaryArch:
     low: float = 0.0
     high: float = 0.0
     original: float = 0.0
+    fast: float = 0.0
+    slow: float = 0.0
 
     def __post_init__(self) -> None:
         if self.dims < 0 or self.dims % 2:
             raise ValueError(f"rotary dims must be even, got {self.dims}")
+        if self.fast > 0.0 and not (self.slow > 0.0 and self.factor > 0.0 and self.original > 0.0 and self.base > 1.0):
+            raise ValueError("rotary scaling by turns needs factor, original, fast and slow, and a base above one")
+
+    @property
+    def amplitude(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0 if self.fast > 0.0 else 1.0
+
+    def _by_turns(self) -> list[float]:
+        """The frequencies with those of slow pairs divided by ``factor``, a ramp over the pairs' numbers between."""
+
+        def pair(turns: float) -> float:
+            return self.dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+
+        lo, hi = max(math.floor(pair(self.fast)), 0), min(math.ceil(pair(self.slow)), self.dims - 1)
+        out = []
+        for i in range(self.dims // 2):
+            f, ramp = self.base ** (-2.0 * i / self.dims), min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            out.append(f / self.factor * ramp + f * (1.0 - ramp))
+        return out
 
     def inv_freq(self) -> list[float]:
+        if self.fast > 0.0:
+            return self._by_turns()
         out = []
         for i in range(self.dims // 2):
             f = self.base ** (-2.0 * i / self.dims)
@@ -638,9 +700,6 @@ class RotaryArch:
                     f = (1.0 - keep) * f / self.factor + keep * f
             out.append(f)
         return out
-
-
-NO_WINDOW = 1 << 30              # a window that no sequence outgrows
 
 
 @dataclass(frozen=True)
@@ -705,7 +764,9 @@ class MixtureArch:
     ``shared_ff`` (0: none) for every token, times a sigmoid per token with ``shared_gate``.  The weights are the softmax over
     the chosen logits, or (``scored``) the chosen scores of a softmax over all, divided by their sum and times ``scale``; then
     a learned correction enters the choice only, ``identity`` more router outputs stand for the input itself, and the
-    choice is among the ``groups_kept`` best of ``groups`` equal groups of neighbours."""
+    choice is among the ``groups_kept`` best of ``groups`` equal groups of neighbours.  ``sigmoid``: the scores are the outputs'
+    own sigmoids instead, not corrected and not divided by their sum, and a group is as good as the sum of its two best.
+    ``limit``: the experts' gates and inputs are bounded (``act(min(g, limit)) * (1 + clamp(u, -limit, limit))``); 0: SiLU."""
 
     experts: int
     top: int
@@ -717,6 +778,8 @@ class MixtureArch:
     groups_kept: int = 1
     scale: float = 1.0
     shared_gate: bool = False
+    sigmoid: bool = False
+    limit: float = 0.0
 
     @property
     def outputs(self) -> int:
@@ -730,6 +793,8 @@ class MixtureArch:
             raise ValueError(f"mixture of experts: {self.top} of {self.outputs} in {self.groups_kept} of {self.groups} groups")
         if not self.scored and (self.identity or self.groups > 1 or self.scale != 1.0):
             raise ValueError("mixture of experts: identity experts, groups and a scale belong to scored routing")
+        if (self.sigmoid and not self.scored) or self.limit < 0.0:
+            raise ValueError("mixture of experts: sigmoid scores belong to scored routing, a limit must not be negative")
 
 
 @dataclass(frozen=True)
@@ -1151,3 +1216,235 @@ class BokoraxArch(LoopedStack):
                           shared_gate=True)
         kinds = [(wkv, sink, tied, replace(sink, kv_from=i - 2))[i % 4] for i in range(layers)]
         return cls(vocab_size=vocab_size, width=width, layers=tuple(BokoraxLayer(m, moe) for m in kinds), embed_scale=8.0)
+
+
+# -------------------------------------------------------------------------------- Fosulix
+@dataclass(frozen=True)
+class ForgetMixArch:
+    """A recurrent mixer with a state per head (``dim`` x ``vdim``) whose forget gate per key channel also weighs what is
+    written; a learned bound keeps the gate from below."""
+
+    heads: int
+    dim: int
+    vdim: int
+
+    def __post_init__(self) -> None:
+        if self.heads < 1 or self.dim < 1 or self.vdim < 1:
+            raise ValueError(f"gated linear attention: {self.heads} heads of {self.dim} x {self.vdim}")
+
+    @property
+    def n(self) -> int:
+        """Key channels padded to whole tensor-core steps, ``m`` the value channels."""
+        return -(-self.dim // 16) * 16
+
+    @property
+    def m(self) -> int:
+        return -(-self.vdim // 16) * 16
+
+    @property
+    def state_size(self) -> int:
+        return self.heads * self.n * self.m
+
+
+@dataclass(frozen=True)
+class FosulixLayer:
+    mixer: LatentAttentionArch | ForgetMixArch
+    moe: MixtureArch | None = None
+
+    @property
+    def recurrent(self) -> bool:
+        return isinstance(self.mixer, ForgetMixArch)
+
+    @property
+    def owns_cache(self) -> bool:
+        return not self.recurrent and self.mixer.kv_from < 0
+
+
+@dataclass(frozen=True)
+class FosulixArch(LoopedStack):
+    vocab_size: int
+    width: int
+    layers: tuple[FosulixLayer, ...]
+    taps: int                        # rows an input convolution sums, the token's own among them
+    embed_scale: float = 1.0
+    residual_mult: float = 1.0
+    norm_eps: float = 1.0e-6
+    eos_token_id: int = -1
+    model_type: str = "fosulix"
+
+    loop_start = loop_stop = loop_times = 0   # every layer runs once
+    tied_head = True
+
+    def __post_init__(self) -> None:
+        self.check_stack()
+        if self.taps < 1:
+            raise ValueError("canon.taps must be positive")
+        for i, l in enumerate(self.layers):
+            if l.recurrent or l.owns_cache:
+                continue
+            m, j = l.mixer, l.mixer.kv_from
+            owner = self.layers[j] if j < i else None
+            if owner is None or not owner.owns_cache:
+                raise ValueError(f"Fosulix layer {i}: kv_from {j} does not name an earlier layer with latents of its own")
+            if (m.kv_rank, m.rot_dim, m.rot) != (owner.mixer.kv_rank, owner.mixer.rot_dim, owner.mixer.rot):
+                raise ValueError(f"Fosulix layer {i}: latents of layer {j} have other sizes or another rotation")
+
+    def cache_slab(self, layer: int) -> int:
+        """Cache slab a layer's attention reads (-1: a recurrent layer)."""
+        l = self.layers[layer]
+        if l.recurrent:
+            return -1
+        owner = layer if l.owns_cache else l.mixer.kv_from
+        return sum(o.owns_cache for o in self.layers[:owner])
+
+    def kv_geometry(self, tp: int = 1) -> KVGeometry:
+        rows = tuple(l.mixer.cache_row for l in self.layers if l.owns_cache) or (64,)   # pages count tokens even without keys
+        return KVGeometry(1, len(rows), 1, max(rows), rows)
+
+    @property
+    def carry_size(self) -> int:
+        """fp32 elements of the rows an input convolution carries on."""
+        return (self.taps - 1) * (-(-self.width // 16) * 16)
+
+    def carry_start(self, layer: int) -> int:
+        """Where they start in the layer's state row, behind the recurrent state."""
+        return self.layers[layer].mixer.state_size if self.layers[layer].recurrent else 0
+
+    def state_sizes(self) -> tuple[int, ...]:
+        return tuple(max(4, self.carry_start(i) + self.carry_size) for i in range(len(self.layers)))
+
+    # ---- checkpoint --------------------------------------------------------------
+    def weight_shapes(self) -> dict[str, tuple[int, ...]]:
+        W = self.width
+        s: dict[str, tuple[int, ...]] = {"embed": (self.vocab_size, W)}
+        for i, l in enumerate(self.layers):
+            m, p = l.mixer, f"l{i}"
+            s[f"{p}.norm1"] = (W,)
+            if l.recurrent:
+                n = m.heads * m.dim
+                s[f"{p}.mix.q"] = s[f"{p}.mix.f"] = (n, W)
+                s[f"{p}.mix.f.b"] = s[f"{p}.mix.lower"] = (n,)
+                s[f"{p}.mix.v"], s[f"{p}.mix.norm"] = (m.heads * m.vdim, W), (m.vdim,)
+            else:
+                s[f"{p}.mix.dq"], s[f"{p}.mix.dq.norm"] = (m.q_rank, W), (m.q_rank,)
+                s[f"{p}.mix.uq"] = (m.heads * (m.dim + m.rot_dim), m.q_rank)
+                if m.kv_from < 0:
+                    s[f"{p}.mix.dkv"], s[f"{p}.mix.dkv.norm"] = (m.kv_rank + m.rot_dim, W), (m.kv_rank,)
+                s[f"{p}.mix.uk"], s[f"{p}.mix.uv"] = (m.heads * m.dim, m.kv_rank), (m.heads * m.vdim, m.kv_rank)
+            s[f"{p}.mix.o"] = (W, m.heads * m.vdim)
+            if l.moe is not None:
+                s[f"{p}.norm2"] = (W,)
+                for e in range(l.moe.experts):
+                    s[f"{p}.mlp.e{e}.gate"] = s[f"{p}.mlp.e{e}.up"] = (l.moe.ff, W)
+                    s[f"{p}.mlp.e{e}.down"] = (W, l.moe.ff)
+                s[f"{p}.mlp.router"] = (l.moe.experts, W)
+            s[f"{p}.canon1"], s[f"{p}.dwa"] = (W, self.taps), (i + 2,)
+        s["final.norm"] = (W,)
+        return s
+
+    @staticmethod
+    def init_kind(name: str) -> str:
+        """How random initialisation draws a tensor: ``norm``, ``bias``, ``embedding`` or ``matrix``."""
+        last = name.rsplit(".", 1)[-1]
+        if last in ("norm", "norm1", "norm2", "dwa"):
+            return "norm"
+        if last in ("b", "lower", "canon1"):
+            return "bias"
+        return "embedding" if name == "embed" else "matrix"
+
+    # ---- factories ---------------------------------------------------------------
+    @classmethod
+    def from_hf_config(cls, cfg: Mapping[str, Any]) -> "FosulixArch":
+        """From the ``config.json`` dictionary."""
+        need = _field_reader("Fosulix")
+
+        def attention(m: Mapping[str, Any], where: str) -> LatentAttentionArch:
+            rot, mask = need(m, "rot", where), m.get("mask") or {}
+            scaling = rot.get("scaling") or {}
+            return LatentAttentionArch(
+                *(int(need(m, k, where)) for k in ("heads", "dim", "vdim", "kv_rank")), float(need(m, "scale", where)),
+                q_rank=int(need(m, "q_rank", where)), rot_dim=int(need(m, "rot_dim", where)),
+                rot=RotaryArch(float(need(rot, "base", where)), int(need(rot, "dims", where)),
+                               **{k: float(need(scaling, k, where)) for k in ("factor", "original", "fast", "slow") if scaling}),
+                window=int(need(mask, "size", where)) if mask else NO_WINDOW, kv_from=-1 if m.get("kv_from") is None else int(m["kv_from"]))
+
+        layers = []
+        for i, entry in enumerate(need(cfg, "layers")):
+            where = f"layer {i}"
+            kind, m = need(entry, "type", where), need(entry, "mixer", where)
+            if kind == "latent_attention":
+                mixer = attention(m, where)
+                if mixer.q_rank < 1:
+                    raise ValueError(f"Fosulix {where}: q_rank must be positive")
+            elif kind == "hgrn2":
+                mixer = ForgetMixArch(*(int(need(m, k, where)) for k in ("heads", "dim", "vdim")))
+            else:
+                raise ValueError(f"Fosulix {where}: unsupported mixer {kind!r}")
+            mlp = entry.get("mlp")
+            if mlp is None:
+                layers.append(FosulixLayer(mixer))
+                continue
+            if mlp.get("kind") != "moe":
+                raise ValueError(f"Fosulix {where}: unsupported feed-forward {mlp.get('kind')!r}")
+            router, expert = need(mlp, "router", where), need(mlp, "expert", where)
+            groups = router.get("groups") or {"count": 1, "keep": 1}
+            moe = MixtureArch(int(need(router, "experts", where)), int(need(router, "top", where)), int(need(expert, "ff", where)), scored=True,
+                              groups=int(need(groups, "count", where)), groups_kept=int(need(groups, "keep", where)),
+                              scale=float(router.get("scale", 1.0)), sigmoid=True, limit=float(need(expert, "limit", where)))
+            if moe.limit <= 0.0:
+                raise ValueError(f"Fosulix {where}: the experts' limit must be positive")
+            layers.append(FosulixLayer(mixer, moe))
+        return cls(vocab_size=int(need(cfg, "vocab")), width=int(need(cfg, "width")), layers=tuple(layers),
+                   taps=int(need(need(cfg, "canon"), "taps", "canon")), embed_scale=float(need(need(cfg, "embedding"), "scale", "embedding")),
+                   residual_mult=float(need(cfg, "residual_mult")), norm_eps=float(need(need(cfg, "norm"), "eps", "norm")))
+
+    def to_hf_config(self) -> dict[str, Any]:
+        """The ``config.json`` dictionary ``from_hf_config`` reads."""
+
+        def layer(l: FosulixLayer) -> dict[str, Any]:
+            m = l.mixer
+            mixer: dict[str, Any] = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+            if not l.recurrent:
+                rot: dict[str, Any] = {"base": m.rot.base, "dims": m.rot.dims}
+                if m.rot.fast > 0.0:
+                    rot["scaling"] = {k: getattr(m.rot, k) for k in ("factor", "original", "fast", "slow")}
+                mixer |= {"kv_rank": m.kv_rank, "q_rank": m.q_rank, "rot_dim": m.rot_dim, "scale": m.scale, "rot": rot}
+                if m.window != NO_WINDOW:
+                    mixer["mask"] = {"size": m.window}
+                if m.kv_from >= 0:
+                    mixer["kv_from"] = m.kv_from
+            mlp: dict[str, Any] | None = None
+            if l.moe is not None:
+                mlp = {"kind": "moe", "expert": {"ff": l.moe.ff, "limit": l.moe.limit},
+                       "router": {"experts": l.moe.experts, "top": l.moe.top, "scale": l.moe.scale,
+                                  "groups": {"count": l.moe.groups, "keep": l.moe.groups_kept}}}
+            return {"type": "hgrn2" if l.recurrent else "latent_attention", "mixer": mixer, "mlp": mlp}
+
+        return {"architecture": "Fosulix", "vocab": self.vocab_size, "width": self.width, "norm": {"eps": self.norm_eps},
+                "canon": {"taps": self.taps}, "embedding": {"scale": self.embed_scale}, "residual_mult": self.residual_mult,
+                "layers": [layer(l) for l in self.layers]}
+
+    @classmethod
+    def tiny(cls) -> "FosulixArch":
+        """The small CPU test model: every size different, both mixers, a layer that reads another's latents."""
+        forget = ForgetMixArch(3, 24, 40)
+        rot = RotaryArch(7000.0, 12, factor=3.0, original=96.0, fast=8.0, slow=1.0)
+        latent = LatentAttentionArch(5, 20, 28, 72, 0.2, q_rank=56, rot_dim=12, rot=rot, window=23)
+        moe = MixtureArch(8, 2, 40, scored=True, groups=4, groups_kept=2, scale=1.5, sigmoid=True, limit=3.0)
+        return cls(vocab_size=300, width=112, layers=(FosulixLayer(latent, moe), FosulixLayer(forget, moe), FosulixLayer(forget),
+                                                      FosulixLayer(replace(latent, window=9, kv_from=0), moe)),
+                   taps=3, embed_scale=4.0, residual_mult=0.6)
+
+    @classmethod
+    def like_8b(cls, layers: int = 4, *, width: int = 4096, heads: int = 32, dim: int = 128, rot_dim: int = 64, q_rank: int = 1536,
+                kv_rank: int = 512, state_dim: int = 128, window: int = 1024, experts: int = 32, top: int = 4, expert_ff: int = 1536,
+                vocab_size: int = 151_936) -> "FosulixArch":
+        """Layers with the widths of an 8B-class decoder (measurement model; random weights): recurrent, latent, latent with the
+        one before it's latents, recurrent, in turn."""
+        forget = ForgetMixArch(width // state_dim, state_dim, state_dim)
+        rot = RotaryArch(1.0e6, rot_dim, factor=4.0, original=8192.0, fast=32.0, slow=1.0)
+        latent = LatentAttentionArch(heads, dim, dim, kv_rank, (dim + rot_dim) ** -0.5, q_rank=q_rank, rot_dim=rot_dim, rot=rot, window=window)
+        moe = MixtureArch(experts, top, expert_ff, scored=True, groups=8, groups_kept=4, scale=1.0, sigmoid=True, limit=7.0)
+        kinds = [(forget, latent, replace(latent, kv_from=i - 1), forget)[i % 4] for i in range(layers)]
+        return cls(vocab_size=vocab_size, width=width, layers=tuple(FosulixLayer(m, moe) for m in kinds), taps=4, embed_scale=8.0,
+                   residual_mult=0.5)

@@ -3,7 +3,7 @@ of a tensor-parallel rank."""
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Optional
 
 import torch
@@ -39,6 +39,8 @@ class AttnMeta:
     # recurrent layers: the state container and the slot of each sequence (decode: of each row, < 0: padding)
     state: Optional[object] = None                 # ops.recurrent.StateCache
     state_slots: Optional[torch.Tensor] = None     # [S] int32
+    host_lens: Optional[list] = None               # (new tokens, tokens up to the last of them) per sequence, on the host
+    plans: dict = field(default_factory=dict)      # what a step's layers derive from them once
     attended_pairs: int = 0                        # sum over the sequences of query rows x visible keys, known on the host
 
 

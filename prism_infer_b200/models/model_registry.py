@@ -82,6 +82,19 @@ def _bokorax_random() -> dict[str, Callable[[], Any]]:
             "bokorax-8b-like-4layer": BokoraxArch.like_8b}
 
 
+def _fosulix_arch(cfg: Any):
+    from .architecture import FosulixArch
+
+    return FosulixArch.from_hf_config(cfg)
+
+
+def _fosulix_random() -> dict[str, Callable[[], Any]]:
+    from .architecture import FosulixArch
+
+    return {"fosulix-tiny": FosulixArch.tiny, "fosulix-8b-like": lambda: FosulixArch.like_8b(36),
+            "fosulix-8b-like-4layer": FosulixArch.like_8b}
+
+
 _FAMILIES = {
     "qwen3_vl": ModelFamily("qwen3_vl", True, _qwen3_vl_arch, "prism_infer_b200.models.qwen3_vl:Qwen3VLModel", _qwen3_vl_random()),
     "poralorn": ModelFamily("poralorn", False, _poralorn_arch, "prism_infer_b200.models.poralorn:PoralornModel", _poralorn_random(),
@@ -95,6 +108,10 @@ _FAMILIES = {
                            float32_on_cuda=True, kv_modes=(0,),
                            kernel_units=("gemm_tcgen05", "gemm_f32", "window_attention", "recurrence", "moe", "residual_stream", "kv_ops",
                                          "sampler")),
+    "fosulix": ModelFamily("fosulix", False, _fosulix_arch, "prism_infer_b200.models.fosulix:FosulixModel", _fosulix_random(),
+                           float32_on_cuda=True, kv_modes=(0,),
+                           kernel_units=("gemm_tcgen05", "gemm_f32", "latent_attention", "window_attention", "recurrence", "moe",
+                                         "residual_stream", "kv_ops", "sampler")),
 }
 
 

@@ -1,4 +1,4 @@
-"""What the families with windowed attention over single-row caches and routed experts share: padded packed weights of a
+"""What the families with attention over single-row caches and routed experts share: padded packed weights of a
 layer, their loading, the layer loop's skeleton, projections, attention, experts, logits and sampling.
 
 Inner dimensions are zero-padded at load time to multiples of 16; padding stays zero through every operation and norms count
@@ -37,6 +37,7 @@ class LayerWeights:
     always: int = 0                         # experts after the routed ones that every token uses
     experts: int = 0
     scored: Optional[moe.Scored] = None
+    limit: float = 0.0                      # bound of the experts' gated units (0: SiLU units)
 
     def tensors(self) -> Iterator[torch.Tensor]:
         a = self.attn or window.WindowWeights()
@@ -56,6 +57,7 @@ class LayerLoopState:
     n: torch.Tensor                        # [T, W] normalised rows: input of the next projection
     raw: torch.Tensor                      # [T, W] the stream in the compute type
     next_layer: int = 0
+    history: Optional[torch.Tensor] = None # [n, T, W] fp32 results of the layers so far, where a design reads them again
 
 
 class WindowedDecoder:
@@ -74,7 +76,8 @@ class WindowedDecoder:
         self.sampled_logits: Optional[torch.Tensor] = None
         self.keep_logits = False
         self._head_sections = lat.Sections([(arch.vocab_size, getattr(arch, "logit_scale", 1.0), None)])
-        self.embed, self.head, self.final_norm = self._z(arch.vocab_size, self.W), self._z(arch.vocab_size, self.W), self._z(self.W)
+        self.embed, self.final_norm = self._z(arch.vocab_size, self.W), self._z(self.W)
+        self.head = self.embed if getattr(arch, "tied_head", False) else self._z(arch.vocab_size, self.W)
         self._alloc()
 
     # ------------------------------------------------------------------- storage
@@ -101,15 +104,15 @@ class WindowedDecoder:
 
     def _alloc_experts(self, w: LayerWeights, m: MixtureArch) -> None:
         F, E = padded(m.ff), m.experts
-        w.top, w.always, w.experts = m.top, -(-m.shared_ff // F), E
+        w.top, w.always, w.experts, w.limit = m.top, -(-m.shared_ff // F), E, m.limit
         w.gate_up, w.down = self._z(E + w.always, 2 * F, self.W), self._z(E + w.always, self.W, F)
         w.router = self._z(m.outputs + m.shared_gate, self.W)
         if m.scored:
             w.scored = moe.Scored(torch.zeros(m.outputs, dtype=torch.float32, device=self.device), m.identity, m.groups, m.groups_kept, m.scale,
-                                  m.shared_gate)
+                                  m.shared_gate, m.sigmoid, 2 if m.sigmoid else 1)
 
     def weight_bytes(self) -> int:
-        tensors = [self.embed, self.head, self.final_norm] + [t for w in self.weights for t in w.tensors()]
+        tensors = [self.embed, self.final_norm] + ([] if self.head is self.embed else [self.head]) + [t for w in self.weights for t in w.tensors()]
         return sum(t.numel() * t.element_size() for t in tensors)
 
     # ------------------------------------------------------------------- loading
@@ -278,7 +281,7 @@ class WindowedDecoder:
     def _experts(self, st: LayerLoopState, w: LayerWeights, h: torch.Tensor) -> lat.Branch:
         routing = moe.route(lat.Branch(slabs=lat.linear_slabs(h, w.router)), w.top, w.experts, w.always, st.meta.slots,
                             f32=self.dtype == torch.float32, scored=w.scored)
-        return moe.expert_ffn(h, routing, w.gate_up, w.down, "silu")
+        return moe.expert_ffn(h, routing, w.gate_up, w.down, "bounded" if w.limit > 0.0 else "silu", w.limit)
 
     @torch.no_grad()
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:

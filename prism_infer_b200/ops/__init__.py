@@ -151,7 +151,18 @@ def glu_act(z: torch.Tensor, act: str) -> torch.Tensor:
     return F.gelu(z, approximate="tanh") if act == "gelu_tanh" else F.silu(z)
 
 
-GLU_ACTS = {"silu": 1, "gelu_tanh": 2}  # 0: silu with the rounding points of the eager graph (gate_up_swiglu)
+GLU_SLOPE = 1.702   # of the bounded unit's sigmoid
+
+
+def gated_unit(g: torch.Tensor, u: torch.Tensor, act: str, limit: float = 0.0) -> torch.Tensor:
+    """``act(g) * u``; ``bounded``: with ``g`` at most ``limit`` and ``u`` within it, ``g * sigmoid(1.702 g) * (u + 1)``."""
+    if act == "bounded":
+        g = g.clamp(max=limit)
+        return g * torch.sigmoid(GLU_SLOPE * g) * (u.clamp(-limit, limit) + 1.0)
+    return glu_act(g, act) * u
+
+
+GLU_ACTS = {"silu": 1, "gelu_tanh": 2, "bounded": 3}  # 0: silu with the rounding points of the eager graph (gate_up_swiglu)
 
 
 def gate_up_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, *, bn: int = 0) -> torch.Tensor:
@@ -183,6 +194,7 @@ def _gate_up(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int, bn: 
 def gate_up_glu(x: torch.Tensor, w_gate_up: torch.Tensor, act: str) -> torch.Tensor:
     """``act(x @ Wg.T) * (x @ Wu.T)``, activation and product in 32-bit; ``act`` is ``silu`` or ``gelu_tanh``.  bf16 or
     (true 32-bit kernels) fp32."""
+    assert act in ("silu", "gelu_tanh")
     T = x.shape[0]
     I = w_gate_up.shape[0] // 2
     if not x.is_cuda:
@@ -194,7 +206,7 @@ def gate_up_glu(x: torch.Tensor, w_gate_up: torch.Tensor, act: str) -> torch.Ten
         gu = torch.empty((T, 2 * I), dtype=torch.float32, device=x.device)
         native.call("prism_gemm_f32", _p(w_gate_up), _p(x), _p(gu), 2 * I, T, x.shape[1], w_gate_up.stride(0), x.stride(0), 2 * I,
                     None, 0, None, None, None, 0.0, _s(), _pdl())
-        native.call("prism_glu_f32", _p(gu), _p(out), T, I, GLU_ACTS[act], _s(), _pdl())
+        native.call("prism_glu_f32", _p(gu), _p(out), T, I, GLU_ACTS[act], 0.0, _s(), _pdl())
     else:
         _gate_up(x, w_gate_up, out, GLU_ACTS[act])
     return out

@@ -79,8 +79,14 @@ __device__ __forceinline__ float gelu_erf(float x) {
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
 // Gated linear units of the two-matrix GEMM epilogues.  SILU_ROUNDED keeps the rounding points of an eager bf16 graph;
 // the others stay in 32-bit until the product is stored.
-enum PrismGlu : int { PRISM_GLU_SILU_ROUNDED = 0, PRISM_GLU_SILU = 1, PRISM_GLU_GELU_TANH = 2 };
-__device__ __forceinline__ float glu(float g, float u, int act) {
+// BOUNDED: with g at most `limit` and u within it, g sigmoid(1.702 g) (u + 1).
+enum PrismGlu : int { PRISM_GLU_SILU_ROUNDED = 0, PRISM_GLU_SILU = 1, PRISM_GLU_GELU_TANH = 2, PRISM_GLU_BOUNDED = 3 };
+constexpr float PRISM_GLU_SLOPE = 1.702f;
+__device__ __forceinline__ float glu(float g, float u, int act, float limit = 0.0f) {
+  if (act == PRISM_GLU_BOUNDED) {
+    g = fminf(g, limit);
+    return g / (1.0f + __expf(-PRISM_GLU_SLOPE * g)) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+  }
   if (act == PRISM_GLU_SILU_ROUNDED) return bf16_round(silu(bf16_round(g))) * bf16_round(u);
   return (act == PRISM_GLU_GELU_TANH ? gelu_tanh(g) : silu(g)) * u;
 }

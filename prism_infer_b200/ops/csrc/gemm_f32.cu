@@ -92,26 +92,33 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const F32Args a) {
   }
 }
 
-// out[n][i] = act(gu[n][i]) * gu[n][F + i]
-__global__ void __launch_bounds__(256) glu_f32_kernel(const float* gu, float* out, long long total, int F, int gelu) {
+// out[n][i] = the gated unit of gu[n][i] and gu[n][F + i]
+__global__ void __launch_bounds__(256) glu_f32_kernel(const float* gu, float* out, long long total, int F, int act, float limit) {
   pdl_launch_dependents();
   pdl_wait();
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
   if (i >= total) return;
   const long long n = i / F;
-  const float z = gu[n * 2 * F + (i - n * F)], u = gu[n * 2 * F + F + (i - n * F)];
-  out[i] = (gelu ? act_f32(z, PRISM_ACT_GELU_TANH, 0.0f) : z / (1.0f + expf(-z))) * u;
+  float z = gu[n * 2 * F + (i - n * F)], u = gu[n * 2 * F + F + (i - n * F)];
+  if (act == PRISM_GLU_BOUNDED) {
+    z = fminf(z, limit);
+    u = fminf(fmaxf(u, -limit), limit) + 1.0f;
+    z /= 1.0f + expf(-PRISM_GLU_SLOPE * z);
+  } else {
+    z = act == PRISM_GLU_GELU_TANH ? act_f32(z, PRISM_ACT_GELU_TANH, 0.0f) : z / (1.0f + expf(-z));
+  }
+  out[i] = z * u;
 }
 
 }  // namespace
 
-// act: 1 silu, 2 gelu (tanh form)
-PRISM_API int prism_glu_f32(const void* gu, void* out, int N, int F, int act, void* stream, int pdl) {
+// act: 1 silu, 2 gelu (tanh form), 3 bounded by `limit`
+PRISM_API int prism_glu_f32(const void* gu, void* out, int N, int F, int act, float limit, void* stream, int pdl) {
   if (N <= 0) return 0;
-  if (F <= 0 || act < 1 || act > 2) return -1;
+  if (F <= 0 || act < PRISM_GLU_SILU || act > PRISM_GLU_BOUNDED) return -1;
   const long long total = (long long)N * F;
   return (int)prism_launch(glu_f32_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream),
-                           pdl != 0, (const float*)gu, (float*)out, total, F, act == 2 ? 1 : 0);
+                           pdl != 0, (const float*)gu, (float*)out, total, F, act, limit);
 }
 
 PRISM_API int prism_gemm_f32(const void* W, const void* X, void* out, int M, int T, int K, long long ldw, long long ldx,

@@ -53,6 +53,7 @@ struct GemmArgs {
   int tokens_fastest;  // grid rasterisation, see the kernel
   int out_f32;       // 1: fp32 partial output, one slab per split
   int act;           // 0 none, 1 gelu(tanh), 2 gelu(erf)
+  float glu_limit;   // bound of a bounded gated unit
   long long ldo;     // output row stride (elements)
   long long ldr;     // residual row stride (elements)
   long long split_stride;  // elements between split slabs
@@ -246,7 +247,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           tmem_ld1(t_lane + c, rg);
           tmem_ld1(t_lane + BN + c, ru);
           tmem_ld_wait();
-          if (m_ok) out_b[(size_t)(group.y + i) * a.ldo + m] = __float2bfloat16_rn(glu(__uint_as_float(rg), __uint_as_float(ru), a.act));
+          if (m_ok) out_b[(size_t)(group.y + i) * a.ldo + m] = __float2bfloat16_rn(glu(__uint_as_float(rg), __uint_as_float(ru), a.act, a.glu_limit));
         }
       } else {
       unsigned long long push_seq = 0;
@@ -354,7 +355,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             __nv_bfloat16* dst = out_b + row0 * a.ldo + m;
 #pragma unroll
             for (int j = 0; j < 16; ++j)
-              if (j < cols) dst[(size_t)j * a.ldo] = __float2bfloat16_rn(glu(__uint_as_float(r[j]), __uint_as_float(r2[j]), a.act));
+              if (j < cols) dst[(size_t)j * a.ldo] = __float2bfloat16_rn(glu(__uint_as_float(r[j]), __uint_as_float(r2[j]), a.act, a.glu_limit));
             break;
           }
         }
@@ -398,6 +399,7 @@ struct PersistArgs {
   int m_tiles, n_tiles;
   int tokens_fastest;
   int act;
+  float glu_limit;   // bound of a bounded gated unit
   int out_f32;  // row-major form without residual or scatter: out is float
   long long ldo, ldr;
   const __nv_bfloat16* bias;
@@ -591,8 +593,8 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
           __nv_bfloat162* op = reinterpret_cast<__nv_bfloat162*>(o);
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
-            op[e] = __floats2bfloat162_rn(glu(__uint_as_float(rg[2 * e]), __uint_as_float(ru[2 * e]), a.act),
-                                          glu(__uint_as_float(rg[2 * e + 1]), __uint_as_float(ru[2 * e + 1]), a.act));
+            op[e] = __floats2bfloat162_rn(glu(__uint_as_float(rg[2 * e]), __uint_as_float(ru[2 * e]), a.act, a.glu_limit),
+                                          glu(__uint_as_float(rg[2 * e + 1]), __uint_as_float(ru[2 * e + 1]), a.act, a.glu_limit));
           }
           __nv_bfloat16* dst = a.out + (size_t)m * a.ldo + f_base + c0;
           *reinterpret_cast<uint4*>(dst) = o[0];
@@ -700,7 +702,7 @@ gemm_wx_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
         if (DUAL) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
-            if (j < cols) dst[(size_t)j * a.ldo] = __float2bfloat16_rn(glu(__uint_as_float(r[j]), __uint_as_float(r2[j]), a.act));
+            if (j < cols) dst[(size_t)j * a.ldo] = __float2bfloat16_rn(glu(__uint_as_float(r[j]), __uint_as_float(r2[j]), a.act, a.glu_limit));
         } else if (plain) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
@@ -1117,15 +1119,16 @@ PRISM_API int prism_gemm_wx_sections(const void* W, const void* X, void* out, in
 }
 
 // Experts' projections of a decode-sized step.  W stacks the experts' matrices (act != 0: M gate rows then M up rows each, the
-// output is act(gate) * up in bf16; act == 0: M rows each, the output fp32 split-K slabs).  Entry i of the table is
+// output is act(gate) * up in bf16, limit the bound of a bounded unit; act == 0: M rows each, the output fp32 split-K slabs).  Entry i of the table is
 // (expert, first row, rows, -) with rows <= T.  row_token != null: X holds the step's T <= 128 tokens and output row n belongs
 // to token row_token[n]; null: X and the output share their row numbers.
 PRISM_API int prism_gemm_grouped_small(const void* W, const void* X, void* out, int M, int T, int X_rows, int K, long long ldx,
                                        long long ldo, const void* groups, int max_groups, const void* n_groups, const void* row_token,
-                                       int N, int experts, int act, int splits, long long split_stride, void* stream, int pdl) {
+                                       int N, int experts, int act, float limit, int splits, long long split_stride, void* stream,
+                                       int pdl) {
   if (M <= 0 || T <= 0 || T > 128 || K <= 0 || K % 8 || max_groups <= 0 || max_groups > 65535 || experts <= 0 || !groups || !n_groups) return -1;
   const bool dual = act != 0;
-  if (act < 0 || act > PRISM_GLU_GELU_TANH || (dual != (row_token != nullptr)) || (dual && splits > 1) || X_rows < (dual ? T : N)) return -2;
+  if (act < 0 || act > PRISM_GLU_BOUNDED || (dual != (row_token != nullptr)) || (dual && splits > 1) || X_rows < (dual ? T : N)) return -2;
   GemmArgs a = {};
   a.M = M;
   a.T = N;
@@ -1137,6 +1140,7 @@ PRISM_API int prism_gemm_grouped_small(const void* W, const void* X, void* out, 
   a.w2_row_off = M;
   a.out_f32 = dual ? 0 : 1;
   a.act = act;
+  a.glu_limit = limit;
   a.ldo = ldo;
   a.split_stride = split_stride;
   a.out = out;
@@ -1167,9 +1171,10 @@ PRISM_API int prism_gemm_grouped_small(const void* W, const void* X, void* out, 
 // Experts' projections of a prompt: X [N][K] and out [N][ldo] (bf16) in expert order, table entries of at most 128 rows.
 // act != 0: W [experts][M gate rows, M up rows][K], out = act(gate) * up; act == 0: W [experts][M][K].  M a multiple of 16.
 PRISM_API int prism_gemm_grouped(const void* W, const void* X, void* out, int M, int N, int K, long long ldx, long long ldo,
-                                 const void* groups, int max_groups, const void* n_groups, int experts, int act, void* stream, int pdl) {
+                                 const void* groups, int max_groups, const void* n_groups, int experts, int act, float limit, void* stream,
+                                 int pdl) {
   if (M <= 0 || M % 16 || N <= 0 || K <= 0 || K % 8 || max_groups <= 0 || experts <= 0 || !groups || !n_groups) return -1;
-  if (act < 0 || act > PRISM_GLU_GELU_TANH || ldo % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return -2;
+  if (act < 0 || act > PRISM_GLU_BOUNDED || ldo % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return -2;
   const bool dual = act != 0;
   PersistArgs pa = {};
   pa.sec.n = 0;
@@ -1182,6 +1187,7 @@ PRISM_API int prism_gemm_grouped(const void* W, const void* X, void* out, int M,
   pa.n_tiles = dual ? (M + 127) / 128 : (M + 255) / 256;
   pa.tokens_fastest = 1;  // consecutive tiles share a token tile: the features of one expert follow one another
   pa.act = act;
+  pa.glu_limit = limit;
   pa.ldo = ldo;
   pa.out = reinterpret_cast<__nv_bfloat16*>(out);
   pa.rows_per_owner = 1;

@@ -13,6 +13,13 @@
 // GEMM makes keys and values of all heads, and the tcgen05 kernel of attention_tcgen05.cu attends over them.
 // The *_f32 kernels are the absorbed form in true 32-bit.
 //
+// Rotated columns.  A row may hold, behind the latent, a rotated key part that all heads share; a head's query then has a
+// rotated part of its own.  With an identity block in U_h for those columns, q~_h holds the rotated query beside U_h^T q_h, so
+// that scores are still q~_h . row and explicit keys still U_h row; values take the row's first Rv elements only.
+//   latent_prepare_kernel    norms of the query latent and of the key latent, rotation and page store of the shared key part
+//   latent_rotate_kernel     rotation of the queries where no absorb kernel does it (explicit keys, 32-bit)
+// A query may see a window of the newest rows only: tiles outside it are not visited.
+//
 // Latent rows are padded with zeros to Rc elements (a multiple of 64), heads to dq / dv elements (multiples of 8).
 #include "mma_sync.cuh"
 
@@ -134,8 +141,197 @@ __global__ void __launch_bounds__(256) latent_norm_store_kernel(const NormStoreA
 }
 
 // -------------------------------------------------------------------------------------------------
+// Rotation of neighbouring columns: the pair (u, v) number i of a row at position p turns by p * freq[i].
+// -------------------------------------------------------------------------------------------------
+struct Rotation {
+  const float* freq;       // [dims / 2] (null: nothing turns)
+  const int* positions;    // [tokens]
+  float amplitude;         // factor on sine and cosine
+  int start, dims;         // columns start .. start + dims - 1
+};
+// Columns c .. c + 3 (c and start multiples of 4) of a row whose position is pos.
+__device__ __forceinline__ void rotate4(float (&v)[4], const Rotation& r, float pos, int c) {
+#pragma unroll
+  for (int e = 0; e < 4; e += 2) {
+    const int i = c + e - r.start;
+    if (i < 0 || i >= r.dims) continue;
+    float sn, cs;
+    sincosf(pos * r.freq[i >> 1], &sn, &cs);
+    sn *= r.amplitude;
+    cs *= r.amplitude;
+    const float a = v[e], b = v[e + 1];
+    v[e] = a * cs - b * sn;
+    v[e + 1] = b * cs + a * sn;
+  }
+}
+
+// Rows of a projection: fp32 split-K slabs [P][tokens][ld] whose sum they are, or rows of the compute type.
+template <typename T>
+struct Source {
+  const float* slabs;
+  long long slab_stride;
+  int P;
+  const T* rows;
+  long long ld;
+};
+__device__ __forceinline__ void get4(float (&v)[4], const float* p) {
+  const float4 f = *reinterpret_cast<const float4*>(p);
+  v[0] = f.x;
+  v[1] = f.y;
+  v[2] = f.z;
+  v[3] = f.w;
+}
+__device__ __forceinline__ void get4(float (&v)[4], const bf16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+  const float2 a = __bfloat1622float2(h[0]), b = __bfloat1622float2(h[1]);
+  v[0] = a.x;
+  v[1] = a.y;
+  v[2] = b.x;
+  v[3] = b.y;
+}
+__device__ __forceinline__ void put4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void put4(bf16* p, const float (&v)[4]) {
+  uint2 o;
+  o.x = pack_bf16(v[0], v[1]);
+  o.y = pack_bf16(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = o;
+}
+template <typename T>
+__device__ __forceinline__ void source4(float (&v)[4], const Source<T>& s, size_t row, int c) {
+  if (s.slabs == nullptr) {
+    get4(v, s.rows + row * s.ld + c);
+    return;
+  }
+  v[0] = v[1] = v[2] = v[3] = 0.0f;
+  const float* src = s.slabs + row * s.ld + c;
+#pragma unroll 8
+  for (int p = 0; p < s.P; ++p) {
+    const float4 f = __ldcg(reinterpret_cast<const float4*>(src + (size_t)p * s.slab_stride));
+    v[0] += f.x;
+    v[1] += f.y;
+    v[2] += f.z;
+    v[3] += f.w;
+  }
+}
+
+// -------------------------------------------------------------------------------------------------
+// The stacked projection [query latent | key latent | shared key part] of a token, one CTA per token: the query latent over
+// its root mean square times a weight, and the token's cache row.  Sections start at multiples of 16 columns and their padding
+// is zero, so that sums over padded columns are sums over real ones.
+// -------------------------------------------------------------------------------------------------
+template <typename T>
+struct PrepareArgs {
+  Source<T> y;
+  const T* q_w;            // [Qp]
+  const T* c_w;            // [Cp]
+  T* q_out;                // [tokens][Qp]
+  T* cache;                // [blocks][page][Rc]
+  const long long* slots;  // flat slot, < 0: not stored
+  long long num_slots;
+  int Q, Qp, R, Cp, Rc;    // real and padded widths of the latents (Cp = 0: queries only), cache row
+  float eps;
+  Rotation rot;            // start: Cp, in columns of the cache row
+};
+
+constexpr int PREP_GROUPS = 4;  // groups of four columns a thread holds
+
+template <typename T>
+__global__ void __launch_bounds__(512) latent_prepare_kernel(const PrepareArgs<T> a) {
+  __shared__ float red[2][16];
+  const size_t t = blockIdx.x;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int total = a.Cp > 0 ? a.Qp + a.Rc : a.Qp, filled = a.Cp > 0 ? a.Qp + a.Cp + (a.rot.dims + 3) / 4 * 4 : a.Qp;
+  float v[PREP_GROUPS][4], sq = 0.0f, sc = 0.0f;
+#pragma unroll
+  for (int u = 0; u < PREP_GROUPS; ++u) {
+    const int c = (tid + u * blockDim.x) * 4;
+    v[u][0] = v[u][1] = v[u][2] = v[u][3] = 0.0f;
+    if (c < filled) source4(v[u], a.y, t, c);
+    const float ss = v[u][0] * v[u][0] + v[u][1] * v[u][1] + v[u][2] * v[u][2] + v[u][3] * v[u][3];
+    if (c < a.Qp) sq += ss;
+    else if (c < a.Qp + a.Cp) sc += ss;
+  }
+  sq = warp_sum(sq);
+  sc = warp_sum(sc);
+  if (lane == 0) {
+    red[0][warp] = sq;
+    red[1][warp] = sc;
+  }
+  __syncthreads();
+  sq = warp_sum(lane < nw ? red[0][lane] : 0.0f);
+  sc = warp_sum(lane < nw ? red[1][lane] : 0.0f);
+  const float iq = 1.0f / sqrtf(sq / (float)a.Q + a.eps), ic = 1.0f / sqrtf(sc / (float)max(a.R, 1) + a.eps);
+  T* row = nullptr;
+  float pos = 0.0f;
+  if (a.Cp > 0) {
+    const long long slot = a.slots[t];
+    if (slot >= a.num_slots) {
+      if (tid == 0) prism_report(PRISM_ERR_BOUNDS, 5);
+    } else if (slot >= 0) {
+      row = a.cache + (size_t)slot * a.Rc;
+    }
+    if (a.rot.dims > 0) pos = (float)a.rot.positions[t];
+  }
+#pragma unroll
+  for (int u = 0; u < PREP_GROUPS; ++u) {
+    const int c = (tid + u * blockDim.x) * 4;
+    if (c >= total) continue;
+    if (c < a.Qp) {
+      float w[4];
+      get4(w, a.q_w + c);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[u][e] *= iq * w[e];
+      put4(a.q_out + t * a.Qp + c, v[u]);
+      continue;
+    }
+    if (row == nullptr) continue;
+    const int r = c - a.Qp;
+    if (r < a.Cp) {
+      float w[4];
+      get4(w, a.c_w + r);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[u][e] *= ic * w[e];
+    } else {
+      rotate4(v[u], a.rot, pos, r);
+    }
+    put4(row + r, v[u]);
+  }
+}
+
+// -------------------------------------------------------------------------------------------------
+// Queries [tokens][H * dq] with the rotated columns of every head turned.  In place only those columns are touched.
+// -------------------------------------------------------------------------------------------------
+template <typename T>
+struct RotateArgs {
+  Source<T> q;
+  T* out;                  // [tokens][ldo]
+  long long ldo;
+  int tokens, H, dq, per;  // per: groups of four columns of a head that are handled
+  int first;               // first of them
+  Rotation rot;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) latent_rotate_kernel(const RotateArgs<T> a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x, per_token = (long long)a.H * a.per;
+  if (i >= a.tokens * per_token) return;
+  const size_t t = (size_t)(i / per_token);
+  const int k = (int)(i - (long long)t * per_token), h = k / a.per, c = a.first + (k - h * a.per) * 4;
+  float v[4];
+  source4(v, a.q, t, h * a.dq + c);
+  if (a.rot.dims > 0) rotate4(v, a.rot, (float)a.rot.positions[t], c);
+  put4(a.out + t * a.ldo + (size_t)h * a.dq + c, v);
+}
+
+// -------------------------------------------------------------------------------------------------
 // q~ = U_h^T q_h for a tile of 16 tokens, one head and 128 latent elements per CTA.  The CTAs with
-// blockIdx.y == H run the norm and store instead, one token per warp.
+// blockIdx.y == H (if the launch has them) run the norm and store instead, one token per warp.  Queries that are rotated, or
+// that come as slabs, are rounded once, on their way into shared memory.
 // -------------------------------------------------------------------------------------------------
 constexpr int ABS_N = 128, ABS_LDW = ABS_N + 8;
 
@@ -146,6 +342,8 @@ struct AbsorbArgs {
   bf16* out;               // [tokens][H][Rc]
   int H, dq, dk16;         // dk16: dq rounded up to 16
   NormStoreArgs<bf16> ns;
+  Source<bf16> src;        // the queries where they are not taken as they are (slabs or rows null otherwise)
+  Rotation rot;            // columns of a head
 };
 
 __global__ void __launch_bounds__(128) latent_absorb_kernel(const AbsorbArgs a) {
@@ -167,10 +365,22 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const AbsorbArgs a) 
     cp_async16(w_s + k * ABS_LDW + c, ok ? a.uk + ((size_t)h * a.dq + k) * Rc + n0 + c : a.uk, ok);
   }
   pdl_wait();
-  for (int i = threadIdx.x; i < 16 * (a.dk16 / 8); i += 128) {
-    const int r = i / (a.dk16 / 8), c = (i % (a.dk16 / 8)) * 8;
-    const bool ok = t0 + r < a.ns.tokens && c < a.dq;
-    cp_async16(q_s + r * ldq_s + c, ok ? a.q + (size_t)(t0 + r) * a.ldq + (size_t)h * a.dq + c : a.q, ok);
+  if (a.src.slabs != nullptr || a.src.rows != nullptr) {
+    for (int i = threadIdx.x; i < 16 * (a.dk16 / 4); i += 128) {
+      const int r = i / (a.dk16 / 4), c = (i % (a.dk16 / 4)) * 4;
+      float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      if (t0 + r < a.ns.tokens && c < a.dq) {
+        source4(v, a.src, (size_t)(t0 + r), h * a.dq + c);
+        if (a.rot.dims > 0) rotate4(v, a.rot, (float)a.rot.positions[t0 + r], c);
+      }
+      put4(q_s + r * ldq_s + c, v);
+    }
+  } else {
+    for (int i = threadIdx.x; i < 16 * (a.dk16 / 8); i += 128) {
+      const int r = i / (a.dk16 / 8), c = (i % (a.dk16 / 8)) * 8;
+      const bool ok = t0 + r < a.ns.tokens && c < a.dq;
+      cp_async16(q_s + r * ldq_s + c, ok ? a.q + (size_t)(t0 + r) * a.ldq + (size_t)h * a.dq + c : a.q, ok);
+    }
   }
   cp_async_commit();
   cp_async_wait_all();
@@ -209,10 +419,11 @@ struct LatentAttnArgs {
   const int* block_tables;  // [S][max_blocks], < 0: hole
   const int* cu_q;          // [S + 1] token offsets; null: sequence s is token s
   const int* kv_lens;       // [S] visible latents of the sequence's last token
-  float* part_o;            // [tokens * H][nsplit][Rc]  (nsplit > 1)
+  float* part_o;            // [tokens * H][nsplit][Rv]  (nsplit > 1)
   float* part_ml;           // [tokens * H][nsplit][2]   maximum (base 2, scaled) and sum
-  bf16* out;                // [tokens * H][Rc] normalised (nsplit == 1)
-  int H, Rc, page, max_blocks, num_blocks, nsplit;
+  bf16* out;                // [tokens * H][Rv] normalised (nsplit == 1)
+  int H, Rc, Rv, page, max_blocks, num_blocks, nsplit;
+  int window;               // a query sees that many newest rows, its own among them
   float scale;
 };
 
@@ -235,18 +446,18 @@ __host__ __device__ constexpr size_t latent_smem_bytes(int Rc) {
 //             for the whole kernel where they fit (QREG), the slices are added when the softmax reads them
 //   softmax   BM / 8 rows per warp; a row's reference maximum is only raised when a tile exceeds it by more than
 //             2^8 (the weights stay below 256), so the accumulators are rarely rescaled
-//   output    every warp accumulates Rc / 8 columns of P C in registers
+//   output    every warp accumulates Rv / 8 columns of P C in registers
 // Latent rows come by one bulk copy each, issued by one thread per row, two tiles in flight.  Tiles that hold only
-// latents of earlier steps are fetched before the previous kernel has finished.
-template <int MT, int NT, int BN>
+// latents of earlier steps are fetched before the previous kernel has finished.  Rv is at most 64 NT, Rc at most 64 QN.
+template <int MT, int NT, int QN, int BN>
 __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAttnArgs a) {
   constexpr int BM = 16 * MT;
   constexpr int KG = BN / 16, KH = 8 / KG;
-  constexpr bool QREG = NT <= 8;
-  constexpr int QS = QREG ? NT * 4 / KH : 1;              // 16-element steps of a warp's slice (compile-time bound)
+  constexpr bool QREG = QN <= 8 || (QN <= 10 && MT == 1);
+  constexpr int QS = QREG ? QN * 4 / KH : 1;              // 16-element steps of a warp's slice (compile-time bound)
   constexpr int LDS = BN + 4, LDP = BN + 8;
   extern __shared__ __align__(128) uint8_t smem_raw[];
-  const int Rc = a.Rc, LD = Rc + 8, nt = Rc >> 6;         // nt: 8-column tiles of the output per warp
+  const int Rc = a.Rc, LD = Rc + 8, nt = a.Rv >> 6;       // nt: 8-column tiles of the output per warp
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);           // [BM][LD]
   bf16* kv_s = q_s + (size_t)BM * LD;                      // [2][BN][LD]
   float* s_s = reinterpret_cast<float*>(kv_s + (size_t)2 * BN * LD);  // [KH][BM][LDS]
@@ -266,8 +477,10 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
   const int kv_len = clamp_context(a.kv_lens[seq], a.max_blocks, a.page);
   const int last_t = min(row0 + BM, n_rows) - 1;
   const int kv_end = max(0, min(kv_len, kv_len - q_len + last_t / a.H + 1));
-  const int tiles = (kv_end + BN - 1) / BN, per = (tiles + a.nsplit - 1) / a.nsplit;
-  const int tb = split * per, te = min(tiles, tb + per);
+  // the first row any query of the tile sees, in whole tiles
+  const int t_first = max(0, kv_len - q_len + row0 / a.H + 1 - a.window) / BN;
+  const int tiles = (kv_end + BN - 1) / BN, per = (max(0, tiles - t_first) + a.nsplit - 1) / a.nsplit;
+  const int tb = t_first + split * per, te = min(tiles, tb + per);
   const size_t out_row0 = (size_t)q_start * a.H + row0;
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
   const uint32_t row_bytes = (uint32_t)Rc * 2;
@@ -393,7 +606,7 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
 #pragma unroll
     for (int i = 0; i < BM / 8; ++i) {
       const int r = warp * (BM / 8) + i;
-      const int limit = lim_s[r] - j * BN;
+      const int limit = lim_s[r] - j * BN, low = limit - a.window;
       float v[BN / 32], mx = -INFINITY;
 #pragma unroll
       for (int e = 0; e < BN / 32; ++e) {
@@ -401,7 +614,7 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
         float t = s_s[r * LDS + c];
 #pragma unroll
         for (int h = 1; h < KH; ++h) t += s_s[(h * BM + r) * LDS + c];
-        v[e] = c < limit ? t * sl2 : -INFINITY;
+        v[e] = c < limit && c >= low ? t * sl2 : -INFINITY;
         mx = fmaxf(mx, v[e]);
       }
       mx = warp_max(mx);
@@ -481,9 +694,9 @@ __global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentAt
         const int col = warp * nt * 8 + n * 8 + 2 * (lane & 3);
         const float v0 = acc[m][n][2 * half] * inv, v1 = acc[m][n][2 * half + 1] * inv;
         if (a.nsplit > 1)
-          *reinterpret_cast<float2*>(a.part_o + ((out_row0 + r) * a.nsplit + split) * Rc + col) = make_float2(v0, v1);
+          *reinterpret_cast<float2*>(a.part_o + ((out_row0 + r) * a.nsplit + split) * a.Rv + col) = make_float2(v0, v1);
         else
-          *reinterpret_cast<uint32_t*>(a.out + (out_row0 + r) * Rc + col) = pack_bf16(v0, v1);
+          *reinterpret_cast<uint32_t*>(a.out + (out_row0 + r) * a.Rv + col) = pack_bf16(v0, v1);
       }
     }
 }
@@ -497,7 +710,8 @@ struct LatentOutArgs {
   const float* part_o;
   const float* part_ml;
   const bf16* lat;         // [tokens * H][Rc] (nsplit == 1)
-  const bf16* uv;          // [H * dv][Rc]
+  const bf16* uv;          // [H * dv][ldw]
+  long long ldw;
   const bf16* gate;        // [tokens][gate_ld], head h at column h * dv (null: one)
   long long gate_ld;
   bf16* out;               // [tokens][ld_out]
@@ -566,7 +780,7 @@ __global__ void __launch_bounds__(OUT_THREADS) latent_out_kernel(const LatentOut
   pdl_launch_dependents();
   for (int r = warp; r < OUT_N; r += OUT_THREADS / 32) {
     const bool ok = n0 + r < a.dv;
-    const bf16* src = ok ? a.uv + ((size_t)h * a.dv + n0 + r) * Rc : a.uv;
+    const bf16* src = ok ? a.uv + ((size_t)h * a.dv + n0 + r) * a.ldw : a.uv;
     for (int c = lane * 8; c < Rc; c += 256) cp_async16(w_s + (size_t)r * LD + c, ok ? src + c : src, ok);
   }
   cp_async_commit();
@@ -664,6 +878,37 @@ __global__ void __launch_bounds__(256) gather_latents_kernel(const GatherLatentA
   for (int i = lane; i < a.row_bytes / 16; i += 32) out[i] = blk >= 0 ? src[i] : make_uint4(0, 0, 0, 0);
 }
 
+// Pages of every sequence from first[s] on, one behind the other from scratch page base[s] on; rows past the sequence's end and
+// holes are zero.  One warp per row.
+struct GatherPagesArgs {
+  const uint8_t* cache;
+  const int* block_tables;
+  const int* kv_lens;
+  const int* first;        // [S]
+  const int* base;         // [S + 1]
+  uint8_t* rows;           // [base[S] * page][row_bytes]
+  int max_blocks, num_blocks, page, row_bytes, total;
+};
+
+__global__ void __launch_bounds__(256) gather_latent_pages_kernel(const GatherPagesArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.y, lane = threadIdx.x & 31, j = blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int base = a.base[seq];
+  if (j >= (a.base[seq + 1] - base) * a.page) return;
+  const long long dst = (long long)base * a.page + j;
+  if (dst < 0 || dst >= a.total) {
+    if (lane == 0) prism_report(PRISM_ERR_BOUNDS, 6);
+    return;
+  }
+  const int page_no = a.first[seq] + j / a.page, key = page_no * a.page + j % a.page;
+  const bool in = key < a.kv_lens[seq] && page_no < a.max_blocks;
+  const int blk = in ? checked_page(a.block_tables[(size_t)seq * a.max_blocks + page_no], a.num_blocks) : -1;
+  const uint4* src = reinterpret_cast<const uint4*>(a.cache + ((size_t)max(blk, 0) * a.page + j % a.page) * a.row_bytes);
+  uint4* out = reinterpret_cast<uint4*>(a.rows + (size_t)dst * a.row_bytes);
+  for (int i = lane; i < a.row_bytes / 16; i += 32) out[i] = blk >= 0 ? src[i] : make_uint4(0, 0, 0, 0);
+}
+
 // -------------------------------------------------------------------------------------------------
 // True 32-bit forms.
 // -------------------------------------------------------------------------------------------------
@@ -707,7 +952,7 @@ struct LatentF32Args {
   const int* cu_q;
   const int* kv_lens;
   float* out;               // [tokens][H][Rc]
-  int H, Rc, page, max_blocks, num_blocks;
+  int H, Rc, page, max_blocks, num_blocks, window;
   float scale;
 };
 
@@ -734,7 +979,7 @@ __global__ void __launch_bounds__(128) latent_attention_f32_kernel(const LatentF
     o[e] = 0.0f;
   }
   float m = -INFINITY, l = 0.0f;
-  for (int j = warp; j < limit; j += 4) {
+  for (int j = max(0, limit - a.window) + warp; j < limit; j += 4) {
     const int blk = checked_page(a.block_tables[(size_t)seq * a.max_blocks + j / a.page], a.num_blocks);
     if (blk < 0) continue;
     const float* c = a.cache + ((size_t)blk * a.page + j % a.page) * a.Rc;
@@ -783,16 +1028,16 @@ __global__ void __launch_bounds__(128) latent_attention_f32_kernel(const LatentF
   }
 }
 
-template <int MT, int NT, int BN>
+template <int MT, int NT, int QN, int BN>
 int launch_latent(const LatentAttnArgs& a, int row_tiles, int S, cudaStream_t stream, bool pdl) {
   const size_t smem = latent_smem_bytes<MT, BN>(a.Rc);
   static size_t configured = 0;
   if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<MT, NT, BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<MT, NT, QN, BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  return (int)prism_launch(latent_attention_kernel<MT, NT, BN>, dim3(row_tiles, a.nsplit, S), dim3(256), smem, stream, pdl, a);
+  return (int)prism_launch(latent_attention_kernel<MT, NT, QN, BN>, dim3(row_tiles, a.nsplit, S), dim3(256), smem, stream, pdl, a);
 }
 
 template <typename T>
@@ -821,12 +1066,16 @@ PRISM_API int prism_latent_norm_store(int f32, const void* raw, long long ld_raw
                            norm_store_args<bf16>(raw, ld_raw, weight, cache, slots, num_slots, rows, tokens, R, Rc, eps));
 }
 
-// q~ [tokens][H][Rc] = U_h^T q_h (bf16), with the norm and store of the same tokens' latents in the same launch.
-PRISM_API int prism_latent_absorb(const void* q, long long ldq, const void* uk, void* out, const void* raw, long long ld_raw,
-                                  const void* weight, void* cache, const void* slots, long long num_slots, int tokens, int H,
+// q~ [tokens][H][Rc] = U_h^T q_h (bf16), with the norm and store of the same tokens' latents in the same launch (raw null:
+// without).  Queries: rows q, or q_slabs [P][tokens][ldq] fp32 whose sum they are; freq (null: none): columns rot_start ..
+// rot_start + rot - 1 of every head are rotated first.
+PRISM_API int prism_latent_absorb(const void* q, const void* q_slabs, long long q_stride, int q_P, long long ldq, const void* freq,
+                                  const void* positions, float amplitude, int rot_start, int rot, const void* uk, void* out, const void* raw,
+                                  long long ld_raw, const void* weight, void* cache, const void* slots, long long num_slots, int tokens, int H,
                                   int dq, int R, int Rc, float eps, void* stream, int pdl) {
   if (tokens <= 0) return 0;
-  if (R <= 0 || R > Rc || Rc % 64 || H <= 0 || dq % 8 || ldq % 8 || Rc > 1024) return -1;
+  if (R <= 0 || R > Rc || Rc % 64 || H <= 0 || dq % 8 || ldq % 8 || Rc > 1024 || (!q && !q_slabs)) return -1;
+  if (freq != nullptr && (!positions || rot_start < 0 || rot_start % 4 || rot < 0 || rot % 2 || rot_start + rot > dq)) return -3;
   AbsorbArgs a;
   a.q = (const bf16*)q;
   a.ldq = ldq;
@@ -836,6 +1085,8 @@ PRISM_API int prism_latent_absorb(const void* q, long long ldq, const void* uk, 
   a.dq = dq;
   a.dk16 = (dq + 15) / 16 * 16;
   a.ns = norm_store_args<bf16>(raw, ld_raw, weight, cache, slots, num_slots, nullptr, tokens, R, Rc, eps);
+  a.src = Source<bf16>{(const float*)q_slabs, q_stride, q_P, freq != nullptr ? (const bf16*)q : nullptr, ldq};
+  a.rot = Rotation{(const float*)freq, (const int*)positions, amplitude, rot_start, freq != nullptr ? rot : 0};
   const size_t smem = ((size_t)a.dk16 * ABS_LDW + 16 * (a.dk16 + 8)) * 2;
   if (smem > 220 * 1024) return -2;
   static size_t configured = 48 * 1024;
@@ -844,43 +1095,46 @@ PRISM_API int prism_latent_absorb(const void* q, long long ldq, const void* uk, 
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  const dim3 grid((Rc + ABS_N - 1) / ABS_N, H + 1, (tokens + 15) / 16);
+  const dim3 grid((Rc + ABS_N - 1) / ABS_N, raw != nullptr ? H + 1 : H, (tokens + 15) / 16);
   return (int)prism_launch(latent_absorb_kernel, grid, dim3(128), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
 }
 
-// Causal attention of q~ over the paged latents.  nsplit > 1: unnormalised fp32 partials and their maxima / sums;
-// nsplit == 1: normalised bf16 rows in out.  Rc at most 1024.
+// Causal attention of q~ over the paged latents, the newest `window` of them.  nsplit > 1: unnormalised fp32 partials and their
+// maxima / sums; nsplit == 1: normalised bf16 rows in out.  Rows of Rc elements, of which the first Rv are summed up; both
+// multiples of 64, Rc at most 1024.
 PRISM_API int prism_latent_attention(const void* q, const void* cache, const void* block_tables, const void* cu_q,
                                      const void* kv_lens, void* part_o, void* part_ml, void* out, int S, int max_q_len, int H,
-                                     int Rc, int page, int max_blocks, int num_blocks, int nsplit, float scale, void* stream,
-                                     int pdl) {
+                                     int Rc, int Rv, int page, int max_blocks, int num_blocks, int nsplit, int window, float scale,
+                                     void* stream, int pdl) {
   if (S <= 0 || max_q_len <= 0) return 0;
-  if (H <= 0 || Rc % 64 || Rc <= 0 || Rc > 1024 || page <= 0 || max_blocks <= 0) return -1;
+  if (H <= 0 || Rc % 64 || Rc <= 0 || Rc > 1024 || Rv % 64 || Rv <= 0 || Rv > Rc || page <= 0 || max_blocks <= 0 || window < 1) return -1;
   if (nsplit < 1 || nsplit > MAX_SPLITS || (nsplit > 1 ? (!part_o || !part_ml) : !out)) return -2;
   LatentAttnArgs a{(const bf16*)q, (const bf16*)cache, (const int*)block_tables, (const int*)cu_q, (const int*)kv_lens,
-                   (float*)part_o, (float*)part_ml, (bf16*)out, H, Rc, page, max_blocks, num_blocks, nsplit, scale};
+                   (float*)part_o, (float*)part_ml, (bf16*)out, H, Rc, Rv, page, max_blocks, num_blocks, nsplit, window, scale};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const long long rows = (long long)max_q_len * H;
   // 16-row tiles read the latents once per 16 heads instead of 32: worth it while they still fit the device in one wave
   const bool narrow = rows <= 16 || (rows + 15) / 16 * nsplit * S <= 148;
   const int tiles = (int)((rows + (narrow ? 15 : 31)) / (narrow ? 16 : 32));
   const bool p = pdl != 0;
-#define PRISM_LATENT_CASE(NT_, BN_)                                    \
-  return narrow ? launch_latent<1, NT_, BN_>(a, tiles, S, s, p) : launch_latent<2, NT_, BN_>(a, tiles, S, s, p);
-  if (Rc <= 128) PRISM_LATENT_CASE(2, 64)
-  if (Rc <= 256) PRISM_LATENT_CASE(4, 64)
-  if (Rc <= 512) PRISM_LATENT_CASE(8, 64)
-  PRISM_LATENT_CASE(16, 32)
+#define PRISM_LATENT_CASE(NT_, QN_, BN_)                                         \
+  return narrow ? launch_latent<1, NT_, QN_, BN_>(a, tiles, S, s, p) : launch_latent<2, NT_, QN_, BN_>(a, tiles, S, s, p);
+  if (Rc <= 128) PRISM_LATENT_CASE(2, 2, 64)
+  if (Rc <= 256) PRISM_LATENT_CASE(4, 4, 64)
+  if (Rc <= 512) PRISM_LATENT_CASE(8, 8, 64)
+  if (Rc <= 640 && Rv <= 512) PRISM_LATENT_CASE(8, 10, 64)
+  PRISM_LATENT_CASE(16, 16, 32)
 #undef PRISM_LATENT_CASE
 }
 
-// out [tokens][ld_out] (head h at column h * dv) = gate * V_h o~_h, o~ merged from the splits of prism_latent_attention.
-PRISM_API int prism_latent_out(const void* part_o, const void* part_ml, const void* lat, const void* uv, const void* gate,
+// out [tokens][ld_out] (head h at column h * dv) = gate * V_h o~_h, o~ merged from the splits of prism_latent_attention.  Rc: the
+// elements that were summed up; uv rows ldw apart.
+PRISM_API int prism_latent_out(const void* part_o, const void* part_ml, const void* lat, const void* uv, long long ldw, const void* gate,
                                long long gate_ld, void* out, long long ld_out, int tokens, int H, int dv, int Rc, int nsplit,
                                void* stream, int pdl) {
   if (tokens <= 0) return 0;
-  if (H <= 0 || dv % 8 || Rc % 64 || Rc <= 0 || Rc > 1024 || nsplit < 1 || nsplit > MAX_SPLITS || gate_ld % 2 || ld_out % 2) return -1;
-  LatentOutArgs a{(const float*)part_o, (const float*)part_ml, (const bf16*)lat, (const bf16*)uv, (const bf16*)gate, gate_ld,
+  if (H <= 0 || dv % 8 || Rc % 64 || Rc <= 0 || Rc > 1024 || nsplit < 1 || nsplit > MAX_SPLITS || gate_ld % 2 || ld_out % 2 || ldw < Rc || ldw % 8) return -1;
+  LatentOutArgs a{(const float*)part_o, (const float*)part_ml, (const bf16*)lat, (const bf16*)uv, ldw, (const bf16*)gate, gate_ld,
                   (bf16*)out, ld_out, tokens, H, dv, Rc, nsplit};
   const size_t smem = (size_t)(OUT_N + 16) * (Rc + 8) * 2;
   static size_t configured = 40 * 1024;
@@ -893,6 +1147,54 @@ PRISM_API int prism_latent_out(const void* part_o, const void* part_ml, const vo
   return (int)prism_launch(latent_out_kernel, grid, dim3(OUT_THREADS), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
 }
 
+// Stacked projection [tokens][ld] (fp32 slabs or rows of the compute type) with Qp columns of a query latent (Q real ones), Cp of
+// a key latent (R real ones) and rot of the shared key part -> q_out [tokens][Qp], normed, and cache rows of Rc elements
+// [Cp | rot | zeros].  Cp = 0: queries only.  Qp and Cp multiples of 16.
+PRISM_API int prism_latent_prepare(int f32, const void* slabs, long long slab_stride, int P, const void* rows, long long ld, const void* q_w,
+                                   const void* c_w, void* q_out, void* cache, const void* slots, long long num_slots, const void* freq,
+                                   const void* positions, float amplitude, int tokens, int Q, int Qp, int R, int Cp, int rot, int Rc, float eps,
+                                   void* stream, int pdl) {
+  if (tokens <= 0) return 0;
+  if (Q <= 0 || Q > Qp || Qp % 16 || Cp < 0 || Cp % 16 || rot < 0 || rot % 2 || ld % 4 || (!slabs && !rows)) return -1;
+  if (Cp > 0 && (R <= 0 || R > Cp || Rc % 64 || Cp + rot > Rc || !cache || !slots || (rot > 0 && (!freq || !positions)))) return -2;
+  const int groups = (Qp + (Cp > 0 ? Rc : 0)) / 4, per = tokens <= 256 ? 1 : PREP_GROUPS;
+  int threads = ((groups + per - 1) / per + 31) / 32 * 32;
+  if (threads > 512) threads = 512;
+  if (groups > threads * PREP_GROUPS) return -3;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  auto run = [&](auto type) -> int {
+    using T = decltype(type);
+    PrepareArgs<T> a{Source<T>{(const float*)slabs, slab_stride, P, (const T*)rows, ld}, (const T*)q_w, (const T*)c_w, (T*)q_out, (T*)cache,
+                     (const long long*)slots, num_slots, Q, Qp, R, Cp, Rc, eps,
+                     Rotation{(const float*)freq, (const int*)positions, amplitude, Cp, Cp > 0 ? rot : 0}};
+    return (int)prism_launch(latent_prepare_kernel<T>, dim3(tokens), dim3(threads), 0, s, pdl != 0, a);
+  };
+  return f32 ? run(float()) : run(bf16());
+}
+
+// Queries as slabs or rows [tokens][ld] -> out [tokens][ldo], columns rot_start .. rot_start + rot - 1 of every head rotated.  rows ==
+// out: only those are touched.
+PRISM_API int prism_latent_rotate(int f32, const void* slabs, long long slab_stride, int P, const void* rows, long long ld, void* out,
+                                  long long ldo, const void* freq, const void* positions, float amplitude, int tokens, int H, int dq,
+                                  int rot_start, int rot, void* stream, int pdl) {
+  if (tokens <= 0) return 0;
+  if (H <= 0 || dq <= 0 || dq % 8 || ld % 4 || ldo % 4 || rot_start < 0 || rot_start % 4 || rot < 0 || rot % 2 || rot_start + rot > dq) return -1;
+  if ((!slabs && !rows) || (rot > 0 && (!freq || !positions))) return -2;
+  const bool in_place = !slabs && rows == out;
+  const int first = in_place ? rot_start : 0, per = in_place ? (rot + 3) / 4 : dq / 4;
+  if (per == 0) return 0;
+  const long long total = (long long)tokens * H * per;
+  if ((total + 255) / 256 > 0x7fffffffll) return -3;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  auto run = [&](auto type) -> int {
+    using T = decltype(type);
+    RotateArgs<T> a{Source<T>{(const float*)slabs, slab_stride, P, (const T*)rows, ld}, (T*)out, ldo, tokens, H, dq, per, first,
+                    Rotation{(const float*)freq, (const int*)positions, amplitude, rot_start, rot}};
+    return (int)prism_launch(latent_rotate_kernel<T>, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, pdl != 0, a);
+  };
+  return f32 ? run(float()) : run(bf16());
+}
+
 // rows [total][row_bytes]: the latents each sequence sees (cu_kv), gathered from their pages.
 PRISM_API int prism_gather_latents(const void* cache, const void* block_tables, const void* cu_kv, void* rows, int S,
                                    int max_kv_len, int total, int max_blocks, int num_blocks, int page, int row_bytes,
@@ -902,6 +1204,19 @@ PRISM_API int prism_gather_latents(const void* cache, const void* block_tables, 
   GatherLatentArgs a{(const uint8_t*)cache, (const int*)block_tables, (const int*)cu_kv, (uint8_t*)rows,
                      max_blocks, num_blocks, page, row_bytes, total};
   return (int)prism_launch(gather_latents_kernel, dim3((max_kv_len + 7) / 8, S), dim3(256), 0,
+                           reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
+}
+
+// rows [total][row_bytes]: of every sequence the pages first[s] .. as scratch pages base[s] .. base[s + 1] - 1, each of `page`
+// rows; max_pages: the most pages of a sequence.
+PRISM_API int prism_gather_latent_pages(const void* cache, const void* block_tables, const void* kv_lens, const void* first, const void* base,
+                                        void* rows, int S, int max_pages, int total, int max_blocks, int num_blocks, int page, int row_bytes,
+                                        void* stream, int pdl) {
+  if (S <= 0 || max_pages <= 0 || total <= 0) return 0;
+  if (row_bytes % 16 || page <= 0 || max_blocks <= 0 || S > 65535) return -1;
+  GatherPagesArgs a{(const uint8_t*)cache, (const int*)block_tables, (const int*)kv_lens, (const int*)first, (const int*)base, (uint8_t*)rows,
+                    max_blocks, num_blocks, page, row_bytes, total};
+  return (int)prism_launch(gather_latent_pages_kernel, dim3((unsigned)(((long long)max_pages * page + 7) / 8), S), dim3(256), 0,
                            reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
 }
 
@@ -917,11 +1232,11 @@ PRISM_API int prism_headwise_f32(const void* x, long long ldx, const void* w, lo
 
 PRISM_API int prism_latent_attention_f32(const void* q, const void* cache, const void* block_tables, const void* cu_q,
                                          const void* kv_lens, void* out, int S, int max_q_len, int H, int Rc, int page,
-                                         int max_blocks, int num_blocks, float scale, void* stream, int pdl) {
+                                         int max_blocks, int num_blocks, int window, float scale, void* stream, int pdl) {
   if (S <= 0 || max_q_len <= 0) return 0;
-  if (H <= 0 || Rc % 64 || Rc <= 0 || Rc > 1024 || page <= 0 || max_blocks <= 0) return -1;
+  if (H <= 0 || Rc % 64 || Rc <= 0 || Rc > 1024 || page <= 0 || max_blocks <= 0 || window < 1) return -1;
   LatentF32Args a{(const float*)q, (const float*)cache, (const int*)block_tables, (const int*)cu_q, (const int*)kv_lens,
-                  (float*)out, H, Rc, page, max_blocks, num_blocks, scale};
+                  (float*)out, H, Rc, page, max_blocks, num_blocks, window, scale};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid((unsigned)max_q_len * H, S);
   const size_t smem = (size_t)4 * Rc * sizeof(float);

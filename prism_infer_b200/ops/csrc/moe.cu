@@ -8,7 +8,8 @@
 //                      over the chosen logits, count per expert and rank of each pair within its chunk and expert.  With a
 //                      single chunk it also places the pairs.  Scored form: the softmax is over all outputs, a correction
 //                      enters the choice only, which is among the best groups of neighbours; outputs E .. choices - 1 stand
-//                      for the token's own row (their weights are summed up for the kernel that adds the branch).
+//                      for the token's own row (their weights are summed up for the kernel that adds the branch).  Scores
+//                      may be the outputs' own sigmoids, and a group as good as the sum of its two best.
 //   moe_place_kernel   one CTA per chunk: first row of every expert, then rows of the chunk's pairs
 //   moe_gather_kernel  copies a token's row to the rows of its pairs
 #include "common.cuh"
@@ -43,6 +44,8 @@ struct RouteArgs {
   int sets, keep;           // the best `keep` of `sets` equal runs of neighbours are open to choice
   int always_col;           // logit whose sigmoid weighs the always-on experts (-1: weight one)
   float scale;
+  int sigmoid;              // 1: the scores are the logits' sigmoids, not divided by their sum
+  int group_best;           // a group's score is its best output's (1) or the sum of its two best (2)
 };
 
 // Exclusive prefix sum over the block of one value per thread; *total gets the sum.
@@ -112,11 +115,20 @@ __device__ __forceinline__ void keep_best_groups(float (&choice)[C], const Route
 #pragma unroll
   for (int c = 0; c < C; ++c) best[c] = -INFINITY;
   for (int g = 0; g < a.sets; ++g) {
-    float m = -INFINITY;
+    float m = -INFINITY, second = -INFINITY;
 #pragma unroll
     for (int c = 0; c < C; ++c)
-      if (of[c] == g) m = fmaxf(m, choice[c]);
-    m = warp_max(m);
+      if (of[c] == g) {
+        second = fmaxf(second, fminf(m, choice[c]));
+        m = fmaxf(m, choice[c]);
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float om = __shfl_xor_sync(0xffffffffu, m, o), os = __shfl_xor_sync(0xffffffffu, second, o);
+      second = fmaxf(fmaxf(second, os), fminf(m, om));
+      m = fmaxf(m, om);
+    }
+    if (a.group_best == 2 && second > -INFINITY) m += second;
 #pragma unroll
     for (int c = 0; c < C; ++c)
       if (c * 32 + lane == g) best[c] = m;
@@ -183,13 +195,20 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArg
         for (int p = 0; p < a.P; ++p) s += __ldcg(a.logits + (size_t)p * a.slab_stride + t * a.ld + a.always_col);
         always_w = 1.0f / (1.0f + expf(-s));
       }
-      float m = v[0], total = 0.0f;
+      float total = 1.0f;
+      if (a.sigmoid) {
 #pragma unroll
-      for (int c = 1; c < C; ++c) m = fmaxf(m, v[c]);
-      m = warp_max(m);
+        for (int c = 0; c < C; ++c) score[c] = 1.0f / (1.0f + expf(-v[c]));
+      } else {
+        float m = v[0];
 #pragma unroll
-      for (int c = 0; c < C; ++c) total += score[c] = expf(v[c] - m);
-      total = 1.0f / warp_sum(total);
+        for (int c = 1; c < C; ++c) m = fmaxf(m, v[c]);
+        m = warp_max(m);
+        total = 0.0f;
+#pragma unroll
+        for (int c = 0; c < C; ++c) total += score[c] = expf(v[c] - m);
+        total = 1.0f / warp_sum(total);
+      }
 #pragma unroll
       for (int c = 0; c < C; ++c) {
         score[c] *= total;
@@ -239,7 +258,7 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RouteArg
       }
     }
     __syncwarp();
-    const float inv = SCORED ? a.scale / (sum + 1e-20f) : 1.0f / sum;
+    const float inv = SCORED ? (a.sigmoid ? a.scale : a.scale / (sum + 1e-20f)) : 1.0f / sum;
     for (int k = lane; k < K; k += 32) {
       if (k >= a.top) expert_s[i * K + k] = live ? a.E + k - a.top : -1;
       a.weight[t * K + k] = live ? (k < a.top ? a.weight[t * K + k] * inv : always_w) : 0.0f;
@@ -304,7 +323,7 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const bf16* x, long lon
 int check_route(const RouteArgs& a) {
   if (a.top < 1 || a.top > a.choices || a.choices < a.E || a.choices > MAX_EXPERTS || a.always < 0 || a.E + a.always > MAX_EXPERTS || a.chunk < 1 || a.tile < 1 || a.max_groups < 1) return -1;
   if ((long long)a.T * (a.top + a.always) > 0x7fffffffll || a.chunk * (a.top + a.always) > 10240) return -2;
-  if (a.correction != nullptr && (!a.self_weight || a.sets < 1 || a.choices % a.sets || a.keep < 1 || a.keep > a.sets)) return -3;
+  if (a.correction != nullptr && (!a.self_weight || a.sets < 1 || a.choices % a.sets || a.keep < 1 || a.keep > a.sets || a.group_best < 1 || a.group_best > 2)) return -3;
   return 0;
 }
 
@@ -321,15 +340,15 @@ int launch_route(const RouteArgs& a, size_t smem, cudaStream_t st, bool pdl) {
 // [chunks][E + always]; groups [max_groups] int4 and n_groups: tiles of at most `tile` rows of one expert.  With more than
 // one chunk prism_moe_place must follow.  correction != null: the scored form, with the logits of `choices` outputs (the E
 // experts, then those that stand for the token's own row, whose weight goes to self_weight [T]) and, at column always_col if
-// that is not negative, the one whose sigmoid weighs the always-on experts.
+// that is not negative, the one whose sigmoid weighs the always-on experts; sigmoid and group_best as in RouteArgs.
 PRISM_API int prism_moe_route(const void* logits, long long slab_stride, long long ld, int P, const void* slots, void* expert, void* pos,
                               void* weight, void* row_token, void* counts, void* groups, int max_groups, void* n_groups, int T, int top,
                               int E, int always, int chunk, int tile, const void* correction, void* self_weight, int choices,
-                              int sets, int keep, int always_col, float scale, void* stream, int pdl) {
+                              int sets, int keep, int always_col, float scale, int sigmoid, int group_best, void* stream, int pdl) {
   if (T <= 0) return 0;
   RouteArgs a{(const float*)logits, slab_stride, ld, P, (const long long*)slots, (int*)expert, (int*)pos, (float*)weight, (int*)row_token,
               (int*)counts, (int4*)groups, max_groups, (int*)n_groups, T, top, E, always, chunk, tile, (const float*)correction,
-              (float*)self_weight, choices, sets, keep, always_col, scale};
+              (float*)self_weight, choices, sets, keep, always_col, scale, sigmoid, group_best};
   if (int rc = check_route(a)) return rc;
   const size_t smem = (size_t)chunk * (top + always) * sizeof(int);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
@@ -344,7 +363,7 @@ PRISM_API int prism_moe_place(void* expert, void* pos, void* weight, void* row_t
                               void* n_groups, int T, int top, int E, int always, int chunk, int tile, void* stream, int pdl) {
   if (T <= 0) return 0;
   RouteArgs a{nullptr, 0, 0, 0, nullptr, (int*)expert, (int*)pos, (float*)weight, (int*)row_token, (int*)counts, (int4*)groups, max_groups,
-              (int*)n_groups, T, top, E, always, chunk, tile, nullptr, nullptr, top > E ? top : E, 1, 1, -1, 1.0f};
+              (int*)n_groups, T, top, E, always, chunk, tile, nullptr, nullptr, top > E ? top : E, 1, 1, -1, 1.0f, 0, 1};
   if (int rc = check_route(a)) return rc;
   return (int)prism_launch(moe_place_kernel, dim3((T + chunk - 1) / chunk), dim3(ROUTE_THREADS), 0, reinterpret_cast<cudaStream_t>(stream),
                            pdl != 0, a);

@@ -1,18 +1,23 @@
-// Recurrent mixers with a matrix state per head, and what they read of the previous token.
+// Recurrent mixers with a matrix state per head, and what a layer reads of the tokens before.
 //
-// A sequence's state of one layer is a row of fp32 in a slot:  [heads][n][n] (key channel, value channel), then the last
-// token's input row [W].  Every slot has two versions: a step that takes a sequence from c tokens to c' reads version c & 1
-// and writes version c' & 1, so a step that is repeated finds what it read before.  A sequence without tokens (c = 0)
+// A sequence's state of one layer is a row of fp32 in a slot:  [heads][n][m] (key channel, value channel), then what it carries
+// of the last tokens' input rows.  Every slot has two versions: a step that takes a sequence from c tokens to c' reads version
+// c & 1 and writes version c' & 1, so a step that is repeated finds what it read before.  A sequence without tokens (c = 0)
 // starts from zero whatever its slot holds.
 //
 //   token_mix_kernel      five blends of a token's row with the previous token's, and the table of a grouped projection
+//   short_conv_kernel     a causal convolution over the last few rows of every channel
 //   decay_project_kernel  decays of many tokens from the narrow projection's rows (bf16; fp32 takes the 32-bit GEMM)
-//   state_step_kernel     one token per sequence: decay, output, state update, norm per head, gate
+//   state_step_kernel     one token per sequence: output, state update, norm per head, gate
 //   state_scan_kernel     many tokens of a sequence: the state stays in registers, loader warps feed token blocks
 //   head_norm_gate_kernel norm per head and gate behind the scan
 //
-// Per head, with r, k, v, the decay d = exp(-exp(z)) and the bonus u (all fp32):
-//   o_t = (S + diag(u) k v^T)^T r,   S <- diag(d) S + k v^T.
+// Per head, with r, k, v, a decay d and a weight b per key channel (all fp32):
+//   o_t = S^T r + (b . 1) v,   S <- diag(d) S + k v^T.
+// The rules (n = m in the first):
+//   RULE_BONUS   r and k as projected, b = r u k, d = exp(-exp(z)): the token itself counts with the bonus u
+//   RULE_FORGET  a gate f = l + (1 - l) sigmoid(z + c) per key channel decays and writes:  d = f, k = 1 - f, and with
+//                q = silu(y) read behind the update r = q f, b = q k
 #include "mma_sync.cuh"
 
 #include <type_traits>
@@ -34,6 +39,7 @@ __device__ __forceinline__ float4 load4(const bf16* p) {
   const float2 a = __bfloat1622float2(h[0]), b = __bfloat1622float2(h[1]);
   return make_float4(a.x, a.y, b.x, b.y);
 }
+enum StateRule : int { RULE_BONUS = 0, RULE_FORGET = 1 };
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ void store4(bf16* p, float4 v) {
@@ -105,6 +111,28 @@ struct RawProj {
     }
   }
 };
+
+// What RULE_FORGET makes of a channel's query y, gate z (bias added) and lower bound l.
+struct Forget {
+  float r, k, d, b;
+};
+template <typename T>
+__device__ __forceinline__ Forget forget_of(float y, float z, float l) {
+  float stay, q;                                  // stay: 1 - sigmoid(z), exact where the gate is all but open
+  if (sizeof(T) == 2) {
+    stay = __fdividef(1.0f, 1.0f + __expf(z));
+    q = __fdividef(y, 1.0f + __expf(-y));
+  } else {
+    stay = 1.0f / (1.0f + expf(z));
+    q = y / (1.0f + expf(-y));
+  }
+  Forget f;
+  f.k = (1.0f - l) * stay;
+  f.d = 1.0f - f.k;
+  f.r = q * f.d;
+  f.b = q * f.k;
+  return f;
+}
 
 // The state slots of a layer and the sequences of a step.
 struct StateArgs {
@@ -193,6 +221,76 @@ __global__ void __launch_bounds__(256) token_mix_kernel(const MixArgs<T> a) {
       store4(a.out + ((size_t)m * a.T_rows + t) * W + c,
              make_float4(fmaf(d.x, mu.x, x.x), fmaf(d.y, mu.y, x.y), fmaf(d.z, mu.z, x.z), fmaf(d.w, mu.w, x.w)));
     }
+  }
+}
+
+// =====================================================================================
+// out_t = x_t + sum_j w_j x_(t - taps + 1 + j) on every channel, rows before the step's from the slot's carry (oldest first) and
+// zeros before the sequence's start.  grid (chunks of a sequence, column blocks, sequences): a thread walks four columns through
+// a chunk.  A chunk is no shorter than the rows that are carried on, so only a sequence's first one reads the carry: it writes the
+// new one too, after it has read the old (both may be the same version).  MT: taps, rounded up.
+// =====================================================================================
+constexpr int CONV_CHUNK = 16;
+template <typename T>
+struct ConvArgs {
+  StateArgs st;            // x is not used
+  const T* x;              // [T][W]
+  const T* w;              // [taps][W]
+  T* out;                  // [T][W]
+  int taps;
+};
+
+template <typename T, int MT>
+__global__ void __launch_bounds__(256) short_conv_kernel(const ConvArgs<T> a) {
+  const int W = a.st.W, s = blockIdx.z, c = (blockIdx.y * 256 + threadIdx.x) * 4, i0 = blockIdx.x * CONV_CHUNK;
+  pdl_launch_dependents();
+  const Span sp = span_of(a.st, s);
+  if (i0 >= sp.len || c >= W) return;             // a row without a slot has a carry of zeros
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 w[MT], h[MT];                            // aligned at the end: tap MT - 1 meets the row itself
+#pragma unroll
+  for (int k = 0; k < MT; ++k) w[k] = k >= MT - a.taps ? load4(a.w + (size_t)(k - (MT - a.taps)) * W + c) : zero;
+  pdl_wait();
+  const T* x = a.x + (size_t)sp.first * W + c;
+  const int keep = a.taps - 1;
+#pragma unroll
+  for (int k = 0; k < MT - 1; ++k) {
+    const int p = i0 - (MT - 1) + k;              // row within the step's part of the sequence
+    h[k] = zero;
+    if (k < MT - a.taps) continue;
+    if (p >= 0) h[k] = load4(x + (size_t)p * W);
+    else if (sp.old_version) h[k] = load4(sp.old_version + a.st.carry + (size_t)(keep + p) * W + c);
+  }
+  if (i0 == 0 && sp.new_version) {
+    float* dst = sp.new_version + a.st.carry + c;
+#pragma unroll
+    for (int k = 0; k < MT - 1; ++k) {
+      if (k < MT - a.taps) continue;
+      const int p = sp.len - (MT - 1) + k;
+      float4 v = zero;
+      if (p >= 0) v = load4(x + (size_t)p * W);
+#pragma unroll
+      for (int q = 0; q < MT - 1; ++q)
+        if (p < 0 && q == MT - 1 + p) v = h[q];
+      store4(dst + (size_t)(k - (MT - a.taps)) * W, v);
+    }
+  }
+  T* out = a.out + (size_t)sp.first * W + c;
+  const int n = min(CONV_CHUNK, sp.len - i0);
+#pragma unroll 4
+  for (int i = 0; i < n; ++i) {
+    h[MT - 1] = load4(x + (size_t)(i0 + i) * W);
+    float4 o = h[MT - 1];
+#pragma unroll
+    for (int k = 0; k < MT; ++k) {
+      o.x = fmaf(w[k].x, h[k].x, o.x);
+      o.y = fmaf(w[k].y, h[k].y, o.y);
+      o.z = fmaf(w[k].z, h[k].z, o.z);
+      o.w = fmaf(w[k].w, h[k].w, o.w);
+    }
+    store4(out + (size_t)(i0 + i) * W, o);
+#pragma unroll
+    for (int k = 0; k < MT - 1; ++k) h[k] = h[k + 1];
   }
 }
 
@@ -340,36 +438,37 @@ __global__ void __launch_bounds__(256) tanh_f32_kernel(const Proj<float> z, floa
 template <typename T>
 struct StepArgs {
   StateArgs st;
-  Proj<T> p;               // r, k, v, gate: rows m * tokens + t, columns head * n
+  // RULE_BONUS: r, k, v, gate, rows m * tokens + t, columns head * n.  RULE_FORGET: a row per token, [queries | gates | values].
+  Proj<T> p;
   Proj<T> w1;              // [tokens][rank] input of the decay's second projection, before tanh
   const T* w2;             // [heads * n][rank]
-  const T* w0;             // [heads * n]
-  const T* u;              // [heads * n]
-  const T* norm;           // [heads * n]
-  T* out;                  // [tokens][heads * n]
-  int tokens, H, n, n_real, rank;
+  const T* w0;             // [heads * n] decays' offsets; RULE_FORGET: gates' bias
+  const T* u;              // [heads * n] bonus; RULE_FORGET: lower bounds
+  const T* norm;           // [heads * m]; RULE_FORGET: [m], for every head
+  T* out;                  // [tokens][heads * m]
+  int tokens, H, n, m, m_real, rank;
   float eps;
 };
 
-template <typename T, int NV, int NT>
+template <typename T, int NV, int NT, int RULE>
 __global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_step_kernel(const StepArgs<T> a) {
   extern __shared__ float sm[];
-  const int n = a.n, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, s = blockIdx.y;
-  float *r_s = sm, *k_s = sm + n, *v_s = sm + 2 * n, *g_s = sm + 3 * n, *d_s = sm + 4 * n, *b_s = sm + 5 * n, *t_s = sm + 6 * n;
-  float* o_s = t_s + a.rank;                      // [rows][n] partial outputs
+  const int n = a.n, m = a.m, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, s = blockIdx.y;
+  float *r_s = sm, *k_s = sm + n, *d_s = sm + 2 * n, *b_s = sm + 3 * n, *v_s = sm + 4 * n, *g_s = v_s + m, *t_s = g_s + m;
+  float* o_s = t_s + a.rank;                      // [rows][m] partial outputs
   __shared__ float red[NT / 32];
-  const int c4 = n >> 2, rows = NT / c4, tx = tid % c4, ty = tid / c4;
+  const int c4 = m >> 2, rows = NT / c4, tx = tid % c4, ty = tid / c4;
   pdl_launch_dependents();
   const Span sp = span_of(a.st, s);
-  const size_t C = (size_t)a.H * n, hc = (size_t)h * n;
-  T* out = a.out + (size_t)s * C + hc;
+  const size_t C = (size_t)a.H * m, hn = (size_t)h * n, hm = (size_t)h * m;
+  T* out = a.out + (size_t)s * C + hm;
   if (sp.new_version == nullptr) {
     pdl_wait();
-    for (int c = tid; c < n; c += NT) put(out + c, 0.0f);
+    for (int c = tid; c < m; c += NT) put(out + c, 0.0f);
     return;
   }
-  const float* old_s = sp.old_version ? sp.old_version + (size_t)h * n * n : nullptr;
-  float* new_s = sp.new_version + (size_t)h * n * n;
+  const float* old_s = sp.old_version ? sp.old_version + (size_t)h * n * m : nullptr;
+  float* new_s = sp.new_version + (size_t)h * n * m;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   const bool active = ty < rows;
   float4 S[NV > 0 ? NV : 1];
@@ -377,38 +476,60 @@ __global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_st
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int key = ty + i * rows;
-      S[i] = active && key < n && old_s ? __ldcs(reinterpret_cast<const float4*>(old_s + (size_t)key * n) + tx) : zero;
+      S[i] = active && key < n && old_s ? __ldcs(reinterpret_cast<const float4*>(old_s + (size_t)key * m) + tx) : zero;
     }
   }
-  for (int i = tid * 128; i < n * a.rank * (int)sizeof(T); i += NT * 128)   // the head's rows of the decay projection
-    asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(a.w2 + hc * a.rank) + i));
-  pdl_wait();
-  // the projections' sums, and the narrow one's tanh
-  for (int i = tid; i < 4 * c4 + a.rank; i += NT) {
-    if (i < 4 * c4) {
-      const int m = i / c4, c = (i - m * c4) * 4;
-      store4(sm + m * n + c, proj4(a.p, (size_t)m * a.tokens + s, (int)hc + c));
-    } else {
-      t_s[i - 4 * c4] = tanhf(proj1(a.w1, (size_t)s, i - 4 * c4));
-    }
-  }
-  __syncthreads();
-  // decay and bonus: eight lanes per channel over the rank
-#pragma unroll 4
-  for (int c0 = 0; c0 < n; c0 += NT / 8) {
-    const int c = c0 + (tid >> 3);
-    float z = 0.0f;
-    if (c < n)
-      for (int j = (tid & 7) * 4; j < a.rank; j += 32) {
-        const float4 w = load4(a.w2 + (hc + c) * a.rank + j), t = load4(t_s + j);
-        z += w.x * t.x + w.y * t.y + w.z * t.z + w.w * t.w;
+  if (RULE == RULE_BONUS) {
+    for (int i = tid * 128; i < n * a.rank * (int)sizeof(T); i += NT * 128)   // the head's rows of the decay projection
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(a.w2 + hn * a.rank) + i));
+    pdl_wait();
+    // the projections' sums, and the narrow one's tanh
+    for (int i = tid; i < 4 * c4 + a.rank; i += NT) {
+      if (i < 4 * c4) {
+        const int q = i / c4, c = (i - q * c4) * 4;
+        float* dst = q == 0 ? r_s : (q == 1 ? k_s : (q == 2 ? v_s : g_s));
+        store4(dst + c, proj4(a.p, (size_t)q * a.tokens + s, (int)hm + c));
+      } else {
+        t_s[i - 4 * c4] = tanhf(proj1(a.w1, (size_t)s, i - 4 * c4));
       }
-    z += __shfl_xor_sync(0xffffffffu, z, 1);
-    z += __shfl_xor_sync(0xffffffffu, z, 2);
-    z += __shfl_xor_sync(0xffffffffu, z, 4);
-    if (c < n && (tid & 7) == 0) {
-      d_s[c] = decay_of(z + to_f(a.w0[hc + c]));
-      b_s[c] = r_s[c] * to_f(a.u[hc + c]) * k_s[c];
+    }
+    __syncthreads();
+    // decay and bonus: eight lanes per channel over the rank
+#pragma unroll 4
+    for (int c0 = 0; c0 < n; c0 += NT / 8) {
+      const int c = c0 + (tid >> 3);
+      float z = 0.0f;
+      if (c < n)
+        for (int j = (tid & 7) * 4; j < a.rank; j += 32) {
+          const float4 w = load4(a.w2 + (hn + c) * a.rank + j), t = load4(t_s + j);
+          z += w.x * t.x + w.y * t.y + w.z * t.z + w.w * t.w;
+        }
+      z += __shfl_xor_sync(0xffffffffu, z, 1);
+      z += __shfl_xor_sync(0xffffffffu, z, 2);
+      z += __shfl_xor_sync(0xffffffffu, z, 4);
+      if (c < n && (tid & 7) == 0) {
+        d_s[c] = decay_of(z + to_f(a.w0[hn + c]));
+        b_s[c] = r_s[c] * to_f(a.u[hn + c]) * k_s[c];
+      }
+    }
+  } else {
+    pdl_wait();
+    const int n4 = n >> 2, Hn = a.H * n;
+    for (int i = tid; i < n4 + c4; i += NT) {
+      if (i < n4) {
+        const int c = i * 4;
+        const float4 y = proj4(a.p, (size_t)s, (int)hn + c), z = proj4(a.p, (size_t)s, Hn + (int)hn + c);
+        const float4 bias = load4(a.w0 + hn + c), low = load4(a.u + hn + c);
+        const Forget f[4] = {forget_of<float>(y.x, z.x + bias.x, low.x), forget_of<float>(y.y, z.y + bias.y, low.y),
+                             forget_of<float>(y.z, z.z + bias.z, low.z), forget_of<float>(y.w, z.w + bias.w, low.w)};
+        store4(r_s + c, make_float4(f[0].r, f[1].r, f[2].r, f[3].r));
+        store4(k_s + c, make_float4(f[0].k, f[1].k, f[2].k, f[3].k));
+        store4(d_s + c, make_float4(f[0].d, f[1].d, f[2].d, f[3].d));
+        store4(b_s + c, make_float4(f[0].b, f[1].b, f[2].b, f[3].b));
+      } else {
+        const int c = (i - n4) * 4;
+        store4(v_s + c, proj4(a.p, (size_t)s, 2 * Hn + (int)hm + c));
+      }
     }
   }
   __syncthreads();
@@ -421,7 +542,7 @@ __global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_st
       o.y = fmaf(b, v.y, fmaf(r, st.y, o.y));
       o.z = fmaf(b, v.z, fmaf(r, st.z, o.z));
       o.w = fmaf(b, v.w, fmaf(r, st.w, o.w));
-      __stcs(reinterpret_cast<float4*>(new_s + (size_t)key * n) + tx,
+      __stcs(reinterpret_cast<float4*>(new_s + (size_t)key * m) + tx,
              make_float4(fmaf(d, st.x, k * v.x), fmaf(d, st.y, k * v.y), fmaf(d, st.z, k * v.z), fmaf(d, st.w, k * v.w)));
     };
     if (NV > 0) {
@@ -430,19 +551,19 @@ __global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_st
         if (ty + i * rows < n) step(ty + i * rows, S[i]);
     } else {
 #pragma unroll 8
-      for (int key = ty; key < n; key += rows) step(key, old_s ? __ldcs(reinterpret_cast<const float4*>(old_s + (size_t)key * n) + tx) : zero);
+      for (int key = ty; key < n; key += rows) step(key, old_s ? __ldcs(reinterpret_cast<const float4*>(old_s + (size_t)key * m) + tx) : zero);
     }
-    store4(o_s + (size_t)ty * n + 4 * tx, o);
+    store4(o_s + (size_t)ty * m + 4 * tx, o);
   }
-  // the last token's row, a share per head
-  for (int c = (h * NT + tid) * 4; c < a.st.W; c += a.H * NT * 4)
-    store4(sp.new_version + a.st.carry + c, load4(a.st.x + (size_t)s * a.st.W + c));
+  if (RULE == RULE_BONUS)                         // the last token's row, a share per head
+    for (int c = (h * NT + tid) * 4; c < a.st.W; c += a.H * NT * 4)
+      store4(sp.new_version + a.st.carry + c, load4(a.st.x + (size_t)s * a.st.W + c));
   __syncthreads();
   float ss = 0.0f;
-  for (int c = tid; c < n; c += NT) {
+  for (int c = tid; c < m; c += NT) {
     float o = 0.0f;
 #pragma unroll 8
-    for (int i = 0; i < rows; ++i) o += o_s[(size_t)i * n + c];
+    for (int i = 0; i < rows; ++i) o += o_s[(size_t)i * m + c];
     o_s[c] = o;                                   // column c is this thread's
     ss += o * o;
   }
@@ -450,8 +571,11 @@ __global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_st
   if (lane == 0) red[warp] = ss;
   __syncthreads();
   ss = warp_sum(lane < NT / 32 ? red[lane] : 0.0f);
-  const float inv = 1.0f / sqrtf(ss / (float)a.n_real + a.eps);
-  for (int c = tid; c < n; c += NT) put(out + c, o_s[c] * inv * to_f(a.norm[hc + c]) * silu_f(g_s[c]));
+  const float inv = 1.0f / sqrtf(ss / (float)a.m_real + a.eps);
+  for (int c = tid; c < m; c += NT) {
+    const float o = o_s[c] * inv * to_f(a.norm[RULE == RULE_BONUS ? hm + c : c]);
+    put(out + c, RULE == RULE_BONUS ? o * silu_f(g_s[c]) : o);
+  }
 }
 
 // =====================================================================================
@@ -459,7 +583,7 @@ __global__ void __launch_bounds__(NT, NV > 8 ? 1 : (NT == 128 ? 7 : 3)) state_st
 // four value columns, sixteen lanes the keys of a column, so that a token costs a lane three 16-byte shared-memory reads per
 // four keys and one for the values; the lanes' partial outputs of four tokens are summed by one reduce-scatter.  Four more
 // warps feed blocks of TB tokens: while a block is worked on they turn the next one's raw rows, already in registers, into
-// what the products need (fp32, the bonus' scalar per token) and fetch rows of the blocks behind it.
+// what the products need (fp32, the scalar b . 1 per token) and fetch rows of the blocks behind it.
 // =====================================================================================
 constexpr int SCAN_COLS = 32;
 constexpr int SCAN_THREADS = 256;
@@ -467,11 +591,12 @@ constexpr int SCAN_THREADS = 256;
 template <typename T>
 struct ScanArgs {
   StateArgs st;
-  Proj<T> p;               // r, k, v: rows m * tokens + t
-  const float* d;          // [tokens][heads * n] decays
-  const T* u;              // [heads * n]
-  float* o;                // [tokens][heads * n]
-  int tokens, H, n;
+  Proj<T> p;               // RULE_BONUS: r, k, v, rows m * tokens + t.  RULE_FORGET: a row per token, [queries | gates | values]
+  const float* d;          // [tokens][heads * n] decays (RULE_BONUS)
+  const T* u;              // [heads * n] bonus; RULE_FORGET: lower bounds
+  const T* bias;           // [heads * n] of the gates (RULE_FORGET)
+  float* o;                // [tokens][heads * m]
+  int tokens, H, n, m;
 };
 
 template <int KL>
@@ -485,23 +610,23 @@ struct ScanTile {
   static constexpr int FLOATS = BONUS + TB * PARTS;             // one buffer: [r | k | d][TB][NP], v [TB][32], bonus
 };
 
-template <typename T, int KL, bool SLABS>
+template <typename T, int KL, bool SLABS, int RULE>
 __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs<T> a) {
   extern __shared__ __align__(16) float sm[];                   // two buffers, then outputs [2][TB][32]
   using Tile = ScanTile<KL>;
   constexpr int TB = Tile::TB, NP = Tile::NP, G = Tile::G, ITEMS = Tile::ITEMS;
-  const int n = a.n, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int blocks = (n + SCAN_COLS - 1) / SCAN_COLS, h = blockIdx.x / blocks, col0 = blockIdx.x % blocks * SCAN_COLS, s = blockIdx.y;
+  const int n = a.n, m = a.m, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int blocks = (m + SCAN_COLS - 1) / SCAN_COLS, h = blockIdx.x / blocks, col0 = blockIdx.x % blocks * SCAN_COLS, s = blockIdx.y;
   float* out_s = sm + 2 * Tile::FLOATS;
   pdl_launch_dependents();
   const Span sp = span_of(a.st, s);
-  const size_t C = (size_t)a.H * n, hc = (size_t)h * n;
+  const size_t C = (size_t)a.H * m, D = (size_t)a.H * n, hc = (size_t)h * n, hm = (size_t)h * m;
   pdl_wait();
   if (sp.len <= 0) return;
   const int nb = (sp.len + TB - 1) / TB;
   if (sp.new_version == nullptr) {                // no slot: outputs are zero
     for (int i = threadIdx.x; i < sp.len * SCAN_COLS; i += SCAN_THREADS)
-      if (col0 + i % SCAN_COLS < n) a.o[(size_t)(sp.first + i / SCAN_COLS) * C + hc + col0 + i % SCAN_COLS] = 0.0f;
+      if (col0 + i % SCAN_COLS < m) a.o[(size_t)(sp.first + i / SCAN_COLS) * C + hm + col0 + i % SCAN_COLS] = 0.0f;
     return;
   }
   if (warp >= 4) {
@@ -509,13 +634,13 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
     const int tid = threadIdx.x - 128, g = tid % G, c = g * 4;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     const bool in = c < n;
-    const float4 u = in ? load4(a.u + hc + c) : zero;
+    const float4 u = in ? load4(a.u + hc + c) : zero, bias = RULE == RULE_FORGET && in ? load4(a.bias + hc + c) : zero;
     const int vi = tid >> 3, vc = (tid & 7) * 4;                // a token in sixteen, a group of value columns
-    const bool v_in = col0 + vc < n;
+    const bool v_in = col0 + vc < m;
     using Raw = RawProj<T, SLABS>;
-    struct Rows {                                               // of one block
+    struct Rows {                                               // of one block (k: the gates under RULE_FORGET)
       typename Raw::type r[ITEMS], k[ITEMS], v[TB / 16];
-      float4 d[ITEMS];
+      float4 d[RULE == RULE_BONUS ? ITEMS : 1];
     };
     constexpr int AHEAD = ITEMS <= 4 ? 2 : 1;                   // blocks held in registers
     Rows held[AHEAD];
@@ -525,19 +650,26 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
       for (int q = 0; q < ITEMS; ++q) {
         const int tok = b * TB + tid / G + q * (128 / G);
         x.r[q] = x.k[q] = Raw::zero();
-        x.d[q] = zero;
-        if (tok >= sp.len) x.d[q].x = x.d[q].y = x.d[q].z = x.d[q].w = 1.0f;   // past the end: no decay, nothing added
-        else if (in) {
+        if constexpr (RULE == RULE_BONUS) {
+          x.d[q] = zero;
+          if (tok >= sp.len) x.d[q].x = x.d[q].y = x.d[q].z = x.d[q].w = 1.0f;   // past the end: no decay, nothing added
+        }
+        if (tok < sp.len && in) {
           const size_t t = (size_t)(sp.first + tok);
           x.r[q] = Raw::load(a.p, t, (int)hc + c);
-          x.k[q] = Raw::load(a.p, (size_t)a.tokens + t, (int)hc + c);
-          x.d[q] = __ldcg(reinterpret_cast<const float4*>(a.d + t * C + hc + c));
+          if constexpr (RULE == RULE_BONUS) {
+            x.k[q] = Raw::load(a.p, (size_t)a.tokens + t, (int)hc + c);
+            x.d[q] = __ldcg(reinterpret_cast<const float4*>(a.d + t * D + hc + c));
+          } else {
+            x.k[q] = Raw::load(a.p, t, (int)(D + hc) + c);
+          }
         }
       }
 #pragma unroll
       for (int q = 0; q < TB / 16; ++q) {
         const int tok = b * TB + vi + 16 * q;
-        x.v[q] = v_in && tok < sp.len ? Raw::load(a.p, (size_t)2 * a.tokens + sp.first + tok, (int)hc + col0 + vc) : Raw::zero();
+        const size_t row = RULE == RULE_BONUS ? (size_t)2 * a.tokens + sp.first + tok : (size_t)(sp.first + tok);
+        x.v[q] = v_in && tok < sp.len ? Raw::load(a.p, row, (int)(RULE == RULE_BONUS ? hm : 2 * D + hm) + col0 + vc) : Raw::zero();
       }
     };
     auto store = [&](const Rows& x, int b) {
@@ -547,10 +679,23 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
       for (int q = 0; q < ITEMS; ++q) {
         const int i = tid / G + q * (128 / G);
         const float4 rq = raw_value(x.r[q]), kq = raw_value(x.k[q]);
-        store4(dst + i * NP + c, rq);
-        store4(dst + Tile::K + i * NP + c, kq);
-        store4(dst + Tile::D + i * NP + c, x.d[q]);
-        float bonus = rq.x * u.x * kq.x + rq.y * u.y * kq.y + rq.z * u.z * kq.z + rq.w * u.w * kq.w;
+        float bonus;
+        if constexpr (RULE == RULE_BONUS) {
+          store4(dst + i * NP + c, rq);
+          store4(dst + Tile::K + i * NP + c, kq);
+          store4(dst + Tile::D + i * NP + c, x.d[q]);
+          bonus = rq.x * u.x * kq.x + rq.y * u.y * kq.y + rq.z * u.z * kq.z + rq.w * u.w * kq.w;
+        } else {
+          // past the sequence's end, and in columns past the head's: no decay, nothing added
+          const bool live = in && b * TB + i < sp.len;
+          const float4 low = live ? u : make_float4(1.f, 1.f, 1.f, 1.f);
+          const Forget f[4] = {forget_of<T>(rq.x, kq.x + bias.x, low.x), forget_of<T>(rq.y, kq.y + bias.y, low.y),
+                               forget_of<T>(rq.z, kq.z + bias.z, low.z), forget_of<T>(rq.w, kq.w + bias.w, low.w)};
+          store4(dst + i * NP + c, make_float4(f[0].r, f[1].r, f[2].r, f[3].r));
+          store4(dst + Tile::K + i * NP + c, make_float4(f[0].k, f[1].k, f[2].k, f[3].k));
+          store4(dst + Tile::D + i * NP + c, make_float4(f[0].d, f[1].d, f[2].d, f[3].d));
+          bonus = f[0].b + f[1].b + f[2].b + f[3].b;
+        }
 #pragma unroll
         for (int o = (G < 32 ? G : 32) / 2; o > 0; o >>= 1) bonus += __shfl_xor_sync(0xffffffffu, bonus, o);
         if (g % 32 == 0) dst[Tile::BONUS + i * Tile::PARTS + g / 32] = bonus;
@@ -573,24 +718,25 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
         __syncthreads();
       }
     }
-    // the last token's row, a share per CTA
-    const float* last = a.st.x + (size_t)(sp.first + sp.len - 1) * a.st.W;
-    for (int i = (blockIdx.x * 128 + tid) * 4; i < a.st.W; i += gridDim.x * 512) store4(sp.new_version + a.st.carry + i, load4(last + i));
+    if (RULE == RULE_BONUS) {                     // the last token's row, a share per CTA
+      const float* last = a.st.x + (size_t)(sp.first + sp.len - 1) * a.st.W;
+      for (int i = (blockIdx.x * 128 + tid) * 4; i < a.st.W; i += gridDim.x * 512) store4(sp.new_version + a.st.carry + i, load4(last + i));
+    }
     return;
   }
   // ------------------------------ state ------------------------------
   const int kl = lane & 15, col = warp * 8 + (lane >> 4) * 4;    // first of the lane's columns in the block
-  const bool live = col0 + col < n;
+  const bool live = col0 + col < m;
   unsigned long long S[KL / 2][4];                // keys 64 g + 4 kl + {0, 1}, {2, 3}
   {
-    const float* src = sp.old_version ? sp.old_version + (size_t)h * n * n + col0 + col : nullptr;
+    const float* src = sp.old_version ? sp.old_version + (size_t)h * n * m + col0 + col : nullptr;
 #pragma unroll
     for (int p = 0; p < KL / 2; ++p) {
       const int key = 64 * (p >> 1) + 4 * kl + 2 * (p & 1);
       float4 lo = make_float4(0.f, 0.f, 0.f, 0.f), hi = lo;
       if (live && src && key < n) {               // n is a multiple of 16
-        lo = load4(src + (size_t)key * n);
-        hi = load4(src + (size_t)(key + 1) * n);
+        lo = load4(src + (size_t)key * m);
+        hi = load4(src + (size_t)(key + 1) * m);
       }
       S[p][0] = pair_of(lo.x, hi.x);
       S[p][1] = pair_of(lo.y, hi.y);
@@ -680,24 +826,26 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
     __syncwarp();
     for (int i = lane >> 1; i < cnt; i += 16) {
       const int c = warp * 8 + (lane & 1) * 4;
-      if (col0 + c < n) store4(a.o + (size_t)(sp.first + b * TB + i) * C + hc + col0 + c, load4(out_b + i * SCAN_COLS + c));
+      if (col0 + c < m) store4(a.o + (size_t)(sp.first + b * TB + i) * C + hm + col0 + c, load4(out_b + i * SCAN_COLS + c));
     }
     __syncthreads();
   }
   if (!live) return;
-  float* dst = sp.new_version + (size_t)h * n * n + col0 + col;
+  float* dst = sp.new_version + (size_t)h * n * m + col0 + col;
 #pragma unroll
   for (int p = 0; p < KL / 2; ++p) {
     const int key = 64 * (p >> 1) + 4 * kl + 2 * (p & 1);
     if (key >= n) continue;
     const float2 f0 = unpair(S[p][0]), f1 = unpair(S[p][1]), f2 = unpair(S[p][2]), f3 = unpair(S[p][3]);
-    store4(dst + (size_t)key * n, make_float4(f0.x, f1.x, f2.x, f3.x));
-    store4(dst + (size_t)(key + 1) * n, make_float4(f0.y, f1.y, f2.y, f3.y));
+    store4(dst + (size_t)key * m, make_float4(f0.x, f1.x, f2.x, f3.x));
+    store4(dst + (size_t)(key + 1) * m, make_float4(f0.y, f1.y, f2.y, f3.y));
   }
 }
 
-// out = o / rms(o) * norm * silu(gate) per head.  A lane holds eight columns, L lanes a head; four rows of a warp at a time.
-template <typename T, int L, bool SLABS>
+// out = o / rms(o) * norm * silu(gate) per head (GATE: none, rows or slabs; without one the norm's weights are those of a head,
+// for every head).  A lane holds eight columns, L lanes a head; four rows of a warp at a time.
+enum GateKind : int { GATE_NONE = 0, GATE_ROWS = 1, GATE_SLABS = 2 };
+template <typename T, int L, int GATE>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, const Proj<T> p, const T* norm, T* out, int tokens, int H, int n,
                                                              int n_real, float eps) {
   constexpr int ROWS = 4;
@@ -706,7 +854,7 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, con
   pdl_launch_dependents();
   pdl_wait();
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  using Raw = RawProj<T, SLABS>;
+  using Raw = RawProj<T, GATE == GATE_SLABS>;
   float4 v[ROWS][2];
   typename Raw::type g[ROWS][2];
   long long t[ROWS];
@@ -721,7 +869,7 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, con
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       v[q][e] = in[q] ? __ldcg(reinterpret_cast<const float4*>(o + t[q] * (size_t)H * n + hc[q] + 4 * e)) : zero;
-      g[q][e] = in[q] ? Raw::load(p, (size_t)3 * tokens + t[q], hc[q] + 4 * e) : Raw::zero();
+      if (GATE != GATE_NONE) g[q][e] = in[q] ? Raw::load(p, (size_t)3 * tokens + t[q], hc[q] + 4 * e) : Raw::zero();
     }
   }
 #pragma unroll
@@ -735,9 +883,13 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, con
     if (!in[q]) continue;
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const float4 w = load4(norm + hc[q] + 4 * e), x = v[q][e], z = raw_value(g[q][e]);
-      store4(out + t[q] * (size_t)H * n + hc[q] + 4 * e, make_float4(x.x * inv * w.x * silu_f(z.x), x.y * inv * w.y * silu_f(z.y),
-                                                                   x.z * inv * w.z * silu_f(z.z), x.w * inv * w.w * silu_f(z.w)));
+      const float4 w = load4(norm + (GATE != GATE_NONE ? hc[q] : c) + 4 * e), x = v[q][e];
+      float4 y = make_float4(x.x * inv * w.x, x.y * inv * w.y, x.z * inv * w.z, x.w * inv * w.w);
+      if (GATE != GATE_NONE) {
+        const float4 z = raw_value(g[q][e]);
+        y = make_float4(y.x * silu_f(z.x), y.y * silu_f(z.y), y.z * silu_f(z.z), y.w * silu_f(z.w));
+      }
+      store4(out + t[q] * (size_t)H * n + hc[q] + 4 * e, y);
     }
   }
 }
@@ -746,8 +898,9 @@ StateArgs state_args(void* state, long long row, int num_slots, int carry, const
                      const void* x, int S, int W) {
   return StateArgs{(float*)state, row, num_slots, carry, (const int*)slots, (const int*)cu_q, (const int*)kv_lens, (const float*)x, S, W};
 }
-int check_state(long long row, int num_slots, int carry, int S, int W) {
-  return row <= 0 || row % 4 || num_slots <= 0 || carry < 0 || carry % 4 || S <= 0 || W <= 0 || W % 8 || carry + W > row ? -1 : 0;
+// W columns in each of `rows` rows that are carried on
+int check_state(long long row, int num_slots, int carry, int S, int W, int rows = 1) {
+  return row <= 0 || row % 4 || num_slots <= 0 || carry < 0 || carry % 4 || S <= 0 || W <= 0 || W % 8 || carry + (long long)rows * W > row ? -1 : 0;
 }
 template <typename T>
 Proj<T> proj_of(const void* slabs, long long stride, int P, const void* rows, long long ld) {
@@ -763,22 +916,49 @@ int allow_smem(K kernel, size_t smem, size_t& configured) {
   return (int)e;
 }
 
-template <typename T, int NV, int NT>
+template <typename T, int NV, int NT, int RULE>
 int launch_step(const StepArgs<T>& a, cudaStream_t stream, bool pdl) {
-  const int rows = NT / (a.n / 4);
-  const size_t smem = (size_t)(6 * a.n + a.rank + rows * a.n) * sizeof(float);
+  const int rows = NT / (a.m / 4);
+  const size_t smem = (size_t)(4 * a.n + 2 * a.m + a.rank + rows * a.m) * sizeof(float);
   static size_t configured = 48 * 1024;
-  if (int rc = allow_smem(state_step_kernel<T, NV, NT>, smem, configured)) return rc;
-  return (int)prism_launch(state_step_kernel<T, NV, NT>, dim3(a.H, a.st.S), dim3(NT), smem, stream, pdl, a);
+  if (int rc = allow_smem(state_step_kernel<T, NV, NT, RULE>, smem, configured)) return rc;
+  return (int)prism_launch(state_step_kernel<T, NV, NT, RULE>, dim3(a.H, a.st.S), dim3(NT), smem, stream, pdl, a);
+}
+// As many float4s of the state per thread as its key rows need.
+template <typename T, int RULE>
+int launch_step_sized(const StepArgs<T>& a, cudaStream_t stream, bool pdl) {
+  auto rows_of = [&](int threads) { return threads / (a.m / 4); };
+  if (rows_of(128) * 8 >= a.n) return launch_step<T, 8, 128, RULE>(a, stream, pdl);
+  if (rows_of(256) * 16 >= a.n) return launch_step<T, 16, 256, RULE>(a, stream, pdl);
+  return launch_step<T, 0, 256, RULE>(a, stream, pdl);
 }
 
-template <typename T, int KL, bool SLABS>
+template <typename T, int KL, bool SLABS, int RULE>
 int launch_scan(const ScanArgs<T>& a, cudaStream_t stream, bool pdl) {
   const size_t smem = (size_t)(2 * ScanTile<KL>::FLOATS + 2 * ScanTile<KL>::TB * SCAN_COLS) * sizeof(float);
   static size_t configured = 48 * 1024;
-  if (int rc = allow_smem(state_scan_kernel<T, KL, SLABS>, smem, configured)) return rc;
-  const dim3 grid(a.H * ((a.n + SCAN_COLS - 1) / SCAN_COLS), a.st.S);
-  return (int)prism_launch(state_scan_kernel<T, KL, SLABS>, grid, dim3(SCAN_THREADS), smem, stream, pdl, a);
+  if (int rc = allow_smem(state_scan_kernel<T, KL, SLABS, RULE>, smem, configured)) return rc;
+  const dim3 grid(a.H * ((a.m + SCAN_COLS - 1) / SCAN_COLS), a.st.S);
+  return (int)prism_launch(state_scan_kernel<T, KL, SLABS, RULE>, grid, dim3(SCAN_THREADS), smem, stream, pdl, a);
+}
+template <typename T, int RULE>
+int launch_scan_sized(const ScanArgs<T>& a, cudaStream_t stream, bool pdl) {
+  auto sized = [&](auto slabs) -> int {
+    constexpr bool SLABS = decltype(slabs)::value;
+    if (a.n <= 64) return launch_scan<T, 4, SLABS, RULE>(a, stream, pdl);
+    if (a.n <= 128) return launch_scan<T, 8, SLABS, RULE>(a, stream, pdl);
+    return launch_scan<T, 16, SLABS, RULE>(a, stream, pdl);
+  };
+  return a.p.slabs ? sized(std::true_type()) : sized(std::false_type());
+}
+
+template <typename T>
+int launch_conv(const StateArgs& st, const void* x, const void* w, void* out, int taps, int max_len, cudaStream_t stream, bool pdl) {
+  ConvArgs<T> a{st, (const T*)x, (const T*)w, (T*)out, taps};
+  const dim3 grid((max_len + CONV_CHUNK - 1) / CONV_CHUNK, (st.W / 4 + 255) / 256, st.S), block(256);
+  if (taps <= 4) return (int)prism_launch(short_conv_kernel<T, 4>, grid, block, 0, stream, pdl, a);
+  if (taps <= 8) return (int)prism_launch(short_conv_kernel<T, 8>, grid, block, 0, stream, pdl, a);
+  return (int)prism_launch(short_conv_kernel<T, 16>, grid, block, 0, stream, pdl, a);
 }
 
 template <typename T>
@@ -851,11 +1031,28 @@ PRISM_API int prism_state_step(int f32, void* state, long long row, int num_slot
   auto run = [&](auto type) -> int {
     using T = decltype(type);
     StepArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), proj_of<T>(w1_slabs, w1_stride, w1_P, w1_rows, w1_ld), (const T*)w2,
-                  (const T*)w0, (const T*)u, (const T*)norm, (T*)out, S, H, n, n_real, rank, eps};
-    // float4s of the state per thread
-    if (n <= 64) return launch_step<T, 8, 128>(a, s, pdl != 0);
-    if (n <= 128) return launch_step<T, 16, 256>(a, s, pdl != 0);
-    return launch_step<T, 0, 256>(a, s, pdl != 0);
+                  (const T*)w0, (const T*)u, (const T*)norm, (T*)out, S, H, n, n, n_real, rank, eps};
+    return launch_step_sized<T, RULE_BONUS>(a, s, pdl != 0);
+  };
+  return f32 ? run(float()) : run(bf16());
+}
+
+// The forget rule, one token per sequence: p [S][ld] = [H n queries | H n gates | H m values] as fp32 slabs or rows; bias and lower
+// [H n] of the gates, norm [m]; out [S][H m].  n and m multiples of 16, at most 256.
+PRISM_API int prism_forget_step(int f32, void* state, long long row, int num_slots, int carry, const void* slots, const void* kv_lens, int S,
+                                const void* p_slabs, long long p_stride, int p_P, const void* p_rows, long long p_ld, const void* bias,
+                                const void* lower, const void* norm, void* out, int H, int n, int m, int m_real, float eps, void* stream, int pdl) {
+  if (S <= 0) return 0;
+  if (int rc = check_state(row, num_slots, carry, S, 8, 0)) return rc;
+  if (H <= 0 || n <= 0 || n % 16 || n > 256 || m <= 0 || m % 16 || m > 256 || m_real <= 0 || m_real > m || (long long)H * n * m > carry || S > 65535) return -2;
+  if ((!p_slabs && !p_rows) || p_ld % 4 || p_ld < (long long)H * (2 * n + m)) return -3;
+  const StateArgs st = state_args(state, row, num_slots, carry, slots, nullptr, kv_lens, nullptr, S, 0);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  auto run = [&](auto type) -> int {
+    using T = decltype(type);
+    StepArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), Proj<T>{}, nullptr, (const T*)bias, (const T*)lower, (const T*)norm, (T*)out,
+                  S, H, n, m, m_real, 0, eps};
+    return launch_step_sized<T, RULE_FORGET>(a, s, pdl != 0);
   };
   return f32 ? run(float()) : run(bf16());
 }
@@ -873,30 +1070,57 @@ PRISM_API int prism_state_scan(int f32, void* state, long long row, int num_slot
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   auto run = [&](auto type) -> int {
     using T = decltype(type);
-    ScanArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), (const float*)decay, (const T*)u, (float*)o, T_rows, H, n};
-    auto sized = [&](auto slabs) -> int {
-      constexpr bool SLABS = decltype(slabs)::value;
-      if (n <= 64) return launch_scan<T, 4, SLABS>(a, s, pdl != 0);
-      if (n <= 128) return launch_scan<T, 8, SLABS>(a, s, pdl != 0);
-      return launch_scan<T, 16, SLABS>(a, s, pdl != 0);
-    };
-    return p_slabs ? sized(std::true_type()) : sized(std::false_type());
+    ScanArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), (const float*)decay, (const T*)u, nullptr, (float*)o, T_rows, H, n, n};
+    return launch_scan_sized<T, RULE_BONUS>(a, s, pdl != 0);
   };
   return f32 ? run(float()) : run(bf16());
 }
 
-// out [T][H n] = o / rms(o) * norm * silu(gate) per head; the gate is block 3 of p.
+// The forget rule over prompts and portions; p [T][ld], bias and lower as in prism_forget_step, o [T][H m] fp32.
+PRISM_API int prism_forget_scan(int f32, void* state, long long row, int num_slots, int carry, const void* slots, const void* cu_q,
+                                const void* kv_lens, int S, const void* p_slabs, long long p_stride, int p_P, const void* p_rows, long long p_ld,
+                                const void* bias, const void* lower, void* o, int T_rows, int H, int n, int m, void* stream, int pdl) {
+  if (T_rows <= 0) return 0;
+  if (int rc = check_state(row, num_slots, carry, S, 8, 0)) return rc;
+  if (H <= 0 || n <= 0 || n % 16 || n > 256 || m <= 0 || m % 16 || m > 256 || (long long)H * n * m > carry || !cu_q || S > 65535) return -2;
+  if ((!p_slabs && !p_rows) || p_ld % 4 || p_ld < (long long)H * (2 * n + m)) return -3;
+  const StateArgs st = state_args(state, row, num_slots, carry, slots, cu_q, kv_lens, nullptr, S, 0);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  auto run = [&](auto type) -> int {
+    using T = decltype(type);
+    ScanArgs<T> a{st, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), nullptr, (const T*)lower, (const T*)bias, (float*)o, T_rows, H, n, m};
+    return launch_scan_sized<T, RULE_FORGET>(a, s, pdl != 0);
+  };
+  return f32 ? run(float()) : run(bf16());
+}
+
+// out [T][W] = x + causal convolution of x with w [taps][W] on every channel, for prompts and portions (max_len: the most tokens of
+// a sequence).  The state's carry is taps - 1 rows of W fp32, oldest first.  taps at most 16.
+PRISM_API int prism_short_conv(int f32, void* state, long long row, int num_slots, int carry, const void* slots, const void* cu_q,
+                               const void* kv_lens, int S, int W, const void* x, const void* w, void* out, int taps, int max_len, void* stream,
+                               int pdl) {
+  if (max_len <= 0) return 0;
+  if (taps < 1 || taps > 16 || !cu_q || S > 65535) return -2;
+  if (int rc = check_state(row, num_slots, carry, S, W, taps - 1)) return rc;
+  const StateArgs st = state_args(state, row, num_slots, carry, slots, cu_q, kv_lens, nullptr, S, W);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  return f32 ? launch_conv<float>(st, x, w, out, taps, max_len, s, pdl != 0) : launch_conv<bf16>(st, x, w, out, taps, max_len, s, pdl != 0);
+}
+
+// out [T][H n] = o / rms(o) * norm * silu(gate) per head; the gate is block 3 of p.  Without p: no gate, and norm
+// [n] holds for every head.
 PRISM_API int prism_head_norm_gate(int f32, const void* o, const void* p_slabs, long long p_stride, int p_P, const void* p_rows,
                                    long long p_ld, const void* norm, void* out, int T_rows, int H, int n, int n_real, float eps,
                                    void* stream, int pdl) {
   if (T_rows <= 0) return 0;
-  if (H <= 0 || n <= 0 || n % 16 || n > 256 || n_real <= 0 || n_real > n || (!p_slabs && !p_rows) || p_ld % 4) return -1;
+  if (H <= 0 || n <= 0 || n % 16 || n > 256 || n_real <= 0 || n_real > n || p_ld % 4) return -1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   auto run = [&](auto type, auto lanes) -> int {
     using T = decltype(type);
     constexpr int L = decltype(lanes)::value, PER_CTA = 8 * (32 / L) * 4;
     const dim3 grid((unsigned)(((long long)T_rows * H + PER_CTA - 1) / PER_CTA));
-    return (int)prism_launch(p_slabs ? head_norm_gate_kernel<T, L, true> : head_norm_gate_kernel<T, L, false>, grid, dim3(256), 0, s, pdl != 0,
+    auto* kernel = p_slabs ? head_norm_gate_kernel<T, L, GATE_SLABS> : (p_rows ? head_norm_gate_kernel<T, L, GATE_ROWS> : head_norm_gate_kernel<T, L, GATE_NONE>);
+    return (int)prism_launch(kernel, grid, dim3(256), 0, s, pdl != 0,
                              (const float*)o, proj_of<T>(p_slabs, p_stride, p_P, p_rows, p_ld), (const T*)norm, (T*)out, T_rows, H, n, n_real, eps);
   };
   auto sized = [&](auto type) -> int {

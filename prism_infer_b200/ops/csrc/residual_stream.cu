@@ -5,10 +5,12 @@
 //   pass      x = sum of the loop projection's slabs + step     (input of a looped section)
 //   layer     x += mult * (gate_a * a + gate_b * b)             (two parallel sublayers, either may be absent)
 //   layer     x += norm(a) * w                                  (a norm behind the sublayer)
+//   average   x = sum of weighted earlier results and this one  (depth average behind a layer)
 // and what the next operation reads of it: the RMS-normalised row (with a weight, or with a scalar gain that the
 // next GEMM's epilogue applies), or the row itself (the loop projection's input, with the embedding beside it).
 // a and b come as fp32 split-K slabs, summed here in a fixed order, or as rows of the compute type; a may also be
-// the weighted sum of several (token, expert) rows, and of the stream's own row.
+// the weighted sum of several (token, expert) rows, and of the stream's own row.  In a decode step the normalised row may also
+// pass through the causal convolution in front of the next mixer, whose earlier rows are in the sequence's state slot.
 #include "common.cuh"
 
 PRISM_DEFINE_TU_STATUS(stream)
@@ -56,6 +58,19 @@ struct Branch {
   const float* self_w;     // [T]: weight of the stream's row in the sum (null: none)
 };
 
+// Causal convolution of one token per sequence over the normalised rows, channel by channel.  The rows carried on, oldest
+// first, are in the slot's version of the tokens so far (version c & 1 at c tokens), from element `carry` on.
+template <typename T>
+struct ConvStep {
+  const T* w;              // [taps][W], the last tap meets the row itself (null: no convolution)
+  int taps;
+  float* state;            // [slots][2][row]
+  long long row;
+  int num_slots, carry;
+  const int* slots;        // [T], < 0: no state
+  const int* kv_lens;      // [T] tokens up to and including this one
+};
+
 template <typename T>
 struct StreamArgs {
   float* x;                // [T][W] the stream
@@ -77,6 +92,12 @@ struct StreamArgs {
   long long embed_ld;
   int W, W_real;           // padded and real width: the padding columns are zero and do not enter the mean
   float eps;
+  // Results of the layers so far [hist_n][T][W] at a stride of hist_stride; this one is stored behind them (null: none kept).
+  float* hist;
+  long long hist_stride;
+  const float* hist_w;     // [hist_n + 1]: x becomes the weighted sum of all of them (null: x stays this one)
+  int hist_n;
+  ConvStep<T> conv;
 };
 
 // Columns i .. i + 3 of row r of a branch, slabs summed.
@@ -217,6 +238,22 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
     } else if (a.embed_out != nullptr) {
       store4(a.embed_out + t * a.embed_ld + i, F4{{0.0f, 0.0f, 0.0f, 0.0f}});
     }
+    if (a.hist != nullptr) {
+      const float* h0 = a.hist + t * a.W + i;
+      store4(a.hist + (size_t)a.hist_n * a.hist_stride + t * a.W + i, acc[u]);
+      if (a.hist_w != nullptr) {
+        const float own = __ldg(a.hist_w + a.hist_n);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[u].v[e] *= own;
+#pragma unroll 8
+        for (int j = 0; j < a.hist_n; ++j) {
+          const float w = __ldg(a.hist_w + j);
+          const F4 h = load4(h0 + (size_t)j * a.hist_stride);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[u].v[e] = fmaf(w, h.v[e], acc[u].v[e]);
+        }
+      }
+    }
     store4(a.x + t * a.W + i, acc[u]);
     if (a.raw_out != nullptr) store4(a.raw_out + t * a.raw_ld + i, acc[u]);
 #pragma unroll
@@ -224,6 +261,18 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
   }
   if (a.norm_out == nullptr) return;
   const float inv = 1.0f / sqrtf(block_sum(ss, red[1]) / (float)a.W_real + a.eps);
+  const float* carry_old = nullptr;
+  float* carry_new = nullptr;
+  if (a.conv.w != nullptr) {
+    const int slot = a.conv.slots[t], end = a.conv.kv_lens[t];
+    if (slot >= a.conv.num_slots) {
+      if (threadIdx.x == 0) prism_report(PRISM_ERR_BOUNDS, 3);
+    } else if (slot >= 0 && end > 0) {
+      float* base = a.conv.state + (size_t)slot * 2 * a.conv.row + a.conv.carry;
+      if (end > 1) carry_old = base + (size_t)((end - 1) & 1) * a.conv.row;
+      carry_new = base + (size_t)(end & 1) * a.conv.row;
+    }
+  }
 #pragma unroll
   for (int u = 0; u < U; ++u) {
     const int i = i0 + u * step;
@@ -235,6 +284,23 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
       const F4 w = load4(a.norm_w + i);
 #pragma unroll
       for (int e = 0; e < 4; ++e) v.v[e] *= a.w_offset + w.v[e];
+    }
+    if (a.conv.w != nullptr) {     // what a row of the compute type would hold meets the taps
+      const int last = a.conv.taps - 1;
+      F4 o = load4(a.conv.w + (size_t)last * a.W + i);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (sizeof(T) == 2) v.v[e] = bf16_round(v.v[e]);
+        o.v[e] = fmaf(o.v[e], v.v[e], v.v[e]);
+      }
+      for (int j = 0; j < last; ++j) {
+        const F4 c = carry_old ? load4(carry_old + (size_t)j * a.W + i) : F4{{0.0f, 0.0f, 0.0f, 0.0f}}, w = load4(a.conv.w + (size_t)j * a.W + i);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o.v[e] = fmaf(w.v[e], c.v[e], o.v[e]);
+        if (carry_new && j > 0) store4(carry_new + (size_t)(j - 1) * a.W + i, c);
+      }
+      if (carry_new && last > 0) store4(carry_new + (size_t)(last - 1) * a.W + i, v);
+      v = o;
     }
     store4(a.norm_out + t * a.norm_ld + i, v);
   }
@@ -289,8 +355,15 @@ int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* ta
                   long long b_stride, int b_P, const void* b_rows, long long b_ld, const void* b_gate, long long gate_ld,
                   const void* a_pos, const void* a_weight, int a_K, const void* a_post, const void* a_self, float mult,
                   float emb_mult, float w_offset, const void* bias, const void* norm_w, void* norm_out, long long norm_ld, void* raw_out, long long raw_ld,
-                  void* embed_out, long long embed_ld, int W, int W_real, float eps, cudaStream_t stream, bool pdl) {
+                  void* embed_out, long long embed_ld, int W, int W_real, float eps, void* hist, long long hist_stride, const void* hist_w,
+                  int hist_n, const void* conv_w, int taps, void* state, long long state_row, int num_slots, int carry, const void* slots,
+                  const void* kv_lens, cudaStream_t stream, bool pdl) {
   StreamArgs<T> a;
+  a.hist = (float*)hist;
+  a.hist_stride = hist_stride;
+  a.hist_w = (const float*)hist_w;
+  a.hist_n = hist_n;
+  a.conv = ConvStep<T>{(const T*)conv_w, taps, (float*)state, state_row, num_slots, carry, (const int*)slots, (const int*)kv_lens};
   a.x = (float*)x;
   a.keep = keep;
   a.ids = (const long long*)ids;
@@ -330,6 +403,9 @@ int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* ta
 
 // f32: 1 = table, rows, gates, bias and outputs are fp32, 0 = bf16.  W a multiple of 8; every row stride a
 // multiple of 4 elements.  a_self [T] (with a branch a): weight of the old stream row in it.  w_offset: added to norm weights.
+// hist: fp32 results of hist_n layers so far at hist_stride elements from one another, this one goes behind them; hist_w
+// [hist_n + 1] fp32: the stream becomes their weighted sum.  conv_w [taps][W] (with norm_out, one token per sequence): the
+// convolution of the normalised row with the taps - 1 rows in the state slots [num_slots][2][state_row] from `carry` on.
 PRISM_API int prism_stream_update(int f32, int T, void* x, int keep, const void* ids, const void* table, long long vocab,
                                   const void* a_slabs, long long a_stride, int a_P, const void* a_rows, long long a_ld,
                                   const void* a_gate, const void* b_slabs, long long b_stride, int b_P, const void* b_rows,
@@ -337,18 +413,26 @@ PRISM_API int prism_stream_update(int f32, int T, void* x, int keep, const void*
                                   const void* a_weight, int a_K, const void* a_post, const void* a_self, float mult,
                                   float emb_mult, float w_offset, const void* bias,
                                   const void* norm_w, void* norm_out, long long norm_ld, void* raw_out, long long raw_ld, void* embed_out,
-                                  long long embed_ld, int W, int W_real, float eps, void* stream, int pdl) {
+                                  long long embed_ld, int W, int W_real, float eps, void* hist, long long hist_stride, const void* hist_w,
+                                  int hist_n, const void* conv_w, int taps, void* state, long long state_row, int num_slots, int carry,
+                                  const void* slots, const void* kv_lens, void* stream, int pdl) {
   if (T <= 0) return 0;
+  if (hist != nullptr && (hist_n < 0 || hist_stride < (long long)T * W)) return -4;
+  if (conv_w != nullptr && (!norm_out || taps < 1 || !state || !slots || !kv_lens || num_slots <= 0 || carry < 0 || carry % 4 || state_row % 4 ||
+                            carry + (long long)(taps - 1) * W > state_row))
+    return -5;
   if (W <= 0 || W % 8 || W_real <= 0 || W_real > W || W > 32768) return -1;
   if ((a_ld | b_ld | gate_ld | norm_ld | raw_ld | embed_ld) % 4) return -2;
   if ((a_pos != nullptr && (a_K <= 0 || !a_weight || a_gate)) || ((a_pos || a_post || a_self) && !a_slabs && !a_rows)) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return f32 ? launch_stream<float>(T, x, keep, ids, table, vocab, a_slabs, a_stride, a_P, a_rows, a_ld, a_gate, b_slabs, b_stride,
                                     b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, a_self, mult, emb_mult, w_offset, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,
-                                    embed_ld, W, W_real, eps, s, pdl != 0)
+                                    embed_ld, W, W_real, eps, hist, hist_stride, hist_w, hist_n, conv_w, taps, state, state_row,
+                                    num_slots, carry, slots, kv_lens, s, pdl != 0)
              : launch_stream<bf16>(T, x, keep, ids, table, vocab, a_slabs, a_stride, a_P, a_rows, a_ld, a_gate, b_slabs, b_stride,
                                    b_P, b_rows, b_ld, b_gate, gate_ld, a_pos, a_weight, a_K, a_post, a_self, mult, emb_mult, w_offset, bias, norm_w, norm_out, norm_ld, raw_out, raw_ld, embed_out,
-                                   embed_ld, W, W_real, eps, s, pdl != 0);
+                                   embed_ld, W, W_real, eps, hist, hist_stride, hist_w, hist_n, conv_w, taps, state, state_row,
+                                    num_slots, carry, slots, kv_lens, s, pdl != 0);
 }
 
 // g [T][D] = gelu_tanh(z) * table[ids[t]][offset ..]; z as fp32 slabs or rows of the compute type.  D, table_ld and offset

@@ -758,7 +758,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   extern __shared__ uint8_t pre_raw[];
   const WinArgs<bf16>& a = p.w;
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(pre_raw) + 1023) & ~uintptr_t(1023));
-  const int qa = a.dq > 64 ? 2 : 1, va = a.dv > 64 ? 2 : 1;          // 64-column atoms of a key / value head
+  const int qa = (a.dq + 63) >> 6, va = a.dv > 64 ? 2 : 1;           // 64-column atoms of a key / value head
   const int q_bytes = qa * Q_ATOM, k_bytes = qa * KV_ATOM, v_bytes = va * KV_ATOM;
   const int stage_bytes = p.k_maps * k_bytes + v_bytes;
   uint8_t* q_s = smem;                                               // [2 streams][qa][128 rows]
@@ -875,7 +875,7 @@ window_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           const uint64_t kd = k_desc + (uint64_t)((uint32_t)(st_next * stage_bytes) >> 4);
           const uint32_t d = s_tmem + (sc & 1) * PKT;
 #pragma unroll
-          for (int k = 0; k < 8; ++k)
+          for (int k = 0; k < 12; ++k)
             if (k < ksteps)
               tc_mma_f16(d, q_desc + ((k >> 2) * (Q_ATOM >> 4) + 2 * (k & 3)), kd + ((k >> 2) * (KV_ATOM >> 4) + 2 * (k & 3)), idesc_s, k != 0);
           tc_commit(&s_full[s * 2 + (sc & 1)]);
@@ -1328,14 +1328,15 @@ PRISM_API int prism_window_decode(const void* q, const void* cache, const void* 
   return launch_decode<1, 32, 0>(a, S, blocks, s, p);
 }
 
-// Prompts and portions (cu_q: token offsets of the sequences), head widths up to 128, pages of a multiple of 8 rows.
+// Prompts and portions (cu_q: token offsets of the sequences), values up to 128 wide, keys up to 128 (one map: 192), pages of a
+// multiple of 8 rows.
 PRISM_API int prism_window_prefill_tc(const void* q, const void* cache, const void* block_tables, const void* cu_q, const void* kv_lens,
                                       const void* gate, const void* sink, void* out, long long out_ld, int T, int S, int max_q_len, int H, int G, int maps,
                                       int dq, int dv, int vdim, int R, int page, int max_blocks, int num_blocks, int window, int keep,
                                       float scale, float lam, float gain, float eps, float cap, void* stream, int pdl) {
   if (T <= 0 || S <= 0 || max_q_len <= 0) return 0;
   if (int rc = check_sizes(H, G, maps, dq, dv, vdim, R, page, max_blocks, window, keep, sink, cap)) return rc;
-  if (dq > 128 || dv > 128 || page % 8 || !cu_q || num_blocks <= 0 || !(scale > 0.0f) || out_ld % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return -3;
+  if (dq > (maps == 1 ? 192 : 128) || dv > 128 || page % 8 || !cu_q || num_blocks <= 0 || !(scale > 0.0f) || out_ld % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) return -3;
   PrefillArgs p;
   p.w = win_args<bf16>(q, cache, block_tables, cu_q, kv_lens, gate, sink, out, out_ld, H, G, maps, dq, dv, vdim, R, page, max_blocks, num_blocks,
                        window, keep, scale, lam, gain, eps, cap);
@@ -1355,7 +1356,7 @@ PRISM_API int prism_window_prefill_tc(const void* q, const void* cache, const vo
   rc = prism_make_head_tensor_map(base + (size_t)G * maps * dq, (unsigned long long)rows, (unsigned)G, (unsigned)dv, (unsigned long long)R,
                                   (unsigned)p.box, &tv);
   if (rc) return rc;
-  const int qa = dq > 64 ? 2 : 1, va = dv > 64 ? 2 : 1;
+  const int qa = (dq + 63) / 64, va = dv > 64 ? 2 : 1;
   const size_t fixed = 1024 + (size_t)2 * qa * Q_ATOM + 21 * 8 + 16 + 4 * PT * sizeof(float);
   const size_t stage = (size_t)(maps * qa + va) * KV_ATOM;
   p.stages = 4;

@@ -20,6 +20,7 @@ from . import SM_COUNT, KVCache, _p, _pdl, _s, choose_splits, linear, linear_par
 ACTS = {None: 0, "gelu_tanh": 1, "gelu": 2, "sigmoid": 3, "softcap": 4, "decay": 5}
 MAX_SPLITS = 64
 MAX_LATENT = 1024       # widest latent row of the attention kernels
+NO_WINDOW = 1 << 30
 FLASH_MAX_HEAD = 128    # widest head of the tcgen05 prefill attention
 EXPAND_MAX_SCRATCH_BYTES = 2 << 30
 
@@ -137,12 +138,15 @@ def stream_update(x: torch.Tensor, width: int, eps: float, *, keep: bool, ids: O
                   table: Optional[torch.Tensor] = None, a: Optional[Branch] = None, b: Optional[Branch] = None, mult: float = 1.0,
                   bias: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, norm_out: Optional[torch.Tensor] = None,
                   raw_out: Optional[torch.Tensor] = None, embed_out: Optional[torch.Tensor] = None, embed_mult: float = 1.0,
-                  norm_offset: float = 0.0) -> None:
+                  norm_offset: float = 0.0, history: Optional[torch.Tensor] = None, depth: int = 0,
+                  depth_weight: Optional[torch.Tensor] = None, conv=None) -> None:
     """``x [T, W]`` (fp32, in place) ``= (x if keep) + embed_mult * table[ids] + mult * (a + b) + bias``, and what follows reads of
     it: ``norm_out`` the rows over their root mean square (``width`` real columns, the rest are zero), times
     ``norm_weight`` if given, ``raw_out`` the rows themselves, ``embed_out`` the embedding rows, each in its own type.
     Only ``a`` may consist of pairs or be normalised (``Branch.post_norm``).  ``norm_offset`` is added to the norm weights (1:
-    weights stored around zero)."""
+    weights stored around zero).  ``history [n, T, W]`` (fp32): the new ``x`` is kept as its row ``depth``, and with
+    ``depth_weight [depth + 1]`` (fp32) becomes the weighted sum of rows ``0 .. depth`` before anything else reads it.  ``conv``
+    (``recurrent.ConvStep``, one token per sequence): ``norm_out`` goes through it."""
     assert b is None or (b.pos is None and b.post_norm is None and b.self_weight is None)
     T, W = x.shape
     if not x.is_cuda:
@@ -162,12 +166,20 @@ def stream_update(x: torch.Tensor, width: int, eps: float, *, keep: bool, ids: O
             new += emb
             if embed_out is not None:
                 embed_out.copy_(emb)
+        if history is not None:
+            history[depth].copy_(new)
+            if depth_weight is not None:
+                new = torch.einsum("j,jtw->tw", depth_weight, history[:depth + 1])
         x.copy_(new)
         if raw_out is not None:
             raw_out.copy_(new)
         if norm_out is not None:
             n = new / torch.sqrt(new.pow(2).sum(-1, keepdim=True) / width + eps)
             norm_out.copy_(n if norm_weight is None else n * (norm_offset + norm_weight.float()))
+            if conv is not None:
+                from .recurrent import short_conv
+
+                norm_out.copy_(short_conv(norm_out, conv.weight, conv.spec, conv.state))
         return
     kinds = [t.dtype for t in (table, bias, norm_weight, norm_out, raw_out, embed_out) if t is not None]
     for branch in (a, b):
@@ -191,26 +203,63 @@ def stream_update(x: torch.Tensor, width: int, eps: float, *, keep: bool, ids: O
     pairs = a is not None and a.pos is not None
     extra = (_p(a.pos) if pairs else None, _p(a.weight) if pairs else None, a.pos.shape[1] if pairs else 0,
              _p(a.post_norm) if a is not None else None, _p(a.self_weight) if a is not None else None)
+    assert history is None or (history.dtype == torch.float32 and history.shape[1:] == x.shape and history[depth].is_contiguous())
+    assert depth_weight is None or (depth_weight.dtype == torch.float32 and depth_weight.shape == (depth + 1,) and history is not None)
+    assert conv is None or (conv.weight.dtype == norm_out.dtype and conv.weight.shape == (conv.spec.taps, W))
+    behind = (_p(history), history.stride(0) if history is not None else 0, _p(depth_weight), depth,
+              *(conv.args() if conv is not None else (None, 0, None, 0, 0, 0, None, None)))
     native.call("prism_stream_update", 1 if kinds[0] == torch.float32 else 0, T, _p(x), 1 if keep else 0, _p(ids), _p(table),
                 table.shape[0] if table is not None else 0, *flat, gate_ld, *extra, float(mult), float(embed_mult), float(norm_offset), _p(bias), _p(norm_weight), _p(norm_out), ld(norm_out),
-                _p(raw_out), ld(raw_out), _p(embed_out), ld(embed_out), W, width, float(eps), _s(),
+                _p(raw_out), ld(raw_out), _p(embed_out), ld(embed_out), W, width, float(eps), *behind, _s(),
                 0 if ids is not None else _pdl())  # the first kernel of a step may follow a copy: full dependency
 
 
 # -------------------------------------------------------------------------------- latent attention
 @dataclass
+class Rotary:
+    """Rotation of neighbouring columns: pair ``i`` of a row at position ``p`` turns by ``p * inv_freq[i]``, sine and cosine times
+    ``amplitude``.  ``start``: first of the ``dims`` columns in a query head, ``row_start`` in a cached row."""
+
+    inv_freq: torch.Tensor   # [dims / 2] fp32
+    dims: int
+    start: int
+    row_start: int
+    amplitude: float = 1.0
+
+    def apply(self, x: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+        """``x [T, ..., dims]`` turned, fp32 (the plain statement)."""
+        a = (positions.float()[:, None] * self.inv_freq[None]).view(x.shape[0], *([1] * (x.dim() - 2)), -1)
+        c, s = a.cos() * self.amplitude, a.sin() * self.amplitude
+        u, v = x[..., 0::2].float(), x[..., 1::2].float()
+        return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
+
+    def args(self, positions: torch.Tensor) -> tuple:
+        assert positions.dtype == torch.int32 and positions.is_contiguous() and self.inv_freq.dtype == torch.float32
+        return _p(self.inv_freq), _p(positions), float(self.amplitude)
+
+
+NO_ROTARY = (None, None, 1.0)
+
+
+@dataclass
 class LatentWeights:
     """What a latent-attention layer multiplies latents with.  ``uk [H * dq, Rc]`` and ``uv [H * dv, Rc]`` are the two
-    halves of ``ukv``; ``norm [R]`` is the latent's RMS-norm weight.  ``dq`` / ``dv`` are the padded head widths, ``Rc``
-    the padded latent width; padding is zero."""
+    halves of ``ukv``; ``norm [R]`` is the latent's RMS-norm weight (padded to 16 where the layer's latents are made by
+    ``latent_prepare``; none: another layer's are read).  ``dq`` / ``dv`` are the padded head widths, ``Rc`` the padded row
+    width; padding is zero.  A rotated key part that all heads share lies behind the latent in the row (``rot``); ``uk`` has an
+    identity block for it, so that a query's rotated columns meet it.  A query sees the ``window`` newest rows."""
 
     heads: int
     dq: int
     dv: int
     rank: int
     scale: float
-    norm: torch.Tensor
+    norm: Optional[torch.Tensor]
     ukv: torch.Tensor
+    rot: Optional[Rotary] = None
+    window: int = NO_WINDOW
+    q_rank: int = 0
+    q_norm: Optional[torch.Tensor] = None    # [q_rank padded to 16] of the query latent
 
     @property
     def uk(self) -> torch.Tensor:
@@ -220,12 +269,78 @@ class LatentWeights:
     def uv(self) -> torch.Tensor:
         return self.ukv[self.heads * self.dq:]
 
+    @property
+    def value_cols(self) -> int:
+        """Columns of a row that values are made of, in whole tiles."""
+        return -(-self.rank // 64) * 64
+
+    def connect_rotary(self) -> None:
+        """The identity blocks of ``uk``."""
+        if self.rot is not None:
+            uk, i = self.uk.view(self.heads, self.dq, -1), torch.arange(self.rot.dims, device=self.ukv.device)
+            uk[:, self.rot.start + i, self.rot.row_start + i] = 1.0
+
+
+def latent_prepare(y: Branch, lw: LatentWeights, eps: float, positions: torch.Tensor, slots: torch.Tensor, cache: KVCache,
+                   layer: int) -> torch.Tensor:
+    """From the stacked projection ``y [T, query latent | key latent | shared key part]`` (sections padded to 16): the normalised
+    query latent ``[T, Qp]``; normalised key latent and rotated key part go to the cache rows at flat ``slots`` (negative = skip).
+    A layer that reads another's rows projects the query latent alone."""
+    src = y.slabs if y.slabs is not None else y.rows
+    T, Qp, Cp = src.shape[-2], lw.q_norm.shape[0], lw.norm.shape[0] if lw.norm is not None else 0
+    pages = cache.latent(layer)
+    if not src.is_cuda:
+        v = y.value()
+
+        def normed(z, real, weight):
+            return z / torch.sqrt(z.pow(2).sum(-1, keepdim=True) / real + eps) * weight.float()
+
+        if Cp:
+            row = torch.zeros((T, pages.shape[-1]))
+            row[:, :Cp] = normed(v[:, Qp:Qp + Cp], lw.rank, lw.norm)
+            if lw.rot is not None:
+                row[:, Cp:Cp + lw.rot.dims] = lw.rot.apply(v[:, Qp + Cp:Qp + Cp + lw.rot.dims], positions)
+            at = slots[slots >= 0]
+            pages[at // cache.page, at % cache.page] = row[slots >= 0].to(pages.dtype)
+        return normed(v[:, :Qp], lw.q_rank, lw.q_norm).to(lw.q_norm.dtype)
+    out = torch.empty((T, Qp), dtype=lw.q_norm.dtype, device=src.device)
+    dims = lw.rot.dims if lw.rot is not None else 0
+    assert slots.dtype == torch.int64 and src.shape[-1] >= Qp + Cp + (-(-dims // 4) * 4 if Cp else 0) and (lw.rot is None or lw.rot.row_start == Cp or not Cp)
+    native.call("prism_latent_prepare", 1 if out.dtype == torch.float32 else 0, *_branch_args(y), _p(lw.q_norm), _p(lw.norm), _p(out), _p(pages),
+                _p(slots), cache.num_blocks * cache.page, *(lw.rot.args(positions) if lw.rot is not None else NO_ROTARY), T, lw.q_rank, Qp, lw.rank,
+                Cp, dims, pages.shape[-1], float(eps), _s(), _pdl())
+    return out
+
+
+def _branch_args(b: Branch) -> tuple:
+    """(slabs, stride between them, their number, rows, stride between rows)"""
+    s, r = b.slabs, b.rows
+    assert s is None or s.stride(2) == 1
+    return (_p(s), s.stride(0) if s is not None else 0, s.shape[0] if s is not None else 0, _p(r), s.stride(1) if s is not None else r.stride(0))
+
+
+def rotate_queries(q: Branch, lw: LatentWeights, positions: torch.Tensor) -> torch.Tensor:
+    """Queries ``[T, H * dq]`` of a projection with their rotated columns turned, in the weights' type; rows are turned in place."""
+    src = q.slabs if q.slabs is not None else q.rows
+    T, H, dtype = src.shape[-2], lw.heads, lw.ukv.dtype
+    if not src.is_cuda:
+        v = q.value().clone().view(T, H, lw.dq)
+        if lw.rot is not None:
+            part = v[..., lw.rot.start:lw.rot.start + lw.rot.dims]
+            part.copy_(lw.rot.apply(part, positions))
+        return v.view(T, H * lw.dq).to(dtype)
+    out = torch.empty((T, H * lw.dq), dtype=dtype, device=src.device) if q.rows is None else q.rows
+    start, dims = (lw.rot.start, lw.rot.dims) if lw.rot is not None else (0, 0)
+    native.call("prism_latent_rotate", 1 if dtype == torch.float32 else 0, *_branch_args(q), _p(out), out.stride(0),
+                *(lw.rot.args(positions) if lw.rot is not None else NO_ROTARY), T, H, lw.dq, start, dims, _s(), _pdl())
+    return out
+
 
 def latent_norm_store(raw: torch.Tensor, lw: LatentWeights, eps: float, slots: torch.Tensor, cache: KVCache, layer: int, *,
                       rows: Optional[torch.Tensor] = None) -> None:
     """RMS-normalise the projected latents ``raw [T, R]`` with their weight and store them at flat ``slots`` (negative =
     skip) of a single-plane cache, and into ``rows [T, Rc]`` when given."""
-    T, Rc = raw.shape[0], cache.head_dim
+    T, Rc = raw.shape[0], cache.latent(layer).shape[-1]
     if not raw.is_cuda:
         v = raw[:, :lw.rank].float()
         c = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps) * lw.norm.float()
@@ -241,28 +356,33 @@ def latent_norm_store(raw: torch.Tensor, lw: LatentWeights, eps: float, slots: t
                 _p(cache.latent(layer)), _p(slots), cache.num_blocks * cache.page, _p(rows), T, lw.rank, Rc, float(eps), _s(), _pdl())
 
 
-def latent_splits(sequences: int, rows: int) -> int:
-    """CTAs per key range: one CTA per SM is resident, so no more than fill the device once."""
+def latent_splits(sequences: int, rows: int, reach: int = NO_WINDOW) -> int:
+    """CTAs per key range: one CTA per SM is resident, so no more than fill the device once, nor than tiles in ``reach`` rows."""
     tiles = sequences * max(1, -(-rows // (16 if rows <= 16 else 32)))
-    return max(1, min(MAX_SPLITS, SM_COUNT // tiles))
+    return max(1, min(MAX_SPLITS, SM_COUNT // tiles, -(-reach // 64) + 1))
 
 
 def latent_attention_absorbed(
-    q: torch.Tensor, raw: torch.Tensor, gate: Optional[torch.Tensor], lw: LatentWeights, eps: float, slots: torch.Tensor,
+    q: "torch.Tensor | Branch", raw: Optional[torch.Tensor], gate: Optional[torch.Tensor], lw: LatentWeights, eps: float, slots: torch.Tensor,
     cache: KVCache, layer: int, block_tables: torch.Tensor, kv_lens: torch.Tensor, *, cu_seqlens_q: Optional[torch.Tensor] = None,
-    max_q_len: int = 1, nsplit: int = 0,
+    max_q_len: int = 1, nsplit: int = 0, positions: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
-    """Store the new tokens' latents, then causal attention of their heads over the paged latents in the absorbed
-    form, times the output ``gate``: ``[T, H * dv]``.
+    """Store the new tokens' latents (``raw``; none: they are in their pages already), then causal attention of their heads
+    over the paged latents in the absorbed form, times the output ``gate``: ``[T, H * dv]``.
 
-    ``q [T, H * dq]``, ``raw [T, R]`` and ``gate [T, H * dv]`` may be column ranges of a stacked projection.  Without
-    ``cu_seqlens_q`` every token is its own sequence (a decode step)."""
-    T, H, Rc = q.shape[0], lw.heads, cache.head_dim
-    if not q.is_cuda:
+    ``q [T, H * dq]``, ``raw [T, R]`` and ``gate [T, H * dv]`` may be column ranges of a stacked projection; ``q`` may be a branch.
+    Its rotated columns are turned here (``positions``).  Without ``cu_seqlens_q`` every token is its own sequence (a decode
+    step)."""
+    if isinstance(q, torch.Tensor):
+        q = Branch(rows=q)
+    src = q.slabs if q.slabs is not None else q.rows
+    pages = cache.latent(layer)
+    T, H, Rc, Rv = src.shape[-2], lw.heads, pages.shape[-1], lw.value_cols
+    if raw is not None and (not src.is_cuda or lw.ukv.dtype == torch.float32):
         latent_norm_store(raw, lw, eps, slots, cache, layer)
-        qa = torch.einsum("thd,hdr->thr", q.reshape(T, H, lw.dq).float(), lw.uk.float().view(H, lw.dq, Rc))
+    if not src.is_cuda:
+        qa = torch.einsum("thd,hdr->thr", rotate_queries(q, lw, positions).view(T, H, lw.dq).float(), lw.uk.float().view(H, lw.dq, Rc))
         lat = torch.zeros((T, H, Rc), dtype=torch.float32)
-        pages = cache.latent(layer).float()
         cu = cu_seqlens_q.tolist() if cu_seqlens_q is not None else list(range(T + 1))
         for s, (lo, hi) in enumerate(zip(cu[:-1], cu[1:])):
             n = int(kv_lens[s])
@@ -270,46 +390,48 @@ def latent_attention_absorbed(
                 continue
             pos = torch.arange(n)
             blk = block_tables[s, pos // cache.page].long()
-            c = pages[blk.clamp_min(0), pos % cache.page]
+            c = pages[blk.clamp_min(0), pos % cache.page].float()
             sc = torch.einsum("thr,nr->thn", qa[lo:hi], c) * lw.scale
-            seen = (pos[None, :] <= torch.arange(n - (hi - lo), n)[:, None]) & (blk >= 0)[None, :]
+            at = torch.arange(n - (hi - lo), n)[:, None]
+            seen = (pos[None, :] <= at) & (at - pos[None, :] < lw.window) & (blk >= 0)[None, :]
             sc = sc.masked_fill(~seen[:, None, :], float("-inf"))
             lat[lo:hi] = torch.einsum("thn,nr->thr", torch.softmax(sc, dim=-1), c)
         o = torch.einsum("thr,hvr->thv", lat, lw.uv.float().view(H, lw.dv, Rc)).reshape(T, H * lw.dv)
-        return (o if gate is None else o * gate.float()).to(q.dtype)
+        return (o if gate is None else o * gate.float()).to(lw.ukv.dtype)
     S = T if cu_seqlens_q is None else cu_seqlens_q.shape[0] - 1
-    dev = q.device
-    pages = cache.latent(layer)
+    dev, dtype = src.device, lw.ukv.dtype
     page_args = (_p(pages), _p(block_tables), _p(cu_seqlens_q), _p(kv_lens))
     assert block_tables.dtype == torch.int32 and kv_lens.dtype == torch.int32 and slots.dtype == torch.int64
     gate_ld = gate.stride(0) if gate is not None else 0
-    if q.dtype == torch.float32:
-        latent_norm_store(raw, lw, eps, slots, cache, layer)
+    if dtype == torch.float32:
+        rows = q.rows if lw.rot is None and q.rows is not None else rotate_queries(q, lw, positions)
         qa = torch.empty((T, H, Rc), dtype=torch.float32, device=dev)
-        native.call("prism_headwise_f32", _p(q), q.stride(0), _p(lw.uk), Rc, None, 0, _p(qa), H * Rc, T, H, lw.dq, Rc, 0, _s(), _pdl())
+        native.call("prism_headwise_f32", _p(rows), rows.stride(0), _p(lw.uk), Rc, None, 0, _p(qa), H * Rc, T, H, lw.dq, Rc, 0, _s(), _pdl())
         lat = torch.empty_like(qa)
         native.call("prism_latent_attention_f32", _p(qa), *page_args, _p(lat), S, max_q_len, H, Rc, cache.page, block_tables.shape[1],
-                    cache.num_blocks, float(lw.scale), _s(), _pdl())
+                    cache.num_blocks, lw.window, float(lw.scale), _s(), _pdl())
         out = torch.empty((T, H * lw.dv), dtype=torch.float32, device=dev)
         native.call("prism_headwise_f32", _p(lat), H * Rc, _p(lw.uv), Rc, _p(gate), gate_ld, _p(out), H * lw.dv, T, H, Rc, lw.dv, 1,
                     _s(), _pdl())
         return out
     if nsplit <= 0:
-        nsplit = latent_splits(S, max_q_len * H)
+        nsplit = latent_splits(S, max_q_len * H, lw.window + max_q_len)
     qa = torch.empty((T, H, Rc), dtype=torch.bfloat16, device=dev)
-    native.call("prism_latent_absorb", _p(q), q.stride(0), _p(lw.uk), _p(qa), _p(raw), raw.stride(0), _p(lw.norm), _p(pages), _p(slots),
-                cache.num_blocks * cache.page, T, H, lw.dq, lw.rank, Rc, float(eps), _s(), _pdl())
+    rot = (*lw.rot.args(positions), lw.rot.start, lw.rot.dims) if lw.rot is not None else (*NO_ROTARY, 0, 0)
+    slabs, stride, P, rows, ld = _branch_args(q)
+    native.call("prism_latent_absorb", rows, slabs, stride, P, ld, *rot, _p(lw.uk), _p(qa), _p(raw), raw.stride(0) if raw is not None else 0,
+                _p(lw.norm), _p(pages), _p(slots), cache.num_blocks * cache.page, T, H, lw.dq, lw.rank, Rc, float(eps), _s(), _pdl())
     part_o = part_ml = lat = None
     if nsplit > 1:
-        part_o = torch.empty((T * H, nsplit, Rc), dtype=torch.float32, device=dev)
+        part_o = torch.empty((T * H, nsplit, Rv), dtype=torch.float32, device=dev)
         part_ml = torch.empty((T * H, nsplit, 2), dtype=torch.float32, device=dev)
     else:
-        lat = torch.empty((T * H, Rc), dtype=torch.bfloat16, device=dev)
-    native.call("prism_latent_attention", _p(qa), *page_args, _p(part_o), _p(part_ml), _p(lat), S, max_q_len, H, Rc, cache.page,
-                block_tables.shape[1], cache.num_blocks, nsplit, float(lw.scale), _s(), _pdl())
+        lat = torch.empty((T * H, Rv), dtype=torch.bfloat16, device=dev)
+    native.call("prism_latent_attention", _p(qa), *page_args, _p(part_o), _p(part_ml), _p(lat), S, max_q_len, H, Rc, Rv, cache.page,
+                block_tables.shape[1], cache.num_blocks, nsplit, lw.window, float(lw.scale), _s(), _pdl())
     out = torch.empty((T, H * lw.dv), dtype=torch.bfloat16, device=dev)
-    native.call("prism_latent_out", _p(part_o), _p(part_ml), _p(lat), _p(lw.uv), _p(gate), gate_ld, _p(out), out.stride(0), T, H, lw.dv,
-                Rc, nsplit, _s(), _pdl())
+    native.call("prism_latent_out", _p(part_o), _p(part_ml), _p(lat), _p(lw.uv), Rc, _p(gate), gate_ld, _p(out), out.stride(0), T, H, lw.dv,
+                Rv, nsplit, _s(), _pdl())
     return out
 
 
@@ -334,7 +456,7 @@ def latent_attention_expanded(
     """The same result from explicit keys and values (bf16, CUDA): the visible latents as contiguous rows (the new
     tokens' own without ``cu_seqlens_kv``, else gathered from their pages), one GEMM for the keys and values of all
     heads, and the tcgen05 attention kernel with the gate in its epilogue."""
-    T, H, Rc = q.shape[0], lw.heads, cache.head_dim
+    T, H, Rc = q.shape[0], lw.heads, cache.latent(layer).shape[-1]
     dev, S = q.device, cu_seqlens_q.shape[0] - 1
     assert q.is_cuda and q.dtype == torch.bfloat16 and lw.dq == lw.dv
     total = T if cu_seqlens_kv is None else int(total_kv)
@@ -350,3 +472,85 @@ def latent_attention_expanded(
                 _p(cu_seqlens_q), _p(cu_seqlens_kv), _p(gate), gate.stride(0) if gate is not None else 0, T, total, S, int(max_q_len),
                 H, H, lw.dq, float(lw.scale), _s(), _pdl())
     return out
+
+
+# ------------------------------------------------------------------------- explicit keys of a window
+@dataclass
+class ExpandPlan:
+    """Where a prompt step's explicit keys and values go: of every sequence the pages that its new tokens see, from ``first[s]``
+    on, become scratch pages ``base[s] ..``; ``table`` is the block table of the scratch."""
+
+    first: torch.Tensor      # [S] int32
+    base: torch.Tensor       # [S + 1] int32
+    table: torch.Tensor      # [S, max_blocks] int32
+    pages: int
+    max_pages: int
+    pairs: int               # (new token, visible row) pairs, rounded up to tiles
+
+    @classmethod
+    def make(cls, lens: Sequence[tuple[int, int]], window: int, page: int, max_blocks: int, device) -> "ExpandPlan":
+        """``lens``: (new tokens, tokens up to the last of them) per sequence."""
+        S = len(lens)
+        host = torch.full((S, max_blocks), -1, dtype=torch.int32)
+        marks = torch.zeros((2, S + 1), dtype=torch.int32)
+        most = pairs = 0
+        for s, (n, kv) in enumerate(lens):
+            first, stop = (max(0, kv - n - window + 1) // page, -(-kv // page)) if n > 0 else (0, 0)
+            base = int(marks[1, s])
+            marks[0, s], marks[1, s + 1] = first, base + stop - first
+            host[s, first:stop] = torch.arange(base, base + stop - first, dtype=torch.int32)
+            most, pairs = max(most, stop - first), pairs + n * min(kv, window + 63)
+
+        def put(t: torch.Tensor) -> torch.Tensor:
+            return t if torch.device(device).type == "cpu" else t.pin_memory().to(device, non_blocking=True)
+
+        marks_d = put(marks)
+        return cls(marks_d[0, :S], marks_d[1], put(host), int(marks[1, S]), most, pairs)
+
+    def is_cheaper(self, lw: LatentWeights, row: int, page: int) -> bool:
+        """Whether explicit keys and values beat the absorbed form.  Per pair that multiplies ``row`` and the latent's elements
+        per head, the explicit form ``dq + dv`` on a tensor-core path that is about 2.5 times as fast, behind a projection of
+        every visible row."""
+        from .window import TC_MAX_HEAD, TC_MAX_KEY
+
+        rows, width = self.pages * page, lw.dq + lw.dv
+        if lw.dq > TC_MAX_KEY or lw.dq % 16 or lw.dv > TC_MAX_HEAD or lw.dv % 16 or page % 8 or lw.scale <= 0.0:
+            return False
+        if rows * 2 * (row + lw.heads * width) > EXPAND_MAX_SCRATCH_BYTES:
+            return False
+        return (self.pairs + rows * row) * width < 2.5 * self.pairs * (row + lw.value_cols)
+
+
+@dataclass
+class _ScratchPages:
+    """Scratch rows as the attention over single-row caches sees a cache."""
+
+    rows: torch.Tensor       # [blocks, page, row]
+
+    def token_rows(self, layer: int) -> torch.Tensor:
+        return self.rows
+
+    @property
+    def num_blocks(self) -> int:
+        return self.rows.shape[0]
+
+    @property
+    def page(self) -> int:
+        return self.rows.shape[1]
+
+
+def latent_attention_windowed(q: torch.Tensor, lw: LatentWeights, cache: KVCache, layer: int, block_tables: torch.Tensor, kv_lens: torch.Tensor,
+                              cu_seqlens_q: torch.Tensor, max_q_len: int, plan: ExpandPlan) -> torch.Tensor:
+    """Attention of rotated queries ``q [T, H * dq]`` (bf16, CUDA) with explicit keys and values: the visible rows gathered page by
+    page, one GEMM for the keys and values of all heads, and the tcgen05 attention over paged rows with a window."""
+    from .window import WindowSpec, window_attention
+
+    pages = cache.latent(layer)
+    H, Rc, page, rows = lw.heads, pages.shape[-1], cache.page, plan.pages * cache.page
+    c = torch.empty((rows, Rc), dtype=torch.bfloat16, device=q.device)
+    native.call("prism_gather_latent_pages", _p(pages), _p(block_tables), _p(kv_lens), _p(plan.first), _p(plan.base), _p(c), kv_lens.shape[0],
+                plan.max_pages, rows, block_tables.shape[1], cache.num_blocks, page, Rc * 2, _s(), _pdl())
+    kv = _ScratchPages(linear(c, lw.ukv).view(plan.pages, page, H * (lw.dq + lw.dv)))
+    spec = WindowSpec(heads=H, kv_heads=H, maps=1, dim=lw.dq, vdim=lw.dv, rot_dims=0, scale=lw.scale, window=lw.window, keep_first=0, gate=False,
+                      eps=0.0)
+    return window_attention(q, spec, None, kv, 0, plan.table, kv_lens, cu_seqlens_q=cu_seqlens_q, max_q_len=max_q_len)

@@ -17,7 +17,7 @@ from typing import Optional
 import torch
 import torch.nn.functional as F
 
-from . import GLU_ACTS, SM_COUNT, _p, _pdl, _s, effective_splits, glu_act, native
+from . import GLU_ACTS, SM_COUNT, _p, _pdl, _s, effective_splits, gated_unit, native
 from .latent import Branch
 
 SMALL_TOKENS = 128      # up to here: one routing CTA, every expert's GEMM reads the step's own rows, no gather
@@ -46,7 +46,8 @@ class Scored:
     """Routing by scores: softmax over all ``experts + identity`` outputs; ``correction`` (fp32, one per output) enters the choice
     only, which is among the ``keep`` best of ``groups`` equal runs of outputs (a group is as good as its best output); the
     weights are the chosen scores over their sum, times ``scale``.  ``always_gate``: one more logit, behind the others, whose
-    sigmoid weighs the always-on experts."""
+    sigmoid weighs the always-on experts.  ``sigmoid``: the scores are the outputs' sigmoids, not divided by their sum;
+    ``group_best`` 2: a group is as good as the sum of its two best outputs."""
 
     correction: torch.Tensor
     identity: int = 0
@@ -54,6 +55,8 @@ class Scored:
     keep: int = 1
     scale: float = 1.0
     always_gate: bool = False
+    sigmoid: bool = False
+    group_best: int = 1
 
 
 def _max_groups(T: int, top: int, experts: int, always: int, tile_rows: int) -> int:
@@ -66,13 +69,14 @@ def _max_groups(T: int, top: int, experts: int, always: int, tile_rows: int) -> 
 def _choose_cpu(z: torch.Tensor, top: int, experts: int, s: Scored):
     """(expert [T, top], ``experts`` where it is the token's own row; weight [T, top]; weight of the own row [T])"""
     n = experts + s.identity
-    score = torch.softmax(z[:, :n], 1)
+    score = torch.sigmoid(z[:, :n]) if s.sigmoid else torch.softmax(z[:, :n], 1)
     choice = score + s.correction
-    best = choice.view(-1, s.groups, n // s.groups).max(2).values.sort(dim=1, descending=True, stable=True).indices[:, :s.keep]
-    open_ = torch.zeros(z.shape[0], s.groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(n // s.groups, 1)
+    size = n // s.groups
+    best = choice.view(-1, s.groups, size).topk(min(s.group_best, size), 2).values.sum(2).sort(dim=1, descending=True, stable=True).indices[:, :s.keep]
+    open_ = torch.zeros(z.shape[0], s.groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(size, 1)
     chosen = choice.masked_fill(~open_, float("-inf")).sort(dim=1, descending=True, stable=True).indices[:, :top]
     w = score.gather(1, chosen)
-    w = w / (w.sum(1, keepdim=True) + 1e-20) * s.scale
+    w = (w if s.sigmoid else w / (w.sum(1, keepdim=True) + 1e-20)) * s.scale
     own = chosen >= experts
     return chosen.clamp_max(experts), w.masked_fill(own, 0.0), (w * own).sum(1)
 
@@ -128,12 +132,13 @@ def route(logits: Branch, top: int, experts: int, always: int, slots: torch.Tens
     n_groups = torch.empty((1,), **i32)
     args = (_p(expert), _p(pos), _p(weight), _p(row_token), _p(counts), _p(groups), groups.shape[0], _p(n_groups), T, top, experts, always,
             chunk, tile)
-    own, rule = None, (None, None, experts, 1, 1, -1, 1.0)
+    own, rule = None, (None, None, experts, 1, 1, -1, 1.0, 0, 1)
     if scored is not None:
         n = experts + scored.identity
         assert scored.correction.dtype == torch.float32 and scored.correction.shape == (n,) and s.shape[2] >= n + scored.always_gate
         own = torch.empty((T,), dtype=torch.float32, device=dev)
-        rule = (_p(scored.correction), _p(own), n, scored.groups, scored.keep, n if scored.always_gate else -1, float(scored.scale))
+        rule = (_p(scored.correction), _p(own), n, scored.groups, scored.keep, n if scored.always_gate else -1, float(scored.scale),
+                1 if scored.sigmoid else 0, scored.group_best)
     native.call("prism_moe_route", _p(s), s.stride(0), s.stride(1), s.shape[0], _p(slots), *args, *rule, _s(), _pdl())
     if chunks > 1:
         native.call("prism_moe_place", *args, _s(), _pdl())
@@ -145,9 +150,10 @@ def _down_splits(m: int, k: int, groups: int) -> int:
     return max(1, min(SM_COUNT // max(1, groups * -(-m // 128)), kb // 4 if kb >= 8 else 1, 8))
 
 
-def expert_ffn(x: torch.Tensor, r: Routing, w_gate_up: torch.Tensor, w_down: torch.Tensor, act: str = "silu") -> Branch:
+def expert_ffn(x: torch.Tensor, r: Routing, w_gate_up: torch.Tensor, w_down: torch.Tensor, act: str = "silu",
+               limit: float = 0.0) -> Branch:
     """Every pair's ``down_e(act(gate_e x) * up_e x)`` as a branch whose value is the weighted sum per token.  ``w_gate_up``
-    ``[E, 2 F, W]`` (gate rows, then up rows), ``w_down [E, W, F]``."""
+    ``[E, 2 F, W]`` (gate rows, then up rows), ``w_down [E, W, F]``; ``act`` as in ``gated_unit``, with its ``limit``."""
     T, W = x.shape
     E, F2, _ = w_gate_up.shape
     I = F2 // 2
@@ -157,7 +163,7 @@ def expert_ffn(x: torch.Tensor, r: Routing, w_gate_up: torch.Tensor, w_down: tor
         y = torch.zeros((N, W))
         for e, first, count, _ in r.groups.tolist():
             h = x[r.row_token[first:first + count].long()].float() @ w_gate_up[e].float().t()
-            a = (glu_act(h[:, :I], act) * h[:, I:]).to(x.dtype).float()
+            a = gated_unit(h[:, :I], h[:, I:], act, limit).to(x.dtype).float()
             y[first:first + count] = a @ w_down[e].float().t()
         return Branch(slabs=y.unsqueeze(0), pos=r.pos, weight=r.weight, self_weight=r.self_weight)
     assert x.dtype == w_gate_up.dtype == w_down.dtype and x.stride(1) == 1 and w_gate_up.is_contiguous() and w_down.is_contiguous()
@@ -168,22 +174,22 @@ def expert_ffn(x: torch.Tensor, r: Routing, w_gate_up: torch.Tensor, w_down: tor
         native.call("prism_gemm_f32_grouped", _p(w_gate_up), _p(x), _p(gu), F2, N, W, W, x.stride(0), F2, *table, _p(r.row_token), T, E, _s(),
                     _pdl())
         a = torch.empty((N, I), dtype=torch.float32, device=dev)
-        native.call("prism_glu_f32", _p(gu), _p(a), N, I, GLU_ACTS[act], _s(), _pdl())
+        native.call("prism_glu_f32", _p(gu), _p(a), N, I, GLU_ACTS[act], float(limit), _s(), _pdl())
         y = torch.empty((1, N, W), dtype=torch.float32, device=dev)
         native.call("prism_gemm_f32_grouped", _p(w_down), _p(a), _p(y), W, N, I, I, I, W, *table, None, N, E, _s(), _pdl())
         return Branch(slabs=y, pos=r.pos, weight=r.weight, self_weight=r.self_weight)
     a = torch.empty((N, I), dtype=torch.bfloat16, device=dev)
     if T <= SMALL_TOKENS:
         native.call("prism_gemm_grouped_small", _p(w_gate_up), _p(x), _p(a), I, T, T, W, x.stride(0), I, *table, _p(r.row_token), N, E,
-                    GLU_ACTS[act], 1, 0, _s(), _pdl())
+                    GLU_ACTS[act], float(limit), 1, 0, _s(), _pdl())
         splits = effective_splits(I, _down_splits(W, I, G))
         y = torch.empty((splits, N, W), dtype=torch.float32, device=dev)
-        native.call("prism_gemm_grouped_small", _p(w_down), _p(a), _p(y), W, T, N, I, I, W, *table, None, N, E, 0, splits, y.stride(0), _s(),
+        native.call("prism_gemm_grouped_small", _p(w_down), _p(a), _p(y), W, T, N, I, I, W, *table, None, N, E, 0, 0.0, splits, y.stride(0), _s(),
                     _pdl())
         return Branch(slabs=y, pos=r.pos, weight=r.weight, self_weight=r.self_weight)
     rows = torch.empty((N, W), dtype=torch.bfloat16, device=dev)
     native.call("prism_moe_gather", _p(x), x.stride(0), _p(r.pos), _p(rows), T, K, W, _s(), _pdl())
-    native.call("prism_gemm_grouped", _p(w_gate_up), _p(rows), _p(a), I, N, W, W, I, *table, E, GLU_ACTS[act], _s(), _pdl())
+    native.call("prism_gemm_grouped", _p(w_gate_up), _p(rows), _p(a), I, N, W, W, I, *table, E, GLU_ACTS[act], float(limit), _s(), _pdl())
     y = torch.empty((N, W), dtype=torch.bfloat16, device=dev)
-    native.call("prism_gemm_grouped", _p(w_down), _p(a), _p(y), W, N, I, I, W, *table, E, 0, _s(), _pdl())
+    native.call("prism_gemm_grouped", _p(w_down), _p(a), _p(y), W, N, I, I, W, *table, E, 0, 0.0, _s(), _pdl())
     return Branch(rows=y, pos=r.pos, weight=r.weight, self_weight=r.self_weight)

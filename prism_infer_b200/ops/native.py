@@ -30,10 +30,10 @@ _SIGNATURES = {
     "prism_gemm_wx_sections": "pppiiilllpipppfiiipi",
     "prism_gemm_f32": "pppiiilllpipppfpi",
     "prism_gemm_f32_grouped": "pppiiilllpippiipi",
-    "prism_glu_f32": "ppiiipi",
-    "prism_gemm_grouped_small": "pppiiiillpippiiiilpi",
-    "prism_gemm_grouped": "pppiiillpipiipi",
-    "prism_moe_route": "pllippppppp" "ip" "iiiiii" "ppiiiifpi",
+    "prism_glu_f32": "ppiiifpi",
+    "prism_gemm_grouped_small": "pppiiiillpippiiifilpi",
+    "prism_gemm_grouped": "pppiiillpipiifpi",
+    "prism_moe_route": "pllippppppp" "ip" "iiiiii" "ppiiiifiipi",
     "prism_moe_place": "pppppp" "ip" "iiiiiipi",
     "prism_moe_gather": "plppiiipi",
     "prism_window_prepare": "ipliplppp" "ppplppp" "iiiiiiiiiiii" "fpi",
@@ -45,16 +45,22 @@ _SIGNATURES = {
     "prism_tanh_f32": "plip" "iipi",
     "prism_state_step": "ipliippp" "ii" "plipl" "plipl" "ppppp" "iiii" "fpi",
     "prism_state_scan": "ipliipppp" "ii" "plipl" "ppp" "iiipi",
+    "prism_forget_step": "ipliippi" "plipl" "pppp" "iiii" "fpi",
+    "prism_forget_scan": "ipliipppi" "plipl" "ppp" "iiiipi",
+    "prism_short_conv": "ipliipppii" "ppp" "iipi",
     "prism_head_norm_gate": "ip" "plipl" "pp" "iiii" "fpi",
     "prism_token_side_gate": "ipliplplllppiipi",
-    "prism_stream_update": "iipippl" "plipl" "p" "plipl" "p" "lppippfffpp" "plplpl" "iifpi",
+    "prism_stream_update": "iipippl" "plipl" "p" "plipl" "p" "lppippfffpp" "plplpl" "iif" "plpi" "pipliipp" "pi",
     "prism_latent_norm_store": "iplppplpiiifpi",
-    "prism_latent_absorb": "plppplppp" "liiiiifpi",
-    "prism_latent_attention": "pppppppp" "iiiiiiiifpi",
-    "prism_latent_out": "ppppplpl" "iiiiipi",
+    "prism_latent_prepare": "ipliplpp" "pppl" "ppf" "iiiiiii" "fpi",
+    "prism_latent_rotate": "iplipl" "pl" "ppf" "iiiiipi",
+    "prism_latent_absorb": "pplil" "ppfii" "pppl" "ppp" "liiiiifpi",
+    "prism_latent_attention": "pppppppp" "iiiiiiiiiifpi",
+    "prism_latent_out": "pppplplpl" "iiiiipi",
+    "prism_gather_latent_pages": "pppppp" "iiiiiiipi",
     "prism_gather_latents": "ppppiiiiiiipi",
     "prism_headwise_f32": "plplplpliiiiipi",
-    "prism_latent_attention_f32": "ppppppiiiiiiifpi",
+    "prism_latent_attention_f32": "ppppppiiiiiiiifpi",
     "prism_flash_attention_tc_kv": "plpplplppp" "liiiiiiifpi",
     "prism_gemm_effective_splits": "ii",
     "prism_gemm_clear_tensor_maps": "",

@@ -1,4 +1,4 @@
-"""Recurrent state of sequences and the time-mixing recurrence with a matrix state per head.
+"""Recurrent state of sequences, recurrences with a matrix state per head, and the short convolution in front of a mixer.
 
 A sequence's state lives in a slot: per recurrent layer a row of fp32, in two versions.  A step that takes a sequence from
 ``c`` tokens to ``c'`` reads version ``c & 1`` and writes version ``c' & 1``; a step that is run again (a decode launch that ran
@@ -10,6 +10,16 @@ With ``h'`` the previous token's row, every projection reads its own blend ``h +
     o_t = (S + diag(u) k v^T)^T r        S <- diag(d) S + k v^T
 
 and the mixer's output is ``o`` over its root mean square per head, times a weight, times ``silu`` of the gate.
+
+The forget rule has no keys: a gate per head and key channel, ``f = l + (1 - l) sigmoid(z + b)`` above a learned bound ``l``, decays
+the state and weighs what is written; the query ``q = silu(y)`` reads behind the update:
+
+    S <- diag(f) S + (1 - f) v^T        o_t = S^T q
+
+and the output is ``o`` over its root mean square per head, times a weight that all heads share.
+
+The short convolution adds a causal sum over the last ``taps`` rows of every channel to a row; the last ``taps - 1`` rows are
+carried on in the state.
 
 CUDA tensors run the kernels of ``csrc/recurrence.cu`` and raise without them; CPU tensors run the plain-PyTorch statement.
 """
@@ -98,9 +108,9 @@ class StateView:
     kv_lens: torch.Tensor                          # [S] int32 tokens up to and including the step's last
     cu_seqlens_q: Optional[torch.Tensor] = None    # [S + 1] int32; None: one token per sequence
 
-    def args(self, spec: TimeMixSpec, cu: bool = True) -> tuple:
+    def args(self, spec: "TimeMixSpec | ForgetSpec | ConvSpec", cu: bool = True) -> tuple:
         t = self.cache.layer(self.layer)
-        assert t.shape[2] == spec.carry + spec.width and self.slots.dtype == torch.int32 and self.kv_lens.dtype == torch.int32
+        assert t.shape[2] >= spec.carry + spec.width and self.slots.dtype == torch.int32 and self.kv_lens.dtype == torch.int32
         return (_p(t), t.shape[2], t.shape[0], spec.carry, _p(self.slots)) + ((_p(self.cu_seqlens_q),) if cu else ()) + (_p(self.kv_lens),)
 
 
@@ -176,11 +186,11 @@ def wide_projections(mixed: torch.Tensor, w: torch.Tensor, table: tuple) -> Bran
     if T <= SMALL_TOKENS:
         splits = effective_splits(W, _grouped_splits(M, W))
         y = torch.empty((splits, N, M), dtype=torch.float32, device=w.device)
-        native.call("prism_gemm_grouped_small", _p(w), _p(mixed), _p(y), M, T, N, W, W, M, *table, None, N, 4, 0, splits, y.stride(0), _s(),
+        native.call("prism_gemm_grouped_small", _p(w), _p(mixed), _p(y), M, T, N, W, W, M, *table, None, N, 4, 0, 0.0, splits, y.stride(0), _s(),
                     _pdl())
         return Branch(slabs=y)
     y = torch.empty((N, M), dtype=torch.bfloat16, device=w.device)
-    native.call("prism_gemm_grouped", _p(w), _p(mixed), _p(y), M, N, W, W, M, *table, 4, 0, _s(), _pdl())
+    native.call("prism_gemm_grouped", _p(w), _p(mixed), _p(y), M, N, W, W, M, *table, 4, 0, 0.0, _s(), _pdl())
     return Branch(rows=y)
 
 
@@ -221,4 +231,147 @@ def time_mix(x: torch.Tensor, spec: TimeMixSpec, w: TimeMixWeights, st: StateVie
                 _s(), _pdl())
     native.call("prism_head_norm_gate", f32, _p(o), *_proj_args(p), _p(w.norm), _p(out), T, spec.heads, spec.n, spec.dim, float(spec.eps), _s(),
                 _pdl())
+    return out
+
+
+# ----------------------------------------------------------------------------------------- the forget rule
+@dataclass(frozen=True)
+class ForgetSpec:
+    """Sizes of one mixer: ``dim`` key and ``vdim`` value channels per head, padded to multiples of 16 (``n``, ``m``)."""
+
+    heads: int
+    dim: int
+    vdim: int
+    eps: float
+
+    width = 0                # it carries no input row on
+
+    @property
+    def n(self) -> int:
+        return -(-self.dim // 16) * 16
+
+    @property
+    def m(self) -> int:
+        return -(-self.vdim // 16) * 16
+
+    @property
+    def gate_col(self) -> int:
+        """First gate column of the stacked projection ``[queries | gates | values]``; ``value_col`` the first value column."""
+        return self.heads * self.n
+
+    @property
+    def value_col(self) -> int:
+        return 2 * self.heads * self.n
+
+    @property
+    def proj_cols(self) -> int:
+        return self.heads * (2 * self.n + self.m)
+
+    @property
+    def carry(self) -> int:
+        """Elements of the state; what a layer carries on besides starts there."""
+        return self.heads * self.n * self.m
+
+
+@dataclass
+class ForgetWeights:
+    bias: torch.Tensor       # [H n] of the gates
+    lower: torch.Tensor      # [H n] bounds of the gates; one in padded channels, which then hold nothing
+    norm: torch.Tensor       # [m]
+
+
+def _forget_cpu(y: torch.Tensor, spec: ForgetSpec, w: ForgetWeights, st: StateView) -> torch.Tensor:
+    H, n, m = spec.heads, spec.n, spec.m
+    rows = st.cache.layer(st.layer)
+    out = torch.zeros((y.shape[0], H * m), dtype=w.norm.dtype)
+    for slot, lo, hi, before in _spans(st, y.shape[0]):
+        q = F.silu(y[lo:hi, :spec.gate_col]).view(-1, H, n)
+        keep = (1.0 - w.lower.float()) * torch.sigmoid(-(y[lo:hi, spec.gate_col:spec.value_col] + w.bias.float()))
+        keep = keep.view(-1, H, n)
+        v = y[lo:hi, spec.value_col:].view(-1, H, m)
+        S = rows[slot, before & 1, :spec.carry].clone().view(H, n, m) if before > 0 else torch.zeros(H, n, m)
+        o = torch.empty((hi - lo, H, m))
+        for i in range(hi - lo):
+            S = (1.0 - keep[i])[:, :, None] * S + keep[i, :, :, None] * v[i, :, None, :]
+            o[i] = (S * q[i, :, :, None]).sum(1)
+        o = o / torch.sqrt(o.pow(2).sum(-1, keepdim=True) / spec.vdim + spec.eps) * w.norm.float()
+        out[lo:hi] = o.reshape(-1, H * m).to(out.dtype)
+        rows[slot, (before + hi - lo) & 1, :spec.carry] = S.reshape(-1)
+    return out
+
+
+def forget_mix(p: Branch, spec: ForgetSpec, w: ForgetWeights, st: StateView) -> torch.Tensor:
+    """The mixer up to its output projection for the step's stacked projection ``p [T, proj_cols]``: ``[T, H m]``, with the state
+    taken from and put back into the sequences' slots.  Rows of sequences without a slot are zero."""
+    src = p.slabs if p.slabs is not None else p.rows
+    if not src.is_cuda:
+        return _forget_cpu(p.value(), spec, w, st)
+    if max(spec.n, spec.m) > MAX_HEAD:
+        raise ValueError(f"gated linear attention: heads of up to {MAX_HEAD} channels, got {spec.dim} x {spec.vdim}")
+    T, S, dev = src.shape[-2], st.slots.shape[0], src.device
+    assert src.shape[-1] == spec.proj_cols and src.stride(-1) == 1
+    f32 = 1 if w.norm.dtype == torch.float32 else 0
+    out = torch.empty((T, spec.heads * spec.m), dtype=w.norm.dtype, device=dev)
+    if st.cu_seqlens_q is None:
+        native.call("prism_forget_step", f32, *st.args(spec, cu=False), S, *_proj_args(p), _p(w.bias), _p(w.lower), _p(w.norm), _p(out), spec.heads,
+                    spec.n, spec.m, spec.vdim, float(spec.eps), _s(), _pdl())
+        return out
+    o = torch.empty((T, spec.heads * spec.m), dtype=torch.float32, device=dev)
+    native.call("prism_forget_scan", f32, *st.args(spec), S, *_proj_args(p), _p(w.bias), _p(w.lower), _p(o), T, spec.heads, spec.n, spec.m, _s(),
+                _pdl())
+    native.call("prism_head_norm_gate", f32, _p(o), None, 0, 0, None, 0, _p(w.norm), _p(out), T, spec.heads, spec.m, spec.vdim, float(spec.eps),
+                _s(), _pdl())
+    return out
+
+
+# ---------------------------------------------------------------------------------- the short convolution
+MAX_TAPS = 16
+
+
+@dataclass(frozen=True)
+class ConvSpec:
+    """``taps`` rows of ``row`` columns; those carried on start at element ``carry`` of the state row."""
+
+    taps: int
+    row: int
+    carry: int
+
+    @property
+    def width(self) -> int:
+        return (self.taps - 1) * self.row
+
+
+@dataclass
+class ConvStep:
+    """The convolution of one token per sequence as a part of the kernel that makes its input rows (``stream_update``)."""
+
+    weight: torch.Tensor     # [taps, W]
+    spec: ConvSpec
+    state: StateView
+
+    def args(self) -> tuple:
+        t = self.state.cache.layer(self.state.layer)
+        _, row, slots, carry, slot_p, lens_p = self.state.args(self.spec, cu=False)
+        return (_p(self.weight), self.spec.taps, _p(t), row, slots, carry, slot_p, lens_p)
+
+
+def short_conv(x: torch.Tensor, weight: torch.Tensor, spec: ConvSpec, st: StateView, *, max_len: int = 1) -> torch.Tensor:
+    """``x_t + sum_j weight[j] x_(t - taps + 1 + j)`` for the step's rows ``x [T, W]``, the rows before them from the sequences'
+    slots, whose carry is renewed.  ``max_len``: the most tokens of a sequence."""
+    if spec.taps > MAX_TAPS:
+        raise ValueError(f"convolutions of up to {MAX_TAPS} taps, got {spec.taps}")
+    keep = spec.taps - 1
+    if not x.is_cuda:
+        rows, out = st.cache.layer(st.layer), x.clone()
+        for slot, lo, hi, before in _spans(st, x.shape[0]):
+            old = rows[slot, before & 1, spec.carry:spec.carry + spec.width].clone().view(keep, spec.row)
+            seen = torch.cat([old if before > 0 else torch.zeros_like(old), x[lo:hi].float()])
+            n = hi - lo
+            out[lo:hi] = (x[lo:hi].float() + sum(weight[j].float() * seen[j:j + n] for j in range(spec.taps))).to(x.dtype)
+            rows[slot, (before + n) & 1, spec.carry:spec.carry + spec.width] = seen[n:].reshape(-1)
+        return out
+    assert x.is_contiguous() and weight.is_contiguous() and x.dtype == weight.dtype and x.shape[1] == spec.row and st.cu_seqlens_q is not None
+    out = torch.empty_like(x)
+    native.call("prism_short_conv", 1 if x.dtype == torch.float32 else 0, *st.args(spec), st.slots.shape[0], spec.row, _p(x), _p(weight), _p(out),
+                spec.taps, int(max_len), _s(), _pdl())
     return out

@@ -22,6 +22,7 @@ from . import SM_COUNT, KVCache, _decode_counters, _p, _pdl, _s, native
 from .latent import Branch
 
 TC_MAX_HEAD = 128        # widest key map and value head of the tcgen05 prefill kernel
+TC_MAX_KEY = 192         # widest key head with a single map
 MMA_MAX_KEY = 512        # widest key row (all maps) and value head of the mma.sync decode kernel
 MMA_MAX_VALUE = 256
 MAX_SPLITS = 32
@@ -226,7 +227,7 @@ def window_attention(q: torch.Tensor, spec: WindowSpec, gate: Optional[torch.Ten
             counters = _decode_counters(q.device, S * blocks)
         native.call("prism_window_decode", *head, _p(po), _p(ml), _p(counters), S, *sizes, mt, ns, *tail)
         return out
-    if fast and not decode and spec.dq <= TC_MAX_HEAD and spec.dv <= TC_MAX_HEAD and cache.page % 8 == 0 and spec.scale > 0.0:
+    if fast and not decode and spec.dq <= (TC_MAX_KEY if M == 1 else TC_MAX_HEAD) and spec.dv <= TC_MAX_HEAD and cache.page % 8 == 0 and spec.scale > 0.0:
         native.call("prism_window_prefill_tc", *head, T, S, int(max_q_len), *sizes, *tail)
         return out
     native.call("prism_window_attention_simple", 1 if q.dtype == torch.float32 else 0, *head, S, int(max_q_len), *sizes, *tail)
