@@ -19,6 +19,7 @@ generated token ids of the request, so that runs at different N can be compared 
     python bench.py --workload latent-layers     (benchmarks/bench_latent_layers.py)
     python bench.py --workload window-layers     (benchmarks/bench_window_layers.py)
     python bench.py --workload recurrent-layers  (benchmarks/bench_recurrent_layers.py)
+    python bench.py --workload hybrid-layers     (benchmarks/bench_hybrid_layers.py)
 """
 
 from __future__ import annotations
@@ -111,17 +112,17 @@ def main() -> None:
     ap.add_argument("--model", default="random:qwen3-vl-8b")
     ap.add_argument("--kv-pages", type=int, default=0)
     ap.add_argument("--logits-precision", default="", choices=["", "model", "fp32", "selective_fp32"])
-    ap.add_argument("--workload", default="headline", choices=["headline", "latent-layers", "window-layers", "recurrent-layers"],
-                    help="latent-layers, window-layers, recurrent-layers: layer throughput and kernel rooflines of the latent-attention family, "
-                         "of the windowed-attention family with experts, or of the family with recurrent layers, beside their closest family "
-                         "at equal size (one GPU; its own JSON line)")
+    ap.add_argument("--workload", default="headline", choices=["headline", "latent-layers", "window-layers", "recurrent-layers", "hybrid-layers"],
+                    help="latent-layers, window-layers, recurrent-layers, hybrid-layers: layer throughput and kernel rooflines of the "
+                         "latent-attention family, of the windowed-attention family with experts, of the family with recurrent layers, or of the "
+                         "one with gated linear attention and windowed latents, beside their closest family at equal size (one GPU; its own JSON line)")
     ap.add_argument("--sizes", default="2048,4096,8192", help="layer widths of the layer workloads")
     args = ap.parse_args()
     if args.workload.endswith("-layers"):
-        from benchmarks import bench_latent_layers, bench_recurrent_layers, bench_window_layers
+        from benchmarks import bench_hybrid_layers, bench_latent_layers, bench_recurrent_layers, bench_window_layers
 
         layers = {"latent-layers": bench_latent_layers, "window-layers": bench_window_layers,
-                  "recurrent-layers": bench_recurrent_layers}[args.workload]
+                  "recurrent-layers": bench_recurrent_layers, "hybrid-layers": bench_hybrid_layers}[args.workload]
         raise SystemExit(layers.main(["--sizes", args.sizes, "--steps", str(args.steps), "--warmup", str(args.warmup)]))
     if args.impl == "reference":
         run_reference(args)

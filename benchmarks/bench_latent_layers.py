@@ -283,15 +283,15 @@ class Kernels:
         p, s, pdl = (lambda t: None if t is None else t.data_ptr()), (lambda: torch.cuda.current_stream().cuda_stream), ops._pdl
 
         def absorb(i):
-            native.call("prism_latent_absorb", p(q), q.stride(0), p(lws[i].uk), p(qa), p(raw), raw.stride(0), p(lws[i].norm), p(cache.latent(i)),
+            native.call("prism_latent_absorb", p(q), None, 0, 0, q.stride(0), *lat.NO_ROTARY, 0, 0, p(lws[i].uk), p(qa), p(raw), raw.stride(0), p(lws[i].norm), p(cache.latent(i)),
                         p(slots), cache.num_blocks * page, batch, H, D, R, R, 1e-5, s(), pdl())
 
         def attend(i):
-            native.call("prism_latent_attention", p(qa), p(cache.latent(i)), p(table), None, p(lens), p(po), p(ml), p(la), batch, 1, H, R, page,
-                        per_seq, cache.num_blocks, ns, D ** -0.5, s(), pdl())
+            native.call("prism_latent_attention", p(qa), p(cache.latent(i)), p(table), None, p(lens), p(po), p(ml), p(la), batch, 1, H, R, R, page,
+                        per_seq, cache.num_blocks, ns, lat.NO_WINDOW, D ** -0.5, s(), pdl())
 
         def output(i):
-            native.call("prism_latent_out", p(po), p(ml), p(la), p(lws[i].uv), p(gate), gate.stride(0), p(out), out.stride(0), batch, H, D, R, ns,
+            native.call("prism_latent_out", p(po), p(ml), p(la), p(lws[i].uv), R, p(gate), gate.stride(0), p(out), out.stride(0), batch, H, D, R, ns,
                         s(), pdl())
 
         def whole(i):
