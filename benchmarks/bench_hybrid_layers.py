@@ -238,9 +238,11 @@ class Kernels(base.Kernels):
         p, s, pdl = (lambda t: None if t is None else t.data_ptr()), (lambda: torch.cuda.current_stream().cuda_stream), ops._pdl
 
         def absorb(i):
-            l = lws[i]
-            slabs, stride, P, rows, ld = lat._branch_args(q)
-            native.call("prism_latent_absorb", rows, slabs, stride, P, ld, *l.rot.args(pos), D, r, p(l.uk), p(qa), None, 0, None, None, p(slots), 0, batch, H, D + r,
+            l, src, rot = lws[i], q, (*lws[i].rot.args(pos), D, r)
+            if batch > lat.ABSORB_ROTATES_TOKENS:
+                src, rot = lat.Branch(rows=lat.rotate_queries(q, l, pos)), (*lat.NO_ROTARY, 0, 0)
+            slabs, stride, P, rows, ld = lat._branch_args(src)
+            native.call("prism_latent_absorb", rows, slabs, stride, P, ld, *rot, p(l.uk), p(qa), None, 0, None, None, p(slots), 0, batch, H, D + r,
                         R, Rc, 1e-6, s(), pdl())
 
         def attend(i):
@@ -289,7 +291,7 @@ class Kernels(base.Kernels):
 
         self.time("fosulix", f"visible rows gathered, {tag}", "", gather, 2, tokens * Rc * 4)
         M = H * (2 * D + r)
-        self.time("fosulix", f"rows -> keys and values, {tag}", f"stacked projection, {tag}" if tokens == 2048 else "", lambda i: ops.linear(rows, lws[i].ukv), 2,
+        self.time("fosulix", f"rows -> keys and values, {tag}", f"latents -> keys and values, {tag}", lambda i: ops.linear(rows, lws[i].ukv), 2,
                   M * (Rc + tokens) * 2, 2.0 * tokens * Rc * M)
         kv = lat._ScratchPages(self.matrix(tokens, M).view(pages, page, M))
         sp = window.WindowSpec(heads=H, kv_heads=H, maps=1, dim=D + r, vdim=D, rot_dims=0, scale=(D + r) ** -0.5, window=WINDOW, keep_first=0, gate=False, eps=0.0)
@@ -330,6 +332,7 @@ def kernel_rows(widths, steps: int, warmup: int) -> list[dict]:
         for tokens in (2048, 8192):
             k.prefill_attention(tokens)
             like.prefill_attention(tokens)
+            latent.prefill_attention(tokens)
             torch.cuda.empty_cache()
         rows += k.rows + like.rows + [r for r in latent.rows if r["family"] == "latent"]
         del k, like, latent

@@ -227,70 +227,113 @@ __global__ void __launch_bounds__(256) token_mix_kernel(const MixArgs<T> a) {
 // =====================================================================================
 // out_t = x_t + sum_j w_j x_(t - taps + 1 + j) on every channel, rows before the step's from the slot's carry (oldest first) and
 // zeros before the sequence's start.  grid (chunks of a sequence, column blocks, sequences): a thread walks four columns through
-// a chunk.  A chunk is no shorter than the rows that are carried on, so only a sequence's first one reads the carry: it writes the
-// new one too, after it has read the old (both may be the same version).  MT: taps, rounded up.
+// a chunk, two groups of rows under way while it works on a third.  A chunk is no shorter than the rows that are carried on, so only
+// a sequence's first one reads the carry: it writes the new one too, after it has read the old (both may be the same version).  MT:
+// taps, rounded up.
 // =====================================================================================
-constexpr int CONV_CHUNK = 16;
+constexpr int CONV_MIN_CHUNK = 16, CONV_THREADS = 128;
 template <typename T>
 struct ConvArgs {
   StateArgs st;            // x is not used
   const T* x;              // [T][W]
   const T* w;              // [taps][W]
   T* out;                  // [T][W]
-  int taps;
+  int taps, chunk;
 };
 
+// Four columns as two packed pairs.
+struct Pairs {
+  unsigned long long lo, hi;
+};
+__device__ __forceinline__ Pairs pairs_of(float4 v) { return Pairs{pair_of(v.x, v.y), pair_of(v.z, v.w)}; }
+
 template <typename T, int MT>
-__global__ void __launch_bounds__(256) short_conv_kernel(const ConvArgs<T> a) {
-  const int W = a.st.W, s = blockIdx.z, c = (blockIdx.y * 256 + threadIdx.x) * 4, i0 = blockIdx.x * CONV_CHUNK;
+__global__ void __launch_bounds__(CONV_THREADS, MT <= 4 ? 5 : 2) short_conv_kernel(const ConvArgs<T> a) {
+  constexpr int ROWS = MT <= 4 && sizeof(T) == 2 ? 8 : 4;
+  using Raw = RawProj<T, false>;
+  using RawT = typename Raw::type;
+  const int W = a.st.W, s = blockIdx.z, c = (blockIdx.y * CONV_THREADS + threadIdx.x) * 4, i0 = blockIdx.x * a.chunk;
   pdl_launch_dependents();
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  Pairs w[MT], h[MT];                             // aligned at the end: tap MT - 1 meets the row itself, whose one it takes in
+#pragma unroll
+  for (int k = 0; k < MT; ++k) {
+    float4 v = k >= MT - a.taps && c < W ? load4(a.w + (size_t)(k - (MT - a.taps)) * W + c) : zero;
+    if (k == MT - 1) v = make_float4(1.0f + v.x, 1.0f + v.y, 1.0f + v.z, 1.0f + v.w);
+    w[k] = pairs_of(v);
+  }
   const Span sp = span_of(a.st, s);
   if (i0 >= sp.len || c >= W) return;             // a row without a slot has a carry of zeros
-  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  float4 w[MT], h[MT];                            // aligned at the end: tap MT - 1 meets the row itself
-#pragma unroll
-  for (int k = 0; k < MT; ++k) w[k] = k >= MT - a.taps ? load4(a.w + (size_t)(k - (MT - a.taps)) * W + c) : zero;
   pdl_wait();
   const T* x = a.x + (size_t)sp.first * W + c;
-  const int keep = a.taps - 1;
+  const int keep = a.taps - 1, n = min(a.chunk, sp.len - i0);
+  const T* src = x + (size_t)i0 * W;              // the next row to fetch
+  T* dst = a.out + (size_t)(sp.first + i0) * W + c;
+  RawT raw[2][ROWS];
+  auto fetch = [&](RawT (&r)[ROWS], int from) {
+    if (from + ROWS <= n) {
+#pragma unroll
+      for (int q = 0; q < ROWS; ++q, src += W) r[q] = *reinterpret_cast<const RawT*>(src);
+    } else {
+#pragma unroll
+      for (int q = 0; q < ROWS; ++q, src += W) r[q] = from + q < n ? *reinterpret_cast<const RawT*>(src) : Raw::zero();
+    }
+  };
+  fetch(raw[0], 0);
 #pragma unroll
   for (int k = 0; k < MT - 1; ++k) {
     const int p = i0 - (MT - 1) + k;              // row within the step's part of the sequence
-    h[k] = zero;
-    if (k < MT - a.taps) continue;
-    if (p >= 0) h[k] = load4(x + (size_t)p * W);
-    else if (sp.old_version) h[k] = load4(sp.old_version + a.st.carry + (size_t)(keep + p) * W + c);
+    float4 v = zero;
+    if (k >= MT - a.taps) {
+      if (p >= 0) v = load4(x + (size_t)p * W);
+      else if (sp.old_version) v = load4(sp.old_version + a.st.carry + (size_t)(keep + p) * W + c);
+    }
+    h[k] = pairs_of(v);
   }
   if (i0 == 0 && sp.new_version) {
-    float* dst = sp.new_version + a.st.carry + c;
+    float* carry = sp.new_version + a.st.carry + c;
+    float4 v[MT];
 #pragma unroll
-    for (int k = 0; k < MT - 1; ++k) {
-      if (k < MT - a.taps) continue;
+    for (int k = 0; k < MT - 1; ++k) {            // all of it is read before any of it is written
       const int p = sp.len - (MT - 1) + k;
-      float4 v = zero;
-      if (p >= 0) v = load4(x + (size_t)p * W);
-#pragma unroll
-      for (int q = 0; q < MT - 1; ++q)
-        if (p < 0 && q == MT - 1 + p) v = h[q];
-      store4(dst + (size_t)(k - (MT - a.taps)) * W, v);
+      v[k] = zero;
+      if (k < MT - a.taps) continue;
+      if (p >= 0) v[k] = load4(x + (size_t)p * W);
+      else if (sp.old_version) v[k] = load4(sp.old_version + a.st.carry + (size_t)(keep + p) * W + c);
     }
+#pragma unroll
+    for (int k = 0; k < MT - 1; ++k)
+      if (k >= MT - a.taps) store4(carry + (size_t)(k - (MT - a.taps)) * W, v[k]);
   }
-  T* out = a.out + (size_t)sp.first * W + c;
-  const int n = min(CONV_CHUNK, sp.len - i0);
-#pragma unroll 4
-  for (int i = 0; i < n; ++i) {
-    h[MT - 1] = load4(x + (size_t)(i0 + i) * W);
-    float4 o = h[MT - 1];
+  fetch(raw[1], ROWS);
+  auto row = [&](RawT r, bool live) {
+    h[MT - 1] = pairs_of(raw_value(r));
+    Pairs o{mul2(w[0].lo, h[0].lo), mul2(w[0].hi, h[0].hi)};
 #pragma unroll
-    for (int k = 0; k < MT; ++k) {
-      o.x = fmaf(w[k].x, h[k].x, o.x);
-      o.y = fmaf(w[k].y, h[k].y, o.y);
-      o.z = fmaf(w[k].z, h[k].z, o.z);
-      o.w = fmaf(w[k].w, h[k].w, o.w);
+    for (int k = 1; k < MT; ++k) {
+      o.lo = fma2(w[k].lo, h[k].lo, o.lo);
+      o.hi = fma2(w[k].hi, h[k].hi, o.hi);
     }
-    store4(out + (size_t)(i0 + i) * W, o);
 #pragma unroll
     for (int k = 0; k < MT - 1; ++k) h[k] = h[k + 1];
+    const float2 l = unpair(o.lo), u = unpair(o.hi);
+    if (live) store4(dst, make_float4(l.x, l.y, u.x, u.y));
+    dst += W;
+  };
+  auto work = [&](const RawT (&r)[ROWS], int from) {
+    if (from + ROWS <= n) {
+#pragma unroll
+      for (int q = 0; q < ROWS; ++q) row(r[q], true);
+    } else {
+#pragma unroll
+      for (int q = 0; q < ROWS; ++q) row(r[q], from + q < n);
+    }
+  };
+  for (int from = 0; from < n; from += 2 * ROWS) {
+    work(raw[0], from);
+    fetch(raw[0], from + 2 * ROWS);
+    work(raw[1], from + ROWS);
+    fetch(raw[1], from + 3 * ROWS);
   }
 }
 
@@ -954,8 +997,11 @@ int launch_scan_sized(const ScanArgs<T>& a, cudaStream_t stream, bool pdl) {
 
 template <typename T>
 int launch_conv(const StateArgs& st, const void* x, const void* w, void* out, int taps, int max_len, cudaStream_t stream, bool pdl) {
-  ConvArgs<T> a{st, (const T*)x, (const T*)w, (T*)out, taps};
-  const dim3 grid((max_len + CONV_CHUNK - 1) / CONV_CHUNK, (st.W / 4 + 255) / 256, st.S), block(256);
+  ConvArgs<T> a{st, (const T*)x, (const T*)w, (T*)out, taps, CONV_MIN_CHUNK};
+  const int across = (st.W / 4 + CONV_THREADS - 1) / CONV_THREADS;
+  // longer chunks while the device stays full
+  while (a.chunk < 64 && (long long)max_len / (2 * a.chunk) * across * st.S >= 6 * 148) a.chunk *= 2;
+  const dim3 grid((max_len + a.chunk - 1) / a.chunk, across, st.S), block(CONV_THREADS);
   if (taps <= 4) return (int)prism_launch(short_conv_kernel<T, 4>, grid, block, 0, stream, pdl, a);
   if (taps <= 8) return (int)prism_launch(short_conv_kernel<T, 8>, grid, block, 0, stream, pdl, a);
   return (int)prism_launch(short_conv_kernel<T, 16>, grid, block, 0, stream, pdl, a);

@@ -13,6 +13,8 @@
 // pass through the causal convolution in front of the next mixer, whose earlier rows are in the sequence's state slot.
 #include "common.cuh"
 
+#include <type_traits>
+
 PRISM_DEFINE_TU_STATUS(stream)
 
 namespace {
@@ -145,14 +147,33 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return warp_sum(lane < nw ? red[lane] : 0.0f);
 }
 
-// A thread holds U groups of four columns in registers from the first load to the last store.
-template <typename T, int U>
+// A thread holds U groups of four columns in registers from the first load to the last store.  DEEP: with earlier results or a
+// convolution.
+template <typename T, int U, bool DEEP>
 __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_update_kernel(const StreamArgs<T> a) {
   __shared__ float red[2][32];
   const size_t t = blockIdx.x;
   const int i0 = threadIdx.x * 4, step = blockDim.x * 4;
   pdl_launch_dependents();
   F4 acc[U], x[U];
+  // A single token's carried rows were written by an earlier step: a few of them are fetched before the previous kernel has finished.
+  constexpr int EARLY = DEEP && U == 1 ? 3 : 0;
+  const F4 zero{{0.0f, 0.0f, 0.0f, 0.0f}};
+  const float* carry_old = nullptr;
+  float* carry_new = nullptr;
+  F4 early[EARLY > 0 ? EARLY : 1];
+  if (DEEP && a.conv.w != nullptr) {
+    const int slot = a.conv.slots[t], end = a.conv.kv_lens[t];
+    if (slot >= a.conv.num_slots) {
+      if (threadIdx.x == 0) prism_report(PRISM_ERR_BOUNDS, 3);
+    } else if (slot >= 0 && end > 0) {
+      float* base = a.conv.state + (size_t)slot * 2 * a.conv.row + a.conv.carry;
+      if (end > 1) carry_old = base + (size_t)((end - 1) & 1) * a.conv.row;
+      carry_new = base + (size_t)(end & 1) * a.conv.row;
+    }
+#pragma unroll
+    for (int j = 0; j < EARLY; ++j) early[j] = carry_old && j < a.conv.taps - 1 && i0 < a.W ? load4(carry_old + (size_t)j * a.W + i0) : zero;
+  }
   pdl_wait();
   const T* emb = nullptr;
   if (a.ids != nullptr) {
@@ -162,6 +183,20 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
   }
   const bool has_a = a.a.slabs != nullptr || a.a.rows != nullptr;
   float bs = 0.0f;
+  auto earlier_results = [&](int i) {                // weighted sum of the results before this one
+    F4 sum = zero;
+    const float* h0 = a.hist + t * a.W + i;
+#pragma unroll 8
+    for (int j = 0; j < a.hist_n; ++j) {
+      const float w = __ldg(a.hist_w + j);
+      const F4 h = load4(h0 + (size_t)j * a.hist_stride);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sum.v[e] = fmaf(w, h.v[e], sum.v[e]);
+    }
+    return sum;
+  };
+  F4 before = zero;
+  if (DEEP && U == 1 && a.hist_w != nullptr && i0 < a.W) before = earlier_results(i0);
 #pragma unroll
   for (int u = 0; u < U; ++u) {
     const int i = i0 + u * step;
@@ -238,20 +273,13 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
     } else if (a.embed_out != nullptr) {
       store4(a.embed_out + t * a.embed_ld + i, F4{{0.0f, 0.0f, 0.0f, 0.0f}});
     }
-    if (a.hist != nullptr) {
-      const float* h0 = a.hist + t * a.W + i;
+    if (DEEP && a.hist != nullptr) {
       store4(a.hist + (size_t)a.hist_n * a.hist_stride + t * a.W + i, acc[u]);
       if (a.hist_w != nullptr) {
         const float own = __ldg(a.hist_w + a.hist_n);
+        const F4 sum = U == 1 ? before : earlier_results(i);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) acc[u].v[e] *= own;
-#pragma unroll 8
-        for (int j = 0; j < a.hist_n; ++j) {
-          const float w = __ldg(a.hist_w + j);
-          const F4 h = load4(h0 + (size_t)j * a.hist_stride);
-#pragma unroll
-          for (int e = 0; e < 4; ++e) acc[u].v[e] = fmaf(w, h.v[e], acc[u].v[e]);
-        }
+        for (int e = 0; e < 4; ++e) acc[u].v[e] = fmaf(own, acc[u].v[e], sum.v[e]);
       }
     }
     store4(a.x + t * a.W + i, acc[u]);
@@ -261,18 +289,6 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
   }
   if (a.norm_out == nullptr) return;
   const float inv = 1.0f / sqrtf(block_sum(ss, red[1]) / (float)a.W_real + a.eps);
-  const float* carry_old = nullptr;
-  float* carry_new = nullptr;
-  if (a.conv.w != nullptr) {
-    const int slot = a.conv.slots[t], end = a.conv.kv_lens[t];
-    if (slot >= a.conv.num_slots) {
-      if (threadIdx.x == 0) prism_report(PRISM_ERR_BOUNDS, 3);
-    } else if (slot >= 0 && end > 0) {
-      float* base = a.conv.state + (size_t)slot * 2 * a.conv.row + a.conv.carry;
-      if (end > 1) carry_old = base + (size_t)((end - 1) & 1) * a.conv.row;
-      carry_new = base + (size_t)(end & 1) * a.conv.row;
-    }
-  }
 #pragma unroll
   for (int u = 0; u < U; ++u) {
     const int i = i0 + u * step;
@@ -285,7 +301,7 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
 #pragma unroll
       for (int e = 0; e < 4; ++e) v.v[e] *= a.w_offset + w.v[e];
     }
-    if (a.conv.w != nullptr) {     // what a row of the compute type would hold meets the taps
+    if (DEEP && a.conv.w != nullptr) {     // what a row of the compute type would hold meets the taps
       const int last = a.conv.taps - 1;
       F4 o = load4(a.conv.w + (size_t)last * a.W + i);
 #pragma unroll
@@ -293,12 +309,16 @@ __global__ void __launch_bounds__(U == 1 ? 1024 : 512, U == 4 ? 2 : 1) stream_up
         if (sizeof(T) == 2) v.v[e] = bf16_round(v.v[e]);
         o.v[e] = fmaf(o.v[e], v.v[e], v.v[e]);
       }
-      for (int j = 0; j < last; ++j) {
-        const F4 c = carry_old ? load4(carry_old + (size_t)j * a.W + i) : F4{{0.0f, 0.0f, 0.0f, 0.0f}}, w = load4(a.conv.w + (size_t)j * a.W + i);
+      auto tap = [&](int j, const F4& c) {
+        const F4 w = load4(a.conv.w + (size_t)j * a.W + i);
 #pragma unroll
         for (int e = 0; e < 4; ++e) o.v[e] = fmaf(w.v[e], c.v[e], o.v[e]);
         if (carry_new && j > 0) store4(carry_new + (size_t)(j - 1) * a.W + i, c);
-      }
+      };
+#pragma unroll
+      for (int j = 0; j < EARLY; ++j)
+        if (j < last) tap(j, early[j]);
+      for (int j = EARLY; j < last; ++j) tap(j, carry_old ? load4(carry_old + (size_t)j * a.W + i) : zero);
       if (carry_new && last > 0) store4(carry_new + (size_t)(last - 1) * a.W + i, v);
       v = o;
     }
@@ -391,12 +411,16 @@ int launch_stream(int T_rows, void* x, int keep, const void* ids, const void* ta
   const int groups = W / 4;
   const int U = groups <= 1024 && (T_rows < 256 || groups < 256) ? 1 : (groups <= 2048 ? 4 : (groups <= 4096 ? 8 : 16));
   const dim3 grid(T_rows), block(((groups + U - 1) / U + 31) / 32 * 32);
-  switch (U) {
-    case 1: return (int)prism_launch(stream_update_kernel<T, 1>, grid, block, 0, stream, pdl, a);
-    case 4: return (int)prism_launch(stream_update_kernel<T, 4>, grid, block, 0, stream, pdl, a);
-    case 8: return (int)prism_launch(stream_update_kernel<T, 8>, grid, block, 0, stream, pdl, a);
-  }
-  return (int)prism_launch(stream_update_kernel<T, 16>, grid, block, 0, stream, pdl, a);
+  auto run = [&](auto deep) -> int {
+    constexpr bool DEEP = decltype(deep)::value;
+    switch (U) {
+      case 1: return (int)prism_launch(stream_update_kernel<T, 1, DEEP>, grid, block, 0, stream, pdl, a);
+      case 4: return (int)prism_launch(stream_update_kernel<T, 4, DEEP>, grid, block, 0, stream, pdl, a);
+      case 8: return (int)prism_launch(stream_update_kernel<T, 8, DEEP>, grid, block, 0, stream, pdl, a);
+    }
+    return (int)prism_launch(stream_update_kernel<T, 16, DEEP>, grid, block, 0, stream, pdl, a);
+  };
+  return hist != nullptr || conv_w != nullptr ? run(std::true_type()) : run(std::false_type());
 }
 
 }  // namespace

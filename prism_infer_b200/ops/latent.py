@@ -23,6 +23,8 @@ MAX_LATENT = 1024       # widest latent row of the attention kernels
 NO_WINDOW = 1 << 30
 FLASH_MAX_HEAD = 128    # widest head of the tcgen05 prefill attention
 EXPAND_MAX_SCRATCH_BYTES = 2 << 30
+# up to here the absorb kernel sums and rotates the queries itself, once per 128 columns of the row; above, a kernel before it
+ABSORB_ROTATES_TOKENS = 16
 
 
 # ------------------------------------------------------------------------------ stacked projections
@@ -416,8 +418,11 @@ def latent_attention_absorbed(
         return out
     if nsplit <= 0:
         nsplit = latent_splits(S, max_q_len * H, lw.window + max_q_len)
+    turned = lw.rot is None
+    if T > ABSORB_ROTATES_TOKENS and (lw.rot is not None or q.rows is None):
+        q, turned = Branch(rows=rotate_queries(q, lw, positions)), True
     qa = torch.empty((T, H, Rc), dtype=torch.bfloat16, device=dev)
-    rot = (*lw.rot.args(positions), lw.rot.start, lw.rot.dims) if lw.rot is not None else (*NO_ROTARY, 0, 0)
+    rot = (*NO_ROTARY, 0, 0) if turned else (*lw.rot.args(positions), lw.rot.start, lw.rot.dims)
     slabs, stride, P, rows, ld = _branch_args(q)
     native.call("prism_latent_absorb", rows, slabs, stride, P, ld, *rot, _p(lw.uk), _p(qa), _p(raw), raw.stride(0) if raw is not None else 0,
                 _p(lw.norm), _p(pages), _p(slots), cache.num_blocks * cache.page, T, H, lw.dq, lw.rank, Rc, float(eps), _s(), _pdl())
