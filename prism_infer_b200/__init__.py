@@ -1,4 +1,4 @@
-"""B200-native inference engine (Qwen3-VL, Poralorn, Dolidra, Bokorax): ``from prism_infer_b200 import LLM, SamplingParams``.
+"""B200-native inference engine (Qwen3-VL, Poralorn, Dolidra, Bokorax, Fosulix): ``from prism_infer_b200 import LLM, SamplingParams``.
 
 ``LLM`` is loaded lazily so importing the package (for its config, ops or analysis
 modules) does not pull in the engine.

@@ -21,7 +21,7 @@ def forget(heads, dim, vdim):
     return {"heads": heads, "dim": dim, "vdim": vdim}
 
 
-def moe(experts, top, ff, *, groups=None, scale=1.0, limit=2.0):
+def moe(experts, top, ff, *, groups=None, scale=1.0, limit=1.75):
     return {"kind": "moe", "expert": {"ff": ff, "limit": limit},
             "router": {"experts": experts, "top": top, "scale": scale, **({"groups": {"count": groups[0], "keep": groups[1]}} if groups else {})}}
 

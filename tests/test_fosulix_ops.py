@@ -501,7 +501,7 @@ def test_a_far_write_is_remembered(backend, decode):
 
 # ------------------------------------------------------------------------------------------- depth average
 @pytest.mark.parametrize("backend", BACKENDS)
-@pytest.mark.parametrize("width,T", [(64, 3), (75, 5), (1200, 2), (4100, 3), (320, 300), (2048, 260)])
+@pytest.mark.parametrize("width,T", [(64, 3), (75, 5), (1200, 2), (4100, 3), (352, 300), (2048, 260)])
 def test_depth_average(backend, width, T):
     """Results are kept in 32-bit and summed with their weights; the norm, the copy and the stream see the sum."""
     device, dtype = backend
@@ -528,7 +528,7 @@ def test_depth_average(backend, width, T):
 
 # ------------------------------------------------------------------------------- routing and bounded experts
 # outputs, chosen, groups, kept, scale
-ROUTES = {"groups": (12, 3, 4, 3, 2.0), "single": (6, 2, 6, 3, 0.7), "one-group": (5, 4, 1, 1, 1.0), "many": (96, 6, 8, 3, 2.5), "wide": (260, 8, 13, 4, 1.5), "all": (4, 4, 2, 2, 1.0)}
+ROUTES = {"groups": (15, 4, 5, 3, 2.2), "single": (6, 2, 6, 3, 0.7), "one-group": (5, 4, 1, 1, 1.0), "many": (96, 6, 8, 3, 2.5), "wide": (260, 8, 13, 4, 1.5), "all": (4, 4, 2, 2, 1.0)}
 
 
 def routing(T, name, device, seed=7):
@@ -573,7 +573,7 @@ def test_two_good_outputs_beat_one_very_good(backend):
 
 @pytest.mark.parametrize("backend", BACKENDS)
 @pytest.mark.parametrize("T", [1, 5, 128, 140, 500])
-@pytest.mark.parametrize("name,W,F", [("groups", 96, 48), ("single", 112, 208), ("one-group", 320, 144)])
+@pytest.mark.parametrize("name,W,F", [("groups", 96, 48), ("single", 112, 208), ("one-group", 336, 144)])
 def test_bounded_experts(backend, T, name, W, F):
     """Gates and inputs on both sides of the bound."""
     device, dtype = backend
